@@ -166,13 +166,18 @@ inline uint64_t layer_flops(const Layer& l, const ModelMeta& meta, const Workloa
     case LayerKind::Embedding: return b * s * l.hidden;
     case LayerKind::RmsNorm: return 5 * b * s * l.hidden;
     case LayerKind::Attention: {
+      if (l.kv_rank > 0) {   // latent attention as the decode step runs it: the projections, then scores and values over the cached rows
+        uint64_t w = l.shared_elems;
+        for (auto& p : l.params) w += p.numel();
+        return 2 * b * s * w + 2 * b * l.num_heads * s * k * (2 * l.kv_rank + l.rot_dim) + 3 * b * l.num_heads * s * k;
+      }
       const uint64_t hidden = meta.hidden, q = l.num_heads * l.head_dim, kv = l.num_kv_heads * l.head_dim;
       const uint64_t qkvo = 2 * b * s * (q + kv + kv + q) * hidden;
       const uint64_t scores = 2 * b * l.num_heads * s * k * l.head_dim;
       const uint64_t softmax = 3 * b * l.num_heads * s * k;
       return qkvo + scores + softmax + scores;
     }
-    case LayerKind::Mlp: return 6 * b * s * l.hidden * l.intermediate;
+    case LayerKind::Mlp: return (l.activation == "silu" ? 6 : 4) * b * s * l.hidden * l.intermediate;   // two or (ungated) one projections up, one down
     case LayerKind::Moe: return 2 * b * s * l.hidden * l.num_experts + 6 * b * s * l.top_k * l.hidden * l.intermediate;
     case LayerKind::Lmhead: return 2 * b * s * l.vocab * l.hidden;
   }
@@ -197,7 +202,7 @@ inline uint64_t attention_dp_ways(const Placement& pl) { return (pl.ep > 1 && pl
 
 inline double layer_stream_bytes(const Layer& l, const ModelMeta& meta, Dtype wd, Dtype kvd, const Placement& pl, const WorkloadCtx& wl) {
   const double div = (double)std::max<uint64_t>(1, compute_divisor(l.kind, pl));
-  double elems = (double)layer_param_elems(l);
+  double elems = (double)(layer_param_elems(l) + l.shared_elems);
   if (l.kind == LayerKind::Embedding) elems = (double)wl.batch * wl.seq_len * l.hidden;  // only the gathered rows
   if (l.kind == LayerKind::Moe && l.num_experts > 0) {
     // experts actually touched by batch*top_k routed tokens (uniform routing): E * (1 - (1 - 1/E)^(b*k))
@@ -207,7 +212,7 @@ inline double layer_stream_bytes(const Layer& l, const ModelMeta& meta, Dtype wd
   }
   double bytes = (double)dtype_bits(wd) / 8.0 * elems / div;
   if (l.kind == LayerKind::Attention)
-    bytes += (double)dtype_bits(kvd) / 8.0 * 2.0 * l.num_kv_heads * l.head_dim * (double)wl.kv_len * wl.batch /
+    bytes += (double)dtype_bits(kvd) / 8.0 * (double)kv_elems_per_token(l) * (double)wl.kv_len * wl.batch /
              (double)(pl.tp * attention_dp_ways(pl));
   (void)meta;
   return bytes;
@@ -235,7 +240,7 @@ inline double compute_time_with_dtype(const Layer& l, const ModelMeta& meta, Dty
     // (bf16 rate) for the KV cache of an attention layer
     double kv_bytes = 0;
     if (l.kind == LayerKind::Attention)
-      kv_bytes = (double)dtype_bits(kvd) / 8.0 * 2.0 * l.num_kv_heads * l.head_dim * (double)wl.kv_len * wl.batch /
+      kv_bytes = (double)dtype_bits(kvd) / 8.0 * (double)kv_elems_per_token(l) * (double)wl.kv_len * wl.batch /
                  (double)(pl.tp * attention_dp_ways(pl));
     const double w_bytes = layer_stream_bytes(l, meta, wd, kvd, pl, wl) - kv_bytes;
     t = std::max(t, (w_bytes / share(wd) + kv_bytes / share(Dtype::Bf16)) / (hb->second * 1e9) * 1e6);
@@ -264,7 +269,7 @@ inline double block_compute_time(size_t block, const Graph& ir, Dtype wd, Dtype 
 // for its unfused graph: crates/skein_cost/src/compute.rs:232-242).
 inline uint32_t kernels_per_layer(const Layer& l) {
   switch (l.kind) {
-    case LayerKind::Attention: return 4;  // qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
+    case LayerKind::Attention: return l.kv_rank > 0 ? (l.q_rank > 0 ? 8 : 7) : 4;  // latent: input projection, append, (q up,) absorb, attention, values, o_proj, norm; qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
     case LayerKind::Mlp: return 3;        // gate/up GEMM (SwiGLU epilogue), down GEMM, reduce+norm
     case LayerKind::Moe: return 3;        // grouped gate/up (gathers its rows), grouped down, combine + norm
     case LayerKind::RmsNorm: return 0;    // fused into the reduce kernels above
@@ -339,13 +344,19 @@ inline uint64_t weight_bytes_on_device(const Plan& plan, const Graph& ir, size_t
     if (layer_on_stage(l, ir.meta.num_layers, pl, pl.stage_of(device), true)) t += layer_weight_bytes(l, plan_weight_dtype(plan, l.block_idx), pl);
   return t;
 }
+inline uint64_t block_kv_elems_per_token(const Graph& ir, size_t block) {
+  if (ir.meta.layered)
+    for (auto& l : ir.layers) if (l.kind == LayerKind::Attention && l.block_idx && *l.block_idx == block) return kv_elems_per_token(l);
+  return 2ull * ir.meta.num_kv_heads * ir.meta.head_dim;
+}
 inline uint64_t kv_bytes_on_device(const Plan& plan, const Graph& ir, const CostConstants& c, size_t device) {
   const Placement pl = Placement::from_plan(plan);
   if (!pl.holds(device)) return 0;
-  const uint64_t per_seq = 2ull * ir.meta.num_kv_heads * ir.meta.head_dim * c.decode_kv_tokens;
   uint64_t t = 0;
-  for (size_t b = 0; b < ir.meta.num_layers; ++b)
+  for (size_t b = 0; b < ir.meta.num_layers; ++b) {
+    const uint64_t per_seq = block_kv_elems_per_token(ir, b) * c.decode_kv_tokens;
     if (block_to_stage(b, ir.meta.num_layers, pl.pp) == pl.stage_of(device)) t += dtype_bytes_for(plan_kv_dtype(plan, b), per_seq) * plan.batching.max_batch;
+  }
   return (plan.kv.kv_sharded && pl.tp > 1) ? t / pl.tp : t;
 }
 inline uint64_t activation_bytes_on_device(const Plan& plan, const Graph& ir, size_t device) {
@@ -362,8 +373,8 @@ inline uint64_t block_weight_bytes(size_t block, const Graph& ir, Dtype wd, cons
   for (auto& l : ir.layers) if (l.block_idx && *l.block_idx == block) t += layer_weight_bytes(l, wd, pl);
   return t;
 }
-inline uint64_t block_kv_bytes(const Graph& ir, Dtype kvd, const Placement& pl, const WorkloadCtx& wl, bool kv_sharded) {
-  const uint64_t bytes = dtype_bytes_for(kvd, 2ull * ir.meta.num_kv_heads * ir.meta.head_dim * wl.kv_len * wl.batch);
+inline uint64_t block_kv_bytes(const Graph& ir, size_t block, Dtype kvd, const Placement& pl, const WorkloadCtx& wl, bool kv_sharded) {
+  const uint64_t bytes = dtype_bytes_for(kvd, block_kv_elems_per_token(ir, block) * wl.kv_len * wl.batch);
   return (kv_sharded && pl.tp > 1) ? bytes / pl.tp : bytes;
 }
 inline uint64_t non_decoder_weight_bytes(const Graph& ir, const Placement& pl) {

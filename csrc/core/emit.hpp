@@ -174,6 +174,7 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
   LoweredDevice d;
   d.device = device;
   if (!pl.holds(device)) return d;
+  if (ir.meta.layered && pl.tp * pl.pp * pl.ep != 1) throw PlanError(ir.meta.architecture + " runs on one device (tp = pp = ep = 1)");
   const uint32_t stage = pl.stage_of(device);
   Segment cur{0, "segment_0", {}, {}, {}};
   auto cut = [&](const std::string& kind, const std::string& tensor, std::vector<size_t> parts) {
@@ -201,6 +202,21 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
     bool moe = false;
     for (auto& l : ir.layers) if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Moe) moe = true;
     const std::string bs = "block_" + std::to_string(b);
+    if (ir.meta.layered) {
+      // post-norm block of latent attention; its feed-forward, if any, is dense or routed
+      bool ffn = false, q_latent = false;
+      for (auto& l : ir.layers)
+        if (l.block_idx && *l.block_idx == b) { ffn |= l.kind == LayerKind::Mlp || l.kind == LayerKind::Moe; q_latent |= l.q_rank > 0; }
+      std::vector<std::string> ops = {"input_conv", "latent_proj", "latent_append"};
+      if (q_latent) ops.push_back("latent_q_up");
+      for (const char* o : {"latent_attention", "latent_o_proj", "post_norm1"}) ops.push_back(o);
+      if (moe) for (const char* o : {"group_router", "glu_gate_up", "glu_down"}) ops.push_back(o);
+      else if (ffn) for (const char* o : {"ff_up", "poly_norm", "ff_down"}) ops.push_back(o);
+      if (ffn) ops.push_back("post_norm2");
+      for (auto& o : ops) cur.ops.push_back(bs + "_" + o);
+      if (moe) d.sequencing.push_back({"moe_route", cur.idx, "", bs + "_group_router", {}});
+      continue;
+    }
     cur.ops.insert(cur.ops.end(), {bs + "_input_layernorm", bs + "_qkv_proj", bs + "_rope_kv_append", bs + "_attention", bs + "_o_proj"});
     if (pl.tp > 1) cut("ring_allreduce", handoff_collective_attn_out(b), pl.tp_group(device));
     cur.ops.push_back(bs + "_post_attention_layernorm");
@@ -216,7 +232,7 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
     if (pl.tp > 1) cut("ring_allreduce", handoff_collective_ffn_out(b), pl.tp_group(device));
   }
   if (stage == pl.pp - 1) {
-    cur.ops.insert(cur.ops.end(), {"norm", "lm_head", "sample"});
+    cur.ops.insert(cur.ops.end(), {ir.meta.layered ? "final_scalar_norm" : "norm", "lm_head", "sample"});
     if (pl.tp > 1) cut("allgather", "logit_candidates", pl.tp_group(device));
     cur.outputs.push_back(handoff_logits());
   } else {

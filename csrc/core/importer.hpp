@@ -20,7 +20,119 @@ inline size_t cfg_usize(const Json& j, const char* k) {
   return (size_t)x;
 }
 
+// A design that lists its layers one by one (Zarorax): post-norm blocks of latent attention and a dense or routed
+// feed-forward, each with sizes of its own. The tensor names are those of the checkpoint ("l<i>.mix.dkv", "l<i>.mlp.e0.up").
+// A block with `weights_of` has no parameters; what it streams is counted in shared_elems.
+inline Graph import_layered(const Json& cfg) {
+  ModelMeta m;
+  m.architecture = cfg.at("architecture").as_string();
+  m.layered = true;
+  m.hidden = cfg_usize(cfg, "width");
+  m.vocab = cfg_usize(cfg, "vocab");
+  m.max_position = cfg.has("max_position_embeddings") && !cfg.at("max_position_embeddings").is_null() ? cfg_usize(cfg, "max_position_embeddings") : 131072;
+  for (const char* k : {"norm", "canon", "postln_alpha", "layers"})
+    if (!cfg.has(k)) throw ImportError(std::string("config.json: missing `") + k + "`");
+  m.rms_norm_eps = cfg.at("norm").at("eps").as_double();
+  const size_t taps = cfg_usize(cfg.at("canon"), "taps");
+  const auto& layers = cfg.at("layers").items();
+  if (layers.empty()) throw ImportError("config.json: `layers` is empty");
+  m.num_layers = layers.size();
+  m.num_kv_heads = 1;
+  Graph g;
+  size_t idx = 0;
+  const uint64_t C = m.hidden;
+  auto add = [&](LayerKind k, std::optional<size_t> block, const std::string& label) -> Layer& {
+    Layer l;
+    l.idx = idx++; l.block_idx = block; l.kind = k; l.label = label; l.hidden = m.hidden; l.eps = m.rms_norm_eps;
+    g.layers.push_back(l);
+    return g.layers.back();
+  };
+  Layer& em = add(LayerKind::Embedding, std::nullopt, "embed_tokens");
+  em.vocab = m.vocab;
+  em.params.push_back({"embed", {m.vocab, C}, Dtype::Bf16});
+  auto elems = [](const std::vector<Param>& ps) { uint64_t n = 0; for (auto& p : ps) n += p.numel(); return n; };
+  for (size_t b = 0; b < layers.size(); ++b) {
+    const Json& d = layers[b];
+    const std::string type = d.at("type").as_string(), p = "l" + std::to_string(b) + ".";
+    const bool q_latent = type == "latent_attention", gated = type == "latent_attention_2";
+    if (!q_latent && !gated) throw ImportError("layer " + std::to_string(b) + ": mixer type `" + type + "` is not supported");
+    const bool shared = d.has("weights_of") && !d.at("weights_of").is_null();
+    const Json& mx = d.at("mixer");
+    const uint64_t H = cfg_usize(mx, "heads"), D = cfg_usize(mx, "dim"), R = cfg_usize(mx, "rot_dim"), V = cfg_usize(mx, "vdim"), K = cfg_usize(mx, "kv_rank");
+    std::vector<Param> ps;
+    if (q_latent) {
+      const uint64_t Q = cfg_usize(mx, "q_rank");
+      ps.push_back({p + "mix.dq", {Q, C}, Dtype::Bf16});
+      ps.push_back({p + "mix.dq.norm", {Q}, Dtype::Bf16});
+      ps.push_back({p + "mix.uq", {H * (D + R), Q}, Dtype::Bf16});
+    } else {
+      ps.push_back({p + "mix.q", {H * (D + R), C}, Dtype::Bf16});
+    }
+    ps.push_back({p + "mix.dkv", {K + R, C}, Dtype::Bf16});
+    ps.push_back({p + "mix.dkv.norm", {K}, Dtype::Bf16});
+    ps.push_back({p + "mix.uk", {H * D, K}, Dtype::Bf16});
+    ps.push_back({p + "mix.uv", {H * V, K}, Dtype::Bf16});
+    if (gated) ps.push_back({p + "mix.g", {H * V, C}, Dtype::Bf16});
+    ps.push_back({p + "mix.o", {C, H * V}, Dtype::Bf16});
+    ps.push_back({p + "canon1", {C, taps}, Dtype::Bf16});
+    {
+      Layer& a = add(LayerKind::Attention, b, type);
+      a.num_heads = H; a.num_kv_heads = 1; a.head_dim = D + R; a.kv_rank = K; a.rot_dim = R; a.v_dim = V; a.gated = gated;
+      a.q_rank = q_latent ? cfg_usize(mx, "q_rank") : 0;
+      a.conv_taps = taps;
+      a.rope_theta = mx.at("rot").at("base").as_double();
+      if (shared) a.shared_elems = elems(ps); else a.params = ps;
+      m.rope_theta = a.rope_theta;
+    }
+    m.num_attention_heads = std::max<size_t>(m.num_attention_heads, H);
+    m.head_dim = std::max<size_t>(m.head_dim, D + R);
+    Layer& n1 = add(LayerKind::RmsNorm, b, "norm1");
+    if (!shared) n1.params.push_back({p + "norm1", {}, Dtype::Bf16});
+    if (!d.has("mlp") || d.at("mlp").is_null()) continue;
+    const Json& ml = d.at("mlp");
+    const std::string kind = ml.at("kind").as_string();
+    ps.clear();
+    if (kind == "dense") {
+      const uint64_t F = cfg_usize(ml, "ff");
+      ps.push_back({p + "mlp.up", {F, C}, Dtype::Bf16});
+      ps.push_back({p + "mlp.down", {C, F}, Dtype::Bf16});
+      ps.push_back({p + "mlp.act", {4}, Dtype::Bf16});
+      Layer& f = add(LayerKind::Mlp, b, "mlp");
+      f.intermediate = F;
+      f.activation = "poly_norm";
+      if (shared) f.shared_elems = elems(ps); else f.params = ps;
+      m.intermediate = std::max<size_t>(m.intermediate, F);
+    } else if (kind == "moe") {
+      const uint64_t F = cfg_usize(ml.at("expert"), "ff"), E = cfg_usize(ml.at("router"), "experts");
+      for (uint64_t e = 0; e < E; ++e) {
+        const std::string q = p + "mlp.e" + std::to_string(e) + ".";
+        ps.push_back({q + "gate", {F, C}, Dtype::Bf16});
+        ps.push_back({q + "up", {F, C}, Dtype::Bf16});
+        ps.push_back({q + "down", {C, F}, Dtype::Bf16});
+      }
+      ps.push_back({p + "mlp.router", {E, C}, Dtype::Bf16});
+      Layer& f = add(LayerKind::Moe, b, "moe");
+      f.intermediate = F; f.num_experts = E; f.top_k = cfg_usize(ml.at("router"), "top");
+      f.activation = "clamped_glu";
+      if (shared) f.shared_elems = elems(ps); else f.params = ps;
+      m.intermediate = std::max<size_t>(m.intermediate, F * E);
+    } else {
+      throw ImportError("layer " + std::to_string(b) + ": feed-forward kind `" + kind + "` is not supported");
+    }
+    Layer& n2 = add(LayerKind::RmsNorm, b, "norm2");
+    if (!shared) n2.params.push_back({p + "norm2", {}, Dtype::Bf16});
+  }
+  Layer& n = add(LayerKind::RmsNorm, std::nullopt, "norm");
+  n.params.push_back({"final.norm", {}, Dtype::Bf16});
+  Layer& l = add(LayerKind::Lmhead, std::nullopt, "lm_head");
+  l.vocab = m.vocab;
+  l.params.push_back({"head", {m.vocab, C}, Dtype::Bf16});
+  g.meta = m;
+  return g;
+}
+
 inline Graph import_model(const Json& cfg) {
+  if (const Json* a = cfg.find("architecture"); a && !a->is_null() && a->as_string() == "Zarorax") return import_layered(cfg);
   const Json* archs = cfg.find("architectures");
   if (!archs || !archs->is_array() || archs->size() == 0) throw ImportError("config.json: `architectures` is missing or empty");
   const std::string arch = archs->items()[0].as_string();

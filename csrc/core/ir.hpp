@@ -72,6 +72,12 @@ struct Layer {
   size_t num_experts = 0, top_k = 0;
   double eps = 0, rope_theta = 0;
   bool tied = false;
+  // latent attention: one cached row of kv_rank + rot_dim elements per token (0: keys and values per kv head)
+  size_t kv_rank = 0, rot_dim = 0, v_dim = 0, q_rank = 0;
+  bool gated = false;
+  size_t conv_taps = 0;       // the layer's input passes a short causal convolution whose last inputs are cached
+  uint64_t shared_elems = 0;  // parameter elements read from another layer's tensors (weights_of), which own no bytes here
+  std::string activation = "silu";
   std::string label;  // e.g. "input_layernorm", "self_attn"
   std::vector<Param> params;
 };
@@ -84,6 +90,7 @@ struct ModelMeta {
   double rope_theta = 1e4, rms_norm_eps = 1e-5;
   bool tied_embeddings = false;
   bool qkv_bias = false;       // the q / k / v projections carry a bias vector each (Qwen2)
+  bool layered = false;        // the configuration lists its layers one by one; runs on one device
 
   Json to_json() const {
     Json j = Json::object();
@@ -95,6 +102,7 @@ struct ModelMeta {
         .set("rms_norm_eps", rms_norm_eps).set("sliding_window", opt(sliding_window))
         .set("tied_embeddings", tied_embeddings);
     if (qkv_bias) j.set("qkv_bias", true);      // written only when set: plans of models without biases keep their hash
+    if (layered) j.set("layered", true);
     return j;
   }
   static ModelMeta from_json(const Json& j) {
@@ -112,10 +120,16 @@ struct ModelMeta {
     m.rope_theta = j.at("rope_theta").as_double(); m.rms_norm_eps = j.at("rms_norm_eps").as_double();
     m.sliding_window = opt("sliding_window"); m.tied_embeddings = j.at("tied_embeddings").as_bool();
     if (const Json* qb = j.find("qkv_bias"); qb && !qb->is_null()) m.qkv_bias = qb->as_bool();
+    if (const Json* ly = j.find("layered"); ly && !ly->is_null()) m.layered = ly->as_bool();
     return m;
   }
   bool is_moe() const { return num_experts && *num_experts > 0; }
 };
+
+// Cache elements that one token adds in an attention layer.
+inline uint64_t kv_elems_per_token(const Layer& l) {
+  return l.kv_rank > 0 ? (uint64_t)(l.kv_rank + l.rot_dim) : 2ull * l.num_kv_heads * l.head_dim;
+}
 
 struct Graph {
   ModelMeta meta;
@@ -150,11 +164,14 @@ inline Json Graph::to_json() const {
       case LayerKind::Attention:
         k.set("num_heads", l.num_heads).set("num_kv_heads", l.num_kv_heads).set("head_dim", l.head_dim)
             .set("position", Json::object().set("kind", "rope").set("theta", l.rope_theta)).set("sliding_window", Json());
+        if (l.kv_rank > 0)
+          k.set("latent", Json::object().set("kv_rank", l.kv_rank).set("rot_dim", l.rot_dim).set("v_dim", l.v_dim).set("q_rank", l.q_rank)
+                              .set("gated", l.gated).set("conv_taps", l.conv_taps));
         break;
-      case LayerKind::Mlp: k.set("hidden", l.hidden).set("intermediate", l.intermediate).set("activation", "silu"); break;
+      case LayerKind::Mlp: k.set("hidden", l.hidden).set("intermediate", l.intermediate).set("activation", l.activation); break;
       case LayerKind::Moe:
         k.set("num_experts", l.num_experts).set("top_k", l.top_k).set("hidden", l.hidden)
-            .set("intermediate", l.intermediate).set("activation", "silu");
+            .set("intermediate", l.intermediate).set("activation", l.activation);
         break;
       case LayerKind::Lmhead: k.set("vocab", l.vocab).set("hidden", l.hidden).set("tied", l.tied); break;
     }

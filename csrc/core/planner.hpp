@@ -124,6 +124,7 @@ inline std::vector<uint32_t> capture_batch_sizes(uint32_t max_batch) {
 
 inline std::vector<ParallelismPlacement> enumerate_parallelism(uint32_t num_devices, const Graph& ir) {
   std::vector<ParallelismPlacement> out;
+  if (ir.meta.layered) return {{1, 1, 1}};   // designs that list their layers run on one device
   const uint32_t ep_max = ir.meta.is_moe() ? std::min<uint32_t>((uint32_t)*ir.meta.num_experts, 8) : 1;
   for (uint32_t tp : {1u, 2u, 4u, 8u})
     for (uint32_t pp : {1u, 2u, 4u})
@@ -148,7 +149,9 @@ inline std::vector<GlobalConfig> enumerate_global_configs(const Cluster& cl, con
   std::vector<KVCacheSpec> kvs;
   // The cost model does not distinguish KV layouts, so ties go to the first one listed: paged with
   // 16-token pages and head-sharded KV, the layout the runtime's kernels use.
-  for (uint32_t n : {16u, 32u, 64u, 128u}) { kvs.push_back({true, n, true}); kvs.push_back({true, n, false}); }
+  // A latent cache row is one small row per token: its pages start at 64 tokens.
+  const std::vector<uint32_t> page_sizes = ir.meta.layered ? std::vector<uint32_t>{64u} : std::vector<uint32_t>{16u, 32u, 64u, 128u};
+  for (uint32_t n : page_sizes) { kvs.push_back({true, n, true}); kvs.push_back({true, n, false}); }
   kvs.push_back({false, 0, true});
   kvs.push_back({false, 0, false});
   std::vector<uint32_t> ladder = opt.batch_ladder;
@@ -196,7 +199,7 @@ inline RejectReason reject(const GlobalConfig& g, const Cluster& cl, const Graph
   const WorkloadCtx wl{g.batch.max_batch, 1, c.decode_kv_tokens};
   uint64_t total = 0;
   for (size_t b = 0; b < ir.meta.num_layers; ++b)
-    total += block_weight_bytes(b, ir, Dtype::Int4, pl) / p.pp + block_kv_bytes(ir, Dtype::Fp8E4m3, pl, wl, g.kv.kv_sharded) / p.pp;
+    total += block_weight_bytes(b, ir, Dtype::Int4, pl) / p.pp + block_kv_bytes(ir, b, Dtype::Fp8E4m3, pl, wl, g.kv.kv_sharded) / p.pp;
   total += non_decoder_weight_bytes(ir, pl);
   if (total > min_device_memory(cl)) return RejectReason::GlobalMemory;
   return RejectReason::None;
@@ -240,7 +243,7 @@ inline std::optional<DpResult> layer_dtype_dp(const Graph& ir, const CostModel& 
   for (size_t b = 0; b < NB; ++b)
     for (size_t ci = 0; ci < NC; ++ci) {
       const auto& cb = combos[ci];
-      const uint64_t mem = block_weight_bytes(b, ir, cb.weight, pl) / pl.pp + block_kv_bytes(ir, cb.kv_cache, pl, wl, g.kv.kv_sharded) / pl.pp;
+      const uint64_t mem = block_weight_bytes(b, ir, cb.weight, pl) / pl.pp + block_kv_bytes(ir, b, cb.kv_cache, pl, wl, g.kv.kv_sharded) / pl.pp;
       const double dr = drift.block_contribution(b, cb.weight, cb.activation, cb.kv_cache);
       if (!std::isfinite(dr)) { ok[b * NC + ci] = 0; continue; }
       mem_step[b * NC + ci] = (size_t)((mem + bytes_per_bucket - 1) / bytes_per_bucket);

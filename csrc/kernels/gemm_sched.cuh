@@ -104,7 +104,7 @@ __device__ __forceinline__ void build_sched(Sched& sched, const SkeinGemmParams&
   }
   sched.pre[G] = acc;
   sched.MT = MT;
-  sched.KB = p.K / k_elems_per_block;
+  sched.KB = (p.K + k_elems_per_block - 1) / k_elems_per_block;   // a short last block is zero-filled by TMA
   sched.U = acc;
   sched.TK = (long long)acc * sched.KB;
   if (sched.TK >= (1ll << 31)) {   // no work is handed out; the host sees the status
@@ -130,6 +130,14 @@ __device__ __forceinline__ void build_sched(Sched& sched, const SkeinGemmParams&
 }
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + __expf(-x)); }
+// activation of a gate / up pair
+__device__ __forceinline__ float glu_act(const SkeinGemmParams& p, float g, float u) {
+  if (p.glu == 0) return silu(g) * u;
+  g = fminf(g, p.glu_limit);
+  u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
+  return g * sigmoid_f(p.glu_slope * g) * (u + 1.0f);
+}
 
 // host helpers defined in gemm_ws.cu
 int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes, uint32_t box_rows);

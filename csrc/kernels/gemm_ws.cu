@@ -200,6 +200,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           const Unit un = decode_unit(sched, p.G, u);
           const int w_row = un.g * p.w_rows_per_group + un.m * TILE_F;
           const int x_row = sched.off[un.g] + un.n * n_tile;
+          const int x_col = un.g * p.x_group_cols;
           // W8: the 128 block scales of each weight tile travel with the stage (512 bytes per tile), unless the tile
           // sticks out of the matrix; the converters then read the few scales they need themselves
           const bool scales_by_copy = W8 && (w_row + (DUAL ? p.up_row_off : 0) + TILE_F <= w_rows_total) &&
@@ -229,7 +230,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               tma_load_2d(st, &tmW, full, kb * k_elems, w_row, pol_w);
               if (DUAL) tma_load_2d(st + W_TILE_BYTES, &tmW, full, kb * k_elems, w_row + p.up_row_off, pol_w);
             }
-            tma_load_2d(st + W_STAGE_BYTES, &tmX, full, kb * k_elems, x_row, pol_x);
+            tma_load_2d(st + W_STAGE_BYTES, &tmX, full, x_col + kb * k_elems, x_row, pol_x);
             // e4m3 weights: a stage covers 128 K elements, i.e. two 64-wide bf16 activation tiles
             if (W8) {
               tma_load_2d(st + W_STAGE_BYTES + a.x_tile_bytes / 2, &tmX, full, kb * k_elems + 64, x_row, pol_x);
@@ -457,10 +458,12 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const int acc_cols = (DUAL ? 2 : 1) * n_tile;
       const size_t slot_elems = (size_t)TILE_F * acc_cols;
       // final value of one output element: activation pair, residual, store (locally or into every peer)
-      auto emit = [&](float g, float u, long long row, int f) {
+      auto emit = [&](float g, float u, long long row, int f, int gcol) {   // gcol: the group's first column (per-head products)
         float y = g;
-        if (DUAL) y = silu(g) * u;
-        const size_t idx = (size_t)row * p.ldo + p.out_col0 + f;
+        if (DUAL) y = glu_act(p, g, u);
+        const size_t idx = (size_t)row * p.ldo + p.out_col0 + gcol + f;
+        if (p.gate) y *= sigmoid_f(__bfloat162float(((const __nv_bfloat16*)p.gate)[(size_t)row * p.gate_ld + gcol + f]));
+        if (p.out_f32) { ((float*)p.out)[idx] = y; return; }
         if (p.residual) y += __bfloat162float(((const __nv_bfloat16*)p.residual)[idx]);
         const __nv_bfloat16 yb = __float2bfloat16(y);
         ((__nv_bfloat16*)p.out)[idx] = yb;
@@ -548,7 +551,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
                 if (c0 + j >= valid) break;
-                emit(__uint_as_float(v[j]), DUAL ? __uint_as_float(w[j]) : 0.f, row0 + c0 + j, f);
+                emit(__uint_as_float(v[j]), DUAL ? __uint_as_float(w[j]) : 0.f, row0 + c0 + j, f, un.g * p.out_group_cols);
               }
             }
           }
@@ -598,16 +601,23 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         if (r_hi > TILE_F) r_hi = TILE_F;
         const int n_grp = r_hi > r_lo ? (r_hi - r_lo) / 8 : 0;
         const int n_items = n_grp * valid;
-        const bool wide_ok = (p.ldo % 8 == 0) && (p.out_col0 % 8 == 0);
+        const int gcol = un.g * p.out_group_cols;
+        const bool wide_ok = (p.ldo % 8 == 0) && ((p.out_col0 + gcol) % 8 == 0) && !p.out_f32 && (!p.gate || (p.gate_ld % 8 == 0 && gcol % 8 == 0));
         // one item = 8 consecutive features of one token column
         auto store_item = [&](int rr, int col, const float* g8, const float* u8) {
           const int f0 = un.m * TILE_F + rr;
           const long long row = row0 + col;
           if (wide_ok && f0 + 8 <= p.F) {
-            const size_t idx = (size_t)row * p.ldo + p.out_col0 + f0;
+            const size_t idx = (size_t)row * p.ldo + p.out_col0 + gcol + f0;
             float y[8];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) y[j] = DUAL ? silu(g8[j]) * u8[j] : g8[j];
+            for (int j = 0; j < 8; ++j) y[j] = DUAL ? glu_act(p, g8[j], u8[j]) : g8[j];
+            if (p.gate) {
+              const uint4 gv = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.gate + (size_t)row * p.gate_ld + gcol + f0);
+              const __nv_bfloat162* gb = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+              for (int j = 0; j < 4; ++j) { const float2 t = __bfloat1622float2(gb[j]); y[2 * j] *= sigmoid_f(t.x); y[2 * j + 1] *= sigmoid_f(t.y); }
+            }
             if (p.residual) {
               const uint4 rv = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.residual + idx);
               const __nv_bfloat162* rb = reinterpret_cast<const __nv_bfloat162*>(&rv);
@@ -622,7 +632,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           } else {
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              if (f0 + j < p.F) emit(g8[j], u8[j], row, f0 + j);
+              if (f0 + j < p.F) emit(g8[j], u8[j], row, f0 + j, gcol);
           }
         };
         // IPB items of a thread are reduced together, CB = 8 / IPB contributors per batch: 16 (32 with the up half)
@@ -823,7 +833,10 @@ static int plan(const SkeinGemmParams* p, KernelArgs* ka, int* grid, size_t* sme
   if (!p || p->G < 1 || p->G > SKEIN_MAX_GROUPS) return -1;
   const bool w8 = p->fp8 == 2;   // e4m3 weights with 1 x 128 block scales, bf16 activations
   const int kelem = w8 ? 128 : 64;
-  if (p->K <= 0 || p->K % kelem != 0) return -2;
+  // K need not fill its last 64-element block when the weights are plain bf16 rows: TMA reads zeros past the row's end
+  if (p->K <= 0 || p->K % ((w8 || p->w_packed) ? kelem : 8) != 0) return -2;
+  if (p->x_ld % 8 != 0 || (p->x_ld != 0 && p->x_ld < p->K) || p->x_group_cols % 8 != 0) return -2;
+  if (p->out_f32 && (p->mode == 2 || p->residual)) return -4;
   const bool dual = p->mode == 1;
   if (p->n_tile < 16 || p->n_tile % 16 != 0 || p->n_tile > (dual ? 128 : 256)) return -3;
   if (p->mode < 0 || p->mode > 2) return -4;
@@ -908,7 +921,7 @@ extern "C" int skein_gemm_ws(const SkeinGemmParams* p, void* stream) {
     rc = cached_tmap_2d(&tmW, p->W, (uint64_t)p->G * p->w_rows_per_group, p->K, w8 ? 1 : 2, TILE_F);
   }
   if (rc) return rc;
-  rc = cached_tmap_2d(&tmX, p->X, p->x_rows, p->K, 2, p->n_tile);
+  rc = cached_tmap_2d(&tmX, p->X, p->x_rows, p->x_ld > 0 ? p->x_ld : p->K, 2, p->n_tile);
   if (rc) return rc;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   static bool attr_done[4] = {false, false, false, false};

@@ -44,6 +44,16 @@ typedef struct SkeinGemmParams {
   int32_t wait_budget_ms;   // 0 -> 2000
   int32_t w_packed;         // W is stored tile by tile: [rows/128][K/64 (or /128 fp8)][128][128 bytes]
   int32_t line_cut_only;    // 1: never use the tile-aligned split (see gemm_sched.cuh), for comparison runs
+  // per-head products: the groups are column blocks of the same rows (group_off / group_cnt null)
+  int32_t x_ld;             // elements between rows of X (0: K); a multiple of 8
+  int32_t x_group_cols;     // group g reads X from column g * x_group_cols (multiple of 8)
+  int32_t out_group_cols;   // group g writes from column out_col0 + g * out_group_cols
+  int32_t glu;              // dual: 0 silu(g) * u; 1 clamped unit: g = min(g, limit), u = clamp(u, +-limit),
+                            //       g * sigmoid(glu_slope * g) * (u + 1)
+  float glu_limit, glu_slope;
+  int32_t out_f32;          // 1: out is fp32 (residual and publish not available)
+  int32_t gate_ld;          // elements between rows of gate
+  const void* gate;         // optional bf16: the value is multiplied by sigmoid(gate[row, column without out_col0])
 } SkeinGemmParams;
 
 // Returns 0 or a cudaError_t / negative argument-error code.

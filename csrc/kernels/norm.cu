@@ -20,6 +20,7 @@
 // (crates/skein_runtime/src/cuda/nccl.rs:196-245).
 #include "ptx.cuh"
 #include "launch.cuh"
+#include "route.cuh"
 #include <cuda_bf16.h>
 #include <math.h>
 
@@ -222,80 +223,21 @@ __global__ void __launch_bounds__(512) reduce_residual_rmsnorm_kernel(const Norm
 //      router kernel produces) and writes its own row to xs[row] for each of its k experts
 // The host only launches this when T CTAs of 512 threads fit on the device at once.
 // ---------------------------------------------------------------------------------------------
-constexpr int NR_MAX_E = 64;
-constexpr int NR_MAX_K = 8;
-constexpr int NR_MAX_PAIRS = 2048;
-
-struct RouteParams {
-  const __nv_bfloat16* wg;   // [E, H]
-  int* expert_ids;           // [T, k]
-  float* expert_w;           // [T, k]
-  int* counts;               // [E]
-  int* offsets;              // [E + 1]
-  int* row_of;               // [T * k]   (-1: expert not on this rank)
-  int* src_token;            // [T * k]
-  __nv_bfloat16* xs;         // [T * k, H] rows in expert-sorted order
-  int* barrier;              // [2] arrive / depart, zero between launches
-  int E, topk, e_first, e_count;
-  unsigned long long barrier_budget_ns;
-};
-
 template <int MAX_PASSES>
 __global__ void __launch_bounds__(512) reduce_norm_route_kernel(const NormParams p, const RouteParams r) {
   __shared__ float sh[32];
   __shared__ int wait_failed;
-  __shared__ float part[16][NR_MAX_E];
-  __shared__ float logit[NR_MAX_E];
-  __shared__ int ids_s[NR_MAX_PAIRS];
-  __shared__ int cnt_s[NR_MAX_E], bef_s[NR_MAX_E], off_s[NR_MAX_E + 1];
-  __shared__ int my_row[NR_MAX_K];
-  __shared__ int barrier_ok;
-  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
+  __shared__ RouteShared rs;
+  const int t = blockIdx.x, tid = threadIdx.x;
   const int T = gridDim.x, E = r.E, topk = r.topk;
   uint4 nb[MAX_PASSES];
   pdl_trigger();
   pdl_wait();
   const bool have_row = reduce_norm_row<MAX_PASSES>(p, t, sh, wait_failed, nb);
   // a row that failed still takes part in the barrier below, so that the other CTAs do not wait for it
-  const int per_pass = blockDim.x * 8;
-  for (int e0 = 0; e0 < E; e0 += 8) {
-    float a[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = 0.f;
-    if (have_row) {
-#pragma unroll
-      for (int ps = 0; ps < MAX_PASSES; ++ps) {
-        const int h = ps * per_pass + tid * 8;
-        if (h >= p.H) break;
-        uint4 wr[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-          wr[i] = (e0 + i < E) ? *reinterpret_cast<const uint4*>(r.wg + (size_t)(e0 + i) * p.H + h) : make_uint4(0, 0, 0, 0);
-        const __nv_bfloat162* xb = reinterpret_cast<const __nv_bfloat162*>(&nb[ps]);
-        float xf[8];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(xb[i]); xf[2 * i] = f.x; xf[2 * i + 1] = f.y; }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const __nv_bfloat162* wb = reinterpret_cast<const __nv_bfloat162*>(&wr[i]);
-#pragma unroll
-          for (int j = 0; j < 4; ++j) { const float2 f = __bfloat1622float2(wb[j]); a[i] += xf[2 * j] * f.x + xf[2 * j + 1] * f.y; }
-        }
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      float v = a[i];
-      for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-      if (lane == 0 && e0 + i < E) part[warp][e0 + i] = v;
-    }
-  }
+  route_partial_logits<MAX_PASSES>(nb, have_row, r.wg, E, p.H, rs);
   __syncthreads();
-  if (tid < E) {
-    float v = 0.f;
-    for (int w = 0; w < nwarps; ++w) v += part[w][tid];
-    logit[tid] = __bfloat162float(__float2bfloat16(v));
-  }
+  if (tid < E) rs.logit[tid] = __bfloat162float(__float2bfloat16(route_sum_logit(rs, tid)));
   __syncthreads();
   if (tid == 0) {
     int ids[NR_MAX_K];
@@ -306,7 +248,7 @@ __global__ void __launch_bounds__(512) reduce_norm_route_kernel(const NormParams
       for (int e = 0; e < E; ++e) {
         bool taken = false;
         for (int q = 0; q < j; ++q) taken |= (ids[q] == e);
-        if (!taken && (best < 0 || logit[e] > bv)) { best = e; bv = logit[e]; }
+        if (!taken && (best < 0 || rs.logit[e] > bv)) { best = e; bv = rs.logit[e]; }
       }
       ids[j] = best; vals[j] = bv;
     }
@@ -317,68 +259,11 @@ __global__ void __launch_bounds__(512) reduce_norm_route_kernel(const NormParams
       r.expert_ids[t * topk + j] = ids[j];
       r.expert_w[t * topk + j] = vals[j] / den;
     }
-    // release at device scope: this thread's stores of the expert ids / weights above are visible to whoever acquires
-    // the counter (one instruction instead of a full fence followed by a relaxed add)
-    asm volatile("red.release.gpu.global.add.s32 [%0], 1;" ::"l"(r.barrier) : "memory");
-    // grid-wide arrival, bounded: all T CTAs are resident, so this only runs out if one never started
-    const bool poisoned = p.status != nullptr && *(volatile int*)p.status == ST_TIMEOUT_GRID_BARRIER;
-    const bool ok = !poisoned && wait_counter_ge_gpu(r.barrier, T, r.barrier_budget_ns);
-    if (!ok) report_status(p.status, ST_TIMEOUT_GRID_BARRIER, t);
-    barrier_ok = ok ? 1 : 0;
+    route_publish_and_wait(r, p.status, t, T, rs);
   }
   __syncthreads();
-  if (!barrier_ok) return;   // the counters stay dirty: the host clears them when it handles the status
-  const int n_pairs = T * topk;
-  for (int i = tid; i < n_pairs; i += blockDim.x) ids_s[i] = __ldcg(r.expert_ids + i);
-  __syncthreads();
-  const int my_first = t * topk;
-  for (int e = warp; e < E; e += nwarps) {
-    int c = 0, before = 0;
-    for (int i0 = 0; i0 < n_pairs; i0 += 32) {
-      const int i = i0 + lane;
-      const bool hit = i < n_pairs && ids_s[i] == e;
-      c += __popc(__ballot_sync(0xffffffffu, hit));
-      before += __popc(__ballot_sync(0xffffffffu, hit && i < my_first));
-    }
-    if (lane == 0) {
-      cnt_s[e] = (e >= r.e_first && e < r.e_first + r.e_count) ? c : 0;
-      bef_s[e] = before;
-    }
-  }
-  __syncthreads();
-  if (tid == 0) {
-    int a = 0;
-    for (int e = 0; e < E; ++e) { off_s[e] = a; a += cnt_s[e]; }
-    off_s[E] = a;
-    if (t == 0) {
-      for (int e = 0; e < E; ++e) { r.counts[e] = cnt_s[e]; r.offsets[e] = off_s[e]; }
-      r.offsets[E] = a;
-    }
-    for (int j = 0; j < topk; ++j) {
-      const int e = ids_s[my_first + j];
-      const bool mine = e >= r.e_first && e < r.e_first + r.e_count;
-      const int row = mine ? off_s[e] + bef_s[e] : -1;   // a token's k experts are distinct
-      my_row[j] = row;
-      r.row_of[my_first + j] = row;
-      if (row >= 0) r.src_token[row] = t;
-    }
-  }
-  __syncthreads();
-  if (have_row && r.xs != nullptr) {
-#pragma unroll
-    for (int ps = 0; ps < MAX_PASSES; ++ps) {
-      const int h = ps * per_pass + tid * 8;
-      if (h >= p.H) break;
-      for (int j = 0; j < topk; ++j) {
-        const int row = my_row[j];
-        if (row >= 0) *reinterpret_cast<uint4*>(r.xs + (size_t)row * p.H + h) = nb[ps];
-      }
-    }
-  }
-  if (tid == 0) {
-    const int old = atomicAdd(r.barrier + 1, 1);
-    if (old == T - 1) { r.barrier[0] = 0; r.barrier[1] = 0; }   // every CTA is past the wait: re-arm
-  }
+  if (!rs.barrier_ok) return;   // the counters stay dirty: the host clears them when it handles the status
+  route_scatter<MAX_PASSES>(r, nb, have_row, p.H, t, T, rs);
 }
 
 }  // namespace skein

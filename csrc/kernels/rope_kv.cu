@@ -80,6 +80,17 @@ __global__ void gather_rows_kernel(const __nv_bfloat16* __restrict__ in, const i
   for (int h = threadIdx.x; h < H / 8; h += blockDim.x) dst[h] = src[h];
 }
 
+// the same for rows that are not a multiple of 16 bytes
+__global__ void gather_rows_ragged_kernel(const __nv_bfloat16* __restrict__ in, const int* __restrict__ src_row,
+                                          __nv_bfloat16* __restrict__ out, int H, int n_rows_max, const int* n_rows_dev) {
+  const int r = blockIdx.x;
+  const int n = n_rows_dev ? *n_rows_dev : n_rows_max;
+  if (r >= n) return;
+  const __nv_bfloat16* src = in + (size_t)src_row[r] * H;
+  __nv_bfloat16* dst = out + (size_t)r * H;
+  for (int h = threadIdx.x; h < H; h += blockDim.x) dst[h] = src[h];
+}
+
 }  // namespace skein
 
 extern "C" int skein_rope_kv_append(void* qkv, const int* positions, const int* seq_of_token, const int* block_table,
@@ -106,7 +117,11 @@ extern "C" int skein_embed_gather(const int* ids, const void* table, void* out, 
 extern "C" int skein_gather_rows(const void* in, const int* src_row, void* out, int n_rows_max, int H,
                                  const int* n_rows_dev, void* stream) {
   if (n_rows_max == 0) return 0;
-  if (H % 8 != 0) return -1;
+  if (H % 8 != 0) {
+    skein::gather_rows_ragged_kernel<<<n_rows_max, 256, 0, (cudaStream_t)stream>>>(
+        (const __nv_bfloat16*)in, src_row, (__nv_bfloat16*)out, H, n_rows_max, n_rows_dev);
+    return (int)cudaGetLastError();
+  }
   skein::gather_rows_kernel<<<n_rows_max, 256, 0, (cudaStream_t)stream>>>(
       (const __nv_bfloat16*)in, src_row, (__nv_bfloat16*)out, H, n_rows_max, n_rows_dev);
   return (int)cudaGetLastError();

@@ -15,6 +15,8 @@
 // segment_runner.rs:249,1417: D2H of the router logits, host top-k softmax, pointer rebinding) and
 // the graph-level iterative-argmax top_k_route (crates/skein_emit/src/op_wiring.rs:1667-1712).
 #include "ptx.cuh"
+#include "launch.cuh"
+#include "route.cuh"
 #include <cuda_bf16.h>
 #include <math.h>
 
@@ -181,7 +183,86 @@ __global__ void __launch_bounds__(1024) router_plan_kernel(const int* __restrict
   router_plan_body(expert_ids, n_pairs, E, topk, counts, offsets, row_of, src_token, e_first, e_count, cnt_s, off_s, nullptr);
 }
 
+// ---- group-limited selection over given logits, and a layout kernel pair for prefill-sized batches -----------------
+// One warp per token; logits fp32 [T, E].
+constexpr int RG_MAX_E = 256;
+__global__ void __launch_bounds__(128) route_select_kernel(const float* __restrict__ logits, int T, int E, int topk, int n_groups, int keep,
+                                                           int* __restrict__ expert_ids, float* __restrict__ expert_w) {
+  __shared__ float z[4][RG_MAX_E];
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 4 + warp;
+  if (t >= T) return;
+  for (int e = lane; e < E; e += 32) z[warp][e] = logits[(size_t)t * E + e];
+  __syncwarp();
+  select_grouped_warp<RG_MAX_E>(z[warp], E, topk, n_groups, keep, expert_ids + (size_t)t * topk, expert_w + (size_t)t * topk);
+}
+
+// Stable expert-sorted layout with one CTA per expert: the first kernel counts, the second derives its expert's offset from
+// all counts and hands out positions chunk by chunk (256 pairs per chunk, warp ballots inside).
+__global__ void __launch_bounds__(256) plan_count_kernel(const int* __restrict__ expert_ids, int n_pairs, int* __restrict__ counts) {
+  __shared__ int sh[8];
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.x;
+  int c = 0;
+  for (int i = threadIdx.x; i < n_pairs; i += 256) c += expert_ids[i] == e;
+  for (int o = 16; o > 0; o >>= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
+  if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = c;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int a = 0;
+    for (int w = 0; w < 8; ++w) a += sh[w];
+    counts[e] = a;
+  }
+}
+__global__ void __launch_bounds__(256) plan_place_kernel(const int* __restrict__ expert_ids, int n_pairs, int E, int topk,
+                                                         const int* __restrict__ counts, int* __restrict__ offsets,
+                                                         int* __restrict__ row_of, int* __restrict__ src_token) {
+  __shared__ int wsum[8];
+  pdl_trigger();
+  pdl_wait();
+  const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int base = 0;
+  for (int i = 0; i < e; ++i) base += counts[i];
+  if (threadIdx.x == 0) {
+    offsets[e] = base;
+    if (e == E - 1) offsets[E] = base + counts[e];
+  }
+  for (int i0 = 0; i0 < n_pairs; i0 += 256) {
+    const int i = i0 + threadIdx.x;
+    const bool hit = i < n_pairs && expert_ids[i] == e;
+    const unsigned bal = __ballot_sync(0xffffffffu, hit);
+    if (lane == 0) wsum[warp] = __popc(bal);
+    __syncthreads();
+    int before = 0, total = 0;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { if (w < warp) before += wsum[w]; total += wsum[w]; }
+    if (hit) {
+      const int r = base + before + __popc(bal & ((1u << lane) - 1));
+      row_of[i] = r;
+      src_token[r] = i / topk;
+    }
+    base += total;
+    __syncthreads();
+  }
+}
+
 }  // namespace skein
+
+// Softmax over all E logits, group-limited top-k, weights not renormalised (route.cuh: select_grouped_warp), then the
+// expert-sorted layout.
+extern "C" int skein_route_grouped(const float* logits, int T, int E, int topk, int n_groups, int keep, int* expert_ids, float* expert_w,
+                                   int* counts, int* offsets, int* row_of, int* src_token, void* stream) {
+  using namespace skein;
+  if (T == 0) return 0;
+  if (E > RG_MAX_E || n_groups < 1 || n_groups > 64 || E % n_groups != 0 || keep < 1 || keep > n_groups || topk < 1 || topk > keep * (E / n_groups)) return -1;
+  cudaStream_t s = (cudaStream_t)stream;
+  cudaError_t rc = launch_pdl(route_select_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, T, E, topk, n_groups, keep, expert_ids, expert_w);
+  if (rc == cudaSuccess) rc = launch_pdl(plan_count_kernel, dim3(E), dim3(256), 0, s, (const int*)expert_ids, T * topk, counts);
+  if (rc == cudaSuccess) rc = launch_pdl(plan_place_kernel, dim3(E), dim3(256), 0, s, (const int*)expert_ids, T * topk, E, topk, (const int*)counts, offsets, row_of, src_token);
+  return (int)rc;
+}
 
 // With done_counter (a zeroed device int) the same launch also produces the expert-sorted layout
 // (counts[E], offsets[E+1], row_of[T*topk], src_token[T*topk]); without it only ids and weights.

@@ -6,10 +6,14 @@ JIT cache in the home directory.
 
     python -m skein_b200._build            # build whatever is out of date
     python -m skein_b200._build --force    # rebuild everything
+
+`ensure_built(architecture)` compiles, in a fresh checkout, only the kernels that architecture's models run.
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import contextlib
+import fcntl
 import os
 import shutil
 import subprocess
@@ -24,6 +28,11 @@ OBJ = ROOT / "build" / "obj"
 
 KERNEL_LIB = NATIVE / "libskein_kernels.so"
 CORE_LIB_STEM = "_skein_core"
+
+# Kernel sources of architectures that need only some of them (the others take the whole library).
+ARCH_SOURCES = {
+    "Zarorax": ("attn_latent_decode", "attn_latent_prefill", "gemm_simt", "gemm_ws", "latent", "postnorm", "rope_kv", "router", "sample"),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -57,13 +66,29 @@ def core_lib_path() -> Path:
     return NATIVE / (CORE_LIB_STEM + sysconfig.get_config_var("EXT_SUFFIX"))
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every csrc/kernels/*.cu for sm_100a and link libskein_kernels.so."""
+@contextlib.contextmanager
+def _locked():
+    """One build at a time in a checkout."""
     NATIVE.mkdir(parents=True, exist_ok=True)
     OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
+
+
+def _link(cmd, out: Path) -> None:
+    """Link beside the target and rename over it: a process that has the old library mapped keeps it."""
+    tmp = out.with_name(f".{out.name}.{os.getpid()}")
+    _run([*cmd[:2], "-o", str(tmp), *cmd[2:]])
+    os.replace(tmp, out)
+
+
+def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path:
+    """Compile csrc/kernels/*.cu for sm_100a (all, or the stems in `only` besides those compiled before) and link
+    libskein_kernels.so from what has been compiled."""
     kdir = CSRC / "kernels"
     headers = sorted(kdir.glob("*.cuh")) + sorted(kdir.glob("*.h"))
-    srcs = sorted(kdir.glob("*.cu"))
+    srcs = [s for s in sorted(kdir.glob("*.cu")) if only is None or s.stem in only or (OBJ / (s.stem + ".o")).exists()]
     nvcc = _nvcc()
     jobs = []
     objs = []
@@ -77,12 +102,12 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
                 cmd.insert(2, "-v")
             jobs.append(cmd)
     if jobs:
-        with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+        with cf.ThreadPoolExecutor(max_workers=min(16, len(jobs))) as ex:
             for out in ex.map(_run, jobs):
                 if verbose and out.strip():
                     print(out)
     if force or jobs or not KERNEL_LIB.exists():
-        _run([nvcc, "-shared", "-o", str(KERNEL_LIB), *map(str, objs), "-lcudart"])
+        _link([nvcc, "-shared", *map(str, objs), "-lcudart"], KERNEL_LIB)
     return KERNEL_LIB
 
 
@@ -90,8 +115,6 @@ def build_core(force: bool = False) -> Path:
     """Compile the C++ host core (planner, cost model, KV manager, batcher, ...) as a pybind11 module."""
     import pybind11
 
-    NATIVE.mkdir(parents=True, exist_ok=True)
-    OBJ.mkdir(parents=True, exist_ok=True)
     srcs = sorted((CSRC / "core").glob("*.cpp")) + sorted((CSRC / "runtime").glob("*.cpp"))
     headers = sorted((CSRC / "core").glob("*.hpp")) + sorted((CSRC / "runtime").glob("*.hpp"))
     if not srcs:
@@ -109,13 +132,24 @@ def build_core(force: bool = False) -> Path:
             list(ex.map(_run, jobs))
     out = core_lib_path()
     if force or jobs or not out.exists():
-        _run(["g++", "-shared", "-o", str(out), *map(str, objs), "-pthread"])
+        _link(["g++", "-shared", *map(str, objs), "-pthread"], out)
     return out
 
 
+def ensure_built(architecture: str, kernels: bool = True) -> None:
+    """What a model of this architecture needs, compiled if it is missing or out of date."""
+    with _locked(), cf.ThreadPoolExecutor(max_workers=2) as ex:
+        jobs = [ex.submit(build_core)]
+        if kernels:
+            jobs.append(ex.submit(build_kernels, only=ARCH_SOURCES.get(architecture)))
+        for j in jobs:
+            j.result()
+
+
 def build_all(force: bool = False, verbose: bool = False) -> None:
-    build_kernels(force=force, verbose=verbose)
-    build_core(force=force)
+    with _locked():
+        build_kernels(force=force, verbose=verbose)
+        build_core(force=force)
 
 
 if __name__ == "__main__":

@@ -30,7 +30,8 @@ import torch
 
 from .. import core
 from ..models.config import ModelConfig, ParallelLayout
-from ..models.decoder import LayerWeights, ModelWeights
+from ..models.layered import random_param
+from ..models.decoder import LayerWeights, ModelWeights, layered_weights
 from ..ops import reference as ref
 
 FP8_DTYPES = ("fp8_e4m3",)
@@ -45,8 +46,8 @@ class WeightSource:
     """Parameters by HuggingFace name. Backed by a safetensors file / sharded checkpoint directory, or by a
     seeded random generator (benchmarks and tests: N(0, std), norm gains 1)."""
 
-    def __init__(self, cfg: ModelConfig, path: str | None = None, seed: int = 0, std: float = 0.02):
-        self.cfg, self.path, self.seed, self.std = cfg, path, seed, std
+    def __init__(self, cfg: ModelConfig, path: str | None = None, seed: int = 0, std: float = 0.02, dtype=torch.bfloat16):
+        self.cfg, self.path, self.seed, self.std, self.dtype = cfg, path, seed, std, dtype
         self._files = {}
         self._index = None
         if path is not None:
@@ -64,7 +65,7 @@ class WeightSource:
 
     def get(self, name: str, shape) -> torch.Tensor:
         if self.path is None:
-            return _random_param(name, shape, self.seed, self.std)
+            return _random_param(name, shape, self.seed, self.std).to(self.dtype)
         from safetensors import safe_open
 
         if self._index is not None and name not in self._index:
@@ -77,7 +78,16 @@ class WeightSource:
         t = self._files[f].get_tensor(name)
         if list(t.shape) != list(shape):
             raise ArtifactError(f"`{name}` has shape {list(t.shape)}, the model expects {list(shape)}")
-        return t.to(torch.bfloat16)
+        return t.to(self.dtype)
+
+
+def load_checkpoint(cfg: ModelConfig, path, device, dtype=torch.bfloat16) -> ModelWeights:
+    """A checkpoint (safetensors file or directory) as one device's weights, without an artifact in between. dtype float32 runs
+    the model in 32-bit (designs that list their layers)."""
+    if dtype != torch.bfloat16 and not cfg.is_layered:
+        raise ArtifactError(f"{cfg.architecture} runs in bfloat16 only")
+    src = WeightSource(cfg, str(path), dtype=dtype)
+    return assemble_weights(cfg, lambda name: src.get(name, _full_shape(cfg, name)).to(device), ParallelLayout())
 
 
 def _stable_name_seed(name: str) -> int:
@@ -86,8 +96,10 @@ def _stable_name_seed(name: str) -> int:
 
 
 def _random_param(name, shape, seed, std):
-    if name.endswith("layernorm.weight") or name == "model.norm.weight":
-        return torch.ones(*shape, dtype=torch.bfloat16)
+    if name.endswith(("layernorm.weight", ".norm", ".norm1", ".norm2")) or name == "model.norm.weight":
+        return torch.ones(tuple(shape), dtype=torch.bfloat16)
+    if name.endswith((".act", ".canon1")):
+        return random_param(name, tuple(shape), torch.Generator().manual_seed(_stable_name_seed(name) ^ (seed * 1000003)), std, torch.bfloat16, "cpu")
     g = torch.Generator().manual_seed(_stable_name_seed(name) ^ (seed * 1000003))
     return (torch.randn(*shape, generator=g) * std).to(torch.bfloat16)
 
@@ -155,6 +167,11 @@ def build_artifact(plan_json: str, config_json: str, out_root: str | Path, sourc
 
 
 def _full_shape(cfg: ModelConfig, name: str):
+    if cfg.is_layered:
+        shapes = cfg.param_shapes()
+        if name not in shapes:
+            raise ArtifactError(f"unknown parameter `{name}`")
+        return shapes[name]
     H, I, D = cfg.hidden_size, cfg.intermediate_size, cfg.head_dim
     if name in ("model.embed_tokens.weight", "lm_head.weight"):
         return (cfg.vocab_size, H)
@@ -244,7 +261,7 @@ class Artifact:
                     t = ref.dequant_fp8_block128(t.view(torch.float8_e4m3fn), sf.get_tensor(name + ".scale")).to(torch.bfloat16)
                 return t.to(device)
 
-            return self._assemble(get, self.layout(device_idx))
+            return assemble_weights(self.cfg, get, self.layout(device_idx))
 
     def load_full_weights(self, device) -> ModelWeights:
         """Reassemble the unsharded model from every device's shard (inverse of the sharder): used by the
@@ -275,37 +292,40 @@ class Artifact:
                 raise ArtifactError(f"no device holds `{name}`")
             return full[name].to(device)
 
-        return self._assemble(get, ParallelLayout())
+        return assemble_weights(self.cfg, get, ParallelLayout())
 
-    def _assemble(self, get, lay: ParallelLayout) -> ModelWeights:
-        cfg = self.cfg
-        layers = []
-        e_local = cfg.num_experts // lay.ep if cfg.is_moe else 0
-        e0 = lay.ep_rank * e_local
-        for b in lay.stage_layers(cfg.num_layers):
-            pre = f"model.layers.{b}."
-            wqkv = torch.cat([get(pre + f"self_attn.{p}_proj.weight") for p in "qkv"], dim=0).contiguous()
-            if cfg.is_moe:
-                w13 = torch.stack([torch.cat([get(pre + f"block_sparse_moe.experts.{e}.w1.weight"),
-                                              get(pre + f"block_sparse_moe.experts.{e}.w3.weight")], dim=0)
-                                   for e in range(e0, e0 + e_local)]).contiguous()
-                w2 = torch.stack([get(pre + f"block_sparse_moe.experts.{e}.w2.weight") for e in range(e0, e0 + e_local)]).contiguous()
-                router = get(pre + "block_sparse_moe.gate.weight")
-            else:
-                w13 = torch.cat([get(pre + "mlp.gate_proj.weight"), get(pre + "mlp.up_proj.weight")], dim=0).contiguous()
-                w2 = get(pre + "mlp.down_proj.weight").contiguous()
-                router = None
-            bqkv = (torch.cat([get(pre + f"self_attn.{p}_proj.bias") for p in "qkv"]).contiguous() if cfg.qkv_bias else None)
-            layers.append(LayerWeights(attn_norm=get(pre + "input_layernorm.weight"), wqkv=wqkv,
-                                       wo=get(pre + "self_attn.o_proj.weight").contiguous(),
-                                       ffn_norm=get(pre + "post_attention_layernorm.weight"), router=router, w13=w13, w2=w2,
-                                       bqkv=bqkv))
-        first, last = lay.pp_rank == 0, lay.pp_rank == lay.pp - 1
-        embed = get("model.embed_tokens.weight") if first else None
-        # tied embeddings: the output projection is the embedding table (under tensor parallelism both are split by
-        # vocabulary rows the same way, so a rank's table shard is its shard of the output projection)
-        lm_head = (embed if cfg.tie_word_embeddings else get("lm_head.weight")) if last else None
-        return ModelWeights(embed=embed, layers=layers, final_norm=get("model.norm.weight") if last else None, lm_head=lm_head)
+
+def assemble_weights(cfg: ModelConfig, get, lay: ParallelLayout) -> ModelWeights:
+    """The tensors the decoder uses (fused projections, stacked experts) from named checkpoint parameters."""
+    if cfg.is_layered:
+        return layered_weights(cfg, get)
+    layers = []
+    e_local = cfg.num_experts // lay.ep if cfg.is_moe else 0
+    e0 = lay.ep_rank * e_local
+    for b in lay.stage_layers(cfg.num_layers):
+        pre = f"model.layers.{b}."
+        wqkv = torch.cat([get(pre + f"self_attn.{p}_proj.weight") for p in "qkv"], dim=0).contiguous()
+        if cfg.is_moe:
+            w13 = torch.stack([torch.cat([get(pre + f"block_sparse_moe.experts.{e}.w1.weight"),
+                                          get(pre + f"block_sparse_moe.experts.{e}.w3.weight")], dim=0)
+                               for e in range(e0, e0 + e_local)]).contiguous()
+            w2 = torch.stack([get(pre + f"block_sparse_moe.experts.{e}.w2.weight") for e in range(e0, e0 + e_local)]).contiguous()
+            router = get(pre + "block_sparse_moe.gate.weight")
+        else:
+            w13 = torch.cat([get(pre + "mlp.gate_proj.weight"), get(pre + "mlp.up_proj.weight")], dim=0).contiguous()
+            w2 = get(pre + "mlp.down_proj.weight").contiguous()
+            router = None
+        bqkv = (torch.cat([get(pre + f"self_attn.{p}_proj.bias") for p in "qkv"]).contiguous() if cfg.qkv_bias else None)
+        layers.append(LayerWeights(attn_norm=get(pre + "input_layernorm.weight"), wqkv=wqkv,
+                                   wo=get(pre + "self_attn.o_proj.weight").contiguous(),
+                                   ffn_norm=get(pre + "post_attention_layernorm.weight"), router=router, w13=w13, w2=w2,
+                                   bqkv=bqkv))
+    first, last = lay.pp_rank == 0, lay.pp_rank == lay.pp - 1
+    embed = get("model.embed_tokens.weight") if first else None
+    # tied embeddings: the output projection is the embedding table (under tensor parallelism both are split by
+    # vocabulary rows the same way, so a rank's table shard is its shard of the output projection)
+    lm_head = (embed if cfg.tie_word_embeddings else get("lm_head.weight")) if last else None
+    return ModelWeights(embed=embed, layers=layers, final_norm=get("model.norm.weight") if last else None, lm_head=lm_head)
 
 
 def verify_shape_compatibility(old: Artifact, new: Artifact) -> None:

@@ -1,7 +1,8 @@
 """Model and parallel-layout descriptions used by the decoder graph.
 
 ModelConfig is read from a HuggingFace ``config.json`` (MixtralForCausalLM, LlamaForCausalLM and
-the Llama-shaped Mistral / Qwen2 families). The reference imports Mixtral only
+the Llama-shaped Mistral / Qwen2 families), or from the configuration of a design that lists its layers one by one
+(models/layered.py). The reference imports Mixtral only
 (crates/skein_ir/src/model/mod.rs:33-47, model/mixtral.rs:74-372) and rejects the rest; here the
 dense Llama-style block is a Mixtral block with a plain SwiGLU MLP instead of routed experts.
 """
@@ -10,6 +11,8 @@ from __future__ import annotations
 import json
 from dataclasses import asdict, dataclass
 from pathlib import Path
+
+from .layered import LAYERED_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers
 
 MOE_ARCHS = {"MixtralForCausalLM"}
 DENSE_ARCHS = {"LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM"}
@@ -39,12 +42,41 @@ class ModelConfig:
     qkv_bias: bool = False        # the q / k / v projections carry a bias each (Qwen2)
     eos_token_id: int = -1        # token that ends a generation (-1: none known)
     rope_scaling: dict | None = None   # the checkpoint's RoPE frequency scaling ("linear" or "llama3"), None = plain RoPE
+    # designs that list their layers (models/layered.py): per-layer specifications, () for the uniform families
+    layers: tuple = ()
+    conv_taps: int = 0            # taps of the input convolution
+    post_alpha: float = 1.0       # weight of the residual inside the post-norms
 
     @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
 
+    @property
+    def is_layered(self) -> bool:
+        return bool(self.layers)
+
+    @property
+    def default_page_size(self) -> int:
+        """Tokens per cache page: a latent cache row is small and one per token, so its pages are larger."""
+        return 64 if self.is_layered else 16
+
+    def cache_bytes_per_page(self, page_size: int, tp: int = 1, blocks=None, elem: int = 2) -> int:
+        """Bytes of one page over the listed blocks (default: all) on one rank."""
+        blocks = range(self.num_layers) if blocks is None else blocks
+        if not self.is_layered:
+            return 2 * (self.num_kv_heads // tp) * page_size * self.head_dim * elem * len(blocks)
+        tail = min(self.conv_taps - 1, page_size) * self.hidden_size
+        return sum((self.layers[b].mixer.cache_width * page_size + tail) * elem for b in blocks)
+
+    def param_shapes(self) -> dict:
+        """Checkpoint tensor name -> shape (designs that list their layers)."""
+        return param_shapes(self)
+
     def validate(self) -> None:
+        if self.is_layered:
+            if self.conv_taps < 1:
+                raise ImportError_("canon.taps must be at least 1")
+            return
         if self.num_heads % self.num_kv_heads != 0:
             raise ImportError_("num_attention_heads must be a multiple of num_key_value_heads")
         if self.is_moe and not (1 <= self.top_k <= self.num_experts):
@@ -53,6 +85,14 @@ class ModelConfig:
             raise ImportError_("head_dim must be even (RoPE rotates pairs)")
 
     def param_count(self) -> int:
+        if self.is_layered:
+            total = 0
+            for shape in self.param_shapes().values():
+                n = 1
+                for d in shape:
+                    n *= d
+                total += n
+            return total
         H, I, D = self.hidden_size, self.intermediate_size, self.head_dim
         attn = H * (self.num_heads * D) * 2 + H * (self.num_kv_heads * D) * 2
         if self.qkv_bias:
@@ -67,6 +107,8 @@ class ModelConfig:
 
     @staticmethod
     def from_hf_dict(d: dict, name: str | None = None) -> "ModelConfig":
+        if d.get("architecture") in LAYERED_ARCHS:
+            return ModelConfig._from_layered_dict(d, name)
         archs = d.get("architectures") or []
         if not archs:
             raise ImportError_("config.json has no `architectures`")
@@ -121,8 +163,43 @@ class ModelConfig:
         cfg.validate()
         return cfg
 
+    @staticmethod
+    def _from_layered_dict(d: dict, name: str | None) -> "ModelConfig":
+        try:
+            layers = parse_layers(d["architecture"], d["layers"])
+            cfg = ModelConfig.layered(d["architecture"], layers, width=int(d["width"]), vocab=int(d["vocab"]), taps=int(d["canon"]["taps"]),
+                                      alpha=float(d["postln_alpha"]), eps=float(d["norm"]["eps"]), name=name or d["architecture"].lower())
+        except KeyError as e:
+            raise ImportError_(f"config.json: missing {e.args[0]!r}") from e
+        except SpecError as e:
+            raise ImportError_(str(e)) from e
+        if not layers:
+            raise ImportError_("config.json: `layers` is empty")
+        cfg.max_position_embeddings = int(d.get("max_position_embeddings", cfg.max_position_embeddings))
+        eos = d.get("eos_token_id")
+        cfg.eos_token_id = int(eos) if eos is not None else -1
+        return cfg
+
+    @staticmethod
+    def layered(arch: str, layers, width: int, vocab: int, taps: int, alpha: float, eps: float = 1e-5, max_pos: int = 131072,
+                name: str = "layered") -> "ModelConfig":
+        """Configuration of a design that lists its layers. The single-valued fields describe its largest layer (planning and
+        display only; the layer specifications decide what runs). The design sets no position limit: max_pos is the engine's."""
+        ff = [l.mlp.ff * (l.mlp.experts if isinstance(l.mlp, RoutedFFSpec) else 1) for l in layers if l.mlp is not None]
+        cfg = ModelConfig(architecture=arch, hidden_size=width, intermediate_size=max(ff, default=0), num_layers=len(layers),
+                          num_heads=max(l.mixer.heads for l in layers) if layers else 0, num_kv_heads=1,
+                          head_dim=max(l.mixer.dim + l.mixer.rot_dim for l in layers) if layers else 0, vocab_size=vocab,
+                          rms_norm_eps=eps, rope_theta=layers[0].mixer.rope_base if layers else 1e4, num_experts=0, top_k=0,
+                          max_position_embeddings=max_pos, name=name, layers=tuple(layers), conv_taps=taps, post_alpha=alpha)
+        cfg.validate()
+        return cfg
+
     def to_hf_dict(self) -> dict:
-        """The HuggingFace config.json fields that describe this model (what the planner and the lowering read)."""
+        """The config.json fields that describe this model (what the planner and the lowering read)."""
+        if self.is_layered:
+            return {"architecture": self.architecture, "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps},
+                    "canon": {"taps": self.conv_taps}, "postln_alpha": self.post_alpha, "layers": layers_to_list(self.layers),
+                    "max_position_embeddings": self.max_position_embeddings}
         d = {"architectures": [self.architecture], "hidden_size": self.hidden_size, "intermediate_size": self.intermediate_size,
              "num_hidden_layers": self.num_layers, "num_attention_heads": self.num_heads, "num_key_value_heads": self.num_kv_heads,
              "head_dim": self.head_dim, "vocab_size": self.vocab_size, "rms_norm_eps": self.rms_norm_eps, "rope_theta": self.rope_theta,
@@ -167,6 +244,16 @@ def tiny_llama(layers=2, hidden=256, inter=512, heads=4, kv_heads=2, vocab=512) 
     return ModelConfig(architecture="LlamaForCausalLM", hidden_size=hidden, intermediate_size=inter,
                        num_layers=layers, num_heads=heads, num_kv_heads=kv_heads, head_dim=128, vocab_size=vocab,
                        rope_theta=5e5, num_experts=0, top_k=0, max_position_embeddings=4096, name="tiny-llama")
+
+
+def tiny_zarorax(width=192, vocab=384, taps=4, alpha=2.5, eps=1e-5) -> ModelConfig:
+    """A small model of the Zarorax design for tests: both mixers, both feed-forwards, one shared layer, one without any."""
+    from .layered import LatentMixerSpec, LayerSpec
+    a = LatentMixerSpec("latent_attention_2", heads=3, dim=48, rot_dim=16, vdim=40, kv_rank=80, rope_base=1e4, scale=0.11, gated=True)
+    b = LatentMixerSpec("latent_attention", heads=5, dim=24, rot_dim=32, vdim=32, kv_rank=96, rope_base=5e3, scale=0.13, q_rank=56)
+    moe = RoutedFFSpec(ff=72, limit=1.5, experts=8, top=2, groups=4, keep=2)
+    return ModelConfig.layered("Zarorax", (LayerSpec(a, DenseFFSpec(160)), LayerSpec(b, moe), LayerSpec(b, moe, weights_of=1), LayerSpec(a, None)),
+                               width=width, vocab=vocab, taps=taps, alpha=alpha, eps=eps, max_pos=4096, name="tiny-zarorax")
 
 
 @dataclass

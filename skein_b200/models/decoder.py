@@ -28,6 +28,8 @@ from .. import ops
 from ..ops import fp8
 from ..ops import reference as ref
 from .config import ModelConfig, ParallelLayout
+from .layered import assemble_layers, random_param
+from .layered_ops import LayeredOps
 
 
 @dataclass
@@ -70,6 +72,8 @@ def random_weights(cfg: ModelConfig, lay: ParallelLayout, device, seed: int = 0,
                    dtype=torch.bfloat16, shard_embed: bool = False) -> ModelWeights:
     """Random-init weights N(0, std) of this rank's shard shapes (norm gains are 1, as HF initialises them).
     shard_embed: the embedding table holds only this rank's vocabulary rows (tensor parallelism)."""
+    if cfg.is_layered:
+        return _random_layered(cfg, device, seed, std, dtype)
     sh = shard_shapes(cfg, lay)
     g = torch.Generator(device=device)
     g.manual_seed(seed * 1000003 + lay.rank)
@@ -101,6 +105,19 @@ def random_weights(cfg: ModelConfig, lay: ParallelLayout, device, seed: int = 0,
                         lm_head=lm_head)
 
 
+def _random_layered(cfg, device, seed, std, dtype) -> ModelWeights:
+    shapes = cfg.param_shapes()
+    g = torch.Generator(device=device)
+    g.manual_seed(seed * 1000003)
+    return layered_weights(cfg, lambda name: random_param(name, shapes[name], g, std, dtype, device))
+
+
+def layered_weights(cfg, get) -> ModelWeights:
+    """Weights of a design that lists its layers; get(name) returns the checkpoint tensor of that name."""
+    return ModelWeights(embed=get("embed").contiguous(), layers=assemble_layers(cfg, get), final_norm=get("final.norm").float().reshape(1),
+                        lm_head=get("head").contiguous())
+
+
 def quantize_blocks(weights: ModelWeights, blocks, names=("wqkv", "wo", "w13", "w2"), drop_bf16: bool = True) -> None:
     """Replace the named projections of the listed blocks (indices into weights.layers) by block-scaled e4m3
     copies, as the plan's per-layer dtype map asks. With drop_bf16 the bf16 tensors are released."""
@@ -129,6 +146,11 @@ class BatchInputs:
     max_q_len: int = 0                         # host int (prefill)
     logit_rows: torch.Tensor | None = None     # [S] int64 rows of the hidden state that produce logits (prefill)
     ctx_hint: int = 1024                       # host-side typical context length (chooses split-KV)
+    # where each sequence's context starts when all of them are laid end to end, the total, and the longest cached prefix
+    # (prefill of latent attention; derived from seq_lens and q_len when absent)
+    kv_start: torch.Tensor | None = None       # [S] int32
+    kv_total: int = 0
+    max_cached: int = 0
 
 
 @dataclass
@@ -141,14 +163,14 @@ class SamplingInputs:
     step: torch.Tensor                 # [B] int32: counter of each row's random stream (the token's position)
 
 
-class Decoder:
+class Decoder(LayeredOps):
     """One rank's share of the model: weights, KV cache and the step function.
 
     The decoder takes ownership of `weights`: on a GPU the expert matrices are replaced in place by their tile-packed
     form (`ops.PackedWeight`: `.shape`, `.cpu()`, `.unpack()`, `.copy_()`), so that no second copy stays alive."""
 
     def __init__(self, cfg: ModelConfig, weights: ModelWeights, layout: ParallelLayout | None = None,
-                 num_pages: int = 0, page_size: int = 16, max_pos: int | None = None, comm=None, comm_moe=None,
+                 num_pages: int = 0, page_size: int | None = None, max_pos: int | None = None, comm=None, comm_moe=None,
                  pack_moe: bool | None = None, kv_pools=None):
         # pack_moe: tile-pack the FFN / expert weights. kv_pools: per-layer page pools allocated by the caller
         # (peer-mapped pools of a prefill/decode pair, parallel/disagg.py) instead of pools allocated here
@@ -157,17 +179,24 @@ class Decoder:
         self.comm_moe = comm_moe  # communicator over all tp x ep ranks of the stage (expert parallelism), or None
         if self.layout.ep > 1 and comm_moe is None:
             raise ValueError("expert parallelism needs a communicator over the stage's tp x ep ranks (comm_moe)")
-        self.sh = shard_shapes(cfg, self.layout)
+        page_size = page_size or cfg.default_page_size
+        self.sh = shard_shapes(cfg, self.layout) if not cfg.is_layered else {"V_local": cfg.vocab_size}
         self.page_size = page_size
         dev = (weights.embed if weights.embed is not None else weights.layers[0].attn_norm).device
         self.device = dev
-        if dev.type == "cuda" and cfg.head_dim != 128:
+        if cfg.is_layered:
+            pass                # the latent kernels take every head size
+        elif dev.type == "cuda" and cfg.head_dim != 128:
             # say so when the model is set up, not in the middle of the first request
             raise ValueError(f"the attention kernels are built for head size 128; this model has {cfg.head_dim}")
         self.max_pos = max_pos or cfg.max_position_embeddings
-        self.cos_sin = ref.rope_cos_sin_table(self.max_pos, cfg.head_dim, cfg.rope_theta, dev, cfg.rope_scaling)
+        self.cos_sin = None if cfg.is_layered else ref.rope_cos_sin_table(self.max_pos, cfg.head_dim, cfg.rope_theta, dev, cfg.rope_scaling)
         self.num_pages = num_pages
-        if kv_pools is not None:
+        if cfg.is_layered:
+            if kv_pools is not None:
+                raise ValueError(f"{cfg.architecture} allocates its own cache pools")
+            self._init_layered(num_pages)
+        elif kv_pools is not None:
             want = (num_pages, 2, self.sh["Hkv"], page_size, cfg.head_dim)
             if len(kv_pools) != len(weights.layers) or any(tuple(p.shape) != want for p in kv_pools):
                 raise ValueError(f"kv_pools must be {len(weights.layers)} tensors of shape {want}")
@@ -199,7 +228,8 @@ class Decoder:
             raise RuntimeError(f"the lowering names operators this runtime does not implement: {missing}")
         if pack_moe is None:
             pack_moe = os.environ.get("SKEIN_PACK_MOE", "1") == "1"
-        if pack_moe and dev.type == "cuda":
+        # (layered designs keep plain rows: their shapes need not be whole tiles, and layers may share one object)
+        if pack_moe and dev.type == "cuda" and not cfg.is_layered:
             # expert weights re-laid tile by tile (ops.pack_weight): each 128 x 64 tile the GEMM streams is one
             # contiguous 16 KB block instead of 128 rows that are a whole K apart. Measured in-graph on B200:
             # gate/up 80.4 -> 71.2 us at the TP=4 shard shape, 43.2 -> 40.4 us at TP=8, unchanged at TP=1 (HBM-bound)
@@ -242,14 +272,14 @@ class Decoder:
     class _Run:
         """State of one pass over the program."""
         __slots__ = ("inp", "residual", "normed", "qkv", "attn", "pending", "pending_kind", "routed", "h", "sp", "T",
-                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts")
+                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts", "dense")
 
         def __init__(self, inp, residual):
             self.inp, self.residual = inp, residual
             self.normed = self.qkv = self.attn = self.pending = self.routed = self.h = None
             self.pending_kind, self.crossing, self.sp, self.T = None, None, False, 0
             self.embed_deferred = False
-            self.row_idx = self.row_w = self.owner = self.wts = None
+            self.row_idx = self.row_w = self.owner = self.wts = self.dense = None
             self.dp = 0          # rows per rank under data-parallel attention (0: every rank holds all rows)
 
     def dp_ways(self) -> int:
@@ -292,7 +322,9 @@ class Decoder:
 
     # ---- operators of the program (one method per operator name of the lowering) -----------------------
     def _op_embed_tokens(self, st, _):
-        if self.embed_vocab_start is not None:
+        if self.cfg.is_layered:
+            st.residual = ops.latent.embed_f32(st.inp.token_ids, self.w.embed)
+        elif self.embed_vocab_start is not None:
             st.embed_deferred = True       # the ranks' lookups are summed where the lowering puts the embed_out all-reduce
         else:
             st.residual = ops.embed(st.inp.token_ids, self.w.embed)
@@ -594,6 +626,10 @@ class Decoder:
             normed = normed.index_select(0, inp.logit_rows).contiguous()
         return ops.linear(normed, self.w.lm_head)
 
+    def forward_logits(self, inp: BatchInputs):
+        """A step without sampling: logits of the rows inp.logit_rows (prefill chunks) or of every row."""
+        return self.logits(self.forward_hidden(inp)[1], inp)
+
     def forward(self, inp: BatchInputs, hidden_in=None, sampling: SamplingInputs | None = None):
         """Full step on a single stage: returns (next tokens int32 [rows], logits shard). Greedy unless `sampling`
         is given."""
@@ -627,6 +663,8 @@ class Decoder:
         per-request random stream), as the reference gathers logits before its sampler
         (crates/skein_runtime/src/cuda/nccl.rs:251-298)."""
         tp = self.comm is not None and self.comm.size > 1
+        if lg.is_cuda and lg.dtype != torch.bfloat16:
+            lg = lg.to(torch.bfloat16)       # the samplers read bf16 logits (a model run in fp32 keeps them in fp32 until here)
         if sampling is None:
             return self.comm.vocab_parallel_argmax(lg, self.sh["V_local"]) if tp else ops.sample_argmax(lg)
         if tp:

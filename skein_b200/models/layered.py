@@ -1,0 +1,264 @@
+"""Designs whose configuration lists the layers one by one, each with its own mixer and feed-forward: specification,
+parameter names and shapes, weights.
+
+A layer of such a design is post-norm: x <- norm1(alpha x + mixer(h)), x <- norm2(alpha x + ff(x)), with RMS norms whose
+gain is one number, and h = x + (short causal convolution of x over time). Several layers may use one layer's tensors
+(`weights_of`); each keeps a cache of its own. The registry below names, per architecture, which mixers exist:
+
+  Zarorax   latent_attention     latent attention, queries through a latent of their own
+            latent_attention_2   latent attention, queries straight from the input, output gated by a sigmoid
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+
+import torch
+
+# architecture -> mixer type -> (queries through a latent, output gate)
+LAYERED_ARCHS = {"Zarorax": {"latent_attention": (True, False), "latent_attention_2": (False, True)}}
+
+GLU_SLOPE = 1.702          # g * sigmoid(GLU_SLOPE * g) of the clamped gated unit
+
+
+@dataclass(frozen=True)
+class LatentMixerSpec:
+    kind: str                # mixer type of the configuration
+    heads: int
+    dim: int                 # unrotated query / key dimensions per head
+    rot_dim: int             # rotated query / key dimensions per head (the key part is shared by all heads)
+    vdim: int
+    kv_rank: int
+    rope_base: float
+    scale: float
+    q_rank: int = 0          # 0: queries straight from the input
+    gated: bool = False
+
+    @property
+    def cache_width(self) -> int:
+        """Elements cached per token: the normed latent and the rotated key part."""
+        return self.kv_rank + self.rot_dim
+
+    @property
+    def q_width(self) -> int:
+        return self.heads * (self.dim + self.rot_dim)
+
+
+@dataclass(frozen=True)
+class DenseFFSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
+class RoutedFFSpec:
+    ff: int                  # of one expert
+    limit: float
+    experts: int
+    top: int
+    groups: int = 1          # neighbouring experts form equal groups ...
+    keep: int = 1            # ... of which the best `keep` are eligible
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: LatentMixerSpec
+    mlp: DenseFFSpec | RoutedFFSpec | None
+    weights_of: int | None = None
+
+
+class SpecError(ValueError):
+    pass
+
+
+def parse_layers(arch: str, layers: list) -> tuple:
+    """The configuration's `layers` list -> LayerSpec tuple (`weights_of` chains resolved to the layer that owns tensors)."""
+    kinds = LAYERED_ARCHS[arch]
+    out = []
+    for i, d in enumerate(layers):
+        if d.get("type") not in kinds:
+            raise SpecError(f"layer {i}: mixer type {d.get('type')!r} is not part of {arch}")
+        q_latent, gated = kinds[d["type"]]
+        m = d["mixer"]
+        rot = m["rot"]
+        if int(rot["dims"]) != int(m["rot_dim"]):
+            raise SpecError(f"layer {i}: rot.dims must equal rot_dim")
+        mixer = LatentMixerSpec(kind=d["type"], heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                                kv_rank=int(m["kv_rank"]), rope_base=float(rot["base"]), scale=float(m["scale"]),
+                                q_rank=int(m["q_rank"]) if q_latent else 0, gated=gated)
+        if mixer.rot_dim % 2:
+            raise SpecError(f"layer {i}: rot_dim must be even (rotation turns pairs)")
+        mlp = d.get("mlp")
+        if mlp is None:
+            ff = None
+        elif mlp["kind"] == "dense":
+            ff = DenseFFSpec(int(mlp["ff"]))
+        elif mlp["kind"] == "moe":
+            r = mlp["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            ff = RoutedFFSpec(int(mlp["expert"]["ff"]), float(mlp["expert"]["limit"]), int(r["experts"]), int(r["top"]),
+                              int(g["count"]), int(g["keep"]))
+            if ff.experts % ff.groups or not 1 <= ff.keep <= ff.groups or not 1 <= ff.top <= ff.keep * (ff.experts // ff.groups):
+                raise SpecError(f"layer {i}: {ff.top} of {ff.experts} experts cannot be chosen from {ff.keep} of {ff.groups} groups")
+        else:
+            raise SpecError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
+        src = d.get("weights_of")
+        if src is not None:
+            src = int(src)
+            if not 0 <= src < i:
+                raise SpecError(f"layer {i}: weights_of {src} does not name an earlier layer")
+            owner = out[src]
+            if (owner.mixer, owner.mlp) != (mixer, ff):
+                raise SpecError(f"layer {i} differs from layer {src}, whose tensors it uses")
+            src = owner.weights_of if owner.weights_of is not None else src
+        out.append(LayerSpec(mixer, ff, src))
+    return tuple(out)
+
+
+def layers_to_list(layers) -> list:
+    """Inverse of parse_layers."""
+    out = []
+    for sp in layers:
+        m = sp.mixer
+        mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
+                 "rot": {"base": m.rope_base, "dims": m.rot_dim}}
+        if m.q_rank:
+            mixer["q_rank"] = m.q_rank
+        if sp.mlp is None:
+            mlp = None
+        elif isinstance(sp.mlp, DenseFFSpec):
+            mlp = {"kind": "dense", "ff": sp.mlp.ff}
+        else:
+            r = {"experts": sp.mlp.experts, "top": sp.mlp.top}
+            if (sp.mlp.groups, sp.mlp.keep) != (1, 1):
+                r["groups"] = {"count": sp.mlp.groups, "keep": sp.mlp.keep}
+            mlp = {"kind": "moe", "expert": {"ff": sp.mlp.ff, "limit": sp.mlp.limit}, "router": r}
+        d = {"type": m.kind, "mixer": mixer, "mlp": mlp}
+        if sp.weights_of is not None:
+            d["weights_of"] = sp.weights_of
+        out.append(d)
+    return out
+
+
+def param_shapes(cfg) -> dict:
+    """Checkpoint tensor name -> shape, in file order (layers with `weights_of` own none)."""
+    C = cfg.hidden_size
+    s = {"embed": (cfg.vocab_size, C)}
+    for i, sp in enumerate(cfg.layers):
+        if sp.weights_of is not None:
+            continue
+        p, m = f"l{i}.", sp.mixer
+        s[p + "norm1"] = ()
+        if sp.mlp is not None:
+            s[p + "norm2"] = ()
+        if m.q_rank:
+            s[p + "mix.dq"], s[p + "mix.dq.norm"], s[p + "mix.uq"] = (m.q_rank, C), (m.q_rank,), (m.q_width, m.q_rank)
+        else:
+            s[p + "mix.q"] = (m.q_width, C)
+        s[p + "mix.dkv"], s[p + "mix.dkv.norm"] = (m.cache_width, C), (m.kv_rank,)
+        s[p + "mix.uk"], s[p + "mix.uv"] = (m.heads * m.dim, m.kv_rank), (m.heads * m.vdim, m.kv_rank)
+        if m.gated:
+            s[p + "mix.g"] = (m.heads * m.vdim, C)
+        s[p + "mix.o"] = (C, m.heads * m.vdim)
+        if isinstance(sp.mlp, DenseFFSpec):
+            s[p + "mlp.up"], s[p + "mlp.down"], s[p + "mlp.act"] = (sp.mlp.ff, C), (C, sp.mlp.ff), (4,)
+        elif isinstance(sp.mlp, RoutedFFSpec):
+            for e in range(sp.mlp.experts):
+                q = f"{p}mlp.e{e}."
+                s[q + "gate"], s[q + "up"], s[q + "down"] = (sp.mlp.ff, C), (sp.mlp.ff, C), (C, sp.mlp.ff)
+            s[p + "mlp.router"] = (sp.mlp.experts, C)
+        s[p + "canon1"] = (C, cfg.conv_taps)
+    s["final.norm"] = ()
+    s["head"] = (cfg.vocab_size, C)
+    return s
+
+
+# ---- weights ------------------------------------------------------------------------------------------------------
+def _up8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass
+class LatentMixerWeights:
+    """Tensors of a latent-attention mixer in the layouts the kernels read.
+
+    w_in stacks every projection of the mixer's input (queries or their latent, cache row, gate); each section starts at a
+    multiple of 8 rows (zero rows in between), so that a row of its output can be read with 16-byte accesses."""
+    w_in: torch.Tensor                 # [in_rows, C]
+    q_norm: torch.Tensor | None        # [q_rank] fp32
+    w_uq: torch.Tensor | None          # [H (dim + rot), q_rank]
+    kv_norm: torch.Tensor              # [kv_rank] fp32
+    w_ukv: torch.Tensor                # [H dim + H vdim, kv_rank]: keys then values of every head from the latent
+    w_uk_t: torch.Tensor               # [H, kv_rank, dim]: the key expansion transposed, applied to the queries
+    wo: torch.Tensor                   # [C, H vdim]
+    off_kv: int = 0                    # first column of the cache row / the gate in the input projection's output
+    off_gate: int = -1
+
+
+@dataclass
+class LayeredWeights:
+    mixer: LatentMixerWeights
+    conv: torch.Tensor                 # [taps, C] fp32
+    norm1: torch.Tensor                # [1] fp32
+    norm2: torch.Tensor | None
+    w_up: torch.Tensor | None = None   # dense feed-forward
+    act: torch.Tensor | None = None    # [4] fp32
+    router: torch.Tensor | None = None
+    w13: torch.Tensor | None = None    # experts: [E, 2 ff, C], gate rows first
+    w2: torch.Tensor | None = None     # experts [E, C, ff], or the dense down projection [C, ff]
+    fp8: dict = field(default_factory=dict)
+
+
+def stack_rows(parts):
+    """Row-stacks matrices, each section padded to a multiple of 8 rows. Returns (stacked, first row of each section)."""
+    rows, offs, at = [], [], 0
+    for p in parts:
+        offs.append(at)
+        rows.append(p)
+        pad = _up8(p.shape[0]) - p.shape[0]
+        if pad:
+            rows.append(torch.zeros(pad, p.shape[1], dtype=p.dtype, device=p.device))
+        at += _up8(p.shape[0])
+    return torch.cat(rows, dim=0).contiguous(), offs
+
+
+def assemble_mixer(m: LatentMixerSpec, get, prefix: str) -> LatentMixerWeights:
+    parts = [get(prefix + ("dq" if m.q_rank else "q")), get(prefix + "dkv")] + ([get(prefix + "g")] if m.gated else [])
+    w_in, offs = stack_rows(parts)
+    uk, uv = get(prefix + "uk"), get(prefix + "uv")
+    return LatentMixerWeights(
+        w_in=w_in, q_norm=get(prefix + "dq.norm").float() if m.q_rank else None, w_uq=get(prefix + "uq").contiguous() if m.q_rank else None,
+        kv_norm=get(prefix + "dkv.norm").float(), w_ukv=torch.cat([uk, uv], dim=0).contiguous(),
+        w_uk_t=uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).contiguous(), wo=get(prefix + "o").contiguous(),
+        off_kv=offs[1], off_gate=offs[2] if m.gated else -1)
+
+
+def assemble_layers(cfg, get) -> list:
+    """One LayeredWeights per layer; layers that share tensors share the object."""
+    out = []
+    for i, sp in enumerate(cfg.layers):
+        if sp.weights_of is not None:
+            out.append(out[sp.weights_of])
+            continue
+        p = f"l{i}."
+        lw = LayeredWeights(mixer=assemble_mixer(sp.mixer, get, p + "mix."), conv=get(p + "canon1").float().t().contiguous(),
+                            norm1=get(p + "norm1").float().reshape(1),
+                            norm2=get(p + "norm2").float().reshape(1) if sp.mlp is not None else None)
+        if isinstance(sp.mlp, DenseFFSpec):
+            lw.w_up, lw.w2, lw.act = get(p + "mlp.up").contiguous(), get(p + "mlp.down").contiguous(), get(p + "mlp.act").float()
+        elif isinstance(sp.mlp, RoutedFFSpec):
+            E = range(sp.mlp.experts)
+            lw.router = get(p + "mlp.router").contiguous()
+            lw.w13 = torch.stack([torch.cat([get(f"{p}mlp.e{e}.gate"), get(f"{p}mlp.e{e}.up")], dim=0) for e in E]).contiguous()
+            lw.w2 = torch.stack([get(f"{p}mlp.e{e}.down") for e in E]).contiguous()
+        out.append(lw)
+    return out
+
+
+def random_param(name: str, shape, gen, std: float, dtype, device):
+    """Seeded random parameter: N(0, std), gains 1, the polynomial activation near its linear term, convolution taps small."""
+    if name.endswith("norm") or name.endswith(("norm1", "norm2")):
+        return torch.ones(shape, dtype=dtype, device=device)
+    t = torch.empty(shape, dtype=torch.float32, device=device)
+    t.normal_(0.0, 0.25 if name.endswith((".act", ".canon1")) else std, generator=gen)
+    if name.endswith(".act"):
+        t += 0.5
+    return t.to(dtype)

@@ -2,3 +2,4 @@
 from . import reference
 from .functional import *  # noqa: F401,F403
 from .functional import workspace, Workspace
+from . import latent  # noqa: F401

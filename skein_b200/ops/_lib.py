@@ -34,6 +34,9 @@ class GemmParams(C.Structure):
         ("t_static", C.c_int32), ("n_tile", C.c_int32), ("ldo", C.c_int32), ("out_col0", C.c_int32),
         ("mode", C.c_int32), ("fp8", C.c_int32), ("stages", C.c_int32), ("grid", C.c_int32),
         ("wait_budget_ms", C.c_int32), ("w_packed", C.c_int32), ("line_cut_only", C.c_int32),
+        ("x_ld", C.c_int32), ("x_group_cols", C.c_int32), ("out_group_cols", C.c_int32), ("glu", C.c_int32),
+        ("glu_limit", C.c_float), ("glu_slope", C.c_float), ("out_f32", C.c_int32), ("gate_ld", C.c_int32),
+        ("gate", C.c_void_p),
     ]
 
 
@@ -46,6 +49,10 @@ def available() -> bool:
 
 
 def _sig(lib, name, restype, argtypes):
+    # a library built for one architecture holds that architecture's kernels only (_build.py): calling an absent one raises
+    # AttributeError naming it
+    if not hasattr(lib, name):
+        return None
     fn = getattr(lib, name)
     fn.restype = restype
     fn.argtypes = argtypes
@@ -109,6 +116,24 @@ def lib():
     _sig(L, "skein_argmax_push", i32, [vp, i64, i32, i32, i32, pvp, pvp, pvp, i32, vp, vp, vp])
     _sig(L, "skein_copy_pages", i32, [vp, vp, vp, vp, i32, i64, vp])
     _sig(L, "skein_wait_flag", i32, [vp, i32, i32, vp, vp])
+    _sig(L, "skein_gemm_simt", i32, [C.POINTER(GemmParams), i32, i32, vp])
+    _sig(L, "skein_embed_f32", i32, [vp, vp, vp, i32, i32, i32, i32, vp])
+    _sig(L, "skein_conv_input", i32, [vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp])
+    _sig(L, "skein_post_norm", i32, [vp, vp, vp, vp, vp, vp, vp, vp, f32, f32, i32, i32, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp])
+    _sig(L, "skein_post_norm_route", i32,
+         [vp, vp, vp, vp, f32, f32, i32, i32, vp, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp])
+    _sig(L, "skein_poly_norm", i32, [vp, vp, vp, i32, i32, f32, i32, vp])
+    _sig(L, "skein_route_grouped", i32, [vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp])
+    _sig(L, "skein_latent_append", i32,
+         [vp, i32, i32, vp, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp, i32, vp])
+    _sig(L, "skein_rope_rows", i32, [vp, i64, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp])
+    _sig(L, "skein_latent_gather", i32, [vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp])
+    _sig(L, "skein_latent_attn_rows", i32,
+         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp])
+    _sig(L, "skein_latent_attn_decode", i32,
+         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp])
+    _sig(L, "skein_latent_attn_prefill", i32,
+         [vp, i64, i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp])
     for name, rt, at in _OPTIONAL:
         if hasattr(L, name):
             _sig(L, name, rt, at)

@@ -134,7 +134,7 @@ def _gemm_launch(p: "_lib.GemmParams", what: str, cfg: dict | None = None):
         # The estimate assumes one token tile per group (decode); a wrong guess only changes the split.
         rows = p.t_static if not p.group_cnt else p.n_tile
         units = p.G * ((p.F + 127) // 128) * max(1, (rows + p.n_tile - 1) // p.n_tile)
-        p.grid = tuning.heuristic_grid(units, p.K // (128 if p.fp8 else 64), ws.sm_count, dual=(p.mode == 1))
+        p.grid = tuning.heuristic_grid(units, (p.K + 63) // (128 if p.fp8 else 64), ws.sm_count, dual=(p.mode == 1))
     _lib.check(_lib.lib().skein_gemm_ws(C.byref(p), _lib.stream_ptr()), what)
     _lib.count_launch()
 
@@ -207,38 +207,64 @@ def _wview(w):
 
 
 def _check_act(x):
-    if x.dtype != torch.bfloat16 or not x.is_contiguous():
-        raise ValueError("activations must be contiguous bf16")
+    if x.dtype not in (torch.bfloat16, torch.float32) or not x.is_contiguous():
+        raise ValueError("activations must be contiguous bf16 (or fp32 in a model run in 32-bit)")
 
 
-def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None):
-    """y[t, f] = sum_k x[t, k] w[f, k] (+ residual[t, f])."""
+def tc_gemm_ok(x, K) -> bool:
+    """Whether a product over K elements runs on the tensor-core GEMM: bf16 rows of a multiple of 16 bytes. The others (fp32,
+    odd row lengths) take the FMA kernel (csrc/kernels/gemm_simt.cu)."""
+    return x.dtype == torch.bfloat16 and K % 8 == 0
+
+
+def simt_launch(p: "_lib.GemmParams", x, max_rows: int, what: str):
+    _lib.check(_lib.lib().skein_gemm_simt(C.byref(p), 1 if x.dtype == torch.float32 else 0, int(max_rows), _lib.stream_ptr()), what)
+    _lib.count_launch()
+
+
+def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False):
+    """y[t, f] = sum_k x[t, k] w[f, k] (+ residual[t, f]). out_f32: the accumulator is stored without rounding to bf16.
+    x may be the first K columns of a wider matrix (rows strided)."""
+    K = w.shape[1]
     if not x.is_cuda:
-        y = ref.linear(x, w.unpack() if isinstance(w, PackedWeight) else w, residual)
+        y = ref.linear(x[:, :K], w.unpack() if isinstance(w, PackedWeight) else w, residual)
         if out is not None:
             out.copy_(y)
             return out
         return y
-    _check_act(x)
-    T, K = x.shape
+    if x.stride(1) != 1 or x.shape[1] < K:
+        raise ValueError("linear: rows of x must hold at least K contiguous elements")
+    T = x.shape[0]
     F = w.shape[0]
     if out is None:
-        out = torch.empty(T, F, dtype=torch.bfloat16, device=x.device)
+        out = torch.empty(T, F, dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
     if T == 0:
         return out
     wv, _, packed = _wview(w)
     p = _base_params(x, wv, out, F, K, n_tile or pick_n_tile(T, False), 0)
-    p.w_rows_per_group, p.w_packed = F, packed
+    p.w_rows_per_group, p.w_packed, p.out_f32 = F, packed, 1 if out_f32 else 0
+    if x.stride(0) != K:
+        p.x_ld = x.stride(0)
     if residual is not None:
         p.residual = residual.data_ptr()
-    _gemm_launch(p, "linear", _cfg)
+    if tc_gemm_ok(x, K) and p.x_ld % 8 == 0 and x.data_ptr() % 16 == 0:
+        _check_bf16(x)
+        _gemm_launch(p, "linear", _cfg)
+    else:
+        simt_launch(p, x, T, "linear")
     return out
+
+
+def _check_bf16(x):
+    if x.dtype != torch.bfloat16:
+        raise ValueError("the tensor-core GEMM takes bf16 activations")
 
 
 def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None):
     """silu(x @ w13[:I].T) * (x @ w13[I:].T) with both products from one pass over x."""
     if not x.is_cuda:
         return ref.swiglu_linear(x, w13.unpack() if isinstance(w13, PackedWeight) else w13)
+    _check_bf16(x)
     _check_act(x)
     T, K = x.shape
     inter = w13.shape[0] // 2
@@ -254,22 +280,31 @@ def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None):
     return out
 
 
-def grouped_linear(xs, w, counts, offsets, swiglu=False, out=None, n_tile=None, rows_hint=None, grid=0, _cfg=None):
-    """Per-expert linear over an expert-sorted activation matrix.
+def grouped_linear(xs, w, counts, offsets, swiglu=False, out=None, n_tile=None, rows_hint=None, grid=0, _cfg=None, glu=None):
+    """Per-expert linear over an expert-sorted activation matrix. glu (limit, slope): the gate/up pair goes through the clamped
+    unit min(g, limit) sigmoid(slope g) (clamp(u, +-limit) + 1) instead of silu(g) u.
 
     xs [rows, K]; w [E, F, K] (or [E, 2I, K] with gate rows first when swiglu); counts / offsets are
     int32 device tensors of E (offsets may have E+1) entries: rows of expert e are
     offsets[e] : offsets[e] + counts[e]. Rows not covered by any expert are left untouched.
     """
     if not xs.is_cuda:
-        return ref.grouped_linear(xs, w.unpack() if isinstance(w, PackedWeight) else w, counts, offsets, swiglu)
+        return ref.grouped_linear(xs, w.unpack() if isinstance(w, PackedWeight) else w, counts, offsets, swiglu, glu)
     _check_act(xs)
     rows, K = xs.shape
     E = w.shape[0]
     F = w.shape[1] // 2 if swiglu else w.shape[1]
     if out is None:
-        out = torch.empty(rows, F, dtype=torch.bfloat16, device=xs.device)
+        out = torch.empty(rows, F, dtype=xs.dtype, device=xs.device)
     if rows == 0:
+        return out
+    if E > _lib.MAX_GROUPS:      # one launch takes up to MAX_GROUPS experts
+        if isinstance(w, PackedWeight):
+            raise ValueError(f"packed expert weights hold at most {_lib.MAX_GROUPS} experts")
+        for e0 in range(0, E, _lib.MAX_GROUPS):
+            e1 = min(E, e0 + _lib.MAX_GROUPS)
+            grouped_linear(xs, w[e0:e1], counts[e0:e1], offsets[e0:e1], swiglu, out, n_tile,
+                           (rows_hint if rows_hint is not None else rows) * (e1 - e0) // E, grid, _cfg, glu)
         return out
     if n_tile is None:
         avg = (rows_hint if rows_hint is not None else rows) / E
@@ -282,7 +317,12 @@ def grouped_linear(xs, w, counts, offsets, swiglu=False, out=None, n_tile=None, 
     p.group_off = offsets.data_ptr()
     p.group_cnt = counts.data_ptr()
     p.grid = grid
-    _gemm_launch(p, "grouped_linear", _cfg)
+    if glu is not None:
+        p.glu, p.glu_limit, p.glu_slope = 1, float(glu[0]), float(glu[1])
+    if tc_gemm_ok(xs, K):
+        _gemm_launch(p, "grouped_linear", _cfg)
+    else:
+        simt_launch(p, xs, rows, "grouped_linear")
     return out
 
 
@@ -708,6 +748,7 @@ def linear_push(x, w, out_local, peer_flag, epoch, done_counter, ldo, grouped=No
     in this process. `epoch` and `done_counter` are local int32 device tensors. grouped = (counts, offsets) selects
     the per-expert form. The consumers pull the buffer over NVLink (reduce_residual_rmsnorm with peer partials).
     """
+    _check_bf16(x)
     _check_act(x)
     rows, K = x.shape
     wv, rows_pg, packed = _wview(w)

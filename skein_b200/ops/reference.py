@@ -26,7 +26,7 @@ def swiglu_linear(x, w13):
     return (torch.nn.functional.silu(g) * u).to(x.dtype)
 
 
-def grouped_linear(xs, w, counts, offsets, swiglu=False):
+def grouped_linear(xs, w, counts, offsets, swiglu=False, glu=None):
     """xs: [rows, K] expert-sorted; w: [E, F(or 2I), K]; rows of expert e are offsets[e] : offsets[e]+counts[e]."""
     E = w.shape[0]
     F = w.shape[1] // 2 if swiglu else w.shape[1]
@@ -37,7 +37,12 @@ def grouped_linear(xs, w, counts, offsets, swiglu=False):
         c, o = counts[e], offsets[e]
         if c == 0:
             continue
-        out[o:o + c] = swiglu_linear(xs[o:o + c], w[e]) if swiglu else linear(xs[o:o + c], w[e])
+        if glu is not None:
+            from .reference_latent import clamped_glu
+            g, u = (xs[o:o + c].float() @ w[e].float().t()).chunk(2, dim=1)
+            out[o:o + c] = clamped_glu(g, u, *glu).to(xs.dtype)
+        else:
+            out[o:o + c] = swiglu_linear(xs[o:o + c], w[e]) if swiglu else linear(xs[o:o + c], w[e])
     return out
 
 

@@ -69,6 +69,8 @@ class _Bucket:
         self.dev_out = torch.zeros(B + N_RESULT_EXTRA, dtype=torch.int32, device=device)
         self.step_counter = torch.zeros(1, dtype=torch.int32, device=device)
         self.graphs = {}           # (feedback, sampling) -> captured step
+        self.logits = None         # logits of the last eager step; of a captured step: graph_logits
+        self.graph_logits = {}
         self.np_views = None
         self.host_in[B:2 * B] = -1
         self.host_in[5 * B:6 * B].view(torch.float32).fill_(1.0)     # top_p
@@ -133,7 +135,7 @@ class ModelRunner:
         if sampling:
             t, k, p, seeds = bk.sampling_views(bk.dev_in)
             smp = SamplingInputs(t, k, p, seeds, pos)      # the random stream is indexed by the token's position
-        sampled, _ = self.dec.forward(inp, sampling=smp)
+        sampled, bk.logits = self.dec.forward(inp, sampling=smp)     # (a captured step rewrites the same logits at every replay)
         bk.dev_out[:bk.B].copy_(sampled)
         if self.device.type == "cuda":
             bk.dev_out[bk.B:].copy_(ops.workspace().status)
@@ -153,6 +155,7 @@ class ModelRunner:
         g = torch.cuda.CUDAGraph()
         with torch.cuda.graph(g):
             self._decode_body(bk, feedback, sampling)
+        bk.graph_logits[key] = bk.logits
         torch.cuda.synchronize()
         bk.dev_in.copy_(saved)  # the capture itself does not run, but keep the inputs pristine
         self.graph_captures += 1
@@ -315,8 +318,9 @@ class ModelRunner:
             self._decode_body(bk, True)
 
     # ---- prefill ----------------------------------------------------------------------------------
-    def _prefill_inputs(self, seqs, sampling):
-        """BatchInputs (and SamplingInputs) of one eager chunk holding every new token of every listed sequence."""
+    def _prefill_inputs(self, seqs, sampling, want=None):
+        """BatchInputs (and SamplingInputs) of one eager chunk holding every new token of every listed sequence. `want` lists, per
+        sequence, the places among its new tokens that produce logits (default: the last one)."""
         dev = self.device
         toks, pos, sot, qs, ql, kl, rows = [], [], [], [], [], [], []
         S = len(seqs)
@@ -324,12 +328,13 @@ class ModelRunner:
         for s, (ids, table, cached) in enumerate(seqs):
             qs.append(len(toks)); ql.append(len(ids)); kl.append(cached + len(ids))
             toks.extend(ids); pos.extend(range(cached, cached + len(ids))); sot.extend([s] * len(ids))
-            rows.append(len(toks) - 1)
+            rows.extend([len(toks) - 1] if want is None else [qs[-1] + i for i in want[s]])
             bt[s, :len(table)] = torch.as_tensor(table, dtype=torch.int32)
         i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
         inp = BatchInputs(token_ids=i32(toks), positions=i32(pos), block_table=bt.to(dev), seq_lens=i32(kl),
                           is_prefill=True, seq_of_token=i32(sot), q_start=i32(qs), q_len=i32(ql), max_q_len=max(ql),
-                          logit_rows=torch.tensor(rows, dtype=torch.int64, device=dev))
+                          logit_rows=torch.tensor(rows, dtype=torch.int64, device=dev), kv_start=i32([sum(kl[:i]) for i in range(S)]),
+                          kv_total=sum(kl), max_cached=max(k - q for k, q in zip(kl, ql)))
         smp = None
         if sampling is not None and any(s[0] > 0 for s in sampling):
             smp = SamplingInputs(torch.tensor([s[0] for s in sampling], dtype=torch.float32, device=dev),
@@ -338,6 +343,19 @@ class ModelRunner:
                                  torch.tensor([s[3] for s in sampling], dtype=torch.int64, device=dev),
                                  i32([n - 1 for n in kl]))
         return inp, smp
+
+    def extend(self, seqs, want):
+        """One step that feeds every listed sequence (new_token_ids, block_table_row, cached_len) its new tokens, portions of
+        prompts beside single decoded tokens, and returns the logits of the wanted places (in order; nothing is sampled). A step
+        of single tokens runs as a decode step, captured like the ones of a generation."""
+        if all(len(s[0]) == 1 for s in seqs):
+            bk = self.bucket(len(seqs))
+            self.load_decode_inputs(bk, [s[0][0] for s in seqs], [s[2] for s in seqs], [s[2] + 1 for s in seqs], [s[1] for s in seqs])
+            self.decode_step(bk)
+            lg = bk.graph_logits[(False, False)] if self.use_graphs else bk.logits
+            return lg[[i for i, w in enumerate(want) for _ in w]]
+        inp, _ = self._prefill_inputs(seqs, None, want)
+        return self.dec.forward_logits(inp)
 
     def prefill(self, seqs, want_logits: bool = False, sampling=None):
         """seqs: list of (new_token_ids, block_table_row, cached_len). Runs one eager chunk holding every new
