@@ -6,8 +6,9 @@
 //   post_norm        x <- g * v / sqrt(mean(v^2) + eps),  v = alpha * x + y,   y a row or a weighted sum of expert rows
 //   poly_norm        a N(z) + b N(z^2) + c N(z^3) + e,   N(v) = v / sqrt(mean(v^2) + eps)
 //
-// The convolution's last inputs are part of a sequence's cache and live with its pages: every page has R = min(taps - 1,
-// page size) tail rows, position p's input sits in row (p mod page size) mod R of p's page. So a page of the prefix cache
+// The convolution's last inputs are part of a sequence's cache and live with its pages: every page has R = min(taps, page
+// size) tail rows, position p's input sits in row (p mod page size) mod R of p's page (taps - 1 rows would hold the state; with
+// one more, a decode step never overwrites a row it reads and can be run again). So a page of the prefix cache
 // brings the convolution's state along, freeing a sequence frees it, and a batch row needs no state slot of its own. The
 // values kept are in the activation type; the convolution reads the same rounded values inside a chunk, so that a result does
 // not depend on how a prompt was cut.

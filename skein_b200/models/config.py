@@ -65,8 +65,13 @@ class ModelConfig:
         blocks = range(self.num_layers) if blocks is None else blocks
         if not self.is_layered:
             return 2 * (self.num_kv_heads // tp) * page_size * self.head_dim * elem * len(blocks)
-        tail = min(self.conv_taps - 1, page_size) * self.hidden_size
+        tail = self.conv_tail_rows(page_size) * self.hidden_size
         return sum((self.layers[b].mixer.cache_width * page_size + tail) * elem for b in blocks)
+
+    def conv_tail_rows(self, page_size: int) -> int:
+        """Rows per cache page that keep the input convolution's last inputs. One more than the taps that look back, so that a
+        step writes no row it reads: running a step twice (a graph's warm-up before its capture) gives the same result twice."""
+        return min(self.conv_taps, page_size) if self.conv_taps > 1 else 0
 
     def param_shapes(self) -> dict:
         """Checkpoint tensor name -> shape (designs that list their layers)."""

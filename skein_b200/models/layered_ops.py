@@ -35,7 +35,7 @@ class LayeredOps:
             if key not in tables:
                 tables[key] = ref.rope_cos_sin_table(self.max_pos, key[0], key[1], dev)
         self.rope_tables = [tables[(sp.mixer.rot_dim, sp.mixer.rope_base)] for sp in cfg.layers]
-        R = min(cfg.conv_taps - 1, self.page_size)
+        R = cfg.conv_tail_rows(self.page_size)
         new = lambda *shape: torch.zeros(*shape, dtype=self.act_dtype, device=dev)      # noqa: E731
         self.kv = [new(num_pages, self.page_size, sp.mixer.cache_width) for sp in cfg.layers] if num_pages else []
         # the input convolution's last inputs live with the pages of the cache (csrc/kernels/postnorm.cu)
