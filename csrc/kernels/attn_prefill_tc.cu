@@ -53,21 +53,6 @@ struct AttnPrefillTcParams {
   float scale_log2e;
 };
 
-// Shared-memory descriptor of an MN-major operand tile (the reduction dimension strides over 128-byte rows): 64
-// elements of the MN dimension are contiguous in a row, 8 rows form a 1024-byte swizzle atom; `lbo` is the distance
-// between consecutive 64-element chunks of the MN dimension, the atoms of consecutive 8-row groups follow at 1024 bytes.
-__device__ __forceinline__ uint64_t umma_desc_sw128_mn(uint32_t smem_addr, uint32_t lbo_bytes) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4);
-  d |= static_cast<uint64_t>(lbo_bytes >> 4) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
-}
-
-__device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-
 __global__ void __launch_bounds__(TC_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        const AttnPrefillTcParams p) {

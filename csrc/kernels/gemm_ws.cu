@@ -35,6 +35,8 @@
 #include <cuda.h>
 #include <cuda_runtime.h>
 #include <cuda_fp16.h>
+#include <array>
+#include <map>
 #include <mutex>
 #include <type_traits>
 #include <unordered_map>
@@ -816,6 +818,34 @@ int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k
     cache.emplace(key, *out);
   }
   return rc;
+}
+
+// [rows, heads, d] bf16 with `head_stride` / `row_stride` elements between heads / rows; box = [box_rows, 1, 64 elements].
+// Elements past d read as zero, so a 64-wide box may cover a shorter head.
+int cached_tmap_heads(CUtensorMap* out, const void* base, uint64_t rows, uint64_t heads, uint64_t d, uint64_t head_stride,
+                      uint64_t row_stride, uint32_t box_rows) {
+  typedef std::array<uint64_t, 7> Key;
+  static std::map<Key, CUtensorMap> cache;
+  static std::mutex mu;
+  const Key key{(uint64_t)(uintptr_t)base, rows, heads, d, head_stride, row_stride, box_rows};
+  std::lock_guard<std::mutex> lk(mu);
+  auto it = cache.find(key);
+  if (it != cache.end()) { *out = it->second; return 0; }
+  EncodeTiledFn fn = get_encode_fn();
+  if (!fn) return -10;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) != 0) return -11;
+  if (head_stride % 8 != 0 || row_stride % 8 != 0) return -12;
+  cuuint64_t dims[3] = {d, heads, rows};
+  cuuint64_t strides[2] = {head_stride * 2, row_stride * 2};
+  cuuint32_t box[3] = {64, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return -13;
+  if (cache.size() > 4096) cache.clear();
+  cache.emplace(key, *out);
+  return 0;
 }
 
 static int sm_count_cached() {
