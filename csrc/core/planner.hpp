@@ -235,7 +235,8 @@ inline std::optional<DpResult> layer_dtype_dp(const Graph& ir, const CostModel& 
   if (bud.memory_bytes == 0) return std::nullopt;
   const uint64_t bytes_per_bucket = std::max<uint64_t>(1, (bud.memory_bytes + MB - 1) / MB);
   const double drift_per_bucket = std::max(bud.drift / (double)DB, std::numeric_limits<double>::min());
-  const std::vector<PerLayerDtype> combos = allowed ? *allowed : all_combos();
+  // designs that list their layers run with bf16 weights and caches
+  const std::vector<PerLayerDtype> combos = ir.meta.layered ? std::vector<PerLayerDtype>{{Dtype::Bf16, Dtype::Bf16, Dtype::Bf16}} : allowed ? *allowed : all_combos();
   const size_t NC = combos.size();
   std::vector<size_t> mem_step(NB * NC), drift_step(NB * NC);
   std::vector<double> cost(NB * NC);

@@ -56,40 +56,64 @@ __device__ __forceinline__ float lt_block_sum(float v, float* sh) {
   return t;
 }
 
-// one CTA per token
+// one CTA per token; a thread keeps up to LT_KEEP of its elements in registers between the sum and the store
+constexpr int LT_THREADS = 256, LT_KEEP = 4;
 template <typename T>
-__global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppendParams p) {
-  __shared__ float sh[32];
+__global__ void __launch_bounds__(LT_THREADS) latent_append_kernel(const LatentAppendParams p) {
+  __shared__ float sh[2][32];
   pdl_trigger();
   pdl_wait();
-  const int t = blockIdx.x, tid = threadIdx.x;
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const T* row = (const T*)p.proj + (size_t)t * p.proj_ld;
-  if (p.q_rank > 0) {
-    float ss = 0.f;
-    for (int i = tid; i < p.q_rank; i += blockDim.x) { const float v = lt_f<T>(row[i]); ss += v * v; }
-    const float inv = 1.f / sqrtf(lt_block_sum(ss, sh) / (float)p.q_rank + p.eps);
-    T* cq = (T*)p.cq + (size_t)t * p.q_rank;
-    for (int i = tid; i < p.q_rank; i += blockDim.x) cq[i] = lt_t<T>(lt_f<T>(row[i]) * inv * p.q_norm[i]);
-  }
-  const int pos = p.positions[t];
-  if (pos < 0) return;
-  if (pos >= p.max_pos) { report_status(p.status, ST_BAD_INDEX, pos); return; }
-  const int seq = p.seq_of_token ? p.seq_of_token[t] : t;
-  const int page = p.block_table[(size_t)seq * p.max_blocks + pos / p.page_size];
-  if (page < 0 || page >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, page); return; }
-  const int L = p.kv_rank + p.rot, slot = pos % p.page_size;
   const T* ckr = row + p.off_kv;
-  float ss = 0.f;
-  for (int i = tid; i < p.kv_rank; i += blockDim.x) { const float v = lt_f<T>(ckr[i]); ss += v * v; }
-  const float inv = 1.f / sqrtf(lt_block_sum(ss, sh) / (float)p.kv_rank + p.eps);
+  int pos = p.positions[t];
+  const int seq = p.seq_of_token ? p.seq_of_token[t] : t;
+  int page = -1;
+  if (pos >= p.max_pos) { report_status(p.status, ST_BAD_INDEX, pos); pos = -1; }
+  if (pos >= 0) {
+    page = p.block_table[(size_t)seq * p.max_blocks + pos / p.page_size];
+    if (page < 0 || page >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, page); page = -1; }
+  }
+  float kv[LT_KEEP], sq = 0.f, sk = 0.f;
+  for (int i = tid; i < p.q_rank; i += LT_THREADS) { const float v = lt_f<T>(row[i]); sq += v * v; }
+#pragma unroll
+  for (int k = 0; k < LT_KEEP; ++k) {
+    const int i = tid + k * LT_THREADS;
+    kv[k] = i < p.kv_rank ? lt_f<T>(ckr[i]) : 0.f;
+    sk += kv[k] * kv[k];
+  }
+  for (int i = tid + LT_KEEP * LT_THREADS; i < p.kv_rank; i += LT_THREADS) { const float v = lt_f<T>(ckr[i]); sk += v * v; }
+  for (int o = 16; o > 0; o >>= 1) { sq += __shfl_xor_sync(0xffffffffu, sq, o); sk += __shfl_xor_sync(0xffffffffu, sk, o); }
+  if (lane == 0) { sh[0][warp] = sq; sh[1][warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < LT_THREADS / 32; ++w) { sq += sh[0][w]; sk += sh[1][w]; }
+  if (p.q_rank > 0) {
+    const float inv = 1.f / sqrtf(sq / (float)p.q_rank + p.eps);
+    T* cq = (T*)p.cq + (size_t)t * p.q_rank;
+    for (int i = tid; i < p.q_rank; i += LT_THREADS) cq[i] = lt_t<T>(lt_f<T>(row[i]) * inv * p.q_norm[i]);
+  }
+  if (page < 0) return;      // padding row
+  const int L = p.kv_rank + p.rot, slot = pos % p.page_size;
+  const float inv = 1.f / sqrtf(sk / (float)p.kv_rank + p.eps);
   T* dst = (T*)p.cache + ((size_t)page * p.page_size + slot) * L;
   T* den = p.dense ? (T*)p.dense + (size_t)(p.dense_start[seq] + pos) * L : nullptr;
-  for (int i = tid; i < p.kv_rank; i += blockDim.x) {
+#pragma unroll
+  for (int k = 0; k < LT_KEEP; ++k) {
+    const int i = tid + k * LT_THREADS;
+    if (i < p.kv_rank) {
+      const T v = lt_t<T>(kv[k] * inv * p.kv_norm[i]);
+      dst[i] = v;
+      if (den) den[i] = v;
+    }
+  }
+  for (int i = tid + LT_KEEP * LT_THREADS; i < p.kv_rank; i += LT_THREADS) {
     const T v = lt_t<T>(lt_f<T>(ckr[i]) * inv * p.kv_norm[i]);
     dst[i] = v;
     if (den) den[i] = v;
   }
-  for (int i = tid; i < p.rot / 2; i += blockDim.x) {
+  for (int i = tid; i < p.rot / 2; i += LT_THREADS) {
     const float2 cs = reinterpret_cast<const float2*>(p.cos_sin)[(size_t)pos * (p.rot / 2) + i];
     const float u = lt_f<T>(ckr[p.kv_rank + 2 * i]), w = lt_f<T>(ckr[p.kv_rank + 2 * i + 1]);
     const T a = lt_t<T>(u * cs.x - w * cs.y), b = lt_t<T>(w * cs.x + u * cs.y);
@@ -100,7 +124,7 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppendPa
   // the page) read
   if (p.x != nullptr && p.R > 0 && (pos >= p.seq_lens[seq] - (p.taps - 1) || slot >= p.page_size - (p.taps - 1))) {
     T* tl = (T*)p.tail + ((size_t)page * p.R + slot % p.R) * p.C;
-    for (int i = tid; i < p.C; i += blockDim.x) tl[i] = lt_t<T>(p.x[(size_t)t * p.C + i]);
+    for (int i = tid; i < p.C; i += LT_THREADS) tl[i] = lt_t<T>(p.x[(size_t)t * p.C + i]);
   }
 }
 
@@ -250,8 +274,8 @@ extern "C" int skein_latent_append(const void* proj, int proj_ld, int off_kv, co
   if (rot % 2 != 0 || kv_rank < 1 || (q_rank > 0 && (q_norm == nullptr || cq == nullptr)) || (dense && !dense_start) || (x && !seq_lens)) return -1;
   LatentAppendParams p{proj, q_norm, kv_norm, cos_sin, positions, seq_of_token, block_table, cache, cq, dense, dense_start, x, tail, seq_lens,
                        status, eps, proj_ld, off_kv, q_rank, kv_rank, rot, max_pos, max_blocks, num_pages, page_size, C, R, taps};
-  if (fp32) return (int)launch_pdl(latent_append_kernel<float>, dim3(T), dim3(128), 0, (cudaStream_t)stream, p);
-  return (int)launch_pdl(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, (cudaStream_t)stream, p);
+  if (fp32) return (int)launch_pdl(latent_append_kernel<float>, dim3(T), dim3(LT_THREADS), 0, (cudaStream_t)stream, p);
+  return (int)launch_pdl(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(LT_THREADS), 0, (cudaStream_t)stream, p);
 }
 
 extern "C" int skein_rope_rows(void* q, long long ld, const int* positions, const float* cos_sin, int T, int H, int D, int rot, int max_pos,

@@ -299,13 +299,14 @@ __global__ void __launch_bounds__(512) post_norm_route_kernel(const PostNormPara
 // ---- polynomial activation ----------------------------------------------------------------------------
 // one CTA per row of F values, parked in dynamic shared memory
 template <typename T, int V>
-__global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, T* __restrict__ out, int F, float eps) {
+__global__ void __launch_bounds__(1024) poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, T* __restrict__ out, int F, float eps) {
   extern __shared__ __align__(16) float row_sm[];
-  __shared__ float sh[32];
+  __shared__ float sh[3][32];
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x;
   float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll 4
   for (int i = threadIdx.x * V; i < F; i += blockDim.x * V) {
     float v[V];
     load_v<T, V>(z + (size_t)b * F + i, v);
@@ -316,9 +317,20 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z,
       s1 += q; s2 += q * q; s3 += q * q * q;
     }
   }
-  s1 = pn_block_sum(s1, sh);
-  s2 = pn_block_sum(s2, sh);
-  s3 = pn_block_sum(s3, sh);
+  for (int o = 16; o > 0; o >>= 1) {
+    s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+    s2 += __shfl_xor_sync(0xffffffffu, s2, o);
+    s3 += __shfl_xor_sync(0xffffffffu, s3, o);
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (lane == 0) { sh[0][warp] = s1; sh[1][warp] = s2; sh[2][warp] = s3; }
+  __syncthreads();
+  s1 = lane < nw ? sh[0][lane] : 0.f; s2 = lane < nw ? sh[1][lane] : 0.f; s3 = lane < nw ? sh[2][lane] : 0.f;
+  for (int o = 16; o > 0; o >>= 1) {
+    s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+    s2 += __shfl_xor_sync(0xffffffffu, s2, o);
+    s3 += __shfl_xor_sync(0xffffffffu, s3, o);
+  }
   const float n = (float)F;
   const float ca = act[0] / sqrtf(s1 / n + eps), cb = act[1] / sqrtf(s2 / n + eps), cc = act[2] / sqrtf(s3 / n + eps), ce = act[3];
   for (int i = threadIdx.x * V; i < F; i += blockDim.x * V) {
@@ -449,7 +461,7 @@ extern "C" int skein_poly_norm(const void* z, const float* act, void* out, int T
   if (F < 1 || F * 4 > 200 * 1024) return -1;
   cudaStream_t s = (cudaStream_t)stream;
   const bool v4 = F % 4 == 0;
-  const dim3 b(row_threads(F, v4 ? 4 : 1, 256));
+  const dim3 b(row_threads(F, v4 ? 4 : 1, T <= 256 ? 1024 : 256));     // few rows: more threads per row
   const size_t sm = (size_t)F * 4;
   auto go = [&](auto fn, auto zz, auto oo) -> int {
     cudaError_t e = allow_smem(fn, (int)sm);

@@ -353,6 +353,19 @@ def autotune_decode_gemms(cfg, tp: int, batch: int, out_path, seed: int = 0, bud
     cache = tuning.KernelConfigCache(out_path)
     x = bf(batch, H, std=1.0)
     found = {}
+    if cfg.is_layered:
+        from .models.layered import decode_gemm_shapes
+        for name, F, K, E, swiglu in decode_gemm_shapes(cfg):
+            if E == 0:
+                found[name] = ops.tune_linear(bf(batch, K, std=1.0), bf(F, K), cache=cache, budget=budget)[0]
+            else:
+                per = max(1, batch * 2 // E)
+                cnt = torch.full((E,), per, dtype=torch.int32, device=dev)
+                off = (torch.arange(E + 1, device=dev) * per).to(torch.int32)
+                found[name] = ops.tune_grouped(bf(E * per, K, std=1.0), bf(E, F, K), cnt, off, swiglu, cache, budget)[0]
+        ops.workspace().check_status()
+        cache.save()
+        return found
     found["qkv"] = ops.tune_linear(x, bf((hq + 2 * hkv) * D, H), cache=cache, budget=budget)[0]
     found["o_proj"] = ops.tune_linear(bf(batch, hq * D, std=1.0), bf(H, hq * D), cache=cache, budget=budget)[0]
     found["lm_head"] = ops.tune_linear(x, bf(cfg.vocab_size // tp, H), cache=cache, budget=budget)[0]

@@ -35,6 +35,8 @@ def _rope(x, pos, theta, scaling=None):
 @torch.no_grad()
 def forward_full(cfg: ModelConfig, w: ModelWeights, token_ids: torch.Tensor, capture_hidden: list | None = None):
     """Full-sequence forward of ONE sequence (unsharded weights). Returns fp32 logits [T, V]."""
+    if cfg.is_layered:
+        return _forward_layered(cfg, w, token_ids, capture_hidden)
     T = token_ids.shape[0]
     H, D, Hq, Hkv = cfg.hidden_size, cfg.head_dim, cfg.num_heads, cfg.num_kv_heads
     x = w.embed[token_ids.long()].float()
@@ -85,3 +87,60 @@ def forward_full(cfg: ModelConfig, w: ModelWeights, token_ids: torch.Tensor, cap
             capture_hidden.append(x.clone())
     h = _rms(x, w.final_norm, cfg.rms_norm_eps)
     return h @ w.lm_head.float().t()
+
+
+def _forward_layered(cfg, w, token_ids, capture_hidden):
+    """The same for designs that list their layers (post-norm blocks of latent attention), keys and values expanded per head."""
+    from .layered import GLU_SLOPE, RoutedFFSpec
+    T, eps = token_ids.shape[0], cfg.rms_norm_eps
+    unit = lambda v: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)      # noqa: E731
+    x = w.embed[token_ids.long()].float()
+    pos = torch.arange(T, device=x.device)
+    mask = torch.triu(torch.full((T, T), float("-inf"), device=x.device), diagonal=1)
+
+    def rotate(v, base):        # neighbouring pairs
+        n = v.shape[-1]
+        ang = pos.double()[:, None] * base ** (-torch.arange(0, n, 2, device=x.device).double() / n)
+        c, s = ang.cos().float(), ang.sin().float()
+        if v.dim() == 3:
+            c, s = c[:, None], s[:, None]
+        return torch.stack([v[..., 0::2] * c - v[..., 1::2] * s, v[..., 1::2] * c + v[..., 0::2] * s], dim=-1).flatten(-2)
+
+    for sp, lw in zip(cfg.layers, w.layers):
+        m, mw = sp.mixer, lw.mixer
+        H, D, V, K = m.heads, m.dim, m.vdim, m.kv_rank
+        taps = lw.conv.shape[0]
+        h = x + sum(lw.conv[j] * torch.nn.functional.pad(x, (0, 0, taps - 1 - j, 0))[:T] for j in range(taps))
+        z = h @ mw.w_in.float().t()
+        q = z[:, :m.q_width] if not m.q_rank else (unit(z[:, :m.q_rank]) * mw.q_norm) @ mw.w_uq.float().t()
+        q = q.view(T, H, D + m.rot_dim)
+        c = unit(z[:, mw.off_kv:mw.off_kv + K]) * mw.kv_norm
+        kr = rotate(z[:, mw.off_kv + K:mw.off_kv + K + m.rot_dim], m.rope_base)
+        kv = c @ mw.w_ukv.float().t()
+        k, v = kv[:, :H * D].view(T, H, D), kv[:, H * D:].view(T, H, V)
+        s = (torch.einsum("qhd,khd->hqk", q[..., :D], k) + torch.einsum("qhr,kr->hqk", rotate(q[..., D:], m.rope_base), kr)) * m.scale
+        o = torch.einsum("hqk,khv->qhv", torch.softmax(s + mask, dim=-1), v).reshape(T, H * V)
+        if m.gated:
+            o = o * torch.sigmoid(z[:, mw.off_gate:mw.off_gate + H * V])
+        x = unit(cfg.post_alpha * x + o @ mw.wo.float().t()) * lw.norm1
+        if isinstance(sp.mlp, RoutedFFSpec):
+            f = sp.mlp
+            sc = torch.softmax(x @ lw.router.float().t(), dim=-1)
+            best = sc.view(T, f.groups, -1).amax(-1).topk(f.keep, dim=-1).indices
+            ok = torch.zeros(T, f.groups, dtype=torch.bool, device=x.device).scatter_(1, best, True).repeat_interleave(f.experts // f.groups, dim=1)
+            ids = sc.masked_fill(~ok, -1.0).topk(f.top, dim=-1).indices
+            y = torch.zeros_like(x)
+            for e in range(f.experts):
+                rows = (ids == e).any(-1).nonzero().squeeze(-1)
+                if rows.numel():
+                    g, u = (x[rows] @ lw.w13[e].float().t()).chunk(2, dim=1)
+                    g, u = g.clamp(max=f.limit), u.clamp(-f.limit, f.limit)
+                    y[rows] += sc[rows, e:e + 1] * ((g * torch.sigmoid(GLU_SLOPE * g) * (u + 1)) @ lw.w2[e].float().t())
+        elif sp.mlp is not None:
+            z = x @ lw.w_up.float().t()
+            y = (lw.act[0] * unit(z) + lw.act[1] * unit(z ** 2) + lw.act[2] * unit(z ** 3) + lw.act[3]) @ lw.w2.float().t()
+        if sp.mlp is not None:
+            x = unit(cfg.post_alpha * x + y) * lw.norm2
+        if capture_hidden is not None:
+            capture_hidden.append(x.clone())
+    return (unit(x) * w.final_norm) @ w.lm_head.float().t()

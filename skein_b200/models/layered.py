@@ -171,6 +171,45 @@ def param_shapes(cfg) -> dict:
     return s
 
 
+def active_params(cfg) -> int:
+    """Weights one token multiplies with (its chosen experts only), output projection included."""
+    C, n = cfg.hidden_size, cfg.vocab_size * cfg.hidden_size
+    for sp in cfg.layers:
+        m = sp.mixer
+        n += C * (m.cache_width + m.heads * m.vdim * (2 if m.gated else 1)) + m.heads * (m.dim + m.vdim) * m.kv_rank
+        n += m.q_rank * (C + m.q_width) if m.q_rank else C * m.q_width
+        if isinstance(sp.mlp, DenseFFSpec):
+            n += 2 * C * sp.mlp.ff
+        elif isinstance(sp.mlp, RoutedFFSpec):
+            n += 3 * C * sp.mlp.ff * sp.mlp.top + C * sp.mlp.experts
+    return n
+
+
+def decode_gemm_shapes(cfg) -> list:
+    """(name, features, K, experts or 0, gate/up pair) of the distinct projections of a decode step that the tensor-core GEMM
+    runs."""
+    C, seen, out = cfg.hidden_size, set(), []
+
+    def add(name, F, K, E=0, swiglu=False):
+        if (F, K, E, swiglu) not in seen and K % 8 == 0 and E <= 64:
+            seen.add((F, K, E, swiglu))
+            out.append((name, F, K, E, swiglu))
+    for i, sp in enumerate(cfg.layers):
+        m = sp.mixer
+        add(f"l{i}.in", _up8(m.q_rank or m.q_width) + _up8(m.cache_width) + (_up8(m.heads * m.vdim) if m.gated else 0), C)
+        if m.q_rank:
+            add(f"l{i}.uq", m.q_width, m.q_rank)
+        add(f"l{i}.o", C, m.heads * m.vdim)
+        if isinstance(sp.mlp, DenseFFSpec):
+            add(f"l{i}.up", sp.mlp.ff, C)
+            add(f"l{i}.down", C, sp.mlp.ff)
+        elif isinstance(sp.mlp, RoutedFFSpec):
+            add(f"l{i}.experts_gate_up", 2 * sp.mlp.ff, C, sp.mlp.experts, True)
+            add(f"l{i}.experts_down", C, sp.mlp.ff, sp.mlp.experts)
+    add("head", cfg.vocab_size, C)
+    return out
+
+
 # ---- weights ------------------------------------------------------------------------------------------------------
 def _up8(n: int) -> int:
     return (n + 7) // 8 * 8

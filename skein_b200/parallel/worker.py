@@ -30,14 +30,13 @@ from ..runtime.tokenizer import Tokenizer
 from . import launcher
 
 
-def size_kv_pool(art: Artifact, lay, device, total_kv_bytes: int, page_size: int = 16, reserve_frac: float = 0.08,
+def size_kv_pool(art: Artifact, lay, device, total_kv_bytes: int, page_size: int | None = None, reserve_frac: float = 0.08,
                  bytes_per_token: int = 0) -> int:
     """Pages in the per-layer pool: from an explicit byte budget (with the model's KV bytes per token on this rank,
     or the caller's `bytes_per_token`), else from the memory left after the weights."""
     cfg = art.cfg
-    n_layers = len(lay.stage_layers(cfg.num_layers))
-    kv_heads = cfg.num_kv_heads // lay.tp
-    page_bytes = 2 * kv_heads * page_size * cfg.head_dim * 2 * n_layers
+    page_size = page_size or cfg.default_page_size
+    page_bytes = cfg.cache_bytes_per_page(page_size, lay.tp, lay.stage_layers(cfg.num_layers))
     if bytes_per_token > 0:
         page_bytes = bytes_per_token * page_size
     if total_kv_bytes > 0:
@@ -67,9 +66,10 @@ def build_engine(art: Artifact, rank: int, device, comm, args, comm_moe=None, pp
         from ..ops import tuning
         tuning.activate(tuning.KernelConfigCache(tuned, strict=False))   # measured configurations win over the heuristics
     weights = art.load_weights(rank, device)
-    pages = size_kv_pool(art, lay, device, args.total_kv_bytes, bytes_per_token=getattr(args, "bytes_per_token", 0))
-    pages = min(pages, max(8, (args.max_seq_len // 16 + 1) * max(1, args.max_batch or art.plan["batching"]["max_batch"]) * 2))
-    dec = Decoder(art.cfg, weights, lay, num_pages=pages, page_size=art.plan["kv"]["layout"].get("page_size", 16),
+    page_size = art.plan["kv"]["layout"].get("page_size", art.cfg.default_page_size)
+    pages = size_kv_pool(art, lay, device, args.total_kv_bytes, page_size, bytes_per_token=getattr(args, "bytes_per_token", 0))
+    pages = min(pages, max(8, (args.max_seq_len // page_size + 1) * max(1, args.max_batch or art.plan["batching"]["max_batch"]) * 2))
+    dec = Decoder(art.cfg, weights, lay, num_pages=pages, page_size=page_size,
                   max_pos=min(args.max_seq_len, art.cfg.max_position_embeddings), comm=comm, comm_moe=comm_moe)
     # Pure expert parallelism decodes with data-parallel attention: every rank attends over its own share of the step's
     # sequences and the MoE blocks exchange tokens over peer memory (SKEIN_EP_DP_ATTENTION=0: attention over all

@@ -18,6 +18,8 @@ of the server life cycle that calls it (crates/skein_runtime/src/server/lifecycl
 """
 from __future__ import annotations
 
+from dataclasses import fields, is_dataclass
+
 import torch
 
 from ..compile.artifact import Artifact, ArtifactError, update_latest_symlink, verify_shape_compatibility
@@ -36,6 +38,16 @@ def _copy_into(old, new) -> None:
     old.copy_(new)
 
 
+def _slots(weights):
+    """Every weight slot of a layer, in declaration order (a layer's mixer is a group of its own)."""
+    for f in fields(weights):
+        v = getattr(weights, f.name)
+        if is_dataclass(v):
+            yield from _slots(v)
+        elif v is None or hasattr(v, "copy_"):
+            yield v
+
+
 def mount_weights(engine, artifact_path, rank: int) -> None:
     """Copy rank `rank`'s shard of the artifact into the engine's live weights and forget cached prefixes."""
     new = Artifact(artifact_path)
@@ -44,8 +56,8 @@ def mount_weights(engine, artifact_path, rank: int) -> None:
     fresh = new.load_weights(rank, inner.device)
     with torch.no_grad():
         for old_l, new_l in zip(inner.w.layers, fresh.layers):
-            for name in ("attn_norm", "wqkv", "wo", "ffn_norm", "router", "w13", "w2", "bqkv"):
-                _copy_into(getattr(old_l, name), getattr(new_l, name))
+            for old_t, new_t in zip(_slots(old_l), _slots(new_l)):
+                _copy_into(old_t, new_t)
             if set(old_l.fp8) != set(new_l.fp8):
                 raise HotSwapError("the artifacts quantise different projections of a block")
             for name, w8 in old_l.fp8.items():
