@@ -1,18 +1,23 @@
-// Attention of single rows over the latent cache: all heads of a row share one cached row of kv_rank + rot elements per token,
-// so the heads are the rows of the MMA tile and every cached byte is read once per 16 / 32 / 64 heads.
+// Attention of single rows over the latent cache on the 5th-generation tensor cores. All heads of a row share one cached row of
+// kv_rank + rot elements per token, so the cached tokens (and then the latent's columns) fill the 128-row side of the MMA and
+// the heads of the row, 16 or 32 per CTA, are its narrow side; more heads of a row read the cache through L2.
 //
 //   score[h, j] = (q_abs[h] . c_j + rot(q_rot[h]) . k_rot_j) * scale          out[h] = sum_j softmax(score)[h, j] c_j
 //
-// grid = (splits, head groups, rows); the splits of a row form a cluster. A CTA has 8 compute warps and a producer warp that
-// streams tiles of 32 or 64 tokens (whole pages or parts of one, 128-byte swizzle, TMA) into a ring. Per tile:
-//   S = Q C^T      a warp owns 8 tokens and one or two 16-head tiles, over all of kv_rank + rot
-//   softmax        in shared memory, a warp owns whole head rows; P in bf16
-//   O += P C       a warp owns an eighth of the kv_rank columns for all heads of the group, accumulators in registers
-// The splits' results are merged through distributed shared memory: every CTA of the cluster parks its unnormalised O with its
-// maxima and sums, and merges a share of the head rows from all of them. Every wait of the ring is bounded.
+// grid = (splits, head groups, rows); the splits of a row form a cluster. A CTA walks its tokens in tiles of 128, kept in shared
+// memory as 64-column blocks of [128 tokens][128 bytes]:
+//
+//   warp 0      TMA producer: pages of the tile, block by block; a block is refilled as soon as the products that read it are done
+//   warp 1      MMA issuer: S^T = C Q^T (tokens x heads, accumulated over the blocks as they land), and after the softmax
+//               O^T += C^T P^T, 128 latent columns at a time (the tile is the transposed A operand, P comes from shared memory)
+//   warps 2-5   softmax, thread = token: column maxima by halving exchanges inside a warp and a step through shared memory, P to
+//               shared memory, per-thread partial sums; O is rescaled in tensor memory only when a maximum moved by more than 2^8
+//
+// At the end the CTA parks its unnormalised O with its maxima and sums in shared memory, and every CTA of the cluster merges a
+// share of the head rows from all of them through distributed shared memory. Every wait is bounded.
 //
 // q_abs holds the queries with the key expansion already applied; the rotated query part is rotated here, on its way to shared
-// memory. Products run on mma.sync m16n8k16 (bf16, fp32 accumulation): with few heads the kernel is bound by the cache's bytes.
+// memory.
 #include "ptx.cuh"
 #include "launch.cuh"
 #include <cuda.h>
@@ -23,10 +28,13 @@ namespace skein {
 
 int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes, uint32_t box_rows);
 
-constexpr int LD_WARPS = 8;
-constexpr int LD_THREADS = (LD_WARPS + 1) * 32;
-constexpr int LD_MAX_STAGES = 6;
+constexpr int LD_THREADS = 192;
+constexpr int LD_BN = 64;                            // tokens per tile
+constexpr int LD_STAGES = 2;
+constexpr int LD_CHUNK = LD_BN * 128;                // a 64-column block of a tile
+constexpr int LD_MAX_GROUPS = 5;                     // groups of blocks with a barrier of their own: 128 latent columns each, the rest
 constexpr int LD_MAX_SPLITS = 8;
+constexpr int LD_TMEM_COLS = 256;
 constexpr uint64_t LD_BUDGET_NS = 2000000000ull;
 
 struct LatentDecodeParams {
@@ -40,27 +48,14 @@ struct LatentDecodeParams {
   int* status;
   long long q_ld;
   float scale_log2e;
-  int H, D, rot, K, max_pos, max_blocks, num_pages, page_size, splits, stages, nch, box_rows;
+  int H, D, rot, K, max_pos, max_blocks, num_pages, page_size, splits, nch, box_rows;
 };
 
-__device__ __forceinline__ void ld_ldsm4(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ld_ldsm4_t(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ld_ldsm2_t(uint32_t addr, uint32_t* r) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
-}
-__device__ __forceinline__ void ld_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// byte offset of 16-byte chunk c of row r in a tile kept as 64-element column blocks of [rows][128 bytes], 128-byte swizzle
+// byte offset of 16-byte chunk c of row r in 64-column blocks of [rows][128 bytes], 128-byte swizzle
 __device__ __forceinline__ uint32_t ld_off(int r, int c, int rows) {
   return (uint32_t)((c >> 3) * rows * 128 + r * 128 + (((c & 7) ^ (r & 7)) << 4));
 }
-__device__ __forceinline__ void ld_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+__device__ __forceinline__ void ld_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 __device__ __forceinline__ void ld_cluster_sync() {
   asm volatile("barrier.cluster.arrive.release;\n\tbarrier.cluster.wait.acquire;" ::: "memory");
 }
@@ -80,101 +75,194 @@ __device__ __forceinline__ float4 ld_remote_f4(uint32_t addr) {
   return v;
 }
 
-// MT: 16-head tiles per CTA; NT: 8-column tiles of O per warp (64 * NT >= kv_rank); BN: tokens per tile
-template <int MT, int NT, int BN>
+// v[NH] per lane -> lane l returns the maximum (or sum) over the warp's lanes of element l mod NH, by halving exchanges
+template <int NH, bool MAX>
+__device__ __forceinline__ float ld_column_reduce(const float* v) {
+  const int lane = threadIdx.x & 31;
+  float a[NH];
+#pragma unroll
+  for (int i = 0; i < NH; ++i) a[i] = v[i];
+  if (NH == 16) {
+#pragma unroll
+    for (int i = 0; i < NH; ++i) {
+      const float o = __shfl_xor_sync(0xffffffffu, a[i], 16);
+      a[i] = MAX ? fmaxf(a[i], o) : a[i] + o;
+    }
+  }
+#pragma unroll
+  for (int s = NH / 2; s > 0; s >>= 1) {
+    const bool up = (lane & s) != 0;       // lanes with this bit keep the upper half
+#pragma unroll
+    for (int i = 0; i < s; ++i) {
+      const float send = up ? a[i] : a[i + s], keep = up ? a[i + s] : a[i];
+      const float o = __shfl_xor_sync(0xffffffffu, send, s);
+      a[i] = MAX ? fmaxf(keep, o) : keep + o;
+    }
+  }
+  return a[0];
+}
+
+template <int NH> __device__ __forceinline__ void ld_tmem_load(uint32_t addr, uint32_t* r) { if (NH == 32) tmem_ld32(addr, r); else tmem_ld16(addr, r); }
+
+// NH: heads per CTA
+template <int NH>
 __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
-  constexpr int ROWS = 16 * MT;
-  constexpr int NB = BN / 8;                       // 8-token units of a tile
-  constexpr int MPW = MT * NB / LD_WARPS;          // head tiles per warp in the S phase
-  constexpr int P_LD = BN + 8;                     // elements per row of P (16 bytes of padding: conflict-free ldmatrix)
-  constexpr int S_LD = BN + 4;
-  static_assert(MPW >= 1 && MPW * LD_WARPS == MT * NB, "tile shape");
   extern __shared__ uint8_t smem_raw[];
-  __shared__ __align__(8) uint64_t bar_full[LD_MAX_STAGES], bar_empty[LD_MAX_STAGES];
-  __shared__ float alpha_s[ROWS], m_s[ROWS], l_s[ROWS];
-  __shared__ int abort_flag;
+  __shared__ __align__(8) uint64_t bar_full[LD_STAGES * LD_MAX_GROUPS], bar_empty[LD_STAGES * LD_MAX_GROUPS], bar_s[2], bar_p, bar_o;
+  __shared__ __align__(16) float m_s[NH];
+  __shared__ float wred[4][NH], l_s[NH], alpha_s[NH], w_s[LD_MAX_SPLITS][NH];
+  __shared__ uint32_t tmem_slot;
+  __shared__ int abort_flag, moved;
   pdl_trigger();
   pdl_wait();
-  const int split = blockIdx.x, h0 = blockIdx.y * ROWS, t = blockIdx.z;
+  const int split = blockIdx.x, h0 = blockIdx.y * NH, t = blockIdx.z, ns = p.splits;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int K = p.K, nch = p.nch;
+  const int K = p.K, nch = p.nch, park_ld = K + 4;
   int pos = p.positions[t];
   if (pos >= p.max_pos) { if (tid == 0) report_status(p.status, ST_BAD_INDEX, pos); pos = -1; }
   if (pos < 0) {      // padding row: the same decision in every CTA of the cluster
     if (split == 0)
-      for (int i = tid; i < ROWS * K; i += LD_THREADS)
+      for (int i = tid; i < NH * K; i += LD_THREADS)
         if (h0 + i / K < p.H) p.out[(size_t)t * p.H * K + (size_t)h0 * K + i] = __float2bfloat16(0.f);
     return;
   }
   const int len = pos + 1, seq = p.seq_of_token ? p.seq_of_token[t] : t;
-  const int n_all = (len + BN - 1) / BN, per = (n_all + p.splits - 1) / p.splits;
-  const int tile0 = split * per;
-  const int n_my = max(0, min(n_all - tile0, per));
+  const int per = ((len + 63) / 64 + ns - 1) / ns * 64;       // tokens of a split: whole 64-token pieces
+  const int t0 = min(len, split * per), t1 = min(len, t0 + per);
+  const int n_my = (t1 - t0 + LD_BN - 1) / LD_BN;
+  const int nlat = (K + 63) / 64;                             // blocks that hold latent columns; the others only the rotated part
+  const int nblk = (K + 127) / 128, ngrp = nblk + (nch > nlat ? 1 : 0);
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  const uint32_t stage_bytes = nch * BN * 128;
-  const uint32_t q_s = base + p.stages * stage_bytes, p_s = q_s + nch * ROWS * 128;
+  const uint32_t q_s = base + LD_STAGES * nch * LD_CHUNK, p_s = q_s + nch * NH * 128;
   uint8_t* q_ptr = base_ptr + (q_s - base);
-  __nv_bfloat16* p_ptr = reinterpret_cast<__nv_bfloat16*>(base_ptr + (p_s - base));
-  float* s_ptr = reinterpret_cast<float*>(base_ptr + (p_s - base) + ROWS * P_LD * 2);
+  uint8_t* p_ptr = base_ptr + (p_s - base);
 
   if (tid == 0) {
     abort_flag = 0;
-    for (int s = 0; s < p.stages; ++s) { mbar_init(smem_u32(&bar_full[s]), 1); mbar_init(smem_u32(&bar_empty[s]), LD_WARPS); }
+    moved = 0;
+    for (int c = 0; c < LD_STAGES * LD_MAX_GROUPS; ++c) { mbar_init(smem_u32(&bar_full[c]), 1); mbar_init(smem_u32(&bar_empty[c]), 1); }
+    mbar_init(smem_u32(&bar_s[0]), 1); mbar_init(smem_u32(&bar_s[1]), 1); mbar_init(smem_u32(&bar_p), 128); mbar_init(smem_u32(&bar_o), 1);
     fence_mbar_init();
   }
+  if (tid >= 64 && tid - 64 < NH) { m_s[tid - 64] = -INFINITY; l_s[tid - 64] = 0.f; }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_slot), LD_TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
   __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_slot, tm_o = tmem_slot + 64;      // two S buffers of up to 32 columns, then O
 
-  float o[MT][NT][4];
-#pragma unroll
-  for (int a = 0; a < MT; ++a)
-#pragma unroll
-    for (int b = 0; b < NT; ++b) o[a][b][0] = o[a][b][1] = o[a][b][2] = o[a][b][3] = 0.f;
-
-  if (warp == LD_WARPS) {
+  if (warp == 0) {
     // ---------------------------------------------------------------- producer
     if (lane == 0) {
       tma_prefetch_desc(&tmC);
       const uint64_t pol = l2_policy_evict_first();
       const int* bt = p.block_table + (size_t)seq * p.max_blocks;
-      const int ps = p.page_size, last_page = (len - 1) / ps;
+      const int ps = p.page_size;
       bool ok = true;
-      int armed = 0;
-      for (int j = 0; j < n_my; ++j) {
-        const int s = j % p.stages;
-        if (j >= p.stages && !mbar_wait(smem_u32(&bar_empty[s]), ((j / p.stages) - 1) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
-        mbar_expect_tx(smem_u32(&bar_full[s]), stage_bytes);
-        armed = j + 1;
-        const uint32_t dst = base + s * stage_bytes;
-        for (int r = 0; r < BN; r += p.box_rows) {
-          const int tok = (tile0 + j) * BN + r;
-          // a box past the end of the sequence repeats its last page: every row of the tile then holds finite values
-          const int blk = min(tok / ps, last_page);
-          int page = bt[blk];
+      int armed = 0;      // blocks armed so far, in order
+      for (int j = 0; j < n_my && ok; ++j) {
+        const int tok0 = t0 + j * LD_BN, rows = min(t1 - tok0, LD_BN);
+        const int boxes = (rows + p.box_rows - 1) / p.box_rows;
+        int row_of[4];    // first cache row of every box of the tile
+#pragma unroll
+        for (int b = 0; b < 4; ++b) {
+          if (b >= boxes) break;
+          const int tok = tok0 + b * p.box_rows;
+          int page = bt[tok / ps];
           if (page < 0 || page >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, page); page = 0; }
-          const int row = page * ps + tok % ps;
-          for (int c = 0; c < nch; ++c) tma_load_2d(dst + c * BN * 128 + r * 128, &tmC, smem_u32(&bar_full[s]), c * 64, row, pol);
+          row_of[b] = page * ps + tok % ps;
+        }
+        const int s0 = j % LD_STAGES;
+        for (int i = 0; i < ngrp; ++i) {
+          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;           // the rotated-only blocks first: they are free first
+          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
+          const uint32_t full = smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]);
+          if (j >= LD_STAGES && !mbar_wait(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES - 1) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+          mbar_expect_tx(full, (uint32_t)(c_hi - c_lo) * boxes * p.box_rows * 128);
+          ++armed;
+          for (int c = c_lo; c < c_hi; ++c)
+            for (int b = 0; b < boxes && b < 4; ++b)
+              tma_load_2d(base + (s0 * nch + c) * LD_CHUNK + b * p.box_rows * 128, &tmC, full, c * 64, row_of[b], pol);
         }
       }
       if (!ok) {
         abort_flag = 1;
         report_status(p.status, ST_TIMEOUT_SMEM_EMPTY, 30);
         volatile int never = 0;      // copies in flight still write this CTA's shared memory: wait for them (bounded)
-        for (int j = max(0, armed - p.stages); j < armed; ++j)
-          mbar_wait(smem_u32(&bar_full[j % p.stages]), (j / p.stages) & 1, &never, LD_BUDGET_NS);
+        for (int a = max(0, armed - LD_STAGES * ngrp); a < armed; ++a) {
+          const int j = a / ngrp, i = a % ngrp, g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
+          mbar_wait(smem_u32(&bar_full[(j % LD_STAGES) * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &never, LD_BUDGET_NS);
+        }
       }
+    }
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- MMA issuer (the queries are in shared memory: barrier 2)
+    asm volatile("bar.sync 2, 160;" ::: "memory");
+    if (elect_one()) {
+      // the 128 rows of S^T's A operand are the tile's 64 tokens and 64 rows of whatever follows them: those lanes are not read
+      const uint32_t idesc_s = umma_idesc(1, 1, 128, NH);
+      const uint32_t idesc_o = umma_idesc(1, 1, 128, NH) | (1u << 15);      // A operand MN-major: latent columns are contiguous
+      bool ok = true;
+      auto issue_s = [&](int j) -> bool {
+        const int s0 = j % LD_STAGES;
+        const uint32_t d = tmem + (j & 1) * 32;
+        for (int i = 0; i < ngrp; ++i) {
+          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
+          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
+          if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) return false;
+          tc_fence_after();
+          for (int c = c_lo; c < c_hi; ++c) {
+            const uint64_t da = umma_desc_sw128(base + (s0 * nch + c) * LD_CHUNK), dq = umma_desc_sw128(q_s + c * NH * 128);
+            mma_f16(d, da, dq, idesc_s, (i > 0 || c > c_lo) ? 1u : 0u);
+#pragma unroll
+            for (int k = 1; k < 4; ++k) mma_f16(d, da + 2 * k, dq + 2 * k, idesc_s, 1u);      // 32 bytes = 2 descriptor units
+          }
+        }
+        if (ngrp > nblk) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + nblk]));
+        tc_commit(smem_u32(&bar_s[j & 1]));
+        return true;
+      };
+      const uint64_t dp = umma_desc_sw128(p_s);
+      if (n_my > 0) ok = issue_s(0);
+      for (int j = 0; j < n_my && ok; ++j) {
+        if (j + 1 < n_my && !issue_s(j + 1)) { ok = false; break; }       // runs while the softmax of tile j does
+        if (!mbar_wait(smem_u32(&bar_p), j & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+        tc_fence_after();
+        const int s0 = j % LD_STAGES, k_steps = (min(t1 - (t0 + j * LD_BN), LD_BN) + 15) / 16;      // 16-token steps with a live token
+        for (int b = 0; b < nblk; ++b) {
+          const uint64_t da = umma_desc_sw128_mn(base + (s0 * nch + 2 * b) * LD_CHUNK, LD_CHUNK);
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (k < k_steps) mma_f16(tm_o + b * NH, da + k * (16 * 128 / 16), dp + 2 * k, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+          tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + b]));
+        }
+        tc_commit(smem_u32(&bar_o));
+      }
+      if (!ok && abort_flag == 0) { abort_flag = 1; report_status(p.status, ST_TIMEOUT_SMEM_FULL, 31); }
     }
   } else {
     // ---------------------------------------------------------------- queries -> shared memory (rows past H are zero)
-    for (int i = tid; i < ROWS * nch * 8; i += LD_WARPS * 32) {
-      const int r = i / (nch * 8), c = i % (nch * 8), col = c * 8, h = h0 + r;
+    const int st = tid - 64, lane_grp = warp & 3;
+    const uint32_t lane_addr = (uint32_t)(lane_grp * 32) << 16;
+    const int kc = K / 8, rest = nch * 8 - kc;
+    for (int i = st; i < NH * kc; i += 128) {
+      const int r = i / kc, c = i % kc, h = h0 + r;
+      const __nv_bfloat16* src = p.q_abs + (size_t)t * p.H * K + (size_t)(h < p.H ? h : 0) * K + c * 8;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_s + ld_off(r, c, NH)), "l"(src), "r"(h < p.H ? 16 : 0) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll 2
+    for (int i = st; i < NH * rest; i += 128) {
+      const int r = i / rest, c = kc + i % rest, col = c * 8 - K, h = h0 + r;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (h < p.H && col < K) {
-        v = *reinterpret_cast<const uint4*>(p.q_abs + (size_t)t * p.H * K + (size_t)h * K + col);
-      } else if (h < p.H && col < K + p.rot) {
-        const __nv_bfloat16* qr = p.q + (size_t)t * p.q_ld + (size_t)h * (p.D + p.rot) + p.D + (col - K);
-        const float2* cs = reinterpret_cast<const float2*>(p.cos_sin) + (size_t)pos * (p.rot / 2) + (col - K) / 2;
+      if (h < p.H && col < p.rot) {
+        const __nv_bfloat16* qr = p.q + (size_t)t * p.q_ld + (size_t)h * (p.D + p.rot) + p.D + col;
+        const float2* cs = reinterpret_cast<const float2*>(p.cos_sin) + (size_t)pos * (p.rot / 2) + col / 2;
         __nv_bfloat162* vb = reinterpret_cast<__nv_bfloat162*>(&v);
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
@@ -183,174 +271,170 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
           vb[k] = __floats2bfloat162_rn(u * a.x - w * a.y, w * a.x + u * a.y);
         }
       }
-      *reinterpret_cast<uint4*>(q_ptr + ld_off(r, c, ROWS)) = v;
+      *reinterpret_cast<uint4*>(q_ptr + ld_off(r, c, NH)) = v;
     }
-    float m_r[2 * MT], l_r[2 * MT];      // running maximum and sum of this warp's head rows warp * 2 MT .. (all lanes alike)
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    fence_proxy_async_smem();
+    asm volatile("bar.sync 2, 160;" ::: "memory");
+
+    const int r = lane_grp * 32 + lane;             // tensor-memory lane: token of the tile (below 64), latent column of a block of O
+    float lp[NH];                                   // this thread's share of the heads' sums
 #pragma unroll
-    for (int i = 0; i < 2 * MT; ++i) { m_r[i] = -INFINITY; l_r[i] = 0.f; }
-    ld_sync();
-    const int nb = warp % NB, mg = warp / NB;      // S phase: 8-token unit, group of head tiles
-    const int mat = lane >> 3;
+    for (int i = 0; i < NH; ++i) lp[i] = 0.f;
+    bool ok = true;
     for (int j = 0; j < n_my; ++j) {
-      const int s = j % p.stages;
-      const uint32_t c_s = base + s * stage_bytes;
-      const bool landed = mbar_wait(smem_u32(&bar_full[s]), (j / p.stages) & 1, &abort_flag, LD_BUDGET_NS);
-      if (!landed) { report_status(p.status, ST_TIMEOUT_SMEM_FULL, 31); abort_flag = 1; }   // carries on: no barrier below is skipped
-      // ---- S = Q C^T ----
-      float sa[MPW][2][4];
+      if (!mbar_wait(smem_u32(&bar_s[j & 1]), (j >> 1) & 1, &abort_flag, LD_BUDGET_NS)) ok = false;     // carries on: no barrier below is skipped
+      tc_fence_after();
+      const bool live = r < LD_BN && t0 + j * LD_BN + r < t1;
+      float x[NH];
+      if (lane_grp < 2) {
+        uint32_t sv[NH];
+        ld_tmem_load<NH>(tmem + (j & 1) * 32 + lane_addr, sv);
+        tmem_ld_wait();
 #pragma unroll
-      for (int a = 0; a < MPW; ++a)
-#pragma unroll
-        for (int b = 0; b < 2; ++b) sa[a][b][0] = sa[a][b][1] = sa[a][b][2] = sa[a][b][3] = 0.f;
-      for (int k = 0; k < nch * 4; k += 2) {       // two 16-element steps at a time (columns past kv_rank + rot are zero)
-        uint32_t b[4];
-        ld_ldsm4(c_s + ld_off(nb * 8 + (lane & 7), k * 2 + mat, BN), b);
-#pragma unroll
-        for (int a = 0; a < MPW; ++a) {
-          uint32_t q0[4], q1[4];
-          const int row = (mg * MPW + a) * 16 + (lane & 15);
-          ld_ldsm4(q_s + ld_off(row, k * 2 + (lane >> 4), ROWS), q0);
-          ld_ldsm4(q_s + ld_off(row, k * 2 + 2 + (lane >> 4), ROWS), q1);
-          ld_mma(sa[a][0], q0, b[0], b[1]);
-          ld_mma(sa[a][1], q1, b[2], b[3]);
-        }
+        for (int i = 0; i < NH; ++i) x[i] = live ? __uint_as_float(sv[i]) * p.scale_log2e : -INFINITY;
       }
-#pragma unroll
-      for (int a = 0; a < MPW; ++a) {
-        const int r = (mg * MPW + a) * 16 + (lane >> 2), c = nb * 8 + (lane & 3) * 2;
-        *reinterpret_cast<float2*>(s_ptr + r * S_LD + c) = make_float2(sa[a][0][0] + sa[a][1][0], sa[a][0][1] + sa[a][1][1]);
-        *reinterpret_cast<float2*>(s_ptr + (r + 8) * S_LD + c) = make_float2(sa[a][0][2] + sa[a][1][2], sa[a][0][3] + sa[a][1][3]);
+      if (lane_grp < 2) {
+        const float wm = ld_column_reduce<NH, true>(x);
+        if (lane < NH) wred[lane_grp][lane] = wm;
       }
       ld_sync();
-      // ---- softmax of this warp's head rows ----
-      const int valid = len - (tile0 + j) * BN;     // columns of the tile that exist (at least one)
-#pragma unroll
-      for (int i = 0; i < 2 * MT; ++i) {
-        const int r = warp * 2 * MT + i;
-        float x[BN / 32], mx = -INFINITY;
-#pragma unroll
-        for (int c = 0; c < BN / 32; ++c) {
-          const int col = c * 32 + lane;
-          x[c] = col < valid ? s_ptr[r * S_LD + col] * p.scale_log2e : -INFINITY;
-          mx = fmaxf(mx, x[c]);
-        }
-#pragma unroll
-        for (int d = 16; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-        const float mn = fmaxf(m_r[i], mx), al = m_r[i] == -INFINITY ? 0.f : exp2f(m_r[i] - mn);
-        float sum = 0.f;
-#pragma unroll
-        for (int c = 0; c < BN / 32; ++c) {
-          const __nv_bfloat16 pb = __float2bfloat16(exp2f(x[c] - mn));
-          sum += __bfloat162float(pb);
-          p_ptr[r * P_LD + c * 32 + lane] = pb;
-        }
-#pragma unroll
-        for (int d = 16; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-        l_r[i] = l_r[i] * al + sum;
-        m_r[i] = mn;
-        if (lane == 0) alpha_s[r] = al;
+      if (st < NH) {
+        const float mx = fmaxf(wred[0][st], wred[1][st]), m = m_s[st];
+        // a tile holds at least one live token; the maximum only moves by more than 2^8 (the sums stay exact in the end)
+        const float mn = (m == -INFINITY || mx > m + 8.f) ? fmaxf(m, mx) : m;
+        alpha_s[st] = m == -INFINITY ? 1.f : exp2f(m - mn);
+        if (m != -INFINITY && mn != m) moved = j + 1;
+        m_s[st] = mn;
       }
       ld_sync();
-      // ---- O = alpha O + P C ----
+      if (j > 0 && !mbar_wait(smem_u32(&bar_o), (j - 1) & 1, &abort_flag, LD_BUDGET_NS)) ok = false;
+      if (moved == j + 1) {
+        tc_fence_after();
+        for (int b = 0; b < nblk; ++b) {
+          uint32_t ov[NH];
+          ld_tmem_load<NH>(tm_o + lane_addr + b * NH, ov);
+          tmem_ld_wait();
 #pragma unroll
-      for (int a = 0; a < MT; ++a) {
-        const float al0 = alpha_s[a * 16 + (lane >> 2)], al1 = alpha_s[a * 16 + (lane >> 2) + 8];
-        if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
+          for (int i = 0; i < NH; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha_s[i]);
 #pragma unroll
-          for (int b = 0; b < NT; ++b) { o[a][b][0] *= al0; o[a][b][1] *= al0; o[a][b][2] *= al1; o[a][b][3] *= al1; }
+          for (int c = 0; c < NH; c += 16) tmem_st16(tm_o + lane_addr + b * NH + c, ov + c);
+        }
+        tmem_st_wait();
+#pragma unroll
+        for (int i = 0; i < NH; ++i) lp[i] *= alpha_s[i];
+      }
+      if (lane_grp < 2) {
+        uint8_t* pr = p_ptr + (r & 7) * 2;           // P[h][token], token-contiguous rows of 128 bytes
+        const int pc = r >> 3;
+#pragma unroll
+        for (int i = 0; i < NH; i += 4) {            // the maxima first: loads do not wait behind the stores below
+          const float4 m4 = *reinterpret_cast<const float4*>(m_s + i);
+          x[i] = exp2f(x[i] - m4.x); x[i + 1] = exp2f(x[i + 1] - m4.y); x[i + 2] = exp2f(x[i + 2] - m4.z); x[i + 3] = exp2f(x[i + 3] - m4.w);
+        }
+#pragma unroll
+        for (int i = 0; i < NH; ++i) {
+          const __nv_bfloat16 pb = __float2bfloat16(x[i]);
+          lp[i] += __bfloat162float(pb);
+          *reinterpret_cast<__nv_bfloat16*>(pr + i * 128 + ((pc ^ (i & 7)) << 4)) = pb;
         }
       }
-#pragma unroll
-      for (int k = 0; k < BN / 16; ++k) {
-        uint32_t pf[MT][4];
-#pragma unroll
-        for (int a = 0; a < MT; ++a) ld_ldsm4(p_s + ((a * 16 + (lane & 15)) * P_LD + k * 16 + (lane >> 4) * 8) * 2, pf[a]);
-        const int tok = k * 16 + (mat & 1) * 8 + (lane & 7);
-        if (NT == 1) {
-          if (warp * 8 < K) {
-            uint32_t b[2];
-            ld_ldsm2_t(c_s + ld_off(tok, warp, BN), b);       // lanes 0..15 give the addresses
-#pragma unroll
-            for (int a = 0; a < MT; ++a) ld_mma(o[a][0], pf[a], b[0], b[1]);
-          }
-        } else {
-#pragma unroll
-          for (int n = 0; n < NT; n += 2) {
-            if ((warp * NT + n) * 8 < K) {
-              uint32_t b[4];
-              ld_ldsm4_t(c_s + ld_off(tok, warp * NT + n + (mat >> 1), BN), b);
-#pragma unroll
-              for (int a = 0; a < MT; ++a) {
-                ld_mma(o[a][n], pf[a], b[0], b[1]);
-                ld_mma(o[a][NT > 1 ? n + 1 : 0], pf[a], b[2], b[3]);
-              }
-            }
-          }
-        }
-      }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(&bar_empty[s]));
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(smem_u32(&bar_p));
     }
-    if (lane == 0) {
-#pragma unroll
-      for (int i = 0; i < 2 * MT; ++i) { m_s[warp * 2 * MT + i] = m_r[i]; l_s[warp * 2 * MT + i] = l_r[i]; }
-    }
-    ld_sync();       // every warp is done with the ring: its memory becomes the parking place of O, [ROWS][K] fp32
+    // ---- sums, then O from tensor memory to its parking place [NH][park_ld] (fp32, over the tile's memory) ----
+    const float ws = ld_column_reduce<NH, false>(lp);
+    if (lane < NH) wred[lane_grp][lane] = ws;
+    ld_sync();
+    if (st < NH) l_s[st] = wred[0][st] + wred[1][st];
+    if (n_my > 0 && !mbar_wait(smem_u32(&bar_o), (n_my - 1) & 1, &abort_flag, LD_BUDGET_NS)) ok = false;
+    if (!ok && abort_flag == 0) { abort_flag = 1; report_status(p.status, ST_TIMEOUT_TMEM_FULL, 32); }
+    tc_fence_after();
     float* park = reinterpret_cast<float*>(base_ptr);
+    for (int b = 0; b < nblk; ++b) {
+      uint32_t ov[NH];
+      if (n_my > 0) { ld_tmem_load<NH>(tm_o + lane_addr + b * NH, ov); tmem_ld_wait(); }
+      const int d = b * 128 + r;
+      if (d < K)
 #pragma unroll
-    for (int a = 0; a < MT; ++a)
-#pragma unroll
-      for (int b = 0; b < NT; ++b) {
-        const int col = (warp * NT + b) * 8 + (lane & 3) * 2, r = a * 16 + (lane >> 2);
-        if (col < K) {
-          *reinterpret_cast<float2*>(park + (size_t)r * K + col) = make_float2(o[a][b][0], o[a][b][1]);
-          *reinterpret_cast<float2*>(park + (size_t)(r + 8) * K + col) = make_float2(o[a][b][2], o[a][b][3]);
-        }
-      }
-  }
-  // ---- merge: CTA `split` of the cluster produces every splits-th head row of the group ----
-  const int ns = p.splits;
-  if (ns > 1) ld_cluster_sync(); else __syncthreads();
-  const uint32_t m_a = smem_u32(m_s), l_a = smem_u32(l_s);
-  const int q4 = K / 4, n_rows = (ROWS - split + ns - 1) / ns;
-  for (int i = tid; i < n_rows * q4; i += LD_THREADS) {
-    const int r = split + (i / q4) * ns, col = (i % q4) * 4;
-    if (h0 + r >= p.H) continue;
-    float M = -INFINITY;
-    for (int c = 0; c < ns; ++c) M = fmaxf(M, ns > 1 ? ld_remote_f(ld_map(m_a + r * 4, c)) : m_s[r]);
-    float L = 0.f;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int c = 0; c < ns; ++c) {
-      const float mc = ns > 1 ? ld_remote_f(ld_map(m_a + r * 4, c)) : m_s[r];
-      const float lc = ns > 1 ? ld_remote_f(ld_map(l_a + r * 4, c)) : l_s[r];
-      const float w = mc == -INFINITY ? 0.f : exp2f(mc - M);
-      const uint32_t oa = base + (uint32_t)(((size_t)r * K + col) * 4);
-      const float4 v = ns > 1 ? ld_remote_f4(ld_map(oa, c)) : *reinterpret_cast<const float4*>(base_ptr + ((size_t)r * K + col) * 4);
-      L += w * lc;
-      acc.x += w * v.x; acc.y += w * v.y; acc.z += w * v.z; acc.w += w * v.w;
+        for (int i = 0; i < NH; ++i) park[i * park_ld + d] = n_my > 0 ? __uint_as_float(ov[i]) : 0.f;
     }
-    const float inv = L > 0.f ? 1.f / L : 0.f;
-    const __nv_bfloat162 a = __floats2bfloat162_rn(acc.x * inv, acc.y * inv), b = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-    uint2 u;
-    u.x = *reinterpret_cast<const uint32_t*>(&a); u.y = *reinterpret_cast<const uint32_t*>(&b);
-    *reinterpret_cast<uint2*>(p.out + (size_t)t * p.H * K + (size_t)(h0 + r) * K + col) = u;
+  }
+  tc_fence_before();
+  // ---- merge: CTA `split` of the cluster produces every splits-th head row of the group ----
+  if (ns > 1) ld_cluster_sync(); else __syncthreads();
+  if (warp == 1) {
+    __syncwarp();
+    tc_fence_after();
+    tmem_dealloc(tmem, LD_TMEM_COLS);
+  }
+  const int q4 = K / 4, n_rows = (NH - split + ns - 1) / ns;
+  // weight of every split's O for this CTA's rows: exp2(m_c - M) / sum_c exp2(m_c - M) l_c
+  for (int i = tid; i < n_rows; i += LD_THREADS) {
+    const int r = split + i * ns;
+    float mc[LD_MAX_SPLITS], lc[LD_MAX_SPLITS];
+#pragma unroll
+    for (int c = 0; c < LD_MAX_SPLITS; ++c) {
+      mc[c] = -INFINITY; lc[c] = 0.f;
+      if (c < ns) {
+        mc[c] = ns > 1 ? ld_remote_f(ld_map(smem_u32(m_s) + r * 4, c)) : m_s[r];
+        lc[c] = ns > 1 ? ld_remote_f(ld_map(smem_u32(l_s) + r * 4, c)) : l_s[r];
+      }
+    }
+    float M = -INFINITY, L = 0.f;
+#pragma unroll
+    for (int c = 0; c < LD_MAX_SPLITS; ++c) M = fmaxf(M, mc[c]);
+#pragma unroll
+    for (int c = 0; c < LD_MAX_SPLITS; ++c) { mc[c] = mc[c] == -INFINITY ? 0.f : exp2f(mc[c] - M); L += mc[c] * lc[c]; }
+#pragma unroll
+    for (int c = 0; c < LD_MAX_SPLITS; ++c) if (c < ns) w_s[c][i] = L > 0.f ? mc[c] / L : 0.f;
+  }
+  __syncthreads();
+  constexpr int U = 4;       // items of a thread in flight together (an item: 4 columns of a row)
+  for (int i0 = tid; i0 < n_rows * q4; i0 += LD_THREADS * U) {
+    float4 acc[U];
+    uint32_t oa[U];
+    int ri[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = min(i0 + u * LD_THREADS, n_rows * q4 - 1);
+      ri[u] = i / q4;
+      oa[u] = base + (uint32_t)(((split + ri[u] * ns) * park_ld + (i % q4) * 4) * 4);
+      acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (int c = 0; c < ns; ++c) {
+      float4 v[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) v[u] = ns > 1 ? ld_remote_f4(ld_map(oa[u], c)) : *reinterpret_cast<const float4*>(base_ptr + (oa[u] - base));
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const float w = w_s[c][ri[u]];
+        acc[u].x += w * v[u].x; acc[u].y += w * v[u].y; acc[u].z += w * v[u].z; acc[u].w += w * v[u].w;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * LD_THREADS, h = h0 + split + ri[u] * ns;
+      if (i >= n_rows * q4 || h >= p.H) continue;
+      const __nv_bfloat162 a = __floats2bfloat162_rn(acc[u].x, acc[u].y), b = __floats2bfloat162_rn(acc[u].z, acc[u].w);
+      uint2 o2;
+      o2.x = *reinterpret_cast<const uint32_t*>(&a); o2.y = *reinterpret_cast<const uint32_t*>(&b);
+      *reinterpret_cast<uint2*>(p.out + (size_t)t * p.H * K + (size_t)h * K + (i % q4) * 4) = o2;
+    }
   }
   if (ns > 1) ld_cluster_sync();      // nobody leaves while another CTA reads its shared memory
 }
 
-template <int MT, int NT, int BN>
+template <int NH>
 static int latent_decode_launch(const CUtensorMap& tm, LatentDecodeParams& p, int T, int groups, cudaStream_t s) {
-  constexpr int ROWS = 16 * MT;
-  const int stage = p.nch * BN * 128;
-  const int fixed = p.nch * ROWS * 128 + ROWS * (BN + 8) * 2 + ROWS * (BN + 4) * 4 + 1024 + 64;
-  int st = (220 * 1024 - fixed) / stage;
-  if (st > LD_MAX_STAGES) st = LD_MAX_STAGES;
-  if (st < 2) return -1;
-  p.stages = st;
-  size_t smem = (size_t)st * stage + fixed;
-  const size_t park = (size_t)ROWS * p.K * 4 + 1024;
+  size_t smem = (size_t)p.nch * (LD_STAGES * LD_CHUNK + NH * 128) + NH * 128 + 1024 + 64;
+  // the operands of the last block reach past the tiles: that memory (unused results) must exist
+  const size_t reach = (size_t)(LD_STAGES * p.nch + 2) * LD_CHUNK + 1024, park = (size_t)NH * (p.K + 4) * 4 + 1024;
+  if (reach > smem) smem = reach;
   if (park > smem) smem = park;
-  auto fn = attn_latent_decode_kernel<MT, NT, BN>;
+  if (smem > 222 * 1024) return -1;
+  auto fn = attn_latent_decode_kernel<NH>;
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, 222 * 1024);
@@ -376,14 +460,14 @@ static int latent_decode_launch(const CUtensorMap& tm, LatentDecodeParams& p, in
 }  // namespace skein
 
 // Returns 0, a cudaError_t, or -1 for shapes this kernel does not take (the caller then uses the plain kernel): kv_rank and rot
-// multiples of 16, kv_rank <= 512, page sizes 16, 32 or a multiple of 64. splits 0: chosen from the row count and ctx_hint.
+// multiples of 8, kv_rank <= 512, page size 16, 32 or a multiple of 64. splits 0: chosen from the row count and ctx_hint.
 extern "C" int skein_latent_attn_decode(const void* q_abs, const void* q, long long q_ld, const float* cos_sin, int max_pos,
                                         const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
                                         const void* cache, int num_pages, int page_size, void* out, int T, int H, int D, int rot, int kv_rank,
                                         float scale, int splits, int ctx_hint, int* status, void* stream) {
   using namespace skein;
   if (T == 0) return 0;
-  if (kv_rank % 16 || rot % 16 || kv_rank < 16 || kv_rank > 512 || rot < 16 || T > 65535 || scale <= 0.f) return -1;
+  if (kv_rank % 8 || rot % 8 || kv_rank < 8 || kv_rank > 512 || rot < 8 || T > 65535 || scale <= 0.f) return -1;
   if (!(page_size == 16 || page_size == 32 || page_size % 64 == 0)) return -1;
   LatentDecodeParams p;
   p.q_abs = (const __nv_bfloat16*)q_abs; p.q = (const __nv_bfloat16*)q; p.cos_sin = cos_sin; p.positions = positions;
@@ -391,25 +475,17 @@ extern "C" int skein_latent_attn_decode(const void* q_abs, const void* q, long l
   p.scale_log2e = scale * 1.4426950408889634f;
   p.H = H; p.D = D; p.rot = rot; p.K = kv_rank; p.max_pos = max_pos; p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size;
   p.nch = (kv_rank + rot + 63) / 64;
-  const int mt = H <= 16 ? 1 : H <= 32 ? 2 : 4, bn = mt == 4 ? 32 : 64;
-  const int groups = (H + 16 * mt - 1) / (16 * mt);
-  p.box_rows = page_size < bn ? page_size : bn;
+  const int nh = H <= 16 ? 16 : 32, groups = (H + nh - 1) / nh;
+  p.box_rows = page_size < 64 ? page_size : 64;
   int dev = 0, sms = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
   if (splits <= 0) {
     splits = sms / (T * groups > 0 ? T * groups : 1);
-    if (splits > ctx_hint / bn) splits = ctx_hint / bn;
+    if (splits > ctx_hint / LD_BN) splits = ctx_hint / LD_BN;
   }
   p.splits = splits < 1 ? 1 : splits > LD_MAX_SPLITS ? LD_MAX_SPLITS : splits;
   CUtensorMap tm;
   const int rc = cached_tmap_2d(&tm, cache, (uint64_t)num_pages * page_size, (uint64_t)(kv_rank + rot), 2, p.box_rows);
   if (rc != 0) return rc;
-  const int nt = kv_rank <= 64 ? 1 : kv_rank <= 128 ? 2 : kv_rank <= 256 ? 4 : 8;
-  cudaStream_t s = (cudaStream_t)stream;
-#define LD_CASE(M, N, B) if (mt == M && nt == N) return latent_decode_launch<M, N, B>(tm, p, T, groups, s);
-  LD_CASE(1, 1, 64) LD_CASE(1, 2, 64) LD_CASE(1, 4, 64) LD_CASE(1, 8, 64)
-  LD_CASE(2, 1, 64) LD_CASE(2, 2, 64) LD_CASE(2, 4, 64) LD_CASE(2, 8, 64)
-  LD_CASE(4, 1, 32) LD_CASE(4, 2, 32) LD_CASE(4, 4, 32) LD_CASE(4, 8, 32)
-#undef LD_CASE
-  return -1;
+  return nh == 16 ? latent_decode_launch<16>(tm, p, T, groups, (cudaStream_t)stream) : latent_decode_launch<32>(tm, p, T, groups, (cudaStream_t)stream);
 }

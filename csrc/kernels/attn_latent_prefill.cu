@@ -125,28 +125,30 @@ attn_latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       }
     }
   } else if (warp == 1) {
-    // ---------------------------------------------------------------- MMA issuer
-    if (lane == 0) {
+    // ---------------------------------------------------------------- MMA issuer (one elected lane: the issue path stays uniform)
+    if (elect_one()) {
       const uint32_t idesc_s = umma_idesc(1, 1, LP_BM, LP_BN);
       const uint32_t idesc_o = umma_idesc(1, 1, LP_BM, p.vc * 64) | (1u << 16);      // B operand MN-major
       const int dsteps = (p.D + 15) / 16, rsteps = (p.rot + 15) / 16;
+      const uint64_t dq0 = umma_desc_sw128(q_s), dk0 = umma_desc_sw128(k_s), dv0 = umma_desc_sw128_mn(v_s, LP_CHUNK);
       auto issue_s = [&](int t) {
-        const uint32_t qa = q_s + t * qk_bytes, d = tmem + t * 128;
-        for (int k = 0; k < dsteps; ++k) {
-          const uint32_t off = (k >> 2) * LP_CHUNK + (k & 3) * 32;
-          mma_f16(d, umma_desc_sw128(qa + off), umma_desc_sw128(k_s + off), idesc_s, k > 0 ? 1u : 0u);
-        }
-        for (int k = 0; k < rsteps; ++k) {
-          const uint32_t off = p.dc * LP_CHUNK + k * 32;
-          mma_f16(d, umma_desc_sw128(qa + off), umma_desc_sw128(k_s + off), idesc_s, 1u);
-        }
+        const uint32_t d = tmem + t * 128;
+        // descriptors count in 16-byte units: a 16-element step is 2, a 64-element block LP_CHUNK / 16
+        const uint64_t dq = dq0 + (t ? qk_bytes / 16 : 0);
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          if (k < dsteps) mma_f16(d, dq + (k >> 2) * (LP_CHUNK / 16) + (k & 3) * 2, dk0 + (k >> 2) * (LP_CHUNK / 16) + (k & 3) * 2, idesc_s, k > 0 ? 1u : 0u);
+        const uint32_t ro = p.dc * (LP_CHUNK / 16);
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (k < rsteps) mma_f16(d, dq + ro + k * 2, dk0 + ro + k * 2, idesc_s, 1u);
         tc_commit(bar_s + 8 * t);
       };
       auto issue_o = [&](int t, int j, int hi) {
         const int k_steps = (min(hi, (j + 1) * LP_BN) - j * LP_BN + 15) / 16;       // 16-token steps with a visible key
-        for (int k = 0; k < k_steps; ++k)
-          mma_f16_ts(tmem + 256 + t * 128, tmem + t * 128 + k * 8, umma_desc_sw128_mn(v_s + k * 16 * 128, LP_CHUNK), idesc_o,
-                     (j > 0 || k > 0) ? 1u : 0u);
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          if (k < k_steps) mma_f16_ts(tmem + 256 + t * 128, tmem + t * 128 + k * 8, dv0 + k * (16 * 128 / 16), idesc_o, (j > 0 || k > 0) ? 1u : 0u);
         tc_commit(bar_o + 8 * t);
       };
       bool ok = mbar_wait(bar_q, 0, abort_flag, LP_BUDGET_NS) && mbar_wait(bar_kfull, 0, abort_flag, LP_BUDGET_NS);

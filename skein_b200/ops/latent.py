@@ -214,13 +214,10 @@ def head_linear(x, x_cols, w, gate=None):
     return out
 
 
-DECODE_TC_MAX_RANK, DECODE_MAX_HEADS = 512, 1 << 16
-
-
 def _decode_tc_ok(q_abs, q, D, rot, K, cache) -> bool:
     ps = cache.shape[1]
-    return (q_abs.dtype == torch.bfloat16 and K % 16 == 0 and rot % 16 == 0 and K <= DECODE_TC_MAX_RANK and D % 2 == 0
-            and (ps % 64 == 0 or ps in (16, 32)) and q.stride(0) % 2 == 0 and os.environ.get("SKEIN_LATENT_DECODE", "mma") == "mma"
+    return (q_abs.dtype == torch.bfloat16 and K % 8 == 0 and rot % 8 == 0 and K <= 512
+            and (ps in (16, 32) or ps % 64 == 0) and os.environ.get("SKEIN_LATENT_DECODE", "tc") == "tc"
             and hasattr(_lib.lib(), "skein_latent_attn_decode"))
 
 
