@@ -208,30 +208,9 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       const uint32_t idesc_s = umma_idesc(1, 1, 128, NH);
       const uint32_t idesc_o = umma_idesc(1, 1, 128, NH) | (1u << 15);      // A operand MN-major: latent columns are contiguous
       bool ok = true;
-      auto issue_s = [&](int j) -> bool {
-        const int s0 = j % LD_STAGES;
-        const uint32_t d = tmem + (j & 1) * 32;
-        for (int i = 0; i < ngrp; ++i) {
-          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
-          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
-          if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) return false;
-          tc_fence_after();
-          for (int c = c_lo; c < c_hi; ++c) {
-            const uint64_t da = umma_desc_sw128(base + (s0 * nch + c) * LD_CHUNK), dq = umma_desc_sw128(q_s + c * NH * 128);
-            mma_f16(d, da, dq, idesc_s, (i > 0 || c > c_lo) ? 1u : 0u);
-#pragma unroll
-            for (int k = 1; k < 4; ++k) mma_f16(d, da + 2 * k, dq + 2 * k, idesc_s, 1u);      // 32 bytes = 2 descriptor units
-          }
-        }
-        if (ngrp > nblk) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + nblk]));
-        tc_commit(smem_u32(&bar_s[j & 1]));
-        return true;
-      };
       const uint64_t dp = umma_desc_sw128(p_s);
-      if (n_my > 0) ok = issue_s(0);
-      for (int j = 0; j < n_my && ok; ++j) {
-        if (j + 1 < n_my && !issue_s(j + 1)) { ok = false; break; }       // runs while the softmax of tile j does
-        if (!mbar_wait(smem_u32(&bar_p), j & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+      int done_o = 0;                   // tiles whose O products are issued
+      auto issue_o = [&](int j) {
         tc_fence_after();
         const int s0 = j % LD_STAGES, k_steps = (min(t1 - (t0 + j * LD_BN), LD_BN) + 15) / 16;      // 16-token steps with a live token
         for (int b = 0; b < nblk; ++b) {
@@ -242,6 +221,36 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
           tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + b]));
         }
         tc_commit(smem_u32(&bar_o));
+        done_o = j + 1;
+      };
+      for (int j = 0; j < n_my && ok; ++j) {
+        const int s0 = j % LD_STAGES;
+        const uint32_t d = tmem + (j & 1) * 32;
+        for (int i = 0; i < ngrp; ++i) {
+          // the previous tile's O as soon as its P is there, between the groups of this tile's S: it frees that tile's memory
+          if (done_o < j && mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
+          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
+          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
+          if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+          tc_fence_after();
+          for (int c = c_lo; c < c_hi; ++c) {
+            const uint64_t da = umma_desc_sw128(base + (s0 * nch + c) * LD_CHUNK), dq = umma_desc_sw128(q_s + c * NH * 128);
+            mma_f16(d, da, dq, idesc_s, (i > 0 || c > c_lo) ? 1u : 0u);
+#pragma unroll
+            for (int k = 1; k < 4; ++k) mma_f16(d, da + 2 * k, dq + 2 * k, idesc_s, 1u);      // 32 bytes = 2 descriptor units
+          }
+        }
+        if (!ok) break;
+        if (ngrp > nblk) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + nblk]));
+        tc_commit(smem_u32(&bar_s[j & 1]));
+        if (done_o < j) {
+          if (!mbar_wait(smem_u32(&bar_p), (j - 1) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+          issue_o(j - 1);
+        }
+      }
+      if (ok && n_my > 0) {
+        if (mbar_wait(smem_u32(&bar_p), (n_my - 1) & 1, &abort_flag, LD_BUDGET_NS)) issue_o(n_my - 1);
+        else ok = false;
       }
       if (!ok && abort_flag == 0) { abort_flag = 1; report_status(p.status, ST_TIMEOUT_SMEM_FULL, 31); }
     }
