@@ -13,8 +13,8 @@
 //   warps 2-5   softmax, thread = token: column maxima by halving exchanges inside a warp and a step through shared memory, P to
 //               shared memory, per-thread partial sums; O is rescaled in tensor memory only when a maximum moved by more than 2^8
 //
-// At the end the CTA parks its unnormalised O with its maxima and sums in shared memory, and every CTA of the cluster merges a
-// share of the head rows from all of them through distributed shared memory. Every wait is bounded.
+// At the end the CTA parks its unnormalised O in shared memory; every CTA of the cluster produces a share of the head rows, which
+// one bulk copy per CTA pair brings to it. Every wait is bounded.
 //
 // q_abs holds the queries with the key expansion already applied; the rotated query part is rotated here, on its way to shared
 // memory.
@@ -64,17 +64,6 @@ __device__ __forceinline__ uint32_t ld_map(uint32_t addr, uint32_t rank) {   // 
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
   return r;
 }
-__device__ __forceinline__ float ld_remote_f(uint32_t addr) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
-  return v;
-}
-__device__ __forceinline__ float4 ld_remote_f4(uint32_t addr) {
-  float4 v;
-  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
-  return v;
-}
-
 // v[NH] per lane -> lane l returns the maximum (or sum) over the warp's lanes of element l mod NH, by halving exchanges
 template <int NH, bool MAX>
 __device__ __forceinline__ float ld_column_reduce(const float* v) {
@@ -108,9 +97,9 @@ template <int NH> __device__ __forceinline__ void ld_tmem_load(uint32_t addr, ui
 template <int NH>
 __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
   extern __shared__ uint8_t smem_raw[];
-  __shared__ __align__(8) uint64_t bar_full[LD_STAGES * LD_MAX_GROUPS], bar_empty[LD_STAGES * LD_MAX_GROUPS], bar_s[2], bar_p, bar_o;
+  __shared__ __align__(8) uint64_t bar_full[LD_STAGES * LD_MAX_GROUPS], bar_empty[LD_STAGES * LD_MAX_GROUPS], bar_s[2], bar_p, bar_o, bar_r;
   __shared__ __align__(16) float m_s[NH];
-  __shared__ float wred[4][NH], l_s[NH], alpha_s[NH], w_s[LD_MAX_SPLITS][NH];
+  __shared__ float wred[4][NH], l_s[NH], alpha_s[NH];
   __shared__ uint32_t tmem_slot;
   __shared__ int abort_flag, moved;
   pdl_trigger();
@@ -118,12 +107,40 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   const int split = blockIdx.x, h0 = blockIdx.y * NH, t = blockIdx.z, ns = p.splits;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int K = p.K, nch = p.nch, park_ld = K + 4;
+  const int ns_log = 31 - __clz(ns), rows_max = NH >> ns_log;       // splits: a power of two
+  if (tid == 0) {
+    abort_flag = 0;
+    moved = 0;
+    for (int c = 0; c < LD_STAGES * LD_MAX_GROUPS; ++c) { mbar_init(smem_u32(&bar_full[c]), 1); mbar_init(smem_u32(&bar_empty[c]), 1); }
+    mbar_init(smem_u32(&bar_s[0]), 1); mbar_init(smem_u32(&bar_s[1]), 1); mbar_init(smem_u32(&bar_p), 128); mbar_init(smem_u32(&bar_o), 1); mbar_init(smem_u32(&bar_r), 1);
+    fence_mbar_init();
+  }
+  if (tid >= 64 && tid - 64 < NH) { m_s[tid - 64] = -INFINITY; l_s[tid - 64] = 0.f; }
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
+  const uint32_t q_s = base + LD_STAGES * nch * LD_CHUNK, p_s = q_s + nch * NH * 128;
+  uint8_t* q_ptr = base_ptr + (q_s - base);
+  uint8_t* p_ptr = base_ptr + (p_s - base);
+  // queries -> shared memory (rows past H are zero), by everyone but the producer and ahead of the cache's tiles, behind which
+  // they would queue: the latent part by asynchronous copies, the rotated part and the padding through registers (below)
+  if (warp > 0) {
+    for (int r = warp - 1; r < NH; r += LD_THREADS / 32 - 1) {
+      const int h = h0 + r;
+      const __nv_bfloat16* src = p.q_abs + (size_t)t * p.H * K + (size_t)(h < p.H ? h : 0) * K;
+      for (int c = lane; c < K / 8; c += 32)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_s + ld_off(r, c, NH)), "l"(src + c * 8), "r"(h < p.H ? 16 : 0) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  if (p.seq_of_token == nullptr && tid == 0)     // the block table's first line, wanted as soon as the position is known
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(p.block_table + (size_t)t * p.max_blocks));
   int pos = p.positions[t];
   if (pos >= p.max_pos) { if (tid == 0) report_status(p.status, ST_BAD_INDEX, pos); pos = -1; }
   if (pos < 0) {      // padding row: the same decision in every CTA of the cluster
     if (split == 0)
       for (int i = tid; i < NH * K; i += LD_THREADS)
         if (h0 + i / K < p.H) p.out[(size_t)t * p.H * K + (size_t)h0 * K + i] = __float2bfloat16(0.f);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     return;
   }
   const int len = pos + 1, seq = p.seq_of_token ? p.seq_of_token[t] : t;
@@ -133,20 +150,6 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   const int nlat = (K + 63) / 64;                             // blocks that hold latent columns; the others only the rotated part
   const int nblk = (K + 127) / 128, ngrp = nblk + (nch > nlat ? 1 : 0);
 
-  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  const uint32_t q_s = base + LD_STAGES * nch * LD_CHUNK, p_s = q_s + nch * NH * 128;
-  uint8_t* q_ptr = base_ptr + (q_s - base);
-  uint8_t* p_ptr = base_ptr + (p_s - base);
-
-  if (tid == 0) {
-    abort_flag = 0;
-    moved = 0;
-    for (int c = 0; c < LD_STAGES * LD_MAX_GROUPS; ++c) { mbar_init(smem_u32(&bar_full[c]), 1); mbar_init(smem_u32(&bar_empty[c]), 1); }
-    mbar_init(smem_u32(&bar_s[0]), 1); mbar_init(smem_u32(&bar_s[1]), 1); mbar_init(smem_u32(&bar_p), 128); mbar_init(smem_u32(&bar_o), 1);
-    fence_mbar_init();
-  }
-  if (tid >= 64 && tid - 64 < NH) { m_s[tid - 64] = -INFINITY; l_s[tid - 64] = 0.f; }
   if (warp == 1) {
     tmem_alloc(smem_u32(&tmem_slot), LD_TMEM_COLS);
     tmem_relinquish();
@@ -155,6 +158,26 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = tmem_slot, tm_o = tmem_slot + 64;      // two S buffers of up to 32 columns, then O
+
+  if (warp > 0) {
+    const int qt = tid - 32, kc = K / 8, rest = nch * 8 - kc;
+    for (int i = qt; i < NH * rest; i += LD_THREADS - 32) {
+      const int r = i / rest, c = kc + i % rest, col = c * 8 - K, h = h0 + r;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (h < p.H && col < p.rot) {
+        const __nv_bfloat16* qr = p.q + (size_t)t * p.q_ld + (size_t)h * (p.D + p.rot) + p.D + col;
+        const float2* cs = reinterpret_cast<const float2*>(p.cos_sin) + (size_t)pos * (p.rot / 2) + col / 2;
+        __nv_bfloat162* vb = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float u = __bfloat162float(qr[2 * k]), w = __bfloat162float(qr[2 * k + 1]);
+          const float2 a = cs[k];
+          vb[k] = __floats2bfloat162_rn(u * a.x - w * a.y, w * a.x + u * a.y);
+        }
+      }
+      *reinterpret_cast<uint4*>(q_ptr + ld_off(r, c, NH)) = v;
+    }
+  }
 
   if (warp == 0) {
     // ---------------------------------------------------------------- producer
@@ -202,10 +225,11 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
     }
   } else if (warp == 1) {
     // ---------------------------------------------------------------- MMA issuer (the queries are in shared memory: barrier 2)
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    fence_proxy_async_smem();
     asm volatile("bar.sync 2, 160;" ::: "memory");
     if (elect_one()) {
-      // the 128 rows of S^T's A operand are the tile's 64 tokens and 64 rows of whatever follows them: those lanes are not read
-      const uint32_t idesc_s = umma_idesc(1, 1, 128, NH);
+      const uint32_t idesc_s = umma_idesc(1, 1, LD_BN, NH);
       const uint32_t idesc_o = umma_idesc(1, 1, 128, NH) | (1u << 15);      // A operand MN-major: latent columns are contiguous
       bool ok = true;
       const uint64_t dp = umma_desc_sw128(p_s);
@@ -255,38 +279,13 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       if (!ok && abort_flag == 0) { abort_flag = 1; report_status(p.status, ST_TIMEOUT_SMEM_FULL, 31); }
     }
   } else {
-    // ---------------------------------------------------------------- queries -> shared memory (rows past H are zero)
     const int st = tid - 64, lane_grp = warp & 3;
     const uint32_t lane_addr = (uint32_t)(lane_grp * 32) << 16;
-    const int kc = K / 8, rest = nch * 8 - kc;
-    for (int i = st; i < NH * kc; i += 128) {
-      const int r = i / kc, c = i % kc, h = h0 + r;
-      const __nv_bfloat16* src = p.q_abs + (size_t)t * p.H * K + (size_t)(h < p.H ? h : 0) * K + c * 8;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_s + ld_off(r, c, NH)), "l"(src), "r"(h < p.H ? 16 : 0) : "memory");
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-#pragma unroll 2
-    for (int i = st; i < NH * rest; i += 128) {
-      const int r = i / rest, c = kc + i % rest, col = c * 8 - K, h = h0 + r;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (h < p.H && col < p.rot) {
-        const __nv_bfloat16* qr = p.q + (size_t)t * p.q_ld + (size_t)h * (p.D + p.rot) + p.D + col;
-        const float2* cs = reinterpret_cast<const float2*>(p.cos_sin) + (size_t)pos * (p.rot / 2) + col / 2;
-        __nv_bfloat162* vb = reinterpret_cast<__nv_bfloat162*>(&v);
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const float u = __bfloat162float(qr[2 * k]), w = __bfloat162float(qr[2 * k + 1]);
-          const float2 a = cs[k];
-          vb[k] = __floats2bfloat162_rn(u * a.x - w * a.y, w * a.x + u * a.y);
-        }
-      }
-      *reinterpret_cast<uint4*>(q_ptr + ld_off(r, c, NH)) = v;
-    }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     fence_proxy_async_smem();
     asm volatile("bar.sync 2, 160;" ::: "memory");
-
-    const int r = lane_grp * 32 + lane;             // tensor-memory lane: token of the tile (below 64), latent column of a block of O
+    const int r = lane_grp * 32 + lane;             // tensor-memory lane = latent column of a block of O
+    const int tok = lane_grp * 16 + lane;           // a 64-row product keeps 16 rows in the first lanes of every warp's 32
     float lp[NH];                                   // this thread's share of the heads' sums
 #pragma unroll
     for (int i = 0; i < NH; ++i) lp[i] = 0.f;
@@ -294,22 +293,20 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
     for (int j = 0; j < n_my; ++j) {
       if (!mbar_wait(smem_u32(&bar_s[j & 1]), (j >> 1) & 1, &abort_flag, LD_BUDGET_NS)) ok = false;     // carries on: no barrier below is skipped
       tc_fence_after();
-      const bool live = r < LD_BN && t0 + j * LD_BN + r < t1;
+      const bool live = lane < 16 && t0 + j * LD_BN + tok < t1;
       float x[NH];
-      if (lane_grp < 2) {
+      {
         uint32_t sv[NH];
         ld_tmem_load<NH>(tmem + (j & 1) * 32 + lane_addr, sv);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < NH; ++i) x[i] = live ? __uint_as_float(sv[i]) * p.scale_log2e : -INFINITY;
       }
-      if (lane_grp < 2) {
-        const float wm = ld_column_reduce<NH, true>(x);
-        if (lane < NH) wred[lane_grp][lane] = wm;
-      }
+      const float wm = ld_column_reduce<NH, true>(x);
+      if (lane < NH) wred[lane_grp][lane] = wm;
       ld_sync();
       if (st < NH) {
-        const float mx = fmaxf(wred[0][st], wred[1][st]), m = m_s[st];
+        const float mx = fmaxf(fmaxf(wred[0][st], wred[1][st]), fmaxf(wred[2][st], wred[3][st])), m = m_s[st];
         // a tile holds at least one live token; the maximum only moves by more than 2^8 (the sums stay exact in the end)
         const float mn = (m == -INFINITY || mx > m + 8.f) ? fmaxf(m, mx) : m;
         alpha_s[st] = m == -INFINITY ? 1.f : exp2f(m - mn);
@@ -333,9 +330,9 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
 #pragma unroll
         for (int i = 0; i < NH; ++i) lp[i] *= alpha_s[i];
       }
-      if (lane_grp < 2) {
-        uint8_t* pr = p_ptr + (r & 7) * 2;           // P[h][token], token-contiguous rows of 128 bytes
-        const int pc = r >> 3;
+      if (lane < 16) {
+        uint8_t* pr = p_ptr + (tok & 7) * 2;         // P[h][token], token-contiguous rows of 128 bytes
+        const int pc = tok >> 3;
 #pragma unroll
         for (int i = 0; i < NH; i += 4) {            // the maxima first: loads do not wait behind the stores below
           const float4 m4 = *reinterpret_cast<const float4*>(m_s + i);
@@ -352,11 +349,11 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       tc_fence_before();
       mbar_arrive(smem_u32(&bar_p));
     }
-    // ---- sums, then O from tensor memory to its parking place [NH][park_ld] (fp32, over the tile's memory) ----
+    // ---- sums, then O from tensor memory to its parking place (fp32, over the tiles' memory): [producer][rows][park_ld] ----
     const float ws = ld_column_reduce<NH, false>(lp);
     if (lane < NH) wred[lane_grp][lane] = ws;
     ld_sync();
-    if (st < NH) l_s[st] = wred[0][st] + wred[1][st];
+    if (st < NH) l_s[st] = wred[0][st] + wred[1][st] + wred[2][st] + wred[3][st];
     if (n_my > 0 && !mbar_wait(smem_u32(&bar_o), (n_my - 1) & 1, &abort_flag, LD_BUDGET_NS)) ok = false;
     if (!ok && abort_flag == 0) { abort_flag = 1; report_status(p.status, ST_TIMEOUT_TMEM_FULL, 32); }
     tc_fence_after();
@@ -367,79 +364,86 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       const int d = b * 128 + r;
       if (d < K)
 #pragma unroll
-        for (int i = 0; i < NH; ++i) park[i * park_ld + d] = n_my > 0 ? __uint_as_float(ov[i]) : 0.f;
+        for (int i = 0; i < NH; ++i) park[((i & (ns - 1)) * rows_max + (i >> ns_log)) * park_ld + d] = n_my > 0 ? __uint_as_float(ov[i]) : 0.f;
     }
+    if (st < NH) {       // a row's maximum and sum ride in its last four floats
+      float* pm = park + ((st & (ns - 1)) * rows_max + (st >> ns_log)) * park_ld + K;
+      pm[0] = m_s[st]; pm[1] = l_s[st];
+    }
+    fence_proxy_async_smem();
   }
   tc_fence_before();
-  // ---- merge: CTA `split` of the cluster produces every splits-th head row of the group ----
+  // ---- exchange: CTA c of the cluster produces the head rows i with i mod splits = c. Behind the barrier the tiles' memory is dead
+  // in every CTA, and one bulk copy per producer brings a CTA's share of its rows there ----
+  const uint32_t block_bytes = (uint32_t)(rows_max * park_ld * 4);
+  const uint32_t recv = base + (uint32_t)(ns * rows_max * park_ld * 4);                  // [split][rows][park_ld]
   if (ns > 1) ld_cluster_sync(); else __syncthreads();
+  if (tid == 0 && ns > 1) {
+    mbar_expect_tx(smem_u32(&bar_r), (uint32_t)(ns - 1) * block_bytes);
+    for (int c = 0; c < ns; ++c)
+      if (c != split)
+        asm volatile("cp.async.bulk.shared::cluster.shared::cta.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                     ::"r"(ld_map(recv + split * block_bytes, c)), "r"(base + c * block_bytes), "r"(block_bytes), "r"(ld_map(smem_u32(&bar_r), c)) : "memory");
+  }
   if (warp == 1) {
     __syncwarp();
     tc_fence_after();
     tmem_dealloc(tmem, LD_TMEM_COLS);
   }
-  const int q4 = K / 4, n_rows = (NH - split + ns - 1) / ns;
-  // weight of every split's O for this CTA's rows: exp2(m_c - M) / sum_c exp2(m_c - M) l_c
-  for (int i = tid; i < n_rows; i += LD_THREADS) {
-    const int r = split + i * ns;
-    float mc[LD_MAX_SPLITS], lc[LD_MAX_SPLITS];
-#pragma unroll
-    for (int c = 0; c < LD_MAX_SPLITS; ++c) {
-      mc[c] = -INFINITY; lc[c] = 0.f;
-      if (c < ns) {
-        mc[c] = ns > 1 ? ld_remote_f(ld_map(smem_u32(m_s) + r * 4, c)) : m_s[r];
-        lc[c] = ns > 1 ? ld_remote_f(ld_map(smem_u32(l_s) + r * 4, c)) : l_s[r];
-      }
-    }
-    float M = -INFINITY, L = 0.f;
-#pragma unroll
-    for (int c = 0; c < LD_MAX_SPLITS; ++c) M = fmaxf(M, mc[c]);
-#pragma unroll
-    for (int c = 0; c < LD_MAX_SPLITS; ++c) { mc[c] = mc[c] == -INFINITY ? 0.f : exp2f(mc[c] - M); L += mc[c] * lc[c]; }
-#pragma unroll
-    for (int c = 0; c < LD_MAX_SPLITS; ++c) if (c < ns) w_s[c][i] = L > 0.f ? mc[c] / L : 0.f;
-  }
+  if (ns > 1 && !mbar_wait(smem_u32(&bar_r), 0, &abort_flag, LD_BUDGET_NS) && tid == 0) report_status(p.status, ST_TIMEOUT_SPLITK, split);
+  // this CTA's rows are here: it reads no other CTA's memory from now on (the wait for the others is at the end)
+  if (ns > 1) asm volatile("barrier.cluster.arrive.release;" ::: "memory");
   __syncthreads();
-  constexpr int U = 4;       // items of a thread in flight together (an item: 4 columns of a row)
-  for (int i0 = tid; i0 < n_rows * q4; i0 += LD_THREADS * U) {
-    float4 acc[U];
-    uint32_t oa[U];
-    int ri[U];
+  for (int row = warp; row < rows_max; row += LD_THREADS / 32) {
+    const int h = h0 + row * ns + split;
+    if (h >= p.H) break;
+    // lane c: split c's maximum and sum of this row, then the weight of its O: exp2(m_c - M) / sum_c exp2(m_c - M) l_c
+    auto part = [&](int c) -> const float* {
+      return reinterpret_cast<const float*>(base_ptr + ((c == split ? base + c * block_bytes : recv + c * block_bytes) - base)) + row * park_ld;
+    };
+    float mc = -INFINITY, lc = 0.f;
+    if (lane < ns) { const float* q = part(lane) + K; mc = q[0]; lc = q[1]; }
+    float M = mc;
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = min(i0 + u * LD_THREADS, n_rows * q4 - 1);
-      ri[u] = i / q4;
-      oa[u] = base + (uint32_t)(((split + ri[u] * ns) * park_ld + (i % q4) * 4) * 4);
-      acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    for (int c = 0; c < ns; ++c) {
-      float4 v[U];
+    for (int o = LD_MAX_SPLITS / 2; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    float w = mc == -INFINITY ? 0.f : exp2f(mc - M), L = w * lc;
 #pragma unroll
-      for (int u = 0; u < U; ++u) v[u] = ns > 1 ? ld_remote_f4(ld_map(oa[u], c)) : *reinterpret_cast<const float4*>(base_ptr + (oa[u] - base));
+    for (int o = LD_MAX_SPLITS / 2; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+    w = L > 0.f ? w / L : 0.f;
+    __nv_bfloat16* orow = p.out + (size_t)t * p.H * K + (size_t)h * K;
+    for (int c0 = 0; c0 < K; c0 += 512) {            // four groups of 4 columns per lane in flight
+      float4 acc[4];
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const float w = w_s[c][ri[u]];
-        acc[u].x += w * v[u].x; acc[u].y += w * v[u].y; acc[u].z += w * v[u].z; acc[u].w += w * v[u].w;
+      for (int u = 0; u < 4; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int c = 0; c < ns; ++c) {
+        const float wc = __shfl_sync(0xffffffffu, w, c);
+        const float* q = part(c) + c0 + lane * 4;
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (c0 + lane * 4 + u * 128 < K) {
+            const float4 v = *reinterpret_cast<const float4*>(q + u * 128);
+            acc[u].x += wc * v.x; acc[u].y += wc * v.y; acc[u].z += wc * v.z; acc[u].w += wc * v.w;
+          }
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int col = c0 + lane * 4 + u * 128;
+        if (col >= K) continue;
+        const __nv_bfloat162 a = __floats2bfloat162_rn(acc[u].x, acc[u].y), b = __floats2bfloat162_rn(acc[u].z, acc[u].w);
+        uint2 o2;
+        o2.x = *reinterpret_cast<const uint32_t*>(&a); o2.y = *reinterpret_cast<const uint32_t*>(&b);
+        *reinterpret_cast<uint2*>(orow + col) = o2;
       }
     }
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = i0 + u * LD_THREADS, h = h0 + split + ri[u] * ns;
-      if (i >= n_rows * q4 || h >= p.H) continue;
-      const __nv_bfloat162 a = __floats2bfloat162_rn(acc[u].x, acc[u].y), b = __floats2bfloat162_rn(acc[u].z, acc[u].w);
-      uint2 o2;
-      o2.x = *reinterpret_cast<const uint32_t*>(&a); o2.y = *reinterpret_cast<const uint32_t*>(&b);
-      *reinterpret_cast<uint2*>(p.out + (size_t)t * p.H * K + (size_t)h * K + (i % q4) * 4) = o2;
-    }
   }
-  if (ns > 1) ld_cluster_sync();      // nobody leaves while another CTA reads its shared memory
+  if (ns > 1) asm volatile("barrier.cluster.wait.acquire;" ::: "memory");      // nobody leaves while its memory is being read
 }
 
 template <int NH>
 static int latent_decode_launch(const CUtensorMap& tm, LatentDecodeParams& p, int T, int groups, cudaStream_t s) {
   size_t smem = (size_t)p.nch * (LD_STAGES * LD_CHUNK + NH * 128) + NH * 128 + 1024 + 64;
   // the operands of the last block reach past the tiles: that memory (unused results) must exist
-  const size_t reach = (size_t)(LD_STAGES * p.nch + 2) * LD_CHUNK + 1024, park = (size_t)NH * (p.K + 4) * 4 + 1024;
+  const size_t reach = (size_t)(LD_STAGES * p.nch + 2) * LD_CHUNK + 1024, park = (size_t)2 * NH * (p.K + 4) * 4 + 1024;
   if (reach > smem) smem = reach;
   if (park > smem) smem = park;
   if (smem > 222 * 1024) return -1;
@@ -492,7 +496,8 @@ extern "C" int skein_latent_attn_decode(const void* q_abs, const void* q, long l
     splits = sms / (T * groups > 0 ? T * groups : 1);
     if (splits > ctx_hint / LD_BN) splits = ctx_hint / LD_BN;
   }
-  p.splits = splits < 1 ? 1 : splits > LD_MAX_SPLITS ? LD_MAX_SPLITS : splits;
+  p.splits = 1;                       // a power of two, so that the head rows divide evenly among the cluster's CTAs
+  while (p.splits * 2 <= splits && p.splits < LD_MAX_SPLITS) p.splits *= 2;
   CUtensorMap tm;
   const int rc = cached_tmap_2d(&tm, cache, (uint64_t)num_pages * page_size, (uint64_t)(kv_rank + rot), 2, p.box_rows);
   if (rc != 0) return rc;
