@@ -34,7 +34,9 @@ constexpr int LD_STAGES = 2;
 constexpr int LD_CHUNK = LD_BN * 128;                // a 64-column block of a tile
 constexpr int LD_MAX_GROUPS = 5;                     // groups of blocks with a barrier of their own: 128 latent columns each, the rest
 constexpr int LD_MAX_SPLITS = 8;
-constexpr int LD_TMEM_COLS = 256;
+constexpr int LD_ACC = 4;                            // accumulators of a score tile: a narrow product waits for the one it adds to, so
+                                                     // neighbouring 16-element steps go to different ones and the softmax adds them up
+constexpr int LD_TMEM_COLS = 512;
 constexpr uint64_t LD_BUDGET_NS = 2000000000ull;
 
 struct LatentDecodeParams {
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = tmem_slot, tm_o = tmem_slot + 64;      // two S buffers of up to 32 columns, then O
+  const uint32_t tmem = tmem_slot, tm_o = tmem_slot + 2 * LD_ACC * 32;      // two buffers of S accumulators, then O
 
   if (warp > 0) {
     const int qt = tid - 32, kc = K / 8, rest = nch * 8 - kc;
@@ -232,24 +234,25 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       const uint32_t idesc_s = umma_idesc(1, 1, LD_BN, NH);
       const uint32_t idesc_o = umma_idesc(1, 1, 128, NH) | (1u << 15);      // A operand MN-major: latent columns are contiguous
       bool ok = true;
-      const uint64_t dp = umma_desc_sw128(p_s);
+      const uint64_t dp = umma_desc_sw128(p_s), da0 = umma_desc_sw128(base), dq0 = umma_desc_sw128(q_s);
       int done_o = 0;                   // tiles whose O products are issued
       auto issue_o = [&](int j) {
         tc_fence_after();
         const int s0 = j % LD_STAGES, k_steps = (min(t1 - (t0 + j * LD_BN), LD_BN) + 15) / 16;      // 16-token steps with a live token
-        for (int b = 0; b < nblk; ++b) {
-          const uint64_t da = umma_desc_sw128_mn(base + (s0 * nch + 2 * b) * LD_CHUNK, LD_CHUNK);
+        const uint64_t da = umma_desc_sw128_mn(base + s0 * nch * LD_CHUNK, LD_CHUNK);
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            if (k < k_steps) mma_f16(tm_o + b * NH, da + k * (16 * 128 / 16), dp + 2 * k, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
-          tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + b]));
-        }
+        for (int k = 0; k < 4; ++k)
+          if (k < k_steps)
+#pragma unroll
+            for (int b = 0; b < 4; ++b)      // neighbouring products add to different accumulators
+              if (b < nblk) mma_f16(tm_o + b * NH, da + b * (2 * LD_CHUNK / 16) + k * (16 * 128 / 16), dp + 2 * k, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+        for (int b = 0; b < nblk; ++b) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + b]));
         tc_commit(smem_u32(&bar_o));
         done_o = j + 1;
       };
       for (int j = 0; j < n_my && ok; ++j) {
         const int s0 = j % LD_STAGES;
-        const uint32_t d = tmem + (j & 1) * 32;
+        const uint32_t d = tmem + (j & 1) * LD_ACC * 32;
         for (int i = 0; i < ngrp; ++i) {
           // the previous tile's O as soon as its P is there, between the groups of this tile's S: it frees that tile's memory
           if (done_o < j && mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
@@ -257,11 +260,14 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
           const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
           if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
           tc_fence_after();
-          for (int c = c_lo; c < c_hi; ++c) {
-            const uint64_t da = umma_desc_sw128(base + (s0 * nch + c) * LD_CHUNK), dq = umma_desc_sw128(q_s + c * NH * 128);
-            mma_f16(d, da, dq, idesc_s, (i > 0 || c > c_lo) ? 1u : 0u);
+          // descriptors count in 16-byte units: a 16-element step is 2
+          const uint64_t da = da0 + (uint32_t)(s0 * nch + c_lo) * (LD_CHUNK / 16), dq = dq0 + (uint32_t)c_lo * (NH * 128 / 16);
+          const uint32_t acc = i > 0 ? 1u : 0u;
 #pragma unroll
-            for (int k = 1; k < 4; ++k) mma_f16(d, da + 2 * k, dq + 2 * k, idesc_s, 1u);      // 32 bytes = 2 descriptor units
+          for (int k = 0; k < 4; ++k) mma_f16(d + k * 32, da + 2 * k, dq + 2 * k, idesc_s, acc);
+          if (c_hi - c_lo == 2) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) mma_f16(d + k * 32, da + LD_CHUNK / 16 + 2 * k, dq + NH * 128 / 16 + 2 * k, idesc_s, 1u);
           }
         }
         if (!ok) break;
@@ -296,11 +302,20 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
       const bool live = lane < 16 && t0 + j * LD_BN + tok < t1;
       float x[NH];
       {
-        uint32_t sv[NH];
-        ld_tmem_load<NH>(tmem + (j & 1) * 32 + lane_addr, sv);
-        tmem_ld_wait();
+        uint32_t sv[2][NH];
+        const uint32_t sa = tmem + (j & 1) * LD_ACC * 32 + lane_addr;
 #pragma unroll
-        for (int i = 0; i < NH; ++i) x[i] = live ? __uint_as_float(sv[i]) * p.scale_log2e : -INFINITY;
+        for (int i = 0; i < NH; ++i) x[i] = 0.f;
+#pragma unroll
+        for (int a = 0; a < LD_ACC; a += 2) {
+          ld_tmem_load<NH>(sa + a * 32, sv[0]);
+          ld_tmem_load<NH>(sa + a * 32 + 32, sv[1]);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < NH; ++i) x[i] += __uint_as_float(sv[0][i]) + __uint_as_float(sv[1][i]);
+        }
+#pragma unroll
+        for (int i = 0; i < NH; ++i) x[i] = live ? x[i] * p.scale_log2e : -INFINITY;
       }
       const float wm = ld_column_reduce<NH, true>(x);
       if (lane < NH) wred[lane_grp][lane] = wm;
