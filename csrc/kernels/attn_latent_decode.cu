@@ -7,7 +7,7 @@
 // grid = (splits, head groups, rows); the splits of a row form a cluster. A CTA walks its tokens in tiles of 128, kept in shared
 // memory as 64-column blocks of [128 tokens][128 bytes]:
 //
-//   warp 0      TMA producer: pages of the tile, block by block; a block is refilled as soon as the products that read it are done
+//   warp 0      TMA producer: pages of the tile, two tiles in flight
 //   warp 1      MMA issuer: S^T = C Q^T (tokens x heads, accumulated over the blocks as they land), and after the softmax
 //               O^T += C^T P^T, 128 latent columns at a time (the tile is the transposed A operand, P comes from shared memory)
 //   warps 2-5   softmax, thread = token: column maxima by halving exchanges inside a warp and a step through shared memory, P to
@@ -32,7 +32,7 @@ constexpr int LD_THREADS = 192;
 constexpr int LD_BN = 64;                            // tokens per tile
 constexpr int LD_STAGES = 2;
 constexpr int LD_CHUNK = LD_BN * 128;                // a 64-column block of a tile
-constexpr int LD_MAX_GROUPS = 5;                     // groups of blocks with a barrier of their own: 128 latent columns each, the rest
+constexpr int LD_MAX_GROUPS = 2;                     // groups of blocks with a barrier of their own: 256 latent columns each
 constexpr int LD_MAX_SPLITS = 8;
 constexpr int LD_ACC = 4;                            // accumulators of a score tile: a narrow product waits for the one it adds to, so
                                                      // neighbouring 16-element steps go to different ones and the softmax adds them up
@@ -150,7 +150,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   const int t0 = min(len, split * per), t1 = min(len, t0 + per);
   const int n_my = (t1 - t0 + LD_BN - 1) / LD_BN;
   const int nlat = (K + 63) / 64;                             // blocks that hold latent columns; the others only the rotated part
-  const int nblk = (K + 127) / 128, ngrp = nblk + (nch > nlat ? 1 : 0);
+  const int nblk = (K + 127) / 128, ngrp = (nlat + 3) / 4;    // group g: blocks 4 g .. 4 g + 3, group 0 also the rotated-only blocks
 
   if (warp == 1) {
     tmem_alloc(smem_u32(&tmem_slot), LD_TMEM_COLS);
@@ -182,8 +182,8 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   }
 
   if (warp == 0) {
-    // ---------------------------------------------------------------- producer
-    if (lane == 0) {
+    // ---------------------------------------------------------------- producer (one elected lane: the issue path stays uniform)
+    if (elect_one()) {
       tma_prefetch_desc(&tmC);
       const uint64_t pol = l2_policy_evict_first();
       const int* bt = p.block_table + (size_t)seq * p.max_blocks;
@@ -203,16 +203,17 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
           row_of[b] = page * ps + tok % ps;
         }
         const int s0 = j % LD_STAGES;
-        for (int i = 0; i < ngrp; ++i) {
-          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;           // the rotated-only blocks first: they are free first
-          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
+        for (int g = 0; g < ngrp; ++g) {
+          const int c_hi = min(4 * g + 4, nlat), extra = g == 0 ? nch - nlat : 0, n = c_hi - 4 * g + extra;
           const uint32_t full = smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]);
           if (j >= LD_STAGES && !mbar_wait(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES - 1) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
-          mbar_expect_tx(full, (uint32_t)(c_hi - c_lo) * boxes * p.box_rows * 128);
+          mbar_expect_tx(full, (uint32_t)n * boxes * p.box_rows * 128);
           ++armed;
-          for (int c = c_lo; c < c_hi; ++c)
+          for (int i = 0; i < n; ++i) {
+            const int c = i < extra ? nlat + i : 4 * g + i - extra;
             for (int b = 0; b < boxes && b < 4; ++b)
               tma_load_2d(base + (s0 * nch + c) * LD_CHUNK + b * p.box_rows * 128, &tmC, full, c * 64, row_of[b], pol);
+          }
         }
       }
       if (!ok) {
@@ -220,8 +221,8 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
         report_status(p.status, ST_TIMEOUT_SMEM_EMPTY, 30);
         volatile int never = 0;      // copies in flight still write this CTA's shared memory: wait for them (bounded)
         for (int a = max(0, armed - LD_STAGES * ngrp); a < armed; ++a) {
-          const int j = a / ngrp, i = a % ngrp, g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
-          mbar_wait(smem_u32(&bar_full[(j % LD_STAGES) * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &never, LD_BUDGET_NS);
+          const int j = a / ngrp;
+          mbar_wait(smem_u32(&bar_full[(j % LD_STAGES) * LD_MAX_GROUPS + a % ngrp]), (j / LD_STAGES) & 1, &never, LD_BUDGET_NS);
         }
       }
     }
@@ -246,32 +247,35 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
 #pragma unroll
             for (int b = 0; b < 4; ++b)      // neighbouring products add to different accumulators
               if (b < nblk) mma_f16(tm_o + b * NH, da + b * (2 * LD_CHUNK / 16) + k * (16 * 128 / 16), dp + 2 * k, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
-        for (int b = 0; b < nblk; ++b) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + b]));
+        for (int g = 0; g < ngrp; ++g) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + g]));
         tc_commit(smem_u32(&bar_o));
         done_o = j + 1;
       };
       for (int j = 0; j < n_my && ok; ++j) {
         const int s0 = j % LD_STAGES;
         const uint32_t d = tmem + (j & 1) * LD_ACC * 32;
-        for (int i = 0; i < ngrp; ++i) {
+        for (int g = 0; g < ngrp; ++g) {
           // the previous tile's O as soon as its P is there, between the groups of this tile's S: it frees that tile's memory
           if (done_o < j && mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
-          const int g = ngrp > nblk ? (i == 0 ? nblk : i - 1) : i;
-          const int c_lo = g < nblk ? 2 * g : nlat, c_hi = g < nblk ? min(2 * g + 2, nlat) : nch;
           if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
           tc_fence_after();
           // descriptors count in 16-byte units: a 16-element step is 2
-          const uint64_t da = da0 + (uint32_t)(s0 * nch + c_lo) * (LD_CHUNK / 16), dq = dq0 + (uint32_t)c_lo * (NH * 128 / 16);
-          const uint32_t acc = i > 0 ? 1u : 0u;
+          const uint64_t da = da0 + (uint32_t)(s0 * nch) * (LD_CHUNK / 16);
+          if (g == 0)
+            for (int c = nlat; c < nch; ++c)
 #pragma unroll
-          for (int k = 0; k < 4; ++k) mma_f16(d + k * 32, da + 2 * k, dq + 2 * k, idesc_s, acc);
-          if (c_hi - c_lo == 2) {
+              for (int k = 0; k < 4; ++k)
+                mma_f16(d + k * 32, da + c * (LD_CHUNK / 16) + 2 * k, dq0 + c * (NH * 128 / 16) + 2 * k, idesc_s, c > nlat ? 1u : 0u);
 #pragma unroll
-            for (int k = 0; k < 4; ++k) mma_f16(d + k * 32, da + LD_CHUNK / 16 + 2 * k, dq + NH * 128 / 16 + 2 * k, idesc_s, 1u);
+          for (int i = 0; i < 4; ++i) {
+            const int c = 4 * g + i;
+            if (c >= nlat) break;
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              mma_f16(d + k * 32, da + c * (LD_CHUNK / 16) + 2 * k, dq0 + c * (NH * 128 / 16) + 2 * k, idesc_s, (c > 0 || nch > nlat) ? 1u : 0u);
           }
         }
         if (!ok) break;
-        if (ngrp > nblk) tc_commit(smem_u32(&bar_empty[s0 * LD_MAX_GROUPS + nblk]));
         tc_commit(smem_u32(&bar_s[j & 1]));
         if (done_o < j) {
           if (!mbar_wait(smem_u32(&bar_p), (j - 1) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }

@@ -94,7 +94,7 @@ attn_latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 
   if (warp == 0) {
     // ---------------------------------------------------------------- TMA producer
-    if (lane == 0) {
+    if (elect_one()) {
       const uint64_t pol_q = l2_policy_evict_first(), pol_kv = l2_policy_evict_last();
       mbar_expect_tx(bar_q, (two ? 2 : 1) * qk_bytes);
       for (int t = 0; t < (two ? 2 : 1); ++t) {
