@@ -103,7 +103,8 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
   __shared__ __align__(16) float m_s[NH];
   __shared__ float wred[4][NH], l_s[NH], alpha_s[NH];
   __shared__ uint32_t tmem_slot;
-  __shared__ int abort_flag, moved;
+  __shared__ volatile int abort_flag;
+  __shared__ int moved;
   pdl_trigger();
   pdl_wait();
   const int split = blockIdx.x, h0 = blockIdx.y * NH, t = blockIdx.z, ns = p.splits;
@@ -255,9 +256,18 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
         const int s0 = j % LD_STAGES;
         const uint32_t d = tmem + (j & 1) * LD_ACC * 32;
         for (int g = 0; g < ngrp; ++g) {
-          // the previous tile's O as soon as its P is there, between the groups of this tile's S: it frees that tile's memory
-          if (done_o < j && mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
-          if (!mbar_wait(smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]), (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
+          // while waiting for the group: the previous tile's O as soon as its P is there, which frees that tile's memory
+          const uint32_t full = smem_u32(&bar_full[s0 * LD_MAX_GROUPS + g]);
+          if (done_o < j) {
+            const uint64_t w0 = global_timer_ns();
+            bool landed = false;
+            while (!landed && done_o < j) {
+              landed = mbar_test_wait(full, (j / LD_STAGES) & 1);
+              if (mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
+              else if (!landed && (abort_flag != 0 || global_timer_ns() - w0 > LD_BUDGET_NS)) break;      // the wait below reports it
+            }
+          }
+          if (!mbar_wait(full, (j / LD_STAGES) & 1, &abort_flag, LD_BUDGET_NS)) { ok = false; break; }
           tc_fence_after();
           // descriptors count in 16-byte units: a 16-element step is 2
           const uint64_t da = da0 + (uint32_t)(s0 * nch) * (LD_CHUNK / 16);
@@ -270,6 +280,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
           for (int i = 0; i < 4; ++i) {
             const int c = 4 * g + i;
             if (c >= nlat) break;
+            if (i == 2 && done_o < j && mbar_test_wait(smem_u32(&bar_p), (j - 1) & 1)) issue_o(j - 1);
 #pragma unroll
             for (int k = 0; k < 4; ++k)
               mma_f16(d + k * 32, da + c * (LD_CHUNK / 16) + 2 * k, dq0 + c * (NH * 128 / 16) + 2 * k, idesc_s, (c > 0 || nch > nlat) ? 1u : 0u);

@@ -229,7 +229,21 @@ def op_ep_dispatch(ep, a):
     return fn, n // ep * H * 2 * 2 + n * 4, n
 
 
+def op_latent(which, tp, a):
+    """Attention over a latent cache (32 / tp heads of 128 + 64, rank 512): --tokens decoding sequences of --ctx tokens, or the
+    expanded prefill of 4 prompts of --ctx tokens."""
+    from . import design_bench
+    new, near = design_bench.size_config("dense-4k")
+    if tp > 1:
+        import dataclasses
+        new.layers = tuple(dataclasses.replace(l, mixer=dataclasses.replace(l.mixer, heads=max(1, 32 // tp))) for l in new.layers)
+    table = design_bench.decode_kernels(new, near, a.tokens, a.ctx) if which == "decode" else design_bench.prefill_kernels(new, near, 4, a.ctx)
+    return next(make for name, make, _ in table if name == "attention")()
+
+
 def build(name, a):
+    if name in ("latent_decode", "latent_prefill"):
+        return op_latent(name.split("_")[1], a.tp, a)
     tp = a.tp
     if name == "moe_gate_up":
         return op_moe("gate_up", tp, a)
@@ -263,7 +277,7 @@ def build(name, a):
 
 
 OPS = ("moe_gate_up", "moe_down", "qkv", "o_proj", "lm_head", "attn_decode", "reduce_norm", "reduce_route", "router",
-       "attn_prefill", "prefill_qkv", "argmax", "quant_fp8", "ep_dispatch")
+       "attn_prefill", "prefill_qkv", "argmax", "quant_fp8", "ep_dispatch", "latent_decode", "latent_prefill")
 
 
 def main(argv=None):
