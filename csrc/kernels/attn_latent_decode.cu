@@ -4,12 +4,13 @@
 //
 //   score[h, j] = (q_abs[h] . c_j + rot(q_rot[h]) . k_rot_j) * scale          out[h] = sum_j softmax(score)[h, j] c_j
 //
-// grid = (splits, head groups, rows); the splits of a row form a cluster. A CTA walks its tokens in tiles of 128, kept in shared
-// memory as 64-column blocks of [128 tokens][128 bytes]:
+// grid = (splits, head groups, rows); the splits of a row form a cluster. A CTA walks its tokens in tiles of 64, kept in shared
+// memory as 64-column blocks of [64 tokens][128 bytes]:
 //
 //   warp 0      TMA producer: pages of the tile, two tiles in flight
-//   warp 1      MMA issuer: S^T = C Q^T (tokens x heads, accumulated over the blocks as they land), and after the softmax
-//               O^T += C^T P^T, 128 latent columns at a time (the tile is the transposed A operand, P comes from shared memory)
+//   warp 1      MMA issuer: S^T = C Q^T (tokens x heads, as the blocks land, spread over four accumulators that the softmax adds
+//               up), and after the softmax O^T += C^T P^T, 128 latent columns at a time (the tile is the transposed A operand, P
+//               comes from shared memory); the O products of a tile are issued between those of the next tile's scores
 //   warps 2-5   softmax, thread = token: column maxima by halving exchanges inside a warp and a step through shared memory, P to
 //               shared memory, per-thread partial sums; O is rescaled in tensor memory only when a maximum moved by more than 2^8
 //

@@ -50,8 +50,9 @@ class Workspace:
         # Splits are only used while (sequences x kv heads x splits) <= SM count (pick_splits) with at most
         # MAX_GROUP query heads per kv head, which bounds B * Hq * splits; the counters are one per (sequence, kv head).
         self.attn_rows_cap = self.sm_count * self.MAX_GROUP
-        self.attn_ws = torch.empty(int(L.skein_attn_decode_workspace_floats(self.attn_rows_cap, 1, 1)),
-                                   dtype=torch.float32, device=device)
+        # A library built for one design may leave the per-head decode kernel out, and its scratch with it.
+        floats = int(L.skein_attn_decode_workspace_floats(self.attn_rows_cap, 1, 1)) if hasattr(L, "skein_attn_decode_workspace_floats") else 0
+        self.attn_ws = torch.empty(floats, dtype=torch.float32, device=device)
         self.attn_counters = torch.zeros(max(self.sm_count, 256), dtype=torch.int32, device=device)
         self.peer_state = []     # (epochs, done) tensors of live communicators, re-armed after a device error
 

@@ -74,7 +74,7 @@ def test_poly_norm(F, dtype):
     close(lat.poly_norm(tiny.to(DEV), act.to(DEV), 1e-5), rl.poly_norm(tiny, act, 1e-5), dtype)
 
 
-@pytest.mark.parametrize("E,top,groups,keep", [(12, 3, 3, 2), (8, 2, 4, 1), (64, 6, 8, 3), (256, 8, 8, 4), (5, 5, 1, 1), (40, 1, 20, 1)])
+@pytest.mark.parametrize("E,top,groups,keep", [(20, 4, 5, 3), (8, 2, 4, 1), (64, 6, 8, 3), (256, 8, 8, 4), (5, 5, 1, 1), (40, 1, 20, 1)])
 def test_grouped_selection_and_layout(E, top, groups, keep):
     T, C = 301, 64
     x, w = rnd(T, C, dtype=F32), rnd(E, C, dtype=F32)
@@ -155,7 +155,7 @@ def test_post_norm(C, dtype):
     close(act, rl.post_norm(want, None, 1.0, fg, 1e-3), dtype, 4)
 
 
-@pytest.mark.parametrize("T,C,E,top,groups,keep", [(5, 192, 12, 3, 3, 2), (64, 1024, 64, 6, 8, 3), (148, 256, 8, 2, 1, 1), (33, 4096, 40, 8, 10, 4)])
+@pytest.mark.parametrize("T,C,E,top,groups,keep", [(5, 192, 18, 4, 6, 3), (64, 1024, 64, 6, 8, 3), (148, 256, 8, 2, 1, 1), (33, 4096, 40, 8, 10, 4)])
 def test_post_norm_route_equals_separate_kernels(T, C, E, top, groups, keep):
     x, y, wg = rnd(T, C, dtype=F32).to(DEV), rnd(T, C).to(DEV), rnd(E, C, scale=C ** -0.5).to(DEV)
     g = torch.tensor([1.3], device=DEV)
@@ -175,7 +175,7 @@ def test_post_norm_route_equals_separate_kernels(T, C, E, top, groups, keep):
 
 
 # heads, dim, rot, kv_rank, page size: every head-tile and column-tile variant of the decode kernel, and sizes it does not take
-SIZES = [(4, 32, 32, 64, 64), (6, 32, 32, 128, 64), (3, 48, 16, 80, 16), (16, 128, 64, 512, 64), (32, 128, 64, 512, 64), (40, 64, 32, 256, 32),
+SIZES = [(4, 48, 32, 96, 64), (7, 64, 32, 128, 64), (3, 48, 16, 80, 16), (16, 128, 64, 512, 64), (32, 128, 64, 512, 64), (40, 64, 32, 256, 32),
          (64, 128, 64, 512, 64), (70, 16, 16, 32, 128), (20, 24, 48, 320, 64), (5, 20, 6, 36, 8), (2, 33, 10, 24, 16)]
 
 
@@ -204,7 +204,7 @@ def test_rows_over_the_cache(H, D, rot, K, ps, dtype):
 
 
 def test_rows_of_a_portion_share_their_sequence():
-    H, D, rot, K, ps = 4, 32, 32, 64, 16
+    H, D, rot, K, ps = 4, 48, 16, 96, 16
     bt = paged(2, 4, ps)
     cache = rnd(bt.numel(), ps, K + rot, scale=0.3)
     cs = ref.rope_cos_sin_table(64, rot, 1e4)
@@ -231,7 +231,7 @@ def plain_prefill(q, dense, kv, H, D, rot, V, scale, q_len, kv_len, gate):
     return out if gate is None else out * torch.sigmoid(gate.float())
 
 
-@pytest.mark.parametrize("H,D,rot,V,K,gated", [(4, 32, 32, 32, 64, True), (2, 128, 64, 128, 512, False), (3, 48, 16, 40, 80, True),
+@pytest.mark.parametrize("H,D,rot,V,K,gated", [(4, 32, 16, 48, 96, True), (2, 128, 64, 128, 512, False), (3, 48, 16, 40, 80, True),
                                                (5, 24, 32, 72, 96, False), (1, 72, 8, 8, 16, True)])
 @pytest.mark.parametrize("q_len,kv_len", [([1], [1]), ([127, 40], [127, 300]), ([128, 129, 3], [128, 129, 260]), ([300, 257], [300, 700]), ([513], [641])])
 def test_expanded_prefill(H, D, rot, V, K, gated, q_len, kv_len):
@@ -254,7 +254,7 @@ def test_expanded_prefill(H, D, rot, V, K, gated, q_len, kv_len):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("q_rank,K,rot,ps", [(0, 64, 32, 64), (56, 80, 16, 16), (33, 21, 6, 3)])
+@pytest.mark.parametrize("q_rank,K,rot,ps", [(0, 72, 24, 64), (56, 80, 16, 16), (33, 21, 6, 3)])
 def test_append_gather_rotate(q_rank, K, rot, ps, dtype):
     lens, cached = [5, 70, 1], [0, 9, 130]
     kv_len = [a + b for a, b in zip(lens, cached)]
