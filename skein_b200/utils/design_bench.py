@@ -39,7 +39,7 @@ def size_config(name: str, layers: int = 4):
         E, top, groups, keep = (64, 6, 8, 3) if name == "moe-2k" else (8, 2, 4, 2)
         mlp = RoutedFFSpec(ff, 7.0, E, top, groups, keep)
     new = mc.ModelConfig.layered("Zarorax", tuple(LayerSpec(b if i % 2 else a, mlp) for i in range(layers)), width=C, vocab=32000, taps=4,
-                                 alpha=3.0, max_pos=8192, name=f"zarorax-{name}")
+                                 alpha=2.0, max_pos=8192, name=f"zarorax-{name}")
     near = mc.ModelConfig(architecture="MixtralForCausalLM" if E else "LlamaForCausalLM", hidden_size=C, intermediate_size=ff, num_layers=layers,
                           num_heads=H, num_kv_heads=max(1, H // 4), head_dim=128, vocab_size=32000, num_experts=E, top_k=top,
                           max_position_embeddings=8192, name=("mixtral" if E else "llama") + f"-{name}")
