@@ -262,9 +262,11 @@ PYBIND11_MODULE(_skein_core, m) {
   // ---- KV manager ----
   py::class_<PageTable>(m, "PageTable")
       .def_readonly("request_id", &PageTable::request_id).def_readonly("pages", &PageTable::pages).def_readonly("num_tokens", &PageTable::num_tokens)
-      .def_readonly("prefix_hit_tokens", &PageTable::prefix_hit_tokens).def_readonly("registered_pages", &PageTable::registered_pages);
+      .def_readonly("prefix_hit_tokens", &PageTable::prefix_hit_tokens).def_readonly("registered_pages", &PageTable::registered_pages)
+      .def_readonly("slot", &PageTable::slot);
   py::class_<KvBlockManager>(m, "KvBlockManager")
-      .def(py::init<uint32_t, uint32_t, bool, uint32_t>(), py::arg("total_pages"), py::arg("page_size"), py::arg("prefix_cache") = true, py::arg("radix_max_depth") = 4096)
+      .def(py::init<uint32_t, uint32_t, bool, uint32_t, uint32_t>(), py::arg("total_pages"), py::arg("page_size"), py::arg("prefix_cache") = true, py::arg("radix_max_depth") = 4096,
+           py::arg("state_slots") = 0)
       .def_static("with_capacity", &KvBlockManager::with_capacity, py::arg("total_kv_bytes"), py::arg("bytes_per_token"), py::arg("page_size"), py::arg("prefix_cache") = true)
       .def_property_readonly("page_size", &KvBlockManager::page_size).def_property_readonly("total_pages", &KvBlockManager::total_pages)
       .def_property_readonly("available_pages", &KvBlockManager::available_pages).def_property_readonly("in_use_pages", &KvBlockManager::in_use_pages)
@@ -276,6 +278,8 @@ PYBIND11_MODULE(_skein_core, m) {
       .def("release", &KvBlockManager::release, py::arg("request_id"), py::arg("discard") = false)
       .def("mark_computed", &KvBlockManager::mark_computed).def("clear_prefix_cache", &KvBlockManager::clear_prefix_cache)
       .def("pages_for", [](const KvBlockManager& k, uint64_t id) -> py::object { auto* t = k.table(id); if (!t) return py::none(); return py::cast(t->pages); })
+      .def("slot_of", [](const KvBlockManager& k, uint64_t id) { auto* t = k.table(id); return t ? t->slot : -1; })
+      .def_property_readonly("state_slots", &KvBlockManager::state_slots).def_property_readonly("free_state_slots", &KvBlockManager::free_state_slots)
       .def("table", [](const KvBlockManager& k, uint64_t id) -> py::object { auto* t = k.table(id); if (!t) return py::none(); return py::cast(*t); });
 
   // ---- batcher ----
@@ -335,10 +339,10 @@ PYBIND11_MODULE(_skein_core, m) {
       })
       // raw host addresses of int32 arrays (the runner's pinned staging buffer): no per-row Python objects on the hot path
       .def("fill_decode_inputs", [](const ContinuousBatcher& b, const std::vector<uint64_t>& ids, uintptr_t tok, uintptr_t pos, uintptr_t lens,
-                                    uintptr_t bt, size_t max_blocks, size_t rows) {
+                                    uintptr_t bt, size_t max_blocks, size_t rows, uintptr_t slots) {
         b.fill_decode_inputs(ids, reinterpret_cast<int32_t*>(tok), reinterpret_cast<int32_t*>(pos), reinterpret_cast<int32_t*>(lens),
-                             reinterpret_cast<int32_t*>(bt), max_blocks, rows);
-      })
+                             reinterpret_cast<int32_t*>(bt), max_blocks, rows, reinterpret_cast<int32_t*>(slots));
+      }, py::arg("ids"), py::arg("tok"), py::arg("pos"), py::arg("lens"), py::arg("block_table"), py::arg("max_blocks"), py::arg("rows"), py::arg("slots") = 0)
       .def("accept_tokens", [](ContinuousBatcher& b, const std::vector<uint64_t>& ids, uintptr_t tokens, uint64_t now, int32_t eos) {
         auto o = b.accept_tokens(ids, reinterpret_cast<const int32_t*>(tokens), now, eos);
         std::vector<uint8_t> fin(o.size());

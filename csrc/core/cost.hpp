@@ -166,6 +166,14 @@ inline uint64_t layer_flops(const Layer& l, const ModelMeta& meta, const Workloa
     case LayerKind::Embedding: return b * s * l.hidden;
     case LayerKind::RmsNorm: return 5 * b * s * l.hidden;
     case LayerKind::Attention: {
+      if (l.parallel) {      // the projections, the attention over its window, read-out and update of the state
+        uint64_t w = l.shared_elems;
+        for (auto& p : l.params) w += p.numel();
+        uint64_t f = 2 * b * s * w + 6 * b * s * l.state_elems;
+        const uint64_t keys = l.window > 0 ? std::min<uint64_t>(k, l.window) : k;
+        if (l.kv_elems > 0) f += b * l.num_heads * s * keys * (2 * (l.head_dim + l.v_dim) + 3);
+        return f;
+      }
       if (l.kv_rank > 0) {   // latent attention as the decode step runs it: the projections, then scores and values over the cached rows
         uint64_t w = l.shared_elems;
         for (auto& p : l.params) w += p.numel();
@@ -200,6 +208,12 @@ inline uint64_t layer_param_elems(const Layer& l) { uint64_t n = 0; for (auto& p
 // pipeline parallelism beside it the attention is replicated across the expert-parallel ranks instead.
 inline uint64_t attention_dp_ways(const Placement& pl) { return (pl.ep > 1 && pl.tp == 1 && pl.pp == 1) ? pl.ep : 1; }
 
+// Cache and state bytes that a step of one token per sequence moves in an attention layer (or recurrence).
+inline double cache_stream_bytes(const Layer& l, Dtype kvd, const WorkloadCtx& wl) {
+  const uint64_t keys = l.window > 0 ? std::min<uint64_t>(wl.kv_len, l.window) : wl.kv_len;
+  return (double)dtype_bits(kvd) / 8.0 * (double)kv_elems_per_token(l) * (double)keys * wl.batch + 2.0 * (double)l.state_bytes * wl.batch;
+}
+
 inline double layer_stream_bytes(const Layer& l, const ModelMeta& meta, Dtype wd, Dtype kvd, const Placement& pl, const WorkloadCtx& wl) {
   const double div = (double)std::max<uint64_t>(1, compute_divisor(l.kind, pl));
   double elems = (double)(layer_param_elems(l) + l.shared_elems);
@@ -212,8 +226,7 @@ inline double layer_stream_bytes(const Layer& l, const ModelMeta& meta, Dtype wd
   }
   double bytes = (double)dtype_bits(wd) / 8.0 * elems / div;
   if (l.kind == LayerKind::Attention)
-    bytes += (double)dtype_bits(kvd) / 8.0 * (double)kv_elems_per_token(l) * (double)wl.kv_len * wl.batch /
-             (double)(pl.tp * attention_dp_ways(pl));
+    bytes += cache_stream_bytes(l, kvd, wl) / (double)(pl.tp * attention_dp_ways(pl));
   (void)meta;
   return bytes;
 }
@@ -240,8 +253,7 @@ inline double compute_time_with_dtype(const Layer& l, const ModelMeta& meta, Dty
     // (bf16 rate) for the KV cache of an attention layer
     double kv_bytes = 0;
     if (l.kind == LayerKind::Attention)
-      kv_bytes = (double)dtype_bits(kvd) / 8.0 * (double)kv_elems_per_token(l) * (double)wl.kv_len * wl.batch /
-                 (double)(pl.tp * attention_dp_ways(pl));
+      kv_bytes = cache_stream_bytes(l, kvd, wl) / (double)(pl.tp * attention_dp_ways(pl));
     const double w_bytes = layer_stream_bytes(l, meta, wd, kvd, pl, wl) - kv_bytes;
     t = std::max(t, (w_bytes / share(wd) + kv_bytes / share(Dtype::Bf16)) / (hb->second * 1e9) * 1e6);
   }
@@ -269,8 +281,10 @@ inline double block_compute_time(size_t block, const Graph& ir, Dtype wd, Dtype 
 // for its unfused graph: crates/skein_cost/src/compute.rs:232-242).
 inline uint32_t kernels_per_layer(const Layer& l) {
   switch (l.kind) {
-    case LayerKind::Attention: return l.kv_rank > 0 ? (l.q_rank > 0 ? 8 : 7) : 4;  // latent: input projection, append, (q up,) absorb, attention, values, o_proj, norm; qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
-    case LayerKind::Mlp: return 3;        // gate/up GEMM (SwiGLU epilogue), down GEMM, reduce+norm
+    case LayerKind::Attention:
+      if (l.parallel) return 3 + (l.kv_elems > 0 ? 2 : 0) + (l.state_elems > 0 ? 2 : 0) + (l.opens_pass ? 2 : 0);  // in, out, sum + norm; append, attention; step, norm
+      return l.kv_rank > 0 ? (l.q_rank > 0 ? 8 : 7) : 4;  // latent: input projection, append, (q up,) absorb, attention, values, o_proj, norm; qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
+    case LayerKind::Mlp: return l.activation == "relu2" ? 0 : 3;   // (of a parallel layer: inside the mixer's two products)        // gate/up GEMM (SwiGLU epilogue), down GEMM, reduce+norm
     case LayerKind::Moe: return 3;        // grouped gate/up (gathers its rows), grouped down, combine + norm
     case LayerKind::RmsNorm: return 0;    // fused into the reduce kernels above
     default: return 1;
@@ -349,13 +363,18 @@ inline uint64_t block_kv_elems_per_token(const Graph& ir, size_t block) {
     for (auto& l : ir.layers) if (l.kind == LayerKind::Attention && l.block_idx && *l.block_idx == block) return kv_elems_per_token(l);
   return 2ull * ir.meta.num_kv_heads * ir.meta.head_dim;
 }
+inline uint64_t block_state_bytes(const Graph& ir, size_t block) {
+  if (ir.meta.parallel)
+    for (auto& l : ir.layers) if (l.kind == LayerKind::Attention && l.block_idx && *l.block_idx == block) return l.state_bytes;
+  return 0;
+}
 inline uint64_t kv_bytes_on_device(const Plan& plan, const Graph& ir, const CostConstants& c, size_t device) {
   const Placement pl = Placement::from_plan(plan);
   if (!pl.holds(device)) return 0;
   uint64_t t = 0;
   for (size_t b = 0; b < ir.meta.num_layers; ++b) {
     const uint64_t per_seq = block_kv_elems_per_token(ir, b) * c.decode_kv_tokens;
-    if (block_to_stage(b, ir.meta.num_layers, pl.pp) == pl.stage_of(device)) t += dtype_bytes_for(plan_kv_dtype(plan, b), per_seq) * plan.batching.max_batch;
+    if (block_to_stage(b, ir.meta.num_layers, pl.pp) == pl.stage_of(device)) t += (dtype_bytes_for(plan_kv_dtype(plan, b), per_seq) + block_state_bytes(ir, b)) * plan.batching.max_batch;
   }
   return (plan.kv.kv_sharded && pl.tp > 1) ? t / pl.tp : t;
 }
@@ -374,7 +393,7 @@ inline uint64_t block_weight_bytes(size_t block, const Graph& ir, Dtype wd, cons
   return t;
 }
 inline uint64_t block_kv_bytes(const Graph& ir, size_t block, Dtype kvd, const Placement& pl, const WorkloadCtx& wl, bool kv_sharded) {
-  const uint64_t bytes = dtype_bytes_for(kvd, block_kv_elems_per_token(ir, block) * wl.kv_len * wl.batch);
+  const uint64_t bytes = dtype_bytes_for(kvd, block_kv_elems_per_token(ir, block) * wl.kv_len * wl.batch) + block_state_bytes(ir, block) * wl.batch;
   return (kv_sharded && pl.tp > 1) ? bytes / pl.tp : bytes;
 }
 inline uint64_t non_decoder_weight_bytes(const Graph& ir, const Placement& pl) {

@@ -202,6 +202,20 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
     bool moe = false;
     for (auto& l : ir.layers) if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Moe) moe = true;
     const std::string bs = "block_" + std::to_string(b);
+    if (ir.meta.parallel) {
+      // one product in, the mixers, one product out (the feed-forward runs inside the two)
+      std::vector<std::string> ops;
+      for (auto& l : ir.layers)
+        if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Attention) {
+          if (l.opens_pass) ops.push_back("loop_mix");
+          for (const char* o : {"tanh_norm", "parallel_in"}) ops.push_back(o);
+          if (l.kv_elems > 0) for (const char* o : {"window_append", "window_attention"}) ops.push_back(o);
+          if (l.state_elems > 0) for (const char* o : {"recurrence", "gated_norm"}) ops.push_back(o);
+          ops.push_back("parallel_out");
+        }
+      for (auto& o : ops) cur.ops.push_back(bs + "_" + o);
+      continue;
+    }
     if (ir.meta.layered) {
       // post-norm block of latent attention; its feed-forward, if any, is dense or routed
       bool ffn = false, q_latent = false;
@@ -232,7 +246,7 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
     if (pl.tp > 1) cut("ring_allreduce", handoff_collective_ffn_out(b), pl.tp_group(device));
   }
   if (stage == pl.pp - 1) {
-    cur.ops.insert(cur.ops.end(), {ir.meta.layered ? "final_scalar_norm" : "norm", "lm_head", "sample"});
+    cur.ops.insert(cur.ops.end(), {ir.meta.parallel ? "final_tanh_norm" : ir.meta.layered ? "final_scalar_norm" : "norm", "lm_head", "sample"});
     if (pl.tp > 1) cut("allgather", "logit_candidates", pl.tp_group(device));
     cur.outputs.push_back(handoff_logits());
   } else {

@@ -131,8 +131,154 @@ inline Graph import_layered(const Json& cfg) {
   return g;
 }
 
+// A design of parallel layers (Sikalorn): x <- x + (mixer(h) + ff(h)) with h = tanh(alpha x) w + b, and a range of layers that
+// may run several times. One block per run; the runs after a layer's first own no parameters.
+inline Graph import_parallel(const Json& cfg) {
+  ModelMeta m;
+  m.architecture = cfg.at("architecture").as_string();
+  m.layered = m.parallel = true;
+  m.hidden = cfg_usize(cfg, "width");
+  m.vocab = cfg_usize(cfg, "vocab");
+  m.max_position = cfg.has("max_position_embeddings") && !cfg.at("max_position_embeddings").is_null() ? cfg_usize(cfg, "max_position_embeddings") : 131072;
+  for (const char* k : {"norm", "layers"})
+    if (!cfg.has(k)) throw ImportError(std::string("config.json: missing `") + k + "`");
+  m.rms_norm_eps = cfg.at("norm").at("eps").as_double();
+  const auto& layers = cfg.at("layers").items();
+  if (layers.empty()) throw ImportError("config.json: `layers` is empty");
+  m.num_kv_heads = 1;
+  size_t start = 0, stop = 0, times = 1;
+  const Json* loop = cfg.find("loop");
+  const bool looped = loop && !loop->is_null();
+  if (looped) {
+    start = cfg_usize(*loop, "start"); stop = cfg_usize(*loop, "stop"); times = cfg_usize(*loop, "times");
+    if (start >= stop || stop > layers.size() || times < 1) throw ImportError("config.json: `loop` is not a range of the layers");
+  }
+  std::vector<std::pair<size_t, size_t>> runs;      // (layer, pass)
+  for (size_t i = 0; i < layers.size();) {
+    if (looped && i == start) {
+      for (size_t t = 0; t < times; ++t)
+        for (size_t j = start; j < stop; ++j) runs.push_back({j, t});
+      i = stop;
+    } else {
+      runs.push_back({i++, 0});
+    }
+  }
+  m.num_layers = runs.size();
+  Graph g;
+  size_t idx = 0;
+  const uint64_t C = m.hidden;
+  auto add = [&](LayerKind k, std::optional<size_t> block, const std::string& label) -> Layer& {
+    Layer l;
+    l.idx = idx++; l.block_idx = block; l.kind = k; l.label = label; l.hidden = m.hidden; l.eps = m.rms_norm_eps;
+    g.layers.push_back(l);
+    return g.layers.back();
+  };
+  auto elems = [](const std::vector<Param>& ps) { uint64_t n = 0; for (auto& p : ps) n += p.numel(); return n; };
+  auto norm_params = [&](const std::string& n) {
+    return std::vector<Param>{{n, {C}, Dtype::Bf16}, {n + ".b", {C}, Dtype::Bf16}, {n + ".alpha", {}, Dtype::Bf16}};
+  };
+  // parameters and cache / state sizes of the mixers
+  auto window_attention = [&](const Json& mx, const std::string& p, Layer& a, std::vector<Param>& ps) {
+    const uint64_t H = cfg_usize(mx, "heads"), K = cfg_usize(mx, "kv_heads"), D = cfg_usize(mx, "dim"), V = cfg_usize(mx, "vdim");
+    ps.push_back({p + "q", {H * D, C}, Dtype::Bf16});
+    ps.push_back({p + "k", {K * D, C}, Dtype::Bf16});
+    ps.push_back({p + "v", {K * V, C}, Dtype::Bf16});
+    ps.push_back({p + "q.norm", {H * D}, Dtype::Bf16});
+    ps.push_back({p + "k.norm", {K * D}, Dtype::Bf16});
+    ps.push_back({p + "o", {C, H * V}, Dtype::Bf16});
+    a.num_heads = H; a.num_kv_heads = K; a.head_dim = D; a.v_dim = V; a.kv_elems = K * (D + V);
+    if (const Json* w = mx.find("mask"); w && !w->is_null() && w->has("size") && !w->at("size").is_null()) a.window = cfg_usize(*w, "size");
+    a.rope_theta = mx.at("rot").at("base").as_double();
+    m.rope_theta = a.rope_theta;
+    m.num_attention_heads = std::max<size_t>(m.num_attention_heads, H);
+    m.head_dim = std::max<size_t>(m.head_dim, D);
+  };
+  auto recurrence = [&](const Json& mx, const std::string& kind, const std::string& p, Layer& a, std::vector<Param>& ps) {
+    const uint64_t H = cfg_usize(mx, "heads"), V = cfg_usize(mx, "vdim"), D = cfg_usize(mx, kind == "ssd" ? "state" : "dim");
+    const uint64_t G = kind == "ssd" ? cfg_usize(mx, "groups") : kind == "delta" ? cfg_usize(mx, "kv_heads") : H;
+    const uint64_t taps = kind == "lightning" ? 1 : cfg_usize(mx, "conv"), channels = kind == "lightning" ? 0 : H * V + 2 * G * D;
+    if (kind == "ssd") {
+      ps.push_back({p + "in", {2 * H * V + 2 * G * D + H, C}, Dtype::Bf16});
+      ps.push_back({p + "conv", {channels, taps}, Dtype::Bf16});
+      ps.push_back({p + "conv.b", {channels}, Dtype::Bf16});
+      for (const char* n : {"dt_bias", "A_log", "D"}) ps.push_back({p + n, {H}, Dtype::Bf16});
+      ps.push_back({p + "norm", {H * V}, Dtype::Bf16});
+    } else {
+      const std::vector<std::pair<std::string, uint64_t>> qkv = {{"q", G * D}, {"k", G * D}, {"v", H * V}};
+      for (auto& [n, rows] : qkv) ps.push_back({p + n, {rows, C}, Dtype::Bf16});
+      ps.push_back({p + "g", {H * V, C}, Dtype::Bf16});
+      if (kind == "delta") {
+        for (const char* n : {"b", "a"}) ps.push_back({p + n, {H, C}, Dtype::Bf16});
+        for (auto& [n, rows] : qkv) ps.push_back({p + n + ".conv", {rows, taps}, Dtype::Bf16});
+        for (const char* n : {"A_log", "dt_bias"}) ps.push_back({p + n, {H}, Dtype::Bf16});
+        ps.push_back({p + "norm", {V}, Dtype::Bf16});
+      } else {
+        ps.push_back({p + "norm", {H * V}, Dtype::Bf16});
+      }
+    }
+    ps.push_back({p + "o", {C, H * V}, Dtype::Bf16});
+    if (a.num_heads == 0) { a.num_heads = H; a.num_kv_heads = G; a.head_dim = D; a.v_dim = V; }
+    m.num_attention_heads = std::max<size_t>(m.num_attention_heads, a.num_heads);
+    m.head_dim = std::max<size_t>(m.head_dim, a.head_dim);
+    a.conv_taps = taps;
+    a.state_elems = H * D * V;
+    a.state_bytes = 4 * a.state_elems + (taps > 1 ? 2 * taps * channels : 0);
+  };
+  Layer& em = add(LayerKind::Embedding, std::nullopt, "embed_tokens");
+  em.vocab = m.vocab;
+  em.params.push_back({"embed", {m.vocab, C}, Dtype::Bf16});
+  for (size_t b = 0; b < runs.size(); ++b) {
+    const auto [i, pass] = runs[b];
+    const bool shared = pass > 0;
+    const Json& d = layers[i];
+    const std::string type = d.at("type").as_string(), p = "l" + std::to_string(i) + ".";
+    {
+      Layer& n1 = add(LayerKind::RmsNorm, b, "norm1");
+      if (!shared) n1.params = norm_params(p + "norm1");
+    }
+    std::vector<Param> ps;
+    Layer& a = add(LayerKind::Attention, b, type);
+    a.parallel = true;
+    const Json& mx = d.at("mixer");
+    if (type == "parallel") {
+      window_attention(mx.at("left"), p + "mix.left.", a, ps);
+      recurrence(mx.at("right"), "ssd", p + "mix.right.", a, ps);
+    } else if (type == "delta" || type == "lightning") {
+      recurrence(mx, type, p + "mix.", a, ps);
+    } else {
+      throw ImportError("layer " + std::to_string(i) + ": mixer type `" + type + "` is not supported");
+    }
+    if (looped && i == start) {
+      a.opens_pass = true;
+      ps.push_back({"loop.in", {C, 2 * C}, Dtype::Bf16});
+      ps.push_back({"loop.step", {times, C}, Dtype::Bf16});
+    }
+    if (shared) a.shared_elems = elems(ps); else a.params = ps;
+    if (!d.has("mlp") || d.at("mlp").is_null()) continue;
+    const Json& ml = d.at("mlp");
+    if (ml.at("kind").as_string() != "dense") throw ImportError("layer " + std::to_string(i) + ": feed-forward kind `" + ml.at("kind").as_string() + "` is not supported");
+    const uint64_t F = cfg_usize(ml, "ff");
+    ps = {{p + "mlp.up", {F, C}, Dtype::Bf16}, {p + "mlp.down", {C, F}, Dtype::Bf16}};
+    Layer& f = add(LayerKind::Mlp, b, "mlp");
+    f.intermediate = F;
+    f.activation = "relu2";
+    if (shared) f.shared_elems = elems(ps); else f.params = ps;
+    m.intermediate = std::max<size_t>(m.intermediate, F);
+  }
+  Layer& n = add(LayerKind::RmsNorm, std::nullopt, "norm");
+  n.params = norm_params("final.norm");
+  Layer& l = add(LayerKind::Lmhead, std::nullopt, "lm_head");
+  l.vocab = m.vocab;
+  l.params.push_back({"head", {m.vocab, C}, Dtype::Bf16});
+  g.meta = m;
+  return g;
+}
+
 inline Graph import_model(const Json& cfg) {
-  if (const Json* a = cfg.find("architecture"); a && !a->is_null() && a->as_string() == "Zarorax") return import_layered(cfg);
+  if (const Json* a = cfg.find("architecture"); a && !a->is_null()) {
+    if (a->as_string() == "Zarorax") return import_layered(cfg);
+    if (a->as_string() == "Sikalorn") return import_parallel(cfg);
+  }
   const Json* archs = cfg.find("architectures");
   if (!archs || !archs->is_array() || archs->size() == 0) throw ImportError("config.json: `architectures` is missing or empty");
   const std::string arch = archs->items()[0].as_string();

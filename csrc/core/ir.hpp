@@ -78,6 +78,14 @@ struct Layer {
   size_t conv_taps = 0;       // the layer's input passes a short causal convolution whose last inputs are cached
   uint64_t shared_elems = 0;  // parameter elements read from another layer's tensors (weights_of), which own no bytes here
   std::string activation = "silu";
+  // mixer of a parallel layer (x + mixer(h) + ff(h)): an attention over a window, a recurrence with a 32-bit state per sequence,
+  // or both beside each other
+  bool parallel = false;
+  size_t window = 0;           // 0: no window
+  uint64_t kv_elems = 0;       // cache elements per token
+  uint64_t state_elems = 0;    // elements of the recurrent state
+  uint64_t state_bytes = 0;    // bytes of one sequence's state, its convolution inputs included
+  bool opens_pass = false;     // the first layer of a pass of the loop
   std::string label;  // e.g. "input_layernorm", "self_attn"
   std::vector<Param> params;
 };
@@ -91,6 +99,7 @@ struct ModelMeta {
   bool tied_embeddings = false;
   bool qkv_bias = false;       // the q / k / v projections carry a bias vector each (Qwen2)
   bool layered = false;        // the configuration lists its layers one by one; runs on one device
+  bool parallel = false;       // ... and they are parallel layers
 
   Json to_json() const {
     Json j = Json::object();
@@ -103,6 +112,7 @@ struct ModelMeta {
         .set("tied_embeddings", tied_embeddings);
     if (qkv_bias) j.set("qkv_bias", true);      // written only when set: plans of models without biases keep their hash
     if (layered) j.set("layered", true);
+    if (parallel) j.set("parallel", true);
     return j;
   }
   static ModelMeta from_json(const Json& j) {
@@ -121,6 +131,7 @@ struct ModelMeta {
     m.sliding_window = opt("sliding_window"); m.tied_embeddings = j.at("tied_embeddings").as_bool();
     if (const Json* qb = j.find("qkv_bias"); qb && !qb->is_null()) m.qkv_bias = qb->as_bool();
     if (const Json* ly = j.find("layered"); ly && !ly->is_null()) m.layered = ly->as_bool();
+    if (const Json* pa = j.find("parallel"); pa && !pa->is_null()) m.parallel = pa->as_bool();
     return m;
   }
   bool is_moe() const { return num_experts && *num_experts > 0; }
@@ -128,6 +139,7 @@ struct ModelMeta {
 
 // Cache elements that one token adds in an attention layer.
 inline uint64_t kv_elems_per_token(const Layer& l) {
+  if (l.parallel) return l.kv_elems;
   return l.kv_rank > 0 ? (uint64_t)(l.kv_rank + l.rot_dim) : 2ull * l.num_kv_heads * l.head_dim;
 }
 
@@ -164,6 +176,8 @@ inline Json Graph::to_json() const {
       case LayerKind::Attention:
         k.set("num_heads", l.num_heads).set("num_kv_heads", l.num_kv_heads).set("head_dim", l.head_dim)
             .set("position", Json::object().set("kind", "rope").set("theta", l.rope_theta)).set("sliding_window", Json());
+        if (l.parallel) k.set("mixer", l.label).set("kv_elems", l.kv_elems).set("state_bytes", l.state_bytes);
+        if (l.parallel && l.window > 0) k.set("sliding_window", l.window);
         if (l.kv_rank > 0)
           k.set("latent", Json::object().set("kv_rank", l.kv_rank).set("rot_dim", l.rot_dim).set("v_dim", l.v_dim).set("q_rank", l.q_rank)
                               .set("gated", l.gated).set("conv_taps", l.conv_taps));

@@ -151,6 +151,9 @@ inline std::vector<GlobalConfig> enumerate_global_configs(const Cluster& cl, con
   // 16-token pages and head-sharded KV, the layout the runtime's kernels use.
   // A latent cache row is one small row per token: its pages start at 64 tokens.
   const std::vector<uint32_t> page_sizes = ir.meta.layered ? std::vector<uint32_t>{64u} : std::vector<uint32_t>{16u, 32u, 64u, 128u};
+  // cached pages do not bring a recurrent state back
+  bool stateful = false;
+  for (auto& l : ir.layers) stateful |= l.state_bytes > 0;
   for (uint32_t n : page_sizes) { kvs.push_back({true, n, true}); kvs.push_back({true, n, false}); }
   kvs.push_back({false, 0, true});
   kvs.push_back({false, 0, false});
@@ -167,7 +170,7 @@ inline std::vector<GlobalConfig> enumerate_global_configs(const Cluster& cl, con
           g.execution.cuda_graphs = opt.enable_cuda_graphs;
           if (opt.enable_cuda_graphs) for (uint32_t b : capture_batch_sizes(mb)) g.execution.capture_classes.push_back({b, 0});
           g.execution.spec_decode = false;
-          g.execution.prefix_cache = true;
+          g.execution.prefix_cache = !stateful;
           out.push_back(g);
         }
   return out;

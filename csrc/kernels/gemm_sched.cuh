@@ -132,6 +132,7 @@ __device__ __forceinline__ void build_sched(Sched& sched, const SkeinGemmParams&
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + __expf(-x)); }
 // activation of a gate / up pair
+__device__ __forceinline__ float relu2(float x) { x = fmaxf(x, 0.f); return x * x; }
 __device__ __forceinline__ float glu_act(const SkeinGemmParams& p, float g, float u) {
   if (p.glu == 0) return silu(g) * u;
   g = fminf(g, p.glu_limit);

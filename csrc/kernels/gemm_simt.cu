@@ -79,7 +79,8 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const SkeinGemmParams p)
       const size_t row = (size_t)(off + t), gcol = (size_t)g * p.out_group_cols + f;
       if (p.gate) y *= sigmoid_f(gs_load<T>(p.gate, row * p.gate_ld + gcol));
       const size_t idx = row * p.ldo + p.out_col0 + gcol;
-      if (p.residual) y += gs_load<T>(p.residual, idx);
+      if (f < p.relu2_cols) y = relu2(y);
+      if (p.residual) y += p.out_f32 ? gs_load<float>(p.residual, idx) : gs_load<T>(p.residual, idx);
       if (p.out_f32 || sizeof(T) == 4) ((float*)p.out)[idx] = y;
       else ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16(y);
     }

@@ -465,7 +465,8 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         if (DUAL) y = glu_act(p, g, u);
         const size_t idx = (size_t)row * p.ldo + p.out_col0 + gcol + f;
         if (p.gate) y *= sigmoid_f(__bfloat162float(((const __nv_bfloat16*)p.gate)[(size_t)row * p.gate_ld + gcol + f]));
-        if (p.out_f32) { ((float*)p.out)[idx] = y; return; }
+        if (f < p.relu2_cols) y = relu2(y);
+        if (p.out_f32) { ((float*)p.out)[idx] = p.residual ? y + ((const float*)p.residual)[idx] : y; return; }
         if (p.residual) y += __bfloat162float(((const __nv_bfloat16*)p.residual)[idx]);
         const __nv_bfloat16 yb = __float2bfloat16(y);
         ((__nv_bfloat16*)p.out)[idx] = yb;
@@ -604,7 +605,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         const int n_grp = r_hi > r_lo ? (r_hi - r_lo) / 8 : 0;
         const int n_items = n_grp * valid;
         const int gcol = un.g * p.out_group_cols;
-        const bool wide_ok = (p.ldo % 8 == 0) && ((p.out_col0 + gcol) % 8 == 0) && !p.out_f32 && (!p.gate || (p.gate_ld % 8 == 0 && gcol % 8 == 0));
+        const bool wide_ok = (p.ldo % 8 == 0) && ((p.out_col0 + gcol) % 8 == 0) && (!p.gate || (p.gate_ld % 8 == 0 && gcol % 8 == 0));
         // one item = 8 consecutive features of one token column
         auto store_item = [&](int rr, int col, const float* g8, const float* u8) {
           const int f0 = un.m * TILE_F + rr;
@@ -619,6 +620,21 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               const __nv_bfloat162* gb = reinterpret_cast<const __nv_bfloat162*>(&gv);
 #pragma unroll
               for (int j = 0; j < 4; ++j) { const float2 t = __bfloat1622float2(gb[j]); y[2 * j] *= sigmoid_f(t.x); y[2 * j + 1] *= sigmoid_f(t.y); }
+            }
+            if (p.relu2_cols > 0) {
+#pragma unroll
+              for (int j = 0; j < 8; ++j) y[j] = f0 + j < p.relu2_cols ? relu2(y[j]) : y[j];
+            }
+            if (p.out_f32) {
+              float4 a = make_float4(y[0], y[1], y[2], y[3]), b = make_float4(y[4], y[5], y[6], y[7]);
+              if (p.residual) {
+                const float4 ra = reinterpret_cast<const float4*>((const float*)p.residual + idx)[0], rb = reinterpret_cast<const float4*>((const float*)p.residual + idx)[1];
+                a.x += ra.x; a.y += ra.y; a.z += ra.z; a.w += ra.w;
+                b.x += rb.x; b.y += rb.y; b.z += rb.z; b.w += rb.w;
+              }
+              reinterpret_cast<float4*>((float*)p.out + idx)[0] = a;
+              reinterpret_cast<float4*>((float*)p.out + idx)[1] = b;
+              return;
             }
             if (p.residual) {
               const uint4 rv = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.residual + idx);
@@ -866,7 +882,7 @@ static int plan(const SkeinGemmParams* p, KernelArgs* ka, int* grid, size_t* sme
   // K need not fill its last 64-element block when the weights are plain bf16 rows: TMA reads zeros past the row's end
   if (p->K <= 0 || p->K % ((w8 || p->w_packed) ? kelem : 8) != 0) return -2;
   if (p->x_ld % 8 != 0 || (p->x_ld != 0 && p->x_ld < p->K) || p->x_group_cols % 8 != 0) return -2;
-  if (p->out_f32 && (p->mode == 2 || p->residual)) return -4;
+  if (p->out_f32 && p->mode == 2) return -4;
   const bool dual = p->mode == 1;
   if (p->n_tile < 16 || p->n_tile % 16 != 0 || p->n_tile > (dual ? 128 : 256)) return -3;
   if (p->mode < 0 || p->mode > 2) return -4;

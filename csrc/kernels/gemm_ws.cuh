@@ -14,7 +14,7 @@ typedef struct SkeinGemmParams {
   const void* W;            // [G * w_rows_per_group, K]
   const void* X;            // [x_rows, K]
   void* out;                // bf16 [*, ldo]: row = off_g + t, column = out_col0 + f
-  const void* residual;     // optional bf16, same indexing as out (added before the store)
+  const void* residual;     // optional, type and indexing of out (added before the store; may be out itself)
   const int32_t* group_off; // device [G] first X/out row of each group; null -> 0
   const int32_t* group_cnt; // device [G] rows in each group; null -> t_static for every group
   float* workspace;         // stream-K partial tiles: grid * 2 * 128 * acc_cols floats
@@ -51,9 +51,11 @@ typedef struct SkeinGemmParams {
   int32_t glu;              // dual: 0 silu(g) * u; 1 clamped unit: g = min(g, limit), u = clamp(u, +-limit),
                             //       g * sigmoid(glu_slope * g) * (u + 1)
   float glu_limit, glu_slope;
-  int32_t out_f32;          // 1: out is fp32 (residual and publish not available)
+  int32_t out_f32;          // 1: out (and residual) is fp32 (publish not available)
   int32_t gate_ld;          // elements between rows of gate
   const void* gate;         // optional bf16: the value is multiplied by sigmoid(gate[row, column without out_col0])
+  int32_t relu2_cols;       // features below this one are stored as max(y, 0)^2
+  int32_t pad;
 } SkeinGemmParams;
 
 // Returns 0 or a cudaError_t / negative argument-error code.

@@ -17,44 +17,13 @@
 #include "ptx.cuh"
 #include "launch.cuh"
 #include "route.cuh"
+#include "vec.cuh"
 #include <cuda_bf16.h>
 #include <math.h>
 
 namespace skein {
 
 constexpr int PN_MAX_TAPS = 32;
-
-template <typename T> __device__ __forceinline__ float to_f(T v);
-template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
-// V consecutive values (V = 1 or 4; with 4 the address is aligned to the access)
-template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* o) {
-  if (V == 1) { o[0] = to_f<T>(p[0]); return; }
-  if (sizeof(T) == 4) {
-    const float4 f = *reinterpret_cast<const float4*>(p);
-    o[0] = f.x; o[1] = f.y; o[2] = f.z; o[3] = f.w;
-  } else {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-    o[0] = a.x; o[1] = a.y; o[2] = b.x; o[3] = b.y;
-  }
-}
-template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float* v) {
-  if (V == 1) { p[0] = from_f<T>(v[0]); return; }
-  if (sizeof(T) == 4) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  } else {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
-    uint2 u;
-    u.x = *reinterpret_cast<const uint32_t*>(&a); u.y = *reinterpret_cast<const uint32_t*>(&b);
-    *reinterpret_cast<uint2*>(p) = u;
-  }
-}
 
 __device__ __forceinline__ float pn_block_sum(float v, float* sh) {
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

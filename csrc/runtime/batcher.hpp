@@ -161,9 +161,10 @@ class ContinuousBatcher {
   // `failed`: the request is dropped after a step that did not complete; its pages leave the prefix cache.
   // The host inputs of a decode step, written straight into the step's staging arrays (pinned memory that one
   // host-to-device copy then moves): row i feeds request ids[i] its last token at its position; id 0 and the rows
-  // from ids.size() to `rows` are padding (position -1, length 0). Block-table rows are `max_blocks` wide.
+  // from ids.size() to `rows` are padding (position -1, length 0). Block-table rows are `max_blocks` wide. `slots`
+  // (or null) receives the requests' state slots.
   void fill_decode_inputs(const std::vector<uint64_t>& ids, int32_t* tok, int32_t* pos, int32_t* lens, int32_t* block_table,
-                          size_t max_blocks, size_t rows) const {
+                          size_t max_blocks, size_t rows, int32_t* slots = nullptr) const {
     if (ids.size() > rows) throw RuntimeError("decode batch is larger than its staging buffer");
     for (size_t i = 0; i < ids.size(); ++i) {
       if (ids[i] == 0) { tok[i] = 0; pos[i] = -1; lens[i] = 0; continue; }   // a padding row inside the batch
@@ -177,6 +178,7 @@ class ContinuousBatcher {
         const PageTable* t = kv_->table(ids[i]);
         if (!t || t->pages.size() > max_blocks) throw RuntimeError("request " + std::to_string(ids[i]) + ": page table does not fit the block table");
         std::copy(t->pages.begin(), t->pages.end(), block_table + i * max_blocks);
+        if (slots) slots[i] = t->slot;
       }
     }
     for (size_t i = ids.size(); i < rows; ++i) { tok[i] = 0; pos[i] = -1; lens[i] = 0; }

@@ -14,6 +14,10 @@
 // allocator.rs:17-308, radix.rs:18-130): same admit / advance / release life cycle, refcounts,
 // generation check against stale trie entries and LRU eviction; block tables are handed to the
 // kernels instead of assembling contiguous host buffers (kv/paged_cache.rs:30-370).
+//
+// A model whose sequences carry a recurrent state has `state_slots` > 0: every admitted request holds one slot (a row of the
+// device's state pools) until it is released. A slot is not cleared in between: a sequence's first token starts from zero.
+// Cached pages do not bring a state back, so there is no prefix cache then.
 #pragma once
 #include <algorithm>
 #include <cstdint>
@@ -37,6 +41,7 @@ struct PageTable {
   uint32_t prefix_hit_tokens = 0;   // tokens served from the prefix cache at admission
   uint32_t registered_pages = 0;    // leading pages that are entered in the trie
   bool no_register = false;         // the prefix cache was cleared while this request was in flight
+  int32_t slot = -1;                // state slot (models with a recurrent state)
 };
 
 class RadixPrefixTree {
@@ -114,10 +119,13 @@ class RadixPrefixTree {
 
 class KvBlockManager {
  public:
-  KvBlockManager(uint32_t total_pages, uint32_t page_size, bool prefix_cache = true, uint32_t radix_max_depth = 4096)
-      : ps_(page_size), radix_depth_(radix_max_depth), refcount_(total_pages, 0), generation_(total_pages, 0), cached_(total_pages, 0) {
+  KvBlockManager(uint32_t total_pages, uint32_t page_size, bool prefix_cache = true, uint32_t radix_max_depth = 4096,
+                 uint32_t state_slots = 0)
+      : state_slots_(state_slots), ps_(page_size), radix_depth_(radix_max_depth), refcount_(total_pages, 0), generation_(total_pages, 0), cached_(total_pages, 0) {
     if (page_size == 0 || total_pages == 0) throw RuntimeError("KV manager needs pages and a page size");
     for (uint32_t p = 0; p < total_pages; ++p) free_.push_back((int32_t)p);
+    for (uint32_t s = 0; s < state_slots; ++s) free_slots_.push_back((int32_t)s);
+    if (prefix_cache && state_slots > 0) throw RuntimeError("a prefix of cached pages does not bring a recurrent state back: no prefix cache with state slots");
     if (prefix_cache) radix_ = std::make_unique<RadixPrefixTree>(page_size, radix_max_depth);
   }
   static KvBlockManager with_capacity(uint64_t total_kv_bytes, uint64_t bytes_per_token, uint32_t page_size, bool prefix_cache = true) {
@@ -127,6 +135,8 @@ class KvBlockManager {
   }
 
   uint32_t page_size() const { return ps_; }
+  uint32_t state_slots() const { return state_slots_; }
+  uint32_t free_state_slots() const { return (uint32_t)free_slots_.size(); }
   uint32_t total_pages() const { return (uint32_t)refcount_.size(); }
   uint32_t available_pages() const { return (uint32_t)(free_.size() + lru_.size()); }
   uint32_t in_use_pages() const { return total_pages() - available_pages(); }
@@ -142,6 +152,7 @@ class KvBlockManager {
     return (uint32_t)(radix_->lookup(prompt, generation_, (prompt.size() - 1) / ps_).size() * ps_);
   }
   bool can_admit(const std::vector<int32_t>& prompt, uint32_t reserve_tokens = 0) {
+    if (state_slots_ > 0 && free_slots_.empty()) return false;
     const uint32_t hit = try_prefix_reuse(prompt);
     const uint32_t need = pages_needed((uint32_t)prompt.size() + reserve_tokens) - hit / ps_;
     // matched pages sitting in the LRU list stop being "available" once we reference them
@@ -151,6 +162,7 @@ class KvBlockManager {
   PageTable admit(uint64_t request_id, const std::vector<int32_t>& prompt) {
     if (tables_.count(request_id)) throw RuntimeError("request " + std::to_string(request_id) + " is already admitted");
     if (prompt.empty()) throw RuntimeError("empty prompt");
+    if (state_slots_ > 0 && free_slots_.empty()) throw RuntimeError("all " + std::to_string(state_slots_) + " state slots are taken");
     std::vector<int32_t> matched;
     if (radix_) matched = radix_->lookup(prompt, generation_, (prompt.size() - 1) / ps_);
     const uint32_t need = pages_needed((uint32_t)prompt.size()) - (uint32_t)matched.size();
@@ -169,6 +181,7 @@ class KvBlockManager {
     pt.prefix_hit_tokens = (uint32_t)matched.size() * ps_;
     hit_tokens_total_ += pt.prefix_hit_tokens;
     pt.registered_pages = (uint32_t)matched.size();   // the matched pages already sit in the trie
+    if (state_slots_ > 0) { pt.slot = free_slots_.front(); free_slots_.pop_front(); }
     tables_[request_id] = pt;
     return pt;
   }
@@ -224,6 +237,7 @@ class KvBlockManager {
       if (discard && refcount_[p] == 1) { ++generation_[p]; cached_[p] = 0; }
       unref(p);
     }
+    if (it->second.slot >= 0) free_slots_.push_back(it->second.slot);
     tables_.erase(it);
   }
   const PageTable* table(uint64_t request_id) const {
@@ -233,6 +247,8 @@ class KvBlockManager {
   size_t num_requests() const { return tables_.size(); }
 
  private:
+  uint32_t state_slots_ = 0;
+  std::deque<int32_t> free_slots_;
   uint32_t ps_, radix_depth_;
   std::vector<uint32_t> refcount_;
   std::vector<uint64_t> generation_;

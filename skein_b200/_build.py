@@ -32,7 +32,11 @@ CORE_LIB_STEM = "_skein_core"
 # Kernel sources of architectures that need only some of them (the others take the whole library).
 ARCH_SOURCES = {
     "Zarorax": ("attn_latent_decode", "attn_latent_prefill", "gemm_simt", "gemm_ws", "latent", "postnorm", "rope_kv", "router", "sample"),
+    "Sikalorn": ("attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_ws", "parallel_layer", "postnorm", "recurrent", "rope_kv",
+                 "sample"),
 }
+# Sources compiled without fast-math: their exponentials, logarithms and tanh keep the accuracy of 32-bit.
+EXACT_SOURCES = ("attn_window", "parallel_layer", "recurrent")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -96,7 +100,8 @@ def build_kernels(force: bool = False, verbose: bool = False, only=None) -> Path
         o = OBJ / (s.stem + ".o")
         objs.append(o)
         if force or _newer(s, o, headers):
-            cmd = [nvcc, *NVCC_FLAGS, "-I", str(kdir), "-c", str(s), "-o", str(o)]
+            flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or s.stem not in EXACT_SOURCES]
+            cmd = [nvcc, *flags, "-I", str(kdir), "-c", str(s), "-o", str(o)]
             if verbose:
                 cmd.insert(1, "-Xptxas")
                 cmd.insert(2, "-v")

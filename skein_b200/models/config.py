@@ -12,7 +12,8 @@ import json
 from dataclasses import asdict, dataclass
 from pathlib import Path
 
-from .layered import LAYERED_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers
+from .layered import LAYERED_ARCHS, PARALLEL_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers, unroll_loop
+from .parallel_layers import attention_of, parse_loop, recurrence_of
 
 MOE_ARCHS = {"MixtralForCausalLM"}
 DENSE_ARCHS = {"LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM"}
@@ -46,6 +47,7 @@ class ModelConfig:
     layers: tuple = ()
     conv_taps: int = 0            # taps of the input convolution
     post_alpha: float = 1.0       # weight of the residual inside the post-norms
+    loop: tuple | None = None     # (start, stop, times): checkpoint layers that run several times (`layers` lists every run)
 
     @property
     def is_moe(self) -> bool:
@@ -54,6 +56,22 @@ class ModelConfig:
     @property
     def is_layered(self) -> bool:
         return bool(self.layers)
+
+    @property
+    def is_parallel(self) -> bool:
+        """Layers are x + mixer(h) + ff(h) (models/parallel_layers.py)."""
+        return self.architecture in PARALLEL_ARCHS
+
+    @property
+    def has_state(self) -> bool:
+        """Sequences carry a recurrent state beside their cache pages: each needs a state slot, and a prefix of cached pages
+        alone does not bring a sequence back."""
+        return self.is_parallel and any(recurrence_of(l.mixer) is not None for l in self.layers)
+
+    def state_bytes_per_slot(self, elem: int = 2) -> int:
+        if not self.has_state:
+            return 0
+        return sum(recurrence_of(l.mixer).state_bytes(elem) for l in self.layers if recurrence_of(l.mixer) is not None)
 
     @property
     def default_page_size(self) -> int:
@@ -66,7 +84,7 @@ class ModelConfig:
         if not self.is_layered:
             return 2 * (self.num_kv_heads // tp) * page_size * self.head_dim * elem * len(blocks)
         tail = self.conv_tail_rows(page_size) * self.hidden_size
-        return sum((self.layers[b].mixer.cache_width * page_size + tail) * elem for b in blocks)
+        return sum((self.layers[b].mixer.cache_elems_per_token * page_size + tail) * elem for b in blocks)
 
     def conv_tail_rows(self, page_size: int) -> int:
         """Rows per cache page that keep the input convolution's last inputs. One more than the taps that look back, so that a
@@ -79,7 +97,7 @@ class ModelConfig:
 
     def validate(self) -> None:
         if self.is_layered:
-            if self.conv_taps < 1:
+            if self.conv_taps < 1 and not self.is_parallel:
                 raise ImportError_("canon.taps must be at least 1")
             return
         if self.num_heads % self.num_kv_heads != 0:
@@ -171,9 +189,13 @@ class ModelConfig:
     @staticmethod
     def _from_layered_dict(d: dict, name: str | None) -> "ModelConfig":
         try:
-            layers = parse_layers(d["architecture"], d["layers"])
-            cfg = ModelConfig.layered(d["architecture"], layers, width=int(d["width"]), vocab=int(d["vocab"]), taps=int(d["canon"]["taps"]),
-                                      alpha=float(d["postln_alpha"]), eps=float(d["norm"]["eps"]), name=name or d["architecture"].lower())
+            arch = d["architecture"]
+            layers = parse_layers(arch, d["layers"], d.get("loop"))
+            only = {} if arch in PARALLEL_ARCHS else {"taps": int(d["canon"]["taps"]), "alpha": float(d["postln_alpha"])}
+            if arch in PARALLEL_ARCHS:
+                only["loop"] = parse_loop(d.get("loop"), len(d["layers"]))
+            cfg = ModelConfig.layered(arch, layers, width=int(d["width"]), vocab=int(d["vocab"]), eps=float(d["norm"]["eps"]),
+                                      name=name or arch.lower(), **only)
         except KeyError as e:
             raise ImportError_(f"config.json: missing {e.args[0]!r}") from e
         except SpecError as e:
@@ -186,21 +208,29 @@ class ModelConfig:
         return cfg
 
     @staticmethod
-    def layered(arch: str, layers, width: int, vocab: int, taps: int, alpha: float, eps: float = 1e-5, max_pos: int = 131072,
-                name: str = "layered") -> "ModelConfig":
+    def layered(arch: str, layers, width: int, vocab: int, taps: int = 0, alpha: float = 1.0, eps: float = 1e-5, max_pos: int = 131072,
+                name: str = "layered", loop: tuple | None = None) -> "ModelConfig":
         """Configuration of a design that lists its layers. The single-valued fields describe its largest layer (planning and
-        display only; the layer specifications decide what runs). The design sets no position limit: max_pos is the engine's."""
+        display only; the layer specifications decide what runs). The design sets no position limit: max_pos is the engine's.
+        `loop` (start, stop, times): `layers` are its runs (models/layered.py: unroll_loop)."""
         ff = [l.mlp.ff * (l.mlp.experts if isinstance(l.mlp, RoutedFFSpec) else 1) for l in layers if l.mlp is not None]
+        bases = [b for b in (getattr(attention_of(l.mixer) or l.mixer, "rope_base", None) for l in layers) if b is not None]
         cfg = ModelConfig(architecture=arch, hidden_size=width, intermediate_size=max(ff, default=0), num_layers=len(layers),
                           num_heads=max(l.mixer.heads for l in layers) if layers else 0, num_kv_heads=1,
-                          head_dim=max(l.mixer.dim + l.mixer.rot_dim for l in layers) if layers else 0, vocab_size=vocab,
-                          rms_norm_eps=eps, rope_theta=layers[0].mixer.rope_base if layers else 1e4, num_experts=0, top_k=0,
-                          max_position_embeddings=max_pos, name=name, layers=tuple(layers), conv_taps=taps, post_alpha=alpha)
+                          head_dim=max(l.mixer.head_size for l in layers) if layers else 0, vocab_size=vocab,
+                          rms_norm_eps=eps, rope_theta=bases[0] if bases else 1e4, num_experts=0, top_k=0,
+                          max_position_embeddings=max_pos, name=name, layers=tuple(layers), conv_taps=taps, post_alpha=alpha, loop=loop)
         cfg.validate()
         return cfg
 
     def to_hf_dict(self) -> dict:
         """The config.json fields that describe this model (what the planner and the lowering read)."""
+        if self.is_parallel:
+            d = {"architecture": self.architecture, "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps},
+                 "layers": layers_to_list(self.layers), "max_position_embeddings": self.max_position_embeddings}
+            if self.loop is not None:
+                d["loop"] = dict(zip(("start", "stop", "times"), self.loop))
+            return d
         if self.is_layered:
             return {"architecture": self.architecture, "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps},
                     "canon": {"taps": self.conv_taps}, "postln_alpha": self.post_alpha, "layers": layers_to_list(self.layers),
@@ -259,6 +289,18 @@ def tiny_zarorax(width=192, vocab=384, taps=4, alpha=2.5, eps=1e-5) -> ModelConf
     moe = RoutedFFSpec(ff=72, limit=1.5, experts=8, top=2, groups=4, keep=2)
     return ModelConfig.layered("Zarorax", (LayerSpec(a, DenseFFSpec(160)), LayerSpec(b, moe), LayerSpec(b, moe, weights_of=1), LayerSpec(a, None)),
                                width=width, vocab=vocab, taps=taps, alpha=alpha, eps=eps, max_pos=4096, name="tiny-zarorax")
+
+
+def tiny_sikalorn(width=96, vocab=384, eps=1e-5) -> ModelConfig:
+    """A small model of the Sikalorn design for tests: every mixer, a layer without feed-forward, three passes over two layers."""
+    from .parallel_layers import MixerPairSpec, RecurrentSpec, WindowAttnSpec
+    pair = MixerPairSpec(WindowAttnSpec(heads=4, kv_heads=2, dim=24, vdim=40, scale=0.17, rot_dims=16, rope_base=5e4, rope_factor=2.0, window=21),
+                         RecurrentSpec("ssd", heads=6, groups=3, dim=20, vdim=16, taps=4, norm_groups=2), 0.8, 0.7)
+    delta = RecurrentSpec("delta", heads=4, groups=2, dim=24, vdim=32, taps=4)
+    light = RecurrentSpec("lightning", heads=3, groups=3, dim=16, vdim=24, decay=(0.5, 0.9, 0.995))
+    specs = [(delta, DenseFFSpec(144)), (pair, DenseFFSpec(120)), (light, None), (pair, DenseFFSpec(64))]
+    loop = (1, 3, 3)
+    return ModelConfig.layered("Sikalorn", unroll_loop(specs, loop), width=width, vocab=vocab, eps=eps, max_pos=4096, name="tiny-sikalorn", loop=loop)
 
 
 @dataclass

@@ -30,6 +30,8 @@ from ..ops import reference as ref
 from .config import ModelConfig, ParallelLayout
 from .layered import assemble_layers, random_param
 from .layered_ops import LayeredOps
+from .parallel_layers import load_loop, load_tanh_norm
+from .parallel_ops import ParallelOps
 
 
 @dataclass
@@ -50,8 +52,9 @@ class LayerWeights:
 class ModelWeights:
     embed: torch.Tensor | None         # [V, H] (first pipeline stage)
     layers: list                       # LayerWeights of this stage's blocks
-    final_norm: torch.Tensor | None    # [H] (last stage)
+    final_norm: torch.Tensor | None    # [H] (last stage); parallel layers: a TanhNorm
     lm_head: torch.Tensor | None       # [V / tp, H] (last stage)
+    loop: object = None                # LoopWeights of a design that runs some layers several times
 
 
 def shard_shapes(cfg: ModelConfig, lay: ParallelLayout):
@@ -114,8 +117,9 @@ def _random_layered(cfg, device, seed, std, dtype) -> ModelWeights:
 
 def layered_weights(cfg, get) -> ModelWeights:
     """Weights of a design that lists its layers; get(name) returns the checkpoint tensor of that name."""
-    return ModelWeights(embed=get("embed").contiguous(), layers=assemble_layers(cfg, get), final_norm=get("final.norm").float().reshape(1),
-                        lm_head=get("head").contiguous())
+    final = load_tanh_norm(get, "final.norm") if cfg.is_parallel else get("final.norm").float().reshape(1)
+    return ModelWeights(embed=get("embed").contiguous(), layers=assemble_layers(cfg, get), final_norm=final, lm_head=get("head").contiguous(),
+                        loop=load_loop(cfg, get))
 
 
 def quantize_blocks(weights: ModelWeights, blocks, names=("wqkv", "wo", "w13", "w2"), drop_bf16: bool = True) -> None:
@@ -151,6 +155,7 @@ class BatchInputs:
     kv_start: torch.Tensor | None = None       # [S] int32
     kv_total: int = 0
     max_cached: int = 0
+    slots: torch.Tensor | None = None          # [S] int32 state slot of every sequence (models with a recurrent state)
 
 
 @dataclass
@@ -163,7 +168,7 @@ class SamplingInputs:
     step: torch.Tensor                 # [B] int32: counter of each row's random stream (the token's position)
 
 
-class Decoder(LayeredOps):
+class Decoder(LayeredOps, ParallelOps):
     """One rank's share of the model: weights, KV cache and the step function.
 
     The decoder takes ownership of `weights`: on a GPU the expert matrices are replaced in place by their tile-packed
@@ -171,9 +176,10 @@ class Decoder(LayeredOps):
 
     def __init__(self, cfg: ModelConfig, weights: ModelWeights, layout: ParallelLayout | None = None,
                  num_pages: int = 0, page_size: int | None = None, max_pos: int | None = None, comm=None, comm_moe=None,
-                 pack_moe: bool | None = None, kv_pools=None):
+                 pack_moe: bool | None = None, kv_pools=None, state_slots: int = 64):
         # pack_moe: tile-pack the FFN / expert weights. kv_pools: per-layer page pools allocated by the caller
-        # (peer-mapped pools of a prefill/decode pair, parallel/disagg.py) instead of pools allocated here
+        # (peer-mapped pools of a prefill/decode pair, parallel/disagg.py) instead of pools allocated here.
+        # state_slots: sequences that can be live at a time in a model with a recurrent state
         self.cfg, self.w, self.layout = cfg, weights, layout or ParallelLayout()
         self.comm = comm          # tensor-parallel communicator over this rank's TP group, or None
         self.comm_moe = comm_moe  # communicator over all tp x ep ranks of the stage (expert parallelism), or None
@@ -192,10 +198,11 @@ class Decoder(LayeredOps):
         self.max_pos = max_pos or cfg.max_position_embeddings
         self.cos_sin = None if cfg.is_layered else ref.rope_cos_sin_table(self.max_pos, cfg.head_dim, cfg.rope_theta, dev, cfg.rope_scaling)
         self.num_pages = num_pages
+        self.num_state_slots = 0
         if cfg.is_layered:
             if kv_pools is not None:
                 raise ValueError(f"{cfg.architecture} allocates its own cache pools")
-            self._init_layered(num_pages)
+            self._init_layered(num_pages, state_slots)
         elif kv_pools is not None:
             want = (num_pages, 2, self.sh["Hkv"], page_size, cfg.head_dim)
             if len(kv_pools) != len(weights.layers) or any(tuple(p.shape) != want for p in kv_pools):
@@ -272,14 +279,14 @@ class Decoder(LayeredOps):
     class _Run:
         """State of one pass over the program."""
         __slots__ = ("inp", "residual", "normed", "qkv", "attn", "pending", "pending_kind", "routed", "h", "sp", "T",
-                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts", "dense")
+                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts", "dense", "cat")
 
         def __init__(self, inp, residual):
             self.inp, self.residual = inp, residual
             self.normed = self.qkv = self.attn = self.pending = self.routed = self.h = None
             self.pending_kind, self.crossing, self.sp, self.T = None, None, False, 0
             self.embed_deferred = False
-            self.row_idx = self.row_w = self.owner = self.wts = self.dense = None
+            self.row_idx = self.row_w = self.owner = self.wts = self.dense = self.cat = None
             self.dp = 0          # rows per rank under data-parallel attention (0: every rank holds all rows)
 
     def dp_ways(self) -> int:
@@ -322,7 +329,9 @@ class Decoder(LayeredOps):
 
     # ---- operators of the program (one method per operator name of the lowering) -----------------------
     def _op_embed_tokens(self, st, _):
-        if self.cfg.is_layered:
+        if self.cfg.is_parallel:
+            self._embed_parallel(st)
+        elif self.cfg.is_layered:
             st.residual = ops.latent.embed_f32(st.inp.token_ids, self.w.embed)
         elif self.embed_vocab_start is not None:
             st.embed_deferred = True       # the ranks' lookups are summed where the lowering puts the embed_out all-reduce

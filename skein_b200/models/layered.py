@@ -1,12 +1,18 @@
 """Designs whose configuration lists the layers one by one, each with its own mixer and feed-forward: specification,
 parameter names and shapes, weights.
 
-A layer of such a design is post-norm: x <- norm1(alpha x + mixer(h)), x <- norm2(alpha x + ff(x)), with RMS norms whose
-gain is one number, and h = x + (short causal convolution of x over time). Several layers may use one layer's tensors
-(`weights_of`); each keeps a cache of its own. The registry below names, per architecture, which mixers exist:
+Two kinds of layers exist. A post-norm layer is x <- norm1(alpha x + mixer(h)), x <- norm2(alpha x + ff(x)), with RMS norms
+whose gain is one number, and h = x + (short causal convolution of x over time). A parallel layer is
+x <- x + (mixer(h) + ff(h)) with h = tanh(a x) w + b (models/parallel_layers.py). Several layers may use one layer's tensors
+(`weights_of`); each keeps a cache of its own. A range of layers may run several times (`loop`): ModelConfig.layers then lists
+every run, the later ones with `weights_of` the first. The registry below names, per architecture, the kind of its layers and
+which mixers exist:
 
   Zarorax   latent_attention     latent attention, queries through a latent of their own
             latent_attention_2   latent attention, queries straight from the input, output gated by a sigmoid
+  Sikalorn  parallel             sliding-window attention beside a state-space recurrence, both on the same input
+            delta                gated delta rule
+            lightning            linear attention with a fixed decay per head
 """
 from __future__ import annotations
 
@@ -14,8 +20,13 @@ from dataclasses import dataclass, field
 
 import torch
 
-# architecture -> mixer type -> (queries through a latent, output gate)
-LAYERED_ARCHS = {"Zarorax": {"latent_attention": (True, False), "latent_attention_2": (False, True)}}
+from . import parallel_layers as pl
+from .parallel_layers import MixerPairSpec, RecurrentSpec, SpecError, WindowAttnSpec  # noqa: F401
+
+# architecture -> mixer type -> (queries through a latent, output gate), or the parser of the mixer
+LAYERED_ARCHS = {"Zarorax": {"latent_attention": (True, False), "latent_attention_2": (False, True)},
+                 "Sikalorn": {"parallel": pl.parse_pair, "delta": pl.parse_delta, "lightning": pl.parse_lightning}}
+PARALLEL_ARCHS = {"Sikalorn"}      # the architectures of parallel layers
 
 GLU_SLOPE = 1.702          # g * sigmoid(GLU_SLOPE * g) of the clamped gated unit
 
@@ -42,6 +53,14 @@ class LatentMixerSpec:
     def q_width(self) -> int:
         return self.heads * (self.dim + self.rot_dim)
 
+    @property
+    def head_size(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def cache_elems_per_token(self) -> int:
+        return self.cache_width
+
 
 @dataclass(frozen=True)
 class DenseFFSpec:
@@ -60,17 +79,18 @@ class RoutedFFSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentMixerSpec
+    mixer: LatentMixerSpec | MixerPairSpec | RecurrentSpec
     mlp: DenseFFSpec | RoutedFFSpec | None
     weights_of: int | None = None
+    tensors: int | None = None     # number of this layer in the checkpoint's names, where that is not its place in the list
+    loop_pass: int | None = None   # this layer opens the loop's pass of that number
 
 
-class SpecError(ValueError):
-    pass
-
-
-def parse_layers(arch: str, layers: list) -> tuple:
-    """The configuration's `layers` list -> LayerSpec tuple (`weights_of` chains resolved to the layer that owns tensors)."""
+def parse_layers(arch: str, layers: list, loop: dict | None = None) -> tuple:
+    """The configuration's `layers` list (and `loop`) -> LayerSpec tuple (`weights_of` chains resolved to the layer that owns
+    tensors, loops to one entry per run)."""
+    if arch in PARALLEL_ARCHS:
+        return _parse_parallel_layers(arch, layers, loop)
     kinds = LAYERED_ARCHS[arch]
     out = []
     for i, d in enumerate(layers):
@@ -113,8 +133,38 @@ def parse_layers(arch: str, layers: list) -> tuple:
     return tuple(out)
 
 
+def _parse_parallel_layers(arch: str, layers: list, loop: dict | None) -> tuple:
+    specs = []
+    for i, d in enumerate(layers):
+        parse = LAYERED_ARCHS[arch].get(d.get("type"))
+        if parse is None:
+            raise SpecError(f"layer {i}: mixer type {d.get('type')!r} is not part of {arch}")
+        mlp = d.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise SpecError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
+        try:
+            specs.append((parse(d["mixer"]), DenseFFSpec(int(mlp["ff"])) if mlp is not None else None))
+        except SpecError as e:
+            raise SpecError(f"layer {i}: {e}") from e
+    return unroll_loop(specs, pl.parse_loop(loop, len(specs)))
+
+
+def unroll_loop(specs, loop) -> tuple:
+    """(mixer, mlp) pairs in checkpoint order and a loop (start, stop, times) or None -> one LayerSpec per run."""
+    first, out = {}, []
+    for i, t in pl.layer_runs(len(specs), loop):
+        opens = t if (loop is not None and i == loop[0]) else None
+        out.append(LayerSpec(*specs[i], weights_of=first.get(i), tensors=i, loop_pass=opens))
+        first.setdefault(i, len(out) - 1)
+    return tuple(out)
+
+
 def layers_to_list(layers) -> list:
     """Inverse of parse_layers."""
+    if layers and layers[0].tensors is not None:
+        own = [sp for sp in layers if sp.weights_of is None]
+        return [{"type": sp.mixer.kind, "mixer": sp.mixer.to_dict(), "mlp": None if sp.mlp is None else {"kind": "dense", "ff": sp.mlp.ff}}
+                for sp in sorted(own, key=lambda sp: sp.tensors)]
     out = []
     for sp in layers:
         m = sp.mixer
@@ -142,6 +192,10 @@ def param_shapes(cfg) -> dict:
     """Checkpoint tensor name -> shape, in file order (layers with `weights_of` own none)."""
     C = cfg.hidden_size
     s = {"embed": (cfg.vocab_size, C)}
+    if cfg.is_parallel:
+        s.update(pl.param_shapes(cfg))
+        s["head"] = (cfg.vocab_size, C)
+        return s
     for i, sp in enumerate(cfg.layers):
         if sp.weights_of is not None:
             continue
@@ -174,6 +228,8 @@ def param_shapes(cfg) -> dict:
 def active_params(cfg) -> int:
     """Weights one token multiplies with (its chosen experts only), output projection included."""
     C, n = cfg.hidden_size, cfg.vocab_size * cfg.hidden_size
+    if cfg.is_parallel:
+        return n + pl.active_params(cfg)
     for sp in cfg.layers:
         m = sp.mixer
         n += C * (m.cache_width + m.heads * m.vdim * (2 if m.gated else 1)) + m.heads * (m.dim + m.vdim) * m.kv_rank
@@ -196,6 +252,11 @@ def decode_gemm_shapes(cfg) -> list:
             out.append((name, F, K, E, swiglu))
     for i, sp in enumerate(cfg.layers):
         m = sp.mixer
+        if cfg.is_parallel:
+            lay = pl.LayerLayout(sp)
+            add(f"l{i}.in", lay.in_rows, C)
+            add(f"l{i}.out", C, lay.out_cols)
+            continue
         add(f"l{i}.in", _up8(m.q_rank or m.q_width) + _up8(m.cache_width) + (_up8(m.heads * m.vdim) if m.gated else 0), C)
         if m.q_rank:
             add(f"l{i}.uq", m.q_width, m.q_rank)
@@ -211,8 +272,7 @@ def decode_gemm_shapes(cfg) -> list:
 
 
 # ---- weights ------------------------------------------------------------------------------------------------------
-def _up8(n: int) -> int:
-    return (n + 7) // 8 * 8
+_up8 = pl.up8
 
 
 @dataclass
@@ -277,6 +337,9 @@ def assemble_layers(cfg, get) -> list:
         if sp.weights_of is not None:
             out.append(out[sp.weights_of])
             continue
+        if cfg.is_parallel:
+            out.append(pl.assemble_layer(sp, get))
+            continue
         p = f"l{i}."
         lw = LayeredWeights(mixer=assemble_mixer(sp.mixer, get, p + "mix."), conv=get(p + "canon1").float().t().contiguous(),
                             norm1=get(p + "norm1").float().reshape(1),
@@ -294,6 +357,9 @@ def assemble_layers(cfg, get) -> list:
 
 def random_param(name: str, shape, gen, std: float, dtype, device):
     """Seeded random parameter: N(0, std), gains 1, the polynomial activation near its linear term, convolution taps small."""
+    special = pl.random_param(name, shape, gen, device)
+    if special is not None:
+        return special.to(dtype)
     if name.endswith("norm") or name.endswith(("norm1", "norm2")):
         return torch.ones(shape, dtype=dtype, device=device)
     t = torch.empty(shape, dtype=torch.float32, device=device)

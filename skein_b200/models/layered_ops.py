@@ -24,10 +24,12 @@ EXPAND_MIN_ROWS = 33      # a chunk of at least this many rows expands keys and 
 
 
 class LayeredOps:
-    def _init_layered(self, num_pages: int) -> None:
+    def _init_layered(self, num_pages: int, state_slots: int) -> None:
         cfg, w, dev = self.cfg, self.w, self.device
         if self.layout.world != 1:
             raise ValueError(f"{cfg.architecture} runs on one device (tp = pp = ep = 1)")
+        if cfg.is_parallel:
+            return self._init_parallel(num_pages, state_slots)
         self.act_dtype = w.embed.dtype
         tables = {}
         for sp in cfg.layers:

@@ -1,0 +1,429 @@
+"""Parallel layers, x <- x + (mixer(h) + ff(h)) with h = tanh(alpha x) w + b: specification, parameter names, weights.
+
+Mixers (specifications are data; a design picks some and fixes nothing else):
+
+  WindowAttnSpec   grouped-query attention over a sliding window; RMS norm of the whole q and k projections, then rotation of
+                   the first rot_dims dimensions of every head (pairs i, i + rot_dims / 2; frequencies divided by rot_factor)
+  RecurrentSpec    a matrix state S [dim, vdim] per head, 32-bit, carried from token to token:
+                       S <- g S + k u^T,   o = S^T q (+ D v)
+                     "delta"      g per head and token, u = beta (v - (g S)^T k), q and k unit vectors
+                     "ssd"        g = exp(-exp(A) dt), u = dt v (Mamba-2; q, k, v are C, B, x)
+                     "lightning"  g fixed per head, u = v
+  MixerPairSpec    an attention and a recurrence beside each other, summed with a weight each
+
+A layer runs as one product from h (w_in: the feed-forward's up projection and every projection of the mixer, stacked), the
+mixer's own kernels, and one product back (w_out: the mixers' output projections and the feed-forward's down projection side
+by side, so that their sum is the product's). LayerLayout says where everything sits in the row between the two products:
+
+    [ mixer outputs | feed-forward (activated in place) | projections of the mixers ]
+      <------------ read by w_out ------------------->
+                      <--------------- written by w_in ------------------------------>
+
+Every section starts at a multiple of 8 elements.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+
+import torch
+
+
+class SpecError(ValueError):
+    pass
+
+
+def up8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class WindowAttnSpec:
+    heads: int
+    kv_heads: int
+    dim: int                 # of a query / key head
+    vdim: int
+    scale: float
+    rot_dims: int
+    rope_base: float
+    rope_factor: float = 1.0
+    window: int = 0          # position i sees j with 0 <= i - j < window (0: every earlier position)
+
+    @property
+    def cache_elems_per_token(self) -> int:
+        return self.kv_heads * (self.dim + self.vdim)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def sections(self) -> list:
+        """(tensor, rows) of the projections of h, in stacking order."""
+        return [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+
+    def param_shapes(self, C: int) -> dict:
+        s = {n: (rows, C) for n, rows in self.sections()}
+        s["q.norm"], s["k.norm"] = (self.heads * self.dim,), (self.kv_heads * self.dim,)
+        s["o"] = (C, self.out_width)
+        return s
+
+    def to_dict(self) -> dict:
+        rot = {"base": self.rope_base, "dims": self.rot_dims}
+        if self.rope_factor != 1.0:
+            rot["scaling"] = {"factor": self.rope_factor}
+        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": rot}
+        if self.window:
+            d["mask"] = {"size": self.window}
+        return d
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    kind: str                # "delta", "ssd" or "lightning"
+    heads: int               # value heads (one state each)
+    groups: int              # query / key heads; head h uses h // (heads / groups)
+    dim: int                 # of a query / key head: rows of the state
+    vdim: int                # columns of the state
+    taps: int = 1            # of the short convolutions over time (1 for "lightning": none)
+    norm_groups: int = 1     # equal parts of the normed output that have a root mean square each ("ssd")
+    decay: tuple = ()        # "lightning"
+
+    @property
+    def cache_elems_per_token(self) -> int:
+        return 0
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def head_size(self) -> int:
+        return self.dim
+
+    @property
+    def conv_channels(self) -> int:
+        """Channels that pass a convolution: queries, keys and values together."""
+        return 2 * self.groups * self.dim + self.heads * self.vdim if self.kind != "lightning" else 0
+
+    @property
+    def conv_rows(self) -> int:
+        """Cached inputs of the convolution. One more than it looks back, so that a step writes no row that it reads."""
+        return self.taps if self.conv_channels and self.taps > 1 else 0
+
+    @property
+    def state_elems(self) -> int:
+        return self.heads * self.dim * self.vdim
+
+    def state_bytes(self, elem: int = 2) -> int:
+        """Bytes of one sequence's state: the 32-bit matrices and the convolution's last inputs."""
+        return 4 * self.state_elems + elem * self.conv_rows * self.conv_channels
+
+    def sections(self) -> list:
+        GD, HV = self.groups * self.dim, self.heads * self.vdim
+        if self.kind == "ssd":      # rows of the one input matrix: z | x | B | C | dt
+            return [("z", HV), ("conv", HV + 2 * GD), ("dt", self.heads)]
+        qkv = [("q", GD), ("k", GD), ("v", HV), ("g", HV)]
+        return qkv + [("b", self.heads), ("a", self.heads)] if self.kind == "delta" else qkv
+
+    def param_shapes(self, C: int) -> dict:
+        H, GD, HV = self.heads, self.groups * self.dim, self.heads * self.vdim
+        if self.kind == "ssd":
+            ch = self.conv_channels
+            return {"in": (2 * HV + 2 * GD + H, C), "conv": (ch, self.taps), "conv.b": (ch,), "dt_bias": (H,), "A_log": (H,), "D": (H,),
+                    "norm": (HV,), "o": (C, HV)}
+        s = {n: (rows, C) for n, rows in self.sections()}
+        if self.kind == "delta":
+            s.update({n + ".conv": (rows, self.taps) for n, rows in self.sections()[:3]})
+            s.update({"A_log": (H,), "dt_bias": (H,), "norm": (self.vdim,)})
+        else:
+            s["norm"] = (HV,)
+        s["o"] = (C, HV)
+        return s
+
+    def to_dict(self) -> dict:
+        d = {"heads": self.heads, "dim": self.dim, "vdim": self.vdim}
+        if self.kind == "ssd":
+            return {"conv": self.taps, "groups": self.groups, "heads": self.heads, "norm_groups": self.norm_groups, "state": self.dim,
+                    "vdim": self.vdim}
+        if self.kind == "delta":
+            return {**d, "conv": self.taps, "kv_heads": self.groups}
+        return {**d, "decay": list(self.decay)}
+
+
+@dataclass(frozen=True)
+class MixerPairSpec:
+    left: WindowAttnSpec
+    right: RecurrentSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    kind: str = "parallel"
+
+    @property
+    def heads(self) -> int:
+        return self.left.heads
+
+    @property
+    def head_size(self) -> int:
+        return self.left.dim
+
+    @property
+    def cache_elems_per_token(self) -> int:
+        return self.left.cache_elems_per_token
+
+    def to_dict(self) -> dict:
+        return {"left": self.left.to_dict(), "left_scale": self.left_scale, "right": self.right.to_dict(), "right_scale": self.right_scale}
+
+
+def attention_of(mixer) -> WindowAttnSpec | None:
+    return mixer.left if isinstance(mixer, MixerPairSpec) else None
+
+
+def recurrence_of(mixer) -> RecurrentSpec | None:
+    return mixer.right if isinstance(mixer, MixerPairSpec) else mixer if isinstance(mixer, RecurrentSpec) else None
+
+
+# ---- configuration -------------------------------------------------------------------------------------------------
+def _need(ok: bool, what: str) -> None:
+    if not ok:
+        raise SpecError(what)
+
+
+def parse_window(m: dict) -> WindowAttnSpec:
+    rot, mask = m["rot"], m.get("mask") or {}
+    a = WindowAttnSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
+                       rot_dims=int(rot["dims"]), rope_base=float(rot["base"]), rope_factor=float((rot.get("scaling") or {}).get("factor", 1.0)),
+                       window=int(mask.get("size") or 0))
+    _need(a.heads % a.kv_heads == 0, "heads must be a multiple of kv_heads")
+    _need(a.rot_dims % 2 == 0 and 0 <= a.rot_dims <= a.dim, "rot.dims must be even and at most dim (rotation turns pairs)")
+    _need(a.window >= 0 and a.rope_factor > 0, "mask.size and rot.scaling.factor must be positive")
+    return a
+
+
+def parse_ssd(m: dict) -> RecurrentSpec:
+    r = RecurrentSpec("ssd", heads=int(m["heads"]), groups=int(m["groups"]), dim=int(m["state"]), vdim=int(m["vdim"]), taps=int(m["conv"]),
+                      norm_groups=int(m["norm_groups"]))
+    _need(r.heads % r.groups == 0, "heads must be a multiple of groups")
+    _need(r.norm_groups >= 1 and r.out_width % r.norm_groups == 0, "norm_groups must divide heads * vdim")
+    _need(r.taps >= 1, "conv must be at least 1")
+    return r
+
+
+def parse_delta(m: dict) -> RecurrentSpec:
+    r = RecurrentSpec("delta", heads=int(m["heads"]), groups=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), taps=int(m["conv"]))
+    _need(r.heads % r.groups == 0, "heads must be a multiple of kv_heads")
+    _need(r.taps >= 1, "conv must be at least 1")
+    return r
+
+
+def parse_lightning(m: dict) -> RecurrentSpec:
+    r = RecurrentSpec("lightning", heads=int(m["heads"]), groups=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                      decay=tuple(float(x) for x in m["decay"]))
+    _need(len(r.decay) == r.heads, "decay must list one number per head")
+    _need(all(0.0 <= d <= 1.0 for d in r.decay), "decay must lie in [0, 1]")
+    return r
+
+
+def parse_pair(m: dict) -> MixerPairSpec:
+    return MixerPairSpec(parse_window(m["left"]), parse_ssd(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+
+
+def parse_loop(loop: dict | None, n: int):
+    """(start, stop, times) or None."""
+    if not loop:
+        return None
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= start < stop <= n or times < 1:
+        raise SpecError(f"loop {start}..{stop} x {times} is not a range of the {n} layers")
+    return start, stop, times
+
+
+def layer_runs(n: int, loop) -> list:
+    """(layer, pass) in the order they run; pass is None outside the loop."""
+    if loop is None:
+        return [(i, None) for i in range(n)]
+    a, b, times = loop
+    return ([(i, None) for i in range(a)] + [(i, t) for t in range(times) for i in range(a, b)] + [(i, None) for i in range(b, n)])
+
+
+# ---- parameters --------------------------------------------------------------------------------------------------
+def _mixer_parts(mixer):
+    """(name prefix under the layer, specification, weight of its output)."""
+    if isinstance(mixer, MixerPairSpec):
+        return [("mix.left.", mixer.left, mixer.left_scale), ("mix.right.", mixer.right, mixer.right_scale)]
+    return [("mix.", mixer, 1.0)]
+
+
+def _norm_shapes(name: str, C: int) -> dict:
+    return {name: (C,), name + ".b": (C,), name + ".alpha": ()}
+
+
+def param_shapes(cfg) -> dict:
+    C, s = cfg.hidden_size, {}
+    if cfg.loop is not None:
+        s["loop.in"], s["loop.step"] = (C, 2 * C), (cfg.loop[2], C)
+    for sp in sorted((sp for sp in cfg.layers if sp.weights_of is None), key=lambda sp: sp.tensors):
+        p = f"l{sp.tensors}."
+        s.update(_norm_shapes(p + "norm1", C))
+        for pre, m, _ in _mixer_parts(sp.mixer):
+            s.update({p + pre + n: shape for n, shape in m.param_shapes(C).items()})
+        if sp.mlp is not None:
+            s[p + "mlp.up"], s[p + "mlp.down"] = (sp.mlp.ff, C), (C, sp.mlp.ff)
+    s.update(_norm_shapes("final.norm", C))
+    return s
+
+
+def active_params(cfg) -> int:
+    C = cfg.hidden_size
+    n = 2 * C * C * cfg.loop[2] if cfg.loop is not None else 0
+    for sp in cfg.layers:
+        lay = LayerLayout(sp)
+        n += C * (lay.in_rows + lay.out_cols)
+    return n
+
+
+@dataclass
+class Section:
+    """Columns of a layer's row (LayerLayout) that belong to one mixer."""
+    spec: object
+    scale: float             # weight of the mixer's output in the layer's sum
+    out: int                 # first column of its output
+    col: dict                # projection -> first column
+
+
+class LayerLayout:
+    def __init__(self, sp):
+        self.parts, at = [], 0
+        parts = _mixer_parts(sp.mixer)
+        for _, m, scale in parts:
+            self.parts.append(Section(m, scale, at, {}))
+            at += up8(m.out_width)
+        self.ff, self.ff_cols = at, up8(sp.mlp.ff) if sp.mlp is not None else 0
+        self.in_first = at               # w_in writes from here
+        at += self.ff_cols
+        self.out_cols = at               # w_out reads up to here
+        for sec in self.parts:
+            for name, rows in sec.spec.sections():
+                sec.col[name] = at
+                at += up8(rows)
+        self.width, self.in_rows = at, at - self.in_first
+        self.zero_fill = any(m.out_width % 8 for _, m, _ in parts)      # columns that w_out reads and nothing writes
+
+    def part(self, cls):
+        return next((s for s in self.parts if isinstance(s.spec, cls)), None)
+
+
+# ---- weights ------------------------------------------------------------------------------------------------------
+@dataclass
+class TanhNorm:
+    """tanh(alpha x) w + b."""
+    alpha: torch.Tensor      # [1] fp32
+    w: torch.Tensor          # [C] fp32
+    b: torch.Tensor          # [C] fp32
+
+
+@dataclass
+class WindowAttnWeights:
+    q_norm: torch.Tensor     # [heads * dim] fp32
+    k_norm: torch.Tensor     # [kv_heads * dim] fp32
+
+
+@dataclass
+class RecurrentWeights:
+    norm: torch.Tensor                     # output norm, fp32: [vdim] ("delta") or [heads * vdim]
+    conv: torch.Tensor | None = None       # [taps, channels] fp32, channels q | k | v (zero taps of "lightning": none)
+    conv_b: torch.Tensor | None = None     # [channels] fp32
+    neg_decay: torch.Tensor | None = None  # [heads] fp32: -exp(A_log), or log(decay) of "lightning"
+    dt_bias: torch.Tensor | None = None    # [heads] fp32
+    skip: torch.Tensor | None = None       # [heads] fp32: D
+
+
+@dataclass
+class ParallelLayerWeights:
+    norm: TanhNorm
+    w_in: torch.Tensor                     # [in_rows, C]
+    w_out: torch.Tensor                    # [C, out_cols]
+    attn: WindowAttnWeights | None = None
+    rec: RecurrentWeights | None = None
+    fp8: dict = field(default_factory=dict)
+
+
+@dataclass
+class LoopWeights:
+    w_in: torch.Tensor                     # [C, 2 C]: the stream, then the embedding output
+    step: torch.Tensor                     # [times, C] fp32
+
+
+def load_tanh_norm(get, name: str) -> TanhNorm:
+    return TanhNorm(get(name + ".alpha").float().reshape(1), get(name).float(), get(name + ".b").float())
+
+
+def load_loop(cfg, get) -> LoopWeights | None:
+    return None if cfg.loop is None else LoopWeights(get("loop.in").contiguous(), get("loop.step").float())
+
+
+def _pad(t: torch.Tensor, dim: int) -> torch.Tensor:
+    n = up8(t.shape[dim]) - t.shape[dim]
+    if n == 0:
+        return t
+    shape = list(t.shape)
+    shape[dim] = n
+    return torch.cat([t, torch.zeros(shape, dtype=t.dtype, device=t.device)], dim=dim)
+
+
+def _load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
+    w = RecurrentWeights(norm=get(p + "norm").float())
+    GD, HV = m.groups * m.dim, m.heads * m.vdim
+    if m.kind == "lightning":
+        w.neg_decay = torch.tensor(m.decay, dtype=torch.float64).log().clamp(min=-1e30).float().to(w.norm.device)
+        return w
+    w.neg_decay, w.dt_bias = -get(p + "A_log").float().exp(), get(p + "dt_bias").float()
+    if m.kind == "delta":
+        w.conv = torch.cat([get(p + n + ".conv").float() for n in ("q", "k", "v")]).t().contiguous()
+    else:      # the checkpoint's order is x (values) | B (keys) | C (queries)
+        c, b = get(p + "conv").float(), get(p + "conv.b").float()
+        order = torch.cat([torch.arange(HV + GD, HV + 2 * GD), torch.arange(HV, HV + GD), torch.arange(HV)]).to(c.device)
+        w.conv, w.conv_b, w.skip = c[order].t().contiguous(), b[order].contiguous(), get(p + "D").float()
+    return w
+
+
+def assemble_layer(sp, get) -> ParallelLayerWeights:
+    p = f"l{sp.tensors}."
+    ins, outs = [], []
+    attn = rec = None
+    if sp.mlp is not None:
+        ins.append(get(p + "mlp.up"))
+    for pre, m, _ in _mixer_parts(sp.mixer):
+        q = p + pre
+        if isinstance(m, WindowAttnSpec):
+            attn = WindowAttnWeights(get(q + "q.norm").float(), get(q + "k.norm").float())
+        else:
+            rec = _load_recurrence(m, get, q)
+        if isinstance(m, RecurrentSpec) and m.kind == "ssd":
+            rows, whole = m.sections(), get(q + "in")
+            ins.extend(whole.split([n for _, n in rows]))
+        else:
+            ins.extend(get(q + n) for n, _ in m.sections())
+        outs.append(_pad(get(q + "o"), 1))
+    if sp.mlp is not None:
+        outs.append(_pad(get(p + "mlp.down"), 1))
+    return ParallelLayerWeights(norm=load_tanh_norm(get, p + "norm1"), w_in=torch.cat([_pad(t, 0) for t in ins]).contiguous(),
+                                w_out=torch.cat(outs, dim=1).contiguous(), attn=attn, rec=rec)
+
+
+def random_param(name: str, shape, gen, device):
+    """Seeded random values of the parameters that are neither projections nor gains: decays between slow and fast, small steps,
+    convolution taps and biases of order one; None for the others."""
+    def normal(std, mean=0.0):
+        return torch.empty(shape, dtype=torch.float32, device=device).normal_(mean, std, generator=gen)
+    if name.endswith(".alpha"):
+        return torch.ones(shape, device=device)
+    if name.endswith((".norm1.b", "norm.b", ".conv.b", "loop.step")):
+        return normal(0.02)
+    if name.endswith(".conv"):
+        return normal(shape[-1] ** -0.5)
+    if name.endswith(".A_log"):
+        return normal(1.0)
+    if name.endswith(".dt_bias"):
+        return normal(1.0, -3.0)
+    if name.endswith(".D"):
+        return torch.ones(shape, device=device)
+    return None

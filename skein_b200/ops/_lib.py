@@ -36,8 +36,23 @@ class GemmParams(C.Structure):
         ("wait_budget_ms", C.c_int32), ("w_packed", C.c_int32), ("line_cut_only", C.c_int32),
         ("x_ld", C.c_int32), ("x_group_cols", C.c_int32), ("out_group_cols", C.c_int32), ("glu", C.c_int32),
         ("glu_limit", C.c_float), ("glu_slope", C.c_float), ("out_f32", C.c_int32), ("gate_ld", C.c_int32),
-        ("gate", C.c_void_p),
+        ("gate", C.c_void_p), ("relu2_cols", C.c_int32), ("pad", C.c_int32),
     ]
+
+
+class RecParams(C.Structure):
+    """Mirror of SkeinRecParams in csrc/kernels/recurrent.cuh (same field order)."""
+
+    _fields_ = [(n, C.c_void_p) for n in ("row", "out", "state", "tail", "conv_w", "conv_b", "neg_decay", "dt_bias", "skip", "positions",
+                                          "slots", "status")] + [("ld", C.c_int64)] + [
+        (n, C.c_int32) for n in ("kind", "H", "G", "D", "V", "taps", "C", "q_col", "k_col", "v_col", "a_col", "b_col", "num_slots")]
+
+
+class RecChunk(C.Structure):
+    """Mirror of SkeinRecChunk in csrc/kernels/recurrent.cuh (same field order)."""
+
+    _fields_ = [(n, C.c_void_p) for n in ("seq_of_token", "q_start", "q_len", "qkv", "gates", "unit", "chunk_mat")] + [
+        ("qkv_ld", C.c_int64), ("v_off", C.c_int32), ("max_q_len", C.c_int32)]
 
 
 def lib_path() -> Path:
@@ -134,6 +149,16 @@ def lib():
          [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp])
     _sig(L, "skein_latent_attn_prefill", i32,
          [vp, i64, i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp])
+    _sig(L, "skein_residual_tanh", i32, [vp, vp, i32, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp])
+    _sig(L, "skein_gated_norm", i32, [vp, vp, i64, vp, i32, vp, i64, i32, i32, i32, i32, i32, f32, f32, i32, vp])
+    _sig(L, "skein_window_append", i32,
+         [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
+    _sig(L, "skein_window_attn_rows", i32, [vp, i64, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, vp])
+    rec, chunk = C.POINTER(RecParams), C.POINTER(RecChunk)
+    _sig(L, "skein_rec_step", i32, [rec, i32, i32, vp])
+    _sig(L, "skein_rec_prep", i32, [rec, chunk, i32, i32, vp])
+    _sig(L, "skein_rec_scan", i32, [rec, chunk, i32, i32, vp])
+    _sig(L, "skein_rec_tail", i32, [rec, chunk, i32, i32, vp])
     for name, rt, at in _OPTIONAL:
         if hasattr(L, name):
             _sig(L, name, rt, at)

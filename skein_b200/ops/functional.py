@@ -223,12 +223,13 @@ def simt_launch(p: "_lib.GemmParams", x, max_rows: int, what: str):
     _lib.count_launch()
 
 
-def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False):
-    """y[t, f] = sum_k x[t, k] w[f, k] (+ residual[t, f]). out_f32: the accumulator is stored without rounding to bf16.
-    x may be the first K columns of a wider matrix (rows strided)."""
+def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False, relu2_cols=0):
+    """y[t, f] = sum_k x[t, k] w[f, k] (+ residual[t, f]). out_f32: the accumulator is stored without rounding to bf16, the
+    residual is fp32 too. x may be the first K columns of a wider matrix (rows strided), and out, which may be the residual, a
+    run of columns of one. The first relu2_cols features are stored as max(y, 0)^2."""
     K = w.shape[1]
     if not x.is_cuda:
-        y = ref.linear(x[:, :K], w.unpack() if isinstance(w, PackedWeight) else w, residual)
+        y = ref.linear(x[:, :K], w.unpack() if isinstance(w, PackedWeight) else w, residual, out_f32, relu2_cols)
         if out is not None:
             out.copy_(y)
             return out
@@ -243,7 +244,7 @@ def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False)
         return out
     wv, _, packed = _wview(w)
     p = _base_params(x, wv, out, F, K, n_tile or pick_n_tile(T, False), 0)
-    p.w_rows_per_group, p.w_packed, p.out_f32 = F, packed, 1 if out_f32 else 0
+    p.w_rows_per_group, p.w_packed, p.out_f32, p.relu2_cols = F, packed, 1 if out_f32 else 0, int(relu2_cols)
     if x.stride(0) != K:
         p.x_ld = x.stride(0)
     if residual is not None:

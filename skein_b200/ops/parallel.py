@@ -1,0 +1,96 @@
+"""Operators of parallel layers (x <- x + mixer(h) + ff(h), h = tanh(alpha x) w + b) and of sliding-window attention.
+
+CUDA tensors run csrc/kernels (parallel_layer.cu, attn_window.cu, attn_prefill_tc.cu, attn_decode_mma.cu); CPU tensors run
+ops/reference_parallel.py. Activations are bf16, or fp32 when a model runs in 32-bit; the residual stream is fp32.
+"""
+from __future__ import annotations
+
+import torch
+
+from . import _lib, functional as F, reference_parallel as rp
+
+
+def _fp32(t) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def residual_tanh(x, y=None, bias=None, norm=None, dtype=torch.bfloat16, out=None, want_x=True):
+    """a = x + y + bias (each may be None), fp32. Returns (a, or None unless want_x; tanh(alpha a) w + b in `dtype` with a norm
+    (models/parallel_layers.py: TanhNorm), else a in `dtype`). `out`: where the latter goes, possibly columns of a wider matrix;
+    False: nowhere."""
+    like = x if x is not None else y
+    T, C = like.shape
+    if not like.is_cuda:
+        a, act = rp.residual_tanh(x, y, bias, norm, dtype)
+        if out is not None and out is not False:
+            out.copy_(act)
+            act = out
+        return (a if want_x else None), (None if out is False else act)
+    if out is None:
+        out = torch.empty(T, C, dtype=dtype, device=like.device)
+    act = None if out is False else out
+    plain = y is None and bias is None      # a is x
+    x_out = torch.empty(T, C, dtype=torch.float32, device=like.device) if want_x and not plain else None
+    if T:
+        _lib.check(_lib.lib().skein_residual_tanh(
+            _lib.ptr(x), _lib.ptr(y), 1 if y is None else _fp32(y), _lib.ptr(bias), _lib.ptr(norm.alpha if norm else None),
+            _lib.ptr(norm.w if norm else None), _lib.ptr(norm.b if norm else None), _lib.ptr(x_out), _lib.ptr(act),
+            act.stride(0) if act is not None else 0, T, C, 1 if dtype == torch.float32 else 0, _lib.stream_ptr()), "residual_tanh")
+        _lib.count_launch()
+    return ((x if plain else x_out) if want_x else None), act
+
+
+def gated_norm(o, gate, w, out, groups, eps, gate_first=False, silu=False, scale=1.0):
+    """o [T, n] in `groups` equal parts, each divided by its root mean square, times w ([n], or one part's or less, repeated) and
+    times the gate's activation (silu or sigmoid), which multiplies before the norm with gate_first; times scale, into `out`
+    (columns of a wider matrix)."""
+    T, n = o.shape
+    if not o.is_cuda:
+        out.copy_(rp.gated_norm(o, gate, w, groups, eps, gate_first, silu, scale))
+        return out
+    if T:
+        _lib.check(_lib.lib().skein_gated_norm(
+            o.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), w.shape[0], out.data_ptr(), out.stride(0), T, n, groups,
+            int(gate_first), int(silu), float(eps), float(scale), _fp32(o), _lib.stream_ptr()), "gated_norm")
+        _lib.count_launch()
+    return out
+
+
+# ---- sliding-window attention -----------------------------------------------------------------------------------------
+def window_cache(num_pages: int, page_size: int, kv_heads: int, dim: int, vdim: int, dtype, device) -> torch.Tensor:
+    """[pages, kv_heads * page_size * (dim + vdim)]: keys [kv_heads, page_size, dim], then values [kv_heads, page_size, vdim]."""
+    return torch.zeros(num_pages, kv_heads * page_size * (dim + vdim), dtype=dtype, device=device)
+
+
+def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
+    """Norm and rotation of q (in place) and k, append of k and v to the cache. q, k, v: columns of one matrix."""
+    T = q.shape[0]
+    if not q.is_cuda:
+        return rp.window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps)
+    if T:
+        _lib.check(_lib.lib().skein_window_append(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), q_norm.data_ptr(), k_norm.data_ptr(), cos_sin.data_ptr(), positions.data_ptr(),
+            _lib.ptr(seq_of_token), block_table.data_ptr(), cache.data_ptr(), F.workspace().status.data_ptr(), T, spec.heads, spec.kv_heads,
+            spec.dim, spec.vdim, spec.rot_dims, cos_sin.shape[0], block_table.stride(0), cache.shape[0], page_size, float(eps), _fp32(q),
+            _lib.stream_ptr()), "window_append")
+        _lib.count_launch()
+
+
+def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out, out_scale=1.0):
+    """Attention of single rows over the cache, any sizes (plain kernel)."""
+    T = q.shape[0]
+    if not q.is_cuda:
+        out.copy_(rp.window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale))
+        return out
+    if T:
+        _lib.check(_lib.lib().skein_window_attn_rows(
+            q.data_ptr(), q.stride(0), cache.data_ptr(), positions.data_ptr(), _lib.ptr(seq_of_token), block_table.data_ptr(), out.data_ptr(),
+            out.stride(0), F.workspace().status.data_ptr(), T, spec.heads, spec.kv_heads, spec.dim, spec.vdim, block_table.stride(0),
+            cache.shape[0], page_size, spec.window, float(spec.scale), float(out_scale), _fp32(q), _lib.stream_ptr()), "window_attn_rows")
+        _lib.count_launch()
+    return out
+
+
+def window_attn(q, spec, inp, cache, page_size, out, out_scale=1.0):
+    """Attention of a step's rows (a decode step or a chunk) over the cache; the tensor-core kernels where they take the sizes."""
+    return window_attn_rows(q, spec, inp.positions, inp.seq_of_token, inp.block_table, cache, page_size, out, out_scale)

@@ -1,0 +1,96 @@
+"""Recurrences with a 32-bit matrix state per head (gated delta rule, state-space duality, fixed decay).
+
+CUDA tensors run csrc/kernels/recurrent.cu and recurrent_tc.cu; CPU tensors run ops/reference_parallel.py. The specification
+(models/parallel_layers.py: RecurrentSpec) says which recurrence; the weights are its RecurrentWeights.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+
+import torch
+
+from . import _lib, functional as F, reference_parallel as rp
+
+KINDS = {"delta": 0, "ssd": 1, "lightning": 2}
+
+
+@dataclass
+class RecState:
+    """State pools of one recurrent layer: matrices [slots, heads, dim, vdim] fp32 and the convolution's last inputs
+    [slots, taps, channels] (None without a convolution), position p in row p mod taps."""
+    mat: torch.Tensor
+    tail: torch.Tensor | None
+
+    @staticmethod
+    def make(spec, slots: int, dtype, device) -> "RecState":
+        mat = torch.zeros(slots, spec.heads, spec.dim, spec.vdim, dtype=torch.float32, device=device)
+        tail = torch.zeros(slots, spec.conv_rows, spec.conv_channels, dtype=dtype, device=device) if spec.conv_rows else None
+        return RecState(mat, tail)
+
+
+@dataclass
+class RecColumns:
+    """First columns of the recurrence's projections in a row."""
+    q: int
+    k: int
+    v: int
+    a: int = 0               # input of the decay (delta: a; ssd: dt)
+    b: int = 0               # input of the write strength (delta)
+
+    @staticmethod
+    def of(spec, col: dict) -> "RecColumns":
+        if spec.kind == "ssd":      # values | keys | queries, the order of the checkpoint's matrix
+            v = col["conv"]
+            k = v + spec.heads * spec.vdim
+            return RecColumns(k + spec.groups * spec.dim, k, v, a=col["dt"])
+        return RecColumns(col["q"], col["k"], col["v"], col.get("a", 0), col.get("b", 0))
+
+
+def _params(row, cols, spec, w, state, positions, slots, out) -> "_lib.RecParams":
+    p = _lib.RecParams()
+    p.row, p.out, p.ld = row.data_ptr(), out.data_ptr(), row.stride(0)
+    p.state, p.tail = state.mat.data_ptr(), _lib.ptr(state.tail)
+    p.conv_w, p.conv_b, p.neg_decay, p.dt_bias, p.skip = (_lib.ptr(t) for t in (w.conv, w.conv_b, w.neg_decay, w.dt_bias, w.skip))
+    p.positions, p.slots, p.status = positions.data_ptr(), slots.data_ptr(), F.workspace().status.data_ptr()
+    p.kind, p.H, p.G, p.D, p.V, p.taps, p.C = KINDS[spec.kind], spec.heads, spec.groups, spec.dim, spec.vdim, spec.taps, spec.conv_channels
+    p.q_col, p.k_col, p.v_col, p.a_col, p.b_col, p.num_slots = cols.q, cols.k, cols.v, cols.a, cols.b, state.mat.shape[0]
+    return p
+
+
+def rec_step(row, cols: RecColumns, spec, w, state: RecState, positions, slots):
+    """One token per sequence: row [B, ld] holds the projections. Returns the read-outs [B, heads * vdim]; the state moves on."""
+    B = row.shape[0]
+    if not row.is_cuda:
+        return rp.rec_chunk(row, cols, spec, w, state, positions, slots, torch.arange(B), torch.ones(B, dtype=torch.int32))
+    out = torch.empty(B, spec.out_width, dtype=row.dtype, device=row.device)
+    p = _params(row, cols, spec, w, state, positions, slots, out)
+    _lib.check(_lib.lib().skein_rec_step(C.byref(p), B, 1 if row.dtype == torch.float32 else 0, _lib.stream_ptr()), "rec_step")
+    _lib.count_launch()
+    return out
+
+
+def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots, seq_of_token, q_start, q_len, max_q_len):
+    """Portions of several sequences: rows q_start[s] .. + q_len[s] are consecutive tokens of the sequence in slots[s]."""
+    T = row.shape[0]
+    if not row.is_cuda:
+        return rp.rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len)
+    dev, fp32, S = row.device, 1 if row.dtype == torch.float32 else 0, q_len.shape[0]
+    out = torch.empty(T, spec.out_width, dtype=row.dtype, device=dev)
+    p = _params(row, cols, spec, w, state, positions, slots, out)
+    c = _lib.RecChunk()
+    c.v_off = (2 * spec.groups * spec.dim + 7) // 8 * 8
+    c.qkv_ld = c.v_off + (spec.out_width + 7) // 8 * 8
+    qkv = torch.empty(T, c.qkv_ld, dtype=row.dtype, device=dev)
+    gates = torch.empty(T, spec.heads, 2, dtype=torch.float32, device=dev)
+    unit = torch.empty(T, 2, spec.groups, dtype=torch.float32, device=dev) if spec.kind == "delta" else None
+    c.seq_of_token, c.q_start, c.q_len, c.max_q_len = seq_of_token.data_ptr(), q_start.data_ptr(), q_len.data_ptr(), int(max_q_len)
+    c.qkv, c.gates, c.unit = qkv.data_ptr(), gates.data_ptr(), _lib.ptr(unit)
+    L, s = _lib.lib(), _lib.stream_ptr()
+    _lib.check(L.skein_rec_prep(C.byref(p), C.byref(c), T, fp32, s), "rec_prep")
+    _lib.check(L.skein_rec_scan(C.byref(p), C.byref(c), S, fp32, s), "rec_scan")
+    _lib.count_launch(2)
+    if state.tail is not None:
+        _lib.check(L.skein_rec_tail(C.byref(p), C.byref(c), S, fp32, s), "rec_tail")
+        _lib.count_launch()
+    return out

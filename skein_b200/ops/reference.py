@@ -11,11 +11,13 @@ import math
 import torch
 
 
-def linear(x, w, residual=None):
+def linear(x, w, residual=None, out_f32=False, relu2_cols=0):
     y = x.float() @ w.float().t()
+    if relu2_cols:
+        y[:, :relu2_cols] = y[:, :relu2_cols].clamp(min=0).square()
     if residual is not None:
         y = y + residual.float()
-    return y.to(x.dtype)
+    return y if out_f32 else y.to(x.dtype)
 
 
 def swiglu_linear(x, w13):

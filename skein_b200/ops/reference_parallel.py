@@ -1,0 +1,114 @@
+"""Plain PyTorch form of the operators of parallel layers, sliding-window attention and recurrences (ops/parallel.py,
+ops/recurrent.py): 32-bit math, results in the activation type."""
+from __future__ import annotations
+
+import torch
+
+
+def residual_tanh(x, y, bias, norm, dtype):
+    a = sum(t.float() for t in (x, y, bias) if t is not None)
+    if norm is None:
+        return a, a.to(dtype)
+    return a, (torch.tanh(norm.alpha * a) * norm.w + norm.b).to(dtype)
+
+
+def gated_norm(o, gate, w, groups, eps, gate_first, silu, scale):
+    T, n = o.shape
+    v, z = o.float(), gate.float()
+    g = torch.nn.functional.silu(z) if silu else torch.sigmoid(z)
+    if gate_first:
+        v = v * g
+    v = v.view(T, groups, -1)
+    v = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, n) * w.repeat(n // w.shape[0])
+    return ((v if gate_first else v * g) * scale).to(o.dtype)
+
+
+def _rotate(x, cos_sin, dims):
+    half = dims // 2
+    c, s = cos_sin[:, None, :half, 0], cos_sin[:, None, :half, 1]
+    u, v = x[..., :half], x[..., half:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], dim=-1)
+
+
+def _pages(cache, K, ps, D, V):
+    """(keys [pages, K, ps, D], values [pages, K, ps, V]) views of a cache."""
+    n = K * ps * D
+    return cache[:, :n].view(-1, K, ps, D), cache[:, n:].view(-1, K, ps, V)
+
+
+def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
+    keys, vals = _pages(cache, spec.kv_heads, page_size, spec.dim, spec.vdim)
+    T = q.shape[0]
+    for t in range(T):
+        pos = int(positions[t])
+        if pos < 0:
+            continue
+        cs = cos_sin[pos:pos + 1]
+        unit = lambda z, w: z.float() / torch.sqrt(z.float().pow(2).mean() + eps) * w        # noqa: E731
+        q[t] = _rotate(unit(q[t], q_norm).view(1, spec.heads, -1), cs, spec.rot_dims).reshape(-1).to(q.dtype)
+        page = int(block_table[int(seq_of_token[t]) if seq_of_token is not None else t, pos // page_size])
+        keys[page, :, pos % page_size] = _rotate(unit(k[t], k_norm).view(1, spec.kv_heads, -1), cs, spec.rot_dims)[0].to(cache.dtype)
+        vals[page, :, pos % page_size] = v[t].view(spec.kv_heads, -1)
+
+
+def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale):
+    keys, vals = _pages(cache, spec.kv_heads, page_size, spec.dim, spec.vdim)
+    T, G = q.shape[0], spec.heads // spec.kv_heads
+    out = torch.zeros(T, spec.heads * spec.vdim, dtype=q.dtype)
+    for t in range(T):
+        pos = int(positions[t])
+        if pos < 0:
+            continue
+        js = torch.arange(max(0, pos - spec.window + 1) if spec.window else 0, pos + 1)
+        pages = block_table[int(seq_of_token[t]) if seq_of_token is not None else t][js // page_size].long()
+        k = keys[pages, :, js % page_size].float().repeat_interleave(G, dim=1)
+        v = vals[pages, :, js % page_size].float().repeat_interleave(G, dim=1)
+        s = torch.einsum("hd,jhd->hj", q[t].float().view(spec.heads, -1), k) * spec.scale
+        out[t] = (torch.einsum("hj,jhv->hv", torch.softmax(s, dim=-1), v) * out_scale).reshape(-1).to(q.dtype)
+    return out
+
+
+def rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len):
+    H, G, D, V, taps = spec.heads, spec.groups, spec.dim, spec.vdim, spec.taps
+    dt = row.dtype
+    out = torch.zeros(row.shape[0], H * V, dtype=dt)
+    for s in range(q_len.shape[0]):
+        t0, n = int(q_start[s]), int(q_len[s])
+        if n < 1 or int(positions[t0]) < 0:
+            continue
+        pos0, slot = int(positions[t0]), int(slots[s])
+        r = row[t0:t0 + n].float()
+        x = torch.cat([r[:, cols.q:cols.q + G * D], r[:, cols.k:cols.k + G * D], r[:, cols.v:cols.v + H * V]], dim=1)
+        if spec.conv_channels:
+            prev = torch.zeros(taps - 1, x.shape[1])
+            for j in range(1, taps):
+                if pos0 - j >= 0:
+                    prev[taps - 1 - j] = state.tail[slot, (pos0 - j) % taps].float()
+            full = torch.cat([prev, x])
+            if state.tail is not None:
+                for j in range(max(0, n - taps + 1), n):
+                    state.tail[slot, (pos0 + j) % taps] = x[j].to(state.tail.dtype)
+            x = sum(w.conv[j] * full[j:j + n] for j in range(taps)) + (w.conv_b if w.conv_b is not None else 0.0)
+        x = torch.nn.functional.silu(x).to(dt).float()
+        q, k, v = x[:, :G * D].view(n, G, D), x[:, G * D:2 * G * D].view(n, G, D), x[:, 2 * G * D:].view(n, H, V)
+        if spec.kind == "delta":
+            q, k = (z / torch.sqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6) for z in (q, k))
+            q = q * D ** -0.5
+        q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)
+        if spec.kind == "lightning":
+            g, coef = w.neg_decay.exp().expand(n, H), torch.ones(n, H)
+        else:
+            step = torch.nn.functional.softplus(r[:, cols.a:cols.a + H] + w.dt_bias, threshold=60.0)
+            g = (w.neg_decay * step).exp()
+            coef = torch.sigmoid(r[:, cols.b:cols.b + H]) if spec.kind == "delta" else step
+        S = state.mat[slot].clone() if pos0 > 0 else torch.zeros(H, D, V)
+        for t in range(n):
+            S = g[t][:, None, None] * S
+            u = v[t] - torch.einsum("hdv,hd->hv", S, k[t]) if spec.kind == "delta" else v[t]
+            S = S + k[t][:, :, None] * (coef[t][:, None] * u)[:, None, :]
+            o = torch.einsum("hdv,hd->hv", S, q[t])
+            if w.skip is not None:
+                o = o + w.skip[:, None] * v[t]
+            out[t0 + t] = o.reshape(-1).to(dt)
+        state.mat[slot] = S
+    return out

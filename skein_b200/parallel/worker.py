@@ -31,12 +31,12 @@ from . import launcher
 
 
 def size_kv_pool(art: Artifact, lay, device, total_kv_bytes: int, page_size: int | None = None, reserve_frac: float = 0.08,
-                 bytes_per_token: int = 0) -> int:
+                 bytes_per_token: int = 0, reserve_bytes: int = 0) -> int:
     """Pages in the per-layer pool: from an explicit byte budget (with the model's KV bytes per token on this rank,
-    or the caller's `bytes_per_token`), else from the memory left after the weights."""
+    or the caller's `bytes_per_token`), else from the memory left after the weights and `reserve_bytes` (recurrent state)."""
     cfg = art.cfg
     page_size = page_size or cfg.default_page_size
-    page_bytes = cfg.cache_bytes_per_page(page_size, lay.tp, lay.stage_layers(cfg.num_layers))
+    page_bytes = max(1, cfg.cache_bytes_per_page(page_size, lay.tp, lay.stage_layers(cfg.num_layers)))
     if bytes_per_token > 0:
         page_bytes = bytes_per_token * page_size
     if total_kv_bytes > 0:
@@ -44,7 +44,7 @@ def size_kv_pool(art: Artifact, lay, device, total_kv_bytes: int, page_size: int
     if device.type != "cuda":
         return 256
     free, total = torch.cuda.mem_get_info(device)
-    return max(8, int((free - reserve_frac * total) // page_bytes))
+    return max(8, min(int((free - reserve_bytes - reserve_frac * total) // page_bytes), 1 << 24))
 
 
 def prefill_slice_for_slo(tpot_ms: float, decode_us_at_b1: float, batch_exponent: float, max_batch: int, prefill_per_token_us: float,
@@ -67,10 +67,13 @@ def build_engine(art: Artifact, rank: int, device, comm, args, comm_moe=None, pp
         tuning.activate(tuning.KernelConfigCache(tuned, strict=False))   # measured configurations win over the heuristics
     weights = art.load_weights(rank, device)
     page_size = art.plan["kv"]["layout"].get("page_size", art.cfg.default_page_size)
-    pages = size_kv_pool(art, lay, device, args.total_kv_bytes, page_size, bytes_per_token=getattr(args, "bytes_per_token", 0))
+    slots = max(1, args.max_batch or art.plan["batching"]["max_batch"])
+    pages = size_kv_pool(art, lay, device, args.total_kv_bytes, page_size, bytes_per_token=getattr(args, "bytes_per_token", 0),
+                         reserve_bytes=slots * art.cfg.state_bytes_per_slot())
     pages = min(pages, max(8, (args.max_seq_len // page_size + 1) * max(1, args.max_batch or art.plan["batching"]["max_batch"]) * 2))
     dec = Decoder(art.cfg, weights, lay, num_pages=pages, page_size=page_size,
-                  max_pos=min(args.max_seq_len, art.cfg.max_position_embeddings), comm=comm, comm_moe=comm_moe)
+                  max_pos=min(args.max_seq_len, art.cfg.max_position_embeddings), comm=comm, comm_moe=comm_moe,
+                  state_slots=slots)
     # Pure expert parallelism decodes with data-parallel attention: every rank attends over its own share of the step's
     # sequences and the MoE blocks exchange tokens over peer memory (SKEIN_EP_DP_ATTENTION=0: attention over all
     # sequences on every rank, the expert outputs all-reduced).

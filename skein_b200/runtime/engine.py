@@ -89,7 +89,9 @@ class Engine:
         c = self.cfg
         if decoder.num_pages <= 0:
             raise ValueError("the decoder was built without a KV page pool")
-        self.kv = core.KvBlockManager(decoder.num_pages, decoder.page_size, c.prefix_cache)
+        # a recurrent state lives in a slot per request, and cached pages alone do not bring it back: no prefix cache then
+        slots = getattr(getattr(decoder, "dec", decoder), "num_state_slots", 0)
+        self.kv = core.KvBlockManager(decoder.num_pages, decoder.page_size, c.prefix_cache and slots == 0, state_slots=slots)
         # Expert parallelism with data-parallel attention: each decoding sequence belongs to one rank's slice of the
         # step's rows for its whole life (only that rank's cache receives its new tokens). Every rank's engine takes
         # the same decisions, so the assignment needs no communication. A slice is never larger than
@@ -265,7 +267,7 @@ class Engine:
         seqs = []
         for rid, start, end, last in prefill:
             prompt = self.batcher.prompt(rid)
-            seqs.append((prompt[start:end], self.kv.pages_for(rid), start))
+            seqs.append((prompt[start:end], self.kv.pages_for(rid), start, self.kv.slot_of(rid)))
         toks = self.runner.prefill(seqs, sampling=self._rows([p[0] for p in prefill]))
         for (rid, start, end, last), tok in zip(prefill, toks):
             self.batcher.prefill_advanced(rid, end)
@@ -341,6 +343,8 @@ class Engine:
         pre, self._pre = self._pre, None
         if pre is not None and pre[1] != list(decode):
             self.runner.decode_wait(pre[0])     # the plan changed under it (requests were dropped): its result is not used
+            if self.kv.state_slots and set(pre[1]) & set(decode):
+                raise RuntimeError("a decode step that is not used has already moved its sequences' recurrent state on")
             pre = None
         if decode:
             if pre is not None:

@@ -62,8 +62,11 @@ def mount_weights(engine, artifact_path, rank: int) -> None:
                 raise HotSwapError("the artifacts quantise different projections of a block")
             for name, w8 in old_l.fp8.items():
                 w8.copy_(new_l.fp8[name])
-        for name in ("embed", "final_norm", "lm_head"):
-            _copy_into(getattr(inner.w, name), getattr(fresh, name))
+        for name in ("embed", "final_norm", "lm_head", "loop"):
+            a, b = getattr(inner.w, name), getattr(fresh, name)
+            pairs = zip(_slots(a), _slots(b)) if is_dataclass(a) and is_dataclass(b) else [(a, b)]
+            for old_t, new_t in pairs:
+                _copy_into(old_t, new_t)
     engine.kv.clear_prefix_cache()
     if inner.device.type == "cuda":
         torch.cuda.synchronize(inner.device)

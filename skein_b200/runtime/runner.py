@@ -5,7 +5,7 @@ sampling included) and replayed. A step's host inputs travel in ONE pinned buffe
 host-to-device copy (int32 words; B = bucket size):
 
     [ token ids B | positions B | seq_lens B | temperature B (fp32) | top_k B | top_p B (fp32)
-      | seeds B (64-bit) | block table B x max_blocks ]
+      | seeds B (64-bit) | block table B x max_blocks | state slots B ]
 
 and its result in one device-to-host copy:
 
@@ -61,7 +61,7 @@ def split_by_tokens(lengths, m: int):
 class _Bucket:
     def __init__(self, B: int, max_blocks: int, device):
         self.B, self.max_blocks = B, max_blocks
-        n_in = 8 * B + B * max_blocks
+        n_in = 9 * B + B * max_blocks
         pin = device.type == "cuda"
         self.host_in = torch.zeros(n_in, dtype=torch.int32, pin_memory=pin)
         self.dev_in = torch.zeros(n_in, dtype=torch.int32, device=device)
@@ -78,7 +78,11 @@ class _Bucket:
     def views(self, buf):
         """(token ids, positions, seq_lens, block table) views of a staging buffer."""
         B, mb = self.B, self.max_blocks
-        return buf[:B], buf[B:2 * B], buf[2 * B:3 * B], buf[8 * B:].view(B, mb)
+        return buf[:B], buf[B:2 * B], buf[2 * B:3 * B], buf[8 * B:(8 + mb) * B].view(B, mb)
+
+    def slots_view(self, buf):
+        """State slots of the rows (models with a recurrent state)."""
+        return buf[(8 + self.max_blocks) * self.B:]
 
     def sampling_views(self, buf):
         """(temperature fp32, top_k int32, top_p fp32, seeds int64) views of a staging buffer."""
@@ -111,6 +115,7 @@ class ModelRunner:
         self.max_blocks = max_blocks_per_seq
         self.use_graphs = use_graphs and self.device.type == "cuda"
         self.ctx_hint = ctx_hint
+        self.stateful = getattr(getattr(decoder, "dec", decoder), "num_state_slots", 0) > 0
         self.buckets: dict[int, _Bucket] = {}
         self.graph_captures = 0
         self.graph_replays = 0
@@ -130,7 +135,8 @@ class ModelRunner:
 
     def _decode_body(self, bk: _Bucket, feedback: bool, sampling: bool = False):
         tok, pos, lens, bt = bk.views(bk.dev_in)
-        inp = BatchInputs(token_ids=tok, positions=pos, block_table=bt, seq_lens=lens, ctx_hint=self.ctx_hint)
+        inp = BatchInputs(token_ids=tok, positions=pos, block_table=bt, seq_lens=lens, ctx_hint=self.ctx_hint,
+                          slots=bk.slots_view(bk.dev_in) if self.stateful else None)
         smp = None
         if sampling:
             t, k, p, seeds = bk.sampling_views(bk.dev_in)
@@ -149,6 +155,11 @@ class ModelRunner:
             return g
         # eager warm-up allocates workspaces and descriptor caches outside the capture
         saved = bk.dev_in.clone()
+        if self.stateful:
+            # a recurrent state must not move on twice: warm up on padding rows
+            _, pos, lens, _ = bk.views(bk.dev_in)
+            pos.fill_(-1)
+            lens.zero_()
         self._decode_body(bk, False, sampling)
         torch.cuda.synchronize()
         bk.dev_in.copy_(saved)
@@ -187,10 +198,13 @@ class ModelRunner:
                 break
         return n
 
-    def load_decode_inputs(self, bk: _Bucket, tokens, positions, seq_lens, block_tables, sampling=None):
+    def load_decode_inputs(self, bk: _Bucket, tokens, positions, seq_lens, block_tables, sampling=None, slots=None):
         """Fill the pinned staging buffer from host lists (rows beyond len(tokens) are padding). `sampling` is a
-        list of (temperature, top_k, top_p, seed) per row, or None for an all-greedy step."""
+        list of (temperature, top_k, top_p, seed) per row, or None for an all-greedy step; `slots` the rows' state slots
+        (default: row i uses slot i)."""
         n = len(tokens)
+        if self.stateful:
+            bk.slots_view(bk.host_in)[:n] = torch.as_tensor(list(slots) if slots is not None else list(range(n)), dtype=torch.int32)
         if bk.np_views is None:   # numpy views share the pinned buffer: no tensor objects per row on the hot path
             bk.np_views = tuple(v.numpy() for v in bk.views(bk.host_in)) + tuple(v.numpy() for v in bk.sampling_views(bk.host_in))
         t, p, l, bt, st, sk, sp, ss = bk.np_views
@@ -215,7 +229,8 @@ class ModelRunner:
         """load_decode_inputs for the serving engine: the C++ batcher writes tokens, positions, lengths and block tables of
         the listed requests straight into the pinned staging buffer (one call, no per-row Python objects)."""
         t, p, l, bt = bk.views(bk.host_in)
-        batcher.fill_decode_inputs(ids, t.data_ptr(), p.data_ptr(), l.data_ptr(), bt.data_ptr(), bk.max_blocks, bk.B)
+        batcher.fill_decode_inputs(ids, t.data_ptr(), p.data_ptr(), l.data_ptr(), bt.data_ptr(), bk.max_blocks, bk.B,
+                                   bk.slots_view(bk.host_in).data_ptr() if self.stateful else 0)
         if bk.np_views is None:
             bk.np_views = tuple(v.numpy() for v in bk.views(bk.host_in)) + tuple(v.numpy() for v in bk.sampling_views(bk.host_in))
         st, sk, sp, ss = bk.np_views[4:]
@@ -322,10 +337,11 @@ class ModelRunner:
         """BatchInputs (and SamplingInputs) of one eager chunk holding every new token of every listed sequence. `want` lists, per
         sequence, the places among its new tokens that produce logits (default: the last one)."""
         dev = self.device
-        toks, pos, sot, qs, ql, kl, rows = [], [], [], [], [], [], []
+        toks, pos, sot, qs, ql, kl, rows, slots = [], [], [], [], [], [], [], []
         S = len(seqs)
         bt = torch.zeros(S, self.max_blocks, dtype=torch.int32)
-        for s, (ids, table, cached) in enumerate(seqs):
+        for s, (ids, table, cached, *slot) in enumerate(seqs):
+            slots.append(slot[0] if slot else s)
             qs.append(len(toks)); ql.append(len(ids)); kl.append(cached + len(ids))
             toks.extend(ids); pos.extend(range(cached, cached + len(ids))); sot.extend([s] * len(ids))
             rows.extend([len(toks) - 1] if want is None else [qs[-1] + i for i in want[s]])
@@ -334,7 +350,8 @@ class ModelRunner:
         inp = BatchInputs(token_ids=i32(toks), positions=i32(pos), block_table=bt.to(dev), seq_lens=i32(kl),
                           is_prefill=True, seq_of_token=i32(sot), q_start=i32(qs), q_len=i32(ql), max_q_len=max(ql),
                           logit_rows=torch.tensor(rows, dtype=torch.int64, device=dev), kv_start=i32([sum(kl[:i]) for i in range(S)]),
-                          kv_total=sum(kl), max_cached=max(k - q for k, q in zip(kl, ql)))
+                          kv_total=sum(kl), max_cached=max(k - q for k, q in zip(kl, ql)),
+                          slots=i32(slots) if self.stateful else None)
         smp = None
         if sampling is not None and any(s[0] > 0 for s in sampling):
             smp = SamplingInputs(torch.tensor([s[0] for s in sampling], dtype=torch.float32, device=dev),
@@ -345,12 +362,13 @@ class ModelRunner:
         return inp, smp
 
     def extend(self, seqs, want):
-        """One step that feeds every listed sequence (new_token_ids, block_table_row, cached_len) its new tokens, portions of
+        """One step that feeds every listed sequence (new_token_ids, block_table_row, cached_len[, state slot]) its new tokens, portions of
         prompts beside single decoded tokens, and returns the logits of the wanted places (in order; nothing is sampled). A step
         of single tokens runs as a decode step, captured like the ones of a generation."""
         if all(len(s[0]) == 1 for s in seqs):
             bk = self.bucket(len(seqs))
-            self.load_decode_inputs(bk, [s[0][0] for s in seqs], [s[2] for s in seqs], [s[2] + 1 for s in seqs], [s[1] for s in seqs])
+            self.load_decode_inputs(bk, [s[0][0] for s in seqs], [s[2] for s in seqs], [s[2] + 1 for s in seqs], [s[1] for s in seqs],
+                                    slots=[s[3] for s in seqs] if self.stateful else None)
             self.decode_step(bk)
             lg = bk.graph_logits[(False, False)] if self.use_graphs else bk.logits
             return lg[[i for i, w in enumerate(want) for _ in w]]
@@ -358,7 +376,7 @@ class ModelRunner:
         return self.dec.forward_logits(inp)
 
     def prefill(self, seqs, want_logits: bool = False, sampling=None):
-        """seqs: list of (new_token_ids, block_table_row, cached_len). Runs one eager chunk holding every new
+        """seqs: list of (new_token_ids, block_table_row, cached_len[, state slot]). Runs one eager chunk holding every new
         token of every listed sequence. Returns the next token of every sequence (host list) [and logits]; greedy
         unless `sampling` gives (temperature, top_k, top_p, seed) per sequence. Behind a pipeline of several stages the
         chunk is cut, at sequence boundaries, into one micro-chunk per stage so that the stages overlap."""

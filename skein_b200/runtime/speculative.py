@@ -79,6 +79,8 @@ class SpeculativeDecoder:
         if k < 1:
             raise ValueError("k must be at least 1")
         for dec in (target, draft):
+            if dec.cfg.has_state:
+                raise ValueError(f"{dec.cfg.architecture}: a recurrent state cannot be rolled back to an accepted prefix")
             if dec.cfg.is_layered and dec.cfg.conv_taps > 1:
                 # a rejected proposal leaves its convolution inputs behind in the rows that earlier positions need again
                 raise ValueError(f"{dec.cfg.architecture}: the input convolution's state cannot be rolled back to an accepted prefix")

@@ -16,14 +16,17 @@ import os
 import sys
 
 
+MAX_LIVE = 4          # state slots: most requests that may be live at a time (models with a recurrent state)
+
+
 class TraceSession:
-    """Requests by name over one decoder and a page pool of `max_tokens` tokens."""
+    """Requests by name over one decoder, a page pool of `max_tokens` tokens and (with a recurrent state) MAX_LIVE state slots."""
 
     def __init__(self, decoder, max_tokens: int, use_graphs: bool = True):
         from .. import core
         from .runner import ModelRunner
         self.dec = decoder
-        self.kv = core.KvBlockManager(decoder.num_pages, decoder.page_size, False)
+        self.kv = core.KvBlockManager(decoder.num_pages, decoder.page_size, False, state_slots=decoder.num_state_slots)
         self.runner = ModelRunner(decoder, max(1, -(-max_tokens // decoder.page_size)), use_graphs=use_graphs, ctx_hint=max_tokens)
         self._rid, self._cached, self._next = {}, {}, 1
 
@@ -38,7 +41,7 @@ class TraceSession:
                 self.kv.admit(self._rid[name], tokens)
             else:
                 self.kv.advance(self._rid[name], len(tokens))
-            seqs.append((tokens, self.kv.pages_for(self._rid[name]), self._cached[name]))
+            seqs.append((tokens, self.kv.pages_for(self._rid[name]), self._cached[name], self.kv.slot_of(self._rid[name])))
             wants.append([int(w) for w in want])
         logits = None
         if seqs:
@@ -64,7 +67,7 @@ def open_session(model_dir, dtype: str, max_tokens: int, device) -> TraceSession
     cfg = ModelConfig.from_file(os.path.join(model_dir, "config.json"))
     weights = load_checkpoint(cfg, model_dir, device, getattr(torch, dtype))
     ps = cfg.default_page_size
-    dec = Decoder(cfg, weights, num_pages=max(1, -(-max_tokens // ps)), page_size=ps, max_pos=max_tokens)
+    dec = Decoder(cfg, weights, num_pages=max(1, -(-max_tokens // ps)), page_size=ps, max_pos=max_tokens, state_slots=MAX_LIVE)
     return TraceSession(dec, max_tokens)
 
 
