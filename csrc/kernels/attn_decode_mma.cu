@@ -27,14 +27,12 @@ namespace skein {
 
 constexpr int AM_THREADS = 128;
 constexpr int AM_WARPS = 4;
-constexpr int AM_D = 128;
 constexpr int AM_TILE = 16;                       // tokens per tile
 // cp.async ring depth per warp: 3 (two CTAs per SM, for launches with more CTAs than SMs) or 6 (one CTA per SM gets
 // the whole shared memory: twice the bytes in flight per CTA when there are fewer CTAs than SMs)
-constexpr int AM_TILE_BYTES = AM_TILE * AM_D * 2;  // 4 KB (K or V)
-constexpr int AM_STAGE_BYTES = 2 * AM_TILE_BYTES;  // K then V
-constexpr int am_warp_bytes(int stages) { return stages * AM_STAGE_BYTES; }
-constexpr int am_smem_bytes(int stages) { return AM_WARPS * am_warp_bytes(stages) + AM_TILE_BYTES; }  // + the Q tile
+__host__ __device__ constexpr int am_tile_bytes(int d) { return AM_TILE * d * 2; }                           // K or V (4 KB at head size 128)
+__host__ __device__ constexpr int am_warp_bytes(int stages, int d) { return stages * 2 * am_tile_bytes(d); }    // a stage: K then V
+__host__ __device__ constexpr int am_smem_bytes(int stages, int d) { return AM_WARPS * am_warp_bytes(stages, d) + am_tile_bytes(d); }  // + the Q tile
 constexpr int AM_MAX_SPLITS = 16;
 
 struct AttnMmaParams {
@@ -57,10 +55,15 @@ struct AttnMmaParams {
   const float* cos_sin;     // [max_pos, D/2, 2] fp32
   const int* positions;     // [B] position of the new token, -1 = padding row
   int max_pos;
+  // sliding window: the new token sees the last `window` tokens, itself included (0: all)
+  int window;
+  long long out_ld;         // elements between rows of out
+  float out_scale;
 };
 
-__device__ __forceinline__ uint32_t am_swz(int row, int chunk) {  // byte offset in a [16][128] bf16 tile
-  return (uint32_t)(row * 256 + ((chunk ^ (row & 7)) << 4));
+template <int AM_D>
+__device__ __forceinline__ uint32_t am_swz(int row, int chunk) {  // byte offset in a [16][AM_D] bf16 tile
+  return (uint32_t)(row * (AM_D * 2) + ((chunk ^ (row & 7)) << 4));
 }
 __device__ __forceinline__ void am_ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -87,9 +90,11 @@ __device__ __forceinline__ void am_commit() { asm volatile("cp.async.commit_grou
 template <int N>
 __device__ __forceinline__ void am_wait() { asm volatile("cp.async.wait_group %0;" :: "n"(N) : "memory"); }
 
-template <int AM_STAGES>
+template <int AM_STAGES, int AM_D>
 __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnMmaParams p) {
+  constexpr int AM_TILE_BYTES = am_tile_bytes(AM_D), AM_STAGE_BYTES = 2 * AM_TILE_BYTES;
   constexpr int AM_WARP_BYTES = AM_STAGES * AM_STAGE_BYTES;
+  constexpr int CH = AM_D / 8, KS = AM_D / 16, ND = AM_D / 8;    // 16-byte chunks of a row, k-steps of Q K^T, n-tiles of P V
   extern __shared__ __align__(128) uint8_t am_smem[];
   __shared__ int is_last;
   pdl_trigger();
@@ -99,10 +104,12 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   const int G = p.G, ps = p.page_size;
   const int len = p.seq_lens[b];
 
-  // this split's token range, rounded to whole pages (pages are multiples of the tile)
-  int per = (len + p.splits - 1) / p.splits;
-  per = (per + ps - 1) / ps * ps;
-  const int t_begin = split * per;
+  // this split's token range, rounded to whole pages (pages are multiples of the tile), with a window to whole tiles
+  const int lo = p.window > 0 && len > p.window ? len - p.window : 0;     // first visible token
+  const int base = lo / AM_TILE * AM_TILE, unit = p.window > 0 ? AM_TILE : ps;
+  int per = (len - base + p.splits - 1) / p.splits;
+  per = (per + unit - 1) / unit * unit;
+  const int t_begin = base + split * per;
   int t_end = t_begin + per;
   if (t_end > len) t_end = len;
   const int tile_begin = t_begin / AM_TILE;
@@ -118,13 +125,13 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   int pos = rope ? p.positions[b] : -1;
   if (rope && pos >= p.max_pos) { report_status(p.status, ST_BAD_INDEX, pos); pos = -1; }
   if (!rope) {
-    for (int c = tid; c < AM_TILE * 16; c += AM_THREADS) {
-      const int r = c >> 4, ch = c & 15;
+    for (int c = tid; c < AM_TILE * CH; c += AM_THREADS) {
+      const int r = c / CH, ch = c % CH;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (r < G) v = *reinterpret_cast<const uint4*>(p.q + (size_t)b * p.q_stride + (size_t)(kvh * G + r) * AM_D + ch * 8);
-      *reinterpret_cast<uint4*>(q_s + am_swz(r, ch)) = v;
+      *reinterpret_cast<uint4*>(q_s + am_swz<AM_D>(r, ch)) = v;
     }
-  } else {
+  } else if (AM_D == 128) {
     // rotate-half RoPE: dim i pairs with dim i + 64, i.e. chunk ch with chunk ch + 8; one pair of chunks per thread
     const int r = tid >> 3, ch = tid & 7;
     uint4 lo = make_uint4(0, 0, 0, 0), hi = make_uint4(0, 0, 0, 0);
@@ -143,8 +150,8 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
         hb[i] = __floats2bfloat162_rn(x1.x * c2.x + x0.x * c2.y, x1.y * c2.z + x0.y * c2.w);
       }
     }
-    *reinterpret_cast<uint4*>(q_s + am_swz(r, ch)) = lo;
-    *reinterpret_cast<uint4*>(q_s + am_swz(r, ch + 8)) = hi;
+    *reinterpret_cast<uint4*>(q_s + am_swz<AM_D>(r, ch)) = lo;
+    *reinterpret_cast<uint4*>(q_s + am_swz<AM_D>(r, ch + 8)) = hi;
     // the CTA whose token range holds the new token rotates its K row and appends K and V to the cache;
     // the barrier below orders these stores before the asynchronous copies that read them back
     if (pos >= 0) {
@@ -173,14 +180,14 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     }
   }
   __syncthreads();
-  uint32_t qf[8][4];
+  uint32_t qf[KS][4];
 #pragma unroll
-  for (int ks = 0; ks < 8; ++ks)
-    am_ldsm_x4(q_base + am_swz(lane & 15, ks * 2 + (lane >> 4)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+  for (int ks = 0; ks < KS; ++ks)
+    am_ldsm_x4(q_base + am_swz<AM_D>(lane & 15, ks * 2 + (lane >> 4)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
 
-  float o[16][4];
+  float o[ND][4];
 #pragma unroll
-  for (int i = 0; i < 16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < ND; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
   // ---- the warp's copy pipeline ----
@@ -206,11 +213,11 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
       const __nv_bfloat16* vp = kp + (size_t)p.Hkv * head_stride;
       const uint32_t dst = st_base + (j % AM_STAGES) * AM_STAGE_BYTES;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int c = lane + 32 * i, r = c >> 4, ch = c & 15;
+      for (int i = 0; i < AM_TILE * CH / 32; ++i) {
+        const int c = lane + 32 * i, r = c / CH, ch = c % CH;
         const int nbytes = (tok0 + r < t_end) ? 16 : 0;
-        am_cp_async(dst + am_swz(r, ch), kp + r * AM_D + ch * 8, nbytes);
-        am_cp_async(dst + AM_TILE_BYTES + am_swz(r, ch), vp + r * AM_D + ch * 8, nbytes);
+        am_cp_async(dst + am_swz<AM_D>(r, ch), kp + r * AM_D + ch * 8, nbytes);
+        am_cp_async(dst + AM_TILE_BYTES + am_swz<AM_D>(r, ch), vp + r * AM_D + ch * 8, nbytes);
       }
     }
     am_commit();
@@ -231,9 +238,9 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     s[1][0] = s[1][1] = s[1][2] = s[1][3] = 0.f;
     const int mat = lane >> 3;
 #pragma unroll
-    for (int ks = 0; ks < 8; ++ks) {
+    for (int ks = 0; ks < KS; ++ks) {
       uint32_t b0, b1, b2, b3;
-      am_ldsm_x4(kb + am_swz((mat >> 1) * 8 + (lane & 7), ks * 2 + (mat & 1)), b0, b1, b2, b3);
+      am_ldsm_x4(kb + am_swz<AM_D>((mat >> 1) * 8 + (lane & 7), ks * 2 + (mat & 1)), b0, b1, b2, b3);
       am_mma(s[0], qf[ks], b0, b1);
       am_mma(s[1], qf[ks], b2, b3);
     }
@@ -242,10 +249,10 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
       const int col = tok0 + nb * 8 + (lane & 3) * 2;
-      s[nb][0] = (col < t_end) ? s[nb][0] * p.scale_log2e : -INFINITY;
-      s[nb][1] = (col + 1 < t_end) ? s[nb][1] * p.scale_log2e : -INFINITY;
-      s[nb][2] = (col < t_end) ? s[nb][2] * p.scale_log2e : -INFINITY;
-      s[nb][3] = (col + 1 < t_end) ? s[nb][3] * p.scale_log2e : -INFINITY;
+      s[nb][0] = (col < t_end && col >= lo) ? s[nb][0] * p.scale_log2e : -INFINITY;
+      s[nb][1] = (col + 1 < t_end && col + 1 >= lo) ? s[nb][1] * p.scale_log2e : -INFINITY;
+      s[nb][2] = (col < t_end && col >= lo) ? s[nb][2] * p.scale_log2e : -INFINITY;
+      s[nb][3] = (col + 1 < t_end && col + 1 >= lo) ? s[nb][3] * p.scale_log2e : -INFINITY;
       mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
       mx1 = fmaxf(mx1, fmaxf(s[nb][2], s[nb][3]));
     }
@@ -269,7 +276,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     l1 = l1 * al1 + rs1;
     if (!__all_sync(0xffffffffu, al0 == 1.f && al1 == 1.f)) {   // the running maxima usually settle early
 #pragma unroll
-      for (int i = 0; i < 16; ++i) { o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1; }
+      for (int i = 0; i < ND; ++i) { o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1; }
     }
     // ---- O += P V (one k-step of 16 tokens, 16 n-tiles of 8 dims) ----
     uint32_t a[4];
@@ -278,9 +285,9 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     a[2] = am_pack(s[1][0], s[1][1]);
     a[3] = am_pack(s[1][2], s[1][3]);
 #pragma unroll
-    for (int db = 0; db < 16; db += 2) {
+    for (int db = 0; db < ND; db += 2) {
       uint32_t b0, b1, b2, b3;
-      am_ldsm_x4_t(vb + am_swz((mat & 1) * 8 + (lane & 7), db + (mat >> 1)), b0, b1, b2, b3);
+      am_ldsm_x4_t(vb + am_swz<AM_D>((mat & 1) * 8 + (lane & 7), db + (mat >> 1)), b0, b1, b2, b3);
       am_mma(o[db], a, b0, b1);
       am_mma(o[db + 1], a, b2, b3);
     }
@@ -291,12 +298,12 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   // ---- park each warp's (m, l, O[16][128]) in shared memory ----
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  float* o_w = reinterpret_cast<float*>(am_smem + warp * AM_WARP_BYTES);   // [16][128] fp32 = 8 KB
+  float* o_w = reinterpret_cast<float*>(am_smem + warp * AM_WARP_BYTES);   // [16][AM_D] fp32 (8 KB at head size 128)
   float* ml_w = o_w + 16 * AM_D;                                           // [16][2]
   {
     const int r0 = lane >> 2, r1 = r0 + 8;
 #pragma unroll
-    for (int db = 0; db < 16; ++db) {
+    for (int db = 0; db < ND; ++db) {
       const int d = db * 8 + (lane & 3) * 2;
       *reinterpret_cast<float2*>(&o_w[r0 * AM_D + d]) = make_float2(o[db][0], o[db][1]);
       *reinterpret_cast<float2*>(&o_w[r1 * AM_D + d]) = make_float2(o[db][2], o[db][3]);
@@ -309,7 +316,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   __syncthreads();
 
   // ---- merge the 4 warps: thread d owns output dim d of every head ----
-  const int d = tid;
+  const int d = AM_D < AM_THREADS ? tid % AM_D : tid;   // (head size 64: the second half of the CTA repeats the first)
   float O_g[16], M_g[16], L_g[16];
 #pragma unroll
   for (int g = 0; g < 16; ++g) {
@@ -334,7 +341,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   if (p.splits == 1) {
 #pragma unroll
     for (int g = 0; g < 16; ++g)
-      if (g < G) p.out[((size_t)b * p.Hq + kvh * G + g) * AM_D + d] = __float2bfloat16(L_g[g] > 0.f ? O_g[g] / L_g[g] : 0.f);
+      if (g < G) p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(L_g[g] > 0.f ? O_g[g] / L_g[g] * p.out_scale : 0.f);
     return;
   }
 #pragma unroll
@@ -379,58 +386,77 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
         O += w * ov[s2];
       }
     }
-    p.out[((size_t)b * p.Hq + kvh * G + g) * AM_D + d] = __float2bfloat16(L > 0.f ? O / L : 0.f);
+    p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(L > 0.f ? O / L * p.out_scale : 0.f);
   }
 }
 
 }  // namespace skein
 
-// Same contract as skein_attn_decode (ws / counters from skein_attn_decode_workspace_floats; counters zero at
-// first use). Requires D = 128, page_size a multiple of 16, at most 16 query heads per kv head.
-static int attn_decode_mma_launch(const void* q, long long q_stride, void* kv, const int* block_table,
-                                  const int* seq_lens, void* out, float* ws, int* counters, int* status, int B,
-                                  int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits,
-                                  float scale, const float* cos_sin, const int* positions, int max_pos, void* stream) {
-  using namespace skein;
-  if (B == 0) return 0;
-  if (D != AM_D || Hq % Hkv != 0 || page_size % AM_TILE != 0) return -1;
-  const int G = Hq / Hkv;
-  if (G > 16) return -1;
-  if (splits < 1 || splits > AM_MAX_SPLITS) return -2;
-  if (splits > 1 && (ws == nullptr || counters == nullptr)) return -2;
+namespace skein {
+
+template <int AM_D>
+static int attn_decode_mma_go(AttnMmaParams& p, float* ws, void* stream) {
   static bool attr_set[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -4;
   if (!attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<3>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         am_smem_bytes(3));
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<3, AM_D>, cudaFuncAttributeMaxDynamicSharedMemorySize, am_smem_bytes(3, AM_D));
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_decode_mma_kernel<6>, cudaFuncAttributeMaxDynamicSharedMemorySize, am_smem_bytes(6));
+      e = cudaFuncSetAttribute(attn_decode_mma_kernel<6, AM_D>, cudaFuncAttributeMaxDynamicSharedMemorySize, am_smem_bytes(6, AM_D));
     if (e != cudaSuccess) return (int)e;
     attr_set[dev] = true;
   }
+  p.ws_o = ws;
+  p.ws_ml = ws ? ws + (size_t)p.B * p.Hq * p.splits * AM_D : nullptr;
+  dim3 grid(p.splits, p.Hkv, p.B);
+  int sms = 0;
+  if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
+  if ((long long)p.splits * p.Hkv * p.B <= sms)
+    return (int)launch_pdl(attn_decode_mma_kernel<6, AM_D>, grid, dim3(AM_THREADS), (size_t)am_smem_bytes(6, AM_D), (cudaStream_t)stream, p);
+  return (int)launch_pdl(attn_decode_mma_kernel<3, AM_D>, grid, dim3(AM_THREADS), (size_t)am_smem_bytes(3, AM_D), (cudaStream_t)stream, p);
+}
+
+}  // namespace skein
+
+// Same contract as skein_attn_decode (ws / counters from skein_attn_decode_workspace_floats; counters zero at
+// first use). Requires D = 128 (64 without RoPE fusion), page_size a multiple of 16, at most 16 query heads per kv head.
+static int attn_decode_mma_launch(const void* q, long long q_stride, void* kv, const int* block_table,
+                                  const int* seq_lens, void* out, long long out_ld, float* ws, int* counters, int* status, int B,
+                                  int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits, int window,
+                                  float scale, float out_scale, const float* cos_sin, const int* positions, int max_pos, void* stream) {
+  using namespace skein;
+  if (B == 0) return 0;
+  if ((D != 128 && (D != 64 || cos_sin != nullptr)) || Hq % Hkv != 0 || page_size % AM_TILE != 0) return -1;
+  const int G = Hq / Hkv;
+  if (G > 16 || q_stride % 8 != 0 || (uintptr_t)q % 16 != 0 || (window > 0 && cos_sin != nullptr)) return -1;
+  if (splits < 1 || splits > AM_MAX_SPLITS) return -2;
+  if (splits > 1 && (ws == nullptr || counters == nullptr)) return -2;
   AttnMmaParams p;
   p.q = (const __nv_bfloat16*)q; p.kv = (const __nv_bfloat16*)kv; p.kv_rw = (__nv_bfloat16*)kv;
   p.block_table = block_table; p.seq_lens = seq_lens;
   p.cos_sin = cos_sin; p.positions = positions; p.max_pos = max_pos;
-  p.out = (__nv_bfloat16*)out; p.ws_o = ws; p.ws_ml = ws ? ws + (size_t)B * Hq * splits * AM_D : nullptr;
+  p.out = (__nv_bfloat16*)out; p.out_ld = out_ld; p.out_scale = out_scale;
   p.counters = counters; p.status = status; p.q_stride = q_stride;
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.page_size = page_size; p.max_blocks = max_blocks; p.num_pages = num_pages;
-  p.splits = splits; p.scale_log2e = scale * 1.4426950408889634f;
-  dim3 grid(splits, Hkv, B);
-  int sms = 0;
-  if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
-  if ((long long)splits * Hkv * B <= sms)
-    return (int)launch_pdl(attn_decode_mma_kernel<6>, grid, dim3(AM_THREADS), (size_t)am_smem_bytes(6), (cudaStream_t)stream, p);
-  return (int)launch_pdl(attn_decode_mma_kernel<3>, grid, dim3(AM_THREADS), (size_t)am_smem_bytes(3), (cudaStream_t)stream, p);
+  p.splits = splits; p.scale_log2e = scale * 1.4426950408889634f; p.window = window;
+  return D == 64 ? attn_decode_mma_go<64>(p, ws, stream) : attn_decode_mma_go<128>(p, ws, stream);
 }
 
 extern "C" int skein_attn_decode_mma(const void* q, long long q_stride, const void* kv, const int* block_table,
                                      const int* seq_lens, void* out, float* ws, int* counters, int* status, int B,
                                      int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits,
                                      float scale, void* stream) {
-  return attn_decode_mma_launch(q, q_stride, const_cast<void*>(kv), block_table, seq_lens, out, ws, counters, status, B,
-                                Hq, Hkv, D, page_size, max_blocks, num_pages, splits, scale, nullptr, nullptr, 0, stream);
+  return attn_decode_mma_launch(q, q_stride, const_cast<void*>(kv), block_table, seq_lens, out, (long long)Hq * D, ws, counters, status, B,
+                                Hq, Hkv, D, page_size, max_blocks, num_pages, splits, 0, scale, 1.f, nullptr, nullptr, 0, stream);
+}
+
+// The same over a sliding window, into rows out_ld apart, times out_scale.
+extern "C" int skein_attn_decode_window(const void* q, long long q_stride, const void* kv, const int* block_table,
+                                        const int* seq_lens, void* out, long long out_ld, float* ws, int* counters, int* status, int B,
+                                        int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits, int window,
+                                        float scale, float out_scale, void* stream) {
+  return attn_decode_mma_launch(q, q_stride, const_cast<void*>(kv), block_table, seq_lens, out, out_ld, ws, counters, status, B, Hq, Hkv, D,
+                                page_size, max_blocks, num_pages, splits, window, scale, out_scale, nullptr, nullptr, 0, stream);
 }
 
 // Decode attention straight from the fused q/k/v projection: rotates q and k (rotate-half RoPE from the fp32
@@ -443,6 +469,6 @@ extern "C" int skein_attn_decode_rope_mma(const void* qkv, long long qkv_stride,
                                           int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits,
                                           float scale, void* stream) {
   if (cos_sin == nullptr || positions == nullptr) return -1;
-  return attn_decode_mma_launch(qkv, qkv_stride, kv, block_table, seq_lens, out, ws, counters, status, B, Hq, Hkv, D,
-                                page_size, max_blocks, num_pages, splits, scale, cos_sin, positions, max_pos, stream);
+  return attn_decode_mma_launch(qkv, qkv_stride, kv, block_table, seq_lens, out, (long long)Hq * D, ws, counters, status, B, Hq, Hkv, D,
+                                page_size, max_blocks, num_pages, splits, 0, scale, 1.f, cos_sin, positions, max_pos, stream);
 }

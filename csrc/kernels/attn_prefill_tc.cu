@@ -1,7 +1,8 @@
 // Causal prefill attention over the paged KV cache on the 5th-generation tensor cores (tcgen05, accumulators in
 // tensor memory, operands staged by TMA). Same contract as attn_prefill.cu (chunked-prefill aware: a chunk of q_len
 // new tokens attends to the kv_len tokens already in the cache, its own included); this is the kernel the prefill
-// path runs for head_dim 128 and 16-token pages, the mma.sync kernel stays as the fallback for other shapes.
+// path runs for head sizes 128 and 64 and pages of whole 16-token groups, the mma.sync kernel stays as the fallback for other
+// shapes. With a sliding window a row sees its last `window` keys only; tiles before the window of a CTA's first row are skipped.
 //
 // One CTA = 128 query rows of one head, walking the context in 128-token tiles:
 //
@@ -34,11 +35,10 @@ namespace skein {
 
 int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes, uint32_t box_rows);
 
-constexpr int TC_BM = 128, TC_BN = 128, TC_D = 128, TC_PS = 16;
+constexpr int TC_BM = 128, TC_BN = 128, TC_PS = 16;    // (TC_PS: tokens of one box; a page is a multiple of it)
 constexpr int TC_THREADS = 192;
 constexpr int TC_HALF_BYTES = 128 * 128;              // one 64-element half of a 128-row tile, 128-byte rows
-constexpr int TC_TILE_BYTES = 2 * TC_HALF_BYTES;
-constexpr int TC_SMEM = 3 * TC_TILE_BYTES + 1024 /* alignment slack */ + 256 /* barriers */;
+constexpr int tc_smem(int d) { return 3 * (d / 64) * TC_HALF_BYTES + 1024 /* alignment slack */ + 256 /* barriers */; }
 constexpr int TC_TMEM_COLS = 256;
 constexpr uint64_t TC_BUDGET_NS = 4000000000ull;
 
@@ -49,13 +49,17 @@ struct AttnPrefillTcParams {
   const int* kv_len;        // [S] tokens in the cache after this chunk was appended
   __nv_bfloat16* out;       // [T, Hq * D]
   int* status;
-  int Hq, Hkv, max_blocks, num_pages;
-  float scale_log2e;
+  int Hq, Hkv, max_blocks, num_pages, page_size;
+  int window;               // keys a row sees, its own included (0: all)
+  long long out_ld;         // elements between rows of out
+  float scale_log2e, out_scale;
 };
 
+template <int TC_D>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        const AttnPrefillTcParams p) {
+  constexpr int HALVES = TC_D / 64, TC_TILE_BYTES = HALVES * TC_HALF_BYTES;
   const int qt = (int)gridDim.x - 1 - (int)blockIdx.x;     // long rows first: the causal work grows with the row
   const int head = blockIdx.y, seq = blockIdx.z;
   const int qlen = p.q_len[seq];
@@ -67,7 +71,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int kvh = head / (p.Hq / p.Hkv);
   int kv_hi = pos0 + min(q0 + TC_BM, qlen);                 // exclusive bound of the keys any row of this tile sees
   if (kv_hi > kvlen) kv_hi = kvlen;
-  const int n_tiles = (kv_hi + TC_BN - 1) / TC_BN;
+  const int kv_lo = p.window > 0 && pos0 + q0 - p.window + 1 > 0 ? pos0 + q0 - p.window + 1 : 0;   // first key of the first row
+  const int first_tile = kv_lo / TC_BN;
+  const int n_tiles = (kv_hi + TC_BN - 1) / TC_BN - first_tile;
 
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -104,26 +110,25 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tma_prefetch_desc(&tmKV);
       const uint64_t pol_q = l2_policy_evict_first(), pol_kv = l2_policy_evict_last();
       mbar_expect_tx(bar_q, TC_TILE_BYTES);
-      tma_load_2d(q_s, &tmQ, bar_q, head * TC_D, qrow0 + q0, pol_q);
-      tma_load_2d(q_s + TC_HALF_BYTES, &tmQ, bar_q, head * TC_D + 64, qrow0 + q0, pol_q);
+      for (int hf = 0; hf < HALVES; ++hf) tma_load_2d(q_s + hf * TC_HALF_BYTES, &tmQ, bar_q, head * TC_D + hf * 64, qrow0 + q0, pol_q);
       bool ok = true;
       int armed_k = 0, armed_v = 0;      // phases armed so far (for the bounded drain on an early exit)
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int n0 = j * TC_BN;
-        const int n_pages = (min(kv_hi, n0 + TC_BN) - n0 + TC_PS - 1) / TC_PS;
-        const int* bt = p.block_table + (size_t)seq * p.max_blocks + n0 / TC_PS;
+        const int n0 = (first_tile + j) * TC_BN;
+        const int n_pages = (min(kv_hi, n0 + TC_BN) - n0 + TC_PS - 1) / TC_PS;      // 16-token boxes
+        const int* bt = p.block_table + (size_t)seq * p.max_blocks;
         for (int kv01 = 0; kv01 < 2 && ok; ++kv01) {
           const uint32_t full = kv01 ? bar_vfull : bar_kfull, empty = kv01 ? bar_vempty : bar_kempty;
           const uint32_t dst = kv01 ? v_s : k_s;
           if (j > 0 && !mbar_wait(empty, (j - 1) & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
-          mbar_expect_tx(full, (uint32_t)n_pages * 2 * TC_PS * 128);
+          mbar_expect_tx(full, (uint32_t)n_pages * HALVES * TC_PS * 128);
           if (kv01) ++armed_v; else ++armed_k;
           for (int pg = 0; pg < n_pages; ++pg) {
-            int page = bt[pg];
+            const int tok = n0 + pg * TC_PS;
+            int page = bt[tok / p.page_size];
             if (page < 0 || page >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, page); page = 0; }
-            const int row = ((page * 2 + kv01) * p.Hkv + kvh) * TC_PS;
-            tma_load_2d(dst + pg * TC_PS * 128, &tmKV, full, 0, row, pol_kv);
-            tma_load_2d(dst + TC_HALF_BYTES + pg * TC_PS * 128, &tmKV, full, 64, row, pol_kv);
+            const int row = ((page * 2 + kv01) * p.Hkv + kvh) * p.page_size + tok % p.page_size;
+            for (int hf = 0; hf < HALVES; ++hf) tma_load_2d(dst + hf * TC_HALF_BYTES + pg * TC_PS * 128, &tmKV, full, hf * 64, row, pol_kv);
           }
         }
       }
@@ -153,7 +158,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         if (!mbar_wait(bar_pfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
         if (!mbar_wait(bar_vfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
         tc_fence_after();
-        const int n_valid = min(kv_hi, (j + 1) * TC_BN) - j * TC_BN;
+        const int n_valid = min(kv_hi, (first_tile + j + 1) * TC_BN) - (first_tile + j) * TC_BN;
         const int k_steps = (n_valid + 15) / 16;               // 16-token steps that hold at least one visible key
         for (int k = 0; k < k_steps; ++k)
           mma_f16_ts(tm_o, tm_p + k * 8, umma_desc_sw128_mn(v_s + k * 16 * 128, TC_HALF_BYTES), idesc_o,
@@ -173,11 +178,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
-      const int n0 = j * TC_BN;
+      const int n0 = (first_tile + j) * TC_BN;
       if (!mbar_wait(bar_sfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
       tc_fence_after();
-      const bool masked = n0 + TC_BN - 1 > pos0 + q0;   // some row of the tile sees only part of these keys
-      const int limit = pos_r - n0;                     // this row sees columns 0 .. limit of the tile
+      // some row of the tile sees only part of these keys (the tile's last row has the latest window)
+      const bool masked = n0 + TC_BN - 1 > pos0 + q0 || (p.window > 0 && n0 < pos0 + q0 + TC_BM - p.window);
+      const int limit = pos_r - n0;                     // this row sees columns first .. limit of the tile
+      const int first = p.window > 0 ? pos_r - p.window + 1 - n0 : -1;
       // pass 1: row maximum of the raw scores (64 columns per round: both loads in flight before the wait)
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -188,7 +195,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_wait();
         if (masked) {
 #pragma unroll
-          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], (h * 64 + i <= limit) ? __uint_as_float(sv[i]) : -INFINITY);
+          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], (h * 64 + i <= limit && h * 64 + i >= first) ? __uint_as_float(sv[i]) : -INFINITY);
         } else {
 #pragma unroll
           for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[i]));
@@ -200,6 +207,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // rescaling; the final division by the row sum undoes whatever reference the row ended on.
       const float m_new = (m == -INFINITY || mx > m + 8.f) ? fmaxf(m, mx) : m;
       const float alpha = (m == -INFINITY) ? 1.f : exp2f(m - m_new);
+      const float ref = m_new == -INFINITY ? 0.f : m_new;      // (a row whose window starts in a later tile)
       if (j > 0) {
         // O of the previous tiles is complete in tensor memory; bring it to the new reference if some row moved
         if (!mbar_wait(bar_odone, (j - 1) & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
@@ -231,11 +239,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         uint32_t pk[32];
 #pragma unroll
         for (int i = 0; i < 64; i += 2) {
-          float x0 = fmaf(__uint_as_float(sv[i]), p.scale_log2e, -m_new);
-          float x1 = fmaf(__uint_as_float(sv[i + 1]), p.scale_log2e, -m_new);
+          float x0 = fmaf(__uint_as_float(sv[i]), p.scale_log2e, -ref);
+          float x1 = fmaf(__uint_as_float(sv[i + 1]), p.scale_log2e, -ref);
           if (masked) {
-            if (h * 64 + i > limit) x0 = -INFINITY;
-            if (h * 64 + i + 1 > limit) x1 = -INFINITY;
+            if (h * 64 + i > limit || h * 64 + i < first) x0 = -INFINITY;
+            if (h * 64 + i + 1 > limit || h * 64 + i + 1 < first) x1 = -INFINITY;
           }
           const float p0 = exp2f(x0), p1 = exp2f(x1);
           // the row sum is taken over the rounded values, the ones the tensor cores multiply
@@ -254,12 +262,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         // written); zero them so that 0 * garbage cannot produce a NaN. Needs V landed; a 128-byte row is a
         // permutation of itself under the swizzle, so whole rows can be cleared without computing it.
         if (!mbar_wait(bar_vfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
-        const int first = kv_hi - n0;
-        const int n_rows = ((first + 15) & ~15) - first;        // rows of the last 16-token step past the context
+        const int past = kv_hi - n0;
+        const int n_rows = ((past + 15) & ~15) - past;        // rows of the last 16-token step past the context
         for (int i = r; i < n_rows * 8; i += 128) {              // 16-byte chunks of those rows, per half
-          const uint32_t a = v_s + first * 128 + i * 16;
-          asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(a), "r"(0) : "memory");
-          asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(a + TC_HALF_BYTES), "r"(0) : "memory");
+          const uint32_t a = v_s + past * 128 + i * 16;
+#pragma unroll
+          for (int hf = 0; hf < HALVES; ++hf)
+            asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(a + hf * TC_HALF_BYTES), "r"(0) : "memory");
         }
         fence_proxy_async_smem();
       }
@@ -269,9 +278,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
     if (ok && mbar_wait(bar_odone, (n_tiles - 1) & 1, abort_flag, TC_BUDGET_NS)) {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = l > 0.f ? p.out_scale / l : 0.f;
       const bool store = q0 + r < qlen;
-      __nv_bfloat16* orow = p.out + (size_t)(qrow0 + q0 + r) * ((size_t)p.Hq * TC_D) + (size_t)head * TC_D;
+      __nv_bfloat16* orow = p.out + (size_t)(qrow0 + q0 + r) * p.out_ld + (size_t)head * TC_D;
 #pragma unroll
       for (int c = 0; c < TC_D / 16; ++c) {
         uint32_t ov[16];
@@ -303,32 +312,53 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 }  // namespace skein
 
-// Returns 0, a cudaError_t, or a negative code for shapes this kernel does not take (the caller then uses the
-// mma.sync kernel): head_dim 128, 16-token pages, 16-byte aligned rows.
-extern "C" int skein_attn_prefill_tc(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,
-                                     const int* q_start, const int* q_len, const int* kv_len, void* out, int* status, int S,
-                                     int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages,
-                                     float scale, void* stream) {
-  using namespace skein;
-  if (S == 0 || max_q_len == 0) return 0;
-  if (D != TC_D || page_size != TC_PS || Hq % Hkv != 0 || q_stride % 8 != 0) return -1;
+namespace skein {
+
+template <int TC_D>
+static int attn_prefill_tc_go(const void* q, long long q_stride, long long q_rows, const void* kv, const AttnPrefillTcParams& p, int S, int max_q_len,
+                              void* stream) {
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, TC_SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<TC_D>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(TC_D));
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
   CUtensorMap tmQ, tmKV;
   int rc = cached_tmap_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)q_stride, 2, TC_BM);
   if (rc != 0) return rc;
-  rc = cached_tmap_2d(&tmKV, kv, (uint64_t)num_pages * 2 * Hkv * TC_PS, TC_D, 2, TC_PS);
+  rc = cached_tmap_2d(&tmKV, kv, (uint64_t)p.num_pages * 2 * p.Hkv * p.page_size, TC_D, 2, TC_PS);
   if (rc != 0) return rc;
+  dim3 grid((max_q_len + TC_BM - 1) / TC_BM, p.Hq, S);
+  attn_prefill_tc_kernel<TC_D><<<grid, TC_THREADS, tc_smem(TC_D), (cudaStream_t)stream>>>(tmQ, tmKV, p);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace skein
+
+// Returns 0, a cudaError_t, or a negative code for shapes this kernel does not take (the caller then uses another kernel): head
+// size 128 or 64, pages of whole 16-token groups, 16-byte aligned rows. window 0: none. Rows of out are out_ld apart.
+extern "C" int skein_attn_prefill_window(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,
+                                         const int* q_start, const int* q_len, const int* kv_len, void* out, long long out_ld, int* status, int S,
+                                         int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int window,
+                                         float scale, float out_scale, void* stream) {
+  using namespace skein;
+  if (S == 0 || max_q_len == 0) return 0;
+  if ((D != 128 && D != 64) || page_size % TC_PS != 0 || Hq % Hkv != 0 || q_stride % 8 != 0 || (uintptr_t)q % 16 != 0) return -1;
+  if (out_ld % 8 != 0 || (uintptr_t)out % 16 != 0 || scale <= 0.f) return -1;
   AttnPrefillTcParams p;
   p.block_table = block_table; p.q_start = q_start; p.q_len = q_len; p.kv_len = kv_len;
-  p.out = (__nv_bfloat16*)out; p.status = status;
-  p.Hq = Hq; p.Hkv = Hkv; p.max_blocks = max_blocks; p.num_pages = num_pages;
+  p.out = (__nv_bfloat16*)out; p.status = status; p.out_ld = out_ld; p.out_scale = out_scale; p.window = window;
+  p.Hq = Hq; p.Hkv = Hkv; p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size;
   p.scale_log2e = scale * 1.4426950408889634f;
-  dim3 grid((max_q_len + TC_BM - 1) / TC_BM, Hq, S);
-  attn_prefill_tc_kernel<<<grid, TC_THREADS, TC_SMEM, (cudaStream_t)stream>>>(tmQ, tmKV, p);
-  return (int)cudaGetLastError();
+  return D == 64 ? attn_prefill_tc_go<64>(q, q_stride, q_rows, kv, p, S, max_q_len, stream)
+                 : attn_prefill_tc_go<128>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
+}
+
+extern "C" int skein_attn_prefill_tc(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,
+                                     const int* q_start, const int* q_len, const int* kv_len, void* out, int* status, int S,
+                                     int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages,
+                                     float scale, void* stream) {
+  if (D != 128 || page_size != 16) return -1;
+  return skein_attn_prefill_window(q, q_stride, q_rows, kv, block_table, q_start, q_len, kv_len, out, (long long)Hq * D, status, S, max_q_len, Hq,
+                                   Hkv, D, page_size, max_blocks, num_pages, 0, scale, 1.f, stream);
 }

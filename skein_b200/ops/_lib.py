@@ -154,10 +154,16 @@ def lib():
     _sig(L, "skein_window_append", i32,
          [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
     _sig(L, "skein_window_attn_rows", i32, [vp, i64, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, vp])
+    _sig(L, "skein_attn_decode_window", i32,
+         [vp, i64, vp, vp, vp, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, vp])
+    _sig(L, "skein_attn_prefill_window", i32,
+         [vp, i64, i64, vp, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, vp])
     rec, chunk = C.POINTER(RecParams), C.POINTER(RecChunk)
     _sig(L, "skein_rec_step", i32, [rec, i32, i32, vp])
     _sig(L, "skein_rec_prep", i32, [rec, chunk, i32, i32, vp])
     _sig(L, "skein_rec_scan", i32, [rec, chunk, i32, i32, vp])
+    _sig(L, "skein_rec_tc", i32, [rec, chunk, i32, i32, vp])
+    _sig(L, "skein_rec_tc_scratch_bytes", i64, [rec, i32, i32])
     _sig(L, "skein_rec_tail", i32, [rec, chunk, i32, i32, vp])
     for name, rt, at in _OPTIONAL:
         if hasattr(L, name):

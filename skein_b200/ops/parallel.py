@@ -92,5 +92,27 @@ def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_
 
 
 def window_attn(q, spec, inp, cache, page_size, out, out_scale=1.0):
-    """Attention of a step's rows (a decode step or a chunk) over the cache; the tensor-core kernels where they take the sizes."""
-    return window_attn_rows(q, spec, inp.positions, inp.seq_of_token, inp.block_table, cache, page_size, out, out_scale)
+    """Attention of a step's rows (a decode step or a chunk) over the cache. bf16 heads of 128 or 64 run the tensor-core kernels
+    (a decode step's with up to 16 query heads per key head), everything else the plain one."""
+    tc = (q.is_cuda and q.dtype == torch.bfloat16 and spec.dim == spec.vdim and spec.dim in (64, 128) and page_size % 16 == 0
+          and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0 and spec.scale > 0)
+    if not tc or (not inp.is_prefill and (inp.seq_of_token is not None or spec.heads // spec.kv_heads > 16)):
+        return window_attn_rows(q, spec, inp.positions, inp.seq_of_token, inp.block_table, cache, page_size, out, out_scale)
+    ws, bt, H, K, D = F.workspace(), inp.block_table, spec.heads, spec.kv_heads, spec.dim
+    if inp.is_prefill:
+        rc = _lib.lib().skein_attn_prefill_window(
+            q.data_ptr(), q.stride(0), q.shape[0], cache.data_ptr(), bt.data_ptr(), inp.q_start.data_ptr(), inp.q_len.data_ptr(),
+            inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), ws.status.data_ptr(), inp.q_len.shape[0], int(inp.max_q_len), H, K, D,
+            page_size, bt.stride(0), cache.shape[0], spec.window, float(spec.scale), float(out_scale), _lib.stream_ptr())
+    else:
+        B = q.shape[0]
+        splits = F.pick_splits(B, K, min(inp.ctx_hint, spec.window or inp.ctx_hint), ws.sm_count)
+        scratch = ws.attn_scratch(B, H, K, splits) if splits > 1 else None
+        splits, (wsf, ctr) = (splits, scratch) if scratch is not None else (1, (None, None))
+        rc = _lib.lib().skein_attn_decode_window(
+            q.data_ptr(), q.stride(0), cache.data_ptr(), bt.data_ptr(), inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), _lib.ptr(wsf),
+            _lib.ptr(ctr), ws.status.data_ptr(), B, H, K, D, page_size, bt.stride(0), cache.shape[0], splits, spec.window, float(spec.scale),
+            float(out_scale), _lib.stream_ptr())
+    _lib.check(rc, "window_attn")
+    _lib.count_launch()
+    return out

@@ -13,6 +13,11 @@ import torch
 from . import _lib, functional as F, reference_parallel as rp
 
 KINDS = {"delta": 0, "ssd": 1, "lightning": 2}
+TC_MIN_ROWS = 17         # portions of at least this many rows take the tensor-core form
+
+
+def tc_ok(spec, row) -> bool:
+    return row.is_cuda and row.dtype == torch.bfloat16 and spec.dim in (64, 128) and spec.vdim % 64 == 0
 
 
 @dataclass
@@ -70,8 +75,10 @@ def rec_step(row, cols: RecColumns, spec, w, state: RecState, positions, slots):
     return out
 
 
-def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots, seq_of_token, q_start, q_len, max_q_len):
-    """Portions of several sequences: rows q_start[s] .. + q_len[s] are consecutive tokens of the sequence in slots[s]."""
+def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots, seq_of_token, q_start, q_len, max_q_len, impl=None):
+    """Portions of several sequences, one after another: rows q_start[s] .. + q_len[s] are consecutive tokens of the sequence in
+    slots[s]. impl "tc" (chunks of 64 tokens on the tensor cores; the default for longer portions where it takes the sizes) or
+    "scan" (one token after the other)."""
     T = row.shape[0]
     if not row.is_cuda:
         return rp.rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len)
@@ -88,8 +95,14 @@ def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots,
     c.qkv, c.gates, c.unit = qkv.data_ptr(), gates.data_ptr(), _lib.ptr(unit)
     L, s = _lib.lib(), _lib.stream_ptr()
     _lib.check(L.skein_rec_prep(C.byref(p), C.byref(c), T, fp32, s), "rec_prep")
-    _lib.check(L.skein_rec_scan(C.byref(p), C.byref(c), S, fp32, s), "rec_scan")
-    _lib.count_launch(2)
+    if (impl or ("tc" if max_q_len >= TC_MIN_ROWS else "scan")) == "tc" and tc_ok(spec, row):
+        scratch = torch.empty(int(L.skein_rec_tc_scratch_bytes(C.byref(p), T, S)), dtype=torch.uint8, device=dev)
+        c.chunk_mat = scratch.data_ptr()
+        _lib.check(L.skein_rec_tc(C.byref(p), C.byref(c), T, S, s), "rec_tc")
+        _lib.count_launch(3)
+    else:
+        _lib.check(L.skein_rec_scan(C.byref(p), C.byref(c), S, fp32, s), "rec_scan")
+        _lib.count_launch(2)
     if state.tail is not None:
         _lib.check(L.skein_rec_tail(C.byref(p), C.byref(c), S, fp32, s), "rec_tail")
         _lib.count_launch()
