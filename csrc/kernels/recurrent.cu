@@ -31,7 +31,10 @@ namespace skein {
 constexpr int RS_THREADS = 256, RS_WARPS = 8;
 constexpr int REC_MAX_D = 512;
 
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// the activation behind a projection or convolution; its result is rounded to bf16 in a bf16 model, so there it is computed fast
+template <typename T> __device__ __forceinline__ float silu_act(float z);
+template <> __device__ __forceinline__ float silu_act<float>(float z) { return z / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // log decay and write coefficient of head h from the row's gate columns
@@ -51,16 +54,30 @@ __device__ __forceinline__ int rec_col(const RecParams& p, int ch) {
 }
 
 // Convolution and silu of channel ch of the row at position pos. prev(j): the channel's input j tokens earlier (only asked for
-// where it exists).
-template <typename T, typename F>
+// where it exists). TAPS 0: any number.
+template <typename T, int TAPS, typename F>
 __device__ __forceinline__ float rec_conv(const RecParams& p, int ch, int pos, float cur, F prev) {
-  if (p.kind == REC_LIGHTNING) return to_f<T>(from_f<T>(silu_f(cur)));
+  if (p.kind == REC_LIGHTNING) return to_f<T>(from_f<T>(silu_act<T>(cur)));
   float a = p.conv_b ? p.conv_b[ch] : 0.f;
-  for (int j = p.taps - 1; j > 0; --j)
-    if (pos >= j) a = fmaf(p.conv_w[(size_t)(p.taps - 1 - j) * p.C + ch], prev(j), a);
+  if (TAPS > 0) {
+    float x[TAPS > 0 ? TAPS : 1], w[TAPS > 0 ? TAPS : 1];
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j) {
+      x[j] = pos >= j ? prev(j) : 0.f;
+      w[j] = p.conv_w[(size_t)(TAPS - 1 - j) * p.C + ch];
+    }
+#pragma unroll
+    for (int j = TAPS - 1; j > 0; --j) a = fmaf(w[j], x[j], a);
+  } else {
+    for (int j = p.taps - 1; j > 0; --j)
+      if (pos >= j) a = fmaf(p.conv_w[(size_t)(p.taps - 1 - j) * p.C + ch], prev(j), a);
+  }
   a = fmaf(p.conv_w[(size_t)(p.taps - 1) * p.C + ch], cur, a);
-  return to_f<T>(from_f<T>(silu_f(a)));
+  return to_f<T>(from_f<T>(silu_act<T>(a)));
 }
+
+// row of the convolution's cache that holds the input j tokens before position pos (at = pos mod taps)
+__device__ __forceinline__ int rec_tail_row(int at, int j, int taps) { return at >= j ? at - j : at - j + taps; }
 
 // Sums of two values over the CTA, returned to every thread
 __device__ __forceinline__ float2 rec_block_sum2(float2 v, float2* sh) {
@@ -109,7 +126,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
   for (int i = tid; i < 2 * p.D + ncol; i += RS_THREADS) {
     const int ch = i < p.D ? grp * p.D + i : i < 2 * p.D ? gd + grp * p.D + i - p.D : 2 * gd + h * p.V + tile0 + i - 2 * p.D;
     const float cur = to_f<T>(row[rec_col(p, ch)]);
-    const float x = rec_conv<T>(p, ch, pos, cur, [&](int j) { return to_f<T>(tail[(size_t)((pos - j) % p.taps) * p.C + ch]); });
+    const float x = rec_conv<T, 0>(p, ch, pos, cur, [&](int j) { return to_f<T>(tail[(size_t)((pos - j) % p.taps) * p.C + ch]); });
     // one CTA of those that share a channel keeps its input for the next steps
     if (tail && (i >= 2 * p.D || (blockIdx.x == 0 && h == first_head))) tail[(size_t)(pos % p.taps) * p.C + ch] = from_f<T>(cur);
     if (i < p.D) { q_s[i] = x; sq.x += x * x; }
@@ -167,6 +184,165 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
   }
 }
 
+// The same with the head's whole state (a contiguous block of up to RSB_MAX bytes) brought to shared memory by one bulk copy: few
+// registers, so that three CTAs fit an SM and one's copy runs behind the others' arithmetic. Thread (c, r): columns 4c .. 4c + 3, rows
+// r, r + R, ... with R = 1024 / V. V a power of two from 32 to 256. A CTA takes `heads` heads of a group, whose states lie one after
+// another and whose queries and keys are the same. grid (H / heads, B).
+constexpr int RSB_MAX = 64 * 1024, RSB_HEADS = 8;
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecParams p, const RecGate gt, const int heads) {
+  extern __shared__ __align__(128) float st_s[];       // states [heads][D][V], then u [V], sums [warps][V], v [heads][V], q [D], k [D]
+  float* u_s = st_s + heads * p.D * p.V;
+  float* part = u_s + p.V;
+  float* v_s = part + RS_WARPS * p.V;
+  float* q_s = v_s + heads * p.V;
+  float* k_s = q_s + p.D;
+  __shared__ float2 red[RS_WARPS], red2[RS_WARPS];
+  __shared__ float2 gate_s[RSB_HEADS];
+  __shared__ __align__(8) uint64_t bar;
+  __shared__ int gone;
+  pdl_trigger();
+  pdl_wait();
+  const int h0 = blockIdx.x * heads, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int pos = p.positions[b];
+  if (pos < 0) return;
+  const int slot = p.slots[b];
+  if (slot < 0 || slot >= p.num_slots) { if (tid == 0) report_status(p.status, ST_BAD_INDEX, slot); return; }
+  const int D = p.D, V = p.V, grp = h0 / (p.H / p.G);
+  float* S = p.state + ((size_t)slot * p.H + h0) * D * V;
+  if (tid == 0) {
+    gone = 0;
+    mbar_init(smem_u32(&bar), 1);
+    fence_mbar_init();
+    if (pos > 0) {
+      mbar_expect_tx(smem_u32(&bar), (uint32_t)(heads * D * V * 4));
+      bulk_load_1d(smem_u32(st_s), S, (uint32_t)(heads * D * V * 4), smem_u32(&bar));
+    }
+  }
+  const T* row = (const T*)p.row + (size_t)b * p.ld;
+  T* tail = p.taps > 1 ? (T*)p.tail + (size_t)slot * p.taps * p.C : nullptr;
+  const int gd = p.G * D;
+  if (warp == RS_WARPS - 1 && lane < heads) {
+    float log_g, coef;
+    rec_gates<T>(p, row, h0 + lane, &log_g, &coef);
+    gate_s[lane] = make_float2(expf(log_g), coef);
+  }
+  float2 sq = make_float2(0.f, 0.f);
+  const int at = p.taps > 1 ? pos % p.taps : 0;
+  const bool owner = h0 % (p.H / p.G) == 0;      // of the group's queries and keys
+#pragma unroll 2
+  for (int i = tid; i < 2 * D + heads * V; i += RS_THREADS) {
+    const int ch = i < D ? grp * D + i : i < 2 * D ? gd + grp * D + i - D : 2 * gd + h0 * V + i - 2 * D;
+    const float cur = to_f<T>(row[rec_col(p, ch)]);
+    const float x = rec_conv<T, TAPS>(p, ch, pos, cur, [&](int j) { return to_f<T>(tail[(size_t)rec_tail_row(at, j, p.taps) * p.C + ch]); });
+    if (tail && (i >= 2 * D || owner)) tail[(size_t)at * p.C + ch] = from_f<T>(cur);
+    if (i < D) { q_s[i] = x; sq.x += x * x; }
+    else if (i < 2 * D) { k_s[i - D] = x; sq.y += x * x; }
+    else v_s[i - 2 * D] = x;
+  }
+  sq = rec_block_sum2(sq, red);      // (also the barrier behind what was written above)
+  float rq = 1.f, rk = 1.f;
+  if (p.kind == REC_DELTA) {
+    rq = 1.f / sqrtf(sq.x + 1e-6f) / sqrtf((float)D);
+    rk = 1.f / sqrtf(sq.y + 1e-6f);
+  }
+  float qk = 0.f;
+  for (int n = tid; n < D; n += RS_THREADS) qk = fmaf(q_s[n], k_s[n], qk);
+  qk = rec_block_sum2(make_float2(qk, 0.f), red2).x * rq * rk;
+  if (pos > 0) {
+    if (!mbar_wait(smem_u32(&bar), 0, &gone, 2000000000ull)) { if (tid == 0) report_status(p.status, ST_TIMEOUT_SMEM_FULL, 30); return; }
+  } else {
+    for (int i = tid; i < heads * D * V; i += RS_THREADS) st_s[i] = 0.f;
+    __syncthreads();
+  }
+  const int CG = V / 4, R = RS_THREADS / CG, cg = tid % CG, r0 = tid / CG;
+  // sums per warp, or (V = 256) per pair of warps that share the columns' halves
+  const int pr = CG <= 32 ? warp : r0, np = CG <= 32 ? RS_WARPS : R;
+  for (int hh = 0; hh < heads; ++hh) {
+    const int h = h0 + hh;
+    float* st = st_s + hh * D * V;
+    const float g = gate_s[hh].x, coef = gate_s[hh].y;
+    float4 ks = make_float4(0.f, 0.f, 0.f, 0.f), qs = ks;
+#pragma unroll 4
+    for (int n = r0; n < D; n += R) {
+      const float4 s = *reinterpret_cast<const float4*>(st + n * V + cg * 4);
+      const float kn = k_s[n], qn = q_s[n];
+      ks.x = fmaf(kn, s.x, ks.x); ks.y = fmaf(kn, s.y, ks.y); ks.z = fmaf(kn, s.z, ks.z); ks.w = fmaf(kn, s.w, ks.w);
+      qs.x = fmaf(qn, s.x, qs.x); qs.y = fmaf(qn, s.y, qs.y); qs.z = fmaf(qn, s.z, qs.z); qs.w = fmaf(qn, s.w, qs.w);
+    }
+    for (int o = CG; o < 32; o <<= 1) {      // several row groups in a warp
+      ks.x += __shfl_xor_sync(0xffffffffu, ks.x, o); ks.y += __shfl_xor_sync(0xffffffffu, ks.y, o);
+      ks.z += __shfl_xor_sync(0xffffffffu, ks.z, o); ks.w += __shfl_xor_sync(0xffffffffu, ks.w, o);
+      qs.x += __shfl_xor_sync(0xffffffffu, qs.x, o); qs.y += __shfl_xor_sync(0xffffffffu, qs.y, o);
+      qs.z += __shfl_xor_sync(0xffffffffu, qs.z, o); qs.w += __shfl_xor_sync(0xffffffffu, qs.w, o);
+    }
+    const bool writes = CG > 32 || lane < CG;
+    float a = 0.f, y = 0.f;
+    if (p.kind == REC_DELTA) {               // only the correction needs S^T k
+      if (writes) *reinterpret_cast<float4*>(part + pr * V + cg * 4) = ks;
+      __syncthreads();
+      if (tid < V) for (int w = 0; w < np; ++w) a += part[w * V + tid];
+      __syncthreads();
+    }
+    if (writes) *reinterpret_cast<float4*>(part + pr * V + cg * 4) = qs;
+    __syncthreads();
+    float o = 0.f;
+    if (tid < V) {
+      for (int w = 0; w < np; ++w) y += part[w * V + tid];
+      const float v = v_s[hh * V + tid];
+      const float u = p.kind == REC_DELTA ? coef * (v - g * rk * a) : coef * v;
+      u_s[tid] = u * rk;
+      o = g * rq * y + qk * u + (p.skip ? p.skip[h] * v : 0.f);
+      if (gt.out == nullptr) ((T*)p.out)[(size_t)b * p.H * V + (size_t)h * V + tid] = from_f<T>(o);
+    }
+    if (gt.out != nullptr) {
+      // the head's own norm and gate
+      const float r = 1.f / sqrtf(rec_block_sum2(make_float2(o * o, 0.f), red).x / (float)V + gt.eps);      // (a barrier behind u_s too)
+      if (tid < V) {
+        const float z = to_f<T>(row[gt.gate_col + h * V + tid]);
+        ((T*)gt.out)[(size_t)b * gt.out_ld + (size_t)h * V + tid] = from_f<T>(o * r * gt.norm[tid] * (z / (1.f + expf(-z))) * gt.scale);
+      }
+    } else {
+      __syncthreads();
+    }
+    const float4 u4 = *reinterpret_cast<const float4*>(u_s + cg * 4);
+#pragma unroll 4
+    for (int n = r0; n < D; n += R) {
+      float4 s = *reinterpret_cast<const float4*>(st + n * V + cg * 4);
+      const float kn = k_s[n];
+      s.x = fmaf(g, s.x, kn * u4.x); s.y = fmaf(g, s.y, kn * u4.y); s.z = fmaf(g, s.z, kn * u4.z); s.w = fmaf(g, s.w, kn * u4.w);
+      *reinterpret_cast<float4*>(S + (size_t)hh * D * V + (size_t)n * V + cg * 4) = s;
+    }
+    if (hh + 1 < heads) __syncthreads();     // u, the sums and the reduction's scratch are used again
+  }
+}
+
+template <typename T, int TAPS>
+static int rec_step_bulk_go(const RecParams& p, const RecGate& g, int B, cudaStream_t s) {
+  int heads = RSB_HEADS;                     // a power of two that divides the heads of a group; enough CTAs before larger ones
+  while (heads > 1 && ((p.H / p.G) % heads != 0 || (long long)heads * p.D * p.V * 4 > RSB_MAX || (long long)B * p.H / heads < 444)) heads /= 2;
+  const int sm = (heads * p.D * p.V + (RS_WARPS + 1 + heads) * p.V + 2 * p.D) * 4;
+  static bool attr_set = false;
+  if (!attr_set) {
+    cudaError_t e = cudaFuncSetAttribute(rec_step_bulk_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, RSB_MAX + 24 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    attr_set = true;
+  }
+  return (int)launch_pdl(rec_step_bulk_kernel<T, TAPS>, dim3(p.H / heads, B), dim3(RS_THREADS), (size_t)sm, s, p, g, heads);
+}
+
+template <typename T>
+static int rec_step_bulk(const RecParams& p, const RecGate& g, int B, cudaStream_t s) {
+  switch (p.taps) {
+    case 1: return rec_step_bulk_go<T, 1>(p, g, B, s);
+    case 2: return rec_step_bulk_go<T, 2>(p, g, B, s);
+    case 3: return rec_step_bulk_go<T, 3>(p, g, B, s);
+    case 4: return rec_step_bulk_go<T, 4>(p, g, B, s);
+    default: return rec_step_bulk_go<T, 0>(p, g, B, s);
+  }
+}
+
 // ---- chunks ---------------------------------------------------------------------------------------
 // grid T. Convolved q | k | v of one token, its heads' gates and (delta) the factors that make q and k unit vectors.
 template <typename T>
@@ -184,7 +360,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
   const int gd = p.G * p.D, n = 2 * gd + p.H * p.V;
   for (int ch = tid; ch < n; ch += blockDim.x) {
     const int col = rec_col(p, ch);
-    const float x = rec_conv<T>(p, ch, pos, to_f<T>(row[col]), [&](int j) {
+    const float x = rec_conv<T, 0>(p, ch, pos, to_f<T>(row[col]), [&](int j) {
       return t - j >= first ? to_f<T>(row[col - (long long)j * p.ld]) : to_f<T>(tail[(size_t)((pos - j) % p.taps) * p.C + ch]);
     });
     out[ch < 2 * gd ? ch : ch - 2 * gd + c.v_off] = from_f<T>(x);
@@ -203,6 +379,117 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
     for (int d = tid & 31; d < p.D; d += 32) { const float x = qk_s[(size_t)u * p.D + d]; ss = fmaf(x, x, ss); }
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if ((tid & 31) == 0) c.unit[(size_t)t * 2 * p.G + u] = 1.f / sqrtf(ss + 1e-6f) / (u < p.G ? sqrtf((float)p.D) : 1.f);
+  }
+}
+
+// The same with 8-byte accesses: a thread takes 4 channels of PV_TOK tokens and keeps the convolution's inputs in registers. Every
+// section starts at a multiple of 4 channels and columns; D / 4 is a power of two up to 32 (delta). The last column of CTAs does the
+// gates. grid (channel blocks + 1, token blocks)
+constexpr int PV_TOK = 32, PV_AHEAD = 8;       // tokens of a thread; loads in flight
+
+__device__ __forceinline__ void unpack4(const uint2& u, float* v) {
+  const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int k = 0; k < 2; ++k) { const float2 f = __bfloat1622float2(b[k]); v[2 * k] = f.x; v[2 * k + 1] = f.y; }
+}
+
+template <int TAPS>      // 1: no convolution ("lightning"), else the taps
+__global__ void __launch_bounds__(256) rec_prep_vec_kernel(const RecParams p, const RecChunk c, int T) {
+  __shared__ int pos_s[PV_TOK], first_s[PV_TOK], slot_s[PV_TOK];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, t0 = blockIdx.y * PV_TOK, nt = min(PV_TOK, T - t0);
+  if ((int)blockIdx.x == (int)gridDim.x - 1) {
+    for (int i = tid; i < nt * p.H; i += 256) {
+      const int t = t0 + i / p.H, h = i % p.H;
+      float log_g, coef;
+      rec_gates<__nv_bfloat16>(p, (const __nv_bfloat16*)p.row + (size_t)t * p.ld, h, &log_g, &coef);
+      reinterpret_cast<float2*>(c.gates)[(size_t)t * p.H + h] = make_float2(log_g, coef);
+    }
+    return;
+  }
+  if (tid < nt) {
+    const int t = t0 + tid, seq = c.seq_of_token[t];
+    int slot = p.slots[seq];
+    if (slot < 0 || slot >= p.num_slots) { report_status(p.status, ST_BAD_INDEX, slot); slot = 0; }
+    pos_s[tid] = p.positions[t];
+    first_s[tid] = c.q_start[seq];
+    slot_s[tid] = slot;
+  }
+  __syncthreads();
+  const int gd = p.G * p.D, n4 = (2 * gd + p.H * p.V) / 4, g4 = blockIdx.x * 256 + tid;
+  const bool live = g4 < n4;
+  const int ch = (live ? g4 : 0) * 4, col = rec_col(p, ch);
+  const __nv_bfloat16* src = (const __nv_bfloat16*)p.row + (size_t)t0 * p.ld + col;
+  __nv_bfloat16* dst = (__nv_bfloat16*)c.qkv + (size_t)t0 * c.qkv_ld + (ch < 2 * gd ? ch : ch - 2 * gd + c.v_off);
+  float w[TAPS][4], bias[4], x[TAPS][4];      // x[j]: the input j tokens back
+#pragma unroll
+  for (int k = 0; k < 4; ++k) bias[k] = (TAPS > 1 && p.conv_b) ? p.conv_b[ch + k] : 0.f;
+  if (TAPS > 1)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) w[j][k] = p.conv_w[(size_t)(TAPS - 1 - j) * p.C + ch + k];
+  const int lanes = p.D / 4;
+  uint2 next[PV_AHEAD], cur[PV_AHEAD];
+  auto load = [&](int i0) {
+#pragma unroll
+    for (int a = 0; a < PV_AHEAD; ++a)
+      if (i0 + a < nt) next[a] = *reinterpret_cast<const uint2*>(src + (long long)(i0 + a) * p.ld);
+  };
+  auto token = [&](int i, const uint2& in) {
+    if (TAPS > 1) {
+      const int t = t0 + i, first = first_s[i], pos = pos_s[i];
+      if (i == 0 || t == first) {
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) {
+          uint2 u = make_uint2(0, 0);
+          if (t - j >= first) u = *reinterpret_cast<const uint2*>(src + (long long)(i - j) * p.ld);
+          else if (pos - j >= 0)
+            u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p.tail + ((size_t)slot_s[i] * TAPS + (pos - j) % TAPS) * p.C + ch);
+          unpack4(u, x[j]);
+        }
+      } else {
+#pragma unroll
+        for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) x[j][k] = x[j - 1][k];
+      }
+    }
+    unpack4(in, x[0]);
+    float y[4], ss = 0.f;
+    uint2 o;
+    __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      float a = TAPS > 1 ? bias[k] : x[0][k];
+      if (TAPS > 1) {
+#pragma unroll
+        for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][k], x[j][k], a);
+      }
+      y[k] = silu_act<__nv_bfloat16>(a);
+    }
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      ob[k] = __floats2bfloat162_rn(y[2 * k], y[2 * k + 1]);
+      const float2 f = __bfloat1622float2(ob[k]);
+      ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
+    }
+    if (live) *reinterpret_cast<uint2*>(dst + (long long)i * c.qkv_ld) = o;
+    if (p.kind == REC_DELTA) {
+      for (int s = 1; s < lanes; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+      if (live && ch < 2 * gd && g4 % lanes == 0)
+        c.unit[(size_t)(t0 + i) * 2 * p.G + ch / p.D] = 1.f / sqrtf(ss + 1e-6f) / (ch < gd ? sqrtf((float)p.D) : 1.f);
+    }
+  };
+  load(0);
+  for (int i0 = 0; i0 < nt; i0 += PV_AHEAD) {
+#pragma unroll
+    for (int a = 0; a < PV_AHEAD; ++a) cur[a] = next[a];
+    load(i0 + PV_AHEAD);
+#pragma unroll
+    for (int a = 0; a < PV_AHEAD; ++a)
+      if (i0 + a < nt) token(i0 + a, cur[a]);
   }
 }
 
@@ -353,10 +640,21 @@ static int rec_check(const RecParams* p) {
 
 }  // namespace skein
 
-extern "C" int skein_rec_step(const SkeinRecParams* p, int B, int fp32, void* stream) {
+// Whether skein_rec_step applies a head's norm and gate too (a RecGate with out set).
+extern "C" int skein_rec_step_gates(const SkeinRecParams* p) {
+  using namespace skein;
+  const bool pow2 = p->V >= 32 && p->V <= 256 && (p->V & (p->V - 1)) == 0;
+  return pow2 && (long long)p->D * p->V * 4 <= RSB_MAX && p->D * p->V >= 2048 ? 1 : 0;
+}
+
+extern "C" int skein_rec_step(const SkeinRecParams* p, const SkeinRecGate* g, int B, int fp32, void* stream) {
   using namespace skein;
   if (B == 0) return 0;
   if (int e = rec_check(p)) return e;
+  // small batches of large states: more, smaller CTAs
+  const bool bulk = skein_rec_step_gates(p) && (g->out != nullptr || (long long)B * p->H >= 148);
+  if (bulk) return fp32 ? rec_step_bulk<float>(*p, *g, B, (cudaStream_t)stream) : rec_step_bulk<__nv_bfloat16>(*p, *g, B, (cudaStream_t)stream);
+  if (g->out != nullptr) return -1;
   return fp32 ? rec_step_any<float>(*p, B, (cudaStream_t)stream) : rec_step_any<__nv_bfloat16>(*p, B, (cudaStream_t)stream);
 }
 
@@ -364,6 +662,20 @@ extern "C" int skein_rec_prep(const SkeinRecParams* p, const SkeinRecChunk* c, i
   using namespace skein;
   if (T == 0) return 0;
   if (int e = rec_check(p)) return e;
+  const int lanes = p->D / 4;
+  const bool vec = !fp32 && p->D % 4 == 0 && p->V % 4 == 0 && p->ld % 4 == 0 && p->q_col % 4 == 0 && p->k_col % 4 == 0 && p->v_col % 4 == 0 &&
+                   c->qkv_ld % 4 == 0 && c->v_off % 4 == 0 && p->taps <= 4 && (p->kind == REC_LIGHTNING || p->taps > 1) && (uintptr_t)p->row % 16 == 0 &&
+                   (p->kind != REC_DELTA || (lanes <= 32 && (lanes & (lanes - 1)) == 0));
+  if (vec) {
+    const dim3 grid(((2 * p->G * p->D + p->H * p->V) / 4 + 255) / 256 + 1, (T + PV_TOK - 1) / PV_TOK);
+    auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(256), 0, (cudaStream_t)stream, *p, *c, T); };
+    switch (p->kind == REC_LIGHTNING ? 1 : p->taps) {
+      case 1: return go(rec_prep_vec_kernel<1>);
+      case 2: return go(rec_prep_vec_kernel<2>);
+      case 3: return go(rec_prep_vec_kernel<3>);
+      default: return go(rec_prep_vec_kernel<4>);
+    }
+  }
   const size_t sm = p->kind == REC_DELTA ? (size_t)2 * p->G * p->D * 4 : 0;
   if (sm > 200 * 1024) return -1;
   auto go = [&](auto fn) -> int {

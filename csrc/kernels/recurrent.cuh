@@ -39,10 +39,21 @@ typedef struct SkeinRecChunk {
   int32_t max_q_len;
 } SkeinRecChunk;
 
+// A head's output norm and gate (delta): o / rms(o) * norm * silu(row[gate_col + ...]) * scale into out; out null: not applied.
+typedef struct SkeinRecGate {
+  const float* norm;         // [V]
+  void* out;                 // [rows, out_ld]
+  int64_t out_ld;
+  int32_t gate_col;
+  float eps, scale;
+  int32_t pad;
+} SkeinRecGate;
+
 }  // extern "C"
 
 namespace skein {
 enum : int { REC_DELTA = 0, REC_SSD = 1, REC_LIGHTNING = 2 };
 using RecParams = SkeinRecParams;
 using RecChunk = SkeinRecChunk;
+using RecGate = SkeinRecGate;
 }  // namespace skein

@@ -58,27 +58,73 @@ __device__ __forceinline__ void rt_mma(float* c, const uint32_t* a, uint32_t b0,
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-constexpr int rt_mats_smem(int d, bool delta) { return 2 * RT_C * (d + 8) * 2 + (delta ? 3 * RT_C * (RT_C + 1) * 4 : 0); }
+__device__ __forceinline__ void rt_ldsm2t(uint32_t addr, uint32_t* r) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+}
 
-// grid (chunks, H, S), 256 threads
+constexpr int RT_LX = RT_C + 8, RT_LY = 40;    // row lengths of the 64-wide and 32-wide bf16 scratch matrices
+__host__ __device__ constexpr int rt_kq_bytes(int d) { return 2 * RT_C * (d + 8) * 2; }
+// K and Q, whose place X and Y take later; then A
+__host__ __device__ constexpr int rt_mats_smem(int d, bool delta) {
+  return (!delta || rt_kq_bytes(d) > 2 * RT_C * RT_LX * 2 + 2 * 32 * RT_LY * 2 ? rt_kq_bytes(d) : 2 * RT_C * RT_LX * 2 + 2 * 32 * RT_LY * 2) +
+         (delta ? 2 * RT_C * RT_LX * 2 + RT_C * 17 * 4 : 0);
+}
+
+// One 16 x 8 tile of L R with both factors as hi + lo: acc over `ks` steps of 16. l, r: shared-memory addresses of the tile's
+// rows in the hi parts; the lo parts lie l_lo, r_lo bytes further.
+__device__ __forceinline__ void rt_tile(float* acc, uint32_t l, uint32_t l_lo, int l_ld, uint32_t r, uint32_t r_lo, int r_ld, int ks) {
+  const int lane = threadIdx.x & 31;
+  acc[0] = acc[1] = acc[2] = acc[3] = 0.f;
+  for (int k = 0; k < ks; ++k) {
+    uint32_t ah[4], al[4], bh[2], bl[2];
+    const uint32_t la = l + ((lane & 15) * l_ld + k * 16 + (lane >> 4) * 8) * 2, ra = r + (k * 16 + (lane & 15)) * r_ld * 2;
+    rt_ldsm4(la, ah);
+    rt_ldsm4(la + l_lo, al);
+    rt_ldsm2t(ra, bh);
+    rt_ldsm2t(ra + r_lo, bl);
+    rt_mma(acc, ah, bh[0], bh[1]);
+    rt_mma(acc, al, bh[0], bh[1]);
+    rt_mma(acc, ah, bl[0], bl[1]);
+  }
+}
+
+// a tile's accumulators, negated or not, as hi + lo into a bf16 scratch matrix
+__device__ __forceinline__ void rt_put_tile(const float* acc, float sign, __nv_bfloat16* hi, __nv_bfloat16* lo, int ld) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    uint32_t h, l;
+    rt_split(sign * acc[2 * e], sign * acc[2 * e + 1], h, l);
+    const int at = ((lane >> 2) + 8 * e) * ld + (lane & 3) * 2;
+    *reinterpret_cast<uint32_t*>(hi + at) = h;
+    *reinterpret_cast<uint32_t*>(lo + at) = l;
+  }
+}
+
+constexpr int RT_HB = 8;         // most heads of a CTA
+
+// grid (chunks, H / heads, S), 256 threads: `heads` heads that share queries and keys, whose products are computed once
 template <int D, bool DELTA>
-__global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, const RecChunk c, __nv_bfloat16* mats, float* factors) {
+__global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, const RecChunk c, __nv_bfloat16* mats, float* factors, int heads) {
   extern __shared__ __align__(16) uint8_t mt_smem[];
-  __shared__ float G_s[RT_C], coef_s[RT_C], rq_s[RT_C], rk_s[RT_C];
+  __shared__ float Gh_all[RT_HB][RT_C], Gl_all[RT_HB][RT_C], coef_all[RT_HB][RT_C], rq_s[RT_C], rk_s[RT_C];
   pdl_trigger();
   pdl_wait();
-  const int h = blockIdx.y, seq = blockIdx.z, len = c.q_len[seq], i0 = blockIdx.x * RT_C;
+  const int h0 = blockIdx.y * heads, seq = blockIdx.z, len = c.q_len[seq], i0 = blockIdx.x * RT_C;
   if (i0 >= len) return;
   const int n = min(RT_C, len - i0), q_start = c.q_start[seq], t0 = q_start + i0;
-  const int unit = (rt_chunk0(q_start, seq) + blockIdx.x) * p.H + h;
-  const int grp = h / (p.H / p.G), gd = p.G * D, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int unit0 = (rt_chunk0(q_start, seq) + blockIdx.x) * p.H + h0;
+  const int grp = h0 / (p.H / p.G), gd = p.G * D, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   constexpr int LD = D + 8;
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(mt_smem);
   __nv_bfloat16* q_s = k_s + RT_C * LD;
-  float* A = reinterpret_cast<float*>(q_s + RT_C * LD);      // [64][65]
-  float* X = A + RT_C * (RT_C + 1);
-  float* Y = X + RT_C * (RT_C + 1);
-  constexpr int LA = RT_C + 1;
+  __nv_bfloat16* Xh = k_s;                                   // [64][RT_LX], once K and Q are done with
+  __nv_bfloat16* Xl = Xh + RT_C * RT_LX;
+  __nv_bfloat16* Yh = Xl + RT_C * RT_LX;                     // [32][RT_LY]
+  __nv_bfloat16* Yl = Yh + 32 * RT_LY;
+  __nv_bfloat16* Ah = reinterpret_cast<__nv_bfloat16*>(mt_smem + rt_mats_smem(D, true) - 2 * RT_C * RT_LX * 2 - RT_C * 17 * 4);
+  __nv_bfloat16* Al = Ah + RT_C * RT_LX;
+  float* Ad = reinterpret_cast<float*>(Al + RT_C * RT_LX);   // [64][17] the 16 x 16 blocks on the diagonal
   for (int i = tid; i < RT_C * (D / 8) * 2; i += 256) {
     const int m = i / (RT_C * (D / 8)), r = i % (RT_C * (D / 8)) / (D / 8), ch = i % (D / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -86,41 +132,36 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
     *reinterpret_cast<uint4*>((m ? q_s : k_s) + r * LD + ch * 8) = v;
   }
   if (tid < RT_C) {
-    const bool in = tid < n;
-    const float* gt = c.gates + ((size_t)(t0 + (in ? tid : 0)) * p.H + h) * 2;
-    const float* un = DELTA ? c.unit + (size_t)(t0 + (in ? tid : 0)) * 2 * p.G : nullptr;
-    G_s[tid] = in ? gt[0] : 0.f;
-    coef_s[tid] = in ? gt[1] : 0.f;
+    const float* un = DELTA ? c.unit + (size_t)(t0 + (tid < n ? tid : 0)) * 2 * p.G : nullptr;
     rq_s[tid] = DELTA ? un[grp] : 1.f;
     rk_s[tid] = DELTA ? un[p.G + grp] : 1.f;
   }
-  __syncthreads();
-  if (warp == 0) {      // running sum of the log decays
-    float a = G_s[2 * lane], b = G_s[2 * lane + 1], s = a + b;
-    for (int o = 1; o < 32; o <<= 1) { const float u = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += u; }
-    const float before = __shfl_up_sync(0xffffffffu, s, 1);
-    a += lane > 0 ? before : 0.f;
-    G_s[2 * lane] = a;
-    G_s[2 * lane + 1] = a + b;
-  }
-  __syncthreads();
-  float* f = factors + (size_t)unit * RT_SC;
-  if (tid < RT_C) {
-    const float eg = expf(G_s[tid]), rest = expf(G_s[RT_C - 1] - G_s[tid]);
-    f[tid] = DELTA ? coef_s[tid] : 1.f;
-    f[RT_C + tid] = eg * rk_s[tid];
-    f[2 * RT_C + tid] = eg * rq_s[tid];
-    f[3 * RT_C + tid] = tid < n ? rest * rk_s[tid] * (DELTA ? 1.f : coef_s[tid]) : 0.f;
-    f[4 * RT_C + tid] = expf(G_s[RT_C - 1]);
-  }
-  __nv_bfloat16* out = mats + (size_t)unit * (DELTA ? 3 : 1) * RT_C * RT_C;
-  {
-    // K K^T by warps 0-3 and Q K^T by warps 4-7 (without K K^T: two warps per 16 rows of Q K^T), 16 rows each
-    const bool qk = !DELTA || warp >= 4;
-    const int r0 = 16 * (warp & 3), nb0 = DELTA ? 0 : 4 * (warp >> 2), nbn = DELTA ? 8 : 4;
-    float acc[8][4];
+  if (warp < heads) {      // a warp per head: running sum of the log decays, whose differences must keep the accuracy of 32-bit
+    const float2* gt = reinterpret_cast<const float2*>(c.gates) + h0 + warp;
+    const float2 g0 = 2 * lane < n ? gt[(size_t)(t0 + 2 * lane) * p.H] : make_float2(0.f, 0.f);
+    const float2 g1 = 2 * lane + 1 < n ? gt[(size_t)(t0 + 2 * lane + 1) * p.H] : make_float2(0.f, 0.f);
+    double a = g0.x, b = g1.x, s = a + b;
+    for (int o = 1; o < 32; o <<= 1) { const double u = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += u; }
+    const double before = __shfl_up_sync(0xffffffffu, s, 1);
+    a += lane > 0 ? before : 0.0;
+    b += a;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int e = 0; e < 2; ++e) {
+      const double g = (e ? b : a) * 1.4426950408889634;      // base 2 from here
+      Gh_all[warp][2 * lane + e] = (float)g;
+      Gl_all[warp][2 * lane + e] = (float)(g - (double)(float)g);
+      coef_all[warp][2 * lane + e] = e ? g1.y : g0.y;
+    }
+  }
+  __syncthreads();
+  // K K^T by warps 0-3 and Q K^T by warps 4-7 (without K K^T: two warps per 16 rows of Q K^T), 16 rows each
+  const bool qk = !DELTA || warp >= 4;
+  const int blk = warp & 3, r0 = 16 * blk, nb0 = DELTA ? 0 : 4 * (warp >> 2);
+  constexpr int nbn = DELTA ? 8 : 4;
+  float prod[nbn][4];
+#pragma unroll
+  for (int i = 0; i < nbn; ++i) prod[i][0] = prod[i][1] = prod[i][2] = prod[i][3] = 0.f;
+  {
     const uint32_t a_base = smem_u32(qk ? q_s : k_s), b_base = smem_u32(k_s);
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks) {
@@ -128,93 +169,130 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
       rt_ldsm4(a_base + ((r0 + (lane & 15)) * LD + ks * 16 + (lane >> 4) * 8) * 2, a);
 #pragma unroll
       for (int nb = 0; nb < nbn; nb += 2) {
+        if ((nb0 + nb) * 8 > r0 + 15) continue;       // above the diagonal
         const int mat = lane >> 3;
         uint32_t b[4];
         rt_ldsm4(b_base + (((nb0 + nb) * 8 + (mat >> 1) * 8 + (lane & 7)) * LD + ks * 16 + (mat & 1) * 8) * 2, b);
-        rt_mma(acc[nb], a, b[0], b[1]);
-        rt_mma(acc[nb + 1], a, b[2], b[3]);
+        rt_mma(prod[nb], a, b[0], b[1]);
+        rt_mma(prod[nb + 1], a, b[2], b[3]);
       }
     }
+  }
+  for (int hh = 0; hh < heads; ++hh) {
+    const float *Gh_s = Gh_all[hh], *Gl_s = Gl_all[hh], *coef_s = coef_all[hh];
+    auto decay = [&](int i, int j) { return exp2f((Gh_s[i] - Gh_s[j]) + (Gl_s[i] - Gl_s[j])); };      // e^(G_i - G_j)
+    const int unit = unit0 + hh;
+    float* f = factors + (size_t)unit * RT_SC;
+    if (tid < RT_C) {
+      const float eg = exp2f(Gh_s[tid]);
+      f[tid] = DELTA ? coef_s[tid] : 1.f;
+      f[RT_C + tid] = eg * rk_s[tid];
+      f[2 * RT_C + tid] = eg * rq_s[tid];
+      f[3 * RT_C + tid] = tid < n ? decay(n - 1, tid) * rk_s[tid] * (DELTA ? 1.f : coef_s[tid]) : 0.f;
+      f[4 * RT_C + tid] = exp2f(Gh_s[n - 1]);
+    }
+    __nv_bfloat16* out = mats + (size_t)unit * (DELTA ? 3 : 1) * RT_C * RT_C;
+    if (DELTA && hh > 0) __syncthreads();        // the previous head's X has been read
 #pragma unroll
     for (int nb = 0; nb < nbn; ++nb)
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
         const int i = r0 + (lane >> 2) + 8 * hf, j = (nb0 + nb) * 8 + (lane & 3) * 2;
-        float v[2];
+        float v[2] = {0.f, 0.f};
+        if ((nb0 + nb) * 8 <= r0 + 15) {
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int jj = j + e;
-          const bool in = qk ? jj <= i : jj < i;
-          const float w = in ? expf(G_s[i] - G_s[jj]) * rk_s[jj] * (qk ? rq_s[i] * (DELTA ? 1.f : coef_s[jj]) : rk_s[i] * coef_s[i]) : 0.f;
-          v[e] = in && i < n ? acc[nb][2 * hf + e] * w : 0.f;
+          for (int e = 0; e < 2; ++e) {
+            const int jj = j + e;
+            if (i < n && (qk ? jj <= i : jj < i))
+              v[e] = prod[nb][2 * hf + e] * decay(i, jj) * rk_s[jj] * (qk ? rq_s[i] * (DELTA ? 1.f : coef_s[jj]) : rk_s[i] * coef_s[i]);
+          }
         }
-        if (qk) *reinterpret_cast<uint32_t*>(out + (DELTA ? 2 : 0) * RT_C * RT_C + i * RT_C + j) = rt_pack(v[0], v[1]);
-        else { A[i * LA + j] = v[0]; A[i * LA + j + 1] = v[1]; }
-      }
-  }
-  if (!DELTA) return;
-  __syncthreads();
-  // X = (I + A)^-1: the 16 x 16 blocks on the diagonal by substitution, then blocks of 32 and 64 from two of half the size,
-  // [[a, 0], [b, d]]^-1 = [[a^-1, 0], [-d^-1 b a^-1, d^-1]]
-  for (int i = tid; i < RT_C * LA; i += 256) X[i] = 0.f;
-  __syncthreads();
-  if (tid < RT_C) {
-    const int b0 = tid & ~15, col = tid & 15;
-    float x[16];
-#pragma unroll
-    for (int r = 0; r < 16; ++r) {
-      float s = r == col ? 1.f : 0.f;
-#pragma unroll
-      for (int m = 0; m < r; ++m) s = fmaf(-A[(b0 + r) * LA + b0 + m], x[m], s);
-      x[r] = s;
-    }
-#pragma unroll
-    for (int r = 0; r < 16; ++r) X[(b0 + r) * LA + b0 + col] = x[r];
-  }
-  __syncthreads();
-  for (int sz = 16; sz < RT_C; sz *= 2) {
-    const int pairs = RT_C / (2 * sz), each = sz * sz;
-    for (int pass = 0; pass < 2; ++pass) {
-      for (int i = tid; i < pairs * each; i += 256) {
-        const int b = i / each * 2 * sz, r = i % each / sz, q = i % sz;
-        float s = 0.f;
-        if (pass == 0) {
-          for (int m = 0; m < sz; ++m) s = fmaf(A[(b + sz + r) * LA + b + m], X[(b + m) * LA + b + q], s);
-          Y[(b + r) * LA + q] = s;
-        } else {
-          for (int m = 0; m < sz; ++m) s = fmaf(X[(b + sz + r) * LA + b + sz + m], Y[(b + m) * LA + q], s);
-          X[(b + sz + r) * LA + b + q] = -s;
+        if (qk) {
+          *reinterpret_cast<uint32_t*>(out + (DELTA ? 2 : 0) * RT_C * RT_C + i * RT_C + j) = rt_pack(v[0], v[1]);
+        } else if (nb >> 1 == blk) {
+          Ad[i * 17 + (j & 15)] = v[0];
+          Ad[i * 17 + (j & 15) + 1] = v[1];
+        } else if (nb >> 1 < blk) {
+          uint32_t hi, lo;
+          rt_split(v[0], v[1], hi, lo);
+          *reinterpret_cast<uint32_t*>(Ah + i * RT_LX + j) = hi;
+          *reinterpret_cast<uint32_t*>(Al + i * RT_LX + j) = lo;
         }
       }
-      __syncthreads();
+    if (!DELTA) continue;
+    __syncthreads();
+    // X = (I + A)^-1: the 16 x 16 blocks on the diagonal by substitution, then blocks of 32 and 64 from two of half the size,
+    // [[a, 0], [b, d]]^-1 = [[a^-1, 0], [-d^-1 b a^-1, d^-1]]
+    for (int i = tid; i < 2 * RT_C * RT_LX / 8; i += 256) reinterpret_cast<uint4*>(Xh)[i] = make_uint4(0, 0, 0, 0);
+    __syncthreads();
+    if (tid < RT_C) {
+      const int b0 = tid & ~15, col = tid & 15;
+      float x[16];
+  #pragma unroll
+      for (int r = 0; r < 16; ++r) {
+        float s = r == col ? 1.f : 0.f;
+  #pragma unroll
+        for (int m = 0; m < r; ++m) s = fmaf(-Ad[(b0 + r) * 17 + m], x[m], s);
+        x[r] = s;
+      }
+  #pragma unroll
+      for (int r = 0; r < 16; ++r) {
+        const __nv_bfloat16 hi = __float2bfloat16(x[r]);
+        Xh[(b0 + r) * RT_LX + b0 + col] = hi;
+        Xl[(b0 + r) * RT_LX + b0 + col] = __float2bfloat16(x[r] - __bfloat162float(hi));
+      }
     }
-  }
-  for (int i = tid; i < RT_C * RT_C / 2; i += 256) {
-    const int r = i / (RT_C / 2), q = i % (RT_C / 2) * 2;
-    uint32_t hi, lo;
-    rt_split(X[r * LA + q], X[r * LA + q + 1], hi, lo);
-    reinterpret_cast<uint32_t*>(out)[i] = hi;
-    reinterpret_cast<uint32_t*>(out + RT_C * RT_C)[i] = lo;
+    __syncthreads();
+    constexpr uint32_t X_LO = RT_C * RT_LX * 2, Y_LO = 32 * RT_LY * 2;
+    const uint32_t xa = smem_u32(Xh), aa = smem_u32(Ah), ya = smem_u32(Yh);
+    auto x_at = [&](int r, int q) { return xa + (r * RT_LX + q) * 2; };
+    float acc[4];
+    const int b16 = 32 * (warp >> 1), q16 = 8 * (warp & 1);              // blocks of 32: a warp per 16 x 8 tile
+    if (warp < 4) {
+      rt_tile(acc, aa + ((b16 + 16) * RT_LX + b16) * 2, X_LO, RT_LX, x_at(b16, b16 + q16), X_LO, RT_LX, 1);
+      rt_put_tile(acc, 1.f, Yh + (b16 / 2) * RT_LY + q16, Yl + (b16 / 2) * RT_LY + q16, RT_LY);
+    }
+    __syncthreads();
+    if (warp < 4) {
+      rt_tile(acc, x_at(b16 + 16, b16 + 16), X_LO, RT_LX, ya + ((b16 / 2) * RT_LY + q16) * 2, Y_LO, RT_LY, 1);
+      rt_put_tile(acc, -1.f, Xh + (b16 + 16) * RT_LX + b16 + q16, Xl + (b16 + 16) * RT_LX + b16 + q16, RT_LX);
+    }
+    __syncthreads();
+    const int r32 = 16 * (warp >> 2), q32 = 8 * (warp & 3);              // the block of 64
+    rt_tile(acc, aa + ((32 + r32) * RT_LX) * 2, X_LO, RT_LX, x_at(0, q32), X_LO, RT_LX, 2);
+    rt_put_tile(acc, 1.f, Yh + r32 * RT_LY + q32, Yl + r32 * RT_LY + q32, RT_LY);
+    __syncthreads();
+    rt_tile(acc, x_at(32 + r32, 32), X_LO, RT_LX, ya + q32 * 2, Y_LO, RT_LY, 2);
+    rt_put_tile(acc, -1.f, Xh + (32 + r32) * RT_LX + q32, Xl + (32 + r32) * RT_LX + q32, RT_LX);
+    __syncthreads();
+    for (int i = tid; i < 2 * RT_C * 8; i += 256) {
+      const int m = i / (RT_C * 8), r = i % (RT_C * 8) / 8, ch = i % 8;
+      reinterpret_cast<uint4*>(out)[i] = *reinterpret_cast<const uint4*>((m ? Xl : Xh) + r * RT_LX + ch * 8);
+    }
   }
 }
 
 // ---- the walk over the chunks -------------------------------------------------------------------------
 constexpr int RT_THREADS = 320, RT_COMPUTE = 256;
-__host__ __device__ constexpr int rt_stage_bytes(int d, bool delta) {   // [K | Q] per 64 columns, V, matrices, factors
-  return d / 64 * 2 * RT_C * 128 + 2 * RT_C * 128 + (delta ? 3 : 1) * RT_MAT_BYTES + 2048;
+__host__ __device__ constexpr int rt_stage_bytes(int d, bool delta, bool pair) {   // [K | Q] per 64 columns, V, matrices, factors
+  return d / 64 * 2 * RT_C * 128 + 2 * RT_C * 128 + (delta ? 3 : pair ? 2 : 1) * RT_MAT_BYTES + 3072;
 }
-__host__ __device__ constexpr int rt_smem(int d, bool delta) { return 2 * rt_stage_bytes(d, delta) + 1024 + 256; }
+constexpr int RT_OUT_BYTES = RT_C * 256;      // a chunk's outputs, [64][128] bf16
+__host__ __device__ constexpr int rt_smem(int d, bool delta, bool pair) { return 2 * (rt_stage_bytes(d, delta, pair) + RT_OUT_BYTES) + 1024 + 256; }
 
+// PAIR (no correction, V = 64): the tile's two halves are two neighbouring heads of a group, each with its own P and factors.
+//
 // tensor-memory columns. delta: A operands S (hi, lo), U'; accumulators [R | O1] of one product, U, O2, dS.
 constexpr uint32_t TM_SH = 0, TM_SL = 64, TM_R = 128, TM_O1 = 192, TM_U = 256, TM_O2 = 320, TM_DS = 384;
 
-template <int D, bool DELTA>
+template <int D, bool DELTA, bool PAIR>
 __global__ void __launch_bounds__(RT_THREADS, 1)
 rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmM, const RecParams p, const RecChunk c,
                     const float* factors) {
-  constexpr int HALVES = D / 64, KQ_HALF = 2 * RT_C * 128, STAGE = rt_stage_bytes(D, DELTA), NMAT = DELTA ? 3 : 1;
+  constexpr int HALVES = D / 64, KQ_HALF = 2 * RT_C * 128, STAGE = rt_stage_bytes(D, DELTA, PAIR), NMAT = DELTA ? 3 : PAIR ? 2 : 1;
+  constexpr int MATS = DELTA ? 3 : 1;            // of one head
   constexpr int OFF_V = HALVES * KQ_HALF, OFF_M = OFF_V + 2 * RT_C * 128, OFF_F = OFF_M + NMAT * RT_MAT_BYTES;
-  const int h = blockIdx.y, seq = blockIdx.z, tile0 = blockIdx.x * 128;
+  const int h = blockIdx.y * (PAIR ? 2 : 1), seq = blockIdx.z, tile0 = blockIdx.x * 128;
   const int len = c.q_len[seq], slot = p.slots[seq];
   if (len < 1 || slot < 0 || slot >= p.num_slots) return;
   const int t0 = c.q_start[seq], n_chunks = (len + RT_C - 1) / RT_C, unit0 = rt_chunk0(t0, seq);
@@ -223,11 +301,11 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  const uint32_t bars = base + 2 * STAGE;
+  const uint32_t bars = base + 2 * (STAGE + RT_OUT_BYTES);
   const uint32_t bar_full = bars, bar_empty = bars + 16, bar_s = bars + 32, bar_r = bars + 40, bar_rr = bars + 48, bar_u = bars + 56,
                  bar_ur = bars + 64, bar_o = bars + 72;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + 2 * STAGE + 96);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(base_ptr + 2 * STAGE + 104);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + 2 * (STAGE + RT_OUT_BYTES) + 96);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(base_ptr + 2 * (STAGE + RT_OUT_BYTES) + 104);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (tid == 0) {
@@ -246,7 +324,8 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
   __syncthreads();
   tc_fence_after();
   const uint32_t tm = *tmem_slot;
-  const int v_halves = min(2, (p.V - tile0 + 63) / 64);
+  const int width = PAIR ? 128 : p.V;             // columns of V from tile0's head on
+  const int v_halves = min(2, (width - tile0 + 63) / 64);
 
   if (warp == 0) {
     // ---------------------------------------------------------------- TMA producer
@@ -254,7 +333,7 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       tma_prefetch_desc(&tmX);
       tma_prefetch_desc(&tmM);
       const uint64_t pol = l2_policy_evict_first(), pol_keep = l2_policy_evict_last();
-      const uint32_t bytes = HALVES * KQ_HALF + v_halves * RT_C * 128 + NMAT * RT_MAT_BYTES + RT_SC * 4;
+      const uint32_t bytes = HALVES * KQ_HALF + v_halves * RT_C * 128 + NMAT * RT_MAT_BYTES + (PAIR ? 2 : 1) * RT_SC * 4;
       bool ok = true;
       int armed[2] = {0, 0};
       for (int j = 0; j < n_chunks; ++j) {
@@ -269,8 +348,8 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
           tma_load_2d(st + hf * KQ_HALF + RT_C * 128, &tmX, full, grp * D + hf * 64, row, pol_keep);
         }
         for (int hf = 0; hf < v_halves; ++hf) tma_load_2d(st + OFF_V + hf * RT_C * 128, &tmX, full, c.v_off + h * p.V + tile0 + hf * 64, row, pol);
-        for (int m = 0; m < NMAT; ++m) tma_load_2d(st + OFF_M + m * RT_MAT_BYTES, &tmM, full, 0, (unit * NMAT + m) * RT_C, pol);
-        bulk_load_1d(st + OFF_F, factors + (size_t)unit * RT_SC, RT_SC * 4, full);
+        for (int m = 0; m < NMAT; ++m) tma_load_2d(st + OFF_M + m * RT_MAT_BYTES, &tmM, full, 0, (unit * MATS + m) * RT_C, pol);
+        bulk_load_1d(st + OFF_F, factors + (size_t)unit * RT_SC, (PAIR ? 2 : 1) * RT_SC * 4, full);
       }
       if (!ok) {
         if (*abort_flag == 0) { *abort_flag = 1; report_status(p.status, ST_TIMEOUT_SMEM_EMPTY, 20); }
@@ -300,6 +379,7 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
             mma_f16_ts(tm + (DELTA ? TM_R : TM_O1), tm + (part ? TM_SL : TM_SH) + k * 8, umma_desc_sw128(b), DELTA ? id_2c : id_c,
                        part > 0 || k > 0 ? 1u : 0u);
           }
+        if (PAIR) tc_commit(bar_r);
         if (DELTA) {
           tc_commit(bar_r);
           ok = mbar_wait(bar_rr, j & 1, abort_flag, RT_BUDGET_NS);
@@ -320,29 +400,38 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
         // O2 = U P^T, dS = U' K. Operands: U in R's columns and U' in S's (delta), U in its own and U' in R's (otherwise)
 #pragma unroll
         for (int k = 0; k < RT_C / 16; ++k)
-          mma_f16_ts(tm + TM_O2, tm + (DELTA ? TM_R : TM_U) + k * 8, umma_desc_sw128(st + OFF_M + (NMAT - 1) * RT_MAT_BYTES + k * 32), id_c, k > 0 ? 1u : 0u);
+          mma_f16_ts(tm + TM_O2, tm + (DELTA ? TM_R : TM_U) + k * 8, umma_desc_sw128(st + OFF_M + (MATS - 1) * RT_MAT_BYTES + k * 32), id_c, k > 0 ? 1u : 0u);
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int k = 0; k < RT_C / 16; ++k)
             mma_f16_ts(tm + TM_DS, tm + (DELTA ? TM_SH : TM_R) + part * 32 + k * 8, umma_desc_sw128_mn(st + k * 16 * 128, KQ_HALF), id_d,
                        part > 0 || k > 0 ? 1u : 0u);
+        if (PAIR) {
+          // the second head's O2 takes the place of S as an operand, whose product has to be complete
+          ok = mbar_wait(bar_r, j & 1, abort_flag, RT_BUDGET_NS);
+          if (!ok) break;
+          tc_fence_after();
+#pragma unroll
+          for (int k = 0; k < RT_C / 16; ++k) mma_f16_ts(tm + TM_SH, tm + TM_U + k * 8, umma_desc_sw128(st + OFF_M + RT_MAT_BYTES + k * 32), id_c, k > 0 ? 1u : 0u);
+        }
         tc_commit(bar_o);
       }
       if (!ok && *abort_flag == 0) { *abort_flag = 1; report_status(p.status, ST_TIMEOUT_SMEM_FULL, 21); }
     }
   } else {
     // ---------------------------------------------------------------- state, splits, outputs: thread <-> column of V, half hf
-    const int quarter = warp & 3, hf = (warp - 2) >> 2, v = quarter * 32 + lane, col = tile0 + v;
+    const int quarter = warp & 3, hf = (warp - 2) >> 2, v = quarter * 32 + lane, col = PAIR ? v & 63 : tile0 + v;
+    const int second = PAIR ? v >> 6 : 0, head = h + second;
     const uint32_t ta = tm + ((uint32_t)(quarter * 32) << 16);
     const bool in = col < p.V;
     constexpr int NS = D / 2;               // rows of the state in this thread
-    float* S = p.state + ((size_t)slot * p.H + h) * D * p.V + (size_t)hf * NS * p.V + col;
+    float* S = p.state + ((size_t)slot * p.H + head) * D * p.V + (size_t)hf * NS * p.V + col;
     const bool fresh = p.positions[t0] == 0;
     float s[NS];
 #pragma unroll
     for (int i = 0; i < NS; ++i) s[i] = (in && !fresh) ? S[(size_t)i * p.V] : 0.f;
-    const float skip = p.skip ? p.skip[h] : 0.f;
+    const float skip = p.skip ? p.skip[head] : 0.f;
     auto put_state = [&]() {                // S as an operand, hi and lo
 #pragma unroll
       for (int b = 0; b < NS / 32; ++b) {
@@ -354,24 +443,25 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       }
     };
     const uint32_t v_byte = (uint32_t)(v & 63) * 2;
-    bool ok = true;
-    for (int j = 0; j < n_chunks && ok; ++j) {
-      const int sg = j & 1, n = min(RT_C, len - j * RT_C);
-      const uint8_t* stp = base_ptr + sg * STAGE;
-      const float* f = reinterpret_cast<const float*>(stp + OFF_F);
-      const uint8_t* vs = stp + OFF_V + (v >> 6) * RT_C * 128;
-      auto value = [&](int i) {             // V[token i][col]; 128-byte rows, 16-byte pieces swizzled by the row
-        return __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(vs + i * 128 + (v_byte ^ ((i & 7) << 4))));
-      };
+    const uint32_t v_half = OFF_V + (v >> 6) * RT_C * 128;
+    const int cols = min(128, width - tile0), ct = tid - 64;      // columns of the tile; number of this thread among the 256
+    // V[token i][col] of a stage; 128-byte rows, 16-byte pieces swizzled by the row
+    auto value = [&](int sg, int i) {
+      return __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(base_ptr + sg * STAGE + v_half + i * 128 + (v_byte ^ ((i & 7) << 4))));
+    };
+    auto factor = [&](int sg) { return reinterpret_cast<const float*>(base_ptr + sg * STAGE + OFF_F) + second * RT_SC; };
+    // what chunk j's first products read: S, and without a correction U = V (exact) and U' = V times its factor
+    auto open_chunk = [&](int j) {
       put_state();
-      if (!mbar_wait(bar_full + 8 * sg, (j >> 1) & 1, abort_flag, RT_BUDGET_NS)) { ok = false; break; }
       if (!DELTA) {
-        // U = V (exact) and U' = V times its factor
+        const int sg = j & 1;
+        if (!mbar_wait(bar_full + 8 * sg, (j >> 1) & 1, abort_flag, RT_BUDGET_NS)) return false;
+        const float* f = factor(sg);
         uint32_t u[16], hi[16], lo[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int t = hf * 32 + 2 * i;
-          const float a = value(t), b = value(t + 1);
+          const float a = value(sg, t), b = value(sg, t + 1);
           u[i] = rt_pack(a, b);
           rt_split(a * f[3 * RT_C + t], b * f[3 * RT_C + t + 1], hi[i], lo[i]);
         }
@@ -382,18 +472,27 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(bar_s);
+      return true;
+    };
+    bool ok = open_chunk(0);
+    for (int j = 0; j < n_chunks && ok; ++j) {
+      const int sg = j & 1, n = min(RT_C, len - j * RT_C);
+      const float* f = factor(sg);
       if (DELTA) {
+        if (!mbar_wait(bar_full + 8 * sg, (j >> 1) & 1, abort_flag, RT_BUDGET_NS)) { ok = false; break; }
+        uint32_t r[32], hi[16], lo[16];
+        float x[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) x[i] = value(sg, hf * 32 + i);       // (while the product runs)
         if (!mbar_wait(bar_r, j & 1, abort_flag, RT_BUDGET_NS)) { ok = false; break; }
         tc_fence_after();
-        uint32_t r[32], hi[16], lo[16];
         tmem_ld32(ta + TM_R + hf * 32, r);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int t = hf * 32 + 2 * i;
-          const float a = f[t] * (value(t) - f[RT_C + t] * __uint_as_float(r[2 * i]));
-          const float b = f[t + 1] * (value(t + 1) - f[RT_C + t + 1] * __uint_as_float(r[2 * i + 1]));
-          rt_split(a, b, hi[i], lo[i]);
+          const float2 b2 = *reinterpret_cast<const float2*>(f + t), e2 = *reinterpret_cast<const float2*>(f + RT_C + t);
+          rt_split(b2.x * (x[2 * i] - e2.x * __uint_as_float(r[2 * i])), b2.y * (x[2 * i + 1] - e2.y * __uint_as_float(r[2 * i + 1])), hi[i], lo[i]);
         }
         tmem_st16(ta + TM_O2 + hf * 16, hi);
         tmem_st16(ta + TM_O2 + 32 + hf * 16, lo);
@@ -408,9 +507,10 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int t = hf * 32 + 2 * i;
+          const float2 s2 = *reinterpret_cast<const float2*>(f + 3 * RT_C + t);
           const float a = __uint_as_float(r[2 * i]), b = __uint_as_float(r[2 * i + 1]);
           u[i] = rt_pack(a, b);
-          rt_split(a * f[3 * RT_C + t], b * f[3 * RT_C + t + 1], hi[i], lo[i]);
+          rt_split(a * s2.x, b * s2.y, hi[i], lo[i]);
         }
         tmem_st16(ta + TM_R + hf * 16, u);
         tmem_st16(ta + TM_SH + hf * 16, hi);
@@ -421,6 +521,22 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       }
       if (!mbar_wait(bar_o, j & 1, abort_flag, RT_BUDGET_NS)) { ok = false; break; }
       tc_fence_after();
+      uint32_t o[16];                       // the chunk's outputs of this thread, pairs of tokens
+      {
+        uint32_t o1[32], o2[32];
+        tmem_ld32(ta + TM_O1 + hf * 32, o1);
+        tmem_ld32(ta + (second ? TM_SH : TM_O2) + hf * 32, o2);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const int t = hf * 32 + 2 * i;
+          const float2 e2 = *reinterpret_cast<const float2*>(f + 2 * RT_C + t);
+          float a = fmaf(e2.x, __uint_as_float(o1[2 * i]), __uint_as_float(o2[2 * i]));
+          float b = fmaf(e2.y, __uint_as_float(o1[2 * i + 1]), __uint_as_float(o2[2 * i + 1]));
+          if (!DELTA) { a = fmaf(skip, value(sg, t), a); b = fmaf(skip, value(sg, t + 1), b); }
+          o[i] = rt_pack(a, b);
+        }
+      }
       const float keep = f[4 * RT_C];
 #pragma unroll
       for (int b = 0; b < NS / 32; ++b) {
@@ -430,20 +546,24 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 32; ++i) s[b * 32 + i] = fmaf(keep, s[b * 32 + i], __uint_as_float(d[i]));
       }
-      uint32_t o1[32], o2[32];
-      tmem_ld32(ta + TM_O1 + hf * 32, o1);
-      tmem_ld32(ta + TM_O2 + hf * 32, o2);
-      tmem_ld_wait();
-      __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)(t0 + j * RT_C + hf * 32) * p.H * p.V + (size_t)h * p.V + col;
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const int t = hf * 32 + i;
-        float o = fmaf(f[2 * RT_C + t], __uint_as_float(o1[i]), __uint_as_float(o2[i]));
-        if (!DELTA) o = fmaf(skip, value(t), o);
-        if (in && t < n) out[(size_t)i * p.H * p.V] = __float2bfloat16(o);
-      }
       tc_fence_before();
       mbar_arrive(bar_empty + 8 * sg);
+      if (j + 1 < n_chunks) ok = open_chunk(j + 1);
+      // the outputs go through shared memory to whole 16-byte pieces of the rows, while the next chunk's product runs. Two buffers:
+      // a thread can be one chunk ahead of another here, not two.
+      uint8_t* ob = base_ptr + 2 * STAGE + (j & 1) * RT_OUT_BYTES;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        *reinterpret_cast<uint16_t*>(ob + (hf * 32 + 2 * i) * 256 + v * 2) = (uint16_t)o[i];
+        *reinterpret_cast<uint16_t*>(ob + (hf * 32 + 2 * i + 1) * 256 + v * 2) = (uint16_t)(o[i] >> 16);
+      }
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      __nv_bfloat16* out = (__nv_bfloat16*)p.out + (size_t)(t0 + j * RT_C) * p.H * p.V + (size_t)h * p.V + tile0;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = (ct >> 4) + 16 * i, ch = ct & 15;
+        if (t < n && ch * 8 < cols) *reinterpret_cast<uint4*>(out + (size_t)t * p.H * p.V + ch * 8) = *reinterpret_cast<const uint4*>(ob + t * 256 + ch * 16);
+      }
     }
     if (ok) {
 #pragma unroll
@@ -462,7 +582,7 @@ rec_tc_chunk_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
   }
 }
 
-template <int D, bool DELTA>
+template <int D, bool DELTA, bool PAIR>
 static int rec_tc_go(const RecParams& p, const RecChunk& c, int T, int S, cudaStream_t s) {
   const int units = (T / RT_C + S + 1) * p.H, nmat = DELTA ? 3 : 1;
   __nv_bfloat16* mats = (__nv_bfloat16*)c.chunk_mat;
@@ -470,7 +590,8 @@ static int rec_tc_go(const RecParams& p, const RecChunk& c, int T, int S, cudaSt
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(rec_tc_mats_kernel<D, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, rt_mats_smem(D, DELTA));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(rec_tc_chunk_kernel<D, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, rt_smem(D, DELTA));
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(rec_tc_chunk_kernel<D, DELTA, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, rt_smem(D, DELTA, PAIR));
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
@@ -478,10 +599,13 @@ static int rec_tc_go(const RecParams& p, const RecChunk& c, int T, int S, cudaSt
   int rc = cached_tmap_2d(&tmX, c.qkv, (uint64_t)T, (uint64_t)c.qkv_ld, 2, RT_C);
   if (rc == 0) rc = cached_tmap_2d(&tmM, mats, (uint64_t)units * nmat * RT_C, RT_C, 2, RT_C);
   if (rc != 0) return rc;
-  const dim3 g1((c.max_q_len + RT_C - 1) / RT_C, p.H, S), g2((p.V + 127) / 128, p.H, S);
-  cudaError_t e = launch_pdl(rec_tc_mats_kernel<D, DELTA>, g1, dim3(256), (size_t)rt_mats_smem(D, DELTA), s, p, c, mats, factors);
+  int heads = RT_HB;                            // of a CTA of the first kernel: a power of two that divides the heads of a group
+  while ((p.H / p.G) % heads != 0) heads /= 2;
+  const dim3 g1((c.max_q_len + RT_C - 1) / RT_C, p.H / heads, S), g2(PAIR ? 1 : (p.V + 127) / 128, PAIR ? p.H / 2 : p.H, S);
+  cudaError_t e = launch_pdl(rec_tc_mats_kernel<D, DELTA>, g1, dim3(256), (size_t)rt_mats_smem(D, DELTA), s, p, c, mats, factors, heads);
   if (e != cudaSuccess) return (int)e;
-  return (int)launch_pdl(rec_tc_chunk_kernel<D, DELTA>, g2, dim3(RT_THREADS), (size_t)rt_smem(D, DELTA), s, tmX, tmM, p, c, (const float*)factors);
+  return (int)launch_pdl(rec_tc_chunk_kernel<D, DELTA, PAIR>, g2, dim3(RT_THREADS), (size_t)rt_smem(D, DELTA, PAIR), s, tmX, tmM, p, c,
+                         (const float*)factors);
 }
 
 }  // namespace skein
@@ -499,6 +623,8 @@ extern "C" int skein_rec_tc(const SkeinRecParams* p, const SkeinRecChunk* c, int
   if ((p->D != 64 && p->D != 128) || p->V % 64 != 0 || p->V < 64 || p->H % p->G != 0 || p->H > 65535 || S > 65535) return -1;
   if (c->qkv_ld % 8 != 0 || c->v_off % 8 != 0 || c->chunk_mat == nullptr || (uintptr_t)c->qkv % 16 != 0) return -1;
   cudaStream_t s = (cudaStream_t)stream;
-  if (p->kind == REC_DELTA) return p->D == 64 ? rec_tc_go<64, true>(*p, *c, T, S, s) : rec_tc_go<128, true>(*p, *c, T, S, s);
-  return p->D == 64 ? rec_tc_go<64, false>(*p, *c, T, S, s) : rec_tc_go<128, false>(*p, *c, T, S, s);
+  if (p->kind == REC_DELTA) return p->D == 64 ? rec_tc_go<64, true, false>(*p, *c, T, S, s) : rec_tc_go<128, true, false>(*p, *c, T, S, s);
+  if (p->V == 64 && (p->H / p->G) % 2 == 0)
+    return p->D == 64 ? rec_tc_go<64, false, true>(*p, *c, T, S, s) : rec_tc_go<128, false, true>(*p, *c, T, S, s);
+  return p->D == 64 ? rec_tc_go<64, false, false>(*p, *c, T, S, s) : rec_tc_go<128, false, false>(*p, *c, T, S, s);
 }

@@ -107,11 +107,16 @@ class ParallelOps:
         cols = rec.RecColumns.of(sec.spec, sec.col)
         args = (st.qkv, cols, sec.spec, self.w.layers[li].rec, self.rec_state[li], inp.positions, self._slots(inp))
         if self._decode_rows(inp):
-            st.attn = rec.rec_step(*args)
+            r, gate = sec.spec, None
+            if r.kind == "delta":
+                gate = rec.HeadGate(self.w.layers[li].rec.norm, sec.col["g"], st.qkv[:, sec.out:sec.out + r.out_width], self.cfg.rms_norm_eps, sec.scale)
+            st.attn = rec.rec_step(*args, gate=gate)
         else:
             st.attn = rec.rec_chunk(*args, inp.seq_of_token, inp.q_start, inp.q_len, inp.max_q_len)
 
     def _op_gated_norm(self, st, li):
+        if st.attn is None:
+            return              # applied by the decode step's kernel
         sec = self.layouts[li].part(RecurrentSpec)
         r, w = sec.spec, self.w.layers[li].rec
         g = sec.col["z" if r.kind == "ssd" else "g"]

@@ -48,6 +48,13 @@ class RecParams(C.Structure):
         (n, C.c_int32) for n in ("kind", "H", "G", "D", "V", "taps", "C", "q_col", "k_col", "v_col", "a_col", "b_col", "num_slots")]
 
 
+class RecGate(C.Structure):
+    """Mirror of SkeinRecGate in csrc/kernels/recurrent.cuh (same field order)."""
+
+    _fields_ = [("norm", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_int64), ("gate_col", C.c_int32), ("eps", C.c_float),
+                ("scale", C.c_float), ("pad", C.c_int32)]
+
+
 class RecChunk(C.Structure):
     """Mirror of SkeinRecChunk in csrc/kernels/recurrent.cuh (same field order)."""
 
@@ -159,7 +166,8 @@ def lib():
     _sig(L, "skein_attn_prefill_window", i32,
          [vp, i64, i64, vp, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, vp])
     rec, chunk = C.POINTER(RecParams), C.POINTER(RecChunk)
-    _sig(L, "skein_rec_step", i32, [rec, i32, i32, vp])
+    _sig(L, "skein_rec_step", i32, [rec, C.POINTER(RecGate), i32, i32, vp])
+    _sig(L, "skein_rec_step_gates", i32, [rec])
     _sig(L, "skein_rec_prep", i32, [rec, chunk, i32, i32, vp])
     _sig(L, "skein_rec_scan", i32, [rec, chunk, i32, i32, vp])
     _sig(L, "skein_rec_tc", i32, [rec, chunk, i32, i32, vp])

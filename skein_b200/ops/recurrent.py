@@ -63,16 +63,31 @@ def _params(row, cols, spec, w, state, positions, slots, out) -> "_lib.RecParams
     return p
 
 
-def rec_step(row, cols: RecColumns, spec, w, state: RecState, positions, slots):
-    """One token per sequence: row [B, ld] holds the projections. Returns the read-outs [B, heads * vdim]; the state moves on."""
+@dataclass
+class HeadGate:
+    """Norm and gate of a head's own read-out (delta): o / rms(o) * norm * silu(row[:, col ...]) * scale, into `out` (columns of a
+    wider matrix)."""
+    norm: torch.Tensor
+    col: int
+    out: torch.Tensor
+    eps: float
+    scale: float = 1.0
+
+
+def rec_step(row, cols: RecColumns, spec, w, state: RecState, positions, slots, gate: HeadGate | None = None):
+    """One token per sequence: row [B, ld] holds the projections. Returns the read-outs [B, heads * vdim], or None when the step
+    applied `gate` to them (it does where a kernel holds whole heads); the state moves on."""
     B = row.shape[0]
     if not row.is_cuda:
         return rp.rec_chunk(row, cols, spec, w, state, positions, slots, torch.arange(B), torch.ones(B, dtype=torch.int32))
     out = torch.empty(B, spec.out_width, dtype=row.dtype, device=row.device)
-    p = _params(row, cols, spec, w, state, positions, slots, out)
-    _lib.check(_lib.lib().skein_rec_step(C.byref(p), B, 1 if row.dtype == torch.float32 else 0, _lib.stream_ptr()), "rec_step")
+    p, g = _params(row, cols, spec, w, state, positions, slots, out), _lib.RecGate()
+    L = _lib.lib()
+    if gate is not None and L.skein_rec_step_gates(C.byref(p)):
+        g.norm, g.out, g.out_ld, g.gate_col, g.eps, g.scale = gate.norm.data_ptr(), gate.out.data_ptr(), gate.out.stride(0), gate.col, gate.eps, gate.scale
+    _lib.check(L.skein_rec_step(C.byref(p), C.byref(g), B, 1 if row.dtype == torch.float32 else 0, _lib.stream_ptr()), "rec_step")
     _lib.count_launch()
-    return out
+    return None if g.out else out
 
 
 def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots, seq_of_token, q_start, q_len, max_q_len, impl=None):

@@ -198,6 +198,9 @@ RECS = {
     "ssd": RecurrentSpec("ssd", heads=6, groups=3, dim=20, vdim=16, taps=4, norm_groups=2),
     "ssd128": RecurrentSpec("ssd", heads=4, groups=1, dim=128, vdim=64, taps=4),
     "ssd64": RecurrentSpec("ssd", heads=4, groups=2, dim=64, vdim=128, taps=3),
+    "ssd64_pairs": RecurrentSpec("ssd", heads=12, groups=3, dim=64, vdim=64, taps=4),
+    "ssd_odd_heads": RecurrentSpec("ssd", heads=3, groups=1, dim=128, vdim=64, taps=6),
+    "delta_v256": RecurrentSpec("delta", heads=2, groups=2, dim=64, vdim=256, taps=3),
     "ssd_big": RecurrentSpec("ssd", heads=2, groups=1, dim=300, vdim=33, taps=2),
     "lightning": RecurrentSpec("lightning", heads=3, groups=3, dim=16, vdim=24, decay=(0.5, 0.9, 1.0)),
     "lightning128": RecurrentSpec("lightning", heads=3, groups=3, dim=128, vdim=128, decay=(0.0, 0.97, 0.9995)),
@@ -269,8 +272,9 @@ def test_recurrence_in_portions_and_steps(name, dtype):
         got = run_steps(r, rows, cols, gw, gs, slots, plan, DEV, impl)
         for s in range(len(lens)):
             close(got[s], want[s], dtype, 1.0 if dtype == BF else 3.0)
-            e = (gs.mat[slots[s]].cpu() - st.mat[slots[s]]).abs().max() / st.mat[slots[s]].abs().max()
-            assert e < 2e-4, (plan is whole, impl, s, e)           # the state is 32-bit in every form
+            # the state is 32-bit in every form (a convolved input may round to the other neighbour in bf16)
+            e = (gs.mat[slots[s]].cpu() - st.mat[slots[s]]).norm() / st.mat[slots[s]].norm()
+            assert e < (3e-4 if dtype == BF else 1e-5), (plan is whole, impl, s, e)
             if gs.tail is not None:
                 keep = [p % r.taps for p in range(max(0, lens[s] - r.taps + 1), lens[s])]
                 assert torch.equal(gs.tail[slots[s]].cpu()[keep], st.tail[slots[s]][keep])
@@ -299,7 +303,7 @@ def test_long_recurrence_keeps_an_early_write(name):
     w.neg_decay = torch.full((r.heads,), -1e-4)
     st = rec.RecState.make(r, 1, BF, "cpu")
     want = run_steps(r, [row], cols, w, st, [0], [[(0, n)]], "cpu")[0]
-    lost = run_steps(r, [torch.cat([row[:8] * 0, row[8:]])], cols, w, rec.RecState.make(r, 1, BF, "cpu"), [0], [[(0, n)]], "cpu")[0]
+    lost = run_steps(r, [torch.cat([row[:60] * 0, row[60:]])], cols, w, rec.RecState.make(r, 1, BF, "cpu"), [0], [[(0, n)]], "cpu")[0]
     assert (lost[-20:] - want[-20:]).norm() > 0.02 * want[-20:].norm()
     for plan in ([[(0, n)]], [[(0, 333)], [(0, n - 333 - 30)]] + [[(0, 1)]] * 30):
         gs = rec.RecState.make(r, 1, BF, DEV)
