@@ -382,15 +382,16 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
   }
 }
 
-// The same with 8-byte accesses: a thread takes 4 channels of PV_TOK tokens and keeps the convolution's inputs in registers. Every
-// section starts at a multiple of 4 channels and columns; D / 4 is a power of two up to 32 (delta). The last column of CTAs does the
-// gates. grid (channel blocks + 1, token blocks)
-constexpr int PV_TOK = 32, PV_AHEAD = 8;       // tokens of a thread; loads in flight
+// The same with 16-byte accesses: a thread takes 8 channels of PV_TOK tokens and keeps the convolution's inputs and (bf16) taps packed
+// in registers. Every section starts at a multiple of 8 channels and columns; D / 8 is a power of two up to 32 (delta). The last column
+// of CTAs does the gates. grid (channel blocks + 1, token blocks)
+constexpr int PV_TOK = 32, PV_AHEAD = 4;       // tokens of a thread; loads in flight
 
-__device__ __forceinline__ void unpack4(const uint2& u, float* v) {
-  const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-  for (int k = 0; k < 2; ++k) { const float2 f = __bfloat1622float2(b[k]); v[2 * k] = f.x; v[2 * k + 1] = f.y; }
+__device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
+__device__ __forceinline__ uint32_t bf_pack(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
 }
 
 template <int TAPS>      // 1: no convolution ("lightning"), else the taps
@@ -417,79 +418,74 @@ __global__ void __launch_bounds__(256) rec_prep_vec_kernel(const RecParams p, co
     slot_s[tid] = slot;
   }
   __syncthreads();
-  const int gd = p.G * p.D, n4 = (2 * gd + p.H * p.V) / 4, g4 = blockIdx.x * 256 + tid;
-  const bool live = g4 < n4;
-  const int ch = (live ? g4 : 0) * 4, col = rec_col(p, ch);
+  const int gd = p.G * p.D, n8 = (2 * gd + p.H * p.V) / 8, g8 = blockIdx.x * 256 + tid;
+  const bool live = g8 < n8;
+  const int ch = (live ? g8 : 0) * 8, col = rec_col(p, ch);
   const __nv_bfloat16* src = (const __nv_bfloat16*)p.row + (size_t)t0 * p.ld + col;
   __nv_bfloat16* dst = (__nv_bfloat16*)c.qkv + (size_t)t0 * c.qkv_ld + (ch < 2 * gd ? ch : ch - 2 * gd + c.v_off);
-  float w[TAPS][4], bias[4], x[TAPS][4];      // x[j]: the input j tokens back
-#pragma unroll
-  for (int k = 0; k < 4; ++k) bias[k] = (TAPS > 1 && p.conv_b) ? p.conv_b[ch + k] : 0.f;
+  uint32_t w[TAPS][4];                        // w[j]: the tap j tokens back
+  uint4 x[TAPS];                              // x[j]: the input j tokens back
   if (TAPS > 1)
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-      for (int k = 0; k < 4; ++k) w[j][k] = p.conv_w[(size_t)(TAPS - 1 - j) * p.C + ch + k];
-  const int lanes = p.D / 4;
-  uint2 next[PV_AHEAD], cur[PV_AHEAD];
-  auto load = [&](int i0) {
-#pragma unroll
-    for (int a = 0; a < PV_AHEAD; ++a)
-      if (i0 + a < nt) next[a] = *reinterpret_cast<const uint2*>(src + (long long)(i0 + a) * p.ld);
-  };
-  auto token = [&](int i, const uint2& in) {
+    for (int j = 0; j < TAPS; ++j) {
+      const float4* wp = reinterpret_cast<const float4*>(p.conv_w + (size_t)(TAPS - 1 - j) * p.C + ch);
+      const float4 a = wp[0], b = wp[1];
+      w[j][0] = bf_pack(a.x, a.y); w[j][1] = bf_pack(a.z, a.w); w[j][2] = bf_pack(b.x, b.y); w[j][3] = bf_pack(b.z, b.w);
+    }
+  const int lanes = p.D / 8;
+  auto token = [&](int i, const uint4& in) {
     if (TAPS > 1) {
       const int t = t0 + i, first = first_s[i], pos = pos_s[i];
       if (i == 0 || t == first) {
 #pragma unroll
         for (int j = 1; j < TAPS; ++j) {
-          uint2 u = make_uint2(0, 0);
-          if (t - j >= first) u = *reinterpret_cast<const uint2*>(src + (long long)(i - j) * p.ld);
+          x[j] = make_uint4(0, 0, 0, 0);
+          if (t - j >= first) x[j] = *reinterpret_cast<const uint4*>(src + (long long)(i - j) * p.ld);
           else if (pos - j >= 0)
-            u = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p.tail + ((size_t)slot_s[i] * TAPS + (pos - j) % TAPS) * p.C + ch);
-          unpack4(u, x[j]);
+            x[j] = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.tail + ((size_t)slot_s[i] * TAPS + (pos - j) % TAPS) * p.C + ch);
         }
       } else {
 #pragma unroll
-        for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-          for (int k = 0; k < 4; ++k) x[j][k] = x[j - 1][k];
+        for (int j = TAPS - 1; j > 0; --j) x[j] = x[j - 1];
       }
     }
-    unpack4(in, x[0]);
-    float y[4], ss = 0.f;
-    uint2 o;
-    __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
+    x[0] = in;
+    float ss = 0.f;
+    uint32_t o[4];
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
-      float a = TAPS > 1 ? bias[k] : x[0][k];
+      float a = 0.f, b = 0.f;
       if (TAPS > 1) {
+        if (p.conv_b) { const float2 f = *reinterpret_cast<const float2*>(p.conv_b + ch + 2 * k); a = f.x; b = f.y; }
 #pragma unroll
-        for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][k], x[j][k], a);
+        for (int j = TAPS - 1; j >= 0; --j) {
+          const uint32_t u = k == 0 ? x[j].x : k == 1 ? x[j].y : k == 2 ? x[j].z : x[j].w;
+          a = fmaf(bf_lo(w[j][k]), bf_lo(u), a);
+          b = fmaf(bf_hi(w[j][k]), bf_hi(u), b);
+        }
+      } else {
+        const uint32_t u = k == 0 ? in.x : k == 1 ? in.y : k == 2 ? in.z : in.w;
+        a = bf_lo(u);
+        b = bf_hi(u);
       }
-      y[k] = silu_act<__nv_bfloat16>(a);
+      o[k] = bf_pack(silu_act<__nv_bfloat16>(a), silu_act<__nv_bfloat16>(b));
+      ss = fmaf(bf_lo(o[k]), bf_lo(o[k]), fmaf(bf_hi(o[k]), bf_hi(o[k]), ss));
     }
-#pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      ob[k] = __floats2bfloat162_rn(y[2 * k], y[2 * k + 1]);
-      const float2 f = __bfloat1622float2(ob[k]);
-      ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
-    }
-    if (live) *reinterpret_cast<uint2*>(dst + (long long)i * c.qkv_ld) = o;
+    if (live) *reinterpret_cast<uint4*>(dst + (long long)i * c.qkv_ld) = make_uint4(o[0], o[1], o[2], o[3]);
     if (p.kind == REC_DELTA) {
       for (int s = 1; s < lanes; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-      if (live && ch < 2 * gd && g4 % lanes == 0)
+      if (live && ch < 2 * gd && g8 % lanes == 0)
         c.unit[(size_t)(t0 + i) * 2 * p.G + ch / p.D] = 1.f / sqrtf(ss + 1e-6f) / (ch < gd ? sqrtf((float)p.D) : 1.f);
     }
   };
-  load(0);
   for (int i0 = 0; i0 < nt; i0 += PV_AHEAD) {
-#pragma unroll
-    for (int a = 0; a < PV_AHEAD; ++a) cur[a] = next[a];
-    load(i0 + PV_AHEAD);
+    uint4 in[PV_AHEAD];
 #pragma unroll
     for (int a = 0; a < PV_AHEAD; ++a)
-      if (i0 + a < nt) token(i0 + a, cur[a]);
+      if (i0 + a < nt) in[a] = *reinterpret_cast<const uint4*>(src + (long long)(i0 + a) * p.ld);
+#pragma unroll
+    for (int a = 0; a < PV_AHEAD; ++a)
+      if (i0 + a < nt) token(i0 + a, in[a]);
   }
 }
 
@@ -662,12 +658,12 @@ extern "C" int skein_rec_prep(const SkeinRecParams* p, const SkeinRecChunk* c, i
   using namespace skein;
   if (T == 0) return 0;
   if (int e = rec_check(p)) return e;
-  const int lanes = p->D / 4;
-  const bool vec = !fp32 && p->D % 4 == 0 && p->V % 4 == 0 && p->ld % 4 == 0 && p->q_col % 4 == 0 && p->k_col % 4 == 0 && p->v_col % 4 == 0 &&
-                   c->qkv_ld % 4 == 0 && c->v_off % 4 == 0 && p->taps <= 4 && (p->kind == REC_LIGHTNING || p->taps > 1) && (uintptr_t)p->row % 16 == 0 &&
+  const int lanes = p->D / 8;
+  const bool vec = !fp32 && p->D % 8 == 0 && p->V % 8 == 0 && p->ld % 8 == 0 && p->q_col % 8 == 0 && p->k_col % 8 == 0 && p->v_col % 8 == 0 &&
+                   c->qkv_ld % 8 == 0 && c->v_off % 8 == 0 && p->taps <= 4 && (p->kind == REC_LIGHTNING || p->taps > 1) && (uintptr_t)p->row % 16 == 0 &&
                    (p->kind != REC_DELTA || (lanes <= 32 && (lanes & (lanes - 1)) == 0));
   if (vec) {
-    const dim3 grid(((2 * p->G * p->D + p->H * p->V) / 4 + 255) / 256 + 1, (T + PV_TOK - 1) / PV_TOK);
+    const dim3 grid(((2 * p->G * p->D + p->H * p->V) / 8 + 255) / 256 + 1, (T + PV_TOK - 1) / PV_TOK);
     auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(256), 0, (cudaStream_t)stream, *p, *c, T); };
     switch (p->kind == REC_LIGHTNING ? 1 : p->taps) {
       case 1: return go(rec_prep_vec_kernel<1>);

@@ -30,6 +30,7 @@ import torch
 
 from .. import core
 from ..models.config import ModelConfig, ParallelLayout
+from ..models import parallel_layers
 from ..models.layered import random_param
 from ..models.decoder import LayerWeights, ModelWeights, layered_weights
 from ..ops import reference as ref
@@ -101,6 +102,9 @@ def _random_param(name, shape, seed, std):
     if name.endswith((".act", ".canon1")):
         return random_param(name, tuple(shape), torch.Generator().manual_seed(_stable_name_seed(name) ^ (seed * 1000003)), std, torch.bfloat16, "cpu")
     g = torch.Generator().manual_seed(_stable_name_seed(name) ^ (seed * 1000003))
+    special = parallel_layers.random_param(name, tuple(shape), g, "cpu")      # decays, step sizes, convolutions
+    if special is not None:
+        return special.to(torch.bfloat16)
     return (torch.randn(*shape, generator=g) * std).to(torch.bfloat16)
 
 

@@ -35,6 +35,8 @@ def _rope(x, pos, theta, scaling=None):
 @torch.no_grad()
 def forward_full(cfg: ModelConfig, w: ModelWeights, token_ids: torch.Tensor, capture_hidden: list | None = None):
     """Full-sequence forward of ONE sequence (unsharded weights). Returns fp32 logits [T, V]."""
+    if cfg.is_parallel:
+        return _forward_parallel(cfg, w, token_ids, capture_hidden)
     if cfg.is_layered:
         return _forward_layered(cfg, w, token_ids, capture_hidden)
     T = token_ids.shape[0]
@@ -144,3 +146,82 @@ def _forward_layered(cfg, w, token_ids, capture_hidden):
         if capture_hidden is not None:
             capture_hidden.append(x.clone())
     return (unit(x) * w.final_norm) @ w.lm_head.float().t()
+
+
+def _forward_parallel(cfg, w, token_ids, capture_hidden):
+    """The same for parallel layers: attention by a full mask, recurrences one token at a time, no state kept."""
+    from .parallel_layers import LayerLayout, WindowAttnSpec
+    T, C, eps = token_ids.shape[0], cfg.hidden_size, cfg.rms_norm_eps
+    unit = lambda v: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)      # noqa: E731
+    norm = lambda v, n: torch.tanh(n.alpha * v) * n.w + n.b                       # noqa: E731
+    act = torch.nn.functional
+    x0 = x = w.embed[token_ids.long()].float()
+    pos = torch.arange(T, device=x.device)
+    back = pos[:, None] - pos[None, :]
+
+    def attention(a, aw, z, at):
+        q, k, v = (z[:, at[n]:at[n] + rows] for n, rows in a.sections())
+        inv = a.rope_base ** (-torch.arange(0, a.rot_dims, 2, device=x.device).double() / max(a.rot_dims, 1)) / a.rope_factor
+        ang = pos.double()[:, None] * inv
+        c, s = ang.cos().float()[:, None], ang.sin().float()[:, None]
+        n = a.rot_dims // 2
+        turn = lambda t: torch.cat([t[..., :n] * c - t[..., n:2 * n] * s, t[..., n:2 * n] * c + t[..., :n] * s, t[..., 2 * n:]], dim=-1)   # noqa: E731
+        q = turn((unit(q) * aw.q_norm).view(T, a.heads, a.dim))
+        k = turn((unit(k) * aw.k_norm).view(T, a.kv_heads, a.dim)).repeat_interleave(a.heads // a.kv_heads, dim=1)
+        v = v.view(T, a.kv_heads, a.vdim).repeat_interleave(a.heads // a.kv_heads, dim=1)
+        seen = (back >= 0) & (back < a.window) if a.window else back >= 0
+        s = (torch.einsum("qhd,khd->hqk", q, k) * a.scale).masked_fill(~seen, float("-inf"))
+        return torch.einsum("hqk,khv->qhv", torch.softmax(s, dim=-1), v).reshape(T, -1)
+
+    def recurrence(r, rw, z, at):
+        H, G, D, V = r.heads, r.groups, r.dim, r.vdim
+        if r.kind == "ssd":
+            v0 = at["conv"]
+            cols = (v0 + H * V + G * D, v0 + H * V, v0)
+        else:
+            cols = (at["q"], at["k"], at["v"])
+        u = torch.cat([z[:, c0:c0 + n] for c0, n in zip(cols, (G * D, G * D, H * V))], dim=1)
+        if r.conv_channels:
+            u = sum(rw.conv[j] * act.pad(u, (0, 0, r.taps - 1 - j, 0))[:T] for j in range(r.taps)) + (rw.conv_b if rw.conv_b is not None else 0.0)
+        u = act.silu(u)
+        q, k, v = u[:, :G * D].view(T, G, D), u[:, G * D:2 * G * D].view(T, G, D), u[:, 2 * G * D:].view(T, H, V)
+        if r.kind == "delta":
+            q, k = (t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6) for t in (q, k))
+            q = q * D ** -0.5
+        q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)
+        if r.kind == "lightning":
+            g, coef = rw.neg_decay.exp().expand(T, H), torch.ones(T, H, device=x.device)
+        else:
+            a0 = at["dt" if r.kind == "ssd" else "a"]
+            step = act.softplus(z[:, a0:a0 + H] + rw.dt_bias)
+            g = (rw.neg_decay * step).exp()
+            coef = torch.sigmoid(z[:, at["b"]:at["b"] + H]) if r.kind == "delta" else step
+        S, out = torch.zeros(H, D, V, device=x.device), []
+        for t in range(T):
+            S = g[t][:, None, None] * S
+            d = v[t] - torch.einsum("hdv,hd->hv", S, k[t]) if r.kind == "delta" else v[t]
+            S = S + k[t][:, :, None] * (coef[t][:, None] * d)[:, None]
+            out.append(torch.einsum("hdv,hd->hv", S, q[t]) + (rw.skip[:, None] * v[t] if rw.skip is not None else 0.0))
+        o = torch.stack(out)
+        if r.kind == "ssd":
+            o = o.reshape(T, -1) * act.silu(z[:, at["z"]:at["z"] + H * V])
+            return unit(o.view(T, r.norm_groups, -1)).reshape(T, -1) * rw.norm
+        gate = z[:, at["g"]:at["g"] + H * V]
+        if r.kind == "delta":
+            return (unit(o) * rw.norm).reshape(T, -1) * act.silu(gate)
+        return unit(o.reshape(T, -1)) * rw.norm * torch.sigmoid(gate)
+
+    for sp, lw in zip(cfg.layers, w.layers):
+        lay = LayerLayout(sp)
+        if sp.loop_pass is not None:
+            x = torch.cat([x, x0], dim=1) @ w.loop.w_in.float().t() + w.loop.step[sp.loop_pass]
+        z = torch.zeros(T, lay.width, device=x.device)
+        z[:, lay.in_first:] = norm(x, lw.norm) @ lw.w_in.float().t()
+        z[:, lay.ff:lay.ff + lay.ff_cols] = z[:, lay.ff:lay.ff + lay.ff_cols].clamp(min=0).square()
+        for sec in lay.parts:
+            f, mw = (attention, lw.attn) if isinstance(sec.spec, WindowAttnSpec) else (recurrence, lw.rec)
+            z[:, sec.out:sec.out + sec.spec.out_width] = sec.scale * f(sec.spec, mw, z, sec.col)
+        x = x + z[:, :lay.out_cols] @ lw.w_out.float().t()
+        if capture_hidden is not None:
+            capture_hidden.append(x.clone())
+    return norm(x, w.final_norm) @ w.lm_head.float().t()

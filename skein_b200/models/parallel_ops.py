@@ -80,7 +80,7 @@ class ParallelOps:
         st.residual = ops.linear(st.qkv[:, :lay.out_cols], self.w.layers[li].w_out, out=st.residual, residual=st.residual, out_f32=True)
         st.qkv = None
         if self.capture_hidden is not None:
-            self.capture_hidden.append(st.residual.detach().float().cpu())
+            self.capture_hidden.append(st.residual.detach().clone().cpu())      # (the next layer adds in place)
 
     def _op_final_tanh_norm(self, st, _):
         _, st.normed = par.residual_tanh(st.residual, norm=self.w.final_norm, dtype=self.act_dtype, want_x=False)

@@ -219,7 +219,7 @@ def rec_case(r, T, dtype, seed=0):
         w.neg_decay = torch.tensor(r.decay, dtype=torch.float64).log().clamp(min=-1e30).float()
     else:
         w.neg_decay, w.dt_bias = -torch.exp(rnd(H, dtype=F32)), rnd(H, dtype=F32, seed=3) - 1.0
-        w.conv = rnd(r.taps, ch, dtype=F32, scale=r.taps ** -0.5)
+        w.conv = rnd(r.taps, ch, scale=r.taps ** -0.5).float()
         if r.kind == "ssd":
             w.conv_b, w.skip = rnd(ch, dtype=F32, scale=0.2), rnd(H, dtype=F32)
     return row, rec.RecColumns.of(r, col), w
