@@ -114,12 +114,14 @@ def _spiked(size, dim, spec_window):
     g = torch.Generator().manual_seed(1)
     u, v = torch.randn(96, generator=g), torch.randn(96, generator=g)
     v -= u * (u @ v) / (u @ u)
-    t["l0.norm1"], t["l0.norm1.b"], t["l0.norm1.alpha"] = torch.ones(96).to(BF), torch.zeros(96).to(BF), torch.tensor(0.01).to(BF)
-    t["embed"][1], t["embed"][2] = (8 * u).to(BF), (8 * v).to(BF)
+    t["l0.norm1"], t["l0.norm1.b"], t["l0.norm1.alpha"] = torch.ones(96).to(BF), torch.zeros(96).to(BF), torch.tensor(0.1).to(BF)
+    t["embed"][1], t["embed"][2] = (2 * u).to(BF), (2 * v).to(BF)
+    for n in ("v", "o"):
+        t["l0.mix.left." + n] = (t["l0.mix.left." + n].float() * 4).to(BF)
     k = torch.randn(dim, generator=g)
     for n in ("q.norm", "k.norm"):
         t["l0.mix.left." + n] = torch.ones_like(t["l0.mix.left." + n])
-    t["l0.mix.left.k"] = (torch.outer(k, u / u.norm()) * 3 + 0.3 * t["l0.mix.left.k"].float()).to(BF)
+    t["l0.mix.left.k"] = (torch.outer(k, u / u.norm()) * 0.2 + 0.3 * t["l0.mix.left.k"].float()).to(BF)
     t["l0.mix.left.q"] = (torch.outer(torch.cat([k, k]), v / v.norm()) * 3 + 0.3 * t["l0.mix.left.q"].float()).to(BF)
     return cfg, raw, t
 
@@ -160,7 +162,7 @@ def test_an_early_token_is_remembered_by_the_states(tmp_path):
     toks = torch.randint(0, cfg.vocab_size, (n,), generator=torch.Generator().manual_seed(4)).tolist()
     want = plain.forward(raw, t, toks)
     lost = plain.forward(raw, t, [(toks[0] + 1) % cfg.vocab_size] + toks[1:])
-    assert rel_err(lost[-1:], want[-1:]) > 1e-2
+    assert rel_err(lost[-1:], want[-1:]) > 3e-3
     s = session(cfg, t, tmp_path, F32)
     for sizes in ([n], [1, n - 1], [1] * 20 + [380] + [1] * 20):
         at, out = 0, []
