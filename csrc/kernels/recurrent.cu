@@ -34,7 +34,12 @@ constexpr int REC_MAX_D = 512;
 // the activation behind a projection or convolution; its result is rounded to bf16 in a bf16 model, so there it is computed fast
 template <typename T> __device__ __forceinline__ float silu_act(float z);
 template <> __device__ __forceinline__ float silu_act<float>(float z) { return z / (1.f + expf(-z)); }
-template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z * -1.44269504f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return z * r;
+}
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // log decay and write coefficient of head h from the row's gate columns
@@ -382,9 +387,9 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
   }
 }
 
-// The same with 16-byte accesses: a thread takes 8 channels of PV_TOK tokens and keeps the convolution's inputs and (bf16) taps packed
-// in registers. Every section starts at a multiple of 8 channels and columns; D / 8 is a power of two up to 32 (delta). The last column
-// of CTAs does the gates. grid (channel blocks + 1, token blocks)
+// The same with 16-byte accesses: a thread takes 8 channels of PV_TOK tokens and keeps the sums of the next TAPS outputs in registers,
+// into which every input goes as it is read. Every section starts at a multiple of 8 channels and columns; D / 8 is a power of two up
+// to 32 (delta). The last column of CTAs does the gates. grid (channel blocks + 1, token blocks)
 constexpr int PV_TOK = 32, PV_AHEAD = 4;       // tokens of a thread; loads in flight
 
 __device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
@@ -393,9 +398,13 @@ __device__ __forceinline__ uint32_t bf_pack(float a, float b) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
+__device__ __forceinline__ void bf_unpack8(const uint4& u, float* v) {
+  v[0] = bf_lo(u.x); v[1] = bf_hi(u.x); v[2] = bf_lo(u.y); v[3] = bf_hi(u.y);
+  v[4] = bf_lo(u.z); v[5] = bf_hi(u.z); v[6] = bf_lo(u.w); v[7] = bf_hi(u.w);
+}
 
 template <int TAPS>      // 1: no convolution ("lightning"), else the taps
-__global__ void __launch_bounds__(256) rec_prep_vec_kernel(const RecParams p, const RecChunk c, int T) {
+__global__ void __launch_bounds__(256, 2) rec_prep_vec_kernel(const RecParams p, const RecChunk c, int T) {
   __shared__ int pos_s[PV_TOK], first_s[PV_TOK], slot_s[PV_TOK];
   pdl_trigger();
   pdl_wait();
@@ -423,56 +432,62 @@ __global__ void __launch_bounds__(256) rec_prep_vec_kernel(const RecParams p, co
   const int ch = (live ? g8 : 0) * 8, col = rec_col(p, ch);
   const __nv_bfloat16* src = (const __nv_bfloat16*)p.row + (size_t)t0 * p.ld + col;
   __nv_bfloat16* dst = (__nv_bfloat16*)c.qkv + (size_t)t0 * c.qkv_ld + (ch < 2 * gd ? ch : ch - 2 * gd + c.v_off);
-  uint32_t w[TAPS][4];                        // w[j]: the tap j tokens back
-  uint4 x[TAPS];                              // x[j]: the input j tokens back
-  if (TAPS > 1)
+  // w[j]: the tap j tokens back. sum[j] (j > 0): what the inputs so far add to the output j - 1 tokens on; the bias is in it
+  float w[TAPS][8], bias[8], sum[TAPS][8];
+  if (TAPS > 1) {
+#pragma unroll
+    for (int k = 0; k < 8; ++k) bias[k] = p.conv_b ? p.conv_b[ch + k] : 0.f;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-      const float4* wp = reinterpret_cast<const float4*>(p.conv_w + (size_t)(TAPS - 1 - j) * p.C + ch);
-      const float4 a = wp[0], b = wp[1];
-      w[j][0] = bf_pack(a.x, a.y); w[j][1] = bf_pack(a.z, a.w); w[j][2] = bf_pack(b.x, b.y); w[j][3] = bf_pack(b.z, b.w);
+      load_v<float, 4>(p.conv_w + (size_t)(TAPS - 1 - j) * p.C + ch, w[j]);
+      load_v<float, 4>(p.conv_w + (size_t)(TAPS - 1 - j) * p.C + ch + 4, w[j] + 4);
     }
+  }
   const int lanes = p.D / 8;
+  const bool units = p.kind == REC_DELTA && blockIdx.x * 2048 < 2 * gd;
   auto token = [&](int i, const uint4& in) {
+    float x[8], y[8];
     if (TAPS > 1) {
       const int t = t0 + i, first = first_s[i], pos = pos_s[i];
       if (i == 0 || t == first) {
+        // start of the block or of a sequence: the inputs before it, from the chunk, from the cache, or none
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j)
+#pragma unroll
+          for (int k = 0; k < 8; ++k) sum[j][k] = bias[k];
 #pragma unroll
         for (int j = 1; j < TAPS; ++j) {
-          x[j] = make_uint4(0, 0, 0, 0);
-          if (t - j >= first) x[j] = *reinterpret_cast<const uint4*>(src + (long long)(i - j) * p.ld);
+          uint4 u = make_uint4(0, 0, 0, 0);
+          if (t - j >= first) u = *reinterpret_cast<const uint4*>(src + (long long)(i - j) * p.ld);
           else if (pos - j >= 0)
-            x[j] = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.tail + ((size_t)slot_s[i] * TAPS + (pos - j) % TAPS) * p.C + ch);
-        }
-      } else {
+            u = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.tail + ((size_t)slot_s[i] * TAPS + (pos - j) % TAPS) * p.C + ch);
+          bf_unpack8(u, x);
 #pragma unroll
-        for (int j = TAPS - 1; j > 0; --j) x[j] = x[j - 1];
+          for (int o = 0; o + j < TAPS; ++o)        // the output o tokens on sees this input o + j back
+#pragma unroll
+            for (int k = 0; k < 8; ++k) sum[o + 1][k] = fmaf(w[o + j][k], x[k], sum[o + 1][k]);
+        }
       }
+      bf_unpack8(in, x);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) y[k] = fmaf(w[0][k], x[k], sum[1][k]);
+#pragma unroll
+      for (int j = 1; j + 1 < TAPS; ++j)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) sum[j][k] = fmaf(w[j][k], x[k], sum[j + 1][k]);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) sum[TAPS - 1][k] = fmaf(w[TAPS - 1][k], x[k], bias[k]);
+    } else {
+      bf_unpack8(in, y);
     }
-    x[0] = in;
-    float ss = 0.f;
     uint32_t o[4];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      float a = 0.f, b = 0.f;
-      if (TAPS > 1) {
-        if (p.conv_b) { const float2 f = *reinterpret_cast<const float2*>(p.conv_b + ch + 2 * k); a = f.x; b = f.y; }
-#pragma unroll
-        for (int j = TAPS - 1; j >= 0; --j) {
-          const uint32_t u = k == 0 ? x[j].x : k == 1 ? x[j].y : k == 2 ? x[j].z : x[j].w;
-          a = fmaf(bf_lo(w[j][k]), bf_lo(u), a);
-          b = fmaf(bf_hi(w[j][k]), bf_hi(u), b);
-        }
-      } else {
-        const uint32_t u = k == 0 ? in.x : k == 1 ? in.y : k == 2 ? in.z : in.w;
-        a = bf_lo(u);
-        b = bf_hi(u);
-      }
-      o[k] = bf_pack(silu_act<__nv_bfloat16>(a), silu_act<__nv_bfloat16>(b));
-      ss = fmaf(bf_lo(o[k]), bf_lo(o[k]), fmaf(bf_hi(o[k]), bf_hi(o[k]), ss));
-    }
+    for (int k = 0; k < 4; ++k) o[k] = bf_pack(silu_act<__nv_bfloat16>(y[2 * k]), silu_act<__nv_bfloat16>(y[2 * k + 1]));
     if (live) *reinterpret_cast<uint4*>(dst + (long long)i * c.qkv_ld) = make_uint4(o[0], o[1], o[2], o[3]);
-    if (p.kind == REC_DELTA) {
+    if (units) {
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) ss = fmaf(bf_lo(o[k]), bf_lo(o[k]), fmaf(bf_hi(o[k]), bf_hi(o[k]), ss));
       for (int s = 1; s < lanes; s <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
       if (live && ch < 2 * gd && g8 % lanes == 0)
         c.unit[(size_t)(t0 + i) * 2 * p.G + ch / p.D] = 1.f / sqrtf(ss + 1e-6f) / (ch < gd ? sqrtf((float)p.D) : 1.f);
@@ -694,7 +709,8 @@ extern "C" int skein_rec_scan(const SkeinRecParams* p, const SkeinRecChunk* c, i
 extern "C" int skein_rec_tail(const SkeinRecParams* p, const SkeinRecChunk* c, int S, int fp32, void* stream) {
   using namespace skein;
   if (S == 0 || p->taps < 2) return 0;
-  const dim3 grid(S, 8);
+  const int want = (p->C * (p->taps - 1) + 255) / 256;
+  const dim3 grid(S, want < 64 ? want : 64);
   return (int)(fp32 ? launch_pdl(rec_tail_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, *p, *c)
                     : launch_pdl(rec_tail_kernel<__nv_bfloat16>, grid, dim3(256), 0, (cudaStream_t)stream, *p, *c));
 }

@@ -62,12 +62,12 @@ __device__ __forceinline__ void rt_ldsm2t(uint32_t addr, uint32_t* r) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
 
-constexpr int RT_LX = RT_C + 8, RT_LY = 40;    // row lengths of the 64-wide and 32-wide bf16 scratch matrices
+constexpr int RT_LX = RT_C + 8, RT_LY = 40, RT_LD = 20;    // row lengths of the 64-wide and 32-wide bf16 and the 16-wide fp32 scratch matrices
 __host__ __device__ constexpr int rt_kq_bytes(int d) { return 2 * RT_C * (d + 8) * 2; }
 // K and Q, whose place X and Y take later; then A
 __host__ __device__ constexpr int rt_mats_smem(int d, bool delta) {
   return (!delta || rt_kq_bytes(d) > 2 * RT_C * RT_LX * 2 + 2 * 32 * RT_LY * 2 ? rt_kq_bytes(d) : 2 * RT_C * RT_LX * 2 + 2 * 32 * RT_LY * 2) +
-         (delta ? 2 * RT_C * RT_LX * 2 + RT_C * 17 * 4 : 0);
+         (delta ? 2 * RT_C * RT_LX * 2 + RT_C * RT_LD * 4 : 0);
 }
 
 // One 16 x 8 tile of L R with both factors as hi + lo: acc over `ks` steps of 16. l, r: shared-memory addresses of the tile's
@@ -105,9 +105,12 @@ constexpr int RT_HB = 8;         // most heads of a CTA
 
 // grid (chunks, H / heads, S), 256 threads: `heads` heads that share queries and keys, whose products are computed once
 template <int D, bool DELTA>
-__global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, const RecChunk c, __nv_bfloat16* mats, float* factors, int heads) {
+__global__ void __launch_bounds__(256, 3) rec_tc_mats_kernel(const RecParams p, const RecChunk c, __nv_bfloat16* mats, float* factors, int heads) {
   extern __shared__ __align__(16) uint8_t mt_smem[];
-  __shared__ float Gh_all[RT_HB][RT_C], Gl_all[RT_HB][RT_C], coef_all[RT_HB][RT_C], rq_s[RT_C], rk_s[RT_C];
+  __shared__ __align__(16) float Gh_all[RT_HB][RT_C];
+  __shared__ __align__(16) float Gl_all[RT_HB][RT_C];
+  __shared__ __align__(16) float coef_all[RT_HB][RT_C];
+  __shared__ __align__(16) float rq_s[RT_C], rk_s[RT_C];
   pdl_trigger();
   pdl_wait();
   const int h0 = blockIdx.y * heads, seq = blockIdx.z, len = c.q_len[seq], i0 = blockIdx.x * RT_C;
@@ -122,9 +125,9 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
   __nv_bfloat16* Xl = Xh + RT_C * RT_LX;
   __nv_bfloat16* Yh = Xl + RT_C * RT_LX;                     // [32][RT_LY]
   __nv_bfloat16* Yl = Yh + 32 * RT_LY;
-  __nv_bfloat16* Ah = reinterpret_cast<__nv_bfloat16*>(mt_smem + rt_mats_smem(D, true) - 2 * RT_C * RT_LX * 2 - RT_C * 17 * 4);
+  __nv_bfloat16* Ah = reinterpret_cast<__nv_bfloat16*>(mt_smem + rt_mats_smem(D, true) - 2 * RT_C * RT_LX * 2 - RT_C * RT_LD * 4);
   __nv_bfloat16* Al = Ah + RT_C * RT_LX;
-  float* Ad = reinterpret_cast<float*>(Al + RT_C * RT_LX);   // [64][17] the 16 x 16 blocks on the diagonal
+  float* Ad = reinterpret_cast<float*>(Al + RT_C * RT_LX);   // [64][RT_LD] the 16 x 16 blocks on the diagonal
   for (int i = tid; i < RT_C * (D / 8) * 2; i += 256) {
     const int m = i / (RT_C * (D / 8)), r = i % (RT_C * (D / 8)) / (D / 8), ch = i % (D / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -193,25 +196,39 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
     }
     __nv_bfloat16* out = mats + (size_t)unit * (DELTA ? 3 : 1) * RT_C * RT_C;
     if (DELTA && hh > 0) __syncthreads();        // the previous head's X has been read
+    float gi[2], gl[2], ri[2];                   // of this thread's two rows
 #pragma unroll
-    for (int nb = 0; nb < nbn; ++nb)
+    for (int hf = 0; hf < 2; ++hf) {
+      const int i = r0 + (lane >> 2) + 8 * hf;
+      gi[hf] = Gh_s[i];
+      gl[hf] = Gl_s[i];
+      ri[hf] = i < n ? (qk ? rq_s[i] : rk_s[i] * coef_s[i]) : 0.f;
+    }
+#pragma unroll
+    for (int nb = 0; nb < nbn; ++nb) {
+      const int j = (nb0 + nb) * 8 + (lane & 3) * 2;
+      const bool below = (nb0 + nb) * 8 <= r0 + 15;
+      float2 gj = make_float2(0.f, 0.f), glj = gj, rj = gj;
+      if (below) {
+        gj = *reinterpret_cast<const float2*>(Gh_s + j);
+        glj = *reinterpret_cast<const float2*>(Gl_s + j);
+        rj = *reinterpret_cast<const float2*>(rk_s + j);
+        if (!DELTA) { const float2 cj = *reinterpret_cast<const float2*>(coef_s + j); rj.x *= cj.x; rj.y *= cj.y; }
+      }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
-        const int i = r0 + (lane >> 2) + 8 * hf, j = (nb0 + nb) * 8 + (lane & 3) * 2;
+        const int i = r0 + (lane >> 2) + 8 * hf;
         float v[2] = {0.f, 0.f};
-        if ((nb0 + nb) * 8 <= r0 + 15) {
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int jj = j + e;
-            if (i < n && (qk ? jj <= i : jj < i))
-              v[e] = prod[nb][2 * hf + e] * decay(i, jj) * rk_s[jj] * (qk ? rq_s[i] * (DELTA ? 1.f : coef_s[jj]) : rk_s[i] * coef_s[i]);
-          }
+        if (below) {
+          const int last = qk ? i : i - 1;       // last column of the row
+          if (j <= last) v[0] = prod[nb][2 * hf] * exp2f((gi[hf] - gj.x) + (gl[hf] - glj.x)) * rj.x * ri[hf];
+          if (j + 1 <= last) v[1] = prod[nb][2 * hf + 1] * exp2f((gi[hf] - gj.y) + (gl[hf] - glj.y)) * rj.y * ri[hf];
         }
         if (qk) {
           *reinterpret_cast<uint32_t*>(out + (DELTA ? 2 : 0) * RT_C * RT_C + i * RT_C + j) = rt_pack(v[0], v[1]);
         } else if (nb >> 1 == blk) {
-          Ad[i * 17 + (j & 15)] = v[0];
-          Ad[i * 17 + (j & 15) + 1] = v[1];
+          Ad[i * RT_LD + (j & 15)] = v[0];
+          Ad[i * RT_LD + (j & 15) + 1] = v[1];
         } else if (nb >> 1 < blk) {
           uint32_t hi, lo;
           rt_split(v[0], v[1], hi, lo);
@@ -219,6 +236,7 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
           *reinterpret_cast<uint32_t*>(Al + i * RT_LX + j) = lo;
         }
       }
+    }
     if (!DELTA) continue;
     __syncthreads();
     // X = (I + A)^-1: the 16 x 16 blocks on the diagonal by substitution, then blocks of 32 and 64 from two of half the size,
@@ -228,14 +246,20 @@ __global__ void __launch_bounds__(256) rec_tc_mats_kernel(const RecParams p, con
     if (tid < RT_C) {
       const int b0 = tid & ~15, col = tid & 15;
       float x[16];
-  #pragma unroll
+#pragma unroll
       for (int r = 0; r < 16; ++r) {
         float s = r == col ? 1.f : 0.f;
-  #pragma unroll
-        for (int m = 0; m < r; ++m) s = fmaf(-Ad[(b0 + r) * 17 + m], x[m], s);
+#pragma unroll
+        for (int m = 0; m < r; m += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(Ad + (b0 + r) * RT_LD + m);
+          s = fmaf(-a.x, x[m], s);
+          if (m + 1 < r) s = fmaf(-a.y, x[m + 1], s);
+          if (m + 2 < r) s = fmaf(-a.z, x[m + 2], s);
+          if (m + 3 < r) s = fmaf(-a.w, x[m + 3], s);
+        }
         x[r] = s;
       }
-  #pragma unroll
+#pragma unroll
       for (int r = 0; r < 16; ++r) {
         const __nv_bfloat16 hi = __float2bfloat16(x[r]);
         Xh[(b0 + r) * RT_LX + b0 + col] = hi;
