@@ -75,10 +75,10 @@ def parse():
     ap.add_argument("--repeats", type=int, default=5, help="how often each timed K-step loop is repeated (median reported)")
     ap.add_argument("--no-selfcheck", action="store_true")
     ap.add_argument("--no-unfused", action="store_true", help="skip the un-fused comparison arm at N > 1")
-    ap.add_argument("--design", default="", choices=["", "zarorax"],
+    ap.add_argument("--design", default="", choices=["", "zarorax", "sikalorn"],
                     help="instead of the headline workload: throughput of this design at a few layer sizes beside the closest uniform model, "
                          "and its kernels' rooflines beside the like kernels (one JSON line per size; skein_b200/utils/design_bench.py)")
-    ap.add_argument("--design-sizes", default="all", help="with --design: comma-separated sizes (moe-2k, moe-4k, dense-4k)")
+    ap.add_argument("--design-sizes", default="all", help="with --design: comma-separated sizes (zarorax: moe-2k, moe-4k, dense-4k; sikalorn: width-2k, width-4k)")
     ap.add_argument("--eager", action="store_true",
                     help="launch the step's kernels one by one instead of replaying the captured graph "
                          "(for a per-kernel launch list; the timed loop sits in an NVTX range named 'timed')")
@@ -551,13 +551,13 @@ def main():
         import torch
 
         from skein_b200.utils import design_bench
-        sizes = design_bench.SIZES if args.design_sizes == "all" else args.design_sizes.split(",")
+        sizes = design_bench.DESIGNS[args.design][0] if args.design_sizes == "all" else args.design_sizes.split(",")
         for size in sizes:
             sampler = ClockSampler(0)
             sampler.start()
             lines = []
             with torch.no_grad():
-                design_bench.run([size], emit=lines.append)
+                design_bench.run(args.design, [size], emit=lines.append)
             out = json.loads(lines[0])
             out["clocks"] = sampler.stop()
             print(json.dumps(out), flush=True)

@@ -45,8 +45,8 @@ __device__ __forceinline__ float wa_block_sum(float v, float* sh) {
 
 // grid (T, 2): queries, then keys and values. VEC elements per access; a rotated pair is two accesses rot / 2 apart.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) window_append_kernel(const WindowAppendParams p) {
-  __shared__ float sh[8];
+__global__ void __launch_bounds__(1024) window_append_kernel(const WindowAppendParams p) {
+  __shared__ float sh[32];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, pos = p.positions[t];
@@ -187,10 +187,13 @@ extern "C" int skein_window_append(void* q, const void* k, const void* v, long l
                        num_pages, page_size, eps};
   const bool v4 = D % 4 == 0 && (rot / 2) % 4 == 0 && ld % 4 == 0 && (size_t)K * page_size * (D + V) % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0;
   const dim3 grid(T, 2);
+  int th = 256;                     // few rows: up to one access per thread
+  while (T <= 512 && th < 1024 && th * (v4 ? 4 : 1) < H * D) th *= 2;
+  const dim3 b(th);
   cudaStream_t s = (cudaStream_t)stream;
-  if (fp32) return (int)(v4 ? launch_pdl(window_append_kernel<float, 4>, grid, dim3(256), 0, s, p) : launch_pdl(window_append_kernel<float, 1>, grid, dim3(256), 0, s, p));
-  return (int)(v4 ? launch_pdl(window_append_kernel<__nv_bfloat16, 4>, grid, dim3(256), 0, s, p)
-                  : launch_pdl(window_append_kernel<__nv_bfloat16, 1>, grid, dim3(256), 0, s, p));
+  if (fp32) return (int)(v4 ? launch_pdl(window_append_kernel<float, 4>, grid, b, 0, s, p) : launch_pdl(window_append_kernel<float, 1>, grid, b, 0, s, p));
+  return (int)(v4 ? launch_pdl(window_append_kernel<__nv_bfloat16, 4>, grid, b, 0, s, p)
+                  : launch_pdl(window_append_kernel<__nv_bfloat16, 1>, grid, b, 0, s, p));
 }
 
 extern "C" int skein_window_attn_rows(const void* q, long long ld, const void* cache, const int* positions, const int* seq_of_token,

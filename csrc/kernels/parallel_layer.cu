@@ -137,6 +137,44 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormParams p
   }
 }
 
+// The same for groups of up to 4096 elements, four of a group in each thread: read once, kept in registers. A warp per group (WARP), or
+// a CTA of the group's size / 4 threads.
+template <typename T, bool WARP>
+__global__ void __launch_bounds__(1024) gated_norm_reg_kernel(const GatedNormParams p) {
+  __shared__ float sh[32];
+  pdl_trigger();
+  pdl_wait();
+  const int size = p.n / p.groups, lane = WARP ? threadIdx.x & 31 : threadIdx.x;
+  const long long u = WARP ? (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
+  if (u >= (long long)p.T * p.groups) return;      // (whole warps or the whole CTA)
+  const int t = (int)(u / p.groups), c0 = (int)(u % p.groups) * size, i = lane * 4;
+  const bool in = i < size;
+  float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f}, w[4] = {0.f, 0.f, 0.f, 0.f}, ss = 0.f;
+  if (in) {
+    load_v<T, 4>((const T*)p.o + (size_t)t * p.n + c0 + i, v);
+    load_v<T, 4>((const T*)p.gate + (size_t)t * p.gate_ld + c0 + i, z);
+    load_v<float, 4>(p.w + (c0 + i) % p.w_period, w);
+  }
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    z[k] = gate_value<T>(p, z[k]);
+    if (p.gate_first) v[k] *= z[k];
+    ss += v[k] * v[k];
+  }
+  for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+  if (!WARP) {
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int k = 0; k < (int)(blockDim.x >> 5); ++k) ss += sh[k];
+  }
+  if (!in) return;
+  const float r = p.scale / sqrtf(ss / (float)size + p.eps);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) v[k] *= p.gate_first ? r * w[k] : z[k] * r * w[k];
+  store_v<T, 4>((T*)p.out + (size_t)t * p.out_ld + c0 + i, v);
+}
+
 }  // namespace skein
 
 extern "C" int skein_residual_tanh(const float* x, const void* y, int y_f32, const float* bias, const float* alpha, const float* w, const float* b,
@@ -168,6 +206,13 @@ extern "C" int skein_gated_norm(const void* o, const void* gate, long long gate_
   const long long units = (long long)T * groups;
   const dim3 grid((unsigned)(warp ? (units + 7) / 8 : units));
   cudaStream_t s = (cudaStream_t)stream;
+  if (v4 && size <= 4096) {
+    const bool w32 = size <= 128;
+    const dim3 g((unsigned)(w32 ? (units + 7) / 8 : units)), b(w32 ? 256 : (size / 4 + 31) / 32 * 32);
+    if (fp32) return (int)(w32 ? launch_pdl(gated_norm_reg_kernel<float, true>, g, b, 0, s, p) : launch_pdl(gated_norm_reg_kernel<float, false>, g, b, 0, s, p));
+    return (int)(w32 ? launch_pdl(gated_norm_reg_kernel<__nv_bfloat16, true>, g, b, 0, s, p)
+                     : launch_pdl(gated_norm_reg_kernel<__nv_bfloat16, false>, g, b, 0, s, p));
+  }
   auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(256), 0, s, p); };
   if (fp32) {
     if (v4) return warp ? go(gated_norm_kernel<float, 4, true>) : go(gated_norm_kernel<float, 4, false>);

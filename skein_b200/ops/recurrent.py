@@ -90,35 +90,57 @@ def rec_step(row, cols: RecColumns, spec, w, state: RecState, positions, slots, 
     return None if g.out else out
 
 
+class ChunkRun:
+    """Portions of several sequences on the GPU: the launches of rec_chunk and what they share."""
+
+    def __init__(self, row, cols, spec, w, state, positions, slots, seq_of_token, q_start, q_len, max_q_len, impl=None):
+        dev, self.T, self.S = row.device, row.shape[0], q_len.shape[0]
+        self.out = torch.empty(self.T, spec.out_width, dtype=row.dtype, device=dev)
+        self.p, self.c = _params(row, cols, spec, w, state, positions, slots, self.out), _lib.RecChunk()
+        self.fp32, self.tail_rows = 1 if row.dtype == torch.float32 else 0, state.tail is not None
+        self.tc = (impl or ("tc" if max_q_len >= TC_MIN_ROWS else "scan")) == "tc" and tc_ok(spec, row)
+        c = self.c
+        c.v_off = (2 * spec.groups * spec.dim + 7) // 8 * 8
+        c.qkv_ld = c.v_off + (spec.out_width + 7) // 8 * 8
+        qkv = torch.empty(self.T, c.qkv_ld, dtype=row.dtype, device=dev)
+        gates = torch.empty(self.T, spec.heads, 2, dtype=torch.float32, device=dev)
+        unit = torch.empty(self.T, 2, spec.groups, dtype=torch.float32, device=dev) if spec.kind == "delta" else None
+        scratch = None
+        if self.tc:
+            scratch = torch.empty(int(_lib.lib().skein_rec_tc_scratch_bytes(C.byref(self.p), self.T, self.S)), dtype=torch.uint8, device=dev)
+        c.seq_of_token, c.q_start, c.q_len, c.max_q_len = seq_of_token.data_ptr(), q_start.data_ptr(), q_len.data_ptr(), int(max_q_len)
+        c.qkv, c.gates, c.unit, c.chunk_mat = qkv.data_ptr(), gates.data_ptr(), _lib.ptr(unit), _lib.ptr(scratch)
+        self._keep = (row, w, state, positions, slots, seq_of_token, q_start, q_len, qkv, gates, unit, scratch)
+
+    def prep(self):
+        """Convolution, silu, gates, unit norms."""
+        _lib.check(_lib.lib().skein_rec_prep(C.byref(self.p), C.byref(self.c), self.T, self.fp32, _lib.stream_ptr()), "rec_prep")
+        _lib.count_launch()
+
+    def walk(self):
+        """The recurrence; the state moves on."""
+        if self.tc:
+            _lib.check(_lib.lib().skein_rec_tc(C.byref(self.p), C.byref(self.c), self.T, self.S, _lib.stream_ptr()), "rec_tc")
+            _lib.count_launch(2)
+        else:
+            _lib.check(_lib.lib().skein_rec_scan(C.byref(self.p), C.byref(self.c), self.S, self.fp32, _lib.stream_ptr()), "rec_scan")
+            _lib.count_launch()
+
+    def tail(self):
+        """The convolution's last inputs, once nothing reads the old ones any more."""
+        if self.tail_rows:
+            _lib.check(_lib.lib().skein_rec_tail(C.byref(self.p), C.byref(self.c), self.S, self.fp32, _lib.stream_ptr()), "rec_tail")
+            _lib.count_launch()
+
+
 def rec_chunk(row, cols: RecColumns, spec, w, state: RecState, positions, slots, seq_of_token, q_start, q_len, max_q_len, impl=None):
     """Portions of several sequences, one after another: rows q_start[s] .. + q_len[s] are consecutive tokens of the sequence in
     slots[s]. impl "tc" (chunks of 64 tokens on the tensor cores; the default for longer portions where it takes the sizes) or
     "scan" (one token after the other)."""
-    T = row.shape[0]
     if not row.is_cuda:
         return rp.rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len)
-    dev, fp32, S = row.device, 1 if row.dtype == torch.float32 else 0, q_len.shape[0]
-    out = torch.empty(T, spec.out_width, dtype=row.dtype, device=dev)
-    p = _params(row, cols, spec, w, state, positions, slots, out)
-    c = _lib.RecChunk()
-    c.v_off = (2 * spec.groups * spec.dim + 7) // 8 * 8
-    c.qkv_ld = c.v_off + (spec.out_width + 7) // 8 * 8
-    qkv = torch.empty(T, c.qkv_ld, dtype=row.dtype, device=dev)
-    gates = torch.empty(T, spec.heads, 2, dtype=torch.float32, device=dev)
-    unit = torch.empty(T, 2, spec.groups, dtype=torch.float32, device=dev) if spec.kind == "delta" else None
-    c.seq_of_token, c.q_start, c.q_len, c.max_q_len = seq_of_token.data_ptr(), q_start.data_ptr(), q_len.data_ptr(), int(max_q_len)
-    c.qkv, c.gates, c.unit = qkv.data_ptr(), gates.data_ptr(), _lib.ptr(unit)
-    L, s = _lib.lib(), _lib.stream_ptr()
-    _lib.check(L.skein_rec_prep(C.byref(p), C.byref(c), T, fp32, s), "rec_prep")
-    if (impl or ("tc" if max_q_len >= TC_MIN_ROWS else "scan")) == "tc" and tc_ok(spec, row):
-        scratch = torch.empty(int(L.skein_rec_tc_scratch_bytes(C.byref(p), T, S)), dtype=torch.uint8, device=dev)
-        c.chunk_mat = scratch.data_ptr()
-        _lib.check(L.skein_rec_tc(C.byref(p), C.byref(c), T, S, s), "rec_tc")
-        _lib.count_launch(3)
-    else:
-        _lib.check(L.skein_rec_scan(C.byref(p), C.byref(c), S, fp32, s), "rec_scan")
-        _lib.count_launch(2)
-    if state.tail is not None:
-        _lib.check(L.skein_rec_tail(C.byref(p), C.byref(c), S, fp32, s), "rec_tail")
-        _lib.count_launch()
-    return out
+    run = ChunkRun(row, cols, spec, w, state, positions, slots, seq_of_token, q_start, q_len, max_q_len, impl)
+    run.prep()
+    run.walk()
+    run.tail()
+    return run.out

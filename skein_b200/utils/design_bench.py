@@ -1,7 +1,7 @@
 """Throughput and per-kernel rooflines of a design that lists its layers, beside the closest uniform family at equal size.
 
-    python bench.py --design zarorax                    # one JSON object per size
-    python -m skein_b200.utils.design_bench --only kernels --size moe-2k
+    python bench.py --design zarorax                    # one JSON object per size; also: sikalorn
+    python -m skein_b200.utils.design_bench --design sikalorn --only kernels --size width-2k
 
 Weights are random. Each size is a few layers of a real model's width; the closest model has the same width, number of layers,
 query heads, experts and feed-forward size (a Mixtral-shaped block for routed layers, a Llama-shaped one for dense layers).
@@ -25,6 +25,7 @@ from ..models.layered import DenseFFSpec, LatentMixerSpec, LayerSpec, RoutedFFSp
 from ..ops import latent as lat
 from ..ops import reference as ref
 from ..runtime.runner import ModelRunner
+from . import design_bench_parallel as parallel
 from .microbench import _bf, peaks, timeit, timeit_graph
 
 
@@ -52,15 +53,15 @@ def throughput(cfg, B=64, prompt=512, steps=64, warmup=8, repeats=3, prompts_per
     w = random_weights(cfg, mc.ParallelLayout(), dev, seed=0)
     ps = cfg.default_page_size
     blocks = (prompt + steps + warmup + ps) // ps + 1
-    dec = Decoder(cfg, w, num_pages=B * blocks + 1, max_pos=prompt + steps + warmup + 64)
+    dec = Decoder(cfg, w, num_pages=B * blocks + 1, max_pos=prompt + steps + warmup + 64, state_slots=B)
     run = ModelRunner(dec, blocks, ctx_hint=prompt + steps // 2)
     g = torch.Generator().manual_seed(1)
     prompts = torch.randint(0, cfg.vocab_size, (B, prompt), generator=g).tolist()
     tables = [list(range(1 + s * blocks, 1 + (s + 1) * blocks)) for s in range(B)]
     first = []
     for c in range(0, B, prompts_per_chunk):
-        first += run.prefill([(prompts[s], tables[s], 0) for s in range(c, min(B, c + prompts_per_chunk))])
-    inp, _ = run._prefill_inputs([(prompts[s], tables[s], 0) for s in range(prompts_per_chunk)], None)
+        first += run.prefill([(prompts[s], tables[s], 0, s) for s in range(c, min(B, c + prompts_per_chunk))])
+    inp, _ = run._prefill_inputs([(prompts[s], tables[s], 0, s) for s in range(prompts_per_chunk)], None)
     ev = lambda: torch.cuda.Event(enable_timing=True)      # noqa: E731
     pf = []
     for _ in range(repeats + 2):
@@ -288,7 +289,11 @@ def prefill_kernels(new, near, S=4, L=2048):
     return out
 
 
-def kernel_rows(new, near, iters=12, warmup=4):
+DESIGNS = {"zarorax": (("moe-2k", "moe-4k", "dense-4k"), size_config, decode_kernels, prefill_kernels),
+           "sikalorn": (parallel.SIZES, parallel.size_config, parallel.decode_kernels, parallel.prefill_kernels)}
+
+
+def kernel_rows(design, new, near, iters=12, warmup=4):
     pk = peaks()
 
     def far(make, graph):
@@ -297,7 +302,7 @@ def kernel_rows(new, near, iters=12, warmup=4):
         best = max(by / (pk["hbm_gbs"] * 1e3), fl / (pk["bf16_tflops"] * 1e6))
         return us, us / best, by, fl
     rows = []
-    for phase, table in (("decode", decode_kernels(new, near)), ("prefill", prefill_kernels(new, near))):
+    for phase, table in (("decode", DESIGNS[design][2](new, near)), ("prefill", DESIGNS[design][3](new, near))):
         for name, a, b in table:
             ua, fa, by, fl = far(a, phase == "decode")
             torch.cuda.empty_cache()
@@ -309,31 +314,30 @@ def kernel_rows(new, near, iters=12, warmup=4):
     return rows
 
 
-SIZES = ("moe-2k", "moe-4k", "dense-4k")
-
-
-def run(sizes=SIZES, only=("throughput", "kernels"), emit=print):
-    for s in sizes:
-        new, near = size_config(s)
-        res = {"size": s, "config": {"batch": 64, "prompt": 512, "decode_context": "512 + steps", "prefill_tokens": 8192, "weights": "random",
-                                     "width": new.hidden_size, "heads": new.num_heads, "kv_rank": 512}, "peaks": peaks()}
+def run(design, sizes=None, only=("throughput", "kernels"), emit=print):
+    for s in sizes or DESIGNS[design][0]:
+        new, near = DESIGNS[design][1](s)
+        about = parallel.describe(new) if new.is_parallel else {"width": new.hidden_size, "heads": new.num_heads, "kv_rank": 512}
+        res = {"size": s, "config": {"batch": 64, "prompt": 512, "decode_context": "512 + steps", "prefill_tokens": 8192, "weights": "random", **about},
+               "peaks": peaks()}
         if "throughput" in only:
             res["design"] = throughput(new)
             torch.cuda.empty_cache()
             res["closest"] = throughput(near)
             torch.cuda.empty_cache()
         if "kernels" in only:
-            res["kernels"] = kernel_rows(new, near)
+            res["kernels"] = kernel_rows(design, new, near)
         emit(json.dumps(res))
 
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("--size", default="all", help="all, or a comma-separated list of: " + ", ".join(SIZES))
+    ap.add_argument("--design", default="zarorax", choices=sorted(DESIGNS))
+    ap.add_argument("--size", default="all", help="all, or a comma-separated list of: " + "; ".join(f"{d}: {', '.join(v[0])}" for d, v in DESIGNS.items()))
     ap.add_argument("--only", default="throughput,kernels")
     a = ap.parse_args(argv)
     with torch.no_grad():
-        run(SIZES if a.size == "all" else a.size.split(","), a.only.split(","))
+        run(a.design, None if a.size == "all" else a.size.split(","), a.only.split(","))
 
 
 if __name__ == "__main__":
