@@ -3,7 +3,7 @@
 //   S <- g S + k u^T,   o = S^T q (+ skip v)
 //     delta      g = exp(neg_decay softplus(a + dt_bias)),  u = beta (v - (g S)^T k),  beta = sigmoid(b);  q, k unit vectors
 //     ssd        g = exp(neg_decay dt),  dt = softplus(dt_raw + dt_bias),  u = dt v
-//     lightning  g = exp(neg_decay),  u = v
+//     lightning  g fixed per head (neg_decay its logarithm),  u = v
 //
 // q, k, v are projections that passed a short causal convolution over time (delta, ssd) and silu. Query / key heads may be
 // shared: head h uses h / (H / G).
@@ -146,7 +146,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
   }
   float log_g, coef;
   rec_gates<T>(p, row, h, &log_g, &coef);
-  const float g = expf(log_g);
+  const float g = p.decay ? p.decay[h] : expf(log_g);
   float qk = 0.f;
   for (int n = tid; n < p.D; n += RS_THREADS) qk += (q_s[n] * rq) * (k_s[n] * rk);
   float ks[VPT], qs[VPT];
@@ -231,7 +231,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
   if (warp == RS_WARPS - 1 && lane < heads) {
     float log_g, coef;
     rec_gates<T>(p, row, h0 + lane, &log_g, &coef);
-    gate_s[lane] = make_float2(expf(log_g), coef);
+    gate_s[lane] = make_float2(p.decay ? p.decay[h0 + lane] : expf(log_g), coef);
   }
   float2 sq = make_float2(0.f, 0.f);
   const int at = p.taps > 1 ? pos % p.taps : 0;
@@ -568,7 +568,7 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, const 
     }
     if (tid < cnt) {
       const float* gt = c.gates + ((size_t)(t0 + b0 + tid) * p.H + h) * 2;
-      g_s[tid] = expf(gt[0]);
+      g_s[tid] = p.decay ? p.decay[h] : expf(gt[0]);
       coef_s[tid] = gt[1];
     }
     __syncthreads();

@@ -12,7 +12,8 @@ typedef struct SkeinRecParams {
   void* tail;                // [slots, taps, C] the convolution's last inputs, or null (taps == 1)
   const float* conv_w;       // [taps, C] channels q | k | v; null without a convolution
   const float* conv_b;       // [C] or null
-  const float* neg_decay;    // [H]
+  const float* neg_decay;    // [H] factor of the step in the log decay; lightning: the log decay
+  const float* decay;        // [H] lightning: the decay itself, which steps one by one take as it is, or null
   const float* dt_bias;      // [H] or null
   const float* skip;         // [H] or null
   const int32_t* positions;  // [rows], -1: padding row

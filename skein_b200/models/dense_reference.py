@@ -190,7 +190,7 @@ def _forward_parallel(cfg, w, token_ids, capture_hidden):
             q = q * D ** -0.5
         q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)
         if r.kind == "lightning":
-            g, coef = rw.neg_decay.exp().expand(T, H), torch.ones(T, H, device=x.device)
+            g, coef = rw.decay.expand(T, H), torch.ones(T, H, device=x.device)
         else:
             a0 = at["dt" if r.kind == "ssd" else "a"]
             step = act.softplus(z[:, a0:a0 + H] + rw.dt_bias)

@@ -332,6 +332,7 @@ class RecurrentWeights:
     conv: torch.Tensor | None = None       # [taps, channels] fp32, channels q | k | v (zero taps of "lightning": none)
     conv_b: torch.Tensor | None = None     # [channels] fp32
     neg_decay: torch.Tensor | None = None  # [heads] fp32: -exp(A_log), or log(decay) of "lightning"
+    decay: torch.Tensor | None = None      # [heads] fp32, "lightning"
     dt_bias: torch.Tensor | None = None    # [heads] fp32
     skip: torch.Tensor | None = None       # [heads] fp32: D
 
@@ -373,7 +374,8 @@ def _load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
     w = RecurrentWeights(norm=get(p + "norm").float())
     GD, HV = m.groups * m.dim, m.heads * m.vdim
     if m.kind == "lightning":
-        w.neg_decay = torch.tensor(m.decay, dtype=torch.float64).log().clamp(min=-1e30).float().to(w.norm.device)
+        d = torch.tensor(m.decay, dtype=torch.float64)
+        w.decay, w.neg_decay = (t.to(w.norm.device) for t in (d.float(), d.log().clamp(min=-1e30).float()))
         return w
     w.neg_decay, w.dt_bias = -get(p + "A_log").float().exp(), get(p + "dt_bias").float()
     if m.kind == "delta":

@@ -43,7 +43,7 @@ class GemmParams(C.Structure):
 class RecParams(C.Structure):
     """Mirror of SkeinRecParams in csrc/kernels/recurrent.cuh (same field order)."""
 
-    _fields_ = [(n, C.c_void_p) for n in ("row", "out", "state", "tail", "conv_w", "conv_b", "neg_decay", "dt_bias", "skip", "positions",
+    _fields_ = [(n, C.c_void_p) for n in ("row", "out", "state", "tail", "conv_w", "conv_b", "neg_decay", "decay", "dt_bias", "skip", "positions",
                                           "slots", "status")] + [("ld", C.c_int64)] + [
         (n, C.c_int32) for n in ("kind", "H", "G", "D", "V", "taps", "C", "q_col", "k_col", "v_col", "a_col", "b_col", "num_slots")]
 

@@ -56,7 +56,8 @@ def _params(row, cols, spec, w, state, positions, slots, out) -> "_lib.RecParams
     p = _lib.RecParams()
     p.row, p.out, p.ld = row.data_ptr(), out.data_ptr(), row.stride(0)
     p.state, p.tail = state.mat.data_ptr(), _lib.ptr(state.tail)
-    p.conv_w, p.conv_b, p.neg_decay, p.dt_bias, p.skip = (_lib.ptr(t) for t in (w.conv, w.conv_b, w.neg_decay, w.dt_bias, w.skip))
+    p.conv_w, p.conv_b, p.neg_decay, p.decay, p.dt_bias, p.skip = (
+        _lib.ptr(t) for t in (w.conv, w.conv_b, w.neg_decay, w.decay, w.dt_bias, w.skip))
     p.positions, p.slots, p.status = positions.data_ptr(), slots.data_ptr(), F.workspace().status.data_ptr()
     p.kind, p.H, p.G, p.D, p.V, p.taps, p.C = KINDS[spec.kind], spec.heads, spec.groups, spec.dim, spec.vdim, spec.taps, spec.conv_channels
     p.q_col, p.k_col, p.v_col, p.a_col, p.b_col, p.num_slots = cols.q, cols.k, cols.v, cols.a, cols.b, state.mat.shape[0]

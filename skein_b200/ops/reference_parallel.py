@@ -96,7 +96,7 @@ def rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len):
             q = q * D ** -0.5
         q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)
         if spec.kind == "lightning":
-            g, coef = w.neg_decay.exp().expand(n, H), torch.ones(n, H)
+            g, coef = (w.neg_decay.exp() if w.decay is None else w.decay).expand(n, H), torch.ones(n, H)
         else:
             step = torch.nn.functional.softplus(r[:, cols.a:cols.a + H] + w.dt_bias, threshold=60.0)
             g = (w.neg_decay * step).exp()

@@ -216,6 +216,7 @@ def rec_case(r, T, dtype, seed=0):
     row = rnd(T, at, dtype=dtype, seed=seed)
     w = RecurrentWeights(norm=torch.ones(1))
     if r.kind == "lightning":
+        w.decay = torch.tensor(r.decay)
         w.neg_decay = torch.tensor(r.decay, dtype=torch.float64).log().clamp(min=-1e30).float()
     else:
         w.neg_decay, w.dt_bias = -torch.exp(rnd(H, dtype=F32)), rnd(H, dtype=F32, seed=3) - 1.0
@@ -300,7 +301,7 @@ def test_long_recurrence_keeps_an_early_write(name):
     r = RECS[name]
     n = 700
     row, cols, w = rec_case(r, n, BF, seed=5)
-    w.neg_decay = torch.full((r.heads,), -1e-4)
+    w.neg_decay, w.decay = torch.full((r.heads,), -1e-4), None
     st = rec.RecState.make(r, 1, BF, "cpu")
     want = run_steps(r, [row], cols, w, st, [0], [[(0, n)]], "cpu")[0]
     lost = run_steps(r, [torch.cat([row[:60] * 0, row[60:]])], cols, w, rec.RecState.make(r, 1, BF, "cpu"), [0], [[(0, n)]], "cpu")[0]
