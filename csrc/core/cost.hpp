@@ -186,7 +186,7 @@ inline uint64_t layer_flops(const Layer& l, const ModelMeta& meta, const Workloa
       return qkvo + scores + softmax + scores;
     }
     case LayerKind::Mlp: return (l.activation == "silu" ? 6 : 4) * b * s * l.hidden * l.intermediate;   // two or (ungated) one projections up, one down
-    case LayerKind::Moe: return 2 * b * s * l.hidden * l.num_experts + 6 * b * s * l.top_k * l.hidden * l.intermediate;
+    case LayerKind::Moe: return 2 * b * s * l.hidden * l.num_experts + 6 * b * s * l.hidden * (l.top_k * l.intermediate + l.always_ff);
     case LayerKind::Lmhead: return 2 * b * s * l.vocab * l.hidden;
   }
   return 0;
@@ -222,7 +222,8 @@ inline double layer_stream_bytes(const Layer& l, const ModelMeta& meta, Dtype wd
     // experts actually touched by batch*top_k routed tokens (uniform routing): E * (1 - (1 - 1/E)^(b*k))
     const double E = (double)l.num_experts, draws = (double)wl.batch * wl.seq_len * l.top_k;
     const double touched = E * (1.0 - std::pow(1.0 - 1.0 / E, draws));
-    elems *= touched / E;
+    const double always = 3.0 * (double)l.hidden * (double)l.always_ff;      // an expert of every token
+    elems = always + (elems - always) * touched / E;
   }
   double bytes = (double)dtype_bits(wd) / 8.0 * elems / div;
   if (l.kind == LayerKind::Attention)
@@ -282,10 +283,10 @@ inline double block_compute_time(size_t block, const Graph& ir, Dtype wd, Dtype 
 inline uint32_t kernels_per_layer(const Layer& l) {
   switch (l.kind) {
     case LayerKind::Attention:
-      if (l.parallel) return 3 + (l.kv_elems > 0 ? 2 : 0) + (l.state_elems > 0 ? 2 : 0) + (l.opens_pass ? 2 : 0);  // in, out, sum + norm; append, attention; step, norm
+      if (l.parallel) return 3 + (l.kv_elems > 0 ? 2 : 0) + (l.state_elems > 0 ? 2 : 0) + (l.opens_pass && !l.selective ? 2 : 0) + (l.selective ? 2 : 0);  // in, out, sum + norm; append, attention; step, norm
       return l.kv_rank > 0 ? (l.q_rank > 0 ? 8 : 7) : 4;  // latent: input projection, append, (q up,) absorb, attention, values, o_proj, norm; qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
     case LayerKind::Mlp: return l.activation == "relu2" ? 0 : 3;   // (of a parallel layer: inside the mixer's two products)        // gate/up GEMM (SwiGLU epilogue), down GEMM, reduce+norm
-    case LayerKind::Moe: return 3;        // grouped gate/up (gathers its rows), grouped down, combine + norm
+    case LayerKind::Moe: return l.always_ff > 0 ? 5 : 3;        // grouped gate/up (gathers its rows), grouped down, combine + norm
     case LayerKind::RmsNorm: return 0;    // fused into the reduce kernels above
     default: return 1;
   }
@@ -364,7 +365,7 @@ inline uint64_t block_kv_elems_per_token(const Graph& ir, size_t block) {
   return 2ull * ir.meta.num_kv_heads * ir.meta.head_dim;
 }
 inline uint64_t block_state_bytes(const Graph& ir, size_t block) {
-  if (ir.meta.parallel)
+  if (ir.meta.layered)
     for (auto& l : ir.layers) if (l.kind == LayerKind::Attention && l.block_idx && *l.block_idx == block) return l.state_bytes;
   return 0;
 }

@@ -131,6 +131,32 @@ inline Graph import_layered(const Json& cfg) {
   return g;
 }
 
+// The runs of a list of layers of which a range may run several times (`loop`).
+struct LoopRuns {
+  size_t start = 0, stop = 0, times = 1;
+  bool looped = false;
+  std::vector<std::pair<size_t, size_t>> runs;      // (layer, pass)
+  bool opens(size_t layer) const { return looped && layer == start; }
+};
+inline LoopRuns read_loop(const Json& cfg, size_t n) {
+  LoopRuns l;
+  if (const Json* loop = cfg.find("loop"); loop && !loop->is_null()) {
+    l.looped = true;
+    l.start = cfg_usize(*loop, "start"); l.stop = cfg_usize(*loop, "stop"); l.times = cfg_usize(*loop, "times");
+    if (l.start >= l.stop || l.stop > n || l.times < 1) throw ImportError("config.json: `loop` is not a range of the layers");
+  }
+  for (size_t i = 0; i < n;) {
+    if (l.opens(i)) {
+      for (size_t t = 0; t < l.times; ++t)
+        for (size_t j = l.start; j < l.stop; ++j) l.runs.push_back({j, t});
+      i = l.stop;
+    } else {
+      l.runs.push_back({i++, 0});
+    }
+  }
+  return l;
+}
+
 // A design of parallel layers (Sikalorn): x <- x + (mixer(h) + ff(h)) with h = tanh(alpha x) w + b, and a range of layers that
 // may run several times. One block per run; the runs after a layer's first own no parameters.
 inline Graph import_parallel(const Json& cfg) {
@@ -146,23 +172,8 @@ inline Graph import_parallel(const Json& cfg) {
   const auto& layers = cfg.at("layers").items();
   if (layers.empty()) throw ImportError("config.json: `layers` is empty");
   m.num_kv_heads = 1;
-  size_t start = 0, stop = 0, times = 1;
-  const Json* loop = cfg.find("loop");
-  const bool looped = loop && !loop->is_null();
-  if (looped) {
-    start = cfg_usize(*loop, "start"); stop = cfg_usize(*loop, "stop"); times = cfg_usize(*loop, "times");
-    if (start >= stop || stop > layers.size() || times < 1) throw ImportError("config.json: `loop` is not a range of the layers");
-  }
-  std::vector<std::pair<size_t, size_t>> runs;      // (layer, pass)
-  for (size_t i = 0; i < layers.size();) {
-    if (looped && i == start) {
-      for (size_t t = 0; t < times; ++t)
-        for (size_t j = start; j < stop; ++j) runs.push_back({j, t});
-      i = stop;
-    } else {
-      runs.push_back({i++, 0});
-    }
-  }
+  const LoopRuns lr = read_loop(cfg, layers.size());
+  const auto& runs = lr.runs;
   m.num_layers = runs.size();
   Graph g;
   size_t idx = 0;
@@ -248,10 +259,10 @@ inline Graph import_parallel(const Json& cfg) {
     } else {
       throw ImportError("layer " + std::to_string(i) + ": mixer type `" + type + "` is not supported");
     }
-    if (looped && i == start) {
+    if (lr.opens(i)) {
       a.opens_pass = true;
       ps.push_back({"loop.in", {C, 2 * C}, Dtype::Bf16});
-      ps.push_back({"loop.step", {times, C}, Dtype::Bf16});
+      ps.push_back({"loop.step", {lr.times, C}, Dtype::Bf16});
     }
     if (shared) a.shared_elems = elems(ps); else a.params = ps;
     if (!d.has("mlp") || d.at("mlp").is_null()) continue;
@@ -274,10 +285,134 @@ inline Graph import_parallel(const Json& cfg) {
   return g;
 }
 
+// A design of pre-norm layers with an fp32 stream (Barorax): differential attention, attention inside chunks, selective scans; routed
+// experts with one that runs for every token; a range of layers that may run several times. One block per run; the runs after a
+// layer's first own no parameters.
+inline Graph import_prenorm(const Json& cfg) {
+  ModelMeta m;
+  m.architecture = cfg.at("architecture").as_string();
+  m.layered = m.prenorm = true;
+  m.hidden = cfg_usize(cfg, "width");
+  m.vocab = cfg_usize(cfg, "vocab");
+  m.max_position = cfg.has("max_position_embeddings") && !cfg.at("max_position_embeddings").is_null() ? cfg_usize(cfg, "max_position_embeddings") : 131072;
+  for (const char* k : {"norm", "layers"})
+    if (!cfg.has(k)) throw ImportError(std::string("config.json: missing `") + k + "`");
+  m.rms_norm_eps = cfg.at("norm").at("eps").as_double();
+  const auto& layers = cfg.at("layers").items();
+  if (layers.empty()) throw ImportError("config.json: `layers` is empty");
+  m.num_kv_heads = 1;
+  const LoopRuns lr = read_loop(cfg, layers.size());
+  m.num_layers = lr.runs.size();
+  Graph g;
+  size_t idx = 0;
+  const uint64_t C = m.hidden;
+  auto add = [&](LayerKind k, std::optional<size_t> block, const std::string& label) -> Layer& {
+    Layer l;
+    l.idx = idx++; l.block_idx = block; l.kind = k; l.label = label; l.hidden = m.hidden; l.eps = m.rms_norm_eps;
+    g.layers.push_back(l);
+    return g.layers.back();
+  };
+  auto elems = [](const std::vector<Param>& ps) { uint64_t n = 0; for (auto& p : ps) n += p.numel(); return n; };
+  Layer& em = add(LayerKind::Embedding, std::nullopt, "embed_tokens");
+  em.vocab = m.vocab;
+  em.params.push_back({"embed", {m.vocab, C}, Dtype::Bf16});
+  for (size_t b = 0; b < lr.runs.size(); ++b) {
+    const auto [i, pass] = lr.runs[b];
+    const bool shared = pass > 0;
+    const Json& d = layers[i];
+    const std::string type = d.at("type").as_string(), p = "l" + std::to_string(i) + ".", q = p + "mix.";
+    {
+      Layer& n1 = add(LayerKind::RmsNorm, b, "norm1");
+      if (!shared) n1.params.push_back({p + "norm1", {C}, Dtype::Bf16});
+    }
+    std::vector<Param> ps;
+    Layer& a = add(LayerKind::Attention, b, type);
+    a.parallel = true;
+    const Json& mx = d.at("mixer");
+    auto param = [&](const std::string& n, std::vector<uint64_t> shape) { ps.push_back({q + n, std::move(shape), Dtype::Bf16}); };
+    if (type == "attention" || type == "attention_2") {
+      const bool differential = type == "attention";
+      const uint64_t H = cfg_usize(mx, "heads"), K = cfg_usize(mx, "kv_heads"), D = cfg_usize(mx, "dim"), V = cfg_usize(mx, "vdim"), M = differential ? 2 : 1;
+      param("q", {H * M * D, C});
+      param("k", {K * M * D, C});
+      param("v", {K * V, C});
+      if (differential) {
+        for (const char* n : {"lq1", "lk1", "lq2", "lk2"}) param(n, {D});
+        param("g", {H * V, C});
+      } else {
+        a.window = cfg_usize(mx.at("mask"), "size");     // a row sees at most its chunk
+      }
+      param("o", {C, H * V});
+      a.num_heads = H * M; a.num_kv_heads = K; a.head_dim = D; a.v_dim = V; a.kv_elems = K * (M * D + V); a.gated = differential;
+      a.rope_theta = mx.at("rot").at("base").as_double();
+      m.rope_theta = a.rope_theta;
+      m.num_attention_heads = std::max<size_t>(m.num_attention_heads, H);
+      m.head_dim = std::max<size_t>(m.head_dim, D);
+    } else if (type == "mamba1") {
+      const uint64_t I = cfg_usize(mx, "inner"), N = cfg_usize(mx, "state"), R = cfg_usize(mx, "dt_rank"), taps = cfg_usize(mx, "conv");
+      param("in", {2 * I, C});
+      param("conv", {I, taps});
+      param("conv.b", {I});
+      param("x", {R + 2 * N, I});
+      param("dt", {I, R});
+      param("dt.b", {I});
+      param("A_log", {I, N});
+      param("D", {I});
+      param("o", {C, I});
+      a.selective = true;
+      a.num_heads = a.num_kv_heads = 1; a.head_dim = N; a.v_dim = I;
+      a.conv_taps = taps;
+      a.state_elems = I * N;
+      a.state_bytes = 4 * I * N + (taps > 1 ? 2 * taps * I : 0);
+      m.num_attention_heads = std::max<size_t>(m.num_attention_heads, 1);
+      m.head_dim = std::max<size_t>(m.head_dim, N);
+    } else {
+      throw ImportError("layer " + std::to_string(i) + ": mixer type `" + type + "` is not supported");
+    }
+    if (lr.opens(i)) {
+      a.opens_pass = true;
+      ps.push_back({"loop.step", {lr.times, C}, Dtype::Bf16});
+    }
+    if (shared) a.shared_elems = elems(ps); else a.params = ps;
+    if (!d.has("mlp") || d.at("mlp").is_null()) continue;
+    const Json& ml = d.at("mlp");
+    if (ml.at("kind").as_string() != "moe") throw ImportError("layer " + std::to_string(i) + ": feed-forward kind `" + ml.at("kind").as_string() + "` is not supported");
+    {
+      Layer& n2 = add(LayerKind::RmsNorm, b, "norm2");
+      if (!shared) n2.params.push_back({p + "norm2", {C}, Dtype::Bf16});
+    }
+    const uint64_t F = cfg_usize(ml.at("expert"), "ff"), E = cfg_usize(ml.at("router"), "experts");
+    ps.clear();
+    auto expert = [&](const std::string& n, uint64_t ff) {
+      ps.push_back({n + "gate", {ff, C}, Dtype::Bf16});
+      ps.push_back({n + "up", {ff, C}, Dtype::Bf16});
+      ps.push_back({n + "down", {C, ff}, Dtype::Bf16});
+    };
+    for (uint64_t e = 0; e < E; ++e) expert(p + "mlp.e" + std::to_string(e) + ".", F);
+    ps.push_back({p + "mlp.router", {E, C}, Dtype::Bf16});
+    Layer& f = add(LayerKind::Moe, b, "moe");
+    if (ml.has("shared") && !ml.at("shared").is_null()) {
+      f.always_ff = cfg_usize(ml.at("shared"), "ff");
+      expert(p + "mlp.shared.", f.always_ff);
+    }
+    f.intermediate = F; f.num_experts = E; f.top_k = cfg_usize(ml.at("router"), "top");
+    if (shared) f.shared_elems = elems(ps); else f.params = ps;
+    m.intermediate = std::max<size_t>(m.intermediate, F * E);
+  }
+  Layer& n = add(LayerKind::RmsNorm, std::nullopt, "norm");
+  n.params.push_back({"final.norm", {C}, Dtype::Bf16});
+  Layer& l = add(LayerKind::Lmhead, std::nullopt, "lm_head");
+  l.vocab = m.vocab;
+  l.params.push_back({"head", {m.vocab, C}, Dtype::Bf16});
+  g.meta = m;
+  return g;
+}
+
 inline Graph import_model(const Json& cfg) {
   if (const Json* a = cfg.find("architecture"); a && !a->is_null()) {
     if (a->as_string() == "Zarorax") return import_layered(cfg);
     if (a->as_string() == "Sikalorn") return import_parallel(cfg);
+    if (a->as_string() == "Barorax") return import_prenorm(cfg);
   }
   const Json* archs = cfg.find("architectures");
   if (!archs || !archs->is_array() || archs->size() == 0) throw ImportError("config.json: `architectures` is missing or empty");

@@ -78,14 +78,16 @@ struct Layer {
   size_t conv_taps = 0;       // the layer's input passes a short causal convolution whose last inputs are cached
   uint64_t shared_elems = 0;  // parameter elements read from another layer's tensors (weights_of), which own no bytes here
   std::string activation = "silu";
-  // mixer of a parallel layer (x + mixer(h) + ff(h)): an attention over a window, a recurrence with a 32-bit state per sequence,
-  // or both beside each other
+  // mixer of a parallel layer (x + mixer(h) + ff(h)) or of a pre-norm layer with an fp32 stream: an attention over a window, a
+  // recurrence with a 32-bit state per sequence, or both beside each other
   bool parallel = false;
   size_t window = 0;           // 0: no window
   uint64_t kv_elems = 0;       // cache elements per token
   uint64_t state_elems = 0;    // elements of the recurrent state
   uint64_t state_bytes = 0;    // bytes of one sequence's state, its convolution inputs included
   bool opens_pass = false;     // the first layer of a pass of the loop
+  bool selective = false;      // the recurrence is a selective scan: two small products of its own in front of it
+  size_t always_ff = 0;        // routed feed-forward: size of an expert that runs for every token
   std::string label;  // e.g. "input_layernorm", "self_attn"
   std::vector<Param> params;
 };
@@ -100,6 +102,7 @@ struct ModelMeta {
   bool qkv_bias = false;       // the q / k / v projections carry a bias vector each (Qwen2)
   bool layered = false;        // the configuration lists its layers one by one; runs on one device
   bool parallel = false;       // ... and they are parallel layers
+  bool prenorm = false;        // ... or pre-norm layers
 
   Json to_json() const {
     Json j = Json::object();
@@ -113,6 +116,7 @@ struct ModelMeta {
     if (qkv_bias) j.set("qkv_bias", true);      // written only when set: plans of models without biases keep their hash
     if (layered) j.set("layered", true);
     if (parallel) j.set("parallel", true);
+    if (prenorm) j.set("prenorm", true);
     return j;
   }
   static ModelMeta from_json(const Json& j) {
@@ -132,6 +136,7 @@ struct ModelMeta {
     if (const Json* qb = j.find("qkv_bias"); qb && !qb->is_null()) m.qkv_bias = qb->as_bool();
     if (const Json* ly = j.find("layered"); ly && !ly->is_null()) m.layered = ly->as_bool();
     if (const Json* pa = j.find("parallel"); pa && !pa->is_null()) m.parallel = pa->as_bool();
+    if (const Json* pr = j.find("prenorm"); pr && !pr->is_null()) m.prenorm = pr->as_bool();
     return m;
   }
   bool is_moe() const { return num_experts && *num_experts > 0; }
@@ -186,6 +191,7 @@ inline Json Graph::to_json() const {
       case LayerKind::Moe:
         k.set("num_experts", l.num_experts).set("top_k", l.top_k).set("hidden", l.hidden)
             .set("intermediate", l.intermediate).set("activation", l.activation);
+        if (l.always_ff > 0) k.set("shared_intermediate", l.always_ff);
         break;
       case LayerKind::Lmhead: k.set("vocab", l.vocab).set("hidden", l.hidden).set("tied", l.tied); break;
     }

@@ -14,10 +14,15 @@
 //   memory; with splits > 1 the CTA parks its state in a workspace and the last CTA of a
 //   (sequence, kv head) to arrive merges the splits, as in the scalar kernel.
 //
+// Differential heads (SkeinAttnRule.maps == 2): a key head holds its two maps side by side in the 128 columns. Each map of a query head is
+// a row of the tile whose other half is zero, so that one product gives the scores of both maps; the maps of a head are subtracted, normed
+// and gated where the rows are merged.
+//
 // Cache layout: kv_cache[page, 0 = K / 1 = V, kv_head, slot, 128] bf16 with page_size % 16 == 0.
 // Same operator as the reference's fused_decode_attn (vendor/luminal/crates/luminal_cuda_lite/src/
 // kernel/decode_attention.rs:66-139) and its FlashInfer batch-decode wrapper
 // (vendor/luminal/crates/luminal_cuda_lite/src/host/flashinfer/wrapper.cu:123-251).
+#include "attn_rule.cuh"
 #include "ptx.cuh"
 #include "launch.cuh"
 #include <cuda_bf16.h>
@@ -47,7 +52,7 @@ struct AttnMmaParams {
   int* counters;            // [B * Hkv], zero at first use
   int* status;
   long long q_stride;
-  int B, Hq, Hkv, G, page_size, max_blocks, num_pages, splits;
+  int B, Hq, Hkv, G, page_size, max_blocks, num_pages, splits;   // Hq, G: query rows, the maps of differential heads counted apart
   float scale_log2e;
   // optional fusion of RoPE and the KV append of the new token (cos_sin == nullptr: q is already rotated and
   // the cache already holds the token). q then points at the raw fused q/k/v projection rows
@@ -55,11 +60,16 @@ struct AttnMmaParams {
   const float* cos_sin;     // [max_pos, D/2, 2] fp32
   const int* positions;     // [B] position of the new token, -1 = padding row
   int max_pos;
-  // sliding window: the new token sees the last `window` tokens, itself included (0: all)
-  int window;
   long long out_ld;         // elements between rows of out
-  float out_scale;
+  SkeinAttnRule r;
 };
+
+// softmax sums (reference m in base 2, denominator l) -> factor that normalises the weighted values
+__device__ __forceinline__ float am_norm(float m, float l, int sink) {
+  if (!sink) return l > 0.f ? 1.f / l : 0.f;
+  const float top = fmaxf(m, 0.f), e = exp2f(m - top);
+  return e / (l * e + exp2f(-top));
+}
 
 template <int AM_D>
 __device__ __forceinline__ uint32_t am_swz(int row, int chunk) {  // byte offset in a [16][AM_D] bf16 tile
@@ -105,8 +115,8 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   const int len = p.seq_lens[b];
 
   // this split's token range, rounded to whole pages (pages are multiples of the tile), with a window to whole tiles
-  const int lo = p.window > 0 && len > p.window ? len - p.window : 0;     // first visible token
-  const int base = lo / AM_TILE * AM_TILE, unit = p.window > 0 ? AM_TILE : ps;
+  const int lo = len > 0 ? attn_first_key(p.r.window, p.r.chunk, len - 1) : 0;     // first visible token
+  const int base = lo / AM_TILE * AM_TILE, unit = p.r.window > 0 || p.r.chunk > 0 ? AM_TILE : ps;
   int per = (len - base + p.splits - 1) / p.splits;
   per = (per + unit - 1) / unit * unit;
   const int t_begin = base + split * per;
@@ -128,7 +138,9 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     for (int c = tid; c < AM_TILE * CH; c += AM_THREADS) {
       const int r = c / CH, ch = c % CH;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < G) v = *reinterpret_cast<const uint4*>(p.q + (size_t)b * p.q_stride + (size_t)(kvh * G + r) * AM_D + ch * 8);
+      const int head = (kvh * G + r) / p.r.maps;      // (two maps: row r holds one, its other half stays zero)
+      if (r < G && (p.r.maps == 1 || (ch >= CH / 2) == (r & 1)))
+        v = *reinterpret_cast<const uint4*>(p.q + (size_t)b * p.q_stride + (size_t)head * AM_D + ch * 8);
       *reinterpret_cast<uint4*>(q_s + am_swz<AM_D>(r, ch)) = v;
     }
   } else if (AM_D == 128) {
@@ -315,6 +327,33 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   }
   __syncthreads();
 
+  // two maps: thread d's values of the rows (normalised) -> difference, head norm, gate
+  auto store_pairs = [&](auto value) {
+    __shared__ float red[AM_WARPS][8];
+    float o2[8];
+    const float lam = p.r.lam[0];
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      o2[n] = 0.f;
+      if (2 * n < G) {
+        o2[n] = value(2 * n) - lam * value(2 * n + 1);
+        float ss = o2[n] * o2[n];
+        for (int o_ = 16; o_ > 0; o_ >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o_);
+        if (lane == 0) red[warp][n] = ss;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      if (2 * n >= G) break;
+      const float ss = red[0][n] + red[1][n] + red[2][n] + red[3][n];
+      float a = o2[n] * p.r.out_scale / sqrtf(ss / (float)AM_D + p.r.eps);
+      const size_t col = (size_t)(kvh * G / 2 + n) * AM_D + tid;
+      if (p.r.gate) a /= 1.f + __expf(-__bfloat162float(((const __nv_bfloat16*)p.r.gate)[(size_t)b * p.r.gate_ld + col]));
+      p.out[(size_t)b * p.out_ld + col] = __float2bfloat16(a);
+    }
+  };
+
   // ---- merge the 4 warps: thread d owns output dim d of every head ----
   const int d = AM_D < AM_THREADS ? tid % AM_D : tid;   // (head size 64: the second half of the CTA repeats the first)
   float O_g[16], M_g[16], L_g[16];
@@ -339,9 +378,13 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     }
   }
   if (p.splits == 1) {
+    if (AM_D == AM_THREADS && p.r.maps == 2) {
+      store_pairs([&](int g) { return O_g[g] * am_norm(M_g[g], L_g[g], p.r.sink); });
+      return;
+    }
 #pragma unroll
     for (int g = 0; g < 16; ++g)
-      if (g < G) p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(L_g[g] > 0.f ? O_g[g] / L_g[g] * p.out_scale : 0.f);
+      if (g < G) p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(O_g[g] * am_norm(M_g[g], L_g[g], p.r.sink) * p.r.out_scale);
     return;
   }
 #pragma unroll
@@ -366,6 +409,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   // last CTA of this (sequence, kv head): merge the splits. (m, l) of all heads and splits are staged in
   // shared memory with one parallel load; each thread then fetches its dim of all splits at once.
   float* ml_s = reinterpret_cast<float*>(am_smem);   // [G][splits][2]
+  float* val_s = ml_s + 16 * AM_MAX_SPLITS * 2;      // [G][AM_D], two maps
   const size_t base0 = ((size_t)b * p.Hq + kvh * G) * p.splits;
   for (int i = tid; i < G * p.splits * 2; i += AM_THREADS) ml_s[i] = __ldcg(&p.ws_ml[base0 * 2 + i]);
   __syncthreads();
@@ -386,8 +430,11 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
         O += w * ov[s2];
       }
     }
-    p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(L > 0.f ? O / L * p.out_scale : 0.f);
+    const float a = O * am_norm(M, L, p.r.sink);
+    if (AM_D == AM_THREADS && p.r.maps == 2) val_s[g * AM_D + d] = a;
+    else p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(a * p.r.out_scale);
   }
+  if (AM_D == AM_THREADS && p.r.maps == 2) store_pairs([&](int g) { return val_s[g * AM_D + d]; });      // (a thread reads what it wrote)
 }
 
 }  // namespace skein
@@ -422,24 +469,32 @@ static int attn_decode_mma_go(AttnMmaParams& p, float* ws, void* stream) {
 // first use). Requires D = 128 (64 without RoPE fusion), page_size a multiple of 16, at most 16 query heads per kv head.
 static int attn_decode_mma_launch(const void* q, long long q_stride, void* kv, const int* block_table,
                                   const int* seq_lens, void* out, long long out_ld, float* ws, int* counters, int* status, int B,
-                                  int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits, int window,
-                                  float scale, float out_scale, const float* cos_sin, const int* positions, int max_pos, void* stream) {
+                                  int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits, const SkeinAttnRule& rule,
+                                  const float* cos_sin, const int* positions, int max_pos, void* stream) {
   using namespace skein;
   if (B == 0) return 0;
+  if (rule.maps < 1 || rule.maps > 2 || (rule.maps == 2 && (D != AM_THREADS || !rule.lam)) || (rule.maps == 1 && rule.gate)) return -1;
+  Hq *= rule.maps;
   if ((D != 128 && (D != 64 || cos_sin != nullptr)) || Hq % Hkv != 0 || page_size % AM_TILE != 0) return -1;
   const int G = Hq / Hkv;
-  if (G > 16 || q_stride % 8 != 0 || (uintptr_t)q % 16 != 0 || (window > 0 && cos_sin != nullptr)) return -1;
+  if (G > 16 || q_stride % 8 != 0 || (uintptr_t)q % 16 != 0 || ((rule.window > 0 || rule.chunk > 0) && cos_sin != nullptr)) return -1;
   if (splits < 1 || splits > AM_MAX_SPLITS) return -2;
   if (splits > 1 && (ws == nullptr || counters == nullptr)) return -2;
   AttnMmaParams p;
   p.q = (const __nv_bfloat16*)q; p.kv = (const __nv_bfloat16*)kv; p.kv_rw = (__nv_bfloat16*)kv;
   p.block_table = block_table; p.seq_lens = seq_lens;
   p.cos_sin = cos_sin; p.positions = positions; p.max_pos = max_pos;
-  p.out = (__nv_bfloat16*)out; p.out_ld = out_ld; p.out_scale = out_scale;
+  p.out = (__nv_bfloat16*)out; p.out_ld = out_ld; p.r = rule;
   p.counters = counters; p.status = status; p.q_stride = q_stride;
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.page_size = page_size; p.max_blocks = max_blocks; p.num_pages = num_pages;
-  p.splits = splits; p.scale_log2e = scale * 1.4426950408889634f; p.window = window;
+  p.splits = splits; p.scale_log2e = rule.scale * 1.4426950408889634f;
   return D == 64 ? attn_decode_mma_go<64>(p, ws, stream) : attn_decode_mma_go<128>(p, ws, stream);
+}
+
+static SkeinAttnRule plain_rule(float scale) {
+  SkeinAttnRule r{};
+  r.maps = 1; r.scale = scale; r.out_scale = 1.f;
+  return r;
 }
 
 extern "C" int skein_attn_decode_mma(const void* q, long long q_stride, const void* kv, const int* block_table,
@@ -447,16 +502,16 @@ extern "C" int skein_attn_decode_mma(const void* q, long long q_stride, const vo
                                      int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits,
                                      float scale, void* stream) {
   return attn_decode_mma_launch(q, q_stride, const_cast<void*>(kv), block_table, seq_lens, out, (long long)Hq * D, ws, counters, status, B,
-                                Hq, Hkv, D, page_size, max_blocks, num_pages, splits, 0, scale, 1.f, nullptr, nullptr, 0, stream);
+                                Hq, Hkv, D, page_size, max_blocks, num_pages, splits, plain_rule(scale), nullptr, nullptr, 0, stream);
 }
 
-// The same over a sliding window, into rows out_ld apart, times out_scale.
+// The same under a rule (attn_rule.cuh), into rows out_ld apart. D is the width of a key head; with two maps it must be 128.
 extern "C" int skein_attn_decode_window(const void* q, long long q_stride, const void* kv, const int* block_table,
                                         const int* seq_lens, void* out, long long out_ld, float* ws, int* counters, int* status, int B,
-                                        int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits, int window,
-                                        float scale, float out_scale, void* stream) {
+                                        int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int splits,
+                                        const SkeinAttnRule* rule, void* stream) {
   return attn_decode_mma_launch(q, q_stride, const_cast<void*>(kv), block_table, seq_lens, out, out_ld, ws, counters, status, B, Hq, Hkv, D,
-                                page_size, max_blocks, num_pages, splits, window, scale, out_scale, nullptr, nullptr, 0, stream);
+                                page_size, max_blocks, num_pages, splits, *rule, nullptr, nullptr, 0, stream);
 }
 
 // Decode attention straight from the fused q/k/v projection: rotates q and k (rotate-half RoPE from the fp32
@@ -470,5 +525,5 @@ extern "C" int skein_attn_decode_rope_mma(const void* qkv, long long qkv_stride,
                                           float scale, void* stream) {
   if (cos_sin == nullptr || positions == nullptr) return -1;
   return attn_decode_mma_launch(qkv, qkv_stride, kv, block_table, seq_lens, out, (long long)Hq * D, ws, counters, status, B, Hq, Hkv, D,
-                                page_size, max_blocks, num_pages, splits, 0, scale, 1.f, cos_sin, positions, max_pos, stream);
+                                page_size, max_blocks, num_pages, splits, plain_rule(scale), cos_sin, positions, max_pos, stream);
 }

@@ -2,7 +2,12 @@
 // tensor memory, operands staged by TMA). Same contract as attn_prefill.cu (chunked-prefill aware: a chunk of q_len
 // new tokens attends to the kv_len tokens already in the cache, its own included); this is the kernel the prefill
 // path runs for head sizes 128 and 64 and pages of whole 16-token groups, the mma.sync kernel stays as the fallback for other
-// shapes. With a sliding window a row sees its last `window` keys only; tiles before the window of a CTA's first row are skipped.
+// shapes. With a window or chunks (SkeinAttnRule) a row sees part of the keys before it only; tiles before the first key of a CTA's first
+// row are skipped.
+//
+// Differential heads (two maps over the same values, side by side in the 128 columns of a query or key head): the tile's 128 rows are two
+// maps of 64 query rows, each with the other map's half set to zero, so that one product gives both maps' scores; at the end the rows of
+// the second map hand their outputs over through shared memory, and the rows of the first one subtract, norm and gate them.
 //
 // One CTA = 128 query rows of one head, walking the context in 128-token tiles:
 //
@@ -26,6 +31,7 @@
 // The reference never runs a prefill attention kernel: its FlashInfer prefill wrapper returns -1
 // (vendor/luminal/crates/luminal_cuda_lite/src/host/flashinfer/wrapper.cu:263-281) and prefill falls back to unfused
 // graph ops (crates/skein_emit/src/op_wiring.rs:2155-2305).
+#include "attn_rule.cuh"
 #include "ptx.cuh"
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -50,28 +56,33 @@ struct AttnPrefillTcParams {
   __nv_bfloat16* out;       // [T, Hq * D]
   int* status;
   int Hq, Hkv, max_blocks, num_pages, page_size;
-  int window;               // keys a row sees, its own included (0: all)
   long long out_ld;         // elements between rows of out
-  float scale_log2e, out_scale;
+  float scale_log2e;
+  SkeinAttnRule r;
 };
 
-template <int TC_D>
+constexpr int TC_X_LD = 132;            // floats between rows of the second map's outputs in shared memory
+
+template <int TC_D, int MAPS>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        const AttnPrefillTcParams p) {
   constexpr int HALVES = TC_D / 64, TC_TILE_BYTES = HALVES * TC_HALF_BYTES;
+  constexpr int QR = TC_BM / MAPS;                          // query rows of a tile
+  static_assert(MAPS == 1 || TC_D == 128, "two maps fill the two halves of a head");
   const int qt = (int)gridDim.x - 1 - (int)blockIdx.x;     // long rows first: the causal work grows with the row
   const int head = blockIdx.y, seq = blockIdx.z;
   const int qlen = p.q_len[seq];
-  const int q0 = qt * TC_BM;
+  const int q0 = qt * QR;
   if (q0 >= qlen) return;
   const int kvlen = p.kv_len[seq];
   const int pos0 = kvlen - qlen;                            // absolute position of the chunk's first token
   const int qrow0 = p.q_start[seq];
   const int kvh = head / (p.Hq / p.Hkv);
-  int kv_hi = pos0 + min(q0 + TC_BM, qlen);                 // exclusive bound of the keys any row of this tile sees
+  int kv_hi = pos0 + min(q0 + QR, qlen);                    // exclusive bound of the keys any row of this tile sees
   if (kv_hi > kvlen) kv_hi = kvlen;
-  const int kv_lo = p.window > 0 && pos0 + q0 - p.window + 1 > 0 ? pos0 + q0 - p.window + 1 : 0;   // first key of the first row
+  const int kv_lo = attn_first_key(p.r.window, p.r.chunk, pos0 + q0);                    // first key of the first row
+  const int last_lo = attn_first_key(p.r.window, p.r.chunk, pos0 + q0 + QR - 1);         // ... and of the last
   const int first_tile = kv_lo / TC_BN;
   const int n_tiles = (kv_hi + TC_BN - 1) / TC_BN - first_tile;
 
@@ -97,6 +108,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     tmem_alloc(smem_u32(tmem_slot), TC_TMEM_COLS);
     tmem_relinquish();
   }
+  if (MAPS == 2) {      // the halves of Q that no copy fills: rows 64 .. of the first, rows .. 63 of the second
+    for (int i = tid; i < 2 * 64 * 8; i += TC_THREADS) {
+      const uint32_t a = q_s + (i < 64 * 8 ? 64 * 128 + i * 16 : TC_HALF_BYTES + (i - 64 * 8) * 16);
+      asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};" ::"r"(a), "r"(0) : "memory");
+    }
+    fence_proxy_async_smem();
+  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -109,8 +127,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmKV);
       const uint64_t pol_q = l2_policy_evict_first(), pol_kv = l2_policy_evict_last();
-      mbar_expect_tx(bar_q, TC_TILE_BYTES);
-      for (int hf = 0; hf < HALVES; ++hf) tma_load_2d(q_s + hf * TC_HALF_BYTES, &tmQ, bar_q, head * TC_D + hf * 64, qrow0 + q0, pol_q);
+      mbar_expect_tx(bar_q, TC_TILE_BYTES / MAPS);
+      for (int hf = 0; hf < HALVES; ++hf)
+        tma_load_2d(q_s + hf * TC_HALF_BYTES + (MAPS == 2 ? hf * 64 * 128 : 0), &tmQ, bar_q, head * TC_D + hf * 64, qrow0 + q0, pol_q);
       bool ok = true;
       int armed_k = 0, armed_v = 0;      // phases armed so far (for the bounded drain on an early exit)
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -173,8 +192,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int lane_grp = warp & 3;                      // the 32 tensor-memory lanes this warp may access
     const int r = lane_grp * 32 + lane;                 // row of the tile
     const uint32_t lane_addr = (uint32_t)(lane_grp * 32) << 16;
-    int pos_r = pos0 + q0 + r;
+    const int qi = r % QR;                              // its query row (rows QR .. are the second map's)
+    int pos_r = pos0 + q0 + qi;
     if (pos_r > kvlen - 1) pos_r = kvlen - 1;           // rows past the chunk are computed, finite, and never stored
+    const int first_key = attn_first_key(p.r.window, p.r.chunk, pos_r);
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
@@ -182,9 +203,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (!mbar_wait(bar_sfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
       tc_fence_after();
       // some row of the tile sees only part of these keys (the tile's last row has the latest window)
-      const bool masked = n0 + TC_BN - 1 > pos0 + q0 || (p.window > 0 && n0 < pos0 + q0 + TC_BM - p.window);
+      const bool masked = n0 + TC_BN - 1 > pos0 + q0 || n0 < last_lo;
       const int limit = pos_r - n0;                     // this row sees columns first .. limit of the tile
-      const int first = p.window > 0 ? pos_r - p.window + 1 - n0 : -1;
+      const int first = first_key - n0;
       // pass 1: row maximum of the raw scores (64 columns per round: both loads in flight before the wait)
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -276,10 +297,77 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_before();
       mbar_arrive(bar_pfull);
     }
-    if (ok && mbar_wait(bar_odone, (n_tiles - 1) & 1, abort_flag, TC_BUDGET_NS)) {
+    const bool done = ok && mbar_wait(bar_odone, (n_tiles - 1) & 1, abort_flag, TC_BUDGET_NS);
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (p.r.sink) {
+      const float top = fmaxf(m, 0.f), e = exp2f(m - top);
+      inv = e / (l * e + exp2f(-top));
+    }
+    const bool store = q0 + qi < qlen;
+    if (MAPS == 2) {
+      // every copy and product of this CTA is complete: the K and V buffers take the second map's outputs
+      float* x_row = reinterpret_cast<float*>(base_ptr + TC_TILE_BYTES) + (size_t)qi * TC_X_LD;
+      if (done && r >= QR) {
+        tc_fence_after();
+        const float f = inv * p.r.lam[0];
+#pragma unroll
+        for (int c = 0; c < TC_D / 16; ++c) {
+          uint32_t ov[16];
+          tmem_ld16(tm_o + lane_addr + c * 16, ov);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; i += 4)
+            *reinterpret_cast<float4*>(x_row + c * 16 + i) = make_float4(__uint_as_float(ov[i]) * f, __uint_as_float(ov[i + 1]) * f,
+                                                                         __uint_as_float(ov[i + 2]) * f, __uint_as_float(ov[i + 3]) * f);
+        }
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");      // the four softmax warps, whatever their waits returned
+      if (done && r < QR) {
+        tc_fence_after();
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < TC_D / 16; ++c) {
+          uint32_t ov[16];
+          tmem_ld16(tm_o + lane_addr + c * 16, ov);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; i += 4) {
+            float4 x = *reinterpret_cast<const float4*>(x_row + c * 16 + i);
+            x.x = __uint_as_float(ov[i]) * inv - x.x; x.y = __uint_as_float(ov[i + 1]) * inv - x.y;
+            x.z = __uint_as_float(ov[i + 2]) * inv - x.z; x.w = __uint_as_float(ov[i + 3]) * inv - x.w;
+            ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            *reinterpret_cast<float4*>(x_row + c * 16 + i) = x;
+          }
+        }
+        const float f = p.r.out_scale / sqrtf(ss / (float)TC_D + p.r.eps);
+        const size_t row = (size_t)(qrow0 + q0 + qi), col = (size_t)head * TC_D;
+        if (store) {
+          const __nv_bfloat16* g_row = p.r.gate ? (const __nv_bfloat16*)p.r.gate + row * p.r.gate_ld + col : nullptr;
+#pragma unroll
+          for (int c = 0; c < TC_D / 8; ++c) {
+            float v[8];
+            *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(x_row + c * 8);
+            *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(x_row + c * 8 + 4);
+            uint4 g4 = make_uint4(0, 0, 0, 0), o4;
+            if (g_row) g4 = *reinterpret_cast<const uint4*>(g_row + c * 8);
+            const __nv_bfloat162* gb = reinterpret_cast<const __nv_bfloat162*>(&g4);
+            __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              float2 a = make_float2(v[2 * i] * f, v[2 * i + 1] * f);
+              if (g_row) {
+                const float2 z = __bfloat1622float2(gb[i]);
+                a.x /= 1.f + __expf(-z.x); a.y /= 1.f + __expf(-z.y);
+              }
+              ob[i] = __floats2bfloat162_rn(a.x, a.y);
+            }
+            *reinterpret_cast<uint4*>(p.out + row * p.out_ld + col + c * 8) = o4;
+          }
+        }
+      }
+    } else if (done) {
       tc_fence_after();
-      const float inv = l > 0.f ? p.out_scale / l : 0.f;
-      const bool store = q0 + r < qlen;
+      inv *= p.r.out_scale;
       __nv_bfloat16* orow = p.out + (size_t)(qrow0 + q0 + r) * p.out_ld + (size_t)head * TC_D;
 #pragma unroll
       for (int c = 0; c < TC_D / 16; ++c) {
@@ -297,7 +385,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           *reinterpret_cast<uint4*>(orow + c * 16 + 8) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
         }
       }
-    } else if (*abort_flag == 0) {
+    }
+    if (!done && *abort_flag == 0) {
       *abort_flag = 1;
       report_status(p.status, ST_TIMEOUT_TMEM_FULL, 12);
     }
@@ -314,44 +403,47 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 namespace skein {
 
-template <int TC_D>
+template <int TC_D, int MAPS>
 static int attn_prefill_tc_go(const void* q, long long q_stride, long long q_rows, const void* kv, const AttnPrefillTcParams& p, int S, int max_q_len,
                               void* stream) {
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<TC_D>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(TC_D));
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<TC_D, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(TC_D));
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
   CUtensorMap tmQ, tmKV;
-  int rc = cached_tmap_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)q_stride, 2, TC_BM);
+  int rc = cached_tmap_2d(&tmQ, q, (uint64_t)q_rows, (uint64_t)q_stride, 2, TC_BM / MAPS);
   if (rc != 0) return rc;
   rc = cached_tmap_2d(&tmKV, kv, (uint64_t)p.num_pages * 2 * p.Hkv * p.page_size, TC_D, 2, TC_PS);
   if (rc != 0) return rc;
-  dim3 grid((max_q_len + TC_BM - 1) / TC_BM, p.Hq, S);
-  attn_prefill_tc_kernel<TC_D><<<grid, TC_THREADS, tc_smem(TC_D), (cudaStream_t)stream>>>(tmQ, tmKV, p);
+  dim3 grid((max_q_len + TC_BM / MAPS - 1) / (TC_BM / MAPS), p.Hq, S);
+  attn_prefill_tc_kernel<TC_D, MAPS><<<grid, TC_THREADS, tc_smem(TC_D), (cudaStream_t)stream>>>(tmQ, tmKV, p);
   return (int)cudaGetLastError();
 }
 
 }  // namespace skein
 
 // Returns 0, a cudaError_t, or a negative code for shapes this kernel does not take (the caller then uses another kernel): head
-// size 128 or 64, pages of whole 16-token groups, 16-byte aligned rows. window 0: none. Rows of out are out_ld apart.
+// size 128 or 64 (D: the width of a key head; 128 with two maps), pages of whole 16-token groups, 16-byte aligned rows. Rows of out are
+// out_ld apart.
 extern "C" int skein_attn_prefill_window(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,
                                          const int* q_start, const int* q_len, const int* kv_len, void* out, long long out_ld, int* status, int S,
-                                         int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages, int window,
-                                         float scale, float out_scale, void* stream) {
+                                         int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages,
+                                         const SkeinAttnRule* rule, void* stream) {
   using namespace skein;
   if (S == 0 || max_q_len == 0) return 0;
   if ((D != 128 && D != 64) || page_size % TC_PS != 0 || Hq % Hkv != 0 || q_stride % 8 != 0 || (uintptr_t)q % 16 != 0) return -1;
-  if (out_ld % 8 != 0 || (uintptr_t)out % 16 != 0 || scale <= 0.f) return -1;
+  if (out_ld % 8 != 0 || (uintptr_t)out % 16 != 0 || rule->scale <= 0.f) return -1;
+  if (rule->maps == 2 ? D != 128 || !rule->lam || rule->gate_ld % 8 != 0 || (uintptr_t)rule->gate % 16 != 0 : rule->maps != 1 || rule->gate) return -1;
   AttnPrefillTcParams p;
   p.block_table = block_table; p.q_start = q_start; p.q_len = q_len; p.kv_len = kv_len;
-  p.out = (__nv_bfloat16*)out; p.status = status; p.out_ld = out_ld; p.out_scale = out_scale; p.window = window;
+  p.out = (__nv_bfloat16*)out; p.status = status; p.out_ld = out_ld; p.r = *rule;
   p.Hq = Hq; p.Hkv = Hkv; p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size;
-  p.scale_log2e = scale * 1.4426950408889634f;
-  return D == 64 ? attn_prefill_tc_go<64>(q, q_stride, q_rows, kv, p, S, max_q_len, stream)
-                 : attn_prefill_tc_go<128>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
+  p.scale_log2e = rule->scale * 1.4426950408889634f;
+  if (rule->maps == 2) return attn_prefill_tc_go<128, 2>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
+  return D == 64 ? attn_prefill_tc_go<64, 1>(q, q_stride, q_rows, kv, p, S, max_q_len, stream)
+                 : attn_prefill_tc_go<128, 1>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
 }
 
 extern "C" int skein_attn_prefill_tc(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,
@@ -359,6 +451,8 @@ extern "C" int skein_attn_prefill_tc(const void* q, long long q_stride, long lon
                                      int max_q_len, int Hq, int Hkv, int D, int page_size, int max_blocks, int num_pages,
                                      float scale, void* stream) {
   if (D != 128 || page_size != 16) return -1;
+  SkeinAttnRule rule{};
+  rule.maps = 1; rule.scale = scale; rule.out_scale = 1.f;
   return skein_attn_prefill_window(q, q_stride, q_rows, kv, block_table, q_start, q_len, kv_len, out, (long long)Hq * D, status, S, max_q_len, Hq,
-                                   Hkv, D, page_size, max_blocks, num_pages, 0, scale, 1.f, stream);
+                                   Hkv, D, page_size, max_blocks, num_pages, &rule, stream);
 }

@@ -207,10 +207,8 @@ __global__ void __launch_bounds__(512) post_norm_kernel(const PostNormParams p, 
 
 // The same for a bf16 model's decode step, followed in the same launch by the router and the scatter of the row into
 // expert-sorted order (route.cuh). One CTA per row, all resident at once; a thread owns 8 consecutive elements per pass.
-struct GroupRule { int n_groups, keep; };
-
 template <int MAX_PASSES>
-__global__ void __launch_bounds__(512) post_norm_route_kernel(const PostNormParams p, const RouteParams r, const GroupRule rule) {
+__global__ void __launch_bounds__(512) post_norm_route_kernel(const PostNormParams p, const RouteParams r, const SkeinRouteRule rule) {
   __shared__ float sh[32];
   __shared__ RouteShared rs;
   __shared__ int sel_id[NR_MAX_K];
@@ -251,7 +249,7 @@ __global__ void __launch_bounds__(512) post_norm_route_kernel(const PostNormPara
   for (int e = tid; e < r.E; e += blockDim.x) rs.logit[e] = route_sum_logit(rs, e);
   __syncthreads();
   if (tid < 32) {
-    select_grouped_warp<NR_MAX_E>(rs.logit, r.E, r.topk, rule.n_groups, rule.keep, sel_id, sel_w);
+    select_grouped_warp<NR_MAX_E>(rs.logit, r.E, r.topk, rule, sel_id, sel_w);
     if (tid == 0) {
       for (int j = 0; j < r.topk; ++j) {
         r.expert_ids[t * r.topk + j] = sel_id[j];
@@ -417,7 +415,7 @@ extern "C" int skein_post_norm_route(const float* x, const void* y, const float*
   r.barrier_budget_ns = (unsigned long long)grid_barrier_budget_ms() * 1000000ull;
   int threads = row_threads(C, 8, 512);
   const int passes = (C + threads * 8 - 1) / (threads * 8);
-  const GroupRule rule{n_groups, keep};
+  const SkeinRouteRule rule{n_groups, keep, ROUTE_SOFTMAX, 1, 0, 1.f};
   cudaStream_t s = (cudaStream_t)stream;
   if (passes <= 1) return (int)launch_pdl(post_norm_route_kernel<1>, dim3(B), dim3(threads), 0, s, p, r, rule);
   if (passes <= 2) return (int)launch_pdl(post_norm_route_kernel<2>, dim3(B), dim3(threads), 0, s, p, r, rule);

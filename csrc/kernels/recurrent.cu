@@ -20,6 +20,7 @@
 //
 // Activations are bf16, or fp32 when a model runs in 32-bit; convolved q, k, v are rounded to the activation type, everything
 // after that is 32-bit. Compiled without fast-math.
+#include "act.cuh"
 #include "ptx.cuh"
 #include "launch.cuh"
 #include "recurrent.cuh"
@@ -30,17 +31,6 @@ namespace skein {
 
 constexpr int RS_THREADS = 256, RS_WARPS = 8;
 constexpr int REC_MAX_D = 512;
-
-// the activation behind a projection or convolution; its result is rounded to bf16 in a bf16 model, so there it is computed fast
-template <typename T> __device__ __forceinline__ float silu_act(float z);
-template <> __device__ __forceinline__ float silu_act<float>(float z) { return z / (1.f + expf(-z)); }
-template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float z) {
-  float e, r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z * -1.44269504f));
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
-  return z * r;
-}
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // log decay and write coefficient of head h from the row's gate columns
 template <typename T>

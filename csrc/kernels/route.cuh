@@ -4,8 +4,24 @@
 #include "ptx.cuh"
 #include <cuda_bf16.h>
 #include <math.h>
+#include <stdint.h>
+
+// Rule of a group-limited choice of experts (mirrored in skein_b200/ops/_lib.py).
+extern "C" typedef struct SkeinRouteRule {
+  int32_t n_groups, keep;    // equal groups of neighbours, of which the best `keep` are eligible
+  int32_t score;             // ROUTE_*
+  int32_t group_best;        // a group's score is the sum of its 1 or 2 best
+  int32_t renorm;            // the chosen scores are divided by their sum
+  float scale;               // ... and multiplied by this
+} SkeinRouteRule;
 
 namespace skein {
+
+enum : int { ROUTE_SOFTMAX = 0, ROUTE_SIGMOID = 1 };
+inline bool route_rule_ok(const SkeinRouteRule& r, int E, int topk) {
+  return r.n_groups >= 1 && r.n_groups <= 64 && E % r.n_groups == 0 && r.keep >= 1 && r.keep <= r.n_groups && topk >= 1 && topk <= r.keep * (E / r.n_groups) &&
+         r.group_best >= 1 && r.group_best <= 2;
+}
 
 constexpr int NR_MAX_E = 64;
 constexpr int NR_MAX_K = 8;
@@ -154,10 +170,10 @@ __device__ __forceinline__ void route_scatter(const RouteParams& r, const uint4 
   }
 }
 
-// Group-limited selection by one warp: softmax over all E logits z (shared memory), experts in n_groups equal groups of
-// neighbours of which the `keep` with the largest logit are eligible, the topk largest eligible logits in descending order
-// (ties to the lower index), their softmax values as weights (not renormalised). Every lane returns with the same results
-// written to ids / w (shared or global memory, by lane 0).
+// Group-limited selection by one warp over the logits z of E experts (shared memory): a score per expert, experts in n_groups equal groups
+// of neighbours of which the `keep` best are eligible (a group counts its best or its two best scores), the topk best eligible experts in
+// descending order (ties to the lower index), their scores as weights, divided by their sum with renorm, times scale. Lane 0 writes ids / w
+// (shared or global memory).
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   for (int o = 16; o > 0; o >>= 1) {
     const float v2 = __shfl_xor_sync(0xffffffffu, v, o);
@@ -165,37 +181,79 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
     if (v2 > v || (v2 == v && i2 < i)) { v = v2; i = i2; }
   }
 }
+__device__ __forceinline__ float warp_sum(float v) {
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
 template <int MAX_E>
-__device__ __forceinline__ void select_grouped_warp(const float* z, int E, int topk, int n_groups, int keep, int* ids, float* w) {
+__device__ __forceinline__ void select_grouped_warp(const float* z, int E, int topk, const SkeinRouteRule& rule, int* ids, float* w) {
   constexpr int PER = (MAX_E + 31) / 32;
   const int lane = threadIdx.x & 31;
+  // v: what is compared. Softmax scores rise with the logits, so there the logits themselves are compared.
   float v[PER];
-  float mx = -INFINITY;
+  float mx = -INFINITY, den = 0.f;
 #pragma unroll
   for (int q = 0; q < PER; ++q) {
     const int e = q * 32 + lane;
     // a logit that is not a number counts as the smallest: the indices below stay valid whatever the input
     v[q] = (e < E && z[e] == z[e]) ? fmaxf(z[e], -3.0e38f) : (e < E ? -3.0e38f : -INFINITY);
+    if (rule.score == ROUTE_SIGMOID && e < E) v[q] = 1.f / (1.f + expf(-v[q]));
     mx = fmaxf(mx, v[q]);
   }
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-  float den = 0.f;
+  if (rule.score == ROUTE_SOFTMAX) {
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
 #pragma unroll
-  for (int q = 0; q < PER; ++q) if (q * 32 + lane < E) den += expf(v[q] - mx);
-  for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
-  if (keep < n_groups) {
-    const int per = E / n_groups;
+    for (int q = 0; q < PER; ++q) if (q * 32 + lane < E) den += expf(v[q] - mx);
+    den = warp_sum(den);
+  }
+  if (rule.keep < rule.n_groups) {
+    const int per = E / rule.n_groups;
     unsigned long long kept = 0;     // at most 64 groups
-    for (int k = 0; k < keep; ++k) {
-      float bv = -INFINITY;
-      int bi = MAX_E;
+    if (rule.group_best > 1) {
+      // lane g owns groups g and g + 32; the members' scores come from the lanes that hold them
+      float worth[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-      for (int q = 0; q < PER; ++q) {
-        const int e = q * 32 + lane;
-        if (e < E && !((kept >> (e / per)) & 1ull) && (v[q] > bv || bi == MAX_E)) { bv = v[q]; bi = e; }
+      for (int h = 0; h < 2; ++h) {
+        if (h * 32 >= rule.n_groups) break;
+        const int g = h * 32 + lane;
+        float b1 = -INFINITY, b2 = -INFINITY;
+        for (int i = 0; i < per; ++i) {
+          const int e = g < rule.n_groups ? g * per + i : 0;
+          float s = 0.f;
+#pragma unroll
+          for (int q = 0; q < PER; ++q) {
+            const float c = __shfl_sync(0xffffffffu, v[q], e & 31);
+            if ((e >> 5) == q) s = c;
+          }
+          if (rule.score == ROUTE_SOFTMAX) s = expf(s - mx);
+          if (s > b1) { b2 = b1; b1 = s; }
+          else if (s > b2) b2 = s;
+        }
+        if (g < rule.n_groups) worth[h] = per > 1 ? b1 + b2 : b1;
       }
-      warp_argmax(bv, bi);
-      if (bi < MAX_E) kept |= 1ull << (bi / per);
+      for (int k = 0; k < rule.keep; ++k) {
+        float bv = -INFINITY;
+        int bi = 64;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int g = h * 32 + lane;
+          if (g < rule.n_groups && !((kept >> g) & 1ull) && (worth[h] > bv || bi == 64)) { bv = worth[h]; bi = g; }
+        }
+        warp_argmax(bv, bi);
+        if (bi < 64) kept |= 1ull << bi;
+      }
+    } else {
+      for (int k = 0; k < rule.keep; ++k) {
+        float bv = -INFINITY;
+        int bi = MAX_E;
+#pragma unroll
+        for (int q = 0; q < PER; ++q) {
+          const int e = q * 32 + lane;
+          if (e < E && !((kept >> (e / per)) & 1ull) && (v[q] > bv || bi == MAX_E)) { bv = v[q]; bi = e; }
+        }
+        warp_argmax(bv, bi);
+        if (bi < MAX_E) kept |= 1ull << (bi / per);
+      }
     }
 #pragma unroll
     for (int q = 0; q < PER; ++q) {
@@ -203,6 +261,7 @@ __device__ __forceinline__ void select_grouped_warp(const float* z, int E, int t
       if (e < E && !((kept >> (e / per)) & 1ull)) v[q] = -INFINITY;
     }
   }
+  float sum = 0.f;
   for (int j = 0; j < topk; ++j) {
     float bv = -INFINITY;
     int bi = MAX_E;
@@ -212,9 +271,15 @@ __device__ __forceinline__ void select_grouped_warp(const float* z, int E, int t
       if (v[q] > -INFINITY && (v[q] > bv || bi == MAX_E)) { bv = v[q]; bi = e; }
     }
     warp_argmax(bv, bi);
-    if (lane == 0) { ids[j] = bi < E ? bi : 0; w[j] = bi < E ? expf(bv - mx) / den : 0.f; }
+    const float s = bi >= E ? 0.f : rule.score == ROUTE_SIGMOID ? bv : expf(bv - mx) / den;
+    sum += s;
+    if (lane == 0) { ids[j] = bi < E ? bi : 0; w[j] = s * rule.scale; }
 #pragma unroll
     for (int q = 0; q < PER; ++q) if (q * 32 + lane == bi) v[q] = -INFINITY;
+  }
+  if (rule.renorm) {
+    __syncwarp();
+    if (lane == 0) for (int j = 0; j < topk; ++j) w[j] = w[j] / (sum + 1e-20f);
   }
 }
 

@@ -186,7 +186,7 @@ __global__ void __launch_bounds__(1024) router_plan_kernel(const int* __restrict
 // ---- group-limited selection over given logits, and a layout kernel pair for prefill-sized batches -----------------
 // One warp per token; logits fp32 [T, E].
 constexpr int RG_MAX_E = 256;
-__global__ void __launch_bounds__(128) route_select_kernel(const float* __restrict__ logits, int T, int E, int topk, int n_groups, int keep,
+__global__ void __launch_bounds__(128) route_select_kernel(const float* __restrict__ logits, int T, int E, int topk, const SkeinRouteRule rule,
                                                            int* __restrict__ expert_ids, float* __restrict__ expert_w) {
   __shared__ float z[4][RG_MAX_E];
   pdl_trigger();
@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(128) route_select_kernel(const float* __restri
   if (t >= T) return;
   for (int e = lane; e < E; e += 32) z[warp][e] = logits[(size_t)t * E + e];
   __syncwarp();
-  select_grouped_warp<RG_MAX_E>(z[warp], E, topk, n_groups, keep, expert_ids + (size_t)t * topk, expert_w + (size_t)t * topk);
+  select_grouped_warp<RG_MAX_E>(z[warp], E, topk, rule, expert_ids + (size_t)t * topk, expert_w + (size_t)t * topk);
 }
 
 // Stable expert-sorted layout with one CTA per expert: the first kernel counts, the second derives its expert's offset from
@@ -250,15 +250,14 @@ __global__ void __launch_bounds__(256) plan_place_kernel(const int* __restrict__
 
 }  // namespace skein
 
-// Softmax over all E logits, group-limited top-k, weights not renormalised (route.cuh: select_grouped_warp), then the
-// expert-sorted layout.
-extern "C" int skein_route_grouped(const float* logits, int T, int E, int topk, int n_groups, int keep, int* expert_ids, float* expert_w,
+// Scores of E logits, group-limited top-k, weights (route.cuh: select_grouped_warp), then the expert-sorted layout.
+extern "C" int skein_route_grouped(const float* logits, int T, int E, int topk, const SkeinRouteRule* rule, int* expert_ids, float* expert_w,
                                    int* counts, int* offsets, int* row_of, int* src_token, void* stream) {
   using namespace skein;
   if (T == 0) return 0;
-  if (E > RG_MAX_E || n_groups < 1 || n_groups > 64 || E % n_groups != 0 || keep < 1 || keep > n_groups || topk < 1 || topk > keep * (E / n_groups)) return -1;
+  if (E > RG_MAX_E || !route_rule_ok(*rule, E, topk)) return -1;
   cudaStream_t s = (cudaStream_t)stream;
-  cudaError_t rc = launch_pdl(route_select_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, T, E, topk, n_groups, keep, expert_ids, expert_w);
+  cudaError_t rc = launch_pdl(route_select_kernel, dim3((T + 3) / 4), dim3(128), 0, s, logits, T, E, topk, *rule, expert_ids, expert_w);
   if (rc == cudaSuccess) rc = launch_pdl(plan_count_kernel, dim3(E), dim3(256), 0, s, (const int*)expert_ids, T * topk, counts);
   if (rc == cudaSuccess) rc = launch_pdl(plan_place_kernel, dim3(E), dim3(256), 0, s, (const int*)expert_ids, T * topk, E, topk, (const int*)counts, offsets, row_of, src_token);
   return (int)rc;

@@ -1,0 +1,386 @@
+// Selective scan (Mamba): a short causal convolution over time with silu, and a diagonal recurrence per channel c and state dimension n
+// with a 32-bit state per sequence:
+//
+//   S[n, c] <- exp(dt[c] A[n, c]) S[n, c] + dt[c] u[c] B[n],    y[c] = sum_n S[n, c] C[n] + D[c] u[c],    out = y silu(z)
+//
+// with u the convolved channels, dt = softplus(raw + bias) and B, C projections of u that all channels share. The products that make
+// B, C and raw from u run between the two kernels.
+//
+// A sequence owns one slot of the state pools: S [slots, N, I] fp32 and the convolution's last inputs [slots, taps, I] in the activation
+// type, position p in row p mod taps (taps - 1 rows would hold the state; with one more, a decode step writes no row it reads). Position 0
+// starts from zero whatever the slot holds.
+//
+//   short_conv   convolution and silu of every row of the step; a decode step also keeps its input
+//   scan_step    decode: one row per sequence. Four channels per thread, the state read and written once
+//   scan_rows    portions of sequences, one token after the other: a channel's states are spread over P lanes of a warp, tiles of tokens
+//                go through shared memory while the next tile is on its way; keeps the convolution's last inputs
+//
+// Activations are bf16, or fp32 when a model runs in 32-bit; decays, step sizes and the state are 32-bit. Compiled without fast-math.
+#include "act.cuh"
+#include "launch.cuh"
+#include "ptx.cuh"
+#include "vec.cuh"
+#include <math.h>
+
+// Mirrored in skein_b200/ops/_lib.py (same field order).
+extern "C" typedef struct SkeinScanParams {
+  const void* x;             // [T, x_ld] inputs of the convolution, activation type
+  void* xc;                  // [T, I] convolved: written by short_conv, read by the scan
+  const void* proj;          // [T, proj_ld] B from column b_col, C from column c_col
+  const float* dt;           // [T, I] step sizes before bias and softplus
+  const void* z;             // [T, x_ld]
+  void* out;                 // [T, out_ld]
+  float* state;              // [slots, N, I]
+  void* tail;                // [slots, taps, I] or null (taps == 1)
+  const float* conv_w;       // [taps, I]
+  const float* conv_b;       // [I]
+  const float* dt_bias;      // [I]
+  const float* neg_a;        // [N, I]
+  const float* skip;         // [I]
+  const int32_t* positions;  // [T], -1: padding row
+  const int32_t* slots;      // [S]
+  const int32_t* seq_of_token;   // [T], null in a decode step (row = sequence)
+  const int32_t* q_start;    // [S] first row of each sequence's portion
+  const int32_t* q_len;      // [S]
+  int32_t* status;
+  int64_t x_ld, proj_ld, out_ld;
+  int32_t I, N, taps, b_col, c_col, num_slots;
+} SkeinScanParams;
+
+namespace skein {
+
+using ScanParams = SkeinScanParams;
+
+// ---- convolution ----------------------------------------------------------------------------------------
+constexpr int SC_RUN = 8;      // consecutive rows of a thread
+
+// V channels per thread; TAPS 0: any number. DECODE: every row is the next token of its own sequence.
+template <typename T, int V, int TAPS, bool DECODE>
+__global__ void __launch_bounds__(128) short_conv_kernel(const ScanParams p, int rows) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V;
+  if (c >= p.I) return;
+  const int taps = TAPS > 0 ? TAPS : p.taps;
+  const int t0 = blockIdx.y * (DECODE ? 1 : SC_RUN), t1 = min(rows, t0 + (DECODE ? 1 : SC_RUN));
+  const T* x = (const T*)p.x;
+  constexpr int HN = TAPS > 1 ? TAPS - 1 : 1;
+  float bias[V], w[TAPS > 0 ? TAPS : 1][V], hist[HN][V];
+  load_v<float, V>(p.conv_b + c, bias);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load_v<float, V>(p.conv_w + (size_t)j * p.I + c, w[j]);
+  for (int t = t0; t < t1; ++t) {
+    const int pos = p.positions[t];
+    if (pos < 0) continue;
+    const int seq = DECODE ? t : p.seq_of_token[t], first = DECODE ? t : p.q_start[seq];
+    // the input j tokens before row t
+    auto prev = [&](int j, float* v) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[k] = 0.f;
+      if (pos < j) return;
+      if (t - j >= first) { load_v<T, V>(x + (size_t)(t - j) * p.x_ld + c, v); return; }
+      const int slot = p.slots[seq];
+      if (slot < 0 || slot >= p.num_slots) { report_status(p.status, ST_BAD_INDEX, slot); return; }
+      load_v<T, V>((const T*)p.tail + ((size_t)slot * taps + (pos - j) % taps) * p.I + c, v);
+    };
+    float cur[V], a[V];
+    load_v<T, V>(x + (size_t)t * p.x_ld + c, cur);
+#pragma unroll
+    for (int k = 0; k < V; ++k) a[k] = bias[k];
+    if (TAPS > 0) {
+      if (t == t0 || t == first)
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) prev(j, hist[j - 1]);
+#pragma unroll
+      for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) a[k] = fmaf(w[TAPS - 1 - j][k], hist[j - 1][k], a[k]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) a[k] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][k], cur[k], a[k]);
+    } else {
+      float v[V], wj[V];
+      for (int j = taps - 1; j >= 0; --j) {
+        if (j > 0) prev(j, v);
+        load_v<float, V>(p.conv_w + (size_t)(taps - 1 - j) * p.I + c, wj);
+#pragma unroll
+        for (int k = 0; k < V; ++k) a[k] = fmaf(wj[k], j > 0 ? v[k] : cur[k], a[k]);
+      }
+    }
+    if (DECODE && taps > 1) {
+      const int slot = p.slots[seq];
+      if (slot < 0 || slot >= p.num_slots) report_status(p.status, ST_BAD_INDEX, slot);
+      else store_v<T, V>((T*)p.tail + ((size_t)slot * taps + pos % taps) * p.I + c, cur);
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) a[k] = silu_act<T>(a[k]);
+    store_v<T, V>((T*)p.xc + (size_t)t * p.I + c, a);
+    if (TAPS > 1) {
+#pragma unroll
+      for (int j = HN - 1; j > 0; --j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) hist[j][k] = hist[j - 1][k];
+#pragma unroll
+      for (int k = 0; k < V; ++k) hist[0][k] = cur[k];
+    }
+  }
+}
+
+// ---- decode -----------------------------------------------------------------------------------------------
+constexpr int ST_THREADS = 128, ST_UNROLL = 8;
+
+// grid (I / (128 V), B)
+template <typename T, int V>
+__global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(const ScanParams p) {
+  extern __shared__ float bc_s[];      // B [N], C [N]
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.y, c = (blockIdx.x * ST_THREADS + threadIdx.x) * V, N = p.N;
+  const int pos = p.positions[b];
+  if (pos < 0) return;
+  const int slot = p.slots[b];
+  if (slot < 0 || slot >= p.num_slots) { if (threadIdx.x == 0) report_status(p.status, ST_BAD_INDEX, slot); return; }
+  const bool in = c < p.I;
+  float* S = p.state + (size_t)slot * N * p.I + c;
+  const float* A = p.neg_a + c;
+  float s[ST_UNROLL][V], an[ST_UNROLL][V];
+  auto fetch = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < ST_UNROLL; ++i) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) s[i][k] = an[i][k] = 0.f;
+      if (in && n0 + i < N) {
+        if (pos > 0) load_v<float, V>(S + (size_t)(n0 + i) * p.I, s[i]);
+        load_v<float, V>(A + (size_t)(n0 + i) * p.I, an[i]);
+      }
+    }
+  };
+  fetch(0);      // the state's latency covers the rest
+  const T* pr = (const T*)p.proj + (size_t)b * p.proj_ld;
+  for (int i = threadIdx.x; i < 2 * N; i += ST_THREADS) bc_s[i] = to_f<T>(pr[i < N ? p.b_col + i : p.c_col + i - N]);
+  float dt[V], u[V], dx[V], y[V], z[V], skip[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) dt[k] = u[k] = dx[k] = y[k] = z[k] = skip[k] = 0.f;
+  if (in) {
+    float bias[V];
+    load_v<float, V>(p.dt + (size_t)b * p.I + c, dt);
+    load_v<float, V>(p.dt_bias + c, bias);
+    load_v<T, V>((const T*)p.xc + (size_t)b * p.I + c, u);
+    load_v<T, V>((const T*)p.z + (size_t)b * p.x_ld + c, z);
+    load_v<float, V>(p.skip + c, skip);
+#pragma unroll
+    for (int k = 0; k < V; ++k) { dt[k] = softplus_f(dt[k] + bias[k]); dx[k] = dt[k] * u[k]; y[k] = skip[k] * u[k]; }
+  }
+  __syncthreads();
+  if (!in) return;
+  for (int n0 = 0; n0 < N; n0 += ST_UNROLL) {
+    if (n0 > 0) fetch(n0);
+#pragma unroll
+    for (int i = 0; i < ST_UNROLL; ++i) {
+      if (n0 + i >= N) break;
+      const float B = bc_s[n0 + i], C = bc_s[N + n0 + i];
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        s[i][k] = fmaf(expf(dt[k] * an[i][k]), s[i][k], dx[k] * B);
+        y[k] = fmaf(s[i][k], C, y[k]);
+      }
+      store_v<float, V>(S + (size_t)(n0 + i) * p.I, s[i]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k) y[k] *= silu_act<T>(z[k]);
+  store_v<T, V>((T*)p.out + (size_t)b * p.out_ld + c, y);
+}
+
+// ---- portions ------------------------------------------------------------------------------------------------
+constexpr int SR_THREADS = 128;
+
+// decay exp(dt a) with `a` as scan_coef left it
+template <typename T> __device__ __forceinline__ float scan_coef(float a);
+template <> __device__ __forceinline__ float scan_coef<float>(float a) { return a; }
+template <> __device__ __forceinline__ float scan_coef<__nv_bfloat16>(float a) { return a * 1.44269504f; }
+template <typename T> __device__ __forceinline__ float scan_decay(float dt, float a);
+template <> __device__ __forceinline__ float scan_decay<float>(float dt, float a) { return expf(dt * a); }
+template <> __device__ __forceinline__ float scan_decay<__nv_bfloat16>(float dt, float a) {
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(dt * a));
+  return e;
+}
+
+// grid (I / CH, S). Lane q of a channel's P lanes holds states q RPT .. q RPT + RPT - 1; TT tokens per tile.
+template <typename T, int P, int RPT, int TT>
+__global__ void __launch_bounds__(SR_THREADS) scan_rows_kernel(const ScanParams p) {
+  constexpr int CH = SR_THREADS / P, NP = P * RPT, EL = TT * CH / SR_THREADS, BL = (TT * NP + SR_THREADS - 1) / SR_THREADS;
+  __shared__ float dt_s[TT][CH], dx_s[TT][CH], y_s[TT][CH];
+  __shared__ __align__(16) float B_s[TT][NP], C_s[TT][NP];
+  pdl_trigger();
+  pdl_wait();
+  const int seq = blockIdx.y, tid = threadIdx.x, c0 = blockIdx.x * CH;
+  const int n_rows = p.q_len[seq];
+  if (n_rows < 1) return;
+  const int t0 = p.q_start[seq], pos0 = p.positions[t0];
+  if (pos0 < 0) return;
+  const int slot = p.slots[seq];
+  if (slot < 0 || slot >= p.num_slots) { if (tid == 0) report_status(p.status, ST_BAD_INDEX, slot); return; }
+  const int q = tid % P, ch = tid / P, c = c0 + ch;
+  const bool in = c < p.I;
+  float* S = p.state + (size_t)slot * p.N * p.I + c;
+  float s[RPT], a[RPT];
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int n = q * RPT + i;
+    const bool have = in && n < p.N;
+    s[i] = have && pos0 > 0 ? S[(size_t)n * p.I] : 0.f;
+    a[i] = have ? scan_coef<T>(p.neg_a[(size_t)n * p.I + c]) : 0.f;
+  }
+  // elements e of a tile that this thread moves: token e / CH, channel e % CH with e = tid + 128 k
+  const int lc = c0 + tid % CH;
+  const bool lin = lc < p.I;
+  const float bias = lin ? p.dt_bias[lc] : 0.f, skip = lin ? p.skip[lc] : 0.f;
+  float u[EL], nu[EL], nd[EL], z[EL], nb[BL], nc[BL];
+  auto fetch = [&](int r0) {
+#pragma unroll
+    for (int k = 0; k < EL; ++k) {
+      const int r = r0 + (tid + k * SR_THREADS) / CH;
+      nu[k] = nd[k] = 0.f;
+      if (lin && r < n_rows) {
+        nu[k] = to_f<T>(((const T*)p.xc)[(size_t)(t0 + r) * p.I + lc]);
+        nd[k] = p.dt[(size_t)(t0 + r) * p.I + lc];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < BL; ++k) {
+      const int e = tid + k * SR_THREADS, r = r0 + e / NP, n = e % NP;
+      nb[k] = nc[k] = 0.f;
+      if (e < TT * NP && r < n_rows && n < p.N) {
+        const T* pr = (const T*)p.proj + (size_t)(t0 + r) * p.proj_ld;
+        nb[k] = to_f<T>(pr[p.b_col + n]);
+        nc[k] = to_f<T>(pr[p.c_col + n]);
+      }
+    }
+  };
+  fetch(0);
+  for (int r0 = 0; r0 < n_rows; r0 += TT) {
+    const int cnt = min(TT, n_rows - r0);
+#pragma unroll
+    for (int k = 0; k < EL; ++k) {
+      const int e = tid + k * SR_THREADS;
+      u[k] = nu[k];
+      const float d = softplus_f(nd[k] + bias);
+      dt_s[e / CH][e % CH] = d;
+      dx_s[e / CH][e % CH] = d * u[k];
+      const int r = r0 + e / CH;
+      z[k] = lin && r < n_rows ? to_f<T>(((const T*)p.z)[(size_t)(t0 + r) * p.x_ld + lc]) : 0.f;
+    }
+#pragma unroll
+    for (int k = 0; k < BL; ++k) {
+      const int e = tid + k * SR_THREADS;
+      if (e < TT * NP) { B_s[e / NP][e % NP] = nb[k]; C_s[e / NP][e % NP] = nc[k]; }
+    }
+    __syncthreads();
+    if (r0 + TT < n_rows) fetch(r0 + TT);
+#pragma unroll 4
+    for (int j = 0; j < cnt; ++j) {
+      const float d = dt_s[j][ch], x = dx_s[j][ch];
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < RPT; ++i) {
+        s[i] = fmaf(scan_decay<T>(d, a[i]), s[i], x * B_s[j][q * RPT + i]);
+        y = fmaf(s[i], C_s[j][q * RPT + i], y);
+      }
+#pragma unroll
+      for (int o = 1; o < P; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+      if (q == 0) y_s[j][ch] = y;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < EL; ++k) {
+      const int e = tid + k * SR_THREADS, r = r0 + e / CH;
+      if (lin && r < n_rows)
+        ((T*)p.out)[(size_t)(t0 + r) * p.out_ld + lc] = from_f<T>((y_s[e / CH][e % CH] + skip * u[k]) * silu_act<T>(z[k]));
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int n = q * RPT + i;
+    if (in && n < p.N) S[(size_t)n * p.I] = s[i];
+  }
+  if (p.taps > 1) {      // every reader of the old inputs (short_conv) is done
+    const int keep = min(p.taps - 1, n_rows);
+    for (int e = tid; e < keep * CH; e += SR_THREADS) {
+      const int r = n_rows - keep + e / CH, cc = c0 + e % CH;
+      if (cc < p.I) ((T*)p.tail)[((size_t)slot * p.taps + (pos0 + r) % p.taps) * p.I + cc] = ((const T*)p.x)[(size_t)(t0 + r) * p.x_ld + cc];
+    }
+  }
+}
+
+template <typename T, int V, bool DECODE>
+static int short_conv_go(const ScanParams& p, int rows, cudaStream_t s) {
+  const dim3 grid((p.I + 128 * V - 1) / (128 * V), DECODE ? rows : (rows + SC_RUN - 1) / SC_RUN);
+  auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(128), 0, s, p, rows); };
+  switch (p.taps) {
+    case 1: return go(short_conv_kernel<T, V, 1, DECODE>);
+    case 2: return go(short_conv_kernel<T, V, 2, DECODE>);
+    case 3: return go(short_conv_kernel<T, V, 3, DECODE>);
+    case 4: return go(short_conv_kernel<T, V, 4, DECODE>);
+    default: return go(short_conv_kernel<T, V, 0, DECODE>);
+  }
+}
+
+template <typename T>
+static int scan_rows_any(const ScanParams& p, int S, cudaStream_t s) {
+  auto go = [&](auto fn, int ch) -> int { return (int)launch_pdl(fn, dim3((p.I + ch - 1) / ch, S), dim3(SR_THREADS), 0, s, p); };
+  if (p.N <= 4) return go(scan_rows_kernel<T, 1, 4, 16>, 128);
+  if (p.N <= 8) return go(scan_rows_kernel<T, 2, 4, 32>, 64);
+  if (p.N <= 16) return go(scan_rows_kernel<T, 4, 4, 32>, 32);
+  if (p.N <= 32) return go(scan_rows_kernel<T, 8, 4, 32>, 16);
+  if (p.N <= 64) return go(scan_rows_kernel<T, 16, 4, 32>, 8);
+  if (p.N <= 128) return go(scan_rows_kernel<T, 16, 8, 16>, 8);
+  if (p.N <= 256) return go(scan_rows_kernel<T, 16, 16, 16>, 8);
+  return -1;
+}
+
+static int scan_check(const ScanParams* p) {
+  if (p->I < 1 || p->N < 1 || p->taps < 1 || (p->taps > 1 && p->tail == nullptr)) return -1;
+  return 0;
+}
+// 4-element accesses to rows of x, z, xc, out and the state
+static bool scan_vec(const ScanParams* p) {
+  auto ok = [](const void* q) { return (uintptr_t)q % 16 == 0; };
+  return p->I % 4 == 0 && p->x_ld % 4 == 0 && p->out_ld % 4 == 0 && ok(p->x) && ok(p->z) && ok(p->out) && ok(p->xc) && ok(p->dt) && ok(p->tail) && ok(p->state);
+}
+
+}  // namespace skein
+
+extern "C" int skein_short_conv(const SkeinScanParams* p, int rows, int decode, int fp32, void* stream) {
+  using namespace skein;
+  if (rows == 0) return 0;
+  if (int e = scan_check(p)) return e;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v = scan_vec(p);
+  if (fp32) {
+    if (decode) return v ? short_conv_go<float, 4, true>(*p, rows, s) : short_conv_go<float, 1, true>(*p, rows, s);
+    return v ? short_conv_go<float, 4, false>(*p, rows, s) : short_conv_go<float, 1, false>(*p, rows, s);
+  }
+  if (decode) return v ? short_conv_go<__nv_bfloat16, 4, true>(*p, rows, s) : short_conv_go<__nv_bfloat16, 1, true>(*p, rows, s);
+  return v ? short_conv_go<__nv_bfloat16, 4, false>(*p, rows, s) : short_conv_go<__nv_bfloat16, 1, false>(*p, rows, s);
+}
+
+extern "C" int skein_scan_step(const SkeinScanParams* p, int B, int fp32, void* stream) {
+  using namespace skein;
+  if (B == 0) return 0;
+  if (int e = scan_check(p)) return e;
+  if (p->N > 4096) return -1;
+  const int v = scan_vec(p) ? 4 : 1;
+  const dim3 grid((p->I + ST_THREADS * v - 1) / (ST_THREADS * v), B);
+  auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(ST_THREADS), (size_t)p->N * 8, (cudaStream_t)stream, *p); };
+  if (fp32) return v == 4 ? go(scan_step_kernel<float, 4>) : go(scan_step_kernel<float, 1>);
+  return v == 4 ? go(scan_step_kernel<__nv_bfloat16, 4>) : go(scan_step_kernel<__nv_bfloat16, 1>);
+}
+
+// State dimensions up to 256.
+extern "C" int skein_scan_rows(const SkeinScanParams* p, int S, int fp32, void* stream) {
+  using namespace skein;
+  if (S == 0) return 0;
+  if (int e = scan_check(p)) return e;
+  return fp32 ? scan_rows_any<float>(*p, S, (cudaStream_t)stream) : scan_rows_any<__nv_bfloat16>(*p, S, (cudaStream_t)stream);
+}

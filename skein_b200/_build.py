@@ -34,9 +34,11 @@ ARCH_SOURCES = {
     "Zarorax": ("attn_latent_decode", "attn_latent_prefill", "gemm_simt", "gemm_ws", "latent", "postnorm", "rope_kv", "router", "sample"),
     "Sikalorn": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_ws", "parallel_layer", "postnorm", "recurrent",
                  "recurrent_tc", "rope_kv", "sample"),
+    "Barorax": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_ws", "postnorm", "prenorm", "rope_kv", "router",
+                "sample", "selective"),
 }
 # Sources compiled without fast-math: their exponentials, logarithms and tanh keep the accuracy of 32-bit.
-EXACT_SOURCES = ("attn_window", "parallel_layer", "recurrent", "recurrent_tc")
+EXACT_SOURCES = ("attn_window", "parallel_layer", "prenorm", "recurrent", "recurrent_tc", "selective")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -12,7 +12,7 @@ import json
 from dataclasses import asdict, dataclass
 from pathlib import Path
 
-from .layered import LAYERED_ARCHS, PARALLEL_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers, unroll_loop
+from .layered import LAYERED_ARCHS, PARALLEL_ARCHS, PRENORM_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers, unroll_loop
 from .parallel_layers import attention_of, parse_loop, recurrence_of
 
 MOE_ARCHS = {"MixtralForCausalLM"}
@@ -63,10 +63,15 @@ class ModelConfig:
         return self.architecture in PARALLEL_ARCHS
 
     @property
+    def is_prenorm(self) -> bool:
+        """Layers are x + mixer(norm1(x)), x + ff(norm2(x)) with an fp32 stream (models/prenorm_layers.py)."""
+        return self.architecture in PRENORM_ARCHS
+
+    @property
     def has_state(self) -> bool:
         """Sequences carry a recurrent state beside their cache pages: each needs a state slot, and a prefix of cached pages
         alone does not bring a sequence back."""
-        return self.is_parallel and any(recurrence_of(l.mixer) is not None for l in self.layers)
+        return any(recurrence_of(l.mixer) is not None for l in self.layers)
 
     def state_bytes_per_slot(self, elem: int = 2) -> int:
         if not self.has_state:
@@ -97,7 +102,7 @@ class ModelConfig:
 
     def validate(self) -> None:
         if self.is_layered:
-            if self.conv_taps < 1 and not self.is_parallel:
+            if self.conv_taps < 1 and not (self.is_parallel or self.is_prenorm):
                 raise ImportError_("canon.taps must be at least 1")
             return
         if self.num_heads % self.num_kv_heads != 0:
@@ -191,9 +196,10 @@ class ModelConfig:
         try:
             arch = d["architecture"]
             layers = parse_layers(arch, d["layers"], d.get("loop"))
-            only = {} if arch in PARALLEL_ARCHS else {"taps": int(d["canon"]["taps"]), "alpha": float(d["postln_alpha"])}
-            if arch in PARALLEL_ARCHS:
-                only["loop"] = parse_loop(d.get("loop"), len(d["layers"]))
+            if arch in PARALLEL_ARCHS | PRENORM_ARCHS:
+                only = {"loop": parse_loop(d.get("loop"), len(d["layers"]))}
+            else:
+                only = {"taps": int(d["canon"]["taps"]), "alpha": float(d["postln_alpha"])}
             cfg = ModelConfig.layered(arch, layers, width=int(d["width"]), vocab=int(d["vocab"]), eps=float(d["norm"]["eps"]),
                                       name=name or arch.lower(), **only)
         except KeyError as e:
@@ -225,7 +231,7 @@ class ModelConfig:
 
     def to_hf_dict(self) -> dict:
         """The config.json fields that describe this model (what the planner and the lowering read)."""
-        if self.is_parallel:
+        if self.is_parallel or self.is_prenorm:
             d = {"architecture": self.architecture, "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps},
                  "layers": layers_to_list(self.layers), "max_position_embeddings": self.max_position_embeddings}
             if self.loop is not None:
@@ -301,6 +307,22 @@ def tiny_sikalorn(width=96, vocab=384, eps=1e-5) -> ModelConfig:
     specs = [(delta, DenseFFSpec(144)), (pair, DenseFFSpec(120)), (light, None), (pair, DenseFFSpec(64))]
     loop = (1, 3, 3)
     return ModelConfig.layered("Sikalorn", unroll_loop(specs, loop), width=width, vocab=vocab, eps=eps, max_pos=4096, name="tiny-sikalorn", loop=loop)
+
+
+def tiny_barorax(width=96, vocab=384, eps=1e-5) -> ModelConfig:
+    """A small model of the Barorax design for tests: every mixer, a layer without feed-forward, two passes over three layers."""
+    from .parallel_layers import SelectiveSpec, WindowAttnSpec
+    diff = WindowAttnSpec(heads=4, kv_heads=2, dim=20, vdim=32, scale=0.3, rot_dims=12, rope_base=5e4, kind="attention", row_norm=False,
+                          interleaved=True, diff=0.6, gated=True)
+    chunk = WindowAttnSpec(heads=6, kv_heads=2, dim=24, vdim=16, scale=0.4, rot_dims=24, rope_base=1e4, kind="attention_2", chunk=21,
+                           row_norm=False, interleaved=True, unit=True, sink=True)
+    scan = SelectiveSpec(inner=120, state=12, dt_rank=9, taps=4)
+
+    def moe(ff, shared, experts=12, top=3, groups=4, keep=2):
+        return RoutedFFSpec(ff, None, experts, top, groups, keep, score="sigmoid", group_best=2, renorm=True, scale=1.7, shared_ff=shared)
+    specs = [(scan, moe(40, 56)), (diff, moe(32, 24)), (chunk, None), (scan, moe(24, 48, 8, 2, 1, 1))]
+    loop = (1, 4, 2)
+    return ModelConfig.layered("Barorax", unroll_loop(specs, loop), width=width, vocab=vocab, eps=eps, max_pos=4096, name="tiny-barorax", loop=loop)
 
 
 @dataclass

@@ -32,6 +32,8 @@ from .layered import assemble_layers, random_param
 from .layered_ops import LayeredOps
 from .parallel_layers import load_loop, load_tanh_norm
 from .parallel_ops import ParallelOps
+from .prenorm_layers import load_loop as load_steps
+from .prenorm_ops import PrenormOps
 
 
 @dataclass
@@ -54,7 +56,7 @@ class ModelWeights:
     layers: list                       # LayerWeights of this stage's blocks
     final_norm: torch.Tensor | None    # [H] (last stage); parallel layers: a TanhNorm
     lm_head: torch.Tensor | None       # [V / tp, H] (last stage)
-    loop: object = None                # LoopWeights of a design that runs some layers several times
+    loop: object = None                # LoopWeights or StepWeights of a design that runs some layers several times
 
 
 def shard_shapes(cfg: ModelConfig, lay: ParallelLayout):
@@ -117,9 +119,11 @@ def _random_layered(cfg, device, seed, std, dtype) -> ModelWeights:
 
 def layered_weights(cfg, get) -> ModelWeights:
     """Weights of a design that lists its layers; get(name) returns the checkpoint tensor of that name."""
-    final = load_tanh_norm(get, "final.norm") if cfg.is_parallel else get("final.norm").float().reshape(1)
+    final = load_tanh_norm(get, "final.norm") if cfg.is_parallel else get("final.norm").float()
+    if not (cfg.is_parallel or cfg.is_prenorm):
+        final = final.reshape(1)
     return ModelWeights(embed=get("embed").contiguous(), layers=assemble_layers(cfg, get), final_norm=final, lm_head=get("head").contiguous(),
-                        loop=load_loop(cfg, get))
+                        loop=(load_steps if cfg.is_prenorm else load_loop)(cfg, get))
 
 
 def quantize_blocks(weights: ModelWeights, blocks, names=("wqkv", "wo", "w13", "w2"), drop_bf16: bool = True) -> None:
@@ -168,7 +172,7 @@ class SamplingInputs:
     step: torch.Tensor                 # [B] int32: counter of each row's random stream (the token's position)
 
 
-class Decoder(LayeredOps, ParallelOps):
+class Decoder(LayeredOps, ParallelOps, PrenormOps):
     """One rank's share of the model: weights, KV cache and the step function.
 
     The decoder takes ownership of `weights`: on a GPU the expert matrices are replaced in place by their tile-packed
@@ -191,7 +195,7 @@ class Decoder(LayeredOps, ParallelOps):
         dev = (weights.embed if weights.embed is not None else weights.layers[0].attn_norm).device
         self.device = dev
         if cfg.is_layered:
-            pass                # the latent kernels take every head size
+            pass                # their kernels take every head size
         elif dev.type == "cuda" and cfg.head_dim != 128:
             # say so when the model is set up, not in the middle of the first request
             raise ValueError(f"the attention kernels are built for head size 128; this model has {cfg.head_dim}")

@@ -1,9 +1,10 @@
 """Designs whose configuration lists the layers one by one, each with its own mixer and feed-forward: specification,
 parameter names and shapes, weights.
 
-Two kinds of layers exist. A post-norm layer is x <- norm1(alpha x + mixer(h)), x <- norm2(alpha x + ff(x)), with RMS norms
+Three kinds of layers exist. A post-norm layer is x <- norm1(alpha x + mixer(h)), x <- norm2(alpha x + ff(x)), with RMS norms
 whose gain is one number, and h = x + (short causal convolution of x over time). A parallel layer is
-x <- x + (mixer(h) + ff(h)) with h = tanh(a x) w + b (models/parallel_layers.py). Several layers may use one layer's tensors
+x <- x + (mixer(h) + ff(h)) with h = tanh(a x) w + b (models/parallel_layers.py). A pre-norm layer is x <- x + mixer(norm1(x)),
+x <- x + ff(norm2(x)) with RMS norms (models/prenorm_layers.py). Several layers may use one layer's tensors
 (`weights_of`); each keeps a cache of its own. A range of layers may run several times (`loop`): ModelConfig.layers then lists
 every run, the later ones with `weights_of` the first. The registry below names, per architecture, the kind of its layers and
 which mixers exist:
@@ -13,6 +14,9 @@ which mixers exist:
   Sikalorn  parallel             sliding-window attention beside a state-space recurrence, both on the same input
             delta                gated delta rule
             lightning            linear attention with a fixed decay per head
+  Barorax   attention            differential attention (two maps per head over the same values), gated
+            attention_2          attention inside chunks, unit queries and keys, a sink
+            mamba1               selective scan
 """
 from __future__ import annotations
 
@@ -21,12 +25,14 @@ from dataclasses import dataclass, field
 import torch
 
 from . import parallel_layers as pl
-from .parallel_layers import MixerPairSpec, RecurrentSpec, SpecError, WindowAttnSpec  # noqa: F401
+from .parallel_layers import MixerPairSpec, RecurrentSpec, SelectiveSpec, SpecError, WindowAttnSpec  # noqa: F401
 
 # architecture -> mixer type -> (queries through a latent, output gate), or the parser of the mixer
 LAYERED_ARCHS = {"Zarorax": {"latent_attention": (True, False), "latent_attention_2": (False, True)},
-                 "Sikalorn": {"parallel": pl.parse_pair, "delta": pl.parse_delta, "lightning": pl.parse_lightning}}
+                 "Sikalorn": {"parallel": pl.parse_pair, "delta": pl.parse_delta, "lightning": pl.parse_lightning},
+                 "Barorax": {"attention": pl.parse_differential, "attention_2": pl.parse_chunked, "mamba1": pl.parse_selective}}
 PARALLEL_ARCHS = {"Sikalorn"}      # the architectures of parallel layers
+PRENORM_ARCHS = {"Barorax"}        # ... and of pre-norm layers
 
 GLU_SLOPE = 1.702          # g * sigmoid(GLU_SLOPE * g) of the clamped gated unit
 
@@ -70,16 +76,25 @@ class DenseFFSpec:
 @dataclass(frozen=True)
 class RoutedFFSpec:
     ff: int                  # of one expert
-    limit: float
+    limit: float | None      # of the clamped gated unit; None: silu(g) u
     experts: int
     top: int
     groups: int = 1          # neighbouring experts form equal groups ...
     keep: int = 1            # ... of which the best `keep` are eligible
+    score: str = "softmax"   # of the router's logits: softmax over all experts, or a sigmoid each
+    group_best: int = 1      # a group's score is the sum of its 1 or 2 largest scores
+    renorm: bool = False     # the chosen scores are divided by their sum
+    scale: float = 1.0       # ... and multiplied by this
+    shared_ff: int = 0       # size of an expert that runs for every token (0: none)
+
+    def check(self) -> None:
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups or not 1 <= self.top <= self.keep * (self.experts // self.groups):
+            raise SpecError(f"{self.top} of {self.experts} experts cannot be chosen from {self.keep} of {self.groups} groups")
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentMixerSpec | MixerPairSpec | RecurrentSpec
+    mixer: LatentMixerSpec | MixerPairSpec | RecurrentSpec | WindowAttnSpec | SelectiveSpec
     mlp: DenseFFSpec | RoutedFFSpec | None
     weights_of: int | None = None
     tensors: int | None = None     # number of this layer in the checkpoint's names, where that is not its place in the list
@@ -89,8 +104,8 @@ class LayerSpec:
 def parse_layers(arch: str, layers: list, loop: dict | None = None) -> tuple:
     """The configuration's `layers` list (and `loop`) -> LayerSpec tuple (`weights_of` chains resolved to the layer that owns
     tensors, loops to one entry per run)."""
-    if arch in PARALLEL_ARCHS:
-        return _parse_parallel_layers(arch, layers, loop)
+    if arch in PARALLEL_ARCHS | PRENORM_ARCHS:
+        return _parse_runs(arch, layers, loop)
     kinds = LAYERED_ARCHS[arch]
     out = []
     for i, d in enumerate(layers):
@@ -116,8 +131,10 @@ def parse_layers(arch: str, layers: list, loop: dict | None = None) -> tuple:
             g = r.get("groups") or {"count": 1, "keep": 1}
             ff = RoutedFFSpec(int(mlp["expert"]["ff"]), float(mlp["expert"]["limit"]), int(r["experts"]), int(r["top"]),
                               int(g["count"]), int(g["keep"]))
-            if ff.experts % ff.groups or not 1 <= ff.keep <= ff.groups or not 1 <= ff.top <= ff.keep * (ff.experts // ff.groups):
-                raise SpecError(f"layer {i}: {ff.top} of {ff.experts} experts cannot be chosen from {ff.keep} of {ff.groups} groups")
+            try:
+                ff.check()
+            except SpecError as e:
+                raise SpecError(f"layer {i}: {e}") from e
         else:
             raise SpecError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
         src = d.get("weights_of")
@@ -133,17 +150,22 @@ def parse_layers(arch: str, layers: list, loop: dict | None = None) -> tuple:
     return tuple(out)
 
 
-def _parse_parallel_layers(arch: str, layers: list, loop: dict | None) -> tuple:
-    specs = []
+def _parse_dense(mlp: dict) -> DenseFFSpec:
+    if mlp["kind"] != "dense":
+        raise SpecError(f"feed-forward kind {mlp['kind']!r} is not supported")
+    return DenseFFSpec(int(mlp["ff"]))
+
+
+def _parse_runs(arch: str, layers: list, loop: dict | None) -> tuple:
+    """Layers whose mixers have a parser each, one entry per run of a loop."""
+    specs, parse_ff = [], pn.parse_ff if arch in PRENORM_ARCHS else _parse_dense
     for i, d in enumerate(layers):
         parse = LAYERED_ARCHS[arch].get(d.get("type"))
         if parse is None:
             raise SpecError(f"layer {i}: mixer type {d.get('type')!r} is not part of {arch}")
         mlp = d.get("mlp")
-        if mlp is not None and mlp["kind"] != "dense":
-            raise SpecError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not supported")
         try:
-            specs.append((parse(d["mixer"]), DenseFFSpec(int(mlp["ff"])) if mlp is not None else None))
+            specs.append((parse(d["mixer"]), parse_ff(mlp) if mlp is not None else None))
         except SpecError as e:
             raise SpecError(f"layer {i}: {e}") from e
     return unroll_loop(specs, pl.parse_loop(loop, len(specs)))
@@ -163,8 +185,7 @@ def layers_to_list(layers) -> list:
     """Inverse of parse_layers."""
     if layers and layers[0].tensors is not None:
         own = [sp for sp in layers if sp.weights_of is None]
-        return [{"type": sp.mixer.kind, "mixer": sp.mixer.to_dict(), "mlp": None if sp.mlp is None else {"kind": "dense", "ff": sp.mlp.ff}}
-                for sp in sorted(own, key=lambda sp: sp.tensors)]
+        return [{"type": sp.mixer.kind, "mixer": sp.mixer.to_dict(), "mlp": _ff_to_dict(sp.mlp)} for sp in sorted(own, key=lambda sp: sp.tensors)]
     out = []
     for sp in layers:
         m = sp.mixer
@@ -172,28 +193,37 @@ def layers_to_list(layers) -> list:
                  "rot": {"base": m.rope_base, "dims": m.rot_dim}}
         if m.q_rank:
             mixer["q_rank"] = m.q_rank
-        if sp.mlp is None:
-            mlp = None
-        elif isinstance(sp.mlp, DenseFFSpec):
-            mlp = {"kind": "dense", "ff": sp.mlp.ff}
-        else:
-            r = {"experts": sp.mlp.experts, "top": sp.mlp.top}
-            if (sp.mlp.groups, sp.mlp.keep) != (1, 1):
-                r["groups"] = {"count": sp.mlp.groups, "keep": sp.mlp.keep}
-            mlp = {"kind": "moe", "expert": {"ff": sp.mlp.ff, "limit": sp.mlp.limit}, "router": r}
-        d = {"type": m.kind, "mixer": mixer, "mlp": mlp}
+        d = {"type": m.kind, "mixer": mixer, "mlp": _ff_to_dict(sp.mlp)}
         if sp.weights_of is not None:
             d["weights_of"] = sp.weights_of
         out.append(d)
     return out
 
 
+def _ff_to_dict(f) -> dict | None:
+    if f is None:
+        return None
+    if isinstance(f, DenseFFSpec):
+        return {"kind": "dense", "ff": f.ff}
+    r, expert = {"experts": f.experts, "top": f.top}, {"ff": f.ff}
+    if (f.groups, f.keep) != (1, 1):
+        r["groups"] = {"count": f.groups, "keep": f.keep}
+    if f.limit is not None:
+        expert["limit"] = f.limit
+    if f.renorm:
+        r["scale"] = f.scale
+    d = {"kind": "moe", "expert": expert, "router": r}
+    if f.shared_ff:
+        d["shared"] = {"ff": f.shared_ff}
+    return d
+
+
 def param_shapes(cfg) -> dict:
     """Checkpoint tensor name -> shape, in file order (layers with `weights_of` own none)."""
     C = cfg.hidden_size
     s = {"embed": (cfg.vocab_size, C)}
-    if cfg.is_parallel:
-        s.update(pl.param_shapes(cfg))
+    if cfg.is_parallel or cfg.is_prenorm:
+        s.update((pl if cfg.is_parallel else pn).param_shapes(cfg))
         s["head"] = (cfg.vocab_size, C)
         return s
     for i, sp in enumerate(cfg.layers):
@@ -228,8 +258,8 @@ def param_shapes(cfg) -> dict:
 def active_params(cfg) -> int:
     """Weights one token multiplies with (its chosen experts only), output projection included."""
     C, n = cfg.hidden_size, cfg.vocab_size * cfg.hidden_size
-    if cfg.is_parallel:
-        return n + pl.active_params(cfg)
+    if cfg.is_parallel or cfg.is_prenorm:
+        return n + (pl if cfg.is_parallel else pn).active_params(cfg)
     for sp in cfg.layers:
         m = sp.mixer
         n += C * (m.cache_width + m.heads * m.vdim * (2 if m.gated else 1)) + m.heads * (m.dim + m.vdim) * m.kv_rank
@@ -252,6 +282,10 @@ def decode_gemm_shapes(cfg) -> list:
             out.append((name, F, K, E, swiglu))
     for i, sp in enumerate(cfg.layers):
         m = sp.mixer
+        if cfg.is_prenorm:
+            for name, F, K, E, swiglu in pn.gemm_shapes(sp, C):
+                add(f"l{i}.{name}", F, K, E, swiglu)
+            continue
         if cfg.is_parallel:
             lay = pl.LayerLayout(sp)
             add(f"l{i}.in", lay.in_rows, C)
@@ -330,6 +364,14 @@ def assemble_mixer(m: LatentMixerSpec, get, prefix: str) -> LatentMixerWeights:
         off_kv=offs[1], off_gate=offs[2] if m.gated else -1)
 
 
+def stack_experts(f: RoutedFFSpec, get, p: str):
+    """(router, gate and up rows of every expert [E, 2 ff, C], down [E, C, ff]) of the layer with prefix p."""
+    E = range(f.experts)
+    return (get(p + "mlp.router").contiguous(),
+            torch.stack([torch.cat([get(f"{p}mlp.e{e}.gate"), get(f"{p}mlp.e{e}.up")], dim=0) for e in E]).contiguous(),
+            torch.stack([get(f"{p}mlp.e{e}.down") for e in E]).contiguous())
+
+
 def assemble_layers(cfg, get) -> list:
     """One LayeredWeights per layer; layers that share tensors share the object."""
     out = []
@@ -337,8 +379,8 @@ def assemble_layers(cfg, get) -> list:
         if sp.weights_of is not None:
             out.append(out[sp.weights_of])
             continue
-        if cfg.is_parallel:
-            out.append(pl.assemble_layer(sp, get))
+        if cfg.is_parallel or cfg.is_prenorm:
+            out.append((pl if cfg.is_parallel else pn).assemble_layer(sp, get))
             continue
         p = f"l{i}."
         lw = LayeredWeights(mixer=assemble_mixer(sp.mixer, get, p + "mix."), conv=get(p + "canon1").float().t().contiguous(),
@@ -347,10 +389,7 @@ def assemble_layers(cfg, get) -> list:
         if isinstance(sp.mlp, DenseFFSpec):
             lw.w_up, lw.w2, lw.act = get(p + "mlp.up").contiguous(), get(p + "mlp.down").contiguous(), get(p + "mlp.act").float()
         elif isinstance(sp.mlp, RoutedFFSpec):
-            E = range(sp.mlp.experts)
-            lw.router = get(p + "mlp.router").contiguous()
-            lw.w13 = torch.stack([torch.cat([get(f"{p}mlp.e{e}.gate"), get(f"{p}mlp.e{e}.up")], dim=0) for e in E]).contiguous()
-            lw.w2 = torch.stack([get(f"{p}mlp.e{e}.down") for e in E]).contiguous()
+            lw.router, lw.w13, lw.w2 = stack_experts(sp.mlp, get, p)
         out.append(lw)
     return out
 
@@ -367,3 +406,6 @@ def random_param(name: str, shape, gen, std: float, dtype, device):
     if name.endswith(".act"):
         t += 0.5
     return t.to(dtype)
+
+
+from . import prenorm_layers as pn  # noqa: E402  (uses the specifications above)

@@ -30,6 +30,8 @@ class LayeredOps:
             raise ValueError(f"{cfg.architecture} runs on one device (tp = pp = ep = 1)")
         if cfg.is_parallel:
             return self._init_parallel(num_pages, state_slots)
+        if cfg.is_prenorm:
+            return self._init_prenorm(num_pages, state_slots)
         self.act_dtype = w.embed.dtype
         tables = {}
         for sp in cfg.layers:
@@ -171,10 +173,13 @@ class LayeredOps:
     def _op_glu_gate_up(self, st, li):
         mlp = self.cfg.layers[li].mlp
         _, _, counts, offsets, _, _, xs = st.routed
-        st.h = ops.grouped_linear(xs, self.w.layers[li].w13, counts, offsets, swiglu=True, glu=(mlp.limit, GLU_SLOPE))
+        st.normed = None
+        st.h = ops.grouped_linear(xs, self.w.layers[li].w13, counts, offsets, swiglu=True, glu=None if mlp.limit is None else (mlp.limit, GLU_SLOPE))
 
     def _op_glu_down(self, st, li):
         ids, wts, counts, offsets, row_of, _, _ = st.routed
         st.pending = ops.grouped_linear(st.h, self.w.layers[li].w2, counts, offsets)
         st.row_idx, st.row_w = row_of.view(ids.shape), wts
         st.h = st.routed = None
+        if self.cfg.is_prenorm:
+            self._layer_done(st)

@@ -1,17 +1,22 @@
-"""Parallel layers, x <- x + (mixer(h) + ff(h)) with h = tanh(alpha x) w + b: specification, parameter names, weights.
+"""Parallel layers, x <- x + (mixer(h) + ff(h)) with h = tanh(alpha x) w + b: specification, parameter names, weights; and the mixers
+that other layers (models/prenorm_layers.py) share with them.
 
 Mixers (specifications are data; a design picks some and fixes nothing else):
 
-  WindowAttnSpec   grouped-query attention over a sliding window; RMS norm of the whole q and k projections, then rotation of
-                   the first rot_dims dimensions of every head (pairs i, i + rot_dims / 2; frequencies divided by rot_factor)
+  WindowAttnSpec   grouped-query attention over a sliding window, over chunks or over everything before; RMS norm of the whole q and k
+                   projections (or none), then rotation of the first rot_dims dimensions of every head (pairs i, i + rot_dims / 2, or
+                   neighbours; frequencies divided by rot_factor), then unit heads (or not); a sink; two maps per head of which the
+                   second is subtracted; an output gate
   RecurrentSpec    a matrix state S [dim, vdim] per head, 32-bit, carried from token to token:
                        S <- g S + k u^T,   o = S^T q (+ D v)
                      "delta"      g per head and token, u = beta (v - (g S)^T k), q and k unit vectors
                      "ssd"        g = exp(-exp(A) dt), u = dt v (Mamba-2; q, k, v are C, B, x)
                      "lightning"  g fixed per head, u = v
+  SelectiveSpec    a diagonal recurrence per channel (Mamba), 32-bit, behind a short convolution:
+                       S[n, c] <- exp(dt[c] A[n, c]) S[n, c] + dt[c] x[c] B[n],   y[c] = sum_n S[n, c] C[n] + D[c] x[c],   y silu(z)
   MixerPairSpec    an attention and a recurrence beside each other, summed with a weight each
 
-A layer runs as one product from h (w_in: the feed-forward's up projection and every projection of the mixer, stacked), the
+A parallel layer runs as one product from h (w_in: the feed-forward's up projection and every projection of the mixer, stacked), the
 mixer's own kernels, and one product back (w_out: the mixers' output projections and the feed-forward's down projection side
 by side, so that their sum is the product's). LayerLayout says where everything sits in the row between the two products:
 
@@ -47,10 +52,31 @@ class WindowAttnSpec:
     rope_base: float
     rope_factor: float = 1.0
     window: int = 0          # position i sees j with 0 <= i - j < window (0: every earlier position)
+    kind: str = ""           # mixer type of the configuration, where the attention is a mixer of its own
+    chunk: int = 0           # position i sees the j of its own chunk of this many positions, counted from 0 (0: no chunks)
+    row_norm: bool = True    # RMS norm over all of q and all of k, with a weight, before the rotation
+    interleaved: bool = False    # rotated pairs are neighbours
+    unit: bool = False       # heads of q and k are divided by their root mean square after the rotation
+    sink: bool = False       # one more term exp(0) in the softmax's denominator
+    diff: float | None = None    # two maps per head over the same values: (1 - diff) N(map 1 - lambda map 2) with lambda learned around diff
+    gated: bool = False      # the output is multiplied by the sigmoid of a projection
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.diff is None else 2
+
+    @property
+    def head_size(self) -> int:
+        return self.dim
+
+    @property
+    def key_width(self) -> int:
+        """Elements of a key head in the cache: its maps side by side."""
+        return self.maps * self.dim
 
     @property
     def cache_elems_per_token(self) -> int:
-        return self.kv_heads * (self.dim + self.vdim)
+        return self.kv_heads * (self.key_width + self.vdim)
 
     @property
     def out_width(self) -> int:
@@ -58,11 +84,15 @@ class WindowAttnSpec:
 
     def sections(self) -> list:
         """(tensor, rows) of the projections of h, in stacking order."""
-        return [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+        s = [("q", self.heads * self.key_width), ("k", self.kv_heads * self.key_width), ("v", self.kv_heads * self.vdim)]
+        return s + [("g", self.out_width)] if self.gated else s
 
     def param_shapes(self, C: int) -> dict:
         s = {n: (rows, C) for n, rows in self.sections()}
-        s["q.norm"], s["k.norm"] = (self.heads * self.dim,), (self.kv_heads * self.dim,)
+        if self.row_norm:
+            s["q.norm"], s["k.norm"] = (self.heads * self.dim,), (self.kv_heads * self.dim,)
+        if self.diff is not None:
+            s.update({n: (self.dim,) for n in LAMBDA_VECTORS})
         s["o"] = (C, self.out_width)
         return s
 
@@ -71,9 +101,14 @@ class WindowAttnSpec:
         if self.rope_factor != 1.0:
             rot["scaling"] = {"factor": self.rope_factor}
         d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": rot}
-        if self.window:
-            d["mask"] = {"size": self.window}
+        if self.window or self.chunk:
+            d["mask"] = {"size": self.window or self.chunk}
+        if self.diff is not None:
+            d["diff"] = self.diff
         return d
+
+
+LAMBDA_VECTORS = ("lq1", "lk1", "lq2", "lk2")      # lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff
 
 
 @dataclass(frozen=True)
@@ -150,6 +185,59 @@ class RecurrentSpec:
 
 
 @dataclass(frozen=True)
+class SelectiveSpec:
+    inner: int               # channels
+    state: int               # state dimensions of a channel
+    dt_rank: int             # width of the step sizes' bottleneck
+    taps: int = 1            # of the short convolution over time
+    kind: str = "mamba1"
+    heads: int = 1
+
+    @property
+    def cache_elems_per_token(self) -> int:
+        return 0
+
+    @property
+    def out_width(self) -> int:
+        return self.inner
+
+    @property
+    def head_size(self) -> int:
+        return self.state
+
+    @property
+    def conv_channels(self) -> int:
+        return self.inner
+
+    @property
+    def conv_rows(self) -> int:
+        """Cached inputs of the convolution. One more than it looks back, so that a step writes no row that it reads."""
+        return self.taps if self.taps > 1 else 0
+
+    @property
+    def state_elems(self) -> int:
+        return self.inner * self.state
+
+    def state_bytes(self, elem: int = 2) -> int:
+        return 4 * self.state_elems + elem * self.conv_rows * self.inner
+
+    def sections(self) -> list:
+        return [("x", self.inner), ("z", self.inner)]
+
+    def x_sections(self) -> list:
+        """(name, rows) of the projections of the convolved x: step sizes' bottleneck, B, C."""
+        return [("dt", self.dt_rank), ("B", self.state), ("C", self.state)]
+
+    def param_shapes(self, C: int) -> dict:
+        I, N, R = self.inner, self.state, self.dt_rank
+        return {"in": (2 * I, C), "conv": (I, self.taps), "conv.b": (I,), "x": (R + 2 * N, I), "dt": (I, R), "dt.b": (I,), "A_log": (I, N),
+                "D": (I,), "o": (C, I)}
+
+    def to_dict(self) -> dict:
+        return {"conv": self.taps, "dt_rank": self.dt_rank, "inner": self.inner, "state": self.state}
+
+
+@dataclass(frozen=True)
 class MixerPairSpec:
     left: WindowAttnSpec
     right: RecurrentSpec
@@ -174,11 +262,11 @@ class MixerPairSpec:
 
 
 def attention_of(mixer) -> WindowAttnSpec | None:
-    return mixer.left if isinstance(mixer, MixerPairSpec) else None
+    return mixer.left if isinstance(mixer, MixerPairSpec) else mixer if isinstance(mixer, WindowAttnSpec) else None
 
 
-def recurrence_of(mixer) -> RecurrentSpec | None:
-    return mixer.right if isinstance(mixer, MixerPairSpec) else mixer if isinstance(mixer, RecurrentSpec) else None
+def recurrence_of(mixer) -> RecurrentSpec | SelectiveSpec | None:
+    return mixer.right if isinstance(mixer, MixerPairSpec) else mixer if isinstance(mixer, (RecurrentSpec, SelectiveSpec)) else None
 
 
 # ---- configuration -------------------------------------------------------------------------------------------------
@@ -187,15 +275,33 @@ def _need(ok: bool, what: str) -> None:
         raise SpecError(what)
 
 
-def parse_window(m: dict) -> WindowAttnSpec:
-    rot, mask = m["rot"], m.get("mask") or {}
+def parse_window(m: dict, mask: str = "window", **fixed) -> WindowAttnSpec:
+    """An attention mixer; `mask` is what mask.size counts ("window" or "chunk"), `fixed` the properties that the design fixes."""
+    rot, size = m["rot"], int((m.get("mask") or {}).get("size") or 0)
     a = WindowAttnSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]),
                        rot_dims=int(rot["dims"]), rope_base=float(rot["base"]), rope_factor=float((rot.get("scaling") or {}).get("factor", 1.0)),
-                       window=int(mask.get("size") or 0))
+                       **{mask: size}, **fixed)
     _need(a.heads % a.kv_heads == 0, "heads must be a multiple of kv_heads")
     _need(a.rot_dims % 2 == 0 and 0 <= a.rot_dims <= a.dim, "rot.dims must be even and at most dim (rotation turns pairs)")
-    _need(a.window >= 0 and a.rope_factor > 0, "mask.size and rot.scaling.factor must be positive")
+    _need(size >= 0 and a.rope_factor > 0, "mask.size and rot.scaling.factor must be positive")
     return a
+
+
+def parse_differential(m: dict) -> WindowAttnSpec:
+    return parse_window(m, kind="attention", row_norm=False, interleaved=True, diff=float(m["diff"]), gated=True)
+
+
+def parse_chunked(m: dict) -> WindowAttnSpec:
+    a = parse_window(m, mask="chunk", kind="attention_2", row_norm=False, interleaved=True, unit=True, sink=True)
+    _need(a.chunk > 0, "mask.size must be positive")
+    return a
+
+
+def parse_selective(m: dict) -> SelectiveSpec:
+    r = SelectiveSpec(inner=int(m["inner"]), state=int(m["state"]), dt_rank=int(m["dt_rank"]), taps=int(m["conv"]))
+    _need(min(r.inner, r.state, r.dt_rank) >= 1, "inner, state and dt_rank must be positive")
+    _need(r.taps >= 1, "conv must be at least 1")
+    return r
 
 
 def parse_ssd(m: dict) -> RecurrentSpec:
@@ -290,13 +396,15 @@ class Section:
 
 
 class LayerLayout:
-    def __init__(self, sp):
+    """`ff` False: the feed-forward is not part of the row (layers that run it behind the mixer)."""
+
+    def __init__(self, sp, ff: bool = True):
         self.parts, at = [], 0
         parts = _mixer_parts(sp.mixer)
         for _, m, scale in parts:
             self.parts.append(Section(m, scale, at, {}))
             at += up8(m.out_width)
-        self.ff, self.ff_cols = at, up8(sp.mlp.ff) if sp.mlp is not None else 0
+        self.ff, self.ff_cols = at, up8(sp.mlp.ff) if ff and sp.mlp is not None else 0
         self.in_first = at               # w_in writes from here
         at += self.ff_cols
         self.out_cols = at               # w_out reads up to here
@@ -322,8 +430,20 @@ class TanhNorm:
 
 @dataclass
 class WindowAttnWeights:
-    q_norm: torch.Tensor     # [heads * dim] fp32
-    k_norm: torch.Tensor     # [kv_heads * dim] fp32
+    q_norm: torch.Tensor | None = None     # [heads * dim] fp32
+    k_norm: torch.Tensor | None = None     # [kv_heads * dim] fp32
+    lam: torch.Tensor | None = None        # [1] fp32: weight of the second map
+
+
+@dataclass
+class SelectiveWeights:
+    w_x: torch.Tensor                      # [x_rows, inner]: the sections of x_sections, each from a multiple of 8 rows
+    w_dt: torch.Tensor                     # [inner, dt_rank], columns padded with zeros to a multiple of 8
+    conv: torch.Tensor                     # [taps, inner] fp32
+    conv_b: torch.Tensor                   # [inner] fp32
+    dt_bias: torch.Tensor                  # [inner] fp32
+    neg_a: torch.Tensor                    # [state, inner] fp32: -exp(A_log)
+    skip: torch.Tensor                     # [inner] fp32: D
 
 
 @dataclass
@@ -370,6 +490,23 @@ def _pad(t: torch.Tensor, dim: int) -> torch.Tensor:
     return torch.cat([t, torch.zeros(shape, dtype=t.dtype, device=t.device)], dim=dim)
 
 
+def load_attention(m: WindowAttnSpec, get, p: str) -> WindowAttnWeights:
+    w = WindowAttnWeights()
+    if m.row_norm:
+        w.q_norm, w.k_norm = get(p + "q.norm").float(), get(p + "k.norm").float()
+    if m.diff is not None:
+        lq1, lk1, lq2, lk2 = (get(p + n).double() for n in LAMBDA_VECTORS)
+        w.lam = ((lq1 * lk1).sum().exp() - (lq2 * lk2).sum().exp() + m.diff).float().reshape(1)
+    return w
+
+
+def load_selective(m: SelectiveSpec, get, p: str) -> SelectiveWeights:
+    x = get(p + "x").split([rows for _, rows in m.x_sections()])
+    return SelectiveWeights(w_x=torch.cat([_pad(t, 0) for t in x]).contiguous(), w_dt=_pad(get(p + "dt"), 1).contiguous(),
+                            conv=get(p + "conv").float().t().contiguous(), conv_b=get(p + "conv.b").float(), dt_bias=get(p + "dt.b").float(),
+                            neg_a=-get(p + "A_log").float().t().exp().contiguous(), skip=get(p + "D").float())
+
+
 def _load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
     w = RecurrentWeights(norm=get(p + "norm").float())
     GD, HV = m.groups * m.dim, m.heads * m.vdim
@@ -396,7 +533,7 @@ def assemble_layer(sp, get) -> ParallelLayerWeights:
     for pre, m, _ in _mixer_parts(sp.mixer):
         q = p + pre
         if isinstance(m, WindowAttnSpec):
-            attn = WindowAttnWeights(get(q + "q.norm").float(), get(q + "k.norm").float())
+            attn = load_attention(m, get, q)
         else:
             rec = _load_recurrence(m, get, q)
         if isinstance(m, RecurrentSpec) and m.kind == "ssd":
@@ -424,8 +561,10 @@ def random_param(name: str, shape, gen, device):
         return normal(shape[-1] ** -0.5)
     if name.endswith(".A_log"):
         return normal(1.0)
-    if name.endswith(".dt_bias"):
+    if name.endswith((".dt_bias", ".dt.b")):
         return normal(1.0, -3.0)
+    if name.endswith(tuple("." + n for n in LAMBDA_VECTORS)):
+        return normal(0.1)
     if name.endswith(".D"):
         return torch.ones(shape, device=device)
     return None

@@ -89,18 +89,23 @@ class ParallelOps:
     def _window_section(self, st, li):
         sec = self.layouts[li].part(WindowAttnSpec)
         a = sec.spec
-        q, k, v = (st.qkv[:, sec.col[n]:sec.col[n] + rows] for n, rows in a.sections())
+        q, k, v = (st.qkv[:, sec.col[n]:sec.col[n] + rows] for n, rows in a.sections()[:3])
         return sec, a, q, k, v
 
     def _op_window_append(self, st, li):
         _, a, q, k, v = self._window_section(st, li)
         w, inp = self.w.layers[li].attn, st.inp
-        par.window_append(q, k, v, w.q_norm, w.k_norm, a, self.rope_tables[li], inp.positions, inp.seq_of_token, inp.block_table, self.kv[li],
-                          self.page_size, self.cfg.rms_norm_eps)
+        args = (self.rope_tables[li], inp.positions, inp.seq_of_token, inp.block_table, self.kv[li], self.page_size, self.cfg.rms_norm_eps)
+        if a.row_norm:
+            par.window_append(q, k, v, w.q_norm, w.k_norm, a, *args)
+        else:
+            par.head_append(q, k, v, a, *args)
 
     def _op_window_attention(self, st, li):
         sec, a, q, _, _ = self._window_section(st, li)
-        par.window_attn(q, a, st.inp, self.kv[li], self.page_size, st.qkv[:, sec.out:sec.out + a.out_width], sec.scale)
+        gate = st.qkv[:, sec.col["g"]:sec.col["g"] + a.out_width] if a.gated else None
+        par.window_attn(q, a, st.inp, self.kv[li], self.page_size, st.qkv[:, sec.out:sec.out + a.out_width], sec.scale,
+                        par.HeadMix(self.w.layers[li].attn.lam, gate, self.cfg.rms_norm_eps))
 
     def _op_recurrence(self, st, li):
         sec, inp = self.layouts[li].part(RecurrentSpec), st.inp

@@ -2,4 +2,4 @@
 from . import reference
 from .functional import *  # noqa: F401,F403
 from .functional import workspace, Workspace
-from . import latent, parallel, recurrent  # noqa: F401
+from . import latent, parallel, prenorm, recurrent, selective  # noqa: F401

@@ -62,6 +62,30 @@ class RecChunk(C.Structure):
         ("qkv_ld", C.c_int64), ("v_off", C.c_int32), ("max_q_len", C.c_int32)]
 
 
+class RouteRule(C.Structure):
+    """Mirror of SkeinRouteRule in csrc/kernels/route.cuh (same field order)."""
+
+    _fields_ = [(n, C.c_int32) for n in ("n_groups", "keep", "score", "group_best", "renorm")] + [("scale", C.c_float)]
+
+
+class AttnRule(C.Structure):
+    """Mirror of SkeinAttnRule in csrc/kernels/attn_rule.cuh (same field order)."""
+
+    _fields_ = [("lam", C.c_void_p), ("gate", C.c_void_p), ("gate_ld", C.c_int64)] + [
+        (n, C.c_int32) for n in ("window", "chunk", "sink", "maps")] + [(n, C.c_float) for n in ("scale", "out_scale", "eps")] + [("pad", C.c_int32)]
+
+
+class ScanParams(C.Structure):
+    """Mirror of SkeinScanParams in csrc/kernels/selective.cu (same field order)."""
+
+    _fields_ = [(n, C.c_void_p) for n in ("x", "xc", "proj", "dt", "z", "out", "state", "tail", "conv_w", "conv_b", "dt_bias", "neg_a", "skip",
+                                          "positions", "slots", "seq_of_token", "q_start", "q_len", "status")] + [
+        (n, C.c_int64) for n in ("x_ld", "proj_ld", "out_ld")] + [(n, C.c_int32) for n in ("I", "N", "taps", "b_col", "c_col", "num_slots")]
+
+
+byref = C.byref
+
+
 def lib_path() -> Path:
     return _LIB_PATH
 
@@ -145,7 +169,10 @@ def lib():
     _sig(L, "skein_post_norm_route", i32,
          [vp, vp, vp, vp, f32, f32, i32, i32, vp, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp])
     _sig(L, "skein_poly_norm", i32, [vp, vp, vp, i32, i32, f32, i32, vp])
-    _sig(L, "skein_route_grouped", i32, [vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, vp, vp, vp])
+    rule = C.POINTER(RouteRule)
+    _sig(L, "skein_route_grouped", i32, [vp, i32, i32, i32, rule, vp, vp, vp, vp, vp, vp, vp])
+    _sig(L, "skein_norm_route", i32, [vp, vp, vp, f32, i32, i32, vp, i32, i32, rule, vp, vp, vp, vp, vp, vp, vp, vp, i32, vp, vp])
+    _sig(L, "skein_add_norm", i32, [vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32, f32, i32, vp])
     _sig(L, "skein_latent_append", i32,
          [vp, i32, i32, vp, i32, vp, i32, i32, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp, i32, vp])
     _sig(L, "skein_rope_rows", i32, [vp, i64, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp])
@@ -160,11 +187,18 @@ def lib():
     _sig(L, "skein_gated_norm", i32, [vp, vp, i64, vp, i32, vp, i64, i32, i32, i32, i32, i32, f32, f32, i32, vp])
     _sig(L, "skein_window_append", i32,
          [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
-    _sig(L, "skein_window_attn_rows", i32, [vp, i64, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, vp])
+    _sig(L, "skein_head_append", i32,
+         [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
+    arule = C.POINTER(AttnRule)
+    _sig(L, "skein_window_attn_rows", i32, [vp, i64, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, arule, i32, vp])
     _sig(L, "skein_attn_decode_window", i32,
-         [vp, i64, vp, vp, vp, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, vp])
+         [vp, i64, vp, vp, vp, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, arule, vp])
     _sig(L, "skein_attn_prefill_window", i32,
-         [vp, i64, i64, vp, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32, vp])
+         [vp, i64, i64, vp, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, arule, vp])
+    scanp = C.POINTER(ScanParams)
+    _sig(L, "skein_short_conv", i32, [scanp, i32, i32, i32, vp])
+    _sig(L, "skein_scan_step", i32, [scanp, i32, i32, vp])
+    _sig(L, "skein_scan_rows", i32, [scanp, i32, i32, vp])
     rec, chunk = C.POINTER(RecParams), C.POINTER(RecChunk)
     _sig(L, "skein_rec_step", i32, [rec, C.POINTER(RecGate), i32, i32, vp])
     _sig(L, "skein_rec_step_gates", i32, [rec])

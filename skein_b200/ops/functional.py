@@ -266,19 +266,21 @@ def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None):
     """silu(x @ w13[:I].T) * (x @ w13[I:].T) with both products from one pass over x."""
     if not x.is_cuda:
         return ref.swiglu_linear(x, w13.unpack() if isinstance(w13, PackedWeight) else w13)
-    _check_bf16(x)
     _check_act(x)
     T, K = x.shape
     inter = w13.shape[0] // 2
     if out is None:
-        out = torch.empty(T, inter, dtype=torch.bfloat16, device=x.device)
+        out = torch.empty(T, inter, dtype=x.dtype, device=x.device)
     if T == 0:
         return out
     wv, rows_pg, packed = _wview(w13)
     p = _base_params(x, wv, out, inter, K, n_tile or pick_n_tile(T, True), 1)
     p.w_rows_per_group, p.w_packed = rows_pg, packed
     p.up_row_off = inter
-    _gemm_launch(p, "swiglu_linear", _cfg)
+    if tc_gemm_ok(x, K):
+        _gemm_launch(p, "swiglu_linear", _cfg)
+    else:
+        simt_launch(p, x, T, "swiglu_linear")
     return out
 
 

@@ -106,11 +106,7 @@ def post_norm_route(x, y, alpha, gain, eps, wg, top, groups, keep):
     E = wg.shape[0]
     dev = x.device
     x_out = torch.empty_like(x)
-    ids = torch.empty(T, top, dtype=torch.int32, device=dev)
-    w = torch.empty(T, top, dtype=torch.float32, device=dev)
-    meta = torch.empty(2 * E + 1 + 2 * T * top, dtype=torch.int32, device=dev)
-    counts, offsets = meta[:E], meta[E:2 * E + 1]
-    row_of, src_token = meta[2 * E + 1:2 * E + 1 + T * top], meta[2 * E + 1 + T * top:]
+    ids, w, counts, offsets, row_of, src_token = route_buffers(T, E, top, dev)
     xs = torch.empty(T * top, C, dtype=torch.bfloat16, device=dev)
     ws = F.workspace()
     rc = _lib.lib().skein_post_norm_route(
@@ -130,17 +126,26 @@ def route_grouped(x, wg, top, groups, keep):
         ids, w = rl.select_grouped(x.float() @ wg.float().t(), top, groups, keep)
         counts, offsets, row_of, src_token = ref.router_plan(ids, E)
         return ids, w, counts, offsets, row_of, src_token, x[src_token.long()]
+    rule = _lib.RouteRule()
+    rule.n_groups, rule.keep, rule.group_best, rule.scale = groups, keep, 1, 1.0
+    return route_by_rule(x, wg, top, rule)
+
+
+def route_buffers(T: int, E: int, top: int, dev):
+    """(ids, weights, counts, offsets, row_of, src_token) of a routed step, uninitialised."""
+    meta = torch.empty(2 * E + 1 + 2 * T * top, dtype=torch.int32, device=dev)
+    return (torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, dtype=torch.float32, device=dev), meta[:E], meta[E:2 * E + 1],
+            meta[2 * E + 1:2 * E + 1 + T * top], meta[2 * E + 1 + T * top:])
+
+
+def route_by_rule(x, wg, top, rule: "_lib.RouteRule"):
+    """Router over the rows of x by any rule (csrc/kernels/route.cuh) and the expert-sorted copy; see route_grouped."""
+    T, E = x.shape[0], wg.shape[0]
     if E > MAX_ROUTE_E:
         raise ValueError(f"the router kernel takes at most {MAX_ROUTE_E} experts")
-    T = x.shape[0]
-    dev = x.device
     logits = F.linear(x, wg, out_f32=True)
-    ids = torch.empty(T, top, dtype=torch.int32, device=dev)
-    w = torch.empty(T, top, dtype=torch.float32, device=dev)
-    meta = torch.empty(2 * E + 1 + 2 * T * top, dtype=torch.int32, device=dev)
-    counts, offsets = meta[:E], meta[E:2 * E + 1]
-    row_of, src_token = meta[2 * E + 1:2 * E + 1 + T * top], meta[2 * E + 1 + T * top:]
-    rc = _lib.lib().skein_route_grouped(logits.data_ptr(), T, E, top, groups, keep, ids.data_ptr(), w.data_ptr(), counts.data_ptr(),
+    ids, w, counts, offsets, row_of, src_token = route_buffers(T, E, top, x.device)
+    rc = _lib.lib().skein_route_grouped(logits.data_ptr(), T, E, top, _lib.byref(rule), ids.data_ptr(), w.data_ptr(), counts.data_ptr(),
                                         offsets.data_ptr(), row_of.data_ptr(), src_token.data_ptr(), _lib.stream_ptr())
     _lib.check(rc, "route_grouped")
     _lib.count_launch(3)

@@ -1,9 +1,13 @@
-"""Operators of parallel layers (x <- x + mixer(h) + ff(h), h = tanh(alpha x) w + b) and of sliding-window attention.
+"""Operators of parallel layers (x <- x + mixer(h) + ff(h), h = tanh(alpha x) w + b) and of grouped-query attention over a window or
+chunks (models/parallel_layers.py: WindowAttnSpec).
 
 CUDA tensors run csrc/kernels (parallel_layer.cu, attn_window.cu, attn_prefill_tc.cu, attn_decode_mma.cu); CPU tensors run
 ops/reference_parallel.py. Activations are bf16, or fp32 when a model runs in 32-bit; the residual stream is fp32.
 """
 from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
 
 import torch
 
@@ -56,9 +60,10 @@ def gated_norm(o, gate, w, out, groups, eps, gate_first=False, silu=False, scale
     return out
 
 
-# ---- sliding-window attention -----------------------------------------------------------------------------------------
+# ---- attention over a window or chunks ----------------------------------------------------------------------------------
 def window_cache(num_pages: int, page_size: int, kv_heads: int, dim: int, vdim: int, dtype, device) -> torch.Tensor:
-    """[pages, kv_heads * page_size * (dim + vdim)]: keys [kv_heads, page_size, dim], then values [kv_heads, page_size, vdim]."""
+    """[pages, kv_heads * page_size * (dim + vdim)]: keys [kv_heads, page_size, dim], then values [kv_heads, page_size, vdim]. `dim` is
+    the width of a key head, its maps side by side."""
     return torch.zeros(num_pages, kv_heads * page_size * (dim + vdim), dtype=dtype, device=device)
 
 
@@ -76,43 +81,81 @@ def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_toke
         _lib.count_launch()
 
 
-def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out, out_scale=1.0):
+def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
+    """Rotation of every head of q (in place) and k, division by its root mean square where the specification asks for it, append of k
+    and v to the cache. q, k, v: columns of one matrix. A head with two maps is two heads here."""
+    T = q.shape[0]
+    if not q.is_cuda:
+        return rp.head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps)
+    if T:
+        _lib.check(_lib.lib().skein_head_append(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), cos_sin.data_ptr(), positions.data_ptr(), _lib.ptr(seq_of_token),
+            block_table.data_ptr(), cache.data_ptr(), F.workspace().status.data_ptr(), T, spec.heads, spec.kv_heads, spec.dim, spec.maps, spec.vdim,
+            spec.rot_dims, int(spec.interleaved), int(spec.unit), cos_sin.shape[0], block_table.stride(0), cache.shape[0], page_size, float(eps),
+            _fp32(q), _lib.stream_ptr()), "head_append")
+        _lib.count_launch()
+
+
+@dataclass
+class HeadMix:
+    """What follows the softmax of a head: the second map's weight (two maps), the gate, the head norm's eps."""
+    lam: torch.Tensor | None = None
+    gate: torch.Tensor | None = None       # [T, heads * vdim], columns of a wider matrix
+    eps: float = 0.0
+
+
+def _attn_rule(spec, mix, out_scale) -> "_lib.AttnRule":
+    """The mask, sink and what follows the softmax, as the kernels take it."""
+    r = _lib.AttnRule()
+    r.window, r.chunk, r.sink, r.maps = spec.window, spec.chunk, int(spec.sink), spec.maps
+    r.scale, r.out_scale = float(spec.scale), float(out_scale)
+    if spec.diff is not None:
+        r.lam, r.eps, r.out_scale = mix.lam.data_ptr(), float(mix.eps), float(out_scale) * (1.0 - spec.diff)
+    if mix is not None and mix.gate is not None:
+        r.gate, r.gate_ld = mix.gate.data_ptr(), mix.gate.stride(0)
+    return r
+
+
+def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out, out_scale=1.0, mix: HeadMix | None = None):
     """Attention of single rows over the cache, any sizes (plain kernel)."""
     T = q.shape[0]
     if not q.is_cuda:
-        out.copy_(rp.window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale))
+        out.copy_(rp.window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale, mix))
         return out
     if T:
+        r = _attn_rule(spec, mix, out_scale)
         _lib.check(_lib.lib().skein_window_attn_rows(
             q.data_ptr(), q.stride(0), cache.data_ptr(), positions.data_ptr(), _lib.ptr(seq_of_token), block_table.data_ptr(), out.data_ptr(),
             out.stride(0), F.workspace().status.data_ptr(), T, spec.heads, spec.kv_heads, spec.dim, spec.vdim, block_table.stride(0),
-            cache.shape[0], page_size, spec.window, float(spec.scale), float(out_scale), _fp32(q), _lib.stream_ptr()), "window_attn_rows")
+            cache.shape[0], page_size, C.byref(r), _fp32(q), _lib.stream_ptr()), "window_attn_rows")
         _lib.count_launch()
     return out
 
 
-def window_attn(q, spec, inp, cache, page_size, out, out_scale=1.0):
-    """Attention of a step's rows (a decode step or a chunk) over the cache. bf16 heads of 128 or 64 run the tensor-core kernels
-    (a decode step's with up to 16 query heads per key head), everything else the plain one."""
-    tc = (q.is_cuda and q.dtype == torch.bfloat16 and spec.dim == spec.vdim and spec.dim in (64, 128) and page_size % 16 == 0
-          and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0 and spec.scale > 0)
-    if not tc or (not inp.is_prefill and (inp.seq_of_token is not None or spec.heads // spec.kv_heads > 16)):
-        return window_attn_rows(q, spec, inp.positions, inp.seq_of_token, inp.block_table, cache, page_size, out, out_scale)
-    ws, bt, H, K, D = F.workspace(), inp.block_table, spec.heads, spec.kv_heads, spec.dim
+def window_attn(q, spec, inp, cache, page_size, out, out_scale=1.0, mix: HeadMix | None = None):
+    """Attention of a step's rows (a decode step or a chunk) over the cache. bf16 heads of 128 or 64 (two maps of 64 over values of 128)
+    run the tensor-core kernels (a decode step's with up to 16 query rows per key head), everything else the plain one."""
+    KW = spec.key_width
+    tc = (q.is_cuda and q.dtype == torch.bfloat16 and KW == spec.vdim and (KW == 128 or (KW == 64 and spec.maps == 1)) and page_size % 16 == 0
+          and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0 and spec.scale > 0)
+    if tc and mix is not None and mix.gate is not None:
+        tc = spec.maps == 2 and mix.gate.data_ptr() % 16 == 0 and mix.gate.stride(0) % 8 == 0
+    if not tc or (not inp.is_prefill and (inp.seq_of_token is not None or spec.maps * (spec.heads // spec.kv_heads) > 16)):
+        return window_attn_rows(q, spec, inp.positions, inp.seq_of_token, inp.block_table, cache, page_size, out, out_scale, mix)
+    ws, bt, H, K, r = F.workspace(), inp.block_table, spec.heads, spec.kv_heads, _attn_rule(spec, mix, out_scale)
     if inp.is_prefill:
         rc = _lib.lib().skein_attn_prefill_window(
             q.data_ptr(), q.stride(0), q.shape[0], cache.data_ptr(), bt.data_ptr(), inp.q_start.data_ptr(), inp.q_len.data_ptr(),
-            inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), ws.status.data_ptr(), inp.q_len.shape[0], int(inp.max_q_len), H, K, D,
-            page_size, bt.stride(0), cache.shape[0], spec.window, float(spec.scale), float(out_scale), _lib.stream_ptr())
+            inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), ws.status.data_ptr(), inp.q_len.shape[0], int(inp.max_q_len), H, K, KW,
+            page_size, bt.stride(0), cache.shape[0], C.byref(r), _lib.stream_ptr())
     else:
-        B = q.shape[0]
-        splits = F.pick_splits(B, K, min(inp.ctx_hint, spec.window or inp.ctx_hint), ws.sm_count)
-        scratch = ws.attn_scratch(B, H, K, splits) if splits > 1 else None
+        B, reach = q.shape[0], spec.window or spec.chunk or inp.ctx_hint
+        splits = F.pick_splits(B, K, min(inp.ctx_hint, reach), ws.sm_count)
+        scratch = ws.attn_scratch(B, H * spec.maps, K, splits) if splits > 1 else None
         splits, (wsf, ctr) = (splits, scratch) if scratch is not None else (1, (None, None))
         rc = _lib.lib().skein_attn_decode_window(
             q.data_ptr(), q.stride(0), cache.data_ptr(), bt.data_ptr(), inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), _lib.ptr(wsf),
-            _lib.ptr(ctr), ws.status.data_ptr(), B, H, K, D, page_size, bt.stride(0), cache.shape[0], splits, spec.window, float(spec.scale),
-            float(out_scale), _lib.stream_ptr())
+            _lib.ptr(ctr), ws.status.data_ptr(), B, H, K, KW, page_size, bt.stride(0), cache.shape[0], splits, C.byref(r), _lib.stream_ptr())
     _lib.check(rc, "window_attn")
     _lib.count_launch()
     return out

@@ -4,6 +4,8 @@ from __future__ import annotations
 
 import torch
 
+from .reference_latent import rotate_pairs
+
 
 def residual_tanh(x, y, bias, norm, dtype):
     a = sum(t.float() for t in (x, y, bias) if t is not None)
@@ -51,20 +53,55 @@ def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_toke
         vals[page, :, pos % page_size] = v[t].view(spec.kv_heads, -1)
 
 
-def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale):
-    keys, vals = _pages(cache, spec.kv_heads, page_size, spec.dim, spec.vdim)
+def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
+    D, W = spec.dim, spec.key_width
+    keys, vals = _pages(cache, spec.kv_heads, page_size, W, spec.vdim)
+
+    def turn(z, cs):
+        z = z.float().view(-1, D)
+        if spec.interleaved:
+            z = torch.cat([rotate_pairs(z[:, :spec.rot_dims], cs), z[:, spec.rot_dims:]], dim=1)
+        else:
+            z = _rotate(z[None], cs, spec.rot_dims)[0]
+        return z / torch.sqrt(z.pow(2).mean(-1, keepdim=True) + eps) if spec.unit else z
+    for t in range(q.shape[0]):
+        pos = int(positions[t])
+        if pos < 0:
+            continue
+        cs = cos_sin[pos:pos + 1]
+        q[t] = turn(q[t], cs).reshape(-1).to(q.dtype)
+        page = int(block_table[int(seq_of_token[t]) if seq_of_token is not None else t, pos // page_size])
+        keys[page, :, pos % page_size] = turn(k[t], cs).view(spec.kv_heads, W).to(cache.dtype)
+        vals[page, :, pos % page_size] = v[t].view(spec.kv_heads, -1)
+
+
+def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale, mix=None):
+    H, D, V, M = spec.heads, spec.dim, spec.vdim, spec.maps
+    keys, vals = _pages(cache, spec.kv_heads, page_size, spec.key_width, V)
     T, G = q.shape[0], spec.heads // spec.kv_heads
-    out = torch.zeros(T, spec.heads * spec.vdim, dtype=q.dtype)
+    out = torch.zeros(T, H * V, dtype=q.dtype)
     for t in range(T):
         pos = int(positions[t])
         if pos < 0:
             continue
-        js = torch.arange(max(0, pos - spec.window + 1) if spec.window else 0, pos + 1)
+        lo = pos // spec.chunk * spec.chunk if spec.chunk else max(0, pos - spec.window + 1) if spec.window else 0
+        js = torch.arange(lo, pos + 1)
         pages = block_table[int(seq_of_token[t]) if seq_of_token is not None else t][js // page_size].long()
-        k = keys[pages, :, js % page_size].float().repeat_interleave(G, dim=1)
+        k = keys[pages, :, js % page_size].float().view(-1, spec.kv_heads, M, D).repeat_interleave(G, dim=1)
         v = vals[pages, :, js % page_size].float().repeat_interleave(G, dim=1)
-        s = torch.einsum("hd,jhd->hj", q[t].float().view(spec.heads, -1), k) * spec.scale
-        out[t] = (torch.einsum("hj,jhv->hv", torch.softmax(s, dim=-1), v) * out_scale).reshape(-1).to(q.dtype)
+        s = torch.einsum("hmd,jhmd->hmj", q[t].float().view(H, M, D), k) * spec.scale
+        if spec.sink:
+            s = torch.cat([s, torch.zeros(H, M, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :len(js)]
+        a = torch.einsum("hmj,jhv->hmv", p, v)
+        o = a[:, 0]
+        if spec.diff is not None:
+            o = a[:, 0] - mix.lam * a[:, 1]
+            o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + mix.eps) * (1.0 - spec.diff)
+        o = o.reshape(-1)
+        if mix is not None and mix.gate is not None:
+            o = o * torch.sigmoid(mix.gate[t].float())
+        out[t] = (o * out_scale).to(q.dtype)
     return out
 
 
