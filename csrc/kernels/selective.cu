@@ -125,6 +125,12 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ScanParams p, int
   }
 }
 
+// exp(dt a) s + b. A decay near one is raised to a high power over a long sequence: in a 32-bit model it is taken as 1 + expm1, whose error
+// shrinks with the step.
+template <typename T> __device__ __forceinline__ float scan_update(float dt, float a, float s, float b);
+template <> __device__ __forceinline__ float scan_update<float>(float dt, float a, float s, float b) { return fmaf(expm1f(dt * a), s, s + b); }
+template <> __device__ __forceinline__ float scan_update<__nv_bfloat16>(float dt, float a, float s, float b) { return fmaf(expf(dt * a), s, b); }
+
 // ---- decode -----------------------------------------------------------------------------------------------
 constexpr int ST_THREADS = 128, ST_UNROLL = 8;
 
@@ -180,7 +186,7 @@ __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(const ScanParams 
       const float B = bc_s[n0 + i], C = bc_s[N + n0 + i];
 #pragma unroll
       for (int k = 0; k < V; ++k) {
-        s[i][k] = fmaf(expf(dt[k] * an[i][k]), s[i][k], dx[k] * B);
+        s[i][k] = scan_update<T>(dt[k], an[i][k], s[i][k], dx[k] * B);
         y[k] = fmaf(s[i][k], C, y[k]);
       }
       store_v<float, V>(S + (size_t)(n0 + i) * p.I, s[i]);
@@ -194,16 +200,16 @@ __global__ void __launch_bounds__(ST_THREADS) scan_step_kernel(const ScanParams 
 // ---- portions ------------------------------------------------------------------------------------------------
 constexpr int SR_THREADS = 128;
 
-// decay exp(dt a) with `a` as scan_coef left it
+// scan_update with `a` as scan_coef left it (in a bf16 model the logarithm's base is 2)
 template <typename T> __device__ __forceinline__ float scan_coef(float a);
 template <> __device__ __forceinline__ float scan_coef<float>(float a) { return a; }
 template <> __device__ __forceinline__ float scan_coef<__nv_bfloat16>(float a) { return a * 1.44269504f; }
-template <typename T> __device__ __forceinline__ float scan_decay(float dt, float a);
-template <> __device__ __forceinline__ float scan_decay<float>(float dt, float a) { return expf(dt * a); }
-template <> __device__ __forceinline__ float scan_decay<__nv_bfloat16>(float dt, float a) {
+template <typename T> __device__ __forceinline__ float scan_update2(float dt, float a, float s, float b);
+template <> __device__ __forceinline__ float scan_update2<float>(float dt, float a, float s, float b) { return scan_update<float>(dt, a, s, b); }
+template <> __device__ __forceinline__ float scan_update2<__nv_bfloat16>(float dt, float a, float s, float b) {
   float e;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(dt * a));
-  return e;
+  return fmaf(e, s, b);
 }
 
 // grid (I / CH, S). Lane q of a channel's P lanes holds states q RPT .. q RPT + RPT - 1; TT tokens per tile.
@@ -284,7 +290,7 @@ __global__ void __launch_bounds__(SR_THREADS) scan_rows_kernel(const ScanParams 
       float y = 0.f;
 #pragma unroll
       for (int i = 0; i < RPT; ++i) {
-        s[i] = fmaf(scan_decay<T>(d, a[i]), s[i], x * B_s[j][q * RPT + i]);
+        s[i] = scan_update2<T>(d, a[i], s[i], x * B_s[j][q * RPT + i]);
         y = fmaf(s[i], C_s[j][q * RPT + i], y);
       }
 #pragma unroll

@@ -37,6 +37,8 @@ def forward_full(cfg: ModelConfig, w: ModelWeights, token_ids: torch.Tensor, cap
     """Full-sequence forward of ONE sequence (unsharded weights). Returns fp32 logits [T, V]."""
     if cfg.is_parallel:
         return _forward_parallel(cfg, w, token_ids, capture_hidden)
+    if cfg.is_prenorm:
+        return _forward_prenorm(cfg, w, token_ids, capture_hidden)
     if cfg.is_layered:
         return _forward_layered(cfg, w, token_ids, capture_hidden)
     T = token_ids.shape[0]
@@ -225,3 +227,91 @@ def _forward_parallel(cfg, w, token_ids, capture_hidden):
         if capture_hidden is not None:
             capture_hidden.append(x.clone())
     return norm(x, w.final_norm) @ w.lm_head.float().t()
+
+
+def _forward_prenorm(cfg, w, token_ids, capture_hidden):
+    """The same for pre-norm layers: attention by a full mask, the scan one token at a time, every expert over all tokens that chose it."""
+    from .parallel_layers import LayerLayout, SelectiveSpec, up8
+    T, eps = token_ids.shape[0], cfg.rms_norm_eps
+    unit = lambda v: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)      # noqa: E731
+    act = torch.nn.functional
+    x = w.embed[token_ids.long()].float()
+    pos = torch.arange(T, device=x.device)
+
+    def attention(a, aw, z, at):
+        H, G, M, D = a.heads, a.kv_heads, a.maps, a.dim
+        q, k, v = (z[:, at[n]:at[n] + rows] for n, rows in a.sections()[:3])
+        n = a.rot_dims
+        ang = pos.double()[:, None] * (a.rope_base ** (-torch.arange(0, n, 2, device=x.device).double() / max(n, 1)) / a.rope_factor)
+        c, s = ang.cos().float()[:, None], ang.sin().float()[:, None]
+
+        def turn(t):
+            if a.interleaved:
+                u, y = t[..., 0:n:2], t[..., 1:n:2]
+                r = torch.stack([u * c - y * s, y * c + u * s], dim=-1).flatten(-2)
+            else:
+                u, y = t[..., :n // 2], t[..., n // 2:n]
+                r = torch.cat([u * c - y * s, y * c + u * s], dim=-1)
+            t = torch.cat([r, t[..., n:]], dim=-1)
+            return unit(t) if a.unit else t
+        q = turn(q.reshape(T, H * M, D)).view(T, H, M, D)
+        k = turn(k.reshape(T, G * M, D)).view(T, G, M, D).repeat_interleave(H // G, dim=1)
+        v = v.reshape(T, G, a.vdim).repeat_interleave(H // G, dim=1)
+        back = pos[:, None] - pos[None, :]
+        seen = back >= 0
+        if a.chunk:
+            seen = seen & (pos[:, None] // a.chunk == pos[None, :] // a.chunk)
+        if a.window:
+            seen = seen & (back < a.window)
+        sc = (torch.einsum("qhmd,khmd->hmqk", q, k) * a.scale).masked_fill(~seen, float("-inf"))
+        if a.sink:
+            sc = torch.cat([sc, torch.zeros_like(sc[..., :1])], dim=-1)
+        o = torch.einsum("hmqk,khv->mqhv", torch.softmax(sc, dim=-1)[..., :T], v)
+        o = o[0] if M == 1 else unit(o[0] - aw.lam * o[1]) * (1.0 - a.diff)
+        o = o.reshape(T, -1)
+        return o * torch.sigmoid(z[:, at["g"]:at["g"] + a.out_width]) if a.gated else o
+
+    def scan(m, sw, z, at):
+        N = m.state
+        u = z[:, at["x"]:at["x"] + m.inner]
+        u = act.silu(sum(sw.conv[j] * act.pad(u, (0, 0, m.taps - 1 - j, 0))[:T] for j in range(m.taps)) + sw.conv_b)
+        p = u @ sw.w_x.float().t()
+        b0, c0 = up8(m.dt_rank), up8(m.dt_rank) + up8(N)
+        dt = act.softplus(p[:, :sw.w_dt.shape[1]] @ sw.w_dt.float().t() + sw.dt_bias)
+        S, ys = torch.zeros(N, m.inner, device=x.device), []
+        for t in range(T):
+            S = torch.exp(dt[t] * sw.neg_a) * S + (dt[t] * u[t]) * p[t, b0:b0 + N, None]
+            ys.append(p[t, c0:c0 + N] @ S + sw.skip * u[t])
+        return torch.stack(ys) * act.silu(z[:, at["z"]:at["z"] + m.inner])
+
+    def glu(h, w13, w2):
+        g, u = (h @ w13.float().t()).chunk(2, dim=1)
+        return (act.silu(g) * u) @ w2.float().t()
+
+    for sp, lw in zip(cfg.layers, w.layers):
+        lay, f = LayerLayout(sp, ff=False), sp.mlp
+        if sp.loop_pass is not None:
+            x = x + w.loop.step[sp.loop_pass]
+        z = torch.zeros(T, lay.width, device=x.device)
+        z[:, lay.in_first:] = (unit(x) * lw.norm1) @ lw.w_in.float().t()
+        sec = lay.parts[0]
+        o = scan(sp.mixer, lw.scan, z, sec.col) if isinstance(sp.mixer, SelectiveSpec) else attention(sp.mixer, lw.attn, z, sec.col)
+        x = x + act.pad(o, (0, lay.out_cols - o.shape[1])) @ lw.w_out.float().t()
+        if f is not None:
+            h = unit(x) * lw.norm2
+            s = h @ lw.router.float().t()
+            s = torch.sigmoid(s) if f.score == "sigmoid" else torch.softmax(s, dim=-1)
+            grouped = s.view(T, f.groups, -1)
+            best = grouped.topk(min(f.group_best, grouped.shape[-1]), dim=-1).values.sum(-1).topk(f.keep, dim=-1).indices
+            ok = torch.zeros(T, f.groups, dtype=torch.bool, device=x.device).scatter_(1, best, True).repeat_interleave(f.experts // f.groups, dim=1)
+            top, ids = s.masked_fill(~ok, -1.0).topk(f.top, dim=-1)
+            top = (top / (top.sum(-1, keepdim=True) + 1e-20) if f.renorm else top) * f.scale
+            y = glu(h, lw.shared13, lw.shared2) if f.shared_ff else torch.zeros_like(x)
+            for e in range(f.experts):
+                rows, slot = (ids == e).nonzero(as_tuple=True)
+                if rows.numel():
+                    y[rows] += top[rows, slot, None] * glu(h[rows], lw.w13[e], lw.w2[e])
+            x = x + y
+        if capture_hidden is not None:
+            capture_hidden.append(x.clone())
+    return (unit(x) * w.final_norm) @ w.lm_head.float().t()
