@@ -543,6 +543,30 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           if (et == 0) TS(4);
           if (n_pseg < 2) ps_u[n_pseg] = u;
           ++n_pseg;
+        } else if (!DUAL && p.out_f32 && p.residual != nullptr && p.gate == nullptr && p.relu2_cols == 0) {
+          // fp32 sum, usually in place: the residuals of 32 columns are on their way before the first sum is stored
+          const size_t first = (size_t)row0 * p.ldo + p.out_col0 + un.g * p.out_group_cols + f;
+          const float* res = (const float*)p.residual + first;
+          float* out = (float*)p.out + first;
+          for (int c0 = 0; c0 < n_tile; c0 += 32) {
+            if (c0 >= valid) break;
+            uint32_t v[32];
+            float rv[32];
+            if (f_ok) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) rv[j] = __ldcg(res + (size_t)min(c0 + j, valid - 1) * p.ldo);
+            }
+            tmem_ld16(t_acc + c0, v);
+            if (c0 + 16 < n_tile) tmem_ld16(t_acc + c0 + 16, v + 16);
+            tmem_ld_wait();
+            if (f_ok) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (c0 + j < valid) out[(size_t)(c0 + j) * p.ldo] = __uint_as_float(v[j]) + rv[j];
+            }
+          }
+          tc_fence_before();
+          mbar_arrive(smem_u32(&bar_tempty[b]));
         } else {
           for (int c0 = 0; c0 < n_tile; c0 += 16) {
             if (c0 >= valid) break;

@@ -73,15 +73,15 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ScanParams p, int
     const int pos = p.positions[t];
     if (pos < 0) continue;
     const int seq = DECODE ? t : p.seq_of_token[t], first = DECODE ? t : p.q_start[seq];
-    // the input j tokens before row t
+    int slot = taps > 1 ? p.slots[seq] : 0;
+    if (slot < 0 || slot >= p.num_slots) { report_status(p.status, ST_BAD_INDEX, slot); slot = 0; }
+    // the input j tokens before row t (loaded from the row itself where there is none)
     auto prev = [&](int j, float* v) {
+      const T* src = x + (size_t)t * p.x_ld + c;
+      if (pos >= j) src = t - j >= first ? src - (size_t)j * p.x_ld : (const T*)p.tail + ((size_t)slot * taps + (pos - j) % taps) * p.I + c;
+      load_v<T, V>(src, v);
 #pragma unroll
-      for (int k = 0; k < V; ++k) v[k] = 0.f;
-      if (pos < j) return;
-      if (t - j >= first) { load_v<T, V>(x + (size_t)(t - j) * p.x_ld + c, v); return; }
-      const int slot = p.slots[seq];
-      if (slot < 0 || slot >= p.num_slots) { report_status(p.status, ST_BAD_INDEX, slot); return; }
-      load_v<T, V>((const T*)p.tail + ((size_t)slot * taps + (pos - j) % taps) * p.I + c, v);
+      for (int k = 0; k < V; ++k) v[k] = pos >= j ? v[k] : 0.f;
     };
     float cur[V], a[V];
     load_v<T, V>(x + (size_t)t * p.x_ld + c, cur);
@@ -106,11 +106,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ScanParams p, int
         for (int k = 0; k < V; ++k) a[k] = fmaf(wj[k], j > 0 ? v[k] : cur[k], a[k]);
       }
     }
-    if (DECODE && taps > 1) {
-      const int slot = p.slots[seq];
-      if (slot < 0 || slot >= p.num_slots) report_status(p.status, ST_BAD_INDEX, slot);
-      else store_v<T, V>((T*)p.tail + ((size_t)slot * taps + pos % taps) * p.I + c, cur);
-    }
+    if (DECODE && taps > 1) store_v<T, V>((T*)p.tail + ((size_t)slot * taps + pos % taps) * p.I + c, cur);
 #pragma unroll
     for (int k = 0; k < V; ++k) a[k] = silu_act<T>(a[k]);
     store_v<T, V>((T*)p.xc + (size_t)t * p.I + c, a);
@@ -212,11 +208,13 @@ template <> __device__ __forceinline__ float scan_update2<__nv_bfloat16>(float d
   return fmaf(e, s, b);
 }
 
-// grid (I / CH, S). Lane q of a channel's P lanes holds states q RPT .. q RPT + RPT - 1; TT tokens per tile.
+// grid (I / CH, S). Lane q of a channel's P lanes holds states q RPT .. q RPT + RPT - 1; TT tokens per tile, four at a time: their decays
+// do not depend on one another, and the P lanes' sums of the four outputs are formed together (a lane ends up with one token's).
 template <typename T, int P, int RPT, int TT>
-__global__ void __launch_bounds__(SR_THREADS) scan_rows_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(SR_THREADS, 4) scan_rows_kernel(const ScanParams p) {
   constexpr int CH = SR_THREADS / P, NP = P * RPT, EL = TT * CH / SR_THREADS, BL = (TT * NP + SR_THREADS - 1) / SR_THREADS;
-  __shared__ float dt_s[TT][CH], dx_s[TT][CH], y_s[TT][CH];
+  constexpr int LD = TT + 4;
+  __shared__ __align__(16) float dt_s[CH][LD], dx_s[CH][LD], y_s[CH][LD];
   __shared__ __align__(16) float B_s[TT][NP], C_s[TT][NP];
   pdl_trigger();
   pdl_wait();
@@ -242,26 +240,24 @@ __global__ void __launch_bounds__(SR_THREADS) scan_rows_kernel(const ScanParams 
   const int lc = c0 + tid % CH;
   const bool lin = lc < p.I;
   const float bias = lin ? p.dt_bias[lc] : 0.f, skip = lin ? p.skip[lc] : 0.f;
-  float u[EL], nu[EL], nd[EL], z[EL], nb[BL], nc[BL];
+  // Loads go to clamped addresses and stay as they are until the next tile starts: all of a tile's are on their way together.
+  const int lcc = lin ? lc : p.I - 1, row_max = n_rows - 1;
+  float u[EL], nd[EL];
+  T nu[EL], nz[EL], z[EL], nb[BL], nc[BL];
   auto fetch = [&](int r0) {
 #pragma unroll
     for (int k = 0; k < EL; ++k) {
-      const int r = r0 + (tid + k * SR_THREADS) / CH;
-      nu[k] = nd[k] = 0.f;
-      if (lin && r < n_rows) {
-        nu[k] = to_f<T>(((const T*)p.xc)[(size_t)(t0 + r) * p.I + lc]);
-        nd[k] = p.dt[(size_t)(t0 + r) * p.I + lc];
-      }
+      const size_t t = t0 + min(r0 + tid / CH + k * P, row_max);
+      nu[k] = ((const T*)p.xc)[t * p.I + lcc];
+      nd[k] = p.dt[t * p.I + lcc];
+      nz[k] = ((const T*)p.z)[t * p.x_ld + lcc];
     }
 #pragma unroll
     for (int k = 0; k < BL; ++k) {
-      const int e = tid + k * SR_THREADS, r = r0 + e / NP, n = e % NP;
-      nb[k] = nc[k] = 0.f;
-      if (e < TT * NP && r < n_rows && n < p.N) {
-        const T* pr = (const T*)p.proj + (size_t)(t0 + r) * p.proj_ld;
-        nb[k] = to_f<T>(pr[p.b_col + n]);
-        nc[k] = to_f<T>(pr[p.c_col + n]);
-      }
+      const int e = tid + k * SR_THREADS, n = min(e % NP, p.N - 1);
+      const T* pr = (const T*)p.proj + (size_t)(t0 + min(r0 + e / NP, row_max)) * p.proj_ld;
+      nb[k] = pr[p.b_col + n];
+      nc[k] = pr[p.c_col + n];
     }
   };
   fetch(0);
@@ -270,39 +266,64 @@ __global__ void __launch_bounds__(SR_THREADS) scan_rows_kernel(const ScanParams 
 #pragma unroll
     for (int k = 0; k < EL; ++k) {
       const int e = tid + k * SR_THREADS;
-      u[k] = nu[k];
-      const float d = softplus_f(nd[k] + bias);
-      dt_s[e / CH][e % CH] = d;
-      dx_s[e / CH][e % CH] = d * u[k];
-      const int r = r0 + e / CH;
-      z[k] = lin && r < n_rows ? to_f<T>(((const T*)p.z)[(size_t)(t0 + r) * p.x_ld + lc]) : 0.f;
+      u[k] = to_f<T>(nu[k]);
+      z[k] = nz[k];
+      const float d = r0 + e / CH < n_rows ? softplus_f(nd[k] + bias) : 0.f;      // a step of size zero past the end
+      dt_s[e % CH][e / CH] = d;
+      dx_s[e % CH][e / CH] = d * u[k];
     }
 #pragma unroll
     for (int k = 0; k < BL; ++k) {
       const int e = tid + k * SR_THREADS;
-      if (e < TT * NP) { B_s[e / NP][e % NP] = nb[k]; C_s[e / NP][e % NP] = nc[k]; }
+      const bool have = e % NP < p.N;      // states past N take part with zeros
+      if (TT * NP % SR_THREADS == 0 || e < TT * NP) {
+        B_s[e / NP][e % NP] = have ? to_f<T>(nb[k]) : 0.f;
+        C_s[e / NP][e % NP] = have ? to_f<T>(nc[k]) : 0.f;
+      }
     }
     __syncthreads();
     if (r0 + TT < n_rows) fetch(r0 + TT);
-#pragma unroll 4
-    for (int j = 0; j < cnt; ++j) {
-      const float d = dt_s[j][ch], x = dx_s[j][ch];
-      float y = 0.f;
+    for (int j = 0; j < cnt; j += 4) {
+      const float4 d4 = *reinterpret_cast<const float4*>(&dt_s[ch][j]), x4 = *reinterpret_cast<const float4*>(&dx_s[ch][j]);
+      const float d[4] = {d4.x, d4.y, d4.z, d4.w}, x[4] = {x4.x, x4.y, x4.z, x4.w};
+      float y[4];
 #pragma unroll
-      for (int i = 0; i < RPT; ++i) {
-        s[i] = scan_update2<T>(d, a[i], s[i], x * B_s[j][q * RPT + i]);
-        y = fmaf(s[i], C_s[j][q * RPT + i], y);
+      for (int h = 0; h < 4; ++h) {
+        y[h] = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPT; i += 4) {
+          const float4 B = *reinterpret_cast<const float4*>(&B_s[j + h][q * RPT + i]), C = *reinterpret_cast<const float4*>(&C_s[j + h][q * RPT + i]);
+          s[i] = scan_update2<T>(d[h], a[i], s[i], x[h] * B.x);
+          s[i + 1] = scan_update2<T>(d[h], a[i + 1], s[i + 1], x[h] * B.y);
+          s[i + 2] = scan_update2<T>(d[h], a[i + 2], s[i + 2], x[h] * B.z);
+          s[i + 3] = scan_update2<T>(d[h], a[i + 3], s[i + 3], x[h] * B.w);
+          y[h] = fmaf(s[i], C.x, fmaf(s[i + 1], C.y, y[h]));
+          y[h] = fmaf(s[i + 2], C.z, fmaf(s[i + 3], C.w, y[h]));
+        }
       }
+      if (P == 1) {
+        *reinterpret_cast<float4*>(&y_s[ch][j]) = make_float4(y[0], y[1], y[2], y[3]);
+      } else {
+        const bool b0 = q & 1, b1 = q & 2;
+        float v = b0 ? y[2] : y[0], w = b0 ? y[3] : y[1];
+        v += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
+        w += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
+        if (P == 2) {
+          *reinterpret_cast<float2*>(&y_s[ch][j + 2 * b0]) = make_float2(v, w);
+        } else {
+          float r = (b1 ? w : v) + __shfl_xor_sync(0xffffffffu, b1 ? v : w, 2);
 #pragma unroll
-      for (int o = 1; o < P; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (q == 0) y_s[j][ch] = y;
+          for (int o = 4; o < P; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+          if (P == 4 || q < 4) y_s[ch][j + 2 * b0 + b1] = r;
+        }
+      }
     }
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < EL; ++k) {
       const int e = tid + k * SR_THREADS, r = r0 + e / CH;
       if (lin && r < n_rows)
-        ((T*)p.out)[(size_t)(t0 + r) * p.out_ld + lc] = from_f<T>((y_s[e / CH][e % CH] + skip * u[k]) * silu_act<T>(z[k]));
+        ((T*)p.out)[(size_t)(t0 + r) * p.out_ld + lc] = from_f<T>((y_s[e % CH][e / CH] + skip * u[k]) * silu_act<T>(to_f<T>(z[k])));
     }
   }
 #pragma unroll

@@ -105,8 +105,13 @@ def _round_up(x, m):
     return (x + m - 1) // m * m
 
 
-def pick_n_tile(rows_hint: int, dual: bool) -> int:
+def pick_n_tile(rows_hint: int, dual: bool, features: int = 0) -> int:
+    """Tokens of a tile. With many rows and few features (given with `features`) the tiles shrink until every SM has one."""
     cap = 128 if dual else 256
+    if features and rows_hint > 256:
+        feature_tiles, sms = (features + 127) // 128, 148
+        if feature_tiles * ((rows_hint + cap - 1) // cap) < sms:
+            cap = max(32, min(cap, _round_up((rows_hint * feature_tiles + sms - 1) // sms, 16)))
     return max(16, min(cap, _round_up(max(rows_hint, 1), 16)))
 
 
@@ -243,7 +248,7 @@ def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False,
     if T == 0:
         return out
     wv, _, packed = _wview(w)
-    p = _base_params(x, wv, out, F, K, n_tile or pick_n_tile(T, False), 0)
+    p = _base_params(x, wv, out, F, K, n_tile or pick_n_tile(T, False, F), 0)
     p.w_rows_per_group, p.w_packed, p.out_f32, p.relu2_cols = F, packed, 1 if out_f32 else 0, int(relu2_cols)
     if x.stride(0) != K:
         p.x_ld = x.stride(0)
