@@ -200,12 +200,26 @@ constexpr int SR_THREADS = 128;
 template <typename T> __device__ __forceinline__ float scan_coef(float a);
 template <> __device__ __forceinline__ float scan_coef<float>(float a) { return a; }
 template <> __device__ __forceinline__ float scan_coef<__nv_bfloat16>(float a) { return a * 1.44269504f; }
-template <typename T> __device__ __forceinline__ float scan_update2(float dt, float a, float s, float b);
-template <> __device__ __forceinline__ float scan_update2<float>(float dt, float a, float s, float b) { return scan_update<float>(dt, a, s, b); }
-template <> __device__ __forceinline__ float scan_update2<__nv_bfloat16>(float dt, float a, float s, float b) {
-  float e;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(dt * a));
-  return fmaf(e, s, b);
+template <typename T> __device__ __forceinline__ float scan_size(float z);
+template <> __device__ __forceinline__ float scan_size<float>(float z) { return softplus_f(z); }
+template <> __device__ __forceinline__ float scan_size<__nv_bfloat16>(float z) { return softplus_series(z); }
+// two of them, and two products summed, as pairs (one instruction each where the model is bf16)
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float x, float y) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y)); return r; }
+__device__ __forceinline__ float2 unpack2(f32x2 v) { float2 r; asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v)); return r; }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) { f32x2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) { f32x2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+template <typename T> __device__ __forceinline__ f32x2 scan_update2(f32x2 dt, f32x2 a, f32x2 s, f32x2 b);
+template <> __device__ __forceinline__ f32x2 scan_update2<float>(f32x2 dt, f32x2 a, f32x2 s, f32x2 b) {
+  const float2 d = unpack2(dt), aa = unpack2(a), ss = unpack2(s), bb = unpack2(b);
+  return pack2(scan_update<float>(d.x, aa.x, ss.x, bb.x), scan_update<float>(d.y, aa.y, ss.y, bb.y));
+}
+template <> __device__ __forceinline__ f32x2 scan_update2<__nv_bfloat16>(f32x2 dt, f32x2 a, f32x2 s, f32x2 b) {
+  const float2 x = unpack2(mul2(dt, a));
+  float e0, e1;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(x.x));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e1) : "f"(x.y));
+  return fma2(pack2(e0, e1), s, b);
 }
 
 // grid (I / CH, S). Lane q of a channel's P lanes holds states q RPT .. q RPT + RPT - 1; TT tokens per tile, four at a time: their decays
@@ -228,13 +242,19 @@ __global__ void __launch_bounds__(SR_THREADS, 4) scan_rows_kernel(const ScanPara
   const int q = tid % P, ch = tid / P, c = c0 + ch;
   const bool in = c < p.I;
   float* S = p.state + (size_t)slot * p.N * p.I + c;
-  float s[RPT], a[RPT];
+  f32x2 s[RPT / 2], a[RPT / 2];      // pairs of states
 #pragma unroll
-  for (int i = 0; i < RPT; ++i) {
-    const int n = q * RPT + i;
-    const bool have = in && n < p.N;
-    s[i] = have && pos0 > 0 ? S[(size_t)n * p.I] : 0.f;
-    a[i] = have ? scan_coef<T>(p.neg_a[(size_t)n * p.I + c]) : 0.f;
+  for (int i = 0; i < RPT; i += 2) {
+    float sv[2], av[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int n = q * RPT + i + k;
+      const bool have = in && n < p.N;
+      sv[k] = have && pos0 > 0 ? S[(size_t)n * p.I] : 0.f;
+      av[k] = have ? scan_coef<T>(p.neg_a[(size_t)n * p.I + c]) : 0.f;
+    }
+    s[i / 2] = pack2(sv[0], sv[1]);
+    a[i / 2] = pack2(av[0], av[1]);
   }
   // elements e of a tile that this thread moves: token e / CH, channel e % CH with e = tid + 128 k
   const int lc = c0 + tid % CH;
@@ -268,7 +288,7 @@ __global__ void __launch_bounds__(SR_THREADS, 4) scan_rows_kernel(const ScanPara
       const int e = tid + k * SR_THREADS;
       u[k] = to_f<T>(nu[k]);
       z[k] = nz[k];
-      const float d = r0 + e / CH < n_rows ? softplus_f(nd[k] + bias) : 0.f;      // a step of size zero past the end
+      const float d = r0 + e / CH < n_rows ? scan_size<T>(nd[k] + bias) : 0.f;      // a step of size zero past the end
       dt_s[e % CH][e / CH] = d;
       dx_s[e % CH][e / CH] = d * u[k];
     }
@@ -289,17 +309,17 @@ __global__ void __launch_bounds__(SR_THREADS, 4) scan_rows_kernel(const ScanPara
       float y[4];
 #pragma unroll
       for (int h = 0; h < 4; ++h) {
-        y[h] = 0.f;
+        const f32x2 d2 = pack2(d[h], d[h]), x2 = pack2(x[h], x[h]);
+        f32x2 y2 = pack2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < RPT; i += 4) {
-          const float4 B = *reinterpret_cast<const float4*>(&B_s[j + h][q * RPT + i]), C = *reinterpret_cast<const float4*>(&C_s[j + h][q * RPT + i]);
-          s[i] = scan_update2<T>(d[h], a[i], s[i], x[h] * B.x);
-          s[i + 1] = scan_update2<T>(d[h], a[i + 1], s[i + 1], x[h] * B.y);
-          s[i + 2] = scan_update2<T>(d[h], a[i + 2], s[i + 2], x[h] * B.z);
-          s[i + 3] = scan_update2<T>(d[h], a[i + 3], s[i + 3], x[h] * B.w);
-          y[h] = fmaf(s[i], C.x, fmaf(s[i + 1], C.y, y[h]));
-          y[h] = fmaf(s[i + 2], C.z, fmaf(s[i + 3], C.w, y[h]));
+          const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(&B_s[j + h][q * RPT + i]), C = *reinterpret_cast<const ulonglong2*>(&C_s[j + h][q * RPT + i]);
+          s[i / 2] = scan_update2<T>(d2, a[i / 2], s[i / 2], mul2(x2, B.x));
+          s[i / 2 + 1] = scan_update2<T>(d2, a[i / 2 + 1], s[i / 2 + 1], mul2(x2, B.y));
+          y2 = fma2(s[i / 2 + 1], C.y, fma2(s[i / 2], C.x, y2));
         }
+        const float2 yv = unpack2(y2);
+        y[h] = yv.x + yv.y;
       }
       if (P == 1) {
         *reinterpret_cast<float4*>(&y_s[ch][j]) = make_float4(y[0], y[1], y[2], y[3]);
@@ -327,9 +347,11 @@ __global__ void __launch_bounds__(SR_THREADS, 4) scan_rows_kernel(const ScanPara
     }
   }
 #pragma unroll
-  for (int i = 0; i < RPT; ++i) {
+  for (int i = 0; i < RPT; i += 2) {
     const int n = q * RPT + i;
-    if (in && n < p.N) S[(size_t)n * p.I] = s[i];
+    const float2 v = unpack2(s[i / 2]);
+    if (in && n < p.N) S[(size_t)n * p.I] = v.x;
+    if (in && n + 1 < p.N) S[(size_t)(n + 1) * p.I] = v.y;
   }
   if (p.taps > 1) {      // every reader of the old inputs (short_conv) is done
     const int keep = min(p.taps - 1, n_rows);
