@@ -31,10 +31,10 @@ CORE_LIB_STEM = "_skein_core"
 
 # Kernel sources of architectures that need only some of them (the others take the whole library).
 ARCH_SOURCES = {
-    "Zarorax": ("attn_latent_decode", "attn_latent_prefill", "gemm_simt", "gemm_ws", "latent", "postnorm", "rope_kv", "router", "sample"),
-    "Sikalorn": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_ws", "parallel_layer", "postnorm", "recurrent",
+    "Zarorax": ("attn_latent_decode", "attn_latent_prefill", "gemm_simt", "gemm_small", "gemm_ws", "latent", "postnorm", "rope_kv", "router", "sample"),
+    "Sikalorn": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_small", "gemm_ws", "parallel_layer", "postnorm", "recurrent",
                  "recurrent_tc", "rope_kv", "sample"),
-    "Barorax": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_ws", "postnorm", "prenorm", "rope_kv", "router",
+    "Barorax": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_small", "gemm_ws", "postnorm", "prenorm", "rope_kv", "router",
                 "sample", "selective"),
 }
 # Sources compiled without fast-math: their exponentials, logarithms and tanh keep the accuracy of 32-bit.

@@ -163,6 +163,7 @@ def lib():
     _sig(L, "skein_copy_pages", i32, [vp, vp, vp, vp, i32, i64, vp])
     _sig(L, "skein_wait_flag", i32, [vp, i32, i32, vp, vp])
     _sig(L, "skein_gemm_simt", i32, [C.POINTER(GemmParams), i32, i32, vp])
+    _sig(L, "skein_gemm_small", i32, [vp, i64, vp, vp, i64, vp, i32, i32, i32, i32, vp])
     _sig(L, "skein_embed_f32", i32, [vp, vp, vp, i32, i32, i32, i32, vp])
     _sig(L, "skein_conv_input", i32, [vp, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp])
     _sig(L, "skein_post_norm", i32, [vp, vp, vp, vp, vp, vp, vp, vp, f32, f32, i32, i32, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp])

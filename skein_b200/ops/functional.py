@@ -223,6 +223,19 @@ def tc_gemm_ok(x, K) -> bool:
     return x.dtype == torch.bfloat16 and K % 8 == 0
 
 
+def _tuned(p) -> bool:
+    """Whether the kernel-configuration cache holds a measured configuration for this product."""
+    cache = tuning.active()
+    return cache is not None and cache.get("gemm", tuning.gemm_shape_key(p.mode, p.G, p.F, p.K, p.x_rows)) is not None
+
+
+def small_gemm_ok(T: int, F: int, K: int) -> bool:
+    """Whether a decode step's product is quicker on the small kernel (csrc/kernels/gemm_small.cu) than on the streaming one. Measured at
+    64 rows: 160 x 4096 6.9 against 11.1 us, 512 x 512 6.5 / 10.1, 1024 x 1024 7.5 / 10.0, 2048 x 2048 9.5 / 10.8; with short rows
+    (4096 x 128) or more weights the streaming kernel is as quick or quicker."""
+    return T <= 64 and F <= 2048 and K >= 512 and F * K <= 2048 * 2048
+
+
 def simt_launch(p: "_lib.GemmParams", x, max_rows: int, what: str):
     _lib.check(_lib.lib().skein_gemm_simt(C.byref(p), 1 if x.dtype == torch.float32 else 0, int(max_rows), _lib.stream_ptr()), what)
     _lib.count_launch()
@@ -254,6 +267,12 @@ def linear(x, w, out=None, residual=None, n_tile=None, _cfg=None, out_f32=False,
         p.x_ld = x.stride(0)
     if residual is not None:
         p.residual = residual.data_ptr()
+    if (_cfg is None and n_tile is None and relu2_cols == 0 and not packed and small_gemm_ok(T, F, K) and tc_gemm_ok(x, K) and x.stride(0) % 8 == 0
+            and x.data_ptr() % 16 == 0 and w.is_contiguous() and not _tuned(p) and hasattr(_lib.lib(), "skein_gemm_small")):
+        _lib.check(_lib.lib().skein_gemm_small(x.data_ptr(), x.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), _lib.ptr(residual), T, F, K,
+                                               int(out_f32), _lib.stream_ptr()), "linear")
+        _lib.count_launch()
+        return out
     if tc_gemm_ok(x, K) and p.x_ld % 8 == 0 and x.data_ptr() % 16 == 0:
         _check_bf16(x)
         _gemm_launch(p, "linear", _cfg)

@@ -58,6 +58,26 @@ def test_add_norm(T, C, top, dtype):
             close(act, wact, dtype, 0.6)
 
 
+@pytest.mark.parametrize("T,F,K", [(1, 32, 512), (64, 160, 4096), (17, 161, 520), (64, 2048, 2048), (50, 33, 1000), (63, 288, 8192)])
+def test_small_product(T, F, K):
+    """Few rows and few weights: strided rows in and out, 16- and 32-bit sums, in place on the residual, the same result every time."""
+    assert ops.functional.small_gemm_ok(T, F, K)
+    x, w = rnd(T, K + 16)[:, 8:8 + K], rnd(F, K, scale=K ** -0.5)
+    gx = rnd(T, K + 16).to(DEV)[:, 8:8 + K]
+    wide = torch.full((T, F + 8), 7.0, dtype=BF, device=DEV)
+    ops.linear(gx, w.to(DEV), out=wide[:, :F])
+    close(wide[:, :F], ref.linear(x, w), BF)
+    assert (wide[:, F:] == 7).all()
+    r = rnd(T, F, dtype=F32, scale=4)
+    a, b = r.to(DEV), r.to(DEV)
+    for o in (a, b):
+        ops.linear(gx, w.to(DEV), out=o, residual=o, out_f32=True)
+    close(a, ref.linear(x, w, r, out_f32=True), F32)
+    assert torch.equal(a, b)
+    rb = rnd(T, F, seed=3)
+    close(ops.linear(gx, w.to(DEV), residual=rb.to(DEV)), ref.linear(x, w, rb), BF)
+
+
 RULES = [moe(experts=12, top=3, groups=4, keep=2), moe(experts=64, top=6, groups=8, keep=4), moe(experts=5, top=2, groups=1, keep=1, scale=1.0),
          moe(experts=8, top=4, groups=8, keep=5), moe(experts=128, top=12, groups=64, keep=9), moe(experts=200, top=7, groups=40, keep=3),
          RoutedFFSpec(8, 7.0, 16, 4, 4, 2), RoutedFFSpec(8, None, 16, 4, 4, 2, group_best=2, renorm=True)]
