@@ -54,7 +54,7 @@ class OpProfiler:
 
     def __enter__(self):
         from .. import ops
-        from ..ops import fp8, functional, latent, parallel, recurrent
+        from ..ops import fp8, functional, latent, parallel, prenorm, recurrent, selective
         names = ("linear", "swiglu_linear", "grouped_linear", "linear_push", "reduce_residual_rmsnorm", "reduce_norm_route",
                  "rmsnorm", "rope_kv_append", "attn_decode", "attn_decode_rope", "attn_prefill", "router_topk", "route",
                  "router_plan", "gather_rows", "embed", "sample_argmax", "sample", "quant_fp8_block128", "advance_decode_state")
@@ -65,10 +65,14 @@ class OpProfiler:
         for n in ("embed_f32", "conv_input", "post_norm", "post_norm_route", "route_grouped", "poly_norm", "latent_append", "head_linear",
                   "latent_attn_rows", "latent_attn_prefill", "latent_gather", "rope_rows"):
             self._patch(latent, n, "latent." + n)
-        for n in ("residual_tanh", "gated_norm", "window_append", "window_attn"):
+        for n in ("residual_tanh", "gated_norm", "window_append", "head_append", "window_attn"):
             self._patch(parallel, n, "parallel." + n)
         for n in ("rec_step", "rec_chunk"):
             self._patch(recurrent, n, "recurrent." + n)
+        for n in ("add_norm", "norm_route", "route"):
+            self._patch(prenorm, n, "prenorm." + n)
+        for n in ("short_conv", "scan"):
+            self._patch(selective, n, "selective." + n)
         for n in ("linear", "grouped_linear", "linear_publish"):
             self._patch(fp8, n, "fp8." + n)
         for obj in self.extra_objects:
