@@ -166,7 +166,7 @@ inline uint64_t layer_flops(const Layer& l, const ModelMeta& meta, const Workloa
     case LayerKind::Embedding: return b * s * l.hidden;
     case LayerKind::RmsNorm: return 5 * b * s * l.hidden;
     case LayerKind::Attention: {
-      if (l.parallel) {      // the projections, the attention over its window, read-out and update of the state
+      if (l.parallel && l.kv_rank == 0) {      // the projections, the attention over its window, read-out and update of the state
         uint64_t w = l.shared_elems;
         for (auto& p : l.params) w += p.numel();
         uint64_t f = 2 * b * s * w + 6 * b * s * l.state_elems;
@@ -185,7 +185,7 @@ inline uint64_t layer_flops(const Layer& l, const ModelMeta& meta, const Workloa
       const uint64_t softmax = 3 * b * l.num_heads * s * k;
       return qkvo + scores + softmax + scores;
     }
-    case LayerKind::Mlp: return (l.activation == "silu" ? 6 : 4) * b * s * l.hidden * l.intermediate;   // two or (ungated) one projections up, one down
+    case LayerKind::Mlp: return (l.activation == "silu" || l.activation == "clamped_glu" ? 6 : 4) * b * s * l.hidden * l.intermediate;   // two or (ungated) one projections up, one down
     case LayerKind::Moe: return 2 * b * s * l.hidden * l.num_experts + 6 * b * s * l.hidden * (l.top_k * l.intermediate + l.always_ff);
     case LayerKind::Lmhead: return 2 * b * s * l.vocab * l.hidden;
   }
@@ -283,7 +283,8 @@ inline double block_compute_time(size_t block, const Graph& ir, Dtype wd, Dtype 
 inline uint32_t kernels_per_layer(const Layer& l) {
   switch (l.kind) {
     case LayerKind::Attention:
-      if (l.parallel) return 3 + (l.kv_elems > 0 ? 2 : 0) + (l.state_elems > 0 ? 2 : 0) + (l.opens_pass && !l.selective ? 2 : 0) + (l.selective ? 2 : 0);  // in, out, sum + norm; append, attention; step, norm
+      if (l.parallel && l.kv_rank > 0) return 7;      // norm, input projection, append, absorb, attention, values, product back
+      if (l.parallel) return 3 + (l.bottlenecks ? 1 : 0) + (l.kv_elems > 0 ? 2 : 0) + (l.state_elems > 0 ? 2 : 0) + (l.opens_pass && !l.selective ? 2 : 0) + (l.selective ? 2 : 0);  // in, out, sum + norm; append, attention; step, norm (products behind bottlenecks, step)
       return l.kv_rank > 0 ? (l.q_rank > 0 ? 8 : 7) : 4;  // latent: input projection, append, (q up,) absorb, attention, values, o_proj, norm; qkv GEMM, RoPE + KV append + attention, o_proj GEMM, reduce + norm (+ router)
     case LayerKind::Mlp: return l.activation == "relu2" ? 0 : 3;   // (of a parallel layer: inside the mixer's two products)        // gate/up GEMM (SwiGLU epilogue), down GEMM, reduce+norm
     case LayerKind::Moe: return l.always_ff > 0 ? 5 : 3;        // grouped gate/up (gathers its rows), grouped down, combine + norm

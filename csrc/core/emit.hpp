@@ -217,19 +217,24 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
       continue;
     }
     if (ir.meta.prenorm) {
-      // norm, one product in, the mixer, one product out; norm, routed feed-forward
+      // norm, one product in, the mixer, one product out; norm, feed-forward
       std::vector<std::string> ops;
-      bool always = false;
+      bool always = false, dense = false;
       for (auto& l : ir.layers)
         if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Attention) {
           if (l.opens_pass) ops.push_back("loop_step");
-          for (const char* o : {"pre_norm1", "mixer_in"}) ops.push_back(o);
-          if (l.kv_elems > 0) for (const char* o : {"window_append", "window_attention"}) ops.push_back(o);
+          for (const char* o : {ir.meta.shifted ? "depth_shift_norm" : "pre_norm1", "mixer_in"}) ops.push_back(o);
+          if (l.kv_rank > 0) for (const char* o : {"latent_append", "latent_attention"}) ops.push_back(o);
+          else if (l.kv_elems > 0) for (const char* o : {"window_append", "window_attention"}) ops.push_back(o);
           if (l.selective) for (const char* o : {"short_conv", "scan_inputs", "selective_scan"}) ops.push_back(o);
+          if (l.bottlenecks) for (const char* o : {"recurrence_inputs", "recurrence", "gated_norm"}) ops.push_back(o);
           ops.push_back("mixer_out");
         } else if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Moe) {
           always = l.always_ff > 0;
+        } else if (l.block_idx && *l.block_idx == b && l.kind == LayerKind::Mlp) {
+          dense = true;
         }
+      if (dense) for (const char* o : {"group_norm2", "clamped_gate_up", "clamped_down"}) ops.push_back(o);
       if (moe) {
         for (const char* o : {"pre_norm2", "score_router"}) ops.push_back(o);
         if (always) for (const char* o : {"shared_gate_up", "shared_down"}) ops.push_back(o);
@@ -269,7 +274,7 @@ inline LoweredDevice lower_device(const Plan& plan, const Graph& ir, size_t devi
     if (pl.tp > 1) cut("ring_allreduce", handoff_collective_ffn_out(b), pl.tp_group(device));
   }
   if (stage == pl.pp - 1) {
-    cur.ops.insert(cur.ops.end(), {ir.meta.parallel ? "final_tanh_norm" : ir.meta.prenorm ? "final_rms_norm" : ir.meta.layered ? "final_scalar_norm" : "norm", "lm_head", "sample"});
+    cur.ops.insert(cur.ops.end(), {ir.meta.parallel ? "final_tanh_norm" : ir.meta.shifted ? "final_depth_norm" : ir.meta.prenorm ? "final_rms_norm" : ir.meta.layered ? "final_scalar_norm" : "norm", "lm_head", "sample"});
     if (pl.tp > 1) cut("allgather", "logit_candidates", pl.tp_group(device));
     cur.outputs.push_back(handoff_logits());
   } else {

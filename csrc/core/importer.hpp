@@ -285,13 +285,17 @@ inline Graph import_parallel(const Json& cfg) {
   return g;
 }
 
-// A design of pre-norm layers with an fp32 stream (Barorax): differential attention, attention inside chunks, selective scans; routed
-// experts with one that runs for every token; a range of layers that may run several times. One block per run; the runs after a
-// layer's first own no parameters.
+// A design of pre-norm layers with an fp32 stream. One block per run of a layer; the runs after a layer's first own no parameters.
+//   Barorax   differential attention, attention inside chunks, selective scans; routed experts with one that runs for every token; a
+//             range of layers that may run several times
+//   Derusun   latent attention, attention over a window that keeps the first tokens, delta rules with a decay per key channel; clamped
+//             gated units; a token shift in front of every mixer (the last normed row is part of a sequence's state) and an average over
+//             depth behind every layer
 inline Graph import_prenorm(const Json& cfg) {
   ModelMeta m;
   m.architecture = cfg.at("architecture").as_string();
   m.layered = m.prenorm = true;
+  m.shifted = m.architecture == "Derusun";
   m.hidden = cfg_usize(cfg, "width");
   m.vocab = cfg_usize(cfg, "vocab");
   m.max_position = cfg.has("max_position_embeddings") && !cfg.at("max_position_embeddings").is_null() ? cfg_usize(cfg, "max_position_embeddings") : 131072;
@@ -330,7 +334,72 @@ inline Graph import_prenorm(const Json& cfg) {
     a.parallel = true;
     const Json& mx = d.at("mixer");
     auto param = [&](const std::string& n, std::vector<uint64_t> shape) { ps.push_back({q + n, std::move(shape), Dtype::Bf16}); };
-    if (type == "attention" || type == "attention_2") {
+    auto heads = [&](uint64_t H, uint64_t K, uint64_t D, uint64_t V) {
+      a.num_heads = H; a.num_kv_heads = K; a.head_dim = D; a.v_dim = V;
+      m.num_attention_heads = std::max<size_t>(m.num_attention_heads, H);
+      m.head_dim = std::max<size_t>(m.head_dim, D);
+    };
+    if (m.shifted) {
+      const uint64_t H = cfg_usize(mx, "heads"), D = cfg_usize(mx, "dim"), V = cfg_usize(mx, "vdim");
+      if (type == "latent_attention") {
+        const uint64_t R = cfg_usize(mx, "rot_dim"), K = cfg_usize(mx, "kv_rank");
+        param("q", {H * (D + R), C});
+        param("dkv", {K + R, C});
+        param("dkv.norm", {K});
+        param("uk", {H * D, K});
+        param("uv", {H * V, K});
+        param("sink", {H});
+        heads(H, 1, D, V);
+        a.kv_rank = K; a.rot_dim = R; a.kv_elems = K + R;
+        a.rope_theta = mx.at("rot").at("base").as_double();
+        m.rope_theta = a.rope_theta;
+      } else if (type == "attention") {
+        const uint64_t K = cfg_usize(mx, "kv_heads");
+        param("q", {H * D, C});
+        param("k", {K * D, C});
+        param("v", {K * V, C});
+        param("q.b", {H * D});
+        param("k.b", {K * D});
+        param("v.b", {K * V});
+        param("q.norm", {D});
+        param("k.norm", {D});
+        if (const Json* vm = mx.find("v_mix"); vm && !vm->is_null() && vm->as_bool()) param("vmix", {});
+        param("sink", {H});
+        heads(H, K, D, V);
+        a.kv_elems = K * (D + V);
+        if (const Json* w = mx.find("mask"); w && !w->is_null() && w->has("size") && !w->at("size").is_null() && cfg_usize(*w, "size") > 0)
+          a.window = cfg_usize(*w, "size") + (w->has("keep_first") && !w->at("keep_first").is_null() ? cfg_usize(*w, "keep_first") : 0);
+      } else if (type == "channel_delta") {
+        const uint64_t G = cfg_usize(mx, "kv_heads"), taps = cfg_usize(mx, "conv"), channels = H * V + 2 * G * D;
+        auto rank = [&](const char* n) { return mx.has(n) && !mx.at(n).is_null() ? (uint64_t)cfg_usize(mx, n) : D; };
+        const uint64_t RA = rank("decay_rank"), RG = rank("gate_rank");
+        param("q", {G * D, C});
+        param("k", {G * D, C});
+        param("v", {H * V, C});
+        param("b", {H, C});
+        param("a1", {RA, C});
+        param("g1", {RG, C});
+        param("q.conv", {G * D, taps});
+        param("k.conv", {G * D, taps});
+        param("v.conv", {H * V, taps});
+        param("A_log", {H});
+        param("norm", {V});
+        param("a2", {H * D, RA});
+        param("dt_bias", {H * D});
+        param("g2", {H * V, RG});
+        heads(H, G, D, V);
+        a.bottlenecks = true;
+        a.conv_taps = taps;
+        a.state_elems = H * D * V;
+        a.state_bytes = 4 * a.state_elems + (taps > 1 ? 2 * taps * channels : 0);
+      } else {
+        throw ImportError("layer " + std::to_string(i) + ": mixer type `" + type + "` is not supported");
+      }
+      param("o", {C, H * V});
+      ps.push_back({p + "shift", {C}, Dtype::Bf16});
+      ps.push_back({p + "dwa", {i + 2}, Dtype::Bf16});
+      a.state_bytes += 4 * C;
+    } else if (type == "attention" || type == "attention_2") {
       const bool differential = type == "attention";
       const uint64_t H = cfg_usize(mx, "heads"), K = cfg_usize(mx, "kv_heads"), D = cfg_usize(mx, "dim"), V = cfg_usize(mx, "vdim"), M = differential ? 2 : 1;
       param("q", {H * M * D, C});
@@ -376,10 +445,20 @@ inline Graph import_prenorm(const Json& cfg) {
     if (shared) a.shared_elems = elems(ps); else a.params = ps;
     if (!d.has("mlp") || d.at("mlp").is_null()) continue;
     const Json& ml = d.at("mlp");
-    if (ml.at("kind").as_string() != "moe") throw ImportError("layer " + std::to_string(i) + ": feed-forward kind `" + ml.at("kind").as_string() + "` is not supported");
+    if (ml.at("kind").as_string() != (m.shifted ? "dense" : "moe"))
+      throw ImportError("layer " + std::to_string(i) + ": feed-forward kind `" + ml.at("kind").as_string() + "` is not supported");
     {
       Layer& n2 = add(LayerKind::RmsNorm, b, "norm2");
       if (!shared) n2.params.push_back({p + "norm2", {C}, Dtype::Bf16});
+    }
+    if (m.shifted) {
+      const uint64_t F = cfg_usize(ml, "ff");
+      Layer& f = add(LayerKind::Mlp, b, "mlp");
+      f.intermediate = F;
+      f.activation = "clamped_glu";
+      f.params = {{p + "mlp.gate", {F, C}, Dtype::Bf16}, {p + "mlp.up", {F, C}, Dtype::Bf16}, {p + "mlp.down", {C, F}, Dtype::Bf16}};
+      m.intermediate = std::max<size_t>(m.intermediate, F);
+      continue;
     }
     const uint64_t F = cfg_usize(ml.at("expert"), "ff"), E = cfg_usize(ml.at("router"), "experts");
     ps.clear();
@@ -412,7 +491,7 @@ inline Graph import_model(const Json& cfg) {
   if (const Json* a = cfg.find("architecture"); a && !a->is_null()) {
     if (a->as_string() == "Zarorax") return import_layered(cfg);
     if (a->as_string() == "Sikalorn") return import_parallel(cfg);
-    if (a->as_string() == "Barorax") return import_prenorm(cfg);
+    if (a->as_string() == "Barorax" || a->as_string() == "Derusun") return import_prenorm(cfg);
   }
   const Json* archs = cfg.find("architectures");
   if (!archs || !archs->is_array() || archs->size() == 0) throw ImportError("config.json: `architectures` is missing or empty");

@@ -87,6 +87,7 @@ struct Layer {
   uint64_t state_bytes = 0;    // bytes of one sequence's state, its convolution inputs included
   bool opens_pass = false;     // the first layer of a pass of the loop
   bool selective = false;      // the recurrence is a selective scan: two small products of its own in front of it
+  bool bottlenecks = false;    // the recurrence's decays and output gate come from a product behind a bottleneck each
   size_t always_ff = 0;        // routed feed-forward: size of an expert that runs for every token
   std::string label;  // e.g. "input_layernorm", "self_attn"
   std::vector<Param> params;
@@ -103,6 +104,7 @@ struct ModelMeta {
   bool layered = false;        // the configuration lists its layers one by one; runs on one device
   bool parallel = false;       // ... and they are parallel layers
   bool prenorm = false;        // ... or pre-norm layers
+  bool shifted = false;        // ... behind a token shift and an average over depth
 
   Json to_json() const {
     Json j = Json::object();
@@ -117,6 +119,7 @@ struct ModelMeta {
     if (layered) j.set("layered", true);
     if (parallel) j.set("parallel", true);
     if (prenorm) j.set("prenorm", true);
+    if (shifted) j.set("shifted", true);
     return j;
   }
   static ModelMeta from_json(const Json& j) {
@@ -137,6 +140,7 @@ struct ModelMeta {
     if (const Json* ly = j.find("layered"); ly && !ly->is_null()) m.layered = ly->as_bool();
     if (const Json* pa = j.find("parallel"); pa && !pa->is_null()) m.parallel = pa->as_bool();
     if (const Json* pr = j.find("prenorm"); pr && !pr->is_null()) m.prenorm = pr->as_bool();
+    if (const Json* sh = j.find("shifted"); sh && !sh->is_null()) m.shifted = sh->as_bool();
     return m;
   }
   bool is_moe() const { return num_experts && *num_experts > 0; }

@@ -14,6 +14,12 @@ def _read(p) -> str:
     return Path(p).read_text()
 
 
+def _read_model(p, checkpoint=None) -> str:
+    """A model's configuration; sizes that its design leaves to the checkpoint come from there (a folder of its own or the configuration's)."""
+    from ..models.config import sized_config
+    return sized_config(_read(p), checkpoint or Path(p).parent)
+
+
 def _search_options(args) -> dict:
     o = {"objective": getattr(args, "objective", "latency")}
     for env, key in (("SKEIN_FORCE_TP", "force_tp"), ("SKEIN_FORCE_PP", "force_pp"), ("SKEIN_FORCE_EP", "force_ep"), ("SKEIN_FORCE_BATCH", "force_batch")):
@@ -31,7 +37,7 @@ def _plan_summary(plan: dict) -> dict:
 
 def cmd_extract(args, emit) -> int:
     t0 = time.time()
-    ins = (_read(args.model), _read(args.cluster), _read(args.trace), _read(args.drift), _read(args.cost))
+    ins = (_read_model(args.model), _read(args.cluster), _read(args.trace), _read(args.drift), _read(args.cost))
     if args.disaggregate_decode_devices:
         r = core.extract_disaggregated_plan(*ins, args.disaggregate_decode_devices, _search_options(args))
     else:
@@ -57,7 +63,7 @@ def cmd_compile(args, emit) -> int:
     prompts = None
     if args.parity_prompts_path:
         prompts = [json.loads(l)["tokens"] for l in _read(args.parity_prompts_path).splitlines() if l.strip()]
-    r = compile_model(_read(args.model), _read(args.cluster), _read(args.trace), _read(args.drift), _read(args.cost), args.out,
+    r = compile_model(_read_model(args.model, args.weights), _read(args.cluster), _read(args.trace), _read(args.drift), _read(args.cost), args.out,
                       weights=args.weights, options=_search_options(args), n_parity_prompts=args.n_parity_prompts, prompts=prompts,
                       enforce_parity=args.enforce_parity, seed=args.seed, search_budget=args.search_budget)
     if r.replans:
@@ -164,7 +170,7 @@ def cmd_calibrate(args, emit) -> int:
         pp_ = Path(args.fit_plan)
         plan_text = _read(pp_ / "plan.json") if pp_.is_dir() else _read(pp_)
         cost_now = _read(args.out_cost)
-        fitted = cal.fit_fixed_costs(plan_text, _read(args.model), _read(args.fit_cluster), cost_now, args.fit_step_ms, args.fit_kv_tokens)
+        fitted = cal.fit_fixed_costs(plan_text, _read_model(args.model), _read(args.fit_cluster), cost_now, args.fit_step_ms, args.fit_kv_tokens)
         Path(args.out_cost).write_text(cal.rewrite_toml_values(cost_now, fitted))
     if args.candidate_artifact:
         from ..compile import parity

@@ -12,8 +12,9 @@ import json
 from dataclasses import asdict, dataclass
 from pathlib import Path
 
-from .layered import LAYERED_ARCHS, PARALLEL_ARCHS, PRENORM_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers, unroll_loop
+from .layered import LAYERED_ARCHS, PARALLEL_ARCHS, PRENORM_ARCHS, SHIFTED_ARCHS, DenseFFSpec, RoutedFFSpec, SpecError, layers_to_list, param_shapes, parse_layers, unroll_loop
 from .parallel_layers import attention_of, parse_loop, recurrence_of
+from .prenorm_layers import fill_ranks
 
 MOE_ARCHS = {"MixtralForCausalLM"}
 DENSE_ARCHS = {"LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM"}
@@ -48,6 +49,7 @@ class ModelConfig:
     conv_taps: int = 0            # taps of the input convolution
     post_alpha: float = 1.0       # weight of the residual inside the post-norms
     loop: tuple | None = None     # (start, stop, times): checkpoint layers that run several times (`layers` lists every run)
+    norm_groups: int = 1          # equal parts of a normed row that have a root mean square each
 
     @property
     def is_moe(self) -> bool:
@@ -68,15 +70,19 @@ class ModelConfig:
         return self.architecture in PRENORM_ARCHS
 
     @property
+    def is_shifted(self) -> bool:
+        """Pre-norm layers whose mixer also reads the previous token's row, and whose stream is averaged over depth."""
+        return self.architecture in SHIFTED_ARCHS
+
+    @property
     def has_state(self) -> bool:
-        """Sequences carry a recurrent state beside their cache pages: each needs a state slot, and a prefix of cached pages
-        alone does not bring a sequence back."""
-        return any(recurrence_of(l.mixer) is not None for l in self.layers)
+        """Sequences carry a recurrent state (or the last token's rows) beside their cache pages: each needs a state slot, and a prefix of
+        cached pages alone does not bring a sequence back."""
+        return self.is_shifted or any(recurrence_of(l.mixer) is not None for l in self.layers)
 
     def state_bytes_per_slot(self, elem: int = 2) -> int:
-        if not self.has_state:
-            return 0
-        return sum(recurrence_of(l.mixer).state_bytes(elem) for l in self.layers if recurrence_of(l.mixer) is not None)
+        rows = 4 * self.hidden_size * self.num_layers if self.is_shifted else 0
+        return rows + sum(recurrence_of(l.mixer).state_bytes(elem) for l in self.layers if recurrence_of(l.mixer) is not None)
 
     @property
     def default_page_size(self) -> int:
@@ -104,6 +110,8 @@ class ModelConfig:
         if self.is_layered:
             if self.conv_taps < 1 and not (self.is_parallel or self.is_prenorm):
                 raise ImportError_("canon.taps must be at least 1")
+            if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+                raise ImportError_("norm.groups must divide width")
             return
         if self.num_heads % self.num_kv_heads != 0:
             raise ImportError_("num_attention_heads must be a multiple of num_key_value_heads")
@@ -200,6 +208,8 @@ class ModelConfig:
                 only = {"loop": parse_loop(d.get("loop"), len(d["layers"]))}
             else:
                 only = {"taps": int(d["canon"]["taps"]), "alpha": float(d["postln_alpha"])}
+            if arch in SHIFTED_ARCHS:
+                only["groups"] = int(d["norm"].get("groups") or 1)
             cfg = ModelConfig.layered(arch, layers, width=int(d["width"]), vocab=int(d["vocab"]), eps=float(d["norm"]["eps"]),
                                       name=name or arch.lower(), **only)
         except KeyError as e:
@@ -215,7 +225,7 @@ class ModelConfig:
 
     @staticmethod
     def layered(arch: str, layers, width: int, vocab: int, taps: int = 0, alpha: float = 1.0, eps: float = 1e-5, max_pos: int = 131072,
-                name: str = "layered", loop: tuple | None = None) -> "ModelConfig":
+                name: str = "layered", loop: tuple | None = None, groups: int = 1) -> "ModelConfig":
         """Configuration of a design that lists its layers. The single-valued fields describe its largest layer (planning and
         display only; the layer specifications decide what runs). The design sets no position limit: max_pos is the engine's.
         `loop` (start, stop, times): `layers` are its runs (models/layered.py: unroll_loop)."""
@@ -225,7 +235,7 @@ class ModelConfig:
                           num_heads=max(l.mixer.heads for l in layers) if layers else 0, num_kv_heads=1,
                           head_dim=max(l.mixer.head_size for l in layers) if layers else 0, vocab_size=vocab,
                           rms_norm_eps=eps, rope_theta=bases[0] if bases else 1e4, num_experts=0, top_k=0,
-                          max_position_embeddings=max_pos, name=name, layers=tuple(layers), conv_taps=taps, post_alpha=alpha, loop=loop)
+                          max_position_embeddings=max_pos, name=name, layers=tuple(layers), conv_taps=taps, post_alpha=alpha, loop=loop, norm_groups=groups)
         cfg.validate()
         return cfg
 
@@ -234,6 +244,8 @@ class ModelConfig:
         if self.is_parallel or self.is_prenorm:
             d = {"architecture": self.architecture, "width": self.hidden_size, "vocab": self.vocab_size, "norm": {"eps": self.rms_norm_eps},
                  "layers": layers_to_list(self.layers), "max_position_embeddings": self.max_position_embeddings}
+            if self.is_shifted:
+                d["norm"]["groups"] = self.norm_groups
             if self.loop is not None:
                 d["loop"] = dict(zip(("start", "stop", "times"), self.loop))
             return d
@@ -255,7 +267,33 @@ class ModelConfig:
     @staticmethod
     def from_file(path) -> "ModelConfig":
         p = Path(path)
-        return ModelConfig.from_hf_dict(json.loads(p.read_text()), name=p.stem.replace("_config", ""))
+        return ModelConfig.from_hf_dict(json.loads(sized_config(p.read_text(), p.parent)), name=p.stem.replace("_config", ""))
+
+
+def checkpoint_shapes(path) -> dict:
+    """Tensor name -> shape of a checkpoint (a safetensors file, or a directory with one or with shards), from the files' headers; empty
+    where there is none."""
+    p = Path(path)
+    index = p / "model.safetensors.index.json"
+    files = [p] if p.is_file() else sorted({p / f for f in json.loads(index.read_text())["weight_map"].values()}) if index.exists() \
+        else [p / "model.safetensors"]
+    shapes = {}
+    for f in files:
+        if f.suffix != ".safetensors" or not f.exists():
+            continue
+        with open(f, "rb") as fh:
+            header = json.loads(fh.read(int.from_bytes(fh.read(8), "little")))
+        shapes.update({n: tuple(t["shape"]) for n, t in header.items() if n != "__metadata__"})
+    return shapes
+
+
+def sized_config(config_json: str, checkpoint) -> str:
+    """The configuration with the sizes that its design leaves to the checkpoint's tensors filled in (where there is a checkpoint)."""
+    d = json.loads(config_json)
+    if d.get("architecture") not in SHIFTED_ARCHS or checkpoint is None or not isinstance(d.get("layers"), list):
+        return config_json
+    shapes = checkpoint_shapes(checkpoint)
+    return json.dumps(fill_ranks(d, shapes.get)) if shapes else config_json
 
 
 def mixtral_8x7b() -> ModelConfig:
@@ -323,6 +361,21 @@ def tiny_barorax(width=96, vocab=384, eps=1e-5) -> ModelConfig:
     specs = [(scan, moe(40, 56)), (diff, moe(32, 24)), (chunk, None), (scan, moe(24, 48, 8, 2, 1, 1))]
     loop = (1, 4, 2)
     return ModelConfig.layered("Barorax", unroll_loop(specs, loop), width=width, vocab=vocab, eps=eps, max_pos=4096, name="tiny-barorax", loop=loop)
+
+
+def tiny_derusun(width=96, vocab=384, eps=1e-5, groups=3) -> ModelConfig:
+    """A small model of the Derusun design for tests: every mixer, layers without feed-forward, values mixed in two of three layers."""
+    from .layered import LatentMixerSpec
+    from .parallel_layers import RecurrentSpec, WindowAttnSpec
+    latent = LatentMixerSpec("latent_attention", heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=56, rope_base=2e4, scale=0.16, sink=True)
+    rec = RecurrentSpec("channel_delta", heads=4, groups=2, dim=24, vdim=32, taps=3, decay_rank=16, gate_rank=8)
+
+    def attn(window, keep, cap, mix=True):
+        return WindowAttnSpec(heads=6, kv_heads=2, dim=28, vdim=20, scale=0.2, rot_dims=0, rope_base=1e4, window=window, kind="attention",
+                              row_norm=False, bias=True, head_norm=True, softcap=cap, keep_first=keep, head_sink=True, v_mix=mix)
+    specs = [(rec, DenseFFSpec(144, 1.5)), (attn(19, 5, 9.0), None), (latent, DenseFFSpec(80, 3.0)), (attn(33, 0, 30.0, False), DenseFFSpec(64, 2.5)),
+             (attn(19, 11, 4.0), DenseFFSpec(120, 1.0)), (rec, None)]
+    return ModelConfig.layered("Derusun", unroll_loop(specs, None), width=width, vocab=vocab, eps=eps, max_pos=4096, name="tiny-derusun", groups=groups)
 
 
 @dataclass

@@ -283,14 +283,14 @@ class Decoder(LayeredOps, ParallelOps, PrenormOps):
     class _Run:
         """State of one pass over the program."""
         __slots__ = ("inp", "residual", "normed", "qkv", "attn", "pending", "pending_kind", "routed", "h", "sp", "T",
-                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts", "dense", "cat")
+                     "crossing", "embed_deferred", "row_idx", "row_w", "owner", "dp", "wts", "dense", "cat", "hist", "v_first")
 
         def __init__(self, inp, residual):
             self.inp, self.residual = inp, residual
             self.normed = self.qkv = self.attn = self.pending = self.routed = self.h = None
             self.pending_kind, self.crossing, self.sp, self.T = None, None, False, 0
             self.embed_deferred = False
-            self.row_idx = self.row_w = self.owner = self.wts = self.dense = self.cat = None
+            self.row_idx = self.row_w = self.owner = self.wts = self.dense = self.cat = self.hist = self.v_first = None
             self.dp = 0          # rows per rank under data-parallel attention (0: every rank holds all rows)
 
     def dp_ways(self) -> int:
@@ -335,6 +335,8 @@ class Decoder(LayeredOps, ParallelOps, PrenormOps):
     def _op_embed_tokens(self, st, _):
         if self.cfg.is_parallel:
             self._embed_parallel(st)
+        elif self.cfg.is_shifted:
+            self._embed_shifted(st)
         elif self.cfg.is_layered:
             st.residual = ops.latent.embed_f32(st.inp.token_ids, self.w.embed)
         elif self.embed_vocab_start is not None:

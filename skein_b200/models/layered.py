@@ -17,6 +17,10 @@ which mixers exist:
   Barorax   attention            differential attention (two maps per head over the same values), gated
             attention_2          attention inside chunks, unit queries and keys, a sink
             mamba1               selective scan
+  Derusun   latent_attention     latent attention, queries straight from the input, a learned sink per head
+            attention            grouped-query attention over a window that keeps the first tokens; biases, head norms, capped scores, a
+                                 learned sink per head, values mixed with the first such layer's
+            channel_delta        gated delta rule with a decay per head and key channel
 """
 from __future__ import annotations
 
@@ -30,9 +34,12 @@ from .parallel_layers import MixerPairSpec, RecurrentSpec, SelectiveSpec, SpecEr
 # architecture -> mixer type -> (queries through a latent, output gate), or the parser of the mixer
 LAYERED_ARCHS = {"Zarorax": {"latent_attention": (True, False), "latent_attention_2": (False, True)},
                  "Sikalorn": {"parallel": pl.parse_pair, "delta": pl.parse_delta, "lightning": pl.parse_lightning},
-                 "Barorax": {"attention": pl.parse_differential, "attention_2": pl.parse_chunked, "mamba1": pl.parse_selective}}
-PARALLEL_ARCHS = {"Sikalorn"}      # the architectures of parallel layers
-PRENORM_ARCHS = {"Barorax"}        # ... and of pre-norm layers
+                 "Barorax": {"attention": pl.parse_differential, "attention_2": pl.parse_chunked, "mamba1": pl.parse_selective},
+                 "Derusun": {"latent_attention": lambda m: parse_latent(m, "latent_attention", False, False, sink=True),
+                             "attention": pl.parse_kept_window, "channel_delta": pl.parse_channel_delta}}
+PARALLEL_ARCHS = {"Sikalorn"}              # the architectures of parallel layers
+PRENORM_ARCHS = {"Barorax", "Derusun"}     # ... and of pre-norm layers
+SHIFTED_ARCHS = {"Derusun"}                # pre-norm layers behind a token shift and an average over depth (models/prenorm_layers.py)
 
 GLU_SLOPE = 1.702          # g * sigmoid(GLU_SLOPE * g) of the clamped gated unit
 
@@ -49,6 +56,7 @@ class LatentMixerSpec:
     scale: float
     q_rank: int = 0          # 0: queries straight from the input
     gated: bool = False
+    sink: bool = False       # one more term exp(a learned number per head) in the softmax's denominator
 
     @property
     def cache_width(self) -> int:
@@ -67,10 +75,44 @@ class LatentMixerSpec:
     def cache_elems_per_token(self) -> int:
         return self.cache_width
 
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def sections(self) -> list:
+        """(tensor, rows) of the projections of a pre-norm layer's input, in stacking order."""
+        return [("q", self.q_width), ("dkv", self.cache_width)]
+
+    def param_shapes(self, C: int) -> dict:
+        s = {n: (rows, C) for n, rows in self.sections()}
+        s["dkv.norm"], s["uk"], s["uv"] = (self.kv_rank,), (self.heads * self.dim, self.kv_rank), (self.heads * self.vdim, self.kv_rank)
+        if self.sink:
+            s["sink"] = (self.heads,)
+        s["o"] = (C, self.out_width)
+        return s
+
+    def to_dict(self) -> dict:
+        d = {"heads": self.heads, "dim": self.dim, "rot_dim": self.rot_dim, "vdim": self.vdim, "kv_rank": self.kv_rank, "scale": self.scale,
+             "rot": {"base": self.rope_base, "dims": self.rot_dim}}
+        return {**d, "q_rank": self.q_rank} if self.q_rank else d
+
+
+def parse_latent(m: dict, kind: str, q_latent: bool, gated: bool, sink: bool = False) -> LatentMixerSpec:
+    rot = m["rot"]
+    if int(rot["dims"]) != int(m["rot_dim"]):
+        raise SpecError("rot.dims must equal rot_dim")
+    mixer = LatentMixerSpec(kind=kind, heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
+                            kv_rank=int(m["kv_rank"]), rope_base=float(rot["base"]), scale=float(m["scale"]),
+                            q_rank=int(m["q_rank"]) if q_latent else 0, gated=gated, sink=sink)
+    if mixer.rot_dim % 2:
+        raise SpecError("rot_dim must be even (rotation turns pairs)")
+    return mixer
+
 
 @dataclass(frozen=True)
 class DenseFFSpec:
     ff: int
+    limit: float | None = None   # of a clamped gated unit (gate and up projections); None: the design's ungated unit
 
 
 @dataclass(frozen=True)
@@ -111,16 +153,10 @@ def parse_layers(arch: str, layers: list, loop: dict | None = None) -> tuple:
     for i, d in enumerate(layers):
         if d.get("type") not in kinds:
             raise SpecError(f"layer {i}: mixer type {d.get('type')!r} is not part of {arch}")
-        q_latent, gated = kinds[d["type"]]
-        m = d["mixer"]
-        rot = m["rot"]
-        if int(rot["dims"]) != int(m["rot_dim"]):
-            raise SpecError(f"layer {i}: rot.dims must equal rot_dim")
-        mixer = LatentMixerSpec(kind=d["type"], heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
-                                kv_rank=int(m["kv_rank"]), rope_base=float(rot["base"]), scale=float(m["scale"]),
-                                q_rank=int(m["q_rank"]) if q_latent else 0, gated=gated)
-        if mixer.rot_dim % 2:
-            raise SpecError(f"layer {i}: rot_dim must be even (rotation turns pairs)")
+        try:
+            mixer = parse_latent(d["mixer"], d["type"], *kinds[d["type"]])
+        except SpecError as e:
+            raise SpecError(f"layer {i}: {e}") from e
         mlp = d.get("mlp")
         if mlp is None:
             ff = None
@@ -158,7 +194,7 @@ def _parse_dense(mlp: dict) -> DenseFFSpec:
 
 def _parse_runs(arch: str, layers: list, loop: dict | None) -> tuple:
     """Layers whose mixers have a parser each, one entry per run of a loop."""
-    specs, parse_ff = [], pn.parse_ff if arch in PRENORM_ARCHS else _parse_dense
+    specs, parse_ff = [], pn.PARSE_FF.get(arch, _parse_dense)
     for i, d in enumerate(layers):
         parse = LAYERED_ARCHS[arch].get(d.get("type"))
         if parse is None:
@@ -168,6 +204,10 @@ def _parse_runs(arch: str, layers: list, loop: dict | None) -> tuple:
             specs.append((parse(d["mixer"]), parse_ff(mlp) if mlp is not None else None))
         except SpecError as e:
             raise SpecError(f"layer {i}: {e}") from e
+    if arch in SHIFTED_ARCHS:
+        if loop:
+            raise SpecError(f"{arch} has no loop")
+        pn.check_value_mixing([m for m, _ in specs])
     return unroll_loop(specs, pl.parse_loop(loop, len(specs)))
 
 
@@ -188,12 +228,7 @@ def layers_to_list(layers) -> list:
         return [{"type": sp.mixer.kind, "mixer": sp.mixer.to_dict(), "mlp": _ff_to_dict(sp.mlp)} for sp in sorted(own, key=lambda sp: sp.tensors)]
     out = []
     for sp in layers:
-        m = sp.mixer
-        mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
-                 "rot": {"base": m.rope_base, "dims": m.rot_dim}}
-        if m.q_rank:
-            mixer["q_rank"] = m.q_rank
-        d = {"type": m.kind, "mixer": mixer, "mlp": _ff_to_dict(sp.mlp)}
+        d = {"type": sp.mixer.kind, "mixer": sp.mixer.to_dict(), "mlp": _ff_to_dict(sp.mlp)}
         if sp.weights_of is not None:
             d["weights_of"] = sp.weights_of
         out.append(d)
@@ -204,7 +239,7 @@ def _ff_to_dict(f) -> dict | None:
     if f is None:
         return None
     if isinstance(f, DenseFFSpec):
-        return {"kind": "dense", "ff": f.ff}
+        return {"kind": "dense", "ff": f.ff} if f.limit is None else {"kind": "dense", "ff": f.ff, "limit": f.limit}
     r, expert = {"experts": f.experts, "top": f.top}, {"ff": f.ff}
     if (f.groups, f.keep) != (1, 1):
         r["groups"] = {"count": f.groups, "keep": f.keep}
@@ -321,9 +356,10 @@ class LatentMixerWeights:
     kv_norm: torch.Tensor              # [kv_rank] fp32
     w_ukv: torch.Tensor                # [H dim + H vdim, kv_rank]: keys then values of every head from the latent
     w_uk_t: torch.Tensor               # [H, kv_rank, dim]: the key expansion transposed, applied to the queries
-    wo: torch.Tensor                   # [C, H vdim]
+    wo: torch.Tensor | None            # [C, H vdim]
     off_kv: int = 0                    # first column of the cache row / the gate in the input projection's output
     off_gate: int = -1
+    sinks: torch.Tensor | None = None  # [H] fp32
 
 
 @dataclass
@@ -353,14 +389,19 @@ def stack_rows(parts):
     return torch.cat(rows, dim=0).contiguous(), offs
 
 
+def expansions(m: LatentMixerSpec, get, prefix: str):
+    """(keys then values of every head from the latent [H dim + H vdim, kv_rank], the key expansion transposed [H, kv_rank, dim])."""
+    uk, uv = get(prefix + "uk"), get(prefix + "uv")
+    return torch.cat([uk, uv], dim=0).contiguous(), uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).contiguous()
+
+
 def assemble_mixer(m: LatentMixerSpec, get, prefix: str) -> LatentMixerWeights:
     parts = [get(prefix + ("dq" if m.q_rank else "q")), get(prefix + "dkv")] + ([get(prefix + "g")] if m.gated else [])
     w_in, offs = stack_rows(parts)
-    uk, uv = get(prefix + "uk"), get(prefix + "uv")
+    w_ukv, w_uk_t = expansions(m, get, prefix)
     return LatentMixerWeights(
         w_in=w_in, q_norm=get(prefix + "dq.norm").float() if m.q_rank else None, w_uq=get(prefix + "uq").contiguous() if m.q_rank else None,
-        kv_norm=get(prefix + "dkv.norm").float(), w_ukv=torch.cat([uk, uv], dim=0).contiguous(),
-        w_uk_t=uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).contiguous(), wo=get(prefix + "o").contiguous(),
+        kv_norm=get(prefix + "dkv.norm").float(), w_ukv=w_ukv, w_uk_t=w_uk_t, wo=get(prefix + "o").contiguous(),
         off_kv=offs[1], off_gate=offs[2] if m.gated else -1)
 
 
@@ -380,7 +421,7 @@ def assemble_layers(cfg, get) -> list:
             out.append(out[sp.weights_of])
             continue
         if cfg.is_parallel or cfg.is_prenorm:
-            out.append((pl if cfg.is_parallel else pn).assemble_layer(sp, get))
+            out.append(pl.assemble_layer(sp, get) if cfg.is_parallel else pn.assemble_layer(sp, get, cfg.is_shifted))
             continue
         p = f"l{i}."
         lw = LayeredWeights(mixer=assemble_mixer(sp.mixer, get, p + "mix."), conv=get(p + "canon1").float().t().contiguous(),

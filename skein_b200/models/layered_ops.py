@@ -70,6 +70,17 @@ class LayeredOps:
         return inp.kv_start, inp.kv_total, inp.max_cached
 
     # ---- mixer ----------------------------------------------------------------------------------------------
+    def _latent_parts(self, st, li):
+        """(weights, first column of the cache row, queries or None when they have a latent, gate or None) of a latent mixer, in the
+        output of its input projection."""
+        m, lw = self.cfg.layers[li].mixer, self.w.layers[li]
+        if self.cfg.is_prenorm:
+            col = self.layouts[li].parts[0].col
+            return lw.latent, col["dkv"], st.qkv[:, col["q"]:col["q"] + m.q_width], None
+        mw = lw.mixer
+        gate = st.qkv[:, mw.off_gate:mw.off_gate + m.heads * m.vdim] if m.gated else None
+        return mw, mw.off_kv, None if m.q_rank else st.qkv[:, :m.q_width], gate
+
     def _op_input_conv(self, st, li):
         if st.normed is not None:
             return              # decode: produced by the kernel that normed the previous layer
@@ -82,7 +93,8 @@ class LayeredOps:
         st.normed = None
 
     def _op_latent_append(self, st, li):
-        inp, m, mw = st.inp, self.cfg.layers[li].mixer, self.w.layers[li].mixer
+        inp, m = st.inp, self.cfg.layers[li].mixer
+        mw, off_kv, _, _ = self._latent_parts(st, li)
         st.dense = None
         kv_start = None
         if self._expanded(inp, m):
@@ -90,30 +102,38 @@ class LayeredOps:
             st.dense = torch.empty(total, m.cache_width, dtype=self.act_dtype, device=self.device)
             if cached > 0:
                 lat.latent_gather(self.kv[li], inp.block_table, inp.seq_lens, inp.q_len, kv_start, st.dense, cached)
-        decode = self._decode_rows(inp)
-        st.attn = lat.latent_append(st.qkv, mw.off_kv, mw.q_norm, mw.kv_norm, m.rot_dim, self.rope_tables[li], inp.positions, inp.seq_of_token,
-                                    inp.block_table, self.kv[li], self.cfg.rms_norm_eps, None if decode else st.residual, self.conv_tail[li],
-                                    inp.seq_lens, self.cfg.conv_taps, st.dense, kv_start)
+        tail, x = None, None
+        if self.conv_tail:
+            tail, x = self.conv_tail[li], None if self._decode_rows(inp) else st.residual
+        st.attn = lat.latent_append(st.qkv, off_kv, mw.q_norm, mw.kv_norm, m.rot_dim, self.rope_tables[li], inp.positions, inp.seq_of_token,
+                                    inp.block_table, self.kv[li], self.cfg.rms_norm_eps, x, tail, inp.seq_lens, max(self.cfg.conv_taps, 1), st.dense,
+                                    kv_start)
 
     def _op_latent_q_up(self, st, li):
         st.attn = ops.linear(st.attn, self.w.layers[li].mixer.w_uq)     # the normed query latent -> queries
 
     def _op_latent_attention(self, st, li):
-        inp, m, mw = st.inp, self.cfg.layers[li].mixer, self.w.layers[li].mixer
-        q = st.attn if m.q_rank else st.qkv[:, :m.q_width]
-        gate = st.qkv[:, mw.off_gate:mw.off_gate + m.heads * m.vdim] if m.gated else None
+        inp, m = st.inp, self.cfg.layers[li].mixer
+        mw, _, q, gate = self._latent_parts(st, li)
+        q = st.attn if q is None else q
         if st.dense is not None:
             lat.rope_rows(q, m.heads, m.dim, m.rot_dim, self.rope_tables[li], inp.positions)
             kv = ops.linear(st.dense, mw.w_ukv)
             st.attn = lat.latent_attn_prefill(q, m.heads, m.dim, m.rot_dim, m.vdim, m.scale, st.dense, kv, inp.q_start, inp.q_len, inp.seq_lens,
-                                              inp.kv_start, inp.max_q_len, gate)
+                                              inp.kv_start, inp.max_q_len, gate, mw.sinks)
         else:
             q_abs = lat.head_linear(q, m.dim + m.rot_dim, mw.w_uk_t)
             o = lat.latent_attn_rows(q_abs, q, m.heads, m.dim, m.rot_dim, m.scale, self.rope_tables[li], inp.positions, inp.seq_of_token,
-                                     inp.block_table, self.kv[li], inp.ctx_hint)
+                                     inp.block_table, self.kv[li], inp.ctx_hint, sinks=mw.sinks)
             w_uv = mw.w_ukv[m.heads * m.dim:].view(m.heads, m.vdim, m.kv_rank)
+            if self.cfg.is_prenorm:      # straight into the row that the product back reads
+                lat.head_linear(o, m.kv_rank, w_uv, gate, out=st.qkv[:, :m.out_width])
+                st.attn = st.dense = None
+                return
             st.attn = lat.head_linear(o, m.kv_rank, w_uv, gate)
-        st.dense = st.qkv = None
+        st.dense = None
+        if not self.cfg.is_prenorm:
+            st.qkv = None
 
     def _op_latent_o_proj(self, st, li):
         st.pending, st.attn = ops.linear(st.attn, self.w.layers[li].mixer.wo), None

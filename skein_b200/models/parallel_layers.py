@@ -6,12 +6,14 @@ Mixers (specifications are data; a design picks some and fixes nothing else):
   WindowAttnSpec   grouped-query attention over a sliding window, over chunks or over everything before; RMS norm of the whole q and k
                    projections (or none), then rotation of the first rot_dims dimensions of every head (pairs i, i + rot_dims / 2, or
                    neighbours; frequencies divided by rot_factor), then unit heads (or not); a sink; two maps per head of which the
-                   second is subtracted; an output gate
+                   second is subtracted; an output gate; biases on the projections; RMS norm with a weight per head; a cap on the scores;
+                   a window's first tokens kept in sight; a learned sink per head; values mixed with those of the first such layer
   RecurrentSpec    a matrix state S [dim, vdim] per head, 32-bit, carried from token to token:
                        S <- g S + k u^T,   o = S^T q (+ D v)
                      "delta"      g per head and token, u = beta (v - (g S)^T k), q and k unit vectors
                      "ssd"        g = exp(-exp(A) dt), u = dt v (Mamba-2; q, k, v are C, B, x)
                      "lightning"  g fixed per head, u = v
+                     "channel_delta"  "delta" with one g per head, token and row of S; g and the output's gate come from a bottleneck each
   SelectiveSpec    a diagonal recurrence per channel (Mamba), 32-bit, behind a short convolution:
                        S[n, c] <- exp(dt[c] A[n, c]) S[n, c] + dt[c] x[c] B[n],   y[c] = sum_n S[n, c] C[n] + D[c] x[c],   y silu(z)
   MixerPairSpec    an attention and a recurrence beside each other, summed with a weight each
@@ -60,6 +62,12 @@ class WindowAttnSpec:
     sink: bool = False       # one more term exp(0) in the softmax's denominator
     diff: float | None = None    # two maps per head over the same values: (1 - diff) N(map 1 - lambda map 2) with lambda learned around diff
     gated: bool = False      # the output is multiplied by the sigmoid of a projection
+    bias: bool = False       # q, k and v have biases
+    head_norm: bool = False  # RMS norm of every head of q and k, with a weight that the heads share, before the rotation
+    softcap: float = 0.0     # scores are softcap * tanh(score / softcap) (0: as they are)
+    keep_first: int = 0      # with a window: the sequence's first tokens that every position sees
+    head_sink: bool = False  # one more term exp(a learned number per head) in the softmax's denominator
+    v_mix: bool = False      # values are mixed with those that the first such layer has for the token
 
     @property
     def maps(self) -> int:
@@ -91,8 +99,16 @@ class WindowAttnSpec:
         s = {n: (rows, C) for n, rows in self.sections()}
         if self.row_norm:
             s["q.norm"], s["k.norm"] = (self.heads * self.dim,), (self.kv_heads * self.dim,)
+        if self.bias:
+            s.update({n + ".b": (rows,) for n, rows in self.sections()[:3]})
+        if self.head_norm:
+            s["q.norm"], s["k.norm"] = (self.dim,), (self.dim,)
         if self.diff is not None:
             s.update({n: (self.dim,) for n in LAMBDA_VECTORS})
+        if self.v_mix:
+            s["vmix"] = ()
+        if self.head_sink:
+            s["sink"] = (self.heads,)
         s["o"] = (C, self.out_width)
         return s
 
@@ -100,9 +116,17 @@ class WindowAttnSpec:
         rot = {"base": self.rope_base, "dims": self.rot_dims}
         if self.rope_factor != 1.0:
             rot["scaling"] = {"factor": self.rope_factor}
-        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": rot}
+        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale}
+        if self.rot_dims or not self.head_norm:
+            d["rot"] = rot
         if self.window or self.chunk:
             d["mask"] = {"size": self.window or self.chunk}
+            if self.keep_first:
+                d["mask"]["keep_first"] = self.keep_first
+        if self.softcap:
+            d["softcap"] = self.softcap
+        if self.v_mix:
+            d["v_mix"] = True
         if self.diff is not None:
             d["diff"] = self.diff
         return d
@@ -113,7 +137,7 @@ LAMBDA_VECTORS = ("lq1", "lk1", "lq2", "lk2")      # lambda = exp(lq1 . lk1) - e
 
 @dataclass(frozen=True)
 class RecurrentSpec:
-    kind: str                # "delta", "ssd" or "lightning"
+    kind: str                # "delta", "channel_delta", "ssd" or "lightning"
     heads: int               # value heads (one state each)
     groups: int              # query / key heads; head h uses h // (heads / groups)
     dim: int                 # of a query / key head: rows of the state
@@ -121,6 +145,13 @@ class RecurrentSpec:
     taps: int = 1            # of the short convolutions over time (1 for "lightning": none)
     norm_groups: int = 1     # equal parts of the normed output that have a root mean square each ("ssd")
     decay: tuple = ()        # "lightning"
+    decay_rank: int = 0      # "channel_delta": widths of the bottlenecks in front of the decays ...
+    gate_rank: int = 0       # ... and of the output's gate
+
+    @property
+    def corrects(self) -> bool:
+        """The delta rules: what the state holds for k is replaced, and q and k are unit vectors."""
+        return self.kind in ("delta", "channel_delta")
 
     @property
     def cache_elems_per_token(self) -> int:
@@ -156,6 +187,8 @@ class RecurrentSpec:
         GD, HV = self.groups * self.dim, self.heads * self.vdim
         if self.kind == "ssd":      # rows of the one input matrix: z | x | B | C | dt
             return [("z", HV), ("conv", HV + 2 * GD), ("dt", self.heads)]
+        if self.kind == "channel_delta":
+            return [("q", GD), ("k", GD), ("v", HV), ("b", self.heads), ("a1", self.decay_rank), ("g1", self.gate_rank)]
         qkv = [("q", GD), ("k", GD), ("v", HV), ("g", HV)]
         return qkv + [("b", self.heads), ("a", self.heads)] if self.kind == "delta" else qkv
 
@@ -169,6 +202,10 @@ class RecurrentSpec:
         if self.kind == "delta":
             s.update({n + ".conv": (rows, self.taps) for n, rows in self.sections()[:3]})
             s.update({"A_log": (H,), "dt_bias": (H,), "norm": (self.vdim,)})
+        elif self.kind == "channel_delta":
+            s.update({n + ".conv": (rows, self.taps) for n, rows in self.sections()[:3]})
+            s.update({"A_log": (H,), "norm": (self.vdim,), "a2": (H * self.dim, self.decay_rank), "dt_bias": (H * self.dim,),
+                      "g2": (HV, self.gate_rank)})
         else:
             s["norm"] = (HV,)
         s["o"] = (C, HV)
@@ -181,6 +218,8 @@ class RecurrentSpec:
                     "vdim": self.vdim}
         if self.kind == "delta":
             return {**d, "conv": self.taps, "kv_heads": self.groups}
+        if self.kind == "channel_delta":
+            return {**d, "conv": self.taps, "kv_heads": self.groups, "decay_rank": self.decay_rank, "gate_rank": self.gate_rank}
         return {**d, "decay": list(self.decay)}
 
 
@@ -320,6 +359,28 @@ def parse_delta(m: dict) -> RecurrentSpec:
     return r
 
 
+def parse_channel_delta(m: dict) -> RecurrentSpec:
+    """A configuration that does not name the bottlenecks' widths leaves them to the checkpoint (models/prenorm_layers.py: fill_ranks); where
+    there is none they are a key head's size."""
+    r = RecurrentSpec("channel_delta", heads=int(m["heads"]), groups=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), taps=int(m["conv"]),
+                      decay_rank=int(m.get("decay_rank") or m["dim"]), gate_rank=int(m.get("gate_rank") or m["dim"]))
+    _need(r.heads % r.groups == 0, "heads must be a multiple of kv_heads")
+    _need(r.taps >= 1, "conv must be at least 1")
+    return r
+
+
+def parse_kept_window(m: dict) -> WindowAttnSpec:
+    """Attention without rotation over a window that keeps the first tokens in sight."""
+    mask = m.get("mask") or {}
+    a = WindowAttnSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]), rot_dims=0,
+                       rope_base=1e4, window=int(mask.get("size") or 0), kind="attention", row_norm=False, bias=True, head_norm=True,
+                       softcap=float(m.get("softcap") or 0.0), keep_first=int(mask.get("keep_first") or 0), head_sink=True,
+                       v_mix=bool(m.get("v_mix")))
+    _need(a.heads % a.kv_heads == 0, "heads must be a multiple of kv_heads")
+    _need(a.window >= 0 and a.keep_first >= 0 and a.softcap >= 0, "mask.size, mask.keep_first and softcap must not be negative")
+    return a
+
+
 def parse_lightning(m: dict) -> RecurrentSpec:
     r = RecurrentSpec("lightning", heads=int(m["heads"]), groups=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
                       decay=tuple(float(x) for x in m["decay"]))
@@ -430,9 +491,14 @@ class TanhNorm:
 
 @dataclass
 class WindowAttnWeights:
-    q_norm: torch.Tensor | None = None     # [heads * dim] fp32
-    k_norm: torch.Tensor | None = None     # [kv_heads * dim] fp32
+    q_norm: torch.Tensor | None = None     # [heads * dim] fp32, or [dim] with a norm per head
+    k_norm: torch.Tensor | None = None     # [kv_heads * dim] fp32, or [dim]
     lam: torch.Tensor | None = None        # [1] fp32: weight of the second map
+    q_bias: torch.Tensor | None = None     # fp32
+    k_bias: torch.Tensor | None = None
+    v_bias: torch.Tensor | None = None
+    sinks: torch.Tensor | None = None      # [heads] fp32
+    vmix: torch.Tensor | None = None       # [1] fp32: weight of the first such layer's values
 
 
 @dataclass
@@ -448,13 +514,15 @@ class SelectiveWeights:
 
 @dataclass
 class RecurrentWeights:
-    norm: torch.Tensor                     # output norm, fp32: [vdim] ("delta") or [heads * vdim]
+    norm: torch.Tensor                     # output norm, fp32: [vdim] (delta rules) or [heads * vdim]
     conv: torch.Tensor | None = None       # [taps, channels] fp32, channels q | k | v (zero taps of "lightning": none)
     conv_b: torch.Tensor | None = None     # [channels] fp32
     neg_decay: torch.Tensor | None = None  # [heads] fp32: -exp(A_log), or log(decay) of "lightning"
     decay: torch.Tensor | None = None      # [heads] fp32, "lightning"
-    dt_bias: torch.Tensor | None = None    # [heads] fp32
+    dt_bias: torch.Tensor | None = None    # [heads] fp32, or [heads * dim] ("channel_delta")
     skip: torch.Tensor | None = None       # [heads] fp32: D
+    w_decay: torch.Tensor | None = None    # [heads * dim, decay_rank], columns padded with zeros to a multiple of 8 ("channel_delta")
+    w_gate: torch.Tensor | None = None     # [heads * vdim, gate_rank], likewise
 
 
 @dataclass
@@ -492,11 +560,17 @@ def _pad(t: torch.Tensor, dim: int) -> torch.Tensor:
 
 def load_attention(m: WindowAttnSpec, get, p: str) -> WindowAttnWeights:
     w = WindowAttnWeights()
-    if m.row_norm:
+    if m.row_norm or m.head_norm:
         w.q_norm, w.k_norm = get(p + "q.norm").float(), get(p + "k.norm").float()
     if m.diff is not None:
         lq1, lk1, lq2, lk2 = (get(p + n).double() for n in LAMBDA_VECTORS)
         w.lam = ((lq1 * lk1).sum().exp() - (lq2 * lk2).sum().exp() + m.diff).float().reshape(1)
+    if m.bias:
+        w.q_bias, w.k_bias, w.v_bias = (get(p + n + ".b").float() for n in ("q", "k", "v"))
+    if m.head_sink:
+        w.sinks = get(p + "sink").float()
+    if m.v_mix:
+        w.vmix = get(p + "vmix").float().reshape(1)
     return w
 
 
@@ -507,7 +581,7 @@ def load_selective(m: SelectiveSpec, get, p: str) -> SelectiveWeights:
                             neg_a=-get(p + "A_log").float().t().exp().contiguous(), skip=get(p + "D").float())
 
 
-def _load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
+def load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
     w = RecurrentWeights(norm=get(p + "norm").float())
     GD, HV = m.groups * m.dim, m.heads * m.vdim
     if m.kind == "lightning":
@@ -515,7 +589,9 @@ def _load_recurrence(m: RecurrentSpec, get, p: str) -> RecurrentWeights:
         w.decay, w.neg_decay = (t.to(w.norm.device) for t in (d.float(), d.log().clamp(min=-1e30).float()))
         return w
     w.neg_decay, w.dt_bias = -get(p + "A_log").float().exp(), get(p + "dt_bias").float()
-    if m.kind == "delta":
+    if m.kind == "channel_delta":
+        w.w_decay, w.w_gate = _pad(get(p + "a2"), 1).contiguous(), _pad(get(p + "g2"), 1).contiguous()
+    if m.corrects:
         w.conv = torch.cat([get(p + n + ".conv").float() for n in ("q", "k", "v")]).t().contiguous()
     else:      # the checkpoint's order is x (values) | B (keys) | C (queries)
         c, b = get(p + "conv").float(), get(p + "conv.b").float()
@@ -535,7 +611,7 @@ def assemble_layer(sp, get) -> ParallelLayerWeights:
         if isinstance(m, WindowAttnSpec):
             attn = load_attention(m, get, q)
         else:
-            rec = _load_recurrence(m, get, q)
+            rec = load_recurrence(m, get, q)
         if isinstance(m, RecurrentSpec) and m.kind == "ssd":
             rows, whole = m.sections(), get(q + "in")
             ins.extend(whole.split([n for _, n in rows]))
@@ -555,7 +631,7 @@ def random_param(name: str, shape, gen, device):
         return torch.empty(shape, dtype=torch.float32, device=device).normal_(mean, std, generator=gen)
     if name.endswith(".alpha"):
         return torch.ones(shape, device=device)
-    if name.endswith((".norm1.b", "norm.b", ".conv.b", "loop.step")):
+    if name.endswith((".norm1.b", "norm.b", ".conv.b", "loop.step", ".q.b", ".k.b", ".v.b", ".sink")):
         return normal(0.02)
     if name.endswith(".conv"):
         return normal(shape[-1] ** -0.5)
@@ -567,4 +643,10 @@ def random_param(name: str, shape, gen, device):
         return normal(0.1)
     if name.endswith(".D"):
         return torch.ones(shape, device=device)
+    if name.endswith((".shift", ".vmix")):
+        return normal(0.1, 0.5)
+    if name.endswith(".dwa"):      # near the layer's own result
+        t = normal(0.02)
+        t[-1] += 1.0
+        return t
     return None

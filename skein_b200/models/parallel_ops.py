@@ -99,13 +99,22 @@ class ParallelOps:
         if a.row_norm:
             par.window_append(q, k, v, w.q_norm, w.k_norm, a, *args)
         else:
-            par.head_append(q, k, v, a, *args)
+            par.head_append(q, k, v, a, *args, w=w, mix=self._value_mix(st, a, v))
+
+    def _value_mix(self, st, a, v):
+        """The first mixing layer keeps its values for the step's later ones."""
+        if not a.v_mix:
+            return None
+        keep = st.v_first is None
+        if keep:
+            st.v_first = torch.empty(v.shape, dtype=v.dtype, device=v.device)
+        return par.ValueMix(st.v_first, keep)
 
     def _op_window_attention(self, st, li):
         sec, a, q, _, _ = self._window_section(st, li)
         gate = st.qkv[:, sec.col["g"]:sec.col["g"] + a.out_width] if a.gated else None
         par.window_attn(q, a, st.inp, self.kv[li], self.page_size, st.qkv[:, sec.out:sec.out + a.out_width], sec.scale,
-                        par.HeadMix(self.w.layers[li].attn.lam, gate, self.cfg.rms_norm_eps))
+                        par.HeadMix(self.w.layers[li].attn.lam, gate, self.cfg.rms_norm_eps, self.w.layers[li].attn.sinks))
 
     def _op_recurrence(self, st, li):
         sec, inp = self.layouts[li].part(RecurrentSpec), st.inp
@@ -113,19 +122,29 @@ class ParallelOps:
         args = (st.qkv, cols, sec.spec, self.w.layers[li].rec, self.rec_state[li], inp.positions, self._slots(inp))
         if self._decode_rows(inp):
             r, gate = sec.spec, None
-            if r.kind == "delta":
-                gate = rec.HeadGate(self.w.layers[li].rec.norm, sec.col["g"], st.qkv[:, sec.out:sec.out + r.out_width], self.cfg.rms_norm_eps, sec.scale)
-            st.attn = rec.rec_step(*args, gate=gate)
+            if r.corrects:
+                gate = rec.HeadGate(self.w.layers[li].rec.norm, self._output_gate(st, sec), st.qkv[:, sec.out:sec.out + r.out_width],
+                                    self.cfg.rms_norm_eps, sec.scale, sigmoid=r.kind == "channel_delta")
+            st.attn = rec.rec_step(*args, gate=gate, step=st.dense)
         else:
-            st.attn = rec.rec_chunk(*args, inp.seq_of_token, inp.q_start, inp.q_len, inp.max_q_len)
+            st.attn = rec.rec_chunk(*args, inp.seq_of_token, inp.q_start, inp.q_len, inp.max_q_len, step=st.dense)
+        st.dense = None
+
+    @staticmethod
+    def _output_gate(st, sec):
+        """Inputs of a recurrence's output gate: columns of the row, or the product behind a bottleneck."""
+        r = sec.spec
+        if r.kind == "channel_delta":
+            return st.cat
+        g = sec.col["z" if r.kind == "ssd" else "g"]
+        return st.qkv[:, g:g + r.out_width]
 
     def _op_gated_norm(self, st, li):
         if st.attn is None:
             return              # applied by the decode step's kernel
         sec = self.layouts[li].part(RecurrentSpec)
         r, w = sec.spec, self.w.layers[li].rec
-        g = sec.col["z" if r.kind == "ssd" else "g"]
-        groups = {"ssd": r.norm_groups, "delta": r.heads, "lightning": 1}[r.kind]
-        par.gated_norm(st.attn, st.qkv[:, g:g + r.out_width], w.norm, st.qkv[:, sec.out:sec.out + r.out_width], groups, self.cfg.rms_norm_eps,
-                       gate_first=r.kind == "ssd", silu=r.kind != "lightning", scale=sec.scale)
+        groups = {"ssd": r.norm_groups, "delta": r.heads, "channel_delta": r.heads, "lightning": 1}[r.kind]
+        par.gated_norm(st.attn, self._output_gate(st, sec), w.norm, st.qkv[:, sec.out:sec.out + r.out_width], groups, self.cfg.rms_norm_eps,
+                       gate_first=r.kind == "ssd", silu=r.kind in ("ssd", "delta"), scale=sec.scale)
         st.attn = None

@@ -43,16 +43,16 @@ class GemmParams(C.Structure):
 class RecParams(C.Structure):
     """Mirror of SkeinRecParams in csrc/kernels/recurrent.cuh (same field order)."""
 
-    _fields_ = [(n, C.c_void_p) for n in ("row", "out", "state", "tail", "conv_w", "conv_b", "neg_decay", "decay", "dt_bias", "skip", "positions",
-                                          "slots", "status")] + [("ld", C.c_int64)] + [
+    _fields_ = [(n, C.c_void_p) for n in ("row", "out", "state", "tail", "conv_w", "conv_b", "neg_decay", "decay", "dt_bias", "skip", "step",
+                                          "positions", "slots", "status")] + [("ld", C.c_int64)] + [
         (n, C.c_int32) for n in ("kind", "H", "G", "D", "V", "taps", "C", "q_col", "k_col", "v_col", "a_col", "b_col", "num_slots")]
 
 
 class RecGate(C.Structure):
     """Mirror of SkeinRecGate in csrc/kernels/recurrent.cuh (same field order)."""
 
-    _fields_ = [("norm", C.c_void_p), ("out", C.c_void_p), ("out_ld", C.c_int64), ("gate_col", C.c_int32), ("eps", C.c_float),
-                ("scale", C.c_float), ("pad", C.c_int32)]
+    _fields_ = [("norm", C.c_void_p), ("out", C.c_void_p), ("gate", C.c_void_p), ("out_ld", C.c_int64), ("gate_ld", C.c_int64),
+                ("sigmoid", C.c_int32), ("eps", C.c_float), ("scale", C.c_float), ("pad", C.c_int32)]
 
 
 class RecChunk(C.Structure):
@@ -71,8 +71,23 @@ class RouteRule(C.Structure):
 class AttnRule(C.Structure):
     """Mirror of SkeinAttnRule in csrc/kernels/attn_rule.cuh (same field order)."""
 
-    _fields_ = [("lam", C.c_void_p), ("gate", C.c_void_p), ("gate_ld", C.c_int64)] + [
-        (n, C.c_int32) for n in ("window", "chunk", "sink", "maps")] + [(n, C.c_float) for n in ("scale", "out_scale", "eps")] + [("pad", C.c_int32)]
+    _fields_ = [("lam", C.c_void_p), ("gate", C.c_void_p), ("sinks", C.c_void_p), ("gate_ld", C.c_int64)] + [
+        (n, C.c_int32) for n in ("window", "chunk", "sink", "maps", "keep_first")] + [(n, C.c_float) for n in ("softcap", "scale", "out_scale", "eps")] + [
+        ("pad", C.c_int32)]
+
+
+class HeadExtras(C.Structure):
+    """Mirror of SkeinHeadExtras in csrc/kernels/attn_rule.cuh (same field order)."""
+
+    _fields_ = [(n, C.c_void_p) for n in ("q_bias", "k_bias", "v_bias", "q_norm", "k_norm", "mix", "v_first", "v_keep")]
+
+
+class DepthNormParams(C.Structure):
+    """Mirror of SkeinDepthNormParams in csrc/kernels/prenorm.cu (same field order)."""
+
+    _fields_ = [(n, C.c_void_p) for n in ("terms", "weights", "x_out", "gain", "act_out", "shift", "state", "positions", "slots", "seq_of_token",
+                                          "q_start", "q_len", "status")] + [("term_stride", C.c_int64)] + [
+        (n, C.c_int32) for n in ("n_terms", "T", "C", "groups", "num_slots")] + [("eps", C.c_float)]
 
 
 class ScanParams(C.Structure):
@@ -179,17 +194,19 @@ def lib():
     _sig(L, "skein_rope_rows", i32, [vp, i64, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp])
     _sig(L, "skein_latent_gather", i32, [vp, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp, i32, vp])
     _sig(L, "skein_latent_attn_rows", i32,
-         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, vp])
+         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, vp, vp, i32, vp])
     _sig(L, "skein_latent_attn_decode", i32,
-         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, i32, i32, vp, vp])
+         [vp, vp, i64, vp, i32, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, i32, vp, vp])
     _sig(L, "skein_latent_attn_prefill", i32,
-         [vp, i64, i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp])
+         [vp, i64, i32, vp, i32, vp, i32, vp, i32, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, f32, vp, vp])
     _sig(L, "skein_residual_tanh", i32, [vp, vp, i32, vp, vp, vp, vp, vp, vp, i64, i32, i32, i32, vp])
     _sig(L, "skein_gated_norm", i32, [vp, vp, i64, vp, i32, vp, i64, i32, i32, i32, i32, i32, f32, f32, i32, vp])
     _sig(L, "skein_window_append", i32,
          [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
     _sig(L, "skein_head_append", i32,
-         [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp])
+         [vp, vp, vp, i64, vp, vp, vp, vp, vp, vp, C.POINTER(HeadExtras), i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32,
+          vp])
+    _sig(L, "skein_depth_norm", i32, [C.POINTER(DepthNormParams), i32, vp])
     arule = C.POINTER(AttnRule)
     _sig(L, "skein_window_attn_rows", i32, [vp, i64, vp, vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, i32, i32, arule, i32, vp])
     _sig(L, "skein_attn_decode_window", i32,

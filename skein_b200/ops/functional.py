@@ -286,10 +286,11 @@ def _check_bf16(x):
         raise ValueError("the tensor-core GEMM takes bf16 activations")
 
 
-def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None):
-    """silu(x @ w13[:I].T) * (x @ w13[I:].T) with both products from one pass over x."""
+def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None, glu=None):
+    """silu(x @ w13[:I].T) * (x @ w13[I:].T) with both products from one pass over x; glu (limit, slope): the clamped unit of
+    grouped_linear instead."""
     if not x.is_cuda:
-        return ref.swiglu_linear(x, w13.unpack() if isinstance(w13, PackedWeight) else w13)
+        return ref.swiglu_linear(x, w13.unpack() if isinstance(w13, PackedWeight) else w13, glu)
     _check_act(x)
     T, K = x.shape
     inter = w13.shape[0] // 2
@@ -301,6 +302,8 @@ def swiglu_linear(x, w13, out=None, n_tile=None, _cfg=None):
     p = _base_params(x, wv, out, inter, K, n_tile or pick_n_tile(T, True), 1)
     p.w_rows_per_group, p.w_packed = rows_pg, packed
     p.up_row_off = inter
+    if glu is not None:
+        p.glu, p.glu_limit, p.glu_slope = 1, float(glu[0]), float(glu[1])
     if tc_gemm_ok(x, K):
         _gemm_launch(p, "swiglu_linear", _cfg)
     else:

@@ -38,12 +38,14 @@ class ConvState:
         return 0 if self.tail is None else self.tail.shape[1]
 
 
-def embed_f32(ids, table):
+def embed_f32(ids, table, out=None):
     """Rows of the embedding table as an fp32 residual stream."""
     if not table.is_cuda:
-        return ref.embed(ids, table).float()
+        x = ref.embed(ids, table).float()
+        return x if out is None else out.copy_(x)
     T, C = ids.shape[0], table.shape[1]
-    out = torch.empty(T, C, dtype=torch.float32, device=table.device)
+    if out is None:
+        out = torch.empty(T, C, dtype=torch.float32, device=table.device)
     _lib.check(_lib.lib().skein_embed_f32(ids.data_ptr(), table.data_ptr(), out.data_ptr(), T, C, table.shape[0], _fp32(table),
                                           _lib.stream_ptr()), "embed_f32")
     _lib.count_launch()
@@ -193,14 +195,16 @@ def latent_append(proj, off_kv, q_norm, kv_norm, rot, cos_sin, positions, seq_of
     return cq
 
 
-def head_linear(x, x_cols, w, gate=None):
-    """Per-head product: head h multiplies columns h * x_cols .. + K of x by w[h] [F, K]; results side by side [T, H * F]. `gate`
-    ([T, H * F], rows may be strided): the result is multiplied by its sigmoid."""
+def head_linear(x, x_cols, w, gate=None, out=None):
+    """Per-head product: head h multiplies columns h * x_cols .. + K of x by w[h] [F, K]; results side by side [T, H * F], possibly
+    columns `out` of a wider matrix. `gate` ([T, H * F], rows may be strided): the result is multiplied by its sigmoid."""
     H, Fo, K = w.shape
     if not x.is_cuda:
-        return rl.head_linear(x, x_cols, w, gate)
+        y = rl.head_linear(x, x_cols, w, gate)
+        return y if out is None else out.copy_(y)
     T = x.shape[0]
-    out = torch.empty(T, H * Fo, dtype=x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty(T, H * Fo, dtype=x.dtype, device=x.device)
     if T == 0:
         return out
     tensor_core = F.tc_gemm_ok(x, K) and x.stride(0) % 8 == 0 and x_cols % 8 == 0 and x.data_ptr() % 16 == 0
@@ -209,7 +213,7 @@ def head_linear(x, x_cols, w, gate=None):
         p = F._base_params(x, w, out, Fo, K, F.pick_n_tile(T, False), 0)
         p.X, p.W = x[:, h0 * x_cols:].data_ptr(), w[h0:].data_ptr()
         p.G, p.w_rows_per_group = hn, Fo
-        p.x_ld, p.x_group_cols, p.ldo, p.out_col0, p.out_group_cols = x.stride(0), x_cols, H * Fo, h0 * Fo, Fo
+        p.x_ld, p.x_group_cols, p.ldo, p.out_col0, p.out_group_cols = x.stride(0), x_cols, out.stride(0), h0 * Fo, Fo
         if gate is not None:
             p.gate, p.gate_ld = gate[:, h0 * Fo:].data_ptr(), gate.stride(0)
         if tensor_core:
@@ -226,15 +230,15 @@ def _decode_tc_ok(q_abs, q, D, rot, K, cache) -> bool:
             and hasattr(_lib.lib(), "skein_latent_attn_decode"))
 
 
-def latent_attn_rows(q_abs, q, H, D, rot, scale, cos_sin, positions, seq_of_token, block_table, cache, ctx_hint=1024, splits=None):
+def latent_attn_rows(q_abs, q, H, D, rot, scale, cos_sin, positions, seq_of_token, block_table, cache, ctx_hint=1024, splits=None, sinks=None):
     """Attention of single rows over the latent cache with the key expansion already applied to the queries.
     q_abs [T, H * K]; q [T, >= H * (D + rot)] whose rotated parts are not rotated yet; row t sees positions 0 .. positions[t] of
-    its sequence. Returns the weighted latents [T, H * K]."""
+    its sequence. sinks [H] fp32: head h's denominator has one more term exp(sinks[h]). Returns the weighted latents [T, H * K]."""
     K = cache.shape[2] - rot
     T = q_abs.shape[0]
     if not q_abs.is_cuda:
         return rl.latent_attention_rows(q_abs.view(T, H, K), q[:, :H * (D + rot)].reshape(T, H, D + rot), D, rot, scale, cos_sin, positions,
-                                        seq_of_token, block_table, cache).reshape(T, H * K)
+                                        seq_of_token, block_table, cache, sinks).reshape(T, H * K)
     out = torch.empty(T, H * K, dtype=q_abs.dtype, device=q_abs.device)
     ws = F.workspace()
     L = _lib.lib()
@@ -242,7 +246,7 @@ def latent_attn_rows(q_abs, q, H, D, rot, scale, cos_sin, positions, seq_of_toke
         rc = L.skein_latent_attn_decode(
             q_abs.data_ptr(), q.data_ptr(), q.stride(0), cos_sin.data_ptr(), cos_sin.shape[0], positions.data_ptr(), _lib.ptr(seq_of_token),
             block_table.data_ptr(), block_table.stride(0), cache.data_ptr(), cache.shape[0], cache.shape[1], out.data_ptr(), T, H, D, rot, K,
-            float(scale), int(splits or 0), int(ctx_hint), ws.status.data_ptr(), _lib.stream_ptr())
+            float(scale), _lib.ptr(sinks), int(splits or 0), int(ctx_hint), ws.status.data_ptr(), _lib.stream_ptr())
         if rc != -1:
             _lib.check(rc, "latent_attn_decode")
             _lib.count_launch()
@@ -250,7 +254,7 @@ def latent_attn_rows(q_abs, q, H, D, rot, scale, cos_sin, positions, seq_of_toke
     rc = L.skein_latent_attn_rows(
         q_abs.data_ptr(), q.data_ptr(), q.stride(0), cos_sin.data_ptr(), cos_sin.shape[0], positions.data_ptr(), _lib.ptr(seq_of_token),
         block_table.data_ptr(), block_table.stride(0), cache.data_ptr(), cache.shape[0], cache.shape[1], out.data_ptr(), T, H, D, rot, K,
-        float(scale), ws.status.data_ptr(), _fp32(q_abs), _lib.stream_ptr())
+        float(scale), _lib.ptr(sinks), ws.status.data_ptr(), _fp32(q_abs), _lib.stream_ptr())
     _lib.check(rc, "latent_attn_rows")
     _lib.count_launch()
     return out
@@ -280,16 +284,18 @@ def rope_rows(q, H, D, rot, cos_sin, positions):
     _lib.count_launch()
 
 
-def latent_attn_prefill(q, H, D, rot, V, scale, dense, kv, q_start, q_len, kv_len, dense_start, max_q_len, gate=None):
+def latent_attn_prefill(q, H, D, rot, V, scale, dense, kv, q_start, q_len, kv_len, dense_start, max_q_len, gate=None, sinks=None):
     """Causal attention of prefill chunks with keys and values expanded per head. q [T, >= H * (D + rot)] rotated; dense
     [ctx, K + rot] the step's context rows (rotated key part in the last columns); kv [ctx, H * (D + V)] keys then values.
-    `gate` [T, H * V] (rows may be strided): the output is multiplied by its sigmoid. Returns [T, H * V]."""
+    `gate` [T, H * V] (rows may be strided): the output is multiplied by its sigmoid. sinks [H] fp32: see latent_attn_rows. Returns
+    [T, H * V]."""
     T = q.shape[0]
     out = torch.empty(T, H * V, dtype=q.dtype, device=q.device)
     rc = _lib.lib().skein_latent_attn_prefill(
         q.data_ptr(), q.stride(0), T, dense.data_ptr(), dense.shape[1], kv.data_ptr(), kv.shape[0], _lib.ptr(gate),
         gate.stride(0) if gate is not None else 0, q_start.data_ptr(), q_len.data_ptr(), kv_len.data_ptr(), dense_start.data_ptr(),
-        out.data_ptr(), F.workspace().status.data_ptr(), q_len.shape[0], int(max_q_len), H, D, rot, V, float(scale), _lib.stream_ptr())
+        out.data_ptr(), F.workspace().status.data_ptr(), q_len.shape[0], int(max_q_len), H, D, rot, V, float(scale), _lib.ptr(sinks),
+        _lib.stream_ptr())
     _lib.check(rc, "latent_attn_prefill")
     _lib.count_launch()
     return out

@@ -81,27 +81,48 @@ def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_toke
         _lib.count_launch()
 
 
-def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
-    """Rotation of every head of q (in place) and k, division by its root mean square where the specification asks for it, append of k
-    and v to the cache. q, k, v: columns of one matrix. A head with two maps is two heads here."""
+@dataclass
+class ValueMix:
+    """The first mixing layer's values of the step's tokens, [T, kv_heads * vdim] in the activation type. `keep`: this layer is the first
+    and writes them; otherwise its values become (1 - lam) v + lam v_first."""
+    v_first: torch.Tensor
+    keep: bool
+
+
+def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps, w=None, mix: ValueMix | None = None):
+    """Per head of q (in place) and k: bias, RMS norm with a weight, rotation, division by the root mean square, each where the
+    specification asks for it; bias and mixing of v; append of k and v to the cache. q, k, v: columns of one matrix. A head with two maps is
+    two heads here. w (models/parallel_layers.py: WindowAttnWeights): biases, norm weights, the mixing weight. cos_sin None: no rotation."""
     T = q.shape[0]
     if not q.is_cuda:
-        return rp.head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps)
+        return rp.head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps, w, mix)
     if T:
+        x = _lib.HeadExtras()
+        if spec.bias:
+            x.q_bias, x.k_bias, x.v_bias = w.q_bias.data_ptr(), w.k_bias.data_ptr(), w.v_bias.data_ptr()
+        if spec.head_norm:
+            x.q_norm, x.k_norm = w.q_norm.data_ptr(), w.k_norm.data_ptr()
+        if mix is not None and mix.keep:
+            x.v_keep = mix.v_first.data_ptr()
+        elif mix is not None:
+            x.mix, x.v_first = w.vmix.data_ptr(), mix.v_first.data_ptr()
+        max_pos = cos_sin.shape[0] if cos_sin is not None else block_table.shape[1] * page_size
         _lib.check(_lib.lib().skein_head_append(
-            q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), cos_sin.data_ptr(), positions.data_ptr(), _lib.ptr(seq_of_token),
-            block_table.data_ptr(), cache.data_ptr(), F.workspace().status.data_ptr(), T, spec.heads, spec.kv_heads, spec.dim, spec.maps, spec.vdim,
-            spec.rot_dims, int(spec.interleaved), int(spec.unit), cos_sin.shape[0], block_table.stride(0), cache.shape[0], page_size, float(eps),
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), _lib.ptr(cos_sin), positions.data_ptr(), _lib.ptr(seq_of_token),
+            block_table.data_ptr(), cache.data_ptr(), F.workspace().status.data_ptr(), C.byref(x), T, spec.heads, spec.kv_heads, spec.dim, spec.maps, spec.vdim,
+            spec.rot_dims, int(spec.interleaved), int(spec.unit), max_pos, block_table.stride(0), cache.shape[0], page_size, float(eps),
             _fp32(q), _lib.stream_ptr()), "head_append")
         _lib.count_launch()
 
 
 @dataclass
 class HeadMix:
-    """What follows the softmax of a head: the second map's weight (two maps), the gate, the head norm's eps."""
+    """What belongs to a head's softmax and what follows it: the second map's weight (two maps), the gate, the head norm's eps, the learned
+    sinks."""
     lam: torch.Tensor | None = None
     gate: torch.Tensor | None = None       # [T, heads * vdim], columns of a wider matrix
     eps: float = 0.0
+    sinks: torch.Tensor | None = None      # [heads] fp32
 
 
 def _attn_rule(spec, mix, out_scale) -> "_lib.AttnRule":
@@ -109,6 +130,9 @@ def _attn_rule(spec, mix, out_scale) -> "_lib.AttnRule":
     r = _lib.AttnRule()
     r.window, r.chunk, r.sink, r.maps = spec.window, spec.chunk, int(spec.sink), spec.maps
     r.scale, r.out_scale = float(spec.scale), float(out_scale)
+    r.softcap, r.keep_first = float(spec.softcap), spec.keep_first if spec.window else 0
+    if spec.head_sink:
+        r.sinks = mix.sinks.data_ptr()
     if spec.diff is not None:
         r.lam, r.eps, r.out_scale = mix.lam.data_ptr(), float(mix.eps), float(out_scale) * (1.0 - spec.diff)
     if mix is not None and mix.gate is not None:
@@ -149,7 +173,7 @@ def window_attn(q, spec, inp, cache, page_size, out, out_scale=1.0, mix: HeadMix
             inp.seq_lens.data_ptr(), out.data_ptr(), out.stride(0), ws.status.data_ptr(), inp.q_len.shape[0], int(inp.max_q_len), H, K, KW,
             page_size, bt.stride(0), cache.shape[0], C.byref(r), _lib.stream_ptr())
     else:
-        B, reach = q.shape[0], spec.window or spec.chunk or inp.ctx_hint
+        B, reach = q.shape[0], spec.window + spec.keep_first if spec.window else spec.chunk or inp.ctx_hint
         splits = F.pick_splits(B, K, min(inp.ctx_hint, reach), ws.sm_count)
         scratch = ws.attn_scratch(B, H * spec.maps, K, splits) if splits > 1 else None
         splits, (wsf, ctr) = (splits, scratch) if scratch is not None else (1, (None, None))

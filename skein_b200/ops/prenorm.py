@@ -1,9 +1,12 @@
-"""Operators of pre-norm layers over an fp32 stream: stream sum + RMS norm, and the router that scores every expert by itself.
+"""Operators of pre-norm layers over an fp32 stream: stream sum + RMS norm, average over depth + RMS norm in groups + token shift, and the
+router that scores every expert by itself.
 
 CUDA tensors run csrc/kernels (prenorm.cu, router.cu); CPU tensors run ops/reference_prenorm.py. Activations are bf16, or fp32 when a
 model runs in 32-bit; the stream is fp32.
 """
 from __future__ import annotations
+
+from dataclasses import dataclass
 
 import torch
 
@@ -32,6 +35,36 @@ def add_norm(x, y=None, row_idx=None, row_w=None, step=None, gain=None, eps=0.0,
             _lib.stream_ptr()), "add_norm")
         _lib.count_launch()
     return x_out, act
+
+
+@dataclass
+class TokenShift:
+    """What the mixer of a shifted layer reads: h + (h' - h) mix with h the normed row and h' the previous token's. state [slots, C] fp32 keeps
+    every sequence's last h; position 0 starts from zero whatever the slot holds."""
+    mix: torch.Tensor            # [C] fp32
+    state: torch.Tensor
+
+
+def depth_norm(terms, weights, gain, groups, eps, dtype, x_out=None, shift: TokenShift | None = None, inp=None, slots=None, decode=False):
+    """x = sum_j weights[j] terms[j] (weights None: the one term itself), fp32, into x_out where given; then its RMS norm over `groups` equal
+    parts of a row times gain; then, with `shift`, the token shift over the step's sequences. terms [n, T, C]; returns [T, C] in `dtype`."""
+    n, T, C = terms.shape
+    if not terms.is_cuda:
+        return rn.depth_norm(terms, weights, gain, groups, eps, dtype, x_out, shift, inp, slots, decode)
+    act = torch.empty(T, C, dtype=dtype, device=terms.device)
+    if T:
+        p = _lib.DepthNormParams()
+        p.terms, p.weights, p.x_out, p.gain, p.act_out = terms.data_ptr(), _lib.ptr(weights), _lib.ptr(x_out), gain.data_ptr(), act.data_ptr()
+        p.term_stride, p.n_terms, p.T, p.C, p.groups, p.eps = terms.stride(0), n, T, C, groups, float(eps)
+        p.status = F.workspace().status.data_ptr()
+        if shift is not None:
+            p.shift, p.state, p.num_slots = shift.mix.data_ptr(), shift.state.data_ptr(), shift.state.shape[0]
+            p.positions, p.slots = inp.positions.data_ptr(), slots.data_ptr()
+            if not decode:
+                p.seq_of_token, p.q_start, p.q_len = inp.seq_of_token.data_ptr(), inp.q_start.data_ptr(), inp.q_len.data_ptr()
+        _lib.check(_lib.lib().skein_depth_norm(_lib.byref(p), 1 if dtype == torch.float32 else 0, _lib.stream_ptr()), "depth_norm")
+        _lib.count_launch()
+    return act
 
 
 def _rule(f) -> "_lib.RouteRule":

@@ -20,11 +20,14 @@ def linear(x, w, residual=None, out_f32=False, relu2_cols=0):
     return y if out_f32 else y.to(x.dtype)
 
 
-def swiglu_linear(x, w13):
+def swiglu_linear(x, w13, glu=None):
     """w13 = [gate rows; up rows] stacked along dim 0."""
     inter = w13.shape[0] // 2
     g = x.float() @ w13[:inter].float().t()
     u = x.float() @ w13[inter:].float().t()
+    if glu is not None:
+        from .reference_latent import clamped_glu
+        return clamped_glu(g, u, *glu).to(x.dtype)
     return (torch.nn.functional.silu(g) * u).to(x.dtype)
 
 
@@ -39,12 +42,7 @@ def grouped_linear(xs, w, counts, offsets, swiglu=False, glu=None):
         c, o = counts[e], offsets[e]
         if c == 0:
             continue
-        if glu is not None:
-            from .reference_latent import clamped_glu
-            g, u = (xs[o:o + c].float() @ w[e].float().t()).chunk(2, dim=1)
-            out[o:o + c] = clamped_glu(g, u, *glu).to(xs.dtype)
-        else:
-            out[o:o + c] = swiglu_linear(xs[o:o + c], w[e]) if swiglu else linear(xs[o:o + c], w[e])
+        out[o:o + c] = swiglu_linear(xs[o:o + c], w[e], glu) if swiglu else linear(xs[o:o + c], w[e])
     return out
 
 

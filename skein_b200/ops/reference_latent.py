@@ -82,7 +82,7 @@ def latent_append(proj, off_kv, q_norm, kv_norm, rot, cos_sin, positions, seq_of
     return cq
 
 
-def latent_attention_rows(q_abs, q, D, rot, scale, cos_sin, positions, seq_of_token, block_table, cache):
+def latent_attention_rows(q_abs, q, D, rot, scale, cos_sin, positions, seq_of_token, block_table, cache, sinks=None):
     """q_abs [T, H, K]; q [T, H, D + rot] (rotated part not yet rotated). Returns [T, H, K]."""
     T, H, K = q_abs.shape
     ps = cache.shape[1]
@@ -101,7 +101,9 @@ def latent_attention_rows(q_abs, q, D, rot, scale, cos_sin, positions, seq_of_to
             ctx[seq] = cache[pages].reshape(-1, cache.shape[2]).float()
         kv = ctx[seq][:n]
         s = (q_abs[t].float() @ kv[:, :K].t() + qr[t] @ kv[:, K:].t()) * scale
-        out[t] = (torch.softmax(s, dim=-1) @ kv[:, :K]).to(out.dtype)
+        if sinks is not None:
+            s = torch.cat([s, sinks[:, None]], dim=-1)
+        out[t] = (torch.softmax(s, dim=-1)[:, :n] @ kv[:, :K]).to(out.dtype)
     return out
 
 

@@ -53,13 +53,20 @@ def window_append(q, k, v, q_norm, k_norm, spec, cos_sin, positions, seq_of_toke
         vals[page, :, pos % page_size] = v[t].view(spec.kv_heads, -1)
 
 
-def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps):
+def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, cache, page_size, eps, w=None, mix=None):
     D, W = spec.dim, spec.key_width
     keys, vals = _pages(cache, spec.kv_heads, page_size, W, spec.vdim)
 
-    def turn(z, cs):
-        z = z.float().view(-1, D)
-        if spec.interleaved:
+    def turn(z, cs, bias, norm):
+        z = z.float()
+        if bias is not None:
+            z = z + bias
+        z = z.view(-1, D)
+        if norm is not None:
+            z = z / torch.sqrt(z.pow(2).mean(-1, keepdim=True) + eps) * norm
+        if cs is None:
+            pass
+        elif spec.interleaved:
             z = torch.cat([rotate_pairs(z[:, :spec.rot_dims], cs), z[:, spec.rot_dims:]], dim=1)
         else:
             z = _rotate(z[None], cs, spec.rot_dims)[0]
@@ -68,11 +75,18 @@ def head_append(q, k, v, spec, cos_sin, positions, seq_of_token, block_table, ca
         pos = int(positions[t])
         if pos < 0:
             continue
-        cs = cos_sin[pos:pos + 1]
-        q[t] = turn(q[t], cs).reshape(-1).to(q.dtype)
+        cs = cos_sin[pos:pos + 1] if cos_sin is not None else None
+        qb, kb, vb = (w.q_bias, w.k_bias, w.v_bias) if spec.bias else (None, None, None)
+        qn, kn = (w.q_norm, w.k_norm) if spec.head_norm else (None, None)
+        q[t] = turn(q[t], cs, qb, qn).reshape(-1).to(q.dtype)
         page = int(block_table[int(seq_of_token[t]) if seq_of_token is not None else t, pos // page_size])
-        keys[page, :, pos % page_size] = turn(k[t], cs).view(spec.kv_heads, W).to(cache.dtype)
-        vals[page, :, pos % page_size] = v[t].view(spec.kv_heads, -1)
+        keys[page, :, pos % page_size] = turn(k[t], cs, kb, kn).view(spec.kv_heads, W).to(cache.dtype)
+        x = v[t].float() + (vb if vb is not None else 0.0)
+        if mix is not None and mix.keep:
+            mix.v_first[t] = x.to(v.dtype)
+        elif mix is not None:
+            x = (1.0 - w.vmix) * x + w.vmix * mix.v_first[t].float()
+        vals[page, :, pos % page_size] = x.to(cache.dtype).view(spec.kv_heads, -1)
 
 
 def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_size, out_scale, mix=None):
@@ -85,13 +99,18 @@ def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_
         if pos < 0:
             continue
         lo = pos // spec.chunk * spec.chunk if spec.chunk else max(0, pos - spec.window + 1) if spec.window else 0
-        js = torch.arange(lo, pos + 1)
+        kept = min(spec.keep_first, lo) if spec.window else 0
+        js = torch.cat([torch.arange(kept), torch.arange(lo, pos + 1)])
         pages = block_table[int(seq_of_token[t]) if seq_of_token is not None else t][js // page_size].long()
         k = keys[pages, :, js % page_size].float().view(-1, spec.kv_heads, M, D).repeat_interleave(G, dim=1)
         v = vals[pages, :, js % page_size].float().repeat_interleave(G, dim=1)
         s = torch.einsum("hmd,jhmd->hmj", q[t].float().view(H, M, D), k) * spec.scale
+        if spec.softcap:
+            s = spec.softcap * torch.tanh(s / spec.softcap)
         if spec.sink:
             s = torch.cat([s, torch.zeros(H, M, 1)], dim=-1)
+        if spec.head_sink:
+            s = torch.cat([s, mix.sinks.view(H, 1, 1).expand(H, M, 1)], dim=-1)
         p = torch.softmax(s, dim=-1)[..., :len(js)]
         a = torch.einsum("hmj,jhv->hmv", p, v)
         o = a[:, 0]
@@ -105,7 +124,7 @@ def window_attn_rows(q, spec, positions, seq_of_token, block_table, cache, page_
     return out
 
 
-def rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len):
+def rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len, step=None):
     H, G, D, V, taps = spec.heads, spec.groups, spec.dim, spec.vdim, spec.taps
     dt = row.dtype
     out = torch.zeros(row.shape[0], H * V, dtype=dt)
@@ -128,20 +147,23 @@ def rec_chunk(row, cols, spec, w, state, positions, slots, q_start, q_len):
             x = sum(w.conv[j] * full[j:j + n] for j in range(taps)) + (w.conv_b if w.conv_b is not None else 0.0)
         x = torch.nn.functional.silu(x).to(dt).float()
         q, k, v = x[:, :G * D].view(n, G, D), x[:, G * D:2 * G * D].view(n, G, D), x[:, 2 * G * D:].view(n, H, V)
-        if spec.kind == "delta":
+        if spec.corrects:
             q, k = (z / torch.sqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6) for z in (q, k))
             q = q * D ** -0.5
         q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)
         if spec.kind == "lightning":
             g, coef = (w.neg_decay.exp() if w.decay is None else w.decay).expand(n, H), torch.ones(n, H)
+        elif spec.kind == "channel_delta":
+            a = torch.nn.functional.softplus(step[t0:t0 + n] + w.dt_bias, threshold=60.0).view(n, H, D)
+            g, coef = (w.neg_decay[:, None] * a).exp(), torch.sigmoid(r[:, cols.b:cols.b + H])
         else:
             step = torch.nn.functional.softplus(r[:, cols.a:cols.a + H] + w.dt_bias, threshold=60.0)
             g = (w.neg_decay * step).exp()
             coef = torch.sigmoid(r[:, cols.b:cols.b + H]) if spec.kind == "delta" else step
         S = state.mat[slot].clone() if pos0 > 0 else torch.zeros(H, D, V)
         for t in range(n):
-            S = g[t][:, None, None] * S
-            u = v[t] - torch.einsum("hdv,hd->hv", S, k[t]) if spec.kind == "delta" else v[t]
+            S = g[t].view(H, -1, 1) * S
+            u = v[t] - torch.einsum("hdv,hd->hv", S, k[t]) if spec.corrects else v[t]
             S = S + k[t][:, :, None] * (coef[t][:, None] * u)[:, None, :]
             o = torch.einsum("hdv,hd->hv", S, q[t])
             if w.skip is not None:

@@ -14,6 +14,29 @@ def add_norm(x, y, row_idx, row_w, step, gain, eps, dtype):
     return a, None if gain is None else (a / torch.sqrt(a.pow(2).mean(-1, keepdim=True) + eps) * gain).to(dtype)
 
 
+def depth_norm(terms, weights, gain, groups, eps, dtype, x_out, shift, inp, slots, decode):
+    x = terms[0] if weights is None else sum(weights[j] * terms[j] for j in range(terms.shape[0]))
+    if x_out is not None:
+        x_out.copy_(x)
+    T, C = x.shape
+    v = x.view(T, groups, C // groups)
+    h = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, C) * gain
+    if shift is None:
+        return h.to(dtype)
+    out = h.clone()
+    n = inp.seq_lens.shape[0]
+    starts, lens = (range(n), [1] * n) if decode else (inp.q_start.tolist(), inp.q_len.tolist())
+    for s, (t0, m) in enumerate(zip(starts, lens)):
+        if m < 1 or int(inp.positions[t0]) < 0:
+            continue
+        before = shift.state[int(slots[s])].clone() if int(inp.positions[t0]) > 0 else torch.zeros(C)
+        for t in range(t0, t0 + m):
+            out[t] = h[t] + (before - h[t]) * shift.mix
+            before = h[t]
+        shift.state[int(slots[s])] = before
+    return out.to(dtype)
+
+
 def select(logits, f):
     """(ids int32 [T, top], weights fp32) by the rule of `f`."""
     T, E = logits.shape

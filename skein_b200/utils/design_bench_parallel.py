@@ -118,7 +118,7 @@ def decode_kernels(new, near, B=64, ctx=640):
             col, width = _columns(r)
             row, w, st = _bf(B, width, std=1.0), _rec_weights(r), rec.RecState.make(r, B, torch.bfloat16, "cuda")
             cols, pos, slots, out = rec.RecColumns.of(r, col), pos1(ctx), torch.arange(B, dtype=torch.int32, device="cuda"), _bf(B, r.out_width)
-            gate = rec.HeadGate(w.norm, col["g"], out, 1e-5) if r.kind == "delta" else None
+            gate = rec.HeadGate(w.norm, row[:, col["g"]:col["g"] + r.out_width], out, 1e-5) if r.kind == "delta" else None
             by = B * (8 * r.state_elems + 2 * (r.conv_channels * (1 + r.conv_rows) + r.out_width * 2))
             return lambda: rec.rec_step(row, cols, r, w, st, pos, slots, gate), by, 6 * B * r.state_elems
         return make
