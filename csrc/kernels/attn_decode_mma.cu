@@ -14,6 +14,8 @@
 //   memory; with splits > 1 the CTA parks its state in a workspace and the last CTA of a
 //   (sequence, kv head) to arrive merges the splits, as in the scalar kernel.
 //
+// Under a rule (SkeinAttnRule) the tiles are those of the window and, in front of them, those of the first tokens that it keeps in sight.
+//
 // Differential heads (SkeinAttnRule.maps == 2): a key head holds its two maps side by side in the 128 columns. Each map of a query head is
 // a row of the tile whose other half is zero, so that one product gives the scores of both maps; the maps of a head are subtracted, normed
 // and gated where the rows are merged.
@@ -53,7 +55,7 @@ struct AttnMmaParams {
   int* status;
   long long q_stride;
   int B, Hq, Hkv, G, page_size, max_blocks, num_pages, splits;   // Hq, G: query rows, the maps of differential heads counted apart
-  float scale_log2e;
+  float scale_log2e, cap_in, cap_log2e;      // (cap_log2e 0: scores are not capped; attn_cap)
   // optional fusion of RoPE and the KV append of the new token (cos_sin == nullptr: q is already rotated and
   // the cache already holds the token). q then points at the raw fused q/k/v projection rows
   // [B, q_stride >= (Hq + 2 * Hkv) * D]: q heads, k heads, v heads.
@@ -63,13 +65,6 @@ struct AttnMmaParams {
   long long out_ld;         // elements between rows of out
   SkeinAttnRule r;
 };
-
-// softmax sums (reference m in base 2, denominator l) -> factor that normalises the weighted values
-__device__ __forceinline__ float am_norm(float m, float l, int sink) {
-  if (!sink) return l > 0.f ? 1.f / l : 0.f;
-  const float top = fmaxf(m, 0.f), e = exp2f(m - top);
-  return e / (l * e + exp2f(-top));
-}
 
 template <int AM_D>
 __device__ __forceinline__ uint32_t am_swz(int row, int chunk) {  // byte offset in a [16][AM_D] bf16 tile
@@ -114,17 +109,22 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   const int G = p.G, ps = p.page_size;
   const int len = p.seq_lens[b];
 
-  // this split's token range, rounded to whole pages (pages are multiples of the tile), with a window to whole tiles
-  const int lo = len > 0 ? attn_first_key(p.r.window, p.r.chunk, len - 1) : 0;     // first visible token
-  const int base = lo / AM_TILE * AM_TILE, unit = p.r.window > 0 || p.r.chunk > 0 ? AM_TILE : ps;
-  int per = (len - base + p.splits - 1) / p.splits;
+  // The visible tiles in a row: those of the kept first tokens, then from the window's first one on. This split's range of the row is
+  // rounded to whole pages (pages are multiples of the tile), with a window to whole tiles.
+  const int lo = len > 0 ? attn_first_key(p.r.window, p.r.chunk, len - 1) : 0;     // first visible token, the kept ones apart
+  const int keep = p.r.keep_first, tile_lo = lo / AM_TILE, unit = p.r.window > 0 || p.r.chunk > 0 ? AM_TILE : ps;
+  const int kept = min((keep + AM_TILE - 1) / AM_TILE, tile_lo), hop = tile_lo - kept;     // tiles of the first tokens; skipped behind them
+  const int row_len = len - hop * AM_TILE;
+  int per = (row_len + p.splits - 1) / p.splits;
   per = (per + unit - 1) / unit * unit;
-  const int t_begin = base + split * per;
-  int t_end = t_begin + per;
-  if (t_end > len) t_end = len;
+  const int t_begin = split * per, t_end = min(t_begin + per, row_len);
   const int tile_begin = t_begin / AM_TILE;
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + AM_TILE - 1) / AM_TILE : 0;
   const int n_my = n_tiles > warp ? (n_tiles - warp + AM_WARPS - 1) / AM_WARPS : 0;   // tiles of this warp
+  auto tile_of = [&](int j) {      // this warp's j-th tile
+    const int t = tile_begin + warp + j * AM_WARPS;
+    return t < kept ? t : t + hop;
+  };
 
   uint8_t* q_s = am_smem + AM_WARPS * AM_WARP_BYTES;
   const uint32_t q_base = smem_u32(q_s);
@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     const int j = j0 + lane;
     int pg = 0;
     if (j < n_my) {
-      const int tile = tile_begin + warp + j * AM_WARPS;
+      const int tile = tile_of(j);
       pg = p.block_table[(size_t)b * p.max_blocks + (tile * AM_TILE) / ps];
       if (pg < 0 || pg >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, pg); pg = 0; }
     }
@@ -219,15 +219,14 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     if (j < n_my) {
       if ((j & 31) == 0) load_pages(j);
       const int pg = __shfl_sync(0xffffffffu, pg_block, j & 31);
-      const int tile = tile_begin + warp + j * AM_WARPS;
-      const int tok0 = tile * AM_TILE;
+      const int tok0 = tile_of(j) * AM_TILE;
       const __nv_bfloat16* kp = p.kv + ((size_t)pg * 2 * p.Hkv + kvh) * head_stride + (size_t)(tok0 % ps) * AM_D;
       const __nv_bfloat16* vp = kp + (size_t)p.Hkv * head_stride;
       const uint32_t dst = st_base + (j % AM_STAGES) * AM_STAGE_BYTES;
 #pragma unroll
       for (int i = 0; i < AM_TILE * CH / 32; ++i) {
         const int c = lane + 32 * i, r = c / CH, ch = c % CH;
-        const int nbytes = (tok0 + r < t_end) ? 16 : 0;
+        const int nbytes = (tok0 + r < len) ? 16 : 0;
         am_cp_async(dst + am_swz<AM_D>(r, ch), kp + r * AM_D + ch * 8, nbytes);
         am_cp_async(dst + AM_TILE_BYTES + am_swz<AM_D>(r, ch), vp + r * AM_D + ch * 8, nbytes);
       }
@@ -242,7 +241,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
     __syncwarp();               // ... and every lane's; all lanes are also done with tile j-1
     issue(j + AM_STAGES - 1);   // refills the stage tile j-1 used
     const uint32_t kb = st_base + (j % AM_STAGES) * AM_STAGE_BYTES, vb = kb + AM_TILE_BYTES;
-    const int tok0 = (tile_begin + warp + j * AM_WARPS) * AM_TILE;
+    const int tok0 = tile_of(j) * AM_TILE;
 
     // ---- S = Q K^T (16 rows x 16 tokens) ----
     float s[2][4];
@@ -261,10 +260,18 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
 #pragma unroll
     for (int nb = 0; nb < 2; ++nb) {
       const int col = tok0 + nb * 8 + (lane & 3) * 2;
-      s[nb][0] = (col < t_end && col >= lo) ? s[nb][0] * p.scale_log2e : -INFINITY;
-      s[nb][1] = (col + 1 < t_end && col + 1 >= lo) ? s[nb][1] * p.scale_log2e : -INFINITY;
-      s[nb][2] = (col < t_end && col >= lo) ? s[nb][2] * p.scale_log2e : -INFINITY;
-      s[nb][3] = (col + 1 < t_end && col + 1 >= lo) ? s[nb][3] * p.scale_log2e : -INFINITY;
+      const bool see0 = col < len && (col >= lo || col < keep), see1 = col + 1 < len && (col + 1 >= lo || col + 1 < keep);
+      if (p.cap_log2e > 0.f) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[nb][i] = attn_cap(s[nb][i], p.cap_in, p.cap_log2e);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[nb][i] *= p.scale_log2e;
+      }
+      s[nb][0] = see0 ? s[nb][0] : -INFINITY;
+      s[nb][1] = see1 ? s[nb][1] : -INFINITY;
+      s[nb][2] = see0 ? s[nb][2] : -INFINITY;
+      s[nb][3] = see1 ? s[nb][3] : -INFINITY;
       mx0 = fmaxf(mx0, fmaxf(s[nb][0], s[nb][1]));
       mx1 = fmaxf(mx1, fmaxf(s[nb][2], s[nb][3]));
     }
@@ -327,6 +334,8 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   }
   __syncthreads();
 
+  auto sink_of = [&](int g) { return attn_sink_log2(p.r, (kvh * G + g) / p.r.maps); };
+
   // two maps: thread d's values of the rows (normalised) -> difference, head norm, gate
   auto store_pairs = [&](auto value) {
     __shared__ float red[AM_WARPS][8];
@@ -379,12 +388,12 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
   }
   if (p.splits == 1) {
     if (AM_D == AM_THREADS && p.r.maps == 2) {
-      store_pairs([&](int g) { return O_g[g] * am_norm(M_g[g], L_g[g], p.r.sink); });
+      store_pairs([&](int g) { return O_g[g] * attn_norm(M_g[g], L_g[g], sink_of(g)); });
       return;
     }
 #pragma unroll
     for (int g = 0; g < 16; ++g)
-      if (g < G) p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(O_g[g] * am_norm(M_g[g], L_g[g], p.r.sink) * p.r.out_scale);
+      if (g < G) p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(O_g[g] * attn_norm(M_g[g], L_g[g], sink_of(g)) * p.r.out_scale);
     return;
   }
 #pragma unroll
@@ -430,7 +439,7 @@ __global__ void __launch_bounds__(AM_THREADS) attn_decode_mma_kernel(const AttnM
         O += w * ov[s2];
       }
     }
-    const float a = O * am_norm(M, L, p.r.sink);
+    const float a = O * attn_norm(M, L, sink_of(g));
     if (AM_D == AM_THREADS && p.r.maps == 2) val_s[g * AM_D + d] = a;
     else p.out[(size_t)b * p.out_ld + (size_t)(kvh * G + g) * AM_D + d] = __float2bfloat16(a * p.r.out_scale);
   }
@@ -488,6 +497,8 @@ static int attn_decode_mma_launch(const void* q, long long q_stride, void* kv, c
   p.counters = counters; p.status = status; p.q_stride = q_stride;
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.page_size = page_size; p.max_blocks = max_blocks; p.num_pages = num_pages;
   p.splits = splits; p.scale_log2e = rule.scale * 1.4426950408889634f;
+  p.cap_log2e = rule.softcap * 1.4426950408889634f;
+  p.cap_in = rule.softcap > 0.f ? 2.f * p.scale_log2e / rule.softcap : 0.f;
   return D == 64 ? attn_decode_mma_go<64>(p, ws, stream) : attn_decode_mma_go<128>(p, ws, stream);
 }
 

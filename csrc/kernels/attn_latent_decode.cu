@@ -19,6 +19,7 @@
 //
 // q_abs holds the queries with the key expansion already applied; the rotated query part is rotated here, on its way to shared
 // memory.
+#include "attn_rule.cuh"
 #include "ptx.cuh"
 #include "launch.cuh"
 #include <cuda.h>
@@ -49,6 +50,7 @@ struct LatentDecodeParams {
   const int* block_table;
   __nv_bfloat16* out;           // [T, H * K]
   int* status;
+  const float* sinks;           // [H] one more term exp(sinks[h]) in head h's denominator, or null
   long long q_ld;
   float scale_log2e;
   int H, D, rot, K, max_pos, max_blocks, num_pages, page_size, splits, nch, box_rows;
@@ -440,7 +442,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) attn_latent_decode_kernel(const
     float w = mc == -INFINITY ? 0.f : exp2f(mc - M), L = w * lc;
 #pragma unroll
     for (int o = LD_MAX_SPLITS / 2; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
-    w = L > 0.f ? w / L : 0.f;
+    w *= attn_norm(M, L, attn_sink_log2(p.sinks, h));
     __nv_bfloat16* orow = p.out + (size_t)t * p.H * K + (size_t)h * K;
     for (int c0 = 0; c0 < K; c0 += 512) {            // four groups of 4 columns per lane in flight
       float4 acc[4];
@@ -508,7 +510,7 @@ static int latent_decode_launch(const CUtensorMap& tm, LatentDecodeParams& p, in
 extern "C" int skein_latent_attn_decode(const void* q_abs, const void* q, long long q_ld, const float* cos_sin, int max_pos,
                                         const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
                                         const void* cache, int num_pages, int page_size, void* out, int T, int H, int D, int rot, int kv_rank,
-                                        float scale, int splits, int ctx_hint, int* status, void* stream) {
+                                        float scale, const float* sinks, int splits, int ctx_hint, int* status, void* stream) {
   using namespace skein;
   if (T == 0) return 0;
   if (kv_rank % 8 || rot % 8 || kv_rank < 8 || kv_rank > 512 || rot < 8 || T > 65535 || scale <= 0.f) return -1;
@@ -516,6 +518,7 @@ extern "C" int skein_latent_attn_decode(const void* q_abs, const void* q, long l
   LatentDecodeParams p;
   p.q_abs = (const __nv_bfloat16*)q_abs; p.q = (const __nv_bfloat16*)q; p.cos_sin = cos_sin; p.positions = positions;
   p.seq_of_token = seq_of_token; p.block_table = block_table; p.out = (__nv_bfloat16*)out; p.status = status; p.q_ld = q_ld;
+  p.sinks = sinks;
   p.scale_log2e = scale * 1.4426950408889634f;
   p.H = H; p.D = D; p.rot = rot; p.K = kv_rank; p.max_pos = max_pos; p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size;
   p.nch = (kv_rank + rot + 63) / 64;

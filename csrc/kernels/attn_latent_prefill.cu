@@ -15,6 +15,7 @@
 //
 // S0 | S1 | O0 | O1 take all 512 tensor-memory columns, Q, K and V up to 176 KB of shared memory: one CTA per SM. Every wait is
 // bounded; on expiry the CTA records a status code, waits for its copies in flight, frees its tensor memory and returns.
+#include "attn_rule.cuh"
 #include "ptx.cuh"
 #include "launch.cuh"
 #include <cuda.h>
@@ -39,6 +40,7 @@ struct LatentPrefillParams {
   const int* ctx_start;     // [S] first context row of the sequence
   const __nv_bfloat16* gate;
   __nv_bfloat16* out;       // [T, H * V]
+  const float* sinks;       // [H] one more term exp(sinks[h]) in head h's denominator, or null
   int* status;
   int gate_ld;
   int H, D, rot, V, kv_rank;
@@ -274,7 +276,7 @@ attn_latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     if (n_tiles > 0) {
       if (ok && mbar_wait(bar_o + 8 * t, (n_tiles - 1) & 1, abort_flag, LP_BUDGET_NS)) {
         tc_fence_after();
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        const float inv = attn_norm(m, l, attn_sink_log2(p.sinks, head));
         const bool store = row0 + r < qlen;
         const size_t row = (size_t)(qrow0 + row0 + r);
         __nv_bfloat16* orow = p.out + row * ((size_t)p.H * p.V) + (size_t)head * p.V;
@@ -330,14 +332,14 @@ attn_latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 extern "C" int skein_latent_attn_prefill(const void* q, long long q_ld, int q_rows, const void* dense, int L, const void* kv, int ctx_rows,
                                          const void* gate, int gate_ld, const int* q_start, const int* q_len, const int* kv_len,
                                          const int* ctx_start, void* out, int* status, int S, int max_q_len, int H, int D, int rot, int V,
-                                         float scale, void* stream) {
+                                         float scale, const float* sinks, void* stream) {
   using namespace skein;
   if (S == 0 || max_q_len == 0) return 0;
   if (D < 1 || D > 128 || V < 1 || V > 128 || rot < 1 || rot > 64 || D % 8 || V % 8 || rot % 8 || q_ld % 8 || L % 8 || L <= rot || scale <= 0.f) return -1;
   if (gate != nullptr && (gate_ld % 8 || ((uintptr_t)gate & 15))) return -1;
   LatentPrefillParams p;
   p.q_start = q_start; p.q_len = q_len; p.kv_len = kv_len; p.ctx_start = ctx_start; p.gate = (const __nv_bfloat16*)gate;
-  p.out = (__nv_bfloat16*)out; p.status = status; p.gate_ld = gate_ld; p.H = H; p.D = D; p.rot = rot; p.V = V; p.kv_rank = L - rot;
+  p.out = (__nv_bfloat16*)out; p.sinks = sinks; p.status = status; p.gate_ld = gate_ld; p.H = H; p.D = D; p.rot = rot; p.V = V; p.kv_rank = L - rot;
   p.dc = (D + 63) / 64; p.vc = (V + 63) / 64; p.scale_log2e = scale * 1.4426950408889634f;
   CUtensorMap tmQ, tmK, tmR, tmV;
   int rc = cached_tmap_heads(&tmQ, q, q_rows, H, D + rot, D + rot, q_ld, LP_BM);

@@ -3,7 +3,7 @@
 // new tokens attends to the kv_len tokens already in the cache, its own included); this is the kernel the prefill
 // path runs for head sizes 128 and 64 and pages of whole 16-token groups, the mma.sync kernel stays as the fallback for other
 // shapes. With a window or chunks (SkeinAttnRule) a row sees part of the keys before it only; tiles before the first key of a CTA's first
-// row are skipped.
+// row are skipped, but for those of the first tokens that the window keeps in sight.
 //
 // Differential heads (two maps over the same values, side by side in the 128 columns of a query or key head): the tile's 128 rows are two
 // maps of 64 query rows, each with the other map's half set to zero, so that one product gives both maps' scores; at the end the rows of
@@ -57,13 +57,13 @@ struct AttnPrefillTcParams {
   int* status;
   int Hq, Hkv, max_blocks, num_pages, page_size;
   long long out_ld;         // elements between rows of out
-  float scale_log2e;
+  float scale_log2e, cap_in, cap_log2e;      // (cap_log2e 0: scores are not capped; attn_cap)
   SkeinAttnRule r;
 };
 
 constexpr int TC_X_LD = 132;            // floats between rows of the second map's outputs in shared memory
 
-template <int TC_D, int MAPS>
+template <int TC_D, int MAPS, bool CAP>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        const AttnPrefillTcParams p) {
@@ -83,8 +83,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (kv_hi > kvlen) kv_hi = kvlen;
   const int kv_lo = attn_first_key(p.r.window, p.r.chunk, pos0 + q0);                    // first key of the first row
   const int last_lo = attn_first_key(p.r.window, p.r.chunk, pos0 + q0 + QR - 1);         // ... and of the last
+  const int keep = p.r.keep_first;
   const int first_tile = kv_lo / TC_BN;
-  const int n_tiles = (kv_hi + TC_BN - 1) / TC_BN - first_tile;
+  const int kept = min((keep + TC_BN - 1) / TC_BN, first_tile);                          // tiles of the kept first tokens ...
+  const int n_tiles = (kv_hi + TC_BN - 1) / TC_BN - first_tile + kept;                   // ... in front of the window's
+  auto tile_at = [&](int j) { return j < kept ? j : first_tile + j - kept; };
+  // tokens of tile j that some row sees, counted from its first
+  auto tile_len = [&](int j) { return min(j < kept ? keep : kv_hi, (tile_at(j) + 1) * TC_BN) - tile_at(j) * TC_BN; };
 
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -133,8 +138,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       bool ok = true;
       int armed_k = 0, armed_v = 0;      // phases armed so far (for the bounded drain on an early exit)
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int n0 = (first_tile + j) * TC_BN;
-        const int n_pages = (min(kv_hi, n0 + TC_BN) - n0 + TC_PS - 1) / TC_PS;      // 16-token boxes
+        const int n0 = tile_at(j) * TC_BN;
+        const int n_pages = (tile_len(j) + TC_PS - 1) / TC_PS;      // 16-token boxes
         const int* bt = p.block_table + (size_t)seq * p.max_blocks;
         for (int kv01 = 0; kv01 < 2 && ok; ++kv01) {
           const uint32_t full = kv01 ? bar_vfull : bar_kfull, empty = kv01 ? bar_vempty : bar_kempty;
@@ -177,8 +182,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         if (!mbar_wait(bar_pfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
         if (!mbar_wait(bar_vfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
         tc_fence_after();
-        const int n_valid = min(kv_hi, (first_tile + j + 1) * TC_BN) - (first_tile + j) * TC_BN;
-        const int k_steps = (n_valid + 15) / 16;               // 16-token steps that hold at least one visible key
+        const int k_steps = (tile_len(j) + 15) / 16;               // 16-token steps that hold at least one visible key
         for (int k = 0; k < k_steps; ++k)
           mma_f16_ts(tm_o, tm_p + k * 8, umma_desc_sw128_mn(v_s + k * 16 * 128, TC_HALF_BYTES), idesc_o,
                      (j > 0 || k > 0) ? 1u : 0u);
@@ -199,13 +203,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
-      const int n0 = (first_tile + j) * TC_BN;
+      const int n0 = tile_at(j) * TC_BN;
       if (!mbar_wait(bar_sfull, j & 1, abort_flag, TC_BUDGET_NS)) { ok = false; break; }
       tc_fence_after();
       // some row of the tile sees only part of these keys (the tile's last row has the latest window)
-      const bool masked = n0 + TC_BN - 1 > pos0 + q0 || n0 < last_lo;
-      const int limit = pos_r - n0;                     // this row sees columns first .. limit of the tile
-      const int first = first_key - n0;
+      const bool masked = n0 + TC_BN - 1 > pos0 + q0 || (n0 < last_lo && n0 + TC_BN > keep);
+      const int limit = pos_r - n0;                     // this row sees columns first .. limit of the tile, and those before `until`
+      const int first = first_key - n0, until = keep - n0;
+      auto seen = [&](int c) { return c <= limit && (c >= first || c < until); };
       // pass 1: row maximum of the raw scores (64 columns per round: both loads in flight before the wait)
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -216,13 +221,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld_wait();
         if (masked) {
 #pragma unroll
-          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], (h * 64 + i <= limit && h * 64 + i >= first) ? __uint_as_float(sv[i]) : -INFINITY);
+          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], seen(h * 64 + i) ? __uint_as_float(sv[i]) : -INFINITY);
         } else {
 #pragma unroll
           for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[i]));
         }
       }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2e;    // the scale is positive
+      const float raw = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));                   // the scale is positive, the cap monotonic
+      const float mx = CAP ? (raw == -INFINITY ? raw : attn_cap(raw, p.cap_in, p.cap_log2e)) : raw * p.scale_log2e;
       // The running maximum only moves when the tile's maximum exceeds it by more than 2^8: until then the
       // probabilities of this tile are at most 256 (exact in bf16 and harmless in the fp32 sums), and O needs no
       // rescaling; the final division by the row sum undoes whatever reference the row ended on.
@@ -260,11 +266,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         uint32_t pk[32];
 #pragma unroll
         for (int i = 0; i < 64; i += 2) {
-          float x0 = fmaf(__uint_as_float(sv[i]), p.scale_log2e, -ref);
-          float x1 = fmaf(__uint_as_float(sv[i + 1]), p.scale_log2e, -ref);
+          float x0, x1;
+          if (CAP) {
+            x0 = attn_cap(__uint_as_float(sv[i]), p.cap_in, p.cap_log2e) - ref;
+            x1 = attn_cap(__uint_as_float(sv[i + 1]), p.cap_in, p.cap_log2e) - ref;
+          } else {
+            x0 = fmaf(__uint_as_float(sv[i]), p.scale_log2e, -ref);
+            x1 = fmaf(__uint_as_float(sv[i + 1]), p.scale_log2e, -ref);
+          }
           if (masked) {
-            if (h * 64 + i > limit || h * 64 + i < first) x0 = -INFINITY;
-            if (h * 64 + i + 1 > limit || h * 64 + i + 1 < first) x1 = -INFINITY;
+            if (!seen(h * 64 + i)) x0 = -INFINITY;
+            if (!seen(h * 64 + i + 1)) x1 = -INFINITY;
           }
           const float p0 = exp2f(x0), p1 = exp2f(x1);
           // the row sum is taken over the rounded values, the ones the tensor cores multiply
@@ -298,11 +310,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       mbar_arrive(bar_pfull);
     }
     const bool done = ok && mbar_wait(bar_odone, (n_tiles - 1) & 1, abort_flag, TC_BUDGET_NS);
-    float inv = l > 0.f ? 1.f / l : 0.f;
-    if (p.r.sink) {
-      const float top = fmaxf(m, 0.f), e = exp2f(m - top);
-      inv = e / (l * e + exp2f(-top));
-    }
+    float inv = attn_norm(m, l, attn_sink_log2(p.r, head));
     const bool store = q0 + qi < qlen;
     if (MAPS == 2) {
       // every copy and product of this CTA is complete: the K and V buffers take the second map's outputs
@@ -403,12 +411,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 namespace skein {
 
-template <int TC_D, int MAPS>
+template <int TC_D, int MAPS, bool CAP>
 static int attn_prefill_tc_go(const void* q, long long q_stride, long long q_rows, const void* kv, const AttnPrefillTcParams& p, int S, int max_q_len,
                               void* stream) {
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<TC_D, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(TC_D));
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<TC_D, MAPS, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(TC_D));
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
@@ -418,7 +426,7 @@ static int attn_prefill_tc_go(const void* q, long long q_stride, long long q_row
   rc = cached_tmap_2d(&tmKV, kv, (uint64_t)p.num_pages * 2 * p.Hkv * p.page_size, TC_D, 2, TC_PS);
   if (rc != 0) return rc;
   dim3 grid((max_q_len + TC_BM / MAPS - 1) / (TC_BM / MAPS), p.Hq, S);
-  attn_prefill_tc_kernel<TC_D, MAPS><<<grid, TC_THREADS, tc_smem(TC_D), (cudaStream_t)stream>>>(tmQ, tmKV, p);
+  attn_prefill_tc_kernel<TC_D, MAPS, CAP><<<grid, TC_THREADS, tc_smem(TC_D), (cudaStream_t)stream>>>(tmQ, tmKV, p);
   return (int)cudaGetLastError();
 }
 
@@ -441,9 +449,12 @@ extern "C" int skein_attn_prefill_window(const void* q, long long q_stride, long
   p.out = (__nv_bfloat16*)out; p.status = status; p.out_ld = out_ld; p.r = *rule;
   p.Hq = Hq; p.Hkv = Hkv; p.max_blocks = max_blocks; p.num_pages = num_pages; p.page_size = page_size;
   p.scale_log2e = rule->scale * 1.4426950408889634f;
-  if (rule->maps == 2) return attn_prefill_tc_go<128, 2>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
-  return D == 64 ? attn_prefill_tc_go<64, 1>(q, q_stride, q_rows, kv, p, S, max_q_len, stream)
-                 : attn_prefill_tc_go<128, 1>(q, q_stride, q_rows, kv, p, S, max_q_len, stream);
+  p.cap_log2e = rule->softcap * 1.4426950408889634f;
+  p.cap_in = rule->softcap > 0.f ? 2.f * p.scale_log2e / rule->softcap : 0.f;
+  auto go = [&](auto fn) { return fn(q, q_stride, q_rows, kv, p, S, max_q_len, stream); };
+  if (rule->maps == 2) return rule->softcap > 0.f ? -1 : go(attn_prefill_tc_go<128, 2, false>);
+  if (rule->softcap > 0.f) return D == 64 ? go(attn_prefill_tc_go<64, 1, true>) : go(attn_prefill_tc_go<128, 1, true>);
+  return D == 64 ? go(attn_prefill_tc_go<64, 1, false>) : go(attn_prefill_tc_go<128, 1, false>);
 }
 
 extern "C" int skein_attn_prefill_tc(const void* q, long long q_stride, long long q_rows, const void* kv, const int* block_table,

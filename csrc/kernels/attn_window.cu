@@ -4,8 +4,9 @@
 //   window_append     per token: q and k divided by the root mean square of all their rows at once, times a weight, the first
 //                     rot_dims dimensions of every head rotated (pairs i, i + rot_dims / 2); q back in place, k and v into the
 //                     paged cache
-//   head_append       per head: the first rot_dims dimensions rotated (neighbouring pairs, or i and i + rot_dims / 2), then optionally the
-//                     head divided by its root mean square; q back in place, k and v into the paged cache
+//   head_append       per head: bias, RMS norm with a weight, the first rot_dims dimensions rotated (neighbouring pairs, or i and
+//                     i + rot_dims / 2), the head divided by its root mean square, each optional; values mixed with another layer's; q back
+//                     in place, k and v into the paged cache
 //   window_attn_rows  attention of single rows under a SkeinAttnRule (attn_rule.cuh)
 //
 // Cache page: [kv_heads, page_size, maps * dim] keys, then [kv_heads, page_size, vdim] values (with key and value heads of one width the
@@ -119,9 +120,39 @@ struct HeadAppendParams {
   long long ld;
   int T, H, K, D, maps, V, rot, interleaved, unit, max_pos, max_blocks, num_pages, page_size;
   float eps;
+  SkeinHeadExtras x;
 };
 
 constexpr int HA_WARPS = 8;
+
+// N elements of a head at element i of it: value, plus the bias
+template <typename T, int N>
+__device__ __forceinline__ void ha_load(const T* src, const float* bias, int i, float* a) {
+  load_v<T, N>(src + i, a);
+  if (bias) {
+    float b[N];
+    load_v<float, N>(bias + i, b);
+#pragma unroll
+    for (int k = 0; k < N; ++k) a[k] += b[k];
+  }
+}
+
+// values of a key head: bias, kept for later layers, mixed with the first such layer's
+template <typename T, int N>
+__device__ __forceinline__ void ha_value(const HeadAppendParams& p, const T* src, T* dst, int t, int n, int i) {
+  float a[N];
+  const size_t at = (size_t)t * p.K * p.V + (size_t)n * p.V + i;
+  ha_load<T, N>(src, p.x.v_bias ? p.x.v_bias + (size_t)n * p.V : nullptr, i, a);
+  if (p.x.v_keep) store_v<T, N>((T*)p.x.v_keep + at, a);
+  if (p.x.mix) {
+    float f[N];
+    const float m = p.x.mix[0];
+    load_v<T, N>((const T*)p.x.v_first + at, f);
+#pragma unroll
+    for (int k = 0; k < N; ++k) a[k] = (1.f - m) * a[k] + m * f[k];
+  }
+  store_v<T, N>(dst + i, a);
+}
 
 // One warp per head of a token. PAIR4: neighbouring pairs in accesses of 4 elements (two pairs), else single pairs.
 template <typename T, bool PAIR4>
@@ -137,7 +168,9 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
   if (pos >= p.max_pos) { if (lane == 0) report_status(p.status, ST_BAD_INDEX, pos); return; }
   const T* src;
   T* dst;
+  const float *bias = nullptr, *nw = n < nq ? p.x.q_norm : p.x.k_norm;
   if (n < nq) {
+    if (p.x.q_bias) bias = p.x.q_bias + (size_t)n * p.D;
     src = dst = (T*)p.q + (size_t)t * p.ld + (size_t)n * p.D;
   } else {
     const int seq = p.seq_of_token ? p.seq_of_token[t] : t;
@@ -146,6 +179,7 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
     T* base = (T*)p.cache + (size_t)page * p.K * p.page_size * (p.maps * p.D + p.V);
     n -= nq;
     if (n < nk) {
+      if (p.x.k_bias) bias = p.x.k_bias + (size_t)n * p.D;
       src = (const T*)p.k + (size_t)t * p.ld + (size_t)n * p.D;
       dst = base + ((size_t)(n / p.maps) * p.page_size + slot) * p.maps * p.D + (size_t)(n % p.maps) * p.D;
     } else {
@@ -153,9 +187,9 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
       src = (const T*)p.v + (size_t)t * p.ld + (size_t)n * p.V;
       dst = base + (size_t)p.K * p.page_size * p.maps * p.D + ((size_t)n * p.page_size + slot) * p.V;
       if (PAIR4 && p.V % 4 == 0) {
-        for (int i = lane * 4; i < p.V; i += 128) { float a[4]; load_v<T, 4>(src + i, a); store_v<T, 4>(dst + i, a); }
+        for (int i = lane * 4; i < p.V; i += 128) ha_value<T, 4>(p, src, dst, t, n, i);
       } else {
-        for (int i = lane; i < p.V; i += 32) dst[i] = src[i];
+        for (int i = lane; i < p.V; i += 32) ha_value<T, 1>(p, src, dst, t, n, i);
       }
       return;
     }
@@ -163,11 +197,11 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
   const float2* cs = reinterpret_cast<const float2*>(p.cos_sin) + (size_t)pos * (p.rot / 2);
   if (PAIR4) {
     float r = 1.f;
-    if (p.unit) {      // a rotation leaves the sum of squares as it is
+    if (p.unit || nw) {      // a rotation leaves the sum of squares as it is
       float ss = 0.f;
       for (int i = lane * 4; i < p.D; i += 128) {
         float a[4];
-        load_v<T, 4>(src + i, a);
+        ha_load<T, 4>(src, bias, i, a);
 #pragma unroll
         for (int k = 0; k < 4; ++k) ss = fmaf(a[k], a[k], ss);
       }
@@ -176,7 +210,13 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
     }
     for (int i = lane * 4; i < p.D; i += 128) {
       float a[4];
-      load_v<T, 4>(src + i, a);
+      ha_load<T, 4>(src, bias, i, a);
+      if (nw) {
+        float w[4];
+        load_v<float, 4>(nw + i, w);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) a[k] *= w[k];
+      }
       if (i < p.rot) {
         const float4 c = *reinterpret_cast<const float4*>(cs + i / 2);
         const float x0 = a[0], x2 = a[2];
@@ -190,9 +230,11 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
     return;
   }
   float r = 1.f;
-  if (p.unit) {
+  auto value = [&](int i) { return to_f<T>(src[i]) + (bias ? bias[i] : 0.f); };
+  auto weight = [&](int i) { return nw ? nw[i] : 1.f; };
+  if (p.unit || nw) {
     float ss = 0.f;
-    for (int i = lane; i < p.D; i += 32) { const float a = to_f<T>(src[i]); ss = fmaf(a, a, ss); }
+    for (int i = lane; i < p.D; i += 32) { const float a = value(i); ss = fmaf(a, a, ss); }
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     r = 1.f / sqrtf(ss / (float)p.D + p.eps);
   }
@@ -200,11 +242,11 @@ __global__ void __launch_bounds__(32 * HA_WARPS) head_append_kernel(const HeadAp
   for (int i = lane; i < half; i += 32) {
     const int i0 = p.interleaved ? 2 * i : i, i1 = p.interleaved ? 2 * i + 1 : i + half;
     const float2 c = cs[i];
-    const float x = to_f<T>(src[i0]), y = to_f<T>(src[i1]);
+    const float x = value(i0) * weight(i0), y = value(i1) * weight(i1);
     dst[i0] = from_f<T>((x * c.x - y * c.y) * r);
     dst[i1] = from_f<T>((y * c.x + x * c.y) * r);
   }
-  for (int i = p.rot + lane; i < p.D; i += 32) dst[i] = from_f<T>(to_f<T>(src[i]) * r);
+  for (int i = p.rot + lane; i < p.D; i += 32) dst[i] = from_f<T>(value(i) * weight(i) * r);
 }
 
 struct WindowAttnParams {
@@ -235,6 +277,7 @@ __global__ void __launch_bounds__(WR_TILE) window_attn_rows_kernel(const WindowA
   if (pos < 0) return;
   const int kvh = h / (p.H / p.K), seq = p.seq_of_token ? p.seq_of_token[t] : t;
   const int lo = attn_first_key(p.r.window, p.r.chunk, pos), KW = maps * p.D;
+  const int kept = min(p.r.keep_first, lo), n_keys = kept + pos + 1 - lo;      // the first tokens, then the window
   const size_t page_elems = (size_t)p.K * p.page_size * (KW + p.V);
   for (int map = 0; map < maps; ++map) {
     float* o_s = q_s + p.D + map * p.V;
@@ -243,11 +286,11 @@ __global__ void __launch_bounds__(WR_TILE) window_attn_rows_kernel(const WindowA
     for (int i = tid; i < p.D; i += WR_TILE) q_s[i] = to_f<T>(q[i]);
     for (int i = tid; i < p.V; i += WR_TILE) o_s[i] = 0.f;
     float m = -INFINITY, l = 0.f;
-    for (int j0 = lo; j0 <= pos; j0 += WR_TILE) {
+    for (int i0 = 0; i0 < n_keys; i0 += WR_TILE) {
       __syncthreads();
-      const int j = j0 + tid, cnt = min(WR_TILE, pos + 1 - j0);
+      const int cnt = min(WR_TILE, n_keys - i0), j = i0 + tid < kept ? i0 + tid : i0 + tid - kept + lo;
       float s = -INFINITY;
-      if (j <= pos) {
+      if (tid < cnt) {
         int page = p.block_table[(size_t)seq * p.max_blocks + j / p.page_size];
         if (page < 0 || page >= p.num_pages) { report_status(p.status, ST_BAD_INDEX, page); page = 0; }
         const T* base = (const T*)p.cache + (size_t)page * page_elems;
@@ -256,13 +299,14 @@ __global__ void __launch_bounds__(WR_TILE) window_attn_rows_kernel(const WindowA
         float a = 0.f;
         for (int d = 0; d < p.D; ++d) a = fmaf(q_s[d], to_f<T>(k[d]), a);
         s = a * p.r.scale;
+        if (p.r.softcap > 0.f) s = p.r.softcap * tanhf(s / p.r.softcap);
       }
       float mx = s;
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       if ((tid & 31) == 0) red[tid >> 5] = mx;
       __syncthreads();
       const float mn = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
-      const float keep = m == -INFINITY ? 0.f : expf(m - mn), e = j <= pos ? expf(s - mn) : 0.f;
+      const float keep = m == -INFINITY ? 0.f : expf(m - mn), e = tid < cnt ? expf(s - mn) : 0.f;
       m = mn;
       prob[tid] = e;
       float sum = e;
@@ -278,9 +322,9 @@ __global__ void __launch_bounds__(WR_TILE) window_attn_rows_kernel(const WindowA
       }
     }
     float inv = 1.f / l;
-    if (p.r.sink) {
-      const float top = fmaxf(m, 0.f), e = expf(m - top);
-      inv = e / (l * e + expf(-top));
+    if (p.r.sink || p.r.sinks) {
+      const float sink = p.r.sinks ? p.r.sinks[h] : 0.f, top = fmaxf(m, sink), e = expf(m - top);
+      inv = e / (l * e + expf(sink - top));
     }
     for (int d = tid; d < p.V; d += WR_TILE) o_s[d] *= inv;
   }
@@ -328,15 +372,16 @@ extern "C" int skein_window_append(void* q, const void* k, const void* v, long l
 }
 
 extern "C" int skein_head_append(void* q, const void* k, const void* v, long long ld, const float* cos_sin, const int* positions,
-                                 const int* seq_of_token, const int* block_table, void* cache, int* status, int T, int H, int K, int D, int maps, int V,
+                                 const int* seq_of_token, const int* block_table, void* cache, int* status, const SkeinHeadExtras* extras, int T, int H,
+                                 int K, int D, int maps, int V,
                                  int rot, int interleaved, int unit, int max_pos, int max_blocks, int num_pages, int page_size, float eps, int fp32,
                                  void* stream) {
   using namespace skein;
   if (T == 0) return 0;
-  if (rot % 2 != 0 || rot > D || rot < 0) return -1;
+  if (rot % 2 != 0 || rot > D || rot < 0 || (rot > 0 && !cos_sin) || (extras->mix && !extras->v_first)) return -1;
   HeadAppendParams p{q, k, v, cos_sin, positions, seq_of_token, block_table, cache, status, ld, T, H, K, D, maps, V, rot, interleaved, unit, max_pos,
-                     max_blocks, num_pages, page_size, eps};
-  const bool v4 = interleaved && D % 4 == 0 && rot % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 &&
+                     max_blocks, num_pages, page_size, eps, *extras};
+  const bool v4 = (interleaved || rot == 0) && D % 4 == 0 && rot % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 &&
                   (uintptr_t)v % 16 == 0 && (uintptr_t)cache % 16 == 0;
   const long long units = (long long)T * (H * maps + K * maps + K);
   const dim3 grid((unsigned)((units + HA_WARPS - 1) / HA_WARPS)), b(32 * HA_WARPS);

@@ -810,15 +810,16 @@ static EncodeTiledFn get_encode_fn() {
   return fn;
 }
 
-// 2-D row-major tensor [rows, k_elems] of 1- or 2-byte elements; box = [box_rows, 128 bytes].
-int make_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes,
+// 2-D row-major tensor [rows, k_elems] of 1- or 2-byte elements, rows `ld` elements apart; box = [box_rows, 128 bytes]. Elements past
+// k_elems read as zero, whatever lies between the rows.
+int make_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, uint64_t ld, int elem_bytes,
                  uint32_t box_rows) {
   EncodeTiledFn fn = get_encode_fn();
   if (!fn) return -10;
   if ((reinterpret_cast<uintptr_t>(base) & 15) != 0) return -11;
-  if ((k_elems * elem_bytes) % 16 != 0) return -12;
+  if ((ld * elem_bytes) % 16 != 0) return -12;
   cuuint64_t dims[2] = {k_elems, rows};
-  cuuint64_t strides[1] = {k_elems * (uint64_t)elem_bytes};
+  cuuint64_t strides[1] = {ld * (uint64_t)elem_bytes};
   cuuint32_t box[2] = {(cuuint32_t)(128 / elem_bytes), box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = fn(out, elem_bytes == 2 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_UINT8, 2,
@@ -829,9 +830,9 @@ int make_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_e
 }
 
 struct TmapKey {
-  const void* base; uint64_t rows, k; int eb; uint32_t box;
+  const void* base; uint64_t rows, k, ld; int eb; uint32_t box;
   bool operator==(const TmapKey& o) const {
-    return base == o.base && rows == o.rows && k == o.k && eb == o.eb && box == o.box;
+    return base == o.base && rows == o.rows && k == o.k && ld == o.ld && eb == o.eb && box == o.box;
   }
 };
 struct TmapKeyHash {
@@ -839,25 +840,29 @@ struct TmapKeyHash {
     size_t h = reinterpret_cast<size_t>(k.base);
     h ^= k.rows * 0x9E3779B97F4A7C15ull + (h << 6) + (h >> 2);
     h ^= k.k * 0xC2B2AE3D27D4EB4Full + (h << 6) + (h >> 2);
-    h ^= (size_t)k.box * 0x165667B19E3779F9ull + k.eb;
+    h ^= (size_t)k.box * 0x165667B19E3779F9ull + k.eb + k.ld * 0x27D4EB2F165667C5ull;
     return h;
   }
 };
 
-int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes,
-                   uint32_t box_rows) {
+static int cached_tmap_2d_ld(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, uint64_t ld, int elem_bytes,
+                             uint32_t box_rows) {
   static std::unordered_map<TmapKey, CUtensorMap, TmapKeyHash> cache;
   static std::mutex mu;
-  TmapKey key{base, rows, k_elems, elem_bytes, box_rows};
+  TmapKey key{base, rows, k_elems, ld, elem_bytes, box_rows};
   std::lock_guard<std::mutex> lk(mu);
   auto it = cache.find(key);
   if (it != cache.end()) { *out = it->second; return 0; }
-  int rc = make_tmap_2d(out, base, rows, k_elems, elem_bytes, box_rows);
+  int rc = make_tmap_2d(out, base, rows, k_elems, ld, elem_bytes, box_rows);
   if (rc == 0) {
     if (cache.size() > 4096) cache.clear();
     cache.emplace(key, *out);
   }
   return rc;
+}
+
+int cached_tmap_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t k_elems, int elem_bytes, uint32_t box_rows) {
+  return cached_tmap_2d_ld(out, base, rows, k_elems, k_elems, elem_bytes, box_rows);
 }
 
 // [rows, heads, d] bf16 with `head_stride` / `row_stride` elements between heads / rows; box = [box_rows, 1, 64 elements].
@@ -991,7 +996,9 @@ extern "C" int skein_gemm_ws(const SkeinGemmParams* p, void* stream) {
     rc = cached_tmap_2d(&tmW, p->W, (uint64_t)p->G * p->w_rows_per_group, p->K, w8 ? 1 : 2, TILE_F);
   }
   if (rc) return rc;
-  rc = cached_tmap_2d(&tmX, p->X, p->x_rows, p->x_ld > 0 ? p->x_ld : p->K, 2, p->n_tile);
+  // strided rows: a last block of K elements that is not whole must not read what lies behind them
+  const uint64_t x_width = (p->x_group_cols > 0 ? (uint64_t)(p->G - 1) * p->x_group_cols : 0) + p->K;
+  rc = cached_tmap_2d_ld(&tmX, p->X, p->x_rows, x_width, p->x_ld > 0 ? p->x_ld : p->K, 2, p->n_tile);
   if (rc) return rc;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   static bool attr_done[4] = {false, false, false, false};

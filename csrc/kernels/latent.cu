@@ -184,6 +184,7 @@ struct LatentAttnParams {
   const void* cache;
   void* out;                 // [T, H * kv_rank]
   int* status;
+  const float* sinks;        // [H] one more term exp(sinks[h]) in the denominator, or null
   long long q_ld;
   float scale;
   int H, D, rot, kv_rank, max_pos, max_blocks, num_pages, page_size;
@@ -259,7 +260,12 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_rows_kernel(const Late
     }
     __syncthreads();
   }
-  for (int i = tid; i < K; i += LA_THREADS) out[i] = lt_t<T>(acc[i] / l);
+  float inv = 1.f / l;
+  if (p.sinks) {
+    const float sink = p.sinks[h], top = fmaxf(m, sink), e = expf(m - top);
+    inv = e / (l * e + expf(sink - top));
+  }
+  for (int i = tid; i < K; i += LA_THREADS) out[i] = lt_t<T>(acc[i] * inv);
 }
 
 }  // namespace skein
@@ -299,12 +305,12 @@ extern "C" int skein_latent_gather(const void* cache, const int* block_table, in
 
 extern "C" int skein_latent_attn_rows(const void* q_abs, const void* q, long long q_ld, const float* cos_sin, int max_pos, const int* positions,
                                       const int* seq_of_token, const int* block_table, int max_blocks, const void* cache, int num_pages,
-                                      int page_size, void* out, int T, int H, int D, int rot, int kv_rank, float scale, int* status, int fp32,
-                                      void* stream) {
+                                      int page_size, void* out, int T, int H, int D, int rot, int kv_rank, float scale, const float* sinks, int* status,
+                                      int fp32, void* stream) {
   using namespace skein;
   if (T == 0) return 0;
   if (rot % 2 != 0 || H > 65535) return -1;
-  LatentAttnParams p{q_abs, q, cos_sin, positions, seq_of_token, block_table, cache, out, status, q_ld, scale, H, D, rot, kv_rank, max_pos,
+  LatentAttnParams p{q_abs, q, cos_sin, positions, seq_of_token, block_table, cache, out, status, sinks, q_ld, scale, H, D, rot, kv_rank, max_pos,
                      max_blocks, num_pages, page_size};
   const size_t sm = (size_t)(2 * kv_rank + rot + LA_THREADS) * 4;
   if (sm > 200 * 1024) return -1;

@@ -2,11 +2,12 @@
 //
 //   S <- g S + k u^T,   o = S^T q (+ skip v)
 //     delta      g = exp(neg_decay softplus(a + dt_bias)),  u = beta (v - (g S)^T k),  beta = sigmoid(b);  q, k unit vectors
+//     channel    the same with one g per row of S: g[n] = exp(neg_decay softplus(step[n] + dt_bias[n]))
 //     ssd        g = exp(neg_decay dt),  dt = softplus(dt_raw + dt_bias),  u = dt v
 //     lightning  g fixed per head (neg_decay its logarithm),  u = v
 //
 // q, k, v are projections that passed a short causal convolution over time (delta, ssd) and silu. Query / key heads may be
-// shared: head h uses h / (H / G).
+// shared: head h uses h / (H / G). A decay just below one is raised to a high power in the end: decays per row enter as s + expm1(log g) s.
 //
 // A sequence owns one slot of the state pools: S [slots, H, D, V] fp32 and the convolution's last inputs [slots, taps, channels]
 // in the activation type, position p in row p mod taps (taps - 1 rows would hold the state; with one more, a step writes no row
@@ -36,10 +37,17 @@ constexpr int REC_MAX_D = 512;
 template <typename T>
 __device__ __forceinline__ void rec_gates(const RecParams& p, const T* row, int h, float* log_g, float* coef) {
   const float nd = p.neg_decay[h];
+  if (p.kind == REC_CHANNEL) { *log_g = 0.f; *coef = 1.f / (1.f + expf(-to_f<T>(row[p.b_col + h]))); return; }      // (decays: rec_row_decay)
   if (p.kind == REC_LIGHTNING) { *log_g = nd; *coef = 1.f; return; }
   const float dt = softplus_f(to_f<T>(row[p.a_col + h]) + p.dt_bias[h]);
   *log_g = nd * dt;
   *coef = p.kind == REC_DELTA ? 1.f / (1.f + expf(-to_f<T>(row[p.b_col + h]))) : dt;
+}
+
+// g - 1 of row n of head h's state (channel) for the step's row t
+__device__ __forceinline__ float rec_row_decay(const RecParams& p, size_t t, int h, int n) {
+  const int i = h * p.D + n;
+  return expm1f(p.neg_decay[h] * softplus_f(p.step[t * p.H * p.D + i] + p.dt_bias[i]));
 }
 
 // column of the projection row and of the convolution's channel order (q | k | v)
@@ -92,7 +100,7 @@ __device__ __forceinline__ float2 rec_block_sum2(float2 v, float2* sh) {
 // whole 32 VPT-wide row pieces. Both products with the old state come from one pass: o = g S^T q + (q . k) u.
 template <typename T, int RPT, int VPT>
 __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p) {
-  __shared__ float q_s[REC_MAX_D], k_s[REC_MAX_D];
+  __shared__ float q_s[REC_MAX_D], k_s[REC_MAX_D], g_s[REC_MAX_D];
   __shared__ float part[2][RS_WARPS][32 * VPT];
   __shared__ float2 red[RS_WARPS], red2[RS_WARPS];
   __shared__ float v_s[32 * VPT];
@@ -117,6 +125,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
   const T* row = (const T*)p.row + (size_t)b * p.ld;
   T* tail = p.taps > 1 ? (T*)p.tail + (size_t)slot * p.taps * p.C : nullptr;
   const int gd = p.G * p.D, ncol = min(32 * VPT, p.V - tile0), first_head = grp * (p.H / p.G);
+  if (p.kind == REC_CHANNEL) for (int n = tid; n < p.D; n += RS_THREADS) g_s[n] = rec_row_decay(p, b, h, n);
   float2 sq = make_float2(0.f, 0.f);
   for (int i = tid; i < 2 * p.D + ncol; i += RS_THREADS) {
     const int ch = i < p.D ? grp * p.D + i : i < 2 * p.D ? gd + grp * p.D + i - p.D : 2 * gd + h * p.V + tile0 + i - 2 * p.D;
@@ -130,7 +139,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
   }
   sq = rec_block_sum2(sq, red);      // (also the barrier behind q_s, k_s, v_s)
   float rq = 1.f, rk = 1.f;
-  if (p.kind == REC_DELTA) {
+  if (rec_corrects(p.kind)) {
     rq = 1.f / sqrtf(sq.x + 1e-6f) / sqrtf((float)p.D);
     rk = 1.f / sqrtf(sq.y + 1e-6f);
   }
@@ -147,6 +156,10 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
     const int n = warp + i * RS_WARPS;
     if (n >= p.D) break;
     const float kn = k_s[n] * rk, qn = q_s[n] * rq;
+    if (p.kind == REC_CHANNEL) {
+#pragma unroll
+      for (int j = 0; j < VPT; ++j) s[i][j] = fmaf(g_s[n], s[i][j], s[i][j]);
+    }
 #pragma unroll
     for (int j = 0; j < VPT; ++j) { ks[j] = fmaf(kn, s[i][j], ks[j]); qs[j] = fmaf(qn, s[i][j], qs[j]); }
   }
@@ -161,7 +174,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
     for (int w = 0; w < RS_WARPS; ++w) { a += part[0][w][lane * VPT + j]; o += part[1][w][lane * VPT + j]; }
     const bool in = c0 + j < p.V;
     const float v = in ? v_s[lane * VPT + j] : 0.f;
-    u[j] = p.kind == REC_DELTA ? coef * (v - g * a) : coef * v;
+    u[j] = rec_corrects(p.kind) ? coef * (v - g * a) : coef * v;
     if (warp == 0 && in) {
       const float y = g * o + qk * u[j] + (p.skip ? p.skip[h] * v : 0.f);
       ((T*)p.out)[(size_t)b * p.H * p.V + (size_t)h * p.V + c0 + j] = from_f<T>(y);
@@ -185,14 +198,16 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_kernel(const RecParams p)
 // another and whose queries and keys are the same. grid (H / heads, B).
 constexpr int RSB_MAX = 64 * 1024, RSB_HEADS = 8;
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool CHANNEL>
 __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecParams p, const RecGate gt, const int heads) {
-  extern __shared__ __align__(128) float st_s[];       // states [heads][D][V], then u [V], sums [warps][V], v [heads][V], q [D], k [D]
+  // states [heads][D][V], then u [V], sums [warps][V], v [heads][V], q [D], k [D], decays [heads][D] (channel)
+  extern __shared__ __align__(128) float st_s[];
   float* u_s = st_s + heads * p.D * p.V;
   float* part = u_s + p.V;
   float* v_s = part + RS_WARPS * p.V;
   float* q_s = v_s + heads * p.V;
   float* k_s = q_s + p.D;
+  float* g_s = k_s + p.D;
   __shared__ float2 red[RS_WARPS], red2[RS_WARPS];
   __shared__ float2 gate_s[RSB_HEADS];
   __shared__ __align__(8) uint64_t bar;
@@ -223,6 +238,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
     rec_gates<T>(p, row, h0 + lane, &log_g, &coef);
     gate_s[lane] = make_float2(p.decay ? p.decay[h0 + lane] : expf(log_g), coef);
   }
+  if (CHANNEL) for (int i = tid; i < heads * D; i += RS_THREADS) g_s[i] = rec_row_decay(p, b, h0 + i / D, i % D);
   float2 sq = make_float2(0.f, 0.f);
   const int at = p.taps > 1 ? pos % p.taps : 0;
   const bool owner = h0 % (p.H / p.G) == 0;      // of the group's queries and keys
@@ -238,7 +254,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
   }
   sq = rec_block_sum2(sq, red);      // (also the barrier behind what was written above)
   float rq = 1.f, rk = 1.f;
-  if (p.kind == REC_DELTA) {
+  if (rec_corrects(p.kind)) {
     rq = 1.f / sqrtf(sq.x + 1e-6f) / sqrtf((float)D);
     rk = 1.f / sqrtf(sq.y + 1e-6f);
   }
@@ -258,10 +274,19 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
     const int h = h0 + hh;
     float* st = st_s + hh * D * V;
     const float g = gate_s[hh].x, coef = gate_s[hh].y;
+    const float* gr = g_s + hh * D;
+    auto row_of = [&](int n) {      // the state's row, decayed (channel)
+      float4 s = *reinterpret_cast<const float4*>(st + n * V + cg * 4);
+      if (CHANNEL) {
+        const float d = gr[n];
+        s.x = fmaf(d, s.x, s.x); s.y = fmaf(d, s.y, s.y); s.z = fmaf(d, s.z, s.z); s.w = fmaf(d, s.w, s.w);
+      }
+      return s;
+    };
     float4 ks = make_float4(0.f, 0.f, 0.f, 0.f), qs = ks;
 #pragma unroll 4
     for (int n = r0; n < D; n += R) {
-      const float4 s = *reinterpret_cast<const float4*>(st + n * V + cg * 4);
+      const float4 s = row_of(n);
       const float kn = k_s[n], qn = q_s[n];
       ks.x = fmaf(kn, s.x, ks.x); ks.y = fmaf(kn, s.y, ks.y); ks.z = fmaf(kn, s.z, ks.z); ks.w = fmaf(kn, s.w, ks.w);
       qs.x = fmaf(qn, s.x, qs.x); qs.y = fmaf(qn, s.y, qs.y); qs.z = fmaf(qn, s.z, qs.z); qs.w = fmaf(qn, s.w, qs.w);
@@ -274,7 +299,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
     }
     const bool writes = CG > 32 || lane < CG;
     float a = 0.f, y = 0.f;
-    if (p.kind == REC_DELTA) {               // only the correction needs S^T k
+    if (rec_corrects(p.kind)) {              // only the correction needs S^T k
       if (writes) *reinterpret_cast<float4*>(part + pr * V + cg * 4) = ks;
       __syncthreads();
       if (tid < V) for (int w = 0; w < np; ++w) a += part[w * V + tid];
@@ -286,7 +311,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
     if (tid < V) {
       for (int w = 0; w < np; ++w) y += part[w * V + tid];
       const float v = v_s[hh * V + tid];
-      const float u = p.kind == REC_DELTA ? coef * (v - g * rk * a) : coef * v;
+      const float u = rec_corrects(p.kind) ? coef * (v - g * rk * a) : coef * v;
       u_s[tid] = u * rk;
       o = g * rq * y + qk * u + (p.skip ? p.skip[h] * v : 0.f);
       if (gt.out == nullptr) ((T*)p.out)[(size_t)b * p.H * V + (size_t)h * V + tid] = from_f<T>(o);
@@ -295,8 +320,8 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
       // the head's own norm and gate
       const float r = 1.f / sqrtf(rec_block_sum2(make_float2(o * o, 0.f), red).x / (float)V + gt.eps);      // (a barrier behind u_s too)
       if (tid < V) {
-        const float z = to_f<T>(row[gt.gate_col + h * V + tid]);
-        ((T*)gt.out)[(size_t)b * gt.out_ld + (size_t)h * V + tid] = from_f<T>(o * r * gt.norm[tid] * (z / (1.f + expf(-z))) * gt.scale);
+        const float z = to_f<T>(((const T*)gt.gate)[(size_t)b * gt.gate_ld + (size_t)h * V + tid]), a = (gt.sigmoid ? 1.f : z) / (1.f + expf(-z));
+        ((T*)gt.out)[(size_t)b * gt.out_ld + (size_t)h * V + tid] = from_f<T>(o * r * gt.norm[tid] * a * gt.scale);
       }
     } else {
       __syncthreads();
@@ -304,7 +329,7 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
     const float4 u4 = *reinterpret_cast<const float4*>(u_s + cg * 4);
 #pragma unroll 4
     for (int n = r0; n < D; n += R) {
-      float4 s = *reinterpret_cast<const float4*>(st + n * V + cg * 4);
+      float4 s = row_of(n);
       const float kn = k_s[n];
       s.x = fmaf(g, s.x, kn * u4.x); s.y = fmaf(g, s.y, kn * u4.y); s.z = fmaf(g, s.z, kn * u4.z); s.w = fmaf(g, s.w, kn * u4.w);
       *reinterpret_cast<float4*>(S + (size_t)hh * D * V + (size_t)n * V + cg * 4) = s;
@@ -313,33 +338,38 @@ __global__ void __launch_bounds__(RS_THREADS) rec_step_bulk_kernel(const RecPara
   }
 }
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool CHANNEL>
 static int rec_step_bulk_go(const RecParams& p, const RecGate& g, int B, cudaStream_t s) {
   int heads = RSB_HEADS;                     // a power of two that divides the heads of a group; enough CTAs before larger ones
   while (heads > 1 && ((p.H / p.G) % heads != 0 || (long long)heads * p.D * p.V * 4 > RSB_MAX || (long long)B * p.H / heads < 444)) heads /= 2;
-  const int sm = (heads * p.D * p.V + (RS_WARPS + 1 + heads) * p.V + 2 * p.D) * 4;
+  const int sm = (heads * p.D * p.V + (RS_WARPS + 1 + heads) * p.V + (2 + (CHANNEL ? heads : 0)) * p.D) * 4;
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(rec_step_bulk_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, RSB_MAX + 24 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(rec_step_bulk_kernel<T, TAPS, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize, RSB_MAX + 24 * 1024);
     if (e != cudaSuccess) return (int)e;
     attr_set = true;
   }
-  return (int)launch_pdl(rec_step_bulk_kernel<T, TAPS>, dim3(p.H / heads, B), dim3(RS_THREADS), (size_t)sm, s, p, g, heads);
+  return (int)launch_pdl(rec_step_bulk_kernel<T, TAPS, CHANNEL>, dim3(p.H / heads, B), dim3(RS_THREADS), (size_t)sm, s, p, g, heads);
+}
+
+template <typename T, bool CHANNEL>
+static int rec_step_bulk_taps(const RecParams& p, const RecGate& g, int B, cudaStream_t s) {
+  switch (p.taps) {
+    case 1: return rec_step_bulk_go<T, 1, CHANNEL>(p, g, B, s);
+    case 2: return rec_step_bulk_go<T, 2, CHANNEL>(p, g, B, s);
+    case 3: return rec_step_bulk_go<T, 3, CHANNEL>(p, g, B, s);
+    case 4: return rec_step_bulk_go<T, 4, CHANNEL>(p, g, B, s);
+    default: return rec_step_bulk_go<T, 0, CHANNEL>(p, g, B, s);
+  }
 }
 
 template <typename T>
 static int rec_step_bulk(const RecParams& p, const RecGate& g, int B, cudaStream_t s) {
-  switch (p.taps) {
-    case 1: return rec_step_bulk_go<T, 1>(p, g, B, s);
-    case 2: return rec_step_bulk_go<T, 2>(p, g, B, s);
-    case 3: return rec_step_bulk_go<T, 3>(p, g, B, s);
-    case 4: return rec_step_bulk_go<T, 4>(p, g, B, s);
-    default: return rec_step_bulk_go<T, 0>(p, g, B, s);
-  }
+  return p.kind == REC_CHANNEL ? rec_step_bulk_taps<T, true>(p, g, B, s) : rec_step_bulk_taps<T, false>(p, g, B, s);
 }
 
 // ---- chunks ---------------------------------------------------------------------------------------
-// grid T. Convolved q | k | v of one token, its heads' gates and (delta) the factors that make q and k unit vectors.
+// grid T. Convolved q | k | v of one token, its heads' gates and (delta rules) the factors that make q and k unit vectors.
 template <typename T>
 __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const RecChunk c) {
   extern __shared__ float qk_s[];        // [2 G D] (delta)
@@ -359,7 +389,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
       return t - j >= first ? to_f<T>(row[col - (long long)j * p.ld]) : to_f<T>(tail[(size_t)((pos - j) % p.taps) * p.C + ch]);
     });
     out[ch < 2 * gd ? ch : ch - 2 * gd + c.v_off] = from_f<T>(x);
-    if (p.kind == REC_DELTA && ch < 2 * gd) qk_s[ch] = x;
+    if (rec_corrects(p.kind) && ch < 2 * gd) qk_s[ch] = x;
   }
   for (int h = tid; h < p.H; h += blockDim.x) {
     float log_g, coef;
@@ -367,7 +397,7 @@ __global__ void __launch_bounds__(256) rec_prep_kernel(const RecParams p, const 
     c.gates[((size_t)t * p.H + h) * 2] = log_g;
     c.gates[((size_t)t * p.H + h) * 2 + 1] = coef;
   }
-  if (p.kind != REC_DELTA) return;
+  if (!rec_corrects(p.kind)) return;
   __syncthreads();
   for (int u = tid >> 5; u < 2 * p.G; u += blockDim.x >> 5) {      // a warp per query / key head
     float ss = 0.f;
@@ -434,7 +464,7 @@ __global__ void __launch_bounds__(256, 2) rec_prep_vec_kernel(const RecParams p,
     }
   }
   const int lanes = p.D / 8;
-  const bool units = p.kind == REC_DELTA && blockIdx.x * 2048 < 2 * gd;
+  const bool units = rec_corrects(p.kind) && blockIdx.x * 2048 < 2 * gd;
   auto token = [&](int i, const uint4& in) {
     float x[8], y[8];
     if (TAPS > 1) {
@@ -516,7 +546,7 @@ constexpr int SC_WARPS = 8;
 // the sums over rows need no more than shuffles.
 template <typename T, int RPT>
 __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, const RecChunk c) {
-  extern __shared__ float sc_s[];      // q [SC_TOK][D], k [SC_TOK][D], v [SC_TOK][32]
+  extern __shared__ float sc_s[];      // q [SC_TOK][D], k [SC_TOK][D], v [SC_TOK][32], decays [SC_TOK][D] (channel)
   __shared__ float g_s[SC_TOK], coef_s[SC_TOK];
   pdl_trigger();
   pdl_wait();
@@ -529,6 +559,8 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, const 
   float* q_s = sc_s;
   float* k_s = q_s + SC_TOK * p.D;
   float* v_s = k_s + SC_TOK * p.D;
+  float* gr_s = v_s + SC_TOK * 32;
+  const bool channel = p.kind == REC_CHANNEL;
   float* S = p.state + ((size_t)slot * p.H + h) * p.D * p.V;
   const bool fresh = p.positions[t0] == 0;
   float s[RPT];
@@ -545,12 +577,13 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, const 
       const int j = i / p.D, d = i % p.D;
       const T* x = (const T*)c.qkv + (size_t)(t0 + b0 + j) * c.qkv_ld + grp * p.D + d;
       float rq = 1.f, rk = 1.f;
-      if (p.kind == REC_DELTA) {
+      if (rec_corrects(p.kind)) {
         rq = c.unit[(size_t)(t0 + b0 + j) * 2 * p.G + grp];
         rk = c.unit[(size_t)(t0 + b0 + j) * 2 * p.G + p.G + grp];
       }
       q_s[i] = to_f<T>(x[0]) * rq;
       k_s[i] = to_f<T>(x[gd]) * rk;
+      if (channel) gr_s[i] = rec_row_decay(p, t0 + b0 + j, h, d);
     }
     for (int i = tid; i < cnt * 32; i += 256) {
       const int j = i / 32, d = i % 32;
@@ -565,7 +598,14 @@ __global__ void __launch_bounds__(256) rec_scan_kernel(const RecParams p, const 
     for (int j = 0; j < cnt; ++j) {
       const float g = g_s[j], v = v_s[j * 32 + warp * SC_COLS + (lane & 3)];
       float u = coef_s[j] * v;
-      if (p.kind == REC_DELTA) {
+      if (channel) {
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) {
+          const int n = r + 8 * i;
+          if (n < p.D) s[i] = fmaf(gr_s[j * p.D + n], s[i], s[i]);
+        }
+      }
+      if (rec_corrects(p.kind)) {
         float a = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
@@ -614,7 +654,7 @@ static int rec_step_any(const RecParams& p, int B, cudaStream_t s) {
 
 template <typename T, int RPT>
 static int rec_scan_go(const RecParams& p, const RecChunk& c, int S, cudaStream_t s) {
-  const int sm = SC_TOK * (2 * p.D + 32) * 4;
+  const int sm = SC_TOK * ((p.kind == REC_CHANNEL ? 3 : 2) * p.D + 32) * 4;
   auto fn = rec_scan_kernel<T, RPT>;
   if (sm > 46 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, sm);
@@ -633,7 +673,7 @@ static int rec_scan_any(const RecParams& p, const RecChunk& c, int S, cudaStream
 }
 
 static int rec_check(const RecParams* p) {
-  if (p->kind < 0 || p->kind > 2 || p->H < 1 || p->G < 1 || p->H % p->G != 0) return -1;
+  if (p->kind < 0 || p->kind > 3 || (p->kind == REC_CHANNEL && (!p->step || !p->dt_bias)) || p->H < 1 || p->G < 1 || p->H % p->G != 0) return -1;
   if (p->D < 1 || p->D > REC_MAX_D || p->V < 1 || p->taps < 1 || p->H > 65535) return -1;
   if (p->taps > 1 && p->tail == nullptr) return -1;
   return 0;
@@ -666,7 +706,7 @@ extern "C" int skein_rec_prep(const SkeinRecParams* p, const SkeinRecChunk* c, i
   const int lanes = p->D / 8;
   const bool vec = !fp32 && p->D % 8 == 0 && p->V % 8 == 0 && p->ld % 8 == 0 && p->q_col % 8 == 0 && p->k_col % 8 == 0 && p->v_col % 8 == 0 &&
                    c->qkv_ld % 8 == 0 && c->v_off % 8 == 0 && p->taps <= 4 && (p->kind == REC_LIGHTNING || p->taps > 1) && (uintptr_t)p->row % 16 == 0 &&
-                   (p->kind != REC_DELTA || (lanes <= 32 && (lanes & (lanes - 1)) == 0));
+                   (!rec_corrects(p->kind) || (lanes <= 32 && (lanes & (lanes - 1)) == 0));
   if (vec) {
     const dim3 grid(((2 * p->G * p->D + p->H * p->V) / 8 + 255) / 256 + 1, (T + PV_TOK - 1) / PV_TOK);
     auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(256), 0, (cudaStream_t)stream, *p, *c, T); };
@@ -677,7 +717,7 @@ extern "C" int skein_rec_prep(const SkeinRecParams* p, const SkeinRecChunk* c, i
       default: return go(rec_prep_vec_kernel<4>);
     }
   }
-  const size_t sm = p->kind == REC_DELTA ? (size_t)2 * p->G * p->D * 4 : 0;
+  const size_t sm = rec_corrects(p->kind) ? (size_t)2 * p->G * p->D * 4 : 0;
   if (sm > 200 * 1024) return -1;
   auto go = [&](auto fn) -> int {
     if (sm > 46 * 1024) {

@@ -14,8 +14,9 @@ typedef struct SkeinRecParams {
   const float* conv_b;       // [C] or null
   const float* neg_decay;    // [H] factor of the step in the log decay; lightning: the log decay
   const float* decay;        // [H] lightning: the decay itself, which steps one by one take as it is, or null
-  const float* dt_bias;      // [H] or null
+  const float* dt_bias;      // [H], [H * D] (channel delta) or null
   const float* skip;         // [H] or null
+  const float* step;         // [rows, H * D] inputs of the decays before bias and softplus (channel delta), or null
   const int32_t* positions;  // [rows], -1: padding row
   const int32_t* slots;      // [sequences]
   int32_t* status;
@@ -40,12 +41,13 @@ typedef struct SkeinRecChunk {
   int32_t max_q_len;
 } SkeinRecChunk;
 
-// A head's output norm and gate (delta): o / rms(o) * norm * silu(row[gate_col + ...]) * scale into out; out null: not applied.
+// A head's output norm and gate (delta rules): o / rms(o) * norm * silu(gate) * scale into out; out null: not applied.
 typedef struct SkeinRecGate {
   const float* norm;         // [V]
   void* out;                 // [rows, out_ld]
-  int64_t out_ld;
-  int32_t gate_col;
+  const void* gate;          // [rows, gate_ld] H * V columns
+  int64_t out_ld, gate_ld;
+  int32_t sigmoid;           // the gate's activation is a sigmoid instead of silu
   float eps, scale;
   int32_t pad;
 } SkeinRecGate;
@@ -53,7 +55,9 @@ typedef struct SkeinRecGate {
 }  // extern "C"
 
 namespace skein {
-enum : int { REC_DELTA = 0, REC_SSD = 1, REC_LIGHTNING = 2 };
+enum : int { REC_DELTA = 0, REC_SSD = 1, REC_LIGHTNING = 2, REC_CHANNEL = 3 };
+// the delta rules: what the state holds for k is replaced, q and k are unit vectors
+__host__ __device__ constexpr bool rec_corrects(int kind) { return kind == REC_DELTA || kind == REC_CHANNEL; }
 using RecParams = SkeinRecParams;
 using RecChunk = SkeinRecChunk;
 using RecGate = SkeinRecGate;
