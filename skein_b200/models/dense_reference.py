@@ -37,6 +37,8 @@ def forward_full(cfg: ModelConfig, w: ModelWeights, token_ids: torch.Tensor, cap
     """Full-sequence forward of ONE sequence (unsharded weights). Returns fp32 logits [T, V]."""
     if cfg.is_parallel:
         return _forward_parallel(cfg, w, token_ids, capture_hidden)
+    if cfg.is_shifted:
+        return _forward_shifted(cfg, w, token_ids, capture_hidden)
     if cfg.is_prenorm:
         return _forward_prenorm(cfg, w, token_ids, capture_hidden)
     if cfg.is_layered:
@@ -315,3 +317,87 @@ def _forward_prenorm(cfg, w, token_ids, capture_hidden):
         if capture_hidden is not None:
             capture_hidden.append(x.clone())
     return (unit(x) * w.final_norm) @ w.lm_head.float().t()
+
+
+def _forward_shifted(cfg, w, token_ids, capture_hidden):
+    """The same for shifted pre-norm layers: attention by a full mask, keys and values of latent attention expanded, the recurrence one token
+    at a time."""
+    from .layered import GLU_SLOPE, LatentMixerSpec
+    from .parallel_layers import LayerLayout, RecurrentSpec
+    act, eps, T = torch.nn.functional, cfg.rms_norm_eps, token_ids.shape[0]
+    unit = lambda v: v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)      # noqa: E731
+    norm = lambda v, g: unit(v.view(T, cfg.norm_groups, -1)).reshape(T, -1) * g  # noqa: E731
+    xs = [w.embed[token_ids.long()].float()]
+    pos = torch.arange(T, device=xs[0].device)
+    back = pos[:, None] - pos[None, :]
+    v_first = None
+
+    def softmax_values(sc, seen, sinks, v):
+        sc = torch.cat([sc.masked_fill(~seen, float("-inf")), sinks[:, None, None].expand(-1, T, 1)], dim=-1)
+        return torch.einsum("hqk,khv->qhv", torch.softmax(sc, dim=-1)[..., :T], v).reshape(T, -1)
+
+    def latent(m, lw, z, at):
+        mw = lw.latent
+        ang = pos.double()[:, None] * m.rope_base ** (-torch.arange(0, m.rot_dim, 2, device=pos.device).double() / m.rot_dim)
+        turn = lambda t: torch.view_as_real(torch.complex(t[..., 0::2], t[..., 1::2])                 # noqa: E731
+                                            * torch.polar(torch.ones_like(ang), ang).to(torch.complex64)[:, None]).flatten(-2)
+        q = z[:, at["q"]:at["q"] + m.q_width].reshape(T, m.heads, -1)
+        ckr = z[:, at["dkv"]:at["dkv"] + m.cache_width]
+        kr = turn(ckr[:, None, m.kv_rank:])[:, 0]
+        kv = (unit(ckr[:, :m.kv_rank]) * mw.kv_norm) @ mw.w_ukv.float().t()
+        k, v = kv[:, :m.heads * m.dim].view(T, m.heads, -1), kv[:, m.heads * m.dim:].view(T, m.heads, -1)
+        sc = (torch.einsum("qhd,khd->hqk", q[..., :m.dim], k) + torch.einsum("qhd,kd->hqk", turn(q[..., m.dim:]), kr)) * m.scale
+        return softmax_values(sc, back >= 0, mw.sinks, v)
+
+    def attention(a, lw, z, at):
+        nonlocal v_first
+        aw = lw.attn
+        q, k, v = (z[:, at[n]:at[n] + rows] + b for (n, rows), b in zip(a.sections(), (aw.q_bias, aw.k_bias, aw.v_bias)))
+        q = unit(q.reshape(T, a.heads, -1)) * aw.q_norm
+        k = (unit(k.reshape(T, a.kv_heads, -1)) * aw.k_norm).repeat_interleave(a.heads // a.kv_heads, dim=1)
+        if a.v_mix and v_first is None:
+            v_first = v
+        elif a.v_mix:
+            v = torch.lerp(v, v_first, aw.vmix)
+        v = v.reshape(T, a.kv_heads, -1).repeat_interleave(a.heads // a.kv_heads, dim=1)
+        seen = back >= 0
+        if a.window:
+            seen = seen & ((back < a.window) | (pos[None, :] < a.keep_first))
+        sc = torch.einsum("qhd,khd->hqk", q, k) * a.scale
+        return softmax_values(a.softcap * torch.tanh(sc / a.softcap) if a.softcap else sc, seen, aw.sinks, v)
+
+    def recurrence(r, lw, z, at):
+        rw, H, G, D, V = lw.rec, r.heads, r.groups, r.dim, r.vdim
+        u = torch.cat([z[:, at[n]:at[n] + rows] for n, rows in r.sections()[:3]], dim=1)
+        u = act.silu(sum(rw.conv[j] * act.pad(u, (0, 0, r.taps - 1 - j, 0))[:T] for j in range(r.taps)))
+        q, k, v = u[:, :G * D].view(T, G, D), u[:, G * D:2 * G * D].view(T, G, D), u[:, 2 * G * D:].view(T, H, V)
+        q, k = ((t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(H // G, dim=1) for t in (q, k))
+        behind = lambda n, wt: z[:, at[n]:at[n] + wt.shape[1]] @ wt.float().t()       # noqa: E731
+        g = (rw.neg_decay[:, None] * act.softplus(behind("a1", rw.w_decay) + rw.dt_bias).view(T, H, D)).exp()
+        beta = torch.sigmoid(z[:, at["b"]:at["b"] + H])
+        S, out = torch.zeros(H, D, V, device=z.device), []
+        for t in range(T):
+            S = g[t][:, :, None] * S
+            S = S + k[t][:, :, None] * (beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t])))[:, None]
+            out.append(torch.einsum("hdv,hd->hv", S, q[t]) * D ** -0.5)
+        return (unit(torch.stack(out)) * rw.norm).reshape(T, -1) * torch.sigmoid(behind("g1", rw.w_gate))
+
+    x = xs[0]
+    for sp, lw in zip(cfg.layers, w.layers):
+        lay = LayerLayout(sp, ff=False)
+        h = norm(x, lw.norm1)
+        h = torch.lerp(h, act.pad(h, (0, 0, 1, 0))[:T], lw.shift)
+        z = torch.zeros(T, lay.width, device=x.device)
+        z[:, lay.in_first:] = h @ lw.w_in.float().t()
+        f = latent if isinstance(sp.mixer, LatentMixerSpec) else recurrence if isinstance(sp.mixer, RecurrentSpec) else attention
+        o = f(sp.mixer, lw, z, lay.parts[0].col)
+        x = x + act.pad(o, (0, lay.out_cols - o.shape[1])) @ lw.w_out.float().t()
+        if sp.mlp is not None:
+            g, u = (norm(x, lw.norm2) @ lw.dense13.float().t()).chunk(2, dim=1)
+            g, u = g.clamp(max=sp.mlp.limit), u.clamp(-sp.mlp.limit, sp.mlp.limit)
+            x = x + (g * torch.sigmoid(GLU_SLOPE * g) * (u + 1.0)) @ lw.dense2.float().t()
+        xs.append(x)
+        x = torch.einsum("j,jtc->tc", lw.depth, torch.stack(xs))
+        if capture_hidden is not None:
+            capture_hidden.append(x.clone())
+    return norm(x, w.final_norm) @ w.lm_head.float().t()
