@@ -37,10 +37,10 @@ ARCH_SOURCES = {
     "Barorax": ("attn_decode", "attn_decode_mma", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_small", "gemm_ws", "postnorm", "prenorm", "rope_kv", "router",
                 "sample", "selective"),
     "Derusun": ("attn_decode", "attn_decode_mma", "attn_latent_decode", "attn_latent_prefill", "attn_prefill_tc", "attn_window", "gemm_simt", "gemm_small",
-                "gemm_ws", "latent", "parallel_layer", "postnorm", "prenorm", "recurrent", "recurrent_tc", "rope_kv", "sample"),
+                "gemm_ws", "latent", "parallel_layer", "postnorm", "prenorm", "recurrent", "recurrent_channel_tc", "recurrent_tc", "rope_kv", "sample"),
 }
 # Sources compiled without fast-math: their exponentials, logarithms and tanh keep the accuracy of 32-bit.
-EXACT_SOURCES = ("attn_window", "parallel_layer", "prenorm", "recurrent", "recurrent_tc", "selective")
+EXACT_SOURCES = ("attn_window", "parallel_layer", "prenorm", "recurrent", "recurrent_channel_tc", "recurrent_tc", "selective")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

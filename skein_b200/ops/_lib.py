@@ -224,6 +224,8 @@ def lib():
     _sig(L, "skein_rec_scan", i32, [rec, chunk, i32, i32, vp])
     _sig(L, "skein_rec_tc", i32, [rec, chunk, i32, i32, vp])
     _sig(L, "skein_rec_tc_scratch_bytes", i64, [rec, i32, i32])
+    _sig(L, "skein_rec_channel", i32, [rec, chunk, i32, i32, vp])
+    _sig(L, "skein_rec_channel_scratch_bytes", i64, [rec, i32, i32])
     _sig(L, "skein_rec_tail", i32, [rec, chunk, i32, i32, vp])
     for name, rt, at in _OPTIONAL:
         if hasattr(L, name):

@@ -1,6 +1,6 @@
 """Recurrences with a 32-bit matrix state per head (gated delta rule with a decay per head or per key channel, state-space duality, fixed decay).
 
-CUDA tensors run csrc/kernels/recurrent.cu and recurrent_tc.cu; CPU tensors run ops/reference_parallel.py. The specification
+CUDA tensors run csrc/kernels/recurrent.cu, recurrent_tc.cu and recurrent_channel_tc.cu; CPU tensors run ops/reference_parallel.py. The specification
 (models/parallel_layers.py: RecurrentSpec) says which recurrence; the weights are its RecurrentWeights.
 """
 from __future__ import annotations
@@ -17,7 +17,7 @@ TC_MIN_ROWS = 17         # portions of at least this many rows take the tensor-c
 
 
 def tc_ok(spec, row) -> bool:
-    return row.is_cuda and row.dtype == torch.bfloat16 and spec.dim in (64, 128) and spec.vdim % 64 == 0 and spec.kind != "channel_delta"
+    return row.is_cuda and row.dtype == torch.bfloat16 and spec.dim in (64, 128) and spec.vdim % 64 == 0
 
 
 @dataclass
@@ -112,7 +112,8 @@ class ChunkRun:
         unit = torch.empty(self.T, 2, spec.groups, dtype=torch.float32, device=dev) if spec.corrects else None
         scratch = None
         if self.tc:
-            scratch = torch.empty(int(_lib.lib().skein_rec_tc_scratch_bytes(C.byref(self.p), self.T, self.S)), dtype=torch.uint8, device=dev)
+            size = _lib.lib().skein_rec_channel_scratch_bytes if spec.kind == "channel_delta" else _lib.lib().skein_rec_tc_scratch_bytes
+            scratch = torch.empty(int(size(C.byref(self.p), self.T, self.S)), dtype=torch.uint8, device=dev)
         c.seq_of_token, c.q_start, c.q_len, c.max_q_len = seq_of_token.data_ptr(), q_start.data_ptr(), q_len.data_ptr(), int(max_q_len)
         c.qkv, c.gates, c.unit, c.chunk_mat = qkv.data_ptr(), gates.data_ptr(), _lib.ptr(unit), _lib.ptr(scratch)
         self._keep = (row, step, w, state, positions, slots, seq_of_token, q_start, q_len, qkv, gates, unit, scratch)
@@ -125,7 +126,8 @@ class ChunkRun:
     def walk(self):
         """The recurrence; the state moves on."""
         if self.tc:
-            _lib.check(_lib.lib().skein_rec_tc(C.byref(self.p), C.byref(self.c), self.T, self.S, _lib.stream_ptr()), "rec_tc")
+            form = _lib.lib().skein_rec_channel if self.p.kind == KINDS["channel_delta"] else _lib.lib().skein_rec_tc
+            _lib.check(form(C.byref(self.p), C.byref(self.c), self.T, self.S, _lib.stream_ptr()), "rec_tc")
             _lib.count_launch(2)
         else:
             _lib.check(_lib.lib().skein_rec_scan(C.byref(self.p), C.byref(self.c), self.S, self.fp32, _lib.stream_ptr()), "rec_scan")
