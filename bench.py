@@ -75,10 +75,10 @@ def parse():
     ap.add_argument("--repeats", type=int, default=5, help="how often each timed K-step loop is repeated (median reported)")
     ap.add_argument("--no-selfcheck", action="store_true")
     ap.add_argument("--no-unfused", action="store_true", help="skip the un-fused comparison arm at N > 1")
-    ap.add_argument("--design", default="", choices=["", "zarorax", "sikalorn", "barorax"],
+    ap.add_argument("--design", default="", choices=["", "zarorax", "sikalorn", "barorax", "derusun"],
                     help="instead of the headline workload: throughput of this design at a few layer sizes beside the closest uniform model, "
                          "and its kernels' rooflines beside the like kernels (one JSON line per size; skein_b200/utils/design_bench.py)")
-    ap.add_argument("--design-sizes", default="all", help="with --design: comma-separated sizes (zarorax: moe-2k, moe-4k, dense-4k; sikalorn: width-2k, width-4k; barorax: scan-2k, scan-4k)")
+    ap.add_argument("--design-sizes", default="all", help="with --design: comma-separated sizes (zarorax: moe-2k, moe-4k, dense-4k; sikalorn: width-2k, width-4k; barorax: scan-2k, scan-4k; derusun: shift-2k, shift-4k)")
     ap.add_argument("--eager", action="store_true",
                     help="launch the step's kernels one by one instead of replaying the captured graph "
                          "(for a per-kernel launch list; the timed loop sits in an NVTX range named 'timed')")

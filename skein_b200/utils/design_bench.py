@@ -1,6 +1,6 @@
 """Throughput and per-kernel rooflines of a design that lists its layers, beside the closest uniform family at equal size.
 
-    python bench.py --design zarorax                    # one JSON object per size; also: sikalorn, barorax
+    python bench.py --design zarorax                    # one JSON object per size; also: sikalorn, barorax, derusun
     python -m skein_b200.utils.design_bench --design sikalorn --only kernels --size width-2k
 
 Weights are random. Each size is a few layers of a real model's width; the closest model has the same width, number of layers,
@@ -25,7 +25,7 @@ from ..models.layered import DenseFFSpec, LatentMixerSpec, LayerSpec, RoutedFFSp
 from ..ops import latent as lat
 from ..ops import reference as ref
 from ..runtime.runner import ModelRunner
-from . import design_bench_parallel as parallel, design_bench_prenorm as prenorm
+from . import design_bench_parallel as parallel, design_bench_prenorm as prenorm, design_bench_shifted as shifted
 from .microbench import _bf, peaks, timeit, timeit_graph
 
 
@@ -291,7 +291,9 @@ def prefill_kernels(new, near, S=4, L=2048):
 
 DESIGNS = {"zarorax": (("moe-2k", "moe-4k", "dense-4k"), size_config, decode_kernels, prefill_kernels),
            "sikalorn": (parallel.SIZES, parallel.size_config, parallel.decode_kernels, parallel.prefill_kernels),
-           "barorax": (prenorm.SIZES, prenorm.size_config, prenorm.decode_kernels, prenorm.prefill_kernels)}
+           "barorax": (prenorm.SIZES, prenorm.size_config, prenorm.decode_kernels, prenorm.prefill_kernels),
+           "derusun": (shifted.SIZES, shifted.size_config, shifted.decode_kernels, shifted.prefill_kernels)}
+DESCRIBE = {"sikalorn": parallel.describe, "barorax": prenorm.describe, "derusun": shifted.describe}
 
 
 def kernel_rows(design, new, near, iters=12, warmup=4):
@@ -318,7 +320,7 @@ def kernel_rows(design, new, near, iters=12, warmup=4):
 def run(design, sizes=None, only=("throughput", "kernels"), emit=print):
     for s in sizes or DESIGNS[design][0]:
         new, near = DESIGNS[design][1](s)
-        about = (parallel if new.is_parallel else prenorm).describe(new) if new.is_parallel or new.is_prenorm else {"width": new.hidden_size, "heads": new.num_heads, "kv_rank": 512}
+        about = DESCRIBE[design](new) if design in DESCRIBE else {"width": new.hidden_size, "heads": new.num_heads, "kv_rank": 512}
         res = {"size": s, "config": {"batch": 64, "prompt": 512, "decode_context": "512 + steps", "prefill_tokens": 8192, "weights": "random", **about},
                "peaks": peaks()}
         if "throughput" in only:
