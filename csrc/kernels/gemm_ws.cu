@@ -567,6 +567,38 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           }
           tc_fence_before();
           mbar_arrive(smem_u32(&bar_tempty[b]));
+        } else if (!DUAL && p.residual == nullptr && p.gate == nullptr && p.relu2_cols == 0) {
+          // plain store, 32 columns (tokens) at a time. bf16: neighbouring lanes (features) exchange, so that a lane stores pairs of features
+          // of every other token
+          const size_t first = (size_t)row0 * p.ldo + p.out_col0 + un.g * p.out_group_cols + f;
+          const bool pairs = !p.out_f32 && p.F % 2 == 0 && p.ldo % 2 == 0 && (p.out_col0 + un.g * p.out_group_cols) % 2 == 0 && ((uintptr_t)p.out & 3) == 0;
+          const int odd = lane & 1;
+          for (int c0 = 0; c0 < n_tile; c0 += 32) {
+            if (c0 >= valid) break;
+            uint32_t v[32];
+            tmem_ld16(t_acc + c0, v);
+            if (c0 + 16 < n_tile) tmem_ld16(t_acc + c0 + 16, v + 16);
+            tmem_ld_wait();
+            if (pairs) {
+              __nv_bfloat16* out = (__nv_bfloat16*)p.out + first - odd + (size_t)(c0 + odd) * p.ldo;
+#pragma unroll
+              for (int j = 0; j < 32; j += 2) {
+                const float got = __uint_as_float(__shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1)), own = __uint_as_float(odd ? v[j + 1] : v[j]);
+                const __nv_bfloat162 y = odd ? __floats2bfloat162_rn(got, own) : __floats2bfloat162_rn(own, got);
+                if (f_ok && c0 + j + odd < valid) *reinterpret_cast<__nv_bfloat162*>(out + (size_t)j * p.ldo) = y;
+              }
+            } else if (f_ok) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) {
+                if (c0 + j >= valid) break;
+                const size_t idx = first + (size_t)(c0 + j) * p.ldo;
+                if (p.out_f32) ((float*)p.out)[idx] = __uint_as_float(v[j]);
+                else ((__nv_bfloat16*)p.out)[idx] = __float2bfloat16(__uint_as_float(v[j]));
+              }
+            }
+          }
+          tc_fence_before();
+          mbar_arrive(smem_u32(&bar_tempty[b]));
         } else {
           for (int c0 = 0; c0 < n_tile; c0 += 16) {
             if (c0 >= valid) break;

@@ -192,7 +192,7 @@ __device__ __forceinline__ void depth_walk(const DepthNormParams& p, int r0, int
 }
 
 // A thread keeps 4 elements per pass in registers; groups of a multiple of DN_SEG elements, so that a warp's pass lies in one.
-template <typename T, int PASSES>
+template <typename T, int PASSES, bool SHIFT>
 __global__ void __launch_bounds__(512) depth_norm_kernel(const DepthNormParams p, int rows) {
   __shared__ float seg[2][DN_MAX_SEGS];
   pdl_trigger();
@@ -263,8 +263,9 @@ __global__ void __launch_bounds__(512) depth_norm_kernel(const DepthNormParams p
   auto keep = [&](int slot, int from) {
     each([&](int i, int ps) { store_v<float, 4>(p.state + (size_t)slot * p.C + i, from == 2 ? b[2][ps] : b[0][ps]); });
   };
-  const int r0 = blockIdx.x * rows;
-  depth_walk(p, r0, min(r0 + rows, p.T), row, put, take, keep);
+  const int r0 = blockIdx.x * rows, r1 = min(r0 + rows, p.T);
+  if (SHIFT) depth_walk(p, r0, r1, row, put, take, keep);
+  else for (int t = r0; t < r1; ++t) { row(t, true, 0); put(t, false); }
 }
 
 // Any row length and group size: the three buffers in shared memory, then a factor per group.
@@ -406,13 +407,14 @@ static int depth_norm_go(const DepthNormParams& p, cudaStream_t s) {
   if (rows > 16) rows = 16;
   const dim3 grid((p.T + rows - 1) / rows);
   if (p.C / p.groups % DN_SEG == 0 && p.C <= DN_MAX_SEGS * DN_SEG) {
+    // few rows: one access per thread, so that a row's latency is that of one; many rows: smaller CTAs
     int th = 128;
-    while (th < 512 && th * 4 < p.C) th *= 2;
+    while (th < (p.T <= 512 || p.C > 4096 ? 512 : 256) && th * 4 < p.C) th *= 2;
     const int passes = (p.C + th * 4 - 1) / (th * 4);
-    auto go = [&](auto fn) -> int { return (int)launch_pdl(fn, grid, dim3(th), 0, s, p, rows); };
-    if (passes <= 1) return go(depth_norm_kernel<T, 1>);
-    if (passes <= 2) return go(depth_norm_kernel<T, 2>);
-    return go(depth_norm_kernel<T, 4>);
+    auto go = [&](auto with, auto without) -> int { return (int)launch_pdl(p.shift ? with : without, grid, dim3(th), 0, s, p, rows); };
+    if (passes <= 1) return go(depth_norm_kernel<T, 1, true>, depth_norm_kernel<T, 1, false>);
+    if (passes <= 2) return go(depth_norm_kernel<T, 2, true>, depth_norm_kernel<T, 2, false>);
+    return go(depth_norm_kernel<T, 4, true>, depth_norm_kernel<T, 4, false>);
   }
   const size_t sm = (size_t)(3 * p.C + p.groups) * 4;
   if (sm > 200 * 1024) return -1;
