@@ -69,7 +69,7 @@ class OpProfiler:
             self._patch(parallel, n, "parallel." + n)
         for n in ("rec_step", "rec_chunk"):
             self._patch(recurrent, n, "recurrent." + n)
-        for n in ("add_norm", "norm_route", "route"):
+        for n in ("add_norm", "depth_norm", "norm_route", "route"):
             self._patch(prenorm, n, "prenorm." + n)
         for n in ("short_conv", "scan"):
             self._patch(selective, n, "selective." + n)
